@@ -68,6 +68,7 @@ struct AttnParams {
   float logit_cap;         // soft cap: score = cap * tanh(score / cap) before the softmax (0 = off)
   float scale;             // softmax scale (used with the soft cap)
   float cap_pre, cap_post; // soft cap: score in the log2 domain = cap_post * tanh(raw * cap_pre)
+  const float* sink;       // [Hq] or null: a learned logit per head that joins the softmax denominator only
   int kv_fmt;              // single-role kernel only: 1 / 2 = the caches hold unscaled e4m3 / e5m2 bytes
   uint32_t idesc_s, idesc_o;
 };
@@ -82,6 +83,18 @@ __device__ __forceinline__ float tanh_approx(float x) {
   float y;
   asm("tanh.approx.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
+}
+// 1 / softmax denominator of a row with sum `l` over its keys, taken relative to 2^m.  A sink adds exp(sink) once: it
+// has no key and no value and is not scaled.
+__device__ __forceinline__ float inv_denominator(float l, float m, const float* sink, int head) {
+  if (!(l > 0.f)) return 0.f;
+  if (sink == nullptr) return 1.f / l;
+  const float d = sink[head] * kLog2e - m;
+  if (d > 0.f) {
+    const float e = exp2f(-d);
+    return e / fmaf(l, e, 1.f);
+  }
+  return 1.f / (l + exp2f(d));
 }
 __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N>
@@ -432,8 +445,8 @@ __global__ void __launch_bounds__(kAttnThreads, FwdCfg<NH>::kCtasPerSm) attn_fwd
   tc_fence_after_sync();
   if (!ok_all && p.status != nullptr) atomicExch(p.status, kStatusPipelineTimeout);
 
-  // ---- epilogue -----------------------------------------------------------------------------
-  const float inv_l = l_sum > 0.f ? 1.f / l_sum : 0.f;
+  // ---- epilogue (partial results of a split leave the sink to the merge) ---------------------
+  const float inv_l = inv_denominator(l_sum, m_used, p.is_decode && p.num_splits > 1 ? nullptr : p.sink, row_head);
   if (p.is_decode && p.num_splits > 1) {
     float* po = p.part_o + ((static_cast<int64_t>(b) * p.hq + row_head) * p.num_splits + split) * kD;
 #pragma unroll 1
@@ -913,8 +926,9 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
         const int c = c0 + i;
         if (c < g && good) {
           const float l = red2[c];
-          const float v = l > 0.f ? __uint_as_float(o[i]) / l : 0.f;
           const int head = hk * g + c;
+          const float v = p.sink != nullptr && p.num_splits == 1 ? __uint_as_float(o[i]) * inv_denominator(l, m_used[c], p.sink, head)
+                          : l > 0.f ? __uint_as_float(o[i]) / l : 0.f;
           if (p.num_splits > 1) {
             p.part_o[((static_cast<int64_t>(b) * p.hq + head) * p.num_splits + split) * kD + tid] = v;
           } else {
@@ -1309,7 +1323,7 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
 
     // ---- epilogue: normalise, park the group's 128 rows x 256 B in its P buffer (free now), then store them
     // row by row: 16 lanes cover one output row, and the g rows of a token are adjacent in memory ----
-    const float inv_l = l_sum > 0.f ? 1.f / l_sum : 0.f;
+    const float inv_l = inv_denominator(l_sum, m_used, p.sink, hk * g + row % g);
 #pragma unroll 1
     for (int c = 0; c < kD; c += 32) {
       uint32_t o[32];
@@ -1370,9 +1384,10 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
   }
 }
 
-// combine decode partials: out[b, h, :] = sum_s w_s * O_s with w_s = 2^(lse_s - max) / sum
+// combine decode partials: out[b, h, :] = sum_s w_s * O_s with w_s = 2^(lse_s - max) / sum; a head's sink is one more
+// term of the sum, without a value
 __global__ void attn_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_lse,
-                                  void* __restrict__ out, int hq, int splits, int out_f16) {
+                                  void* __restrict__ out, int hq, int splits, int out_f16, const float* __restrict__ sink) {
   pdl_launch_dependents();
   pdl_wait();
   const int b = blockIdx.y, h = blockIdx.x, d = threadIdx.x;
@@ -1381,6 +1396,11 @@ __global__ void attn_merge_kernel(const float* __restrict__ part_o, const float*
   float m = -INFINITY;
   for (int s = 0; s < splits; ++s) m = fmaxf(m, part_lse[base + s]);
   float den = 0.f, acc = 0.f;
+  if (sink != nullptr) {
+    const float sl = sink[h] * kLog2e;
+    m = fmaxf(m, sl);
+    den = exp2f(sl - m);
+  }
   for (int s = 0; s < splits; ++s) {
     const float l = part_lse[base + s];
     const float w = (l == -INFINITY) ? 0.f : exp2f(l - m);
@@ -1516,6 +1536,7 @@ int launch_attention(const AttnArgs& a, cudaStream_t s) {
   p.cap_pre = p.logit_cap > 0.f ? a.scale / p.logit_cap : 0.f;
   p.cap_post = p.logit_cap * kLog2e;
   p.kv_fmt = a.kv_fmt;
+  p.sink = a.sink;
   const uint32_t fmt = a.dt == kF16 ? 0u : 1u;
   p.idesc_s = umma_idesc(kRows, kKV, 1, fmt, fmt, 0, 0);
   p.idesc_o = umma_idesc(kRows, hd, 1, fmt, fmt, 0, 1);
@@ -1529,7 +1550,7 @@ int launch_attention(const AttnArgs& a, cudaStream_t s) {
     const int rc = nq == 16 ? launch_decode_cfg<16>(p, a, grid, s) : launch_decode_cfg<32>(p, a, grid, s);
     if (rc != 0) return rc;
     if (p.num_splits > 1) {
-      launch_pdl(attn_merge_kernel, dim3(a.hq, a.batch), dim3(kD), 0, s, a.part_o, a.part_lse, a.out, a.hq, p.num_splits, p.out_f16);
+      launch_pdl(attn_merge_kernel, dim3(a.hq, a.batch), dim3(kD), 0, s, a.part_o, a.part_lse, a.out, a.hq, p.num_splits, p.out_f16, a.sink);
       note_launch();
     }
     return cudaGetLastError() == cudaSuccess ? 0 : -4;
@@ -1548,7 +1569,7 @@ int launch_attention(const AttnArgs& a, cudaStream_t s) {
   const int rc = hd == 64 ? launch_fwd_cfg<1>(p, grid, s) : hd == 128 ? launch_fwd_cfg<2>(p, grid, s) : launch_fwd_cfg<4>(p, grid, s);
   if (rc != 0) return rc;
   if (a.is_decode && p.num_splits > 1) {
-    launch_pdl(attn_merge_kernel, dim3(a.hq, a.batch), dim3(hd), 0, s, a.part_o, a.part_lse, a.out, a.hq, p.num_splits, p.out_f16);
+    launch_pdl(attn_merge_kernel, dim3(a.hq, a.batch), dim3(hd), 0, s, a.part_o, a.part_lse, a.out, a.hq, p.num_splits, p.out_f16, a.sink);
     note_launch();
   }
   return cudaGetLastError() == cudaSuccess ? 0 : -4;

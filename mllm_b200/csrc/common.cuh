@@ -18,6 +18,8 @@
 #include <cuda_runtime.h>
 #include <stdint.h>
 
+#include <type_traits>
+
 namespace mb200 {
 
 // ---------------------------------------------------------------------------
@@ -399,6 +401,16 @@ template <>
 __device__ __forceinline__ __half from_f32<__half>(float v) {
   return __float2half_rn(v);
 }
+template <>
+__device__ __forceinline__ float from_f32<float>(float v) {
+  return v;
+}
+
+// tanh form of the GELU
+__device__ __forceinline__ float gelu_tanh_f(float v) {
+  const float k = 0.7978845608028654f;
+  return 0.5f * v * (1.f + tanhf(k * (v + 0.044715f * v * v * v)));
+}
 
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
@@ -420,6 +432,14 @@ __device__ __forceinline__ float warp_max(float v) {
     using T = __half;                         \
     __VA_ARGS__;                              \
   }
+
+// the same with fp32 as a third element type
+#define MB200_DISPATCH_FLOAT(dt, ...)         \
+  if ((dt) == ::mb200::kF32) {                \
+    using T = float;                          \
+    __VA_ARGS__;                              \
+  } else                                      \
+    MB200_DISPATCH_HALF(dt, __VA_ARGS__)
 
 // Host side: raises `kernel`'s dynamic shared-memory limit to `bytes`, once per (kernel, device).
 // cudaFuncSetAttribute acts on the current device only, so the record of what was set is kept per

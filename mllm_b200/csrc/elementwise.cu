@@ -242,11 +242,6 @@ __global__ void layernorm_kernel(const T* __restrict__ x, const T* __restrict__ 
 // gated activations
 // ---------------------------------------------------------------------------
 __device__ __forceinline__ float silu_f(float v) { return v / (1.f + __expf(-v)); }
-__device__ __forceinline__ float gelu_tanh_f(float v) {
-  const float k = 0.7978845608028654f;
-  return 0.5f * v * (1.f + tanhf(k * (v + 0.044715f * v * v * v)));
-}
-
 template <typename T, int kAct>
 __global__ void act_and_mul_kernel(const T* __restrict__ x, T* __restrict__ out, int rows, int inter) {
   pdl_launch_dependents();
@@ -265,6 +260,84 @@ __global__ void act_and_mul_kernel(const T* __restrict__ x, T* __restrict__ out,
     for (int j = 0; j < 8; ++j) o[j] = (kAct == 0 ? silu_f(g[j]) : gelu_tanh_f(g[j])) * u[j];
     reinterpret_cast<uint4*>(out + r * inter)[v] = pack8<T>(o);
   }
+}
+
+// the same one element at a time: fp32 tensors and widths that are no multiple of 8
+template <typename T>
+__global__ void act_and_mul_any_kernel(const T* __restrict__ x, T* __restrict__ out, int64_t total, int inter, int act) {
+  pdl_launch_dependents();
+  pdl_wait();
+  for (int64_t i = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x; i < total;
+       i += static_cast<int64_t>(gridDim.x) * blockDim.x) {
+    const int64_t r = i / inter;
+    const int64_t at = r * 2 * inter + (i - r * inter);
+    const float g = to_f32(x[at]), u = to_f32(x[at + inter]);
+    out[i] = from_f32<T>((act == 0 ? g / (1.f + expf(-g)) : gelu_tanh_f(g)) * u);
+  }
+}
+
+// Dynamic Tanh norm on an fp32 residual stream: x += mult * y (y may be absent), h = tanh(alpha * x) * w + b.  Purely
+// element-wise (no row statistic), so a thread takes V neighbouring channels of any row.
+template <typename T, int V>
+__global__ void residual_dyt_kernel(float* __restrict__ x, const T* __restrict__ y, float mult, const float* __restrict__ alpha,
+                                    const float* __restrict__ w, const float* __restrict__ b, T* __restrict__ h, int64_t groups,
+                                    int groups_per_row) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const float al = *alpha;
+  for (int64_t i = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x; i < groups;
+       i += static_cast<int64_t>(gridDim.x) * blockDim.x) {
+    const int c = static_cast<int>(i % groups_per_row) * V;
+    float xv[V], yv[V];
+    T hv[V];
+    if constexpr (V == 4) {
+      *reinterpret_cast<float4*>(xv) = reinterpret_cast<const float4*>(x)[i];
+    } else {
+      xv[0] = x[i];
+    }
+    if (y != nullptr) {
+      T yr[V];
+      if constexpr (V == 4 && sizeof(T) == 2) {
+        *reinterpret_cast<uint2*>(yr) = reinterpret_cast<const uint2*>(y)[i];
+      } else if constexpr (V == 4) {
+        *reinterpret_cast<float4*>(yr) = reinterpret_cast<const float4*>(y)[i];
+      } else {
+        yr[0] = y[i];
+      }
+#pragma unroll
+      for (int j = 0; j < V; ++j) {
+        yv[j] = to_f32(yr[j]);
+        xv[j] = fmaf(mult, yv[j], xv[j]);
+      }
+      if constexpr (V == 4) {
+        reinterpret_cast<float4*>(x)[i] = *reinterpret_cast<const float4*>(xv);
+      } else {
+        x[i] = xv[0];
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < V; ++j) hv[j] = from_f32<T>(fmaf(tanhf(al * xv[j]), w[c + j], b[c + j]));
+    if constexpr (V == 4 && sizeof(T) == 2) {
+      reinterpret_cast<uint2*>(h)[i] = *reinterpret_cast<const uint2*>(hv);
+    } else if constexpr (V == 4) {
+      reinterpret_cast<float4*>(h)[i] = *reinterpret_cast<const float4*>(hv);
+    } else {
+      h[i] = hv[0];
+    }
+  }
+}
+
+// embedding rows widened to fp32 (the start of an fp32 residual stream); one CTA per token
+template <typename T>
+__global__ void embedding_f32_kernel(const int64_t* __restrict__ ids, const T* __restrict__ table, float* __restrict__ out,
+                                     int width, int vocab, int* status) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int64_t id = ids[blockIdx.x];
+  const bool ok = id >= 0 && id < vocab;
+  if (!ok && threadIdx.x == 0 && status != nullptr) atomicExch(status, kStatusBadIndex);
+  for (int c = threadIdx.x; c < width; c += blockDim.x)
+    out[static_cast<int64_t>(blockIdx.x) * width + c] = ok ? to_f32(table[id * width + c]) : 0.f;
 }
 
 template <typename T>
@@ -663,8 +736,16 @@ void launch_layernorm(const void* x, const void* w, const void* b, void* out, in
 
 void launch_act_and_mul(const void* x, void* out, int rows, int inter, int act, DType dt, cudaStream_t s) {
   if (rows == 0) return;
-  const int64_t total = static_cast<int64_t>(rows) * (inter >> 3);
   const int threads = 256;
+  if (dt == kF32 || inter % 8 != 0) {
+    const int64_t n = static_cast<int64_t>(rows) * inter;
+    const int grid = static_cast<int>(std::min<int64_t>((n + threads - 1) / threads, 148 * 16));
+    MB200_DISPATCH_FLOAT(dt, (launch_pdl(act_and_mul_any_kernel<T>, dim3(grid), dim3(threads), 0, s, static_cast<const T*>(x),
+                                         static_cast<T*>(out), n, inter, act)));
+    note_launch();
+    return;
+  }
+  const int64_t total = static_cast<int64_t>(rows) * (inter >> 3);
   const int blocks = static_cast<int>(std::min<int64_t>((total + threads - 1) / threads, 148 * 16));
   if (act == 0) {
     MB200_DISPATCH_HALF(dt, (launch_pdl(act_and_mul_kernel<T, 0>, dim3(blocks), dim3(threads), 0, s, static_cast<const T*>(x),
@@ -673,6 +754,32 @@ void launch_act_and_mul(const void* x, void* out, int rows, int inter, int act, 
     MB200_DISPATCH_HALF(dt, (launch_pdl(act_and_mul_kernel<T, 1>, dim3(blocks), dim3(threads), 0, s, static_cast<const T*>(x),
                                                                                   static_cast<T*>(out), rows, inter)));
   }
+  note_launch();
+}
+
+void launch_residual_dyt(float* x, const void* y, float mult, const float* alpha, const float* w, const float* b, void* h,
+                         int rows, int width, DType dt, cudaStream_t s) {
+  if (rows == 0) return;
+  const int threads = 256;
+  const int v = width % 4 == 0 ? 4 : 1;
+  const int64_t groups = static_cast<int64_t>(rows) * (width / v);
+  const int blocks = static_cast<int>(std::min<int64_t>((groups + threads - 1) / threads, 148 * 16));
+  if (v == 4) {
+    MB200_DISPATCH_FLOAT(dt, (launch_pdl(residual_dyt_kernel<T, 4>, dim3(blocks), dim3(threads), 0, s, x, static_cast<const T*>(y),
+                                         mult, alpha, w, b, static_cast<T*>(h), groups, width / 4)));
+  } else {
+    MB200_DISPATCH_FLOAT(dt, (launch_pdl(residual_dyt_kernel<T, 1>, dim3(blocks), dim3(threads), 0, s, x, static_cast<const T*>(y),
+                                         mult, alpha, w, b, static_cast<T*>(h), groups, width)));
+  }
+  note_launch();
+}
+
+void launch_embedding_f32(const int64_t* ids, const void* table, float* out, int tokens, int width, int vocab, DType dt,
+                          int* status, cudaStream_t s) {
+  if (tokens == 0) return;
+  const int threads = width >= 256 ? 256 : (width + 31) / 32 * 32;
+  MB200_DISPATCH_FLOAT(dt, (launch_pdl(embedding_f32_kernel<T>, dim3(tokens), dim3(threads), 0, s, ids, static_cast<const T*>(table),
+                                       out, width, vocab, status)));
   note_launch();
 }
 

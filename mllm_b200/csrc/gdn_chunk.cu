@@ -12,7 +12,9 @@
 // (request, head) and a block of BV value features: grid (128 / BV, heads, batch), 256 threads.  The products
 // K K^T, Q K^T, K S0, Q S0, P U and K^T U' run on the tensor cores through warp-level MMA on tf32 operands with
 // fp32 accumulation (tiles of 16 x 16 x 8 read from shared memory); the state stays in fp32 in shared memory for
-// the whole sequence and is rounded to tf32 only as an MMA operand.  The substitution is the one sequential step;
+// the whole sequence and is rounded to tf32 only as an MMA operand.  SPLIT: every operand enters as two tf32 terms
+// (its rounding and the remainder), three products per tile, which carries 21 bits of each operand through the
+// recurrence.  Heads of fewer than 128 features are zero-padded on their way into shared memory.  The substitution is the one sequential step;
 // it runs 16 rows at a time (one thread per value feature inside a block, a tensor-core product to carry a solved
 // block into the rows below): one thread walking all 64 rows kept the other warps at a barrier for a quarter of
 // the kernel's issue slots.
@@ -64,13 +66,43 @@ __device__ __forceinline__ void to_tf32(F& f) {
   for (int i = 0; i < f.num_elements; ++i) f.x[i] = wmma::__float_to_tf32(f.x[i]);
 }
 
-template <typename T, int BV>
-__global__ void __launch_bounds__(kGThreads, 1)
-gdn_chunk_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, const float* __restrict__ g,
-                 const float* __restrict__ beta, float* __restrict__ state, const int* __restrict__ slots,
-                 const int* __restrict__ lens, const int* __restrict__ has_state, const int* __restrict__ q_start,
-                 T* __restrict__ out, int heads) {
+// acc += A B with fp32 operands: one tf32 product, or (SPLIT) the three leading products of two-term operands
+template <bool SPLIT, typename FA, typename FB>
+__device__ __forceinline__ void mma_f32(FragC& acc, FA& fa, FB& fb) {
+  if constexpr (SPLIT) {
+    FA la;
+    FB lb;
+#pragma unroll
+    for (int i = 0; i < fa.num_elements; ++i) {
+      const float hi = wmma::__float_to_tf32(fa.x[i]);
+      la.x[i] = wmma::__float_to_tf32(fa.x[i] - hi);
+      fa.x[i] = hi;
+    }
+#pragma unroll
+    for (int i = 0; i < fb.num_elements; ++i) {
+      const float hi = wmma::__float_to_tf32(fb.x[i]);
+      lb.x[i] = wmma::__float_to_tf32(fb.x[i] - hi);
+      fb.x[i] = hi;
+    }
+    wmma::mma_sync(acc, la, fb, acc);
+    wmma::mma_sync(acc, fa, lb, acc);
+  } else {
+    to_tf32(fa);
+    to_tf32(fb);
+  }
+  wmma::mma_sync(acc, fa, fb, acc);
+}
+
+template <typename T, int BV, bool SPLIT>
+__global__ void __launch_bounds__(kGThreads, 1) gdn_chunk_kernel(const GdnRuleParams p) {
   pdl_wait();
+  const T* __restrict__ q = static_cast<const T*>(p.q);
+  const T* __restrict__ k = static_cast<const T*>(p.k);
+  const T* __restrict__ v = static_cast<const T*>(p.v);
+  const float* __restrict__ g = p.g;
+  const float* __restrict__ beta = p.beta;
+  T* __restrict__ out = static_cast<T*>(p.out);
+  const int heads = p.heads, dk = p.dk, dv = p.dv;
   using C = GdnChunkCfg<BV>;
   constexpr int kLdV = C::kLdV;
   constexpr int kVT = BV / 16;   // 16-wide tiles across the value block
@@ -98,31 +130,34 @@ gdn_chunk_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __re
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int vb = blockIdx.x, h = blockIdx.y, b = blockIdx.z;
-  const int n = lens[b];
+  const int n = p.lens[b];
   if (n <= 0) return;
-  const int64_t row0 = q_start[b];
-  float* S = state + ((static_cast<int64_t>(slots[b]) * heads + h) * kGD) * kGD + vb * BV;   // element (i, c) at S[i * 128 + c]
-  const bool resume = has_state[b] != 0;
+  const int hk = h / (heads / p.k_heads);
+  const int cols = min(BV, dv - vb * BV);     // value features of this block
+  const int64_t row0 = p.q_start[b];
+  float* S = p.state + (static_cast<int64_t>(p.slots[b]) * heads + h) * dk * dv + vb * BV;   // element (i, c) at S[i * dv + c]
+  const bool resume = p.has_state[b] != 0;
   for (int idx = tid; idx < kGD * BV; idx += kGThreads) {
     const int i = idx / BV, c = idx % BV;
-    sS[i * kLdV + c] = resume ? S[i * kGD + c] : 0.f;
+    sS[i * kLdV + c] = resume && i < dk && c < cols ? S[i * dv + c] : 0.f;
   }
-  const float qscale = rsqrtf(static_cast<float>(kGD));
+  const float qscale = 1.f / sqrtf(static_cast<float>(dk));
 
   // every copy of one chunk: 64 rows x 16 pieces of K and of Q, 64 x BV / 8 pieces of V, 64 scalars of g and beta
   auto stage_chunk = [&](int c0) {
     const int nv = min(kGC, n - c0);
     for (int idx = tid; idx < kGC * 16; idx += kGThreads) {
       const int r = idx >> 4, piece = idx & 15;
-      const bool valid = r < nv;
-      const int64_t at = ((row0 + c0 + (valid ? r : 0)) * heads + h) * kGD + piece * 8;
-      stage16(sKn + r * kGD + piece * 8, k + at, valid);
-      stage16(sQn + r * kGD + piece * 8, q + at, valid);
+      const bool valid = r < nv && piece * 8 < dk;
+      const int64_t row = row0 + c0 + (valid ? r : 0), at = static_cast<int64_t>(hk) * dk + (valid ? piece * 8 : 0);
+      stage16(sKn + r * kGD + piece * 8, k + row * p.k_ld + at, valid);
+      stage16(sQn + r * kGD + piece * 8, q + row * p.q_ld + at, valid);
     }
     for (int idx = tid; idx < kGC * (BV / 8); idx += kGThreads) {
       const int r = idx / (BV / 8), piece = idx % (BV / 8);
-      const bool valid = r < nv;
-      stage16(sVn + r * BV + piece * 8, v + ((row0 + c0 + (valid ? r : 0)) * heads + h) * kGD + vb * BV + piece * 8, valid);
+      const bool valid = r < nv && piece * 8 < cols;
+      stage16(sVn + r * BV + piece * 8,
+              v + (row0 + c0 + (valid ? r : 0)) * p.v_ld + static_cast<int64_t>(h) * dv + vb * BV + (valid ? piece * 8 : 0), valid);
     }
     if (tid < kGC) {
       const bool valid = tid < nv;
@@ -214,9 +249,7 @@ gdn_chunk_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __re
           FragBT fb;
           wmma::load_matrix_sync(fa, left + k0, kGLd);
           wmma::load_matrix_sync(fb, right + k0, kGLd);     // B[k][j] = K[j][k]
-          to_tf32(fa);
-          to_tf32(fb);
-          wmma::mma_sync(acc, fa, fb, acc);
+          mma_f32<SPLIT>(acc, fa, fb);
         }
         wmma::store_matrix_sync((which ? sP : sA) + ti * 16 * kGLdC + tj * 16, acc, kGLdC, wmma::mem_row_major);
       } else {
@@ -228,9 +261,7 @@ gdn_chunk_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __re
           FragB fb;
           wmma::load_matrix_sync(fa, left + k0, kGLd);
           wmma::load_matrix_sync(fb, sS + k0 * kLdV + tc * 16, kLdV);
-          to_tf32(fa);
-          to_tf32(fb);
-          wmma::mma_sync(acc, fa, fb, acc);
+          mma_f32<SPLIT>(acc, fa, fb);
         }
         wmma::store_matrix_sync((which ? sY : sX) + ti * 16 * kLdV + tc * 16, acc, kLdV, wmma::mem_row_major);
       }
@@ -296,9 +327,8 @@ gdn_chunk_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __re
             wmma::load_matrix_sync(fa, sA + ti * 16 * kGLdC + blk * 16 + k0, kGLdC);
             wmma::load_matrix_sync(fb, sU + (blk * 16 + k0) * kLdV + tc * 16, kLdV);
 #pragma unroll
-            for (int i = 0; i < fa.num_elements; ++i) fa.x[i] = wmma::__float_to_tf32(-fa.x[i]);
-            to_tf32(fb);
-            wmma::mma_sync(acc, fa, fb, acc);
+            for (int i = 0; i < fa.num_elements; ++i) fa.x[i] = -fa.x[i];
+            mma_f32<SPLIT>(acc, fa, fb);
           }
           wmma::store_matrix_sync(tile, acc, kLdV, wmma::mem_row_major);
         }
@@ -319,9 +349,7 @@ gdn_chunk_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __re
           FragB fb;
           wmma::load_matrix_sync(fa, sP + ti * 16 * kGLdC + k0, kGLdC);
           wmma::load_matrix_sync(fb, sU + k0 * kLdV + tc * 16, kLdV);
-          to_tf32(fa);
-          to_tf32(fb);
-          wmma::mma_sync(acc, fa, fb, acc);
+          mma_f32<SPLIT>(acc, fa, fb);
         }
         wmma::store_matrix_sync(tile, acc, kLdV, wmma::mem_row_major);
       } else {
@@ -336,9 +364,7 @@ gdn_chunk_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __re
           FragB fb;
           wmma::load_matrix_sync(fa, sK + k0 * kGLd + tm * 16, kGLd);    // A[m][k] = K[k][m]
           wmma::load_matrix_sync(fb, sX + k0 * kLdV + tc * 16, kLdV);
-          to_tf32(fa);
-          to_tf32(fb);
-          wmma::mma_sync(acc, fa, fb, acc);
+          mma_f32<SPLIT>(acc, fa, fb);
         }
         wmma::store_matrix_sync(tile, acc, kLdV, wmma::mem_row_major);
       }
@@ -348,42 +374,46 @@ gdn_chunk_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __re
     // ---- outputs of the chunk ----
     for (int idx = tid; idx < nv * BV; idx += kGThreads) {
       const int i = idx / BV, c = idx % BV;
-      out[((row0 + c0 + i) * heads + h) * kGD + vb * BV + c] = from_f32<T>(sY[i * kLdV + c]);
+      if (c < cols) out[((row0 + c0 + i) * heads + h) * dv + vb * BV + c] = from_f32<T>(sY[i * kLdV + c]);
     }
     // the next iteration starts with a barrier, so sY is rewritten only after these reads
   }
   for (int idx = tid; idx < kGD * BV; idx += kGThreads) {
     const int i = idx / BV, c = idx % BV;
-    S[i * kGD + c] = sS[i * kLdV + c];
+    if (i < dk && c < cols) S[i * dv + c] = sS[i * kLdV + c];
   }
 }
 
-template <typename T, int BV>
-int launch_chunk_cfg(const T* q, const T* k, const T* v, const float* g, const float* beta, float* state, const int* slots,
-                     const int* lens, const int* has_state, const int* q_start, T* out, int batch, int heads, cudaStream_t s) {
-  if (ensure_dynamic_smem(reinterpret_cast<const void*>(gdn_chunk_kernel<T, BV>), GdnChunkCfg<BV>::kSmem) != cudaSuccess) return -3;
-  const cudaError_t err = launch_pdl(gdn_chunk_kernel<T, BV>, dim3(kGD / BV, heads, batch), dim3(kGThreads), GdnChunkCfg<BV>::kSmem,
-                                     s, q, k, v, g, beta, state, slots, lens, has_state, q_start, out, heads);
+template <typename T, int BV, bool SPLIT>
+int launch_chunk_cfg(const GdnRuleParams& p, cudaStream_t s) {
+  if (ensure_dynamic_smem(reinterpret_cast<const void*>(gdn_chunk_kernel<T, BV, SPLIT>), GdnChunkCfg<BV>::kSmem) != cudaSuccess)
+    return -3;
+  const cudaError_t err = launch_pdl(gdn_chunk_kernel<T, BV, SPLIT>, dim3((p.dv + BV - 1) / BV, p.heads, p.batch), dim3(kGThreads),
+                                     GdnChunkCfg<BV>::kSmem, s, p);
   note_launch();
   return err == cudaSuccess ? 0 : -4;
+}
+template <typename T>
+int launch_chunk_t(const GdnRuleParams& p, bool narrow, cudaStream_t s) {
+  if (p.split_tf32) return narrow ? launch_chunk_cfg<T, 32, true>(p, s) : launch_chunk_cfg<T, 64, true>(p, s);
+  return narrow ? launch_chunk_cfg<T, 32, false>(p, s) : launch_chunk_cfg<T, 64, false>(p, s);
 }
 
 }  // namespace
 
-int launch_gdn_chunk(const void* q, const void* k, const void* v, const float* g, const float* beta, float* state,
-                     const int* slots, const int* lens, const int* has_state, const int* q_start, void* out, int batch,
-                     int heads, int dk, int dv, int num_sms, DType dt, cudaStream_t s) {
-  if (batch <= 0) return 0;
-  if (dk != kGD || dv != kGD) return -1;
+bool gdn_chunk_covers(const GdnRuleParams& p) {
+  // rows move in 16-byte pieces
+  return p.dt != kF32 && p.dk <= kGD && p.dk % 8 == 0 && p.dv % 8 == 0 && p.q_ld % 8 == 0 && p.k_ld % 8 == 0 && p.v_ld % 8 == 0 &&
+         ((reinterpret_cast<uintptr_t>(p.q) | reinterpret_cast<uintptr_t>(p.k) | reinterpret_cast<uintptr_t>(p.v)) & 15) == 0;
+}
+
+int launch_gdn_chunk(const GdnRuleParams& p, int num_sms, cudaStream_t s) {
+  if (p.batch <= 0) return 0;
+  if (!gdn_chunk_covers(p) || p.heads % p.k_heads != 0 || p.g == nullptr) return -1;
   // narrower value blocks when the batch alone does not fill the GPU
-  const bool narrow = batch * heads * 2 < num_sms;
+  const bool narrow = p.batch * p.heads * 2 < num_sms || p.dv <= 32;
   int rc = 0;
-  MB200_DISPATCH_HALF(dt, (rc = narrow ? launch_chunk_cfg<T, 32>(static_cast<const T*>(q), static_cast<const T*>(k),
-                                                                 static_cast<const T*>(v), g, beta, state, slots, lens, has_state,
-                                                                 q_start, static_cast<T*>(out), batch, heads, s)
-                                       : launch_chunk_cfg<T, 64>(static_cast<const T*>(q), static_cast<const T*>(k),
-                                                                 static_cast<const T*>(v), g, beta, state, slots, lens, has_state,
-                                                                 q_start, static_cast<T*>(out), batch, heads, s)));
+  MB200_DISPATCH_HALF(p.dt, rc = launch_chunk_t<T>(p, narrow, s));
   return rc;
 }
 

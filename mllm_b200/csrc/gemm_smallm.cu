@@ -284,7 +284,7 @@ __global__ void __launch_bounds__(kSmThreads, 1) gemm_smallm_kernel(const SmallM
                   for (int w8 = 0; w8 < kSmWarps; ++w8) up += partial[buf][w8][t + 4];
                   const int blk = cu >> 5, q = cu & 31;
                   const int64_t col = static_cast<int64_t>(blk) * 128 + q * 4 + slot;
-                  const float y = v / (1.f + __expf(-v)) * up;
+                  const float y = (p.swiglu == 2 ? gelu_tanh_f(v) : v / (1.f + __expf(-v))) * up;
                   static_cast<uint16_t*>(p.out)[mrow * p.ldc + col] = f_to_half<F16>(y);
                 }
               } else {

@@ -57,6 +57,7 @@ struct KParams {
   int is_int8;
   int row_static;        // swap tiling: the row operand (weights) is not written by earlier kernels of the stream
   int cluster_k;         // swap tiling: > 1 = the k range of a tile is split over the CTAs of a cluster of this size
+  int gate_gelu;         // gated epilogue: GELU (tanh form) of the gate rows instead of SiLU
   int early_trigger;     // swap tiling: let the kernels behind this one start their set-up as soon as this one runs
   uint32_t idesc;
   // ---- tensor-parallel fusion (normal tiling only) ----
@@ -136,6 +137,8 @@ __device__ __forceinline__ void st_cluster_v4f(uint32_t cluster_addr, float a, f
 __device__ __forceinline__ void fence_acq_rel_cluster() { asm volatile("fence.acq_rel.cluster;" ::: "memory"); }
 
 __device__ __forceinline__ float silu_f(float v) { return v / (1.f + __expf(-v)); }
+// activation of the gate rows of a gated epilogue: SiLU, or the tanh form of the GELU
+__device__ __forceinline__ float gate_act(float v, int gelu) { return gelu ? gelu_tanh_f(v) : silu_f(v); }
 
 __device__ __forceinline__ uint32_t pack_out2(float lo, float hi, int out_f16) {
   if (out_f16) {
@@ -508,7 +511,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
                       x *= sa * p.b_scale[tc * BN + cc];
                       u *= sa * p.b_scale[tc * BN + BN / 2 + cc];
                     }
-                    x = silu_f(x) * u;
+                    x = gate_act(x, p.gate_gelu) * u;
                   } else {
                     const int64_t col = col0 + cc;
                     if (p.is_int8 && col < n_out) x *= sa * p.b_scale[col];
@@ -565,7 +568,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
                   x *= sa * p.b_scale[tc * BN + c + v8 * 8 + j];
                   u *= sa * p.b_scale[tc * BN + BN / 2 + c + v8 * 8 + j];
                 }
-                x = silu_f(x) * u;
+                x = gate_act(x, p.gate_gelu) * u;
               } else {
                 if (p.is_int8) x *= sa * p.b_scale[col + j];
                 if (p.bias != nullptr) x += load_out1(p.bias, col + j, p.out_f16);
@@ -708,7 +711,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
                       xv *= p.a_scale[j] * p.b_scale[wrow];
                       uv *= p.a_scale[j] * p.b_scale[wrow + kBM];
                     }
-                    xv = silu_f(xv) * uv;
+                    xv = gate_act(xv, p.gate_gelu) * uv;
                     ocol = static_cast<int64_t>(tr) * kBM + row_in_tile;
                   } else {
                     if (p.is_int8) xv *= p.a_scale[j] * p.b_scale[wrow];
@@ -759,7 +762,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
                   x *= p.a_scale[mi] * p.b_scale[wrow];
                   u *= p.a_scale[mi] * p.b_scale[wrow + kBM];
                 }
-                x = silu_f(x) * u;
+                x = gate_act(x, p.gate_gelu) * u;
                 ocol = static_cast<int64_t>(tr) * kBM + row_in_tile;
               } else {
                 if (p.is_int8) x *= p.a_scale[mi] * p.b_scale[wrow];
@@ -1157,7 +1160,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_consta
                 x *= sa * p.b_scale[tc * kPairBN + c + v8 * 8 + j];
                 u *= sa * p.b_scale[tc * kPairBN + kPairBN / 2 + c + v8 * 8 + j];
               }
-              x = silu_f(x) * u;
+              x = gate_act(x, p.gate_gelu) * u;
             } else {
               if (p.is_int8) x *= sa * p.b_scale[col + j];
               if (p.bias != nullptr) x += load_out1(p.bias, col + j, p.out_f16);
@@ -1363,6 +1366,7 @@ int launch_gemm(const GemmArgs& a, cudaStream_t s) {
   p.out_f16 = (a.dt == kF16) ? 1 : 0;
   p.is_int8 = a.is_int8;
   p.row_static = a.b_static;
+  p.gate_gelu = a.swiglu == 2 ? 1 : 0;
   {
     // The CTAs of a following small-batch GEMM fit beside ours when both keep their rings short: they are
     // then launched while this kernel still streams, fetch their first weight tiles, and take over the memory

@@ -24,6 +24,11 @@ void launch_layernorm(const void* x, const void* w, const void* b, void* out, in
                       DType dt, cudaStream_t s);
 // act: 0 = silu(gate)*up, 1 = gelu_tanh(gate)*up ; x is [rows, 2*inter] = [gate | up]
 void launch_act_and_mul(const void* x, void* out, int rows, int inter, int act, DType dt, cudaStream_t s);
+// fp32 residual stream with a Dynamic Tanh norm: x += mult * y (y may be null), h = tanh(alpha x) * w + b
+void launch_residual_dyt(float* x, const void* y, float mult, const float* alpha, const float* w, const float* b, void* h,
+                         int rows, int width, DType dt, cudaStream_t s);
+void launch_embedding_f32(const int64_t* ids, const void* table, float* out, int tokens, int width, int vocab, DType dt,
+                          int* status, cudaStream_t s);
 void launch_gelu_tanh(const void* x, void* out, int64_t n, DType dt, cudaStream_t s);
 void launch_embedding(const int64_t* ids, const void* table, void* out, int tokens, int hidden, int vocab,
                       DType dt, int* status, cudaStream_t s);
@@ -84,7 +89,7 @@ struct GemmArgs {
   const float* b_scale;  // int8 only: per-column scale [n]
   int m, n, k;
   int64_t lda, ldb, ldc, ld_res;
-  int swiglu;            // 1: b rows alternate 128 gate / 128 up rows; out is [m, n/2]
+  int swiglu;            // 1: b rows alternate 128 gate / 128 up rows; out is [m, n/2] = silu(gate) * up; 2: gelu_tanh(gate) * up
   DType dt;              // element type of a, b (kBF16 / kF16) ; out has the same type
   int is_int8;           // 1: a, b are int8, out type given by dt
   float* workspace;      // split-K partial sums (small-m path), may be null when not needed
@@ -224,26 +229,83 @@ struct AttnArgs {
   int window;               // > 0: a query at position i sees keys i - window + 1 .. i only (causal attention)
   float logit_cap;          // > 0: scores pass through cap * tanh(score / cap) before the softmax
   DType dt;
+  const float* sink;        // [Hq] or null: per head, exp(sink) joins the softmax denominator (no key, no value, unscaled)
   int kv_fmt;               // 0: the caches hold dt; 1 / 2: unscaled e4m3 / e5m2 bytes (strides then count bytes)
 };
 int launch_attention(const AttnArgs& args, cudaStream_t s);
 int decode_num_splits(int batch, int hkv, int max_seq_len, int num_sms);
 
+// ----- latent attention (one cached row of `rank` features per token, shared by all heads) ------------
+// RMS norm of both parts of the down projections' rows [q_rank | kv_rank]: the first into cq [tokens, q_rank], the
+// second into the cache row loc[t].  kv_rank 0: the layer reads another layer's latents and writes none.
+void launch_latent_prologue(const void* y, int64_t ld, int tokens, int q_rank, int kv_rank, const float* q_w, const float* kv_w,
+                            float eps, void* cq, const int64_t* loc, void* cache, int64_t cache_ld, int64_t num_slots, DType dt,
+                            int* status, cudaStream_t s);
+// out[start[b] + j] = latent of token j of request b, j < lens[b]
+void launch_latent_gather(const void* cache, int64_t cache_ld, int rank, int elem_bytes, const int* rtt, int64_t rtt_stride,
+                          const int* req, const int* lens, const int* start, int batch, int max_len, void* out,
+                          int64_t num_slots, int* status, cudaStream_t s);
+// out[t, h, :] = w[h] x[t, h, :] with w [heads, N, K], K % 8 == 0, 16-bit types (else -1)
+int launch_head_linear(const void* x, int64_t x_tok, int64_t x_head, const void* w, void* out, int64_t out_tok, int64_t out_head,
+                       int tokens, int heads, int N, int K, int num_sms, DType dt, cudaStream_t s);
+struct LatentAttnArgs {
+  const void* q;            // [rows, heads, rank] queries taken to the latent space
+  const void* cache;        // latent of slot s at s * cache_ld (elements)
+  void* out;                // [rows, heads, rank]
+  float* part_o;            // splits > 1: [rows, heads, splits, rank]
+  float* part_lse;          // splits > 1: [rows, heads, splits]
+  const int* req_to_token;
+  const int* row_req;       // [rows] request-table row of each query
+  const int64_t* row_pos;   // [rows] its position: it sees keys 0 .. position
+  const float* sink;        // [heads] or null
+  int* status;
+  int64_t rtt_stride, cache_ld, num_slots;
+  int rows, heads, rank, splits;
+  float scale;
+  DType dt;
+};
+int launch_latent_attention(const LatentAttnArgs& args, cudaStream_t s);
+int latent_num_splits(int rows, int heads, int max_seq_len, int num_sms);
+bool latent_mma_covers(int rank, int64_t cache_ld, DType dt);   // false: the fp32 kernel runs, splits must be 1
+
 // ----- gated delta net (hybrid models) -----------------------------------------------------------
 // Ragged sequences: request b owns rows q_start[b] .. q_start[b] + lens[b] of the token-major inputs and
 // row slots[b] of the state tensors; has_state[b] != 0 resumes from the stored state.
-int launch_gdn_conv1d_silu(const void* x, const void* w, void* conv_state, const int* slots, const int* lens,
+int launch_gdn_conv1d_silu(const void* x, int64_t x_ld, const void* w, void* conv_state, const int* slots, const int* lens,
                            const int* has_state, const int* q_start, void* out, int batch, int max_tokens, int channels, int K,
                            DType dt, cudaStream_t s);
-int launch_gdn_recurrent(const void* q, const void* k, const void* v, const float* g, const float* beta, float* state,
-                         const int* slots, const int* lens, const int* has_state, const int* q_start, void* out, int batch,
-                         int heads, int dk, int dv, DType dt, cudaStream_t s);
-// The same rule evaluated 64 tokens at a time with tensor-core products (prefill); same arguments and state layout.
-int launch_gdn_chunk(const void* q, const void* k, const void* v, const float* g, const float* beta, float* state,
-                     const int* slots, const int* lens, const int* has_state, const int* q_start, void* out, int batch,
-                     int heads, int dk, int dv, int num_sms, DType dt, cudaStream_t s);
-void launch_rmsnorm_gated(const void* x, const void* gate, const void* w, void* out, int rows, int width, float eps, DType dt,
-                          cudaStream_t s);
+// beta = sigmoid(b), g = -exp(a_log) * softplus(a + dt_bias); b and a [tokens, heads] with rows ld apart
+void launch_gdn_gates(const void* b, const void* a, int64_t ld, const float* a_log, const float* dt_bias, float* g, float* beta,
+                      int64_t tokens, int heads, DType dt, cudaStream_t s);
+struct GdnRuleParams {
+  const void* q;            // [T, k_heads, dk], token rows q_ld apart (elements)
+  const void* k;            // [T, k_heads, dk]
+  const void* v;            // [T, heads, dv]
+  void* out;                // [T, heads, dv] contiguous
+  const float* g;           // log decay [T, heads], or null: gates from the four fields below (recurrent kernel only)
+  const float* beta;
+  const void* b_raw;        // [T, heads] with rows gate_ld apart
+  const void* a_raw;
+  const float* a_log;       // [heads]
+  const float* dt_bias;     // [heads]
+  float* state;             // [rows, heads, dk, dv]
+  const int* slots;
+  const int* lens;
+  const int* has_state;
+  const int* q_start;
+  int64_t q_ld, k_ld, v_ld, gate_ld;
+  int batch, heads, k_heads, dk, dv;
+  int split_tf32;           // chunk kernel: two-term tf32 operands (fp32-like products)
+  DType dt;
+};
+// token by token; dk up to 512, any dv
+int launch_gdn_recurrent(const GdnRuleParams& p, cudaStream_t s);
+// the same rule evaluated 64 tokens at a time with tensor-core products (prefill); dk up to 128, multiples of 8
+int launch_gdn_chunk(const GdnRuleParams& p, int num_sms, cudaStream_t s);
+bool gdn_chunk_covers(const GdnRuleParams& p);
+// x, out [rows = tokens * heads, width] contiguous, gate [tokens, heads * width] with rows gate_ld apart
+void launch_rmsnorm_gated(const void* x, const void* gate, int64_t gate_ld, const void* w, void* out, int64_t rows, int heads,
+                          int width, float eps, int round_norm, DType dt, cudaStream_t s);
 
 // ----- vision tower helpers ------------------------------------------------------------------
 // qkv [T, 3, H, D] (D <= 128, D % 8 == 0) -> q, k, v [T, H, 128] zero-padded; q and k get the 2-D rotary

@@ -1,0 +1,685 @@
+// Latent attention: every token leaves ONE row c of `rank` features in the cache, shared by all heads; a head's keys
+// and values are W_uk[h] c and W_uv[h] c.  Two ways to evaluate it, both causal, both with an optional sink per head:
+//
+//   expanded (many new tokens): K and V of the whole context are formed by matrix products and the ordinary
+//       attention kernels run on them; this file only gathers the context's latents (latent_gather).
+//   absorbed (decode, short extends): the products move to the query side.  q' = W_uk[h]^T q has `rank` features,
+//       score = q' . c, and the weighted sum of the c rows is carried through W_uv[h] once per query.  The cache is
+//       read once for all heads and nothing per head is stored.
+//
+// latent_attn_mma_kernel is the absorbed form for 16-bit types.  A CTA owns one query token, 16 or 32 heads (the MMA
+// M dimension) and a range of the context, 32 tokens at a time.  The rank features are dealt to the warps, CW each:
+// a warp moves its own feature slice of every c row with cp.async, keeps its slice of q' in registers, multiplies
+// the slice's share of the scores and owns the same slice of the output.  So c is read from shared memory twice (as
+// keys, and transposed as values) by the same warp, tiles need no block barrier on their way in, and the warps meet
+// only to add up the partial scores.  This is a stream of the cache with little arithmetic per byte (2 x heads
+// multiply-adds per element): warp-level MMA keeps up with HBM for the 16 to 32 heads of a tile, and its operands
+// come from shared memory in any width, which is what lets one kernel serve every rank that is a multiple of 8.
+#include <algorithm>
+
+#include "common.cuh"
+#include "kernels.h"
+
+namespace mb200 {
+namespace {
+
+constexpr float kLatLog2e = 1.4426950408889634f;
+
+// ---------------------------------------------------------------------------------------------
+// Prologue: the down projections' output rows are [query latent | cache latent]; both are RMS-normed in 32-bit, the
+// first goes to `cq`, the second to the cache row of the token.  grid (tokens, 1 or 2).
+// ---------------------------------------------------------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(128) latent_prologue_kernel(const T* __restrict__ y, int64_t ld, int q_rank, int kv_rank,
+                                                              const float* __restrict__ q_w, const float* __restrict__ kv_w,
+                                                              float eps, T* __restrict__ cq, const int64_t* __restrict__ loc,
+                                                              T* __restrict__ cache, int64_t cache_ld, int64_t num_slots,
+                                                              int* status) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float red[4];
+  const int t = blockIdx.x, part = blockIdx.y, tid = threadIdx.x;
+  const int n = part == 0 ? q_rank : kv_rank;
+  const T* row = y + static_cast<int64_t>(t) * ld + (part == 0 ? 0 : q_rank);
+  const float* w = part == 0 ? q_w : kv_w;
+  T* dst;
+  if (part == 0) {
+    dst = cq + static_cast<int64_t>(t) * q_rank;
+  } else {
+    const int64_t slot = loc[t];
+    if (slot < 0 || slot >= num_slots) {
+      if (tid == 0 && status != nullptr) atomicExch(status, kStatusBadIndex);
+      return;
+    }
+    dst = cache + slot * cache_ld;
+  }
+  float ss = 0.f;
+  for (int c = tid; c < n; c += 128) {
+    const float f = to_f32(row[c]);
+    ss = fmaf(f, f, ss);
+  }
+  ss = warp_sum(ss);
+  if ((tid & 31) == 0) red[tid >> 5] = ss;
+  __syncthreads();
+  ss = red[0] + red[1] + red[2] + red[3];
+  const float r = 1.f / sqrtf(ss / static_cast<float>(n) + eps);
+  for (int c = tid; c < n; c += 128) dst[c] = from_f32<T>(to_f32(row[c]) * r * w[c]);
+}
+
+// Rows of a request's context, in position order: out[start[b] + j] = cache[rtt[req[b]][j]] for j < lens[b].
+template <typename V>
+__global__ void __launch_bounds__(256) latent_gather_kernel(const V* __restrict__ cache, int64_t cache_ld_v, int row_v,
+                                                            const int* __restrict__ rtt, int64_t rtt_stride,
+                                                            const int* __restrict__ req, const int* __restrict__ lens,
+                                                            const int* __restrict__ start, V* __restrict__ out,
+                                                            int64_t num_slots, int* status) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int b = blockIdx.y, n = lens[b];
+  const int lane = threadIdx.x & 31;
+  const int* slots = rtt + static_cast<int64_t>(req[b]) * rtt_stride;
+  for (int j = blockIdx.x * 8 + (threadIdx.x >> 5); j < n; j += gridDim.x * 8) {
+    const int s = slots[j];
+    const bool ok = s >= 0 && s < num_slots;
+    if (!ok && lane == 0 && status != nullptr) atomicExch(status, kStatusBadIndex);
+    V* dst = out + static_cast<int64_t>(start[b] + j) * row_v;
+    const V* src = cache + static_cast<int64_t>(ok ? s : 0) * cache_ld_v;
+    for (int c = lane; c < row_v; c += 32) dst[c] = src[c];
+  }
+}
+
+// ---------------------------------------------------------------------------------------------
+// Per-head projection out[t, h, :] = W[h] x[t, h, :], W [H, N, K].  A warp owns 16 rows of one head's W (the MMA M
+// dimension) and tiles of 8 tokens; a lane feeds 16 contiguous bytes of W and of x to two MMAs, the same
+// permutation of k in both operands.  KS > 1: the warps of the CTA split k of the same 16 rows.
+// ---------------------------------------------------------------------------------------------
+template <typename T>
+__device__ __forceinline__ void mma_16816(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0,
+                                          uint32_t b1) {
+  if constexpr (sizeof(T) == 2 && std::is_same<T, __half>::value) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.f16.f16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+                 : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+  } else {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+                 : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+  }
+}
+
+constexpr int kHlTokTiles = 4;   // tiles of 8 tokens per CTA
+
+template <typename T, int KS>
+__global__ void __launch_bounds__(128) head_linear_kernel(const T* __restrict__ x, int64_t x_tok, int64_t x_head,
+                                                          const T* __restrict__ w, T* __restrict__ out, int64_t out_tok,
+                                                          int64_t out_head, int tokens, int N, int K) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float part[KS > 1 ? KS : 1][kHlTokTiles][16][8];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int h = blockIdx.y;
+  const int n0 = KS > 1 ? blockIdx.x * 16 : (blockIdx.x * 4 + warp) * 16;
+  const int t0 = blockIdx.z * kHlTokTiles * 8;
+  const int g = lane >> 2, q = lane & 3;
+  float acc[kHlTokTiles][4];
+#pragma unroll
+  for (int i = 0; i < kHlTokTiles; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+  if (n0 < N) {
+    const T* wr0 = w + (static_cast<int64_t>(h) * N + n0 + g) * K;
+    const T* wr1 = wr0 + 8 * static_cast<int64_t>(K);
+    const bool ok0 = n0 + g < N, ok1 = n0 + g + 8 < N;
+    const uint4 zero = make_uint4(0, 0, 0, 0);
+#pragma unroll 4
+    for (int k0 = KS > 1 ? warp * 32 : 0; k0 < K; k0 += 32 * KS) {
+      const int k = k0 + q * 8;
+      const bool okk = k < K;
+      const uint4 a = ok0 && okk ? __ldg(reinterpret_cast<const uint4*>(wr0 + k)) : zero;
+      const uint4 b = ok1 && okk ? __ldg(reinterpret_cast<const uint4*>(wr1 + k)) : zero;
+#pragma unroll
+      for (int i = 0; i < kHlTokTiles; ++i) {
+        const int t = t0 + i * 8 + g;
+        if (t0 + i * 8 < tokens) {
+          const uint4 v = t < tokens && okk ? *reinterpret_cast<const uint4*>(x + t * x_tok + h * x_head + k) : zero;
+          mma_16816<T>(acc[i], a.x, b.x, a.y, b.y, v.x, v.y);
+          mma_16816<T>(acc[i], a.z, b.z, a.w, b.w, v.z, v.w);
+        }
+      }
+    }
+  }
+  // acc[i]: rows g and g + 8 of W, tokens i * 8 + 2 q and + 1
+  if constexpr (KS > 1) {
+#pragma unroll
+    for (int i = 0; i < kHlTokTiles; ++i) {
+      part[warp][i][g][2 * q] = acc[i][0];
+      part[warp][i][g][2 * q + 1] = acc[i][1];
+      part[warp][i][g + 8][2 * q] = acc[i][2];
+      part[warp][i][g + 8][2 * q + 1] = acc[i][3];
+    }
+    __syncthreads();
+    for (int e = threadIdx.x; e < kHlTokTiles * 128; e += 128) {
+      const int i = e >> 7, tok = (e >> 4) & 7, r = e & 15;
+      const int t = t0 + i * 8 + tok;
+      if (t < tokens && n0 + r < N) {
+        float v = 0.f;
+#pragma unroll
+        for (int s = 0; s < KS; ++s) v += part[s][i][r][tok];
+        out[t * out_tok + h * out_head + n0 + r] = from_f32<T>(v);
+      }
+    }
+  } else if (n0 < N) {
+#pragma unroll
+    for (int i = 0; i < kHlTokTiles; ++i) {
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int t = t0 + i * 8 + 2 * q + (j & 1), r = n0 + g + (j >> 1) * 8;
+        if (t < tokens && r < N) out[t * out_tok + h * out_head + r] = from_f32<T>(acc[i][j]);
+      }
+    }
+  }
+}
+
+// ---------------------------------------------------------------------------------------------
+// Absorbed attention
+// ---------------------------------------------------------------------------------------------
+struct LatentParams {
+  const void* q;            // [rows, heads, rank]
+  const void* cache;        // latent of slot s at s * cache_ld
+  void* out;                // [rows, heads, rank]
+  float* part_o;            // splits > 1: [rows, heads, splits, rank]
+  float* part_lse;          // splits > 1: [rows, heads, splits], log2 domain
+  const int* rtt;
+  const int* row_req;       // [rows] row of the request table
+  const int64_t* row_pos;   // [rows] position of the query: it sees keys 0 .. pos
+  const float* sink;        // [heads] or null
+  int* status;
+  int64_t rtt_stride, cache_ld, num_slots;
+  int rows, heads, rank, splits;
+  float scale;
+};
+
+__device__ __forceinline__ float lat_inv_denominator(float l, float m, const float* sink, int head) {
+  if (!(l > 0.f)) return 0.f;
+  if (sink == nullptr) return 1.f / l;
+  const float d = sink[head] * kLatLog2e - m;
+  if (d > 0.f) {
+    const float e = exp2f(-d);
+    return e / fmaf(l, e, 1.f);
+  }
+  return 1.f / (l + exp2f(d));
+}
+
+__device__ __forceinline__ void lat_cp16(uint32_t dst, const void* src, bool valid) {
+  const int sz = valid ? 16 : 0;
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(sz) : "memory");
+}
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(addr)
+               : "memory");
+}
+__device__ __forceinline__ void ldsm4_t(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(addr)
+               : "memory");
+}
+
+constexpr int kLatTok = 32;        // context tokens per tile
+constexpr int kLatSLd = kLatTok + 8;
+
+template <int CW, int MT>
+struct LatCfg {
+  static constexpr int kStages = CW >= 64 ? 2 : 3;
+  static constexpr int kRowBytes = CW * 2 + 16;                // one token of a warp's slice, padded: ldmatrix without conflicts
+  static constexpr int kSliceBytes = kLatTok * kRowBytes;
+  static constexpr int smem(int warps) {
+    return kStages * warps * kSliceBytes + (warps + 1) * MT * 16 * kLatSLd * 4;
+  }
+};
+
+template <typename T, int CW, int MT>
+__global__ void __launch_bounds__(256) latent_attn_mma_kernel(const LatentParams p) {
+  using C = LatCfg<CW, MT>;
+  constexpr int kM = MT * 16;
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ __align__(16) uint8_t lat_smem[];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, warps = blockDim.x >> 5;
+  const int g = lane >> 2, q = lane & 3;
+  const int row = blockIdx.z, h0 = blockIdx.y * kM, split = blockIdx.x;
+  float* sp = reinterpret_cast<float*>(lat_smem + C::kStages * warps * C::kSliceBytes);   // [warps][kM][kLatSLd] partial scores
+  float* ss = sp + warps * kM * kLatSLd;                                                  // [kM][kLatSLd] scores
+  const uint32_t slice0 = smem_u32(lat_smem) + warp * C::kSliceBytes;                     // stage s: + s * warps * kSliceBytes
+  const uint32_t stage_step = warps * C::kSliceBytes;
+
+  const int n = static_cast<int>(p.row_pos[row]) + 1;
+  const int tiles = (n + kLatTok - 1) / kLatTok;
+  const int per = (tiles + p.splits - 1) / p.splits;
+  const int tile0 = split * per, tile1 = min(tiles, tile0 + per);
+  if (tile0 >= tile1) {   // empty split: a neutral partial
+    for (int i = tid; i < kM * p.rank; i += blockDim.x) {
+      const int h = h0 + i / p.rank;
+      if (h < p.heads) p.part_o[((static_cast<int64_t>(row) * p.heads + h) * p.splits + split) * p.rank + i % p.rank] = 0.f;
+    }
+    if (tid < kM && h0 + tid < p.heads)
+      p.part_lse[(static_cast<int64_t>(row) * p.heads + h0 + tid) * p.splits + split] = -INFINITY;
+    return;
+  }
+  const int* slots = p.rtt + static_cast<int64_t>(p.row_req[row]) * p.rtt_stride;
+  const T* cache = static_cast<const T*>(p.cache);
+  const int c0 = warp * CW;
+
+  // this warp's slice of q' as MMA A fragments
+  uint32_t qa[MT][CW / 16][4];
+  {
+    const T* qb = static_cast<const T*>(p.q) + static_cast<int64_t>(row) * p.heads * p.rank;
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+      for (int ks = 0; ks < CW / 16; ++ks)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const int h = h0 + mt * 16 + g + (j & 1) * 8, c = c0 + ks * 16 + 2 * q + (j >> 1) * 8;
+          qa[mt][ks][j] = (h < p.heads && c < p.rank) ? *reinterpret_cast<const uint32_t*>(qb + static_cast<int64_t>(h) * p.rank + c) : 0u;
+        }
+  }
+  float o[MT][CW / 8][4];
+  float m_run[MT][2], l_run[MT][2];
+#pragma unroll
+  for (int mt = 0; mt < MT; ++mt) {
+#pragma unroll
+    for (int i = 0; i < CW / 8; ++i) o[mt][i][0] = o[mt][i][1] = o[mt][i][2] = o[mt][i][3] = 0.f;
+    m_run[mt][0] = m_run[mt][1] = -INFINITY;
+    l_run[mt][0] = l_run[mt][1] = 0.f;
+  }
+
+  auto slot_of = [&](int tile) {   // lane's token of the tile, -1 past the end
+    const int tk = tile * kLatTok + lane;
+    int s = (tile < tile1 && tk < n) ? __ldg(slots + tk) : -1;
+    if (s < -1 || s >= p.num_slots) {
+      if (p.status != nullptr) atomicExch(p.status, kStatusBadIndex);
+      s = -1;
+    }
+    return s;
+  };
+  auto fetch = [&](int stage, int my_slot) {
+    constexpr int kCh = CW / 8;                 // 16-byte pieces per token of the slice
+    const uint32_t dst = slice0 + stage * stage_step;
+#pragma unroll
+    for (int i = 0; i < kCh; ++i) {
+      const int piece = i * 32 + lane, tk = piece / kCh, ch = piece % kCh;
+      const int s = __shfl_sync(0xffffffffu, my_slot, tk);
+      const int c = c0 + ch * 8;
+      const bool ok = s >= 0 && c < p.rank;
+      lat_cp16(dst + tk * C::kRowBytes + ch * 16, cache + (ok ? static_cast<int64_t>(s) * p.cache_ld + c : 0), ok);
+    }
+  };
+
+  int slot_next = slot_of(tile0);
+#pragma unroll
+  for (int s = 0; s < C::kStages - 1; ++s) {
+    fetch(s, slot_next);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    slot_next = slot_of(tile0 + s + 1);
+  }
+  const float scale_log2 = p.scale * kLatLog2e;
+
+  for (int t = tile0, it = 0; t < tile1; ++t, ++it) {
+    const int stage = it % C::kStages;
+    // the stage filled now was read by the previous tile of this warp only
+    fetch((it + C::kStages - 1) % C::kStages, slot_next);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    slot_next = slot_of(t + C::kStages);
+    asm volatile("cp.async.wait_group %0;" ::"n"(C::kStages - 1) : "memory");
+    __syncwarp();
+    const uint32_t tile = slice0 + stage * stage_step;
+
+    // ---- the slice's share of the scores ----
+    {
+      float s[MT][kLatTok / 8][4];
+#pragma unroll
+      for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+        for (int i = 0; i < kLatTok / 8; ++i) s[mt][i][0] = s[mt][i][1] = s[mt][i][2] = s[mt][i][3] = 0.f;
+#pragma unroll
+      for (int ks = 0; ks < CW / 16; ++ks) {
+#pragma unroll
+        for (int np = 0; np < kLatTok / 16; ++np) {
+          uint32_t b[4];   // tokens np*16 + 0..7: k 0-7, k 8-15; tokens + 8: the same
+          ldsm4(b, tile + (np * 16 + (lane & 7) + ((lane >> 4) << 3)) * C::kRowBytes + ks * 32 + ((lane >> 3) & 1) * 16);
+#pragma unroll
+          for (int mt = 0; mt < MT; ++mt) {
+            mma_16816<T>(s[mt][np * 2], qa[mt][ks][0], qa[mt][ks][1], qa[mt][ks][2], qa[mt][ks][3], b[0], b[1]);
+            mma_16816<T>(s[mt][np * 2 + 1], qa[mt][ks][0], qa[mt][ks][1], qa[mt][ks][2], qa[mt][ks][3], b[2], b[3]);
+          }
+        }
+      }
+      float* mine = sp + warp * kM * kLatSLd;
+#pragma unroll
+      for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+        for (int i = 0; i < kLatTok / 8; ++i) {
+          *reinterpret_cast<float2*>(mine + (mt * 16 + g) * kLatSLd + i * 8 + 2 * q) = make_float2(s[mt][i][0], s[mt][i][1]);
+          *reinterpret_cast<float2*>(mine + (mt * 16 + g + 8) * kLatSLd + i * 8 + 2 * q) = make_float2(s[mt][i][2], s[mt][i][3]);
+        }
+    }
+    __syncthreads();
+    for (int e = tid; e < kM * kLatTok; e += blockDim.x) {
+      const int at = (e / kLatTok) * kLatSLd + e % kLatTok;
+      float v = 0.f;
+      for (int w = 0; w < warps; ++w) v += sp[w * kM * kLatSLd + at];
+      ss[at] = (t * kLatTok + e % kLatTok < n) ? v * scale_log2 : -INFINITY;
+    }
+    __syncthreads();
+
+    // ---- softmax (every warp the same rows) and this warp's slice of the output ----
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt) {
+      float2 sv[2][4];     // [row g / g + 8][column pair]
+      float mx[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+      for (int r = 0; r < 2; ++r)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          sv[r][i] = *reinterpret_cast<const float2*>(ss + (mt * 16 + g + r * 8) * kLatSLd + i * 8 + 2 * q);
+          mx[r] = fmaxf(mx[r], fmaxf(sv[r][i].x, sv[r][i].y));
+        }
+      float f[2];
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
+        mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
+        mx[r] = fmaxf(mx[r], m_run[mt][r]);       // a tile has a visible key, so this is finite
+        f[r] = exp2f(m_run[mt][r] - mx[r]);
+        m_run[mt][r] = mx[r];
+        l_run[mt][r] *= f[r];
+      }
+      uint32_t pa[2][4];   // P of two k-steps of 16 tokens as A fragments
+#pragma unroll
+      for (int r = 0; r < 2; ++r)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          T two[2] = {from_f32<T>(exp2f(sv[r][i].x - mx[r])), from_f32<T>(exp2f(sv[r][i].y - mx[r]))};
+          l_run[mt][r] += to_f32(two[0]) + to_f32(two[1]);      // what the product sees
+          pa[i >> 1][r + (i & 1) * 2] = *reinterpret_cast<const uint32_t*>(two);
+        }
+      if (__any_sync(0xffffffffu, f[0] != 1.f || f[1] != 1.f)) {
+#pragma unroll
+        for (int i = 0; i < CW / 8; ++i) {
+          o[mt][i][0] *= f[0];
+          o[mt][i][1] *= f[0];
+          o[mt][i][2] *= f[1];
+          o[mt][i][3] *= f[1];
+        }
+      }
+#pragma unroll
+      for (int ks = 0; ks < 2; ++ks)
+#pragma unroll
+        for (int np = 0; np < CW / 16; ++np) {
+          uint32_t b[4];   // features np*16 + 0..7: tokens 0-7, tokens 8-15; features + 8: the same
+          ldsm4_t(b, tile + (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * C::kRowBytes + np * 32 + (lane >> 4) * 16);
+          mma_16816<T>(o[mt][np * 2], pa[ks][0], pa[ks][1], pa[ks][2], pa[ks][3], b[0], b[1]);
+          mma_16816<T>(o[mt][np * 2 + 1], pa[ks][0], pa[ks][1], pa[ks][2], pa[ks][3], b[2], b[3]);
+        }
+    }
+    __syncwarp();
+  }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+
+#pragma unroll
+  for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      float l = l_run[mt][r];
+      l += __shfl_xor_sync(0xffffffffu, l, 1);
+      l += __shfl_xor_sync(0xffffffffu, l, 2);
+      const int h = h0 + mt * 16 + g + r * 8;
+      if (h >= p.heads) continue;
+      const int64_t at = static_cast<int64_t>(row) * p.heads + h;
+      if (p.splits > 1) {
+        const float inv = 1.f / l;
+        float* po = p.part_o + (at * p.splits + split) * p.rank;
+#pragma unroll
+        for (int i = 0; i < CW / 8; ++i) {
+          const int c = c0 + i * 8 + 2 * q;
+          if (c < p.rank) *reinterpret_cast<float2*>(po + c) = make_float2(o[mt][i][r * 2] * inv, o[mt][i][r * 2 + 1] * inv);
+        }
+        if (warp == 0 && q == 0) p.part_lse[at * p.splits + split] = m_run[mt][r] + log2f(l);
+      } else {
+        const float inv = lat_inv_denominator(l, m_run[mt][r], p.sink, h);
+        T* po = static_cast<T*>(p.out) + at * p.rank;
+#pragma unroll
+        for (int i = 0; i < CW / 8; ++i) {
+          const int c = c0 + i * 8 + 2 * q;
+          if (c < p.rank) {
+            T two[2] = {from_f32<T>(o[mt][i][r * 2] * inv), from_f32<T>(o[mt][i][r * 2 + 1] * inv)};
+            *reinterpret_cast<uint32_t*>(po + c) = *reinterpret_cast<const uint32_t*>(two);
+          }
+        }
+      }
+    }
+}
+
+// out = sum_s w_s * O_s, w_s = 2^(lse_s - max) / (sum + sink); grid (heads, rows)
+template <typename T>
+__global__ void __launch_bounds__(128) latent_merge_kernel(const LatentParams p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int h = blockIdx.x, row = blockIdx.y;
+  const int64_t at = static_cast<int64_t>(row) * p.heads + h;
+  const float* lse = p.part_lse + at * p.splits;
+  float m = -INFINITY;
+  for (int s = 0; s < p.splits; ++s) m = fmaxf(m, lse[s]);
+  float den = 0.f;
+  if (p.sink != nullptr) {
+    const float sl = p.sink[h] * kLatLog2e;
+    m = fmaxf(m, sl);
+    den = exp2f(sl - m);
+  }
+  for (int s = 0; s < p.splits; ++s) den += exp2f(lse[s] - m);
+  const float inv = 1.f / den;
+  for (int c = threadIdx.x; c < p.rank; c += blockDim.x) {
+    float acc = 0.f;
+    for (int s = 0; s < p.splits; ++s) {
+      const float w = exp2f(lse[s] - m);
+      if (w > 0.f) acc = fmaf(w, p.part_o[(at * p.splits + s) * p.rank + c], acc);
+    }
+    static_cast<T*>(p.out)[at * p.rank + c] = from_f32<T>(acc * inv);
+  }
+}
+
+// Any element type and any rank up to 1024, all in fp32: one CTA per (query token, head), tiles of 64 context tokens.
+constexpr int kLatAnyTok = 64, kLatAnyThreads = 128, kLatAnyCols = 8;
+
+template <typename T>
+__global__ void __launch_bounds__(kLatAnyThreads) latent_attn_any_kernel(const LatentParams p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float sq[kLatAnyThreads * kLatAnyCols];
+  __shared__ float sc[kLatAnyTok];
+  __shared__ int sl[kLatAnyTok];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int h = blockIdx.x, row = blockIdx.y;
+  const int64_t at = (static_cast<int64_t>(row) * p.heads + h) * p.rank;
+  const T* qr = static_cast<const T*>(p.q) + at;
+  for (int c = tid; c < p.rank; c += kLatAnyThreads) sq[c] = to_f32(qr[c]);
+  const int n = static_cast<int>(p.row_pos[row]) + 1;
+  const int* slots = p.rtt + static_cast<int64_t>(p.row_req[row]) * p.rtt_stride;
+  const T* cache = static_cast<const T*>(p.cache);
+  float acc[kLatAnyCols];
+#pragma unroll
+  for (int i = 0; i < kLatAnyCols; ++i) acc[i] = 0.f;
+  float m = -INFINITY, l = 0.f;
+  for (int t0 = 0; t0 < n; t0 += kLatAnyTok) {
+    const int nt = min(kLatAnyTok, n - t0);
+    __syncthreads();      // sc and sl of the previous tile are no longer read; sq is written
+    if (tid < nt) {
+      int s = slots[t0 + tid];
+      if (s < 0 || s >= p.num_slots) {
+        if (p.status != nullptr) atomicExch(p.status, kStatusBadIndex);
+        s = 0;
+      }
+      sl[tid] = s;
+    }
+    __syncthreads();
+    for (int j = warp; j < nt; j += kLatAnyThreads / 32) {
+      const T* cr = cache + static_cast<int64_t>(sl[j]) * p.cache_ld;
+      float d = 0.f;
+      for (int c = lane; c < p.rank; c += 32) d = fmaf(sq[c], to_f32(cr[c]), d);
+      d = warp_sum(d);
+      if (lane == 0) sc[j] = d * p.scale;
+    }
+    __syncthreads();
+    float mt = m;
+    for (int j = 0; j < nt; ++j) mt = fmaxf(mt, sc[j]);
+    const float f = expf(m - mt);
+    m = mt;
+    __syncthreads();      // every thread has the maximum before the scores become weights
+    if (tid < nt) sc[tid] = expf(sc[tid] - m);
+    __syncthreads();
+    l *= f;
+#pragma unroll
+    for (int i = 0; i < kLatAnyCols; ++i) acc[i] *= f;
+    for (int j = 0; j < nt; ++j) {
+      const float w = sc[j];
+      l += w;
+      const T* cr = cache + static_cast<int64_t>(sl[j]) * p.cache_ld;
+#pragma unroll
+      for (int i = 0; i < kLatAnyCols; ++i) {
+        const int c = tid + i * kLatAnyThreads;
+        if (c < p.rank) acc[i] = fmaf(w, to_f32(cr[c]), acc[i]);
+      }
+    }
+  }
+  float inv;
+  if (p.sink == nullptr) {
+    inv = 1.f / l;
+  } else {
+    const float d = p.sink[h] - m;
+    inv = d > 0.f ? expf(-d) / fmaf(l, expf(-d), 1.f) : 1.f / (l + expf(d));
+  }
+#pragma unroll
+  for (int i = 0; i < kLatAnyCols; ++i) {
+    const int c = tid + i * kLatAnyThreads;
+    if (c < p.rank) static_cast<T*>(p.out)[at + c] = from_f32<T>(acc[i] * inv);
+  }
+}
+
+template <typename T, int CW, int MT>
+int launch_latent_cfg(const LatentParams& p, cudaStream_t s) {
+  const int warps = (p.rank + CW - 1) / CW;
+  const int smem = LatCfg<CW, MT>::smem(warps);
+  if (ensure_dynamic_smem(reinterpret_cast<const void*>(latent_attn_mma_kernel<T, CW, MT>), LatCfg<CW, MT>::smem(8)) != cudaSuccess)
+    return -3;
+  const cudaError_t err = launch_pdl(latent_attn_mma_kernel<T, CW, MT>, dim3(p.splits, (p.heads + MT * 16 - 1) / (MT * 16), p.rows),
+                                     dim3(warps * 32), smem, s, p);
+  note_launch();
+  return err == cudaSuccess ? 0 : -4;
+}
+
+template <typename T, int CW>
+int launch_latent_mt(const LatentParams& p, cudaStream_t s) {
+  return p.heads > 16 ? launch_latent_cfg<T, CW, 2>(p, s) : launch_latent_cfg<T, CW, 1>(p, s);
+}
+
+}  // namespace
+
+void launch_latent_prologue(const void* y, int64_t ld, int tokens, int q_rank, int kv_rank, const float* q_w, const float* kv_w,
+                            float eps, void* cq, const int64_t* loc, void* cache, int64_t cache_ld, int64_t num_slots, DType dt,
+                            int* status, cudaStream_t s) {
+  if (tokens == 0) return;
+  MB200_DISPATCH_FLOAT(dt, (launch_pdl(latent_prologue_kernel<T>, dim3(tokens, kv_rank > 0 ? 2 : 1), dim3(128), 0, s,
+                                       static_cast<const T*>(y), ld, q_rank, kv_rank, q_w, kv_w, eps, static_cast<T*>(cq), loc,
+                                       static_cast<T*>(cache), cache_ld, num_slots, status)));
+  note_launch();
+}
+
+void launch_latent_gather(const void* cache, int64_t cache_ld, int rank, int elem_bytes, const int* rtt, int64_t rtt_stride,
+                          const int* req, const int* lens, const int* start, int batch, int max_len, void* out,
+                          int64_t num_slots, int* status, cudaStream_t s) {
+  if (batch == 0 || max_len == 0) return;
+  const dim3 grid(std::min((max_len + 7) / 8, 2048), batch), block(256);
+  const int row_bytes = rank * elem_bytes;
+  const int64_t ld_bytes = cache_ld * elem_bytes;
+  if (row_bytes % 16 == 0 && ld_bytes % 16 == 0) {
+    launch_pdl(latent_gather_kernel<uint4>, grid, block, 0, s, static_cast<const uint4*>(cache), ld_bytes / 16, row_bytes / 16, rtt,
+               rtt_stride, req, lens, start, static_cast<uint4*>(out), num_slots, status);
+  } else {
+    launch_pdl(latent_gather_kernel<uint16_t>, grid, block, 0, s, static_cast<const uint16_t*>(cache), ld_bytes / 2, row_bytes / 2,
+               rtt, rtt_stride, req, lens, start, static_cast<uint16_t*>(out), num_slots, status);
+  }
+  note_launch();
+}
+
+int launch_head_linear(const void* x, int64_t x_tok, int64_t x_head, const void* w, void* out, int64_t out_tok, int64_t out_head,
+                       int tokens, int heads, int N, int K, int num_sms, DType dt, cudaStream_t s) {
+  if (tokens == 0) return 0;
+  if (dt == kF32 || K % 8 != 0 || x_tok % 8 != 0 || x_head % 8 != 0) return -1;
+  const int groups = (tokens + kHlTokTiles * 8 - 1) / (kHlTokTiles * 8);
+  const bool split_k = static_cast<int64_t>(heads) * ((N + 63) / 64) * groups < num_sms && K >= 128;
+  MB200_DISPATCH_HALF(dt, {
+    if (split_k)
+      launch_pdl(head_linear_kernel<T, 4>, dim3((N + 15) / 16, heads, groups), dim3(128), 0, s, static_cast<const T*>(x), x_tok,
+                 x_head, static_cast<const T*>(w), static_cast<T*>(out), out_tok, out_head, tokens, N, K);
+    else
+      launch_pdl(head_linear_kernel<T, 1>, dim3((N + 63) / 64, heads, groups), dim3(128), 0, s, static_cast<const T*>(x), x_tok,
+                 x_head, static_cast<const T*>(w), static_cast<T*>(out), out_tok, out_head, tokens, N, K);
+  });
+  note_launch();
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+int latent_num_splits(int rows, int heads, int max_seq_len, int num_sms) {
+  const int ctas = std::max(1, rows * ((heads + 31) / 32));
+  const int tiles = std::max(1, (max_seq_len + kLatTok - 1) / kLatTok);
+  const int splits = std::min(2 * num_sms / ctas, std::max(1, tiles / 4));   // two CTAs fit an SM
+  return std::max(1, std::min(splits, 64));
+}
+
+bool latent_mma_covers(int rank, int64_t cache_ld, DType dt) {
+  return dt != kF32 && rank % 8 == 0 && rank <= 1024 && cache_ld % 8 == 0;
+}
+
+int launch_latent_attention(const LatentAttnArgs& a, cudaStream_t s) {
+  if (a.rows == 0) return 0;
+  if (a.rank > kLatAnyThreads * kLatAnyCols || a.splits < 1) return -1;
+  LatentParams p{};
+  p.q = a.q;
+  p.cache = a.cache;
+  p.out = a.out;
+  p.part_o = a.part_o;
+  p.part_lse = a.part_lse;
+  p.rtt = a.req_to_token;
+  p.row_req = a.row_req;
+  p.row_pos = a.row_pos;
+  p.sink = a.sink;
+  p.status = a.status;
+  p.rtt_stride = a.rtt_stride;
+  p.cache_ld = a.cache_ld;
+  p.num_slots = a.num_slots;
+  p.rows = a.rows;
+  p.heads = a.heads;
+  p.rank = a.rank;
+  p.splits = a.splits;
+  p.scale = a.scale;
+  if (!latent_mma_covers(a.rank, a.cache_ld, a.dt)) {
+    if (a.splits != 1) return -1;
+    MB200_DISPATCH_FLOAT(a.dt, (launch_pdl(latent_attn_any_kernel<T>, dim3(a.heads, a.rows), dim3(kLatAnyThreads), 0, s, p)));
+    note_launch();
+    return cudaGetLastError() == cudaSuccess ? 0 : -4;
+  }
+  int rc = 0;
+  MB200_DISPATCH_HALF(a.dt, (rc = a.rank <= 128   ? launch_latent_mt<T, 16>(p, s)
+                                  : a.rank <= 256 ? launch_latent_mt<T, 32>(p, s)
+                                  : a.rank <= 512 ? launch_latent_mt<T, 64>(p, s)
+                                                  : launch_latent_mt<T, 128>(p, s)));
+  if (rc != 0) return rc;
+  if (a.splits > 1) {
+    MB200_DISPATCH_HALF(a.dt, (launch_pdl(latent_merge_kernel<T>, dim3(a.heads, a.rows), dim3(128), 0, s, p)));
+    note_launch();
+  }
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+}  // namespace mb200

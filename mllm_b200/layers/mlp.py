@@ -1,4 +1,4 @@
-"""Gated MLP: fused gate/up projection with the SwiGLU folded into the GEMM epilogue, then the
+"""Gated MLP: fused gate/up projection with the gated activation (SwiGLU or GeGLU) folded into the GEMM epilogue, then the
 down projection (roles of pymllm/layers/mlp.py:58-231; the tensor-parallel form splits gate/up by
 columns and down by rows, one reduction per MLP)."""
 
@@ -14,7 +14,7 @@ from .linear import MergedLinear, RowParallelLinear
 
 class MLP(nn.Module):
     def __init__(self, hidden_size: int, intermediate_size: int, quant_config=None, prefix: str = "",
-                 params_dtype: Optional[torch.dtype] = None, reduce_results: bool = False) -> None:
+                 params_dtype: Optional[torch.dtype] = None, reduce_results: bool = False, activation: str = "silu") -> None:
         super().__init__()
 
         def qm(name):
@@ -24,6 +24,7 @@ class MLP(nn.Module):
                                          quant_method=qm("gate_up_proj"), params_dtype=params_dtype,
                                          prefix=f"{prefix}.gate_up_proj")
         self.gate_up_proj.swiglu_fused = True
+        self.gate_up_proj.gate_activation = activation        # silu | gelu_tanh
         self.down_proj = RowParallelLinear(intermediate_size, hidden_size, quant_method=qm("down_proj"),
                                            params_dtype=params_dtype, prefix=f"{prefix}.down_proj",
                                            reduce_results=reduce_results)

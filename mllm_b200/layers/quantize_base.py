@@ -45,8 +45,9 @@ class LinearMethodBase(QuantizeMethodBase):
         raise NotImplementedError
 
     def apply_swiglu(self, layer: nn.Module, x: torch.Tensor) -> torch.Tensor:
-        """Fused gate/up projection + SwiGLU; default = apply then activation."""
-        return ops.silu_and_mul(self.apply(layer, x))
+        """Fused gate/up projection + gated activation (``layer.gate_activation``, SiLU unless set); default =
+        apply then activation."""
+        return ops.act_and_mul(self.apply(layer, x), getattr(layer, "gate_activation", "silu"))
 
 
 class UnquantizedLinearMethod(LinearMethodBase):
@@ -73,6 +74,7 @@ class UnquantizedLinearMethod(LinearMethodBase):
         return ops.linear(x, layer.weight, bias, residual)
 
     def apply_swiglu(self, layer, x):
+        act = getattr(layer, "gate_activation", "silu")
         if getattr(layer, "_gate_up_interleaved", False):
-            return ops.linear_swiglu(x, layer.weight, ops.SWIGLU_BLOCK)
-        return ops.silu_and_mul(ops.linear(x, layer.weight))
+            return ops.linear_swiglu(x, layer.weight, ops.SWIGLU_BLOCK, act)
+        return ops.act_and_mul(ops.linear(x, layer.weight), act)

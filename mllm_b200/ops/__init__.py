@@ -112,6 +112,11 @@ def gelu_tanh_and_mul(x: torch.Tensor) -> torch.Tensor:
     return out.view(*x.shape[:-1], -1)
 
 
+def act_and_mul(x: torch.Tensor, act: str) -> torch.Tensor:
+    """``act(gate) * up`` over the two halves of the last dimension; ``act``: ``silu`` or ``gelu_tanh``."""
+    return gelu_tanh_and_mul(x) if act == "gelu_tanh" else silu_and_mul(x)
+
+
 def gelu_tanh(x: torch.Tensor) -> torch.Tensor:
     if not use_kernels(x) or x.numel() % 8:
         return ref.gelu_tanh(x)
@@ -130,12 +135,33 @@ def embedding(ids: torch.Tensor, table: torch.Tensor) -> torch.Tensor:
     return out.view(*ids.shape, table.shape[1])
 
 
+def embedding_f32(ids: torch.Tensor, table: torch.Tensor) -> torch.Tensor:
+    """Embedding rows widened to fp32: the start of a residual stream that is kept in 32-bit."""
+    if not use_kernels(table):
+        return ref.embedding(ids, table).float()
+    flat = ids.reshape(-1).to(torch.int64).contiguous()
+    out = torch.empty((flat.numel(), table.shape[1]), dtype=torch.float32, device=table.device)
+    ext().embedding_f32(flat, table, out)
+    return out.view(*ids.shape, table.shape[1])
+
+
+def residual_dyt(x: torch.Tensor, y: Optional[torch.Tensor], mult: float, alpha: torch.Tensor, weight: torch.Tensor,
+                 bias: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
+    """``x += mult * y`` in place (``x`` [T, W] fp32, ``y`` may be None), then the Dynamic Tanh norm of the new ``x``:
+    ``tanh(alpha * x) * weight + bias``, returned in ``dtype``."""
+    if not use_kernels(x):
+        return ref.residual_dyt(x, y, mult, alpha, weight, bias, dtype)
+    h = torch.empty(x.shape, dtype=dtype, device=x.device)
+    ext().residual_dyt(x, y, float(mult), alpha, weight, bias, h)
+    return h
+
+
 # --------------------------------------------------------------------------
 # GEMMs
 # --------------------------------------------------------------------------
 def _gemm(a, b, out, bias, residual, swiglu, a_scale, b_scale) -> None:
     # a Parameter is a model weight: nothing in the stream writes it, so the kernel may fetch it early
-    rc = ext().gemm(a, b, out, bias, residual, swiglu, a_scale, b_scale, isinstance(b, torch.nn.Parameter))
+    rc = ext().gemm(a, b, out, bias, residual, int(swiglu), a_scale, b_scale, isinstance(b, torch.nn.Parameter))
     if rc != 0:
         raise RuntimeError(f"mllm_b200 gemm: unsupported shape or launch failure (code {rc}) for "
                            f"M={a.shape[0]} N={b.shape[0]} K={a.shape[1]}")
@@ -238,9 +264,10 @@ def tp_rs_add_rmsnorm_ag(partial, residual: torch.Tensor, weight: torch.Tensor, 
 
 
 def _gemm_shape_ok(x2: torch.Tensor, weight: torch.Tensor) -> bool:
-    """The tcgen05 GEMM needs 16-byte aligned rows on every operand and the output."""
+    """The tcgen05 GEMM needs 16-byte aligned rows on every operand and the output, and a 16-bit type (32-bit products
+    are library calls)."""
     per16 = 16 // x2.element_size()
-    return weight.shape[0] % 8 == 0 and x2.shape[1] % per16 == 0 and weight.stride(0) % per16 == 0 and weight.stride(1) == 1
+    return x2.dtype != torch.float32 and weight.shape[0] % 8 == 0 and x2.shape[1] % per16 == 0 and weight.stride(0) % per16 == 0 and weight.stride(1) == 1
 
 
 SWIGLU_BLOCK = 128  # row interleave of fused gate/up weights expected by linear_swiglu
@@ -278,19 +305,20 @@ def linear(
     return o.view(*x.shape[:-1], weight.shape[0]) if out is None else out
 
 
-def linear_swiglu(x: torch.Tensor, weight: torch.Tensor, block: int = SWIGLU_BLOCK) -> torch.Tensor:
-    """``silu(x Wg^T) * (x Wu^T)`` in one GEMM; ``weight`` rows alternate ``block`` gate / ``block`` up rows."""
-    if not use_kernels(x) or block != SWIGLU_BLOCK or weight.shape[0] % 256:
-        return ref.linear_swiglu(x, weight, block)
+def linear_swiglu(x: torch.Tensor, weight: torch.Tensor, block: int = SWIGLU_BLOCK, act: str = "silu") -> torch.Tensor:
+    """``act(x Wg^T) * (x Wu^T)`` in one GEMM; ``weight`` rows alternate ``block`` gate / ``block`` up rows.
+    ``act``: ``silu`` or ``gelu_tanh``."""
     x2 = _2d(x)
+    if not use_kernels(x) or block != SWIGLU_BLOCK or weight.shape[0] % 256 or not _gemm_shape_ok(x2, weight):
+        return ref.linear_swiglu(x, weight, block, act)
     if x2.stride(-1) != 1 or (x2.stride(0) * x2.element_size()) % 16:
         x2 = x2.contiguous()
     o = torch.empty((x2.shape[0], weight.shape[0] // 2), dtype=x.dtype, device=x.device)
-    gate = _take_gate(x2, gated_ok=True)
+    gate = _take_gate(x2, gated_ok=act == "silu")
     if gate is not None:
         _gemm_tp(x2, weight, o, True, gate=gate)
     else:
-        _gemm(x2, weight, o, None, None, True, None, None)
+        _gemm(x2, weight, o, None, None, 2 if act == "gelu_tanh" else 1, None, None)
     return o.view(*x.shape[:-1], weight.shape[0] // 2)
 
 
@@ -597,18 +625,19 @@ def _attention_kernel_ok(q: torch.Tensor, k_cache: torch.Tensor, window, logit_c
 
 def attention_prefill(q, k_cache, v_cache, req_to_token, req_pool_indices, seq_lens, prefix_lens,
                       q_start_loc, scale: float, out=None, max_q_len: int = 0, window: Optional[int] = None,
-                      logit_cap: float = 0.0, seq_lens_cpu=None, prefix_lens_cpu=None) -> torch.Tensor:
+                      logit_cap: float = 0.0, seq_lens_cpu=None, prefix_lens_cpu=None, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of new tokens over cached prefix + themselves.  ``window``: sliding-window attention
     (each query sees its last ``window`` keys); ``logit_cap``: soft-capping of the scores; both are mask /
-    score options of the tcgen05 kernels.  Head sizes other than 64 / 128 / 256 and caches that hold neither the
+    score options of the tcgen05 kernels.  ``sink`` [Hq] fp32: ``exp(sink)`` joins each head's softmax denominator.
+    Head sizes other than 64 / 128 / 256 and caches that hold neither the
     activation dtype nor an 8-bit float take library / PyTorch fallbacks."""
     if _attention_kernel_ok(q, k_cache, window, logit_cap) and hasattr(ext(), "attention_prefill"):
         if out is None:
             out = torch.empty((q.shape[0], q.shape[1], q.shape[2]), dtype=q.dtype, device=q.device)
         ext().attention_prefill(q, k_cache, v_cache, req_to_token, req_pool_indices, seq_lens, prefix_lens,
-                                q_start_loc, scale, out, max_q_len, True, int(window or 0), float(logit_cap or 0.0))
+                                q_start_loc, scale, out, max_q_len, True, int(window or 0), float(logit_cap or 0.0), sink)
         return out
-    if q.is_cuda and not logit_cap:
+    if q.is_cuda and not logit_cap and sink is None:
         o = ref.attention_prefill_sdpa(q, k_cache, v_cache, req_to_token, req_pool_indices, seq_lens, prefix_lens,
                                        q_start_loc, scale, seq_lens_cpu, prefix_lens_cpu, window)
         if out is None:
@@ -616,22 +645,23 @@ def attention_prefill(q, k_cache, v_cache, req_to_token, req_pool_indices, seq_l
         out.copy_(o)
         return out
     return ref.attention_prefill(q, k_cache, v_cache, req_to_token, req_pool_indices, seq_lens, prefix_lens,
-                                 q_start_loc, scale, out, window=window, logit_cap=logit_cap)
+                                 q_start_loc, scale, out, window=window, logit_cap=logit_cap, sink=sink)
 
 
 def attention_decode(q, k_cache, v_cache, req_to_token, req_pool_indices, seq_lens, scale: float,
-                     out=None, max_seq_len: int = 0, window: Optional[int] = None, logit_cap: float = 0.0) -> torch.Tensor:
+                     out=None, max_seq_len: int = 0, window: Optional[int] = None, logit_cap: float = 0.0,
+                     sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     if _attention_kernel_ok(q, k_cache, window, logit_cap) and hasattr(ext(), "attention_decode"):
         if out is None:
             out = torch.empty((q.shape[0], q.shape[1], q.shape[2]), dtype=q.dtype, device=q.device)
         ext().attention_decode(q, k_cache, v_cache, req_to_token, req_pool_indices, seq_lens, scale, out, max_seq_len,
-                               int(window or 0), float(logit_cap or 0.0))
+                               int(window or 0), float(logit_cap or 0.0), sink)
         return out
-    if q.is_cuda and max_seq_len:
+    if q.is_cuda and max_seq_len and sink is None:
         return ref.attention_decode_batched(q, k_cache, v_cache, req_to_token, req_pool_indices, seq_lens, scale,
                                             max_seq_len, out, window, logit_cap)
     return ref.attention_decode(q, k_cache, v_cache, req_to_token, req_pool_indices, seq_lens, scale, out,
-                                window=window, logit_cap=logit_cap)
+                                window=window, logit_cap=logit_cap, sink=sink)
 
 
 def attention_varlen_bidirectional(q, k, v, cu_seqlens, scale: float) -> torch.Tensor:
@@ -720,34 +750,106 @@ def gelu_erf(x: torch.Tensor) -> torch.Tensor:
 
 
 # --------------------------------------------------------------------------
+# latent attention (one cached row per token, shared by all heads)
+# --------------------------------------------------------------------------
+def latent_prologue(y: torch.Tensor, q_weight: torch.Tensor, kv_weight: Optional[torch.Tensor], eps: float,
+                    loc: Optional[torch.Tensor] = None, cache: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """RMS norm (fp32) of the down projections' rows ``y = [query latent | cache latent]``: returns the normed query
+    latent [T, q_rank] and writes the normed cache latent to ``cache[loc]`` (``kv_weight`` None: the layer reads
+    another layer's latents and writes none)."""
+    if not use_kernels(y):
+        return ref.latent_prologue(y, q_weight, kv_weight, eps, loc, cache)
+    cq = torch.empty((y.shape[0], q_weight.numel()), dtype=y.dtype, device=y.device)
+    ext().latent_prologue(y, q_weight, kv_weight, eps, cq, None if loc is None else loc.to(torch.int64).contiguous(), cache)
+    return cq
+
+
+def latent_gather(cache, req_to_token, req, lens, start, total: int, max_len: int) -> torch.Tensor:
+    """[total, rank]: the latents of every request's context back to back (request b's rows begin at ``start[b]``)."""
+    if not use_kernels(cache):
+        return ref.latent_gather(cache, req_to_token, req, lens)
+    out = torch.empty((total, cache.shape[1]), dtype=cache.dtype, device=cache.device)
+    ext().latent_gather(cache, req_to_token, req, lens, start, max_len, out)
+    return out
+
+
+def head_linear(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
+    """``out[t, h] = weight[h] @ x[t, h]``: x [T, H, K], weight [H, N, K] -> [T, H, N]."""
+    if use_kernels(x) and x.dtype != torch.float32:
+        out = torch.empty((x.shape[0], x.shape[1], weight.shape[1]), dtype=x.dtype, device=x.device)
+        if x.shape[0] == 0 or ext().head_linear(x, weight, out) == 0:
+            return out
+    # 32-bit and unaligned sizes: a library batched product
+    return torch.bmm(x.transpose(0, 1), weight.transpose(1, 2)).transpose(0, 1).contiguous()
+
+
+_LATENT_ROWS = 32768     # query rows of one launch (they are a grid dimension)
+
+
+def latent_attention(q: torch.Tensor, cache: torch.Tensor, req_to_token, row_req, row_pos, scale: float,
+                     sink: Optional[torch.Tensor] = None, max_seq_len: int = 0) -> torch.Tensor:
+    """Attention of queries in the latent space over the cached latents, which are keys and values at once: row t is a
+    token of request ``row_req[t]`` at position ``row_pos[t]`` and sees the keys 0 .. its position.
+    q [rows, H, rank] -> [rows, H, rank]; ``sink`` [H] fp32 joins the denominator as ``exp(sink)``."""
+    if not use_kernels(q):
+        return ref.latent_attention(q, cache, req_to_token, row_req, row_pos, scale, sink)
+    q = q.contiguous()
+    out = torch.empty_like(q)
+    for r in range(0, q.shape[0], _LATENT_ROWS):
+        e = min(q.shape[0], r + _LATENT_ROWS)
+        ext().latent_attention(q[r:e], cache, req_to_token, row_req[r:e], row_pos[r:e], float(scale), sink, out[r:e], int(max_seq_len))
+    return out
+
+
+# --------------------------------------------------------------------------
 # gated delta net (linear attention of the hybrid models)
 # --------------------------------------------------------------------------
-def rmsnorm_gated(x: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float) -> torch.Tensor:
-    if use_kernels(x) and hasattr(ext(), "rmsnorm_gated") and x.shape[-1] % 8 == 0:
-        x2, g2 = _2d(x).contiguous(), _2d(gate).contiguous()
+def rmsnorm_gated(x: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, round_norm: bool = True) -> torch.Tensor:
+    """``weight * rmsnorm(x) * silu(gate)``, the norm taken over runs of ``weight.numel()`` features of the last
+    dimension.  ``gate`` may be a column slice of a wider matrix.  ``round_norm``: the normed value is rounded to the
+    tensors' type before it is multiplied."""
+    if use_kernels(x):
+        W = weight.numel()
+        x2 = x.reshape(-1, x.shape[-1])
+        g2 = gate if gate.dim() == 2 and gate.stride(-1) == 1 else gate.reshape(-1, gate.shape[-1]).contiguous()
+        if x2.shape[-1] % W:
+            raise ValueError("rmsnorm_gated: the last dimension must hold whole heads")
+        x2 = x2.contiguous()
         out = torch.empty_like(x2)
-        ext().rmsnorm_gated(x2, g2, weight, out, eps)
+        ext().rmsnorm_gated(x2, g2, weight, out, eps, round_norm)
         return out.view(x.shape)
-    return ref.rmsnorm_gated(x, gate, weight, eps)
+    return ref.rmsnorm_gated(x, gate, weight, eps, round_norm)
 
 
-def causal_conv1d_silu(x, weight, conv_state, state_indices, seq_lens, has_state, q_start=None) -> torch.Tensor:
+def causal_conv1d_silu(x, weight, conv_state, state_indices, seq_lens, has_state, q_start=None, max_len: int = 0) -> torch.Tensor:
     """Depth-wise causal conv (kernel K) + SiLU over the new tokens of every request, reading / updating
     the per-request history rows of ``conv_state``.  ``seq_lens`` / ``has_state`` may be host lists (CPU
-    path) or device int32 tensors (GPU path, no host sync; ``q_start`` = first row of each request)."""
-    if use_kernels(x) and hasattr(ext(), "gdn_conv1d_silu"):
+    path) or device int32 tensors (GPU path, no host sync; ``q_start`` = first row of each request).  ``x`` may be a
+    column slice of a wider matrix; ``max_len``: the longest run of new tokens, when the host knows it."""
+    if use_kernels(x):
         dev = x.device
         lens = seq_lens if isinstance(seq_lens, torch.Tensor) else torch.tensor(list(seq_lens), dtype=torch.int32, device=dev)
         has = has_state if isinstance(has_state, torch.Tensor) else torch.tensor([int(h) for h in has_state], dtype=torch.int32, device=dev)
         if q_start is None:
             q_start = torch.cumsum(lens, 0, dtype=torch.int32) - lens
-        out = torch.empty_like(x)
-        ext().gdn_conv1d_silu(x.contiguous(), weight.contiguous(), conv_state, state_indices.to(torch.int32), lens.to(torch.int32),
-                              has.to(torch.int32), q_start.to(torch.int32), out)
+        out = torch.empty(x.shape, dtype=x.dtype, device=dev)
+        ext().gdn_conv1d_silu(x if x.stride(-1) == 1 else x.contiguous(), weight.contiguous(), conv_state,
+                              state_indices.to(torch.int32), lens.to(torch.int32), has.to(torch.int32), q_start.to(torch.int32),
+                              out, int(max_len))
         return out
     lens = seq_lens.tolist() if isinstance(seq_lens, torch.Tensor) else seq_lens
     has = has_state.tolist() if isinstance(has_state, torch.Tensor) else has_state
     return ref.causal_conv1d_silu(x, weight, conv_state, state_indices, lens, has)
+
+
+def gdn_gates(b: torch.Tensor, a: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor) -> Tuple[torch.Tensor, torch.Tensor]:
+    """``(g, beta)`` fp32 [T, H]: log decay ``-exp(a_log) * softplus(a + dt_bias)`` and step size ``sigmoid(b)``."""
+    if not use_kernels(b):
+        return ref.gdn_gates(b, a, a_log, dt_bias)
+    g = torch.empty(b.shape, dtype=torch.float32, device=b.device)
+    beta = torch.empty_like(g)
+    ext().gdn_gates(b, a, a_log, dt_bias, g, beta)
+    return g, beta
 
 
 _GDN_EXTEND_BACKEND = "auto"
@@ -762,23 +864,47 @@ def set_gdn_extend_backend(name: str) -> None:
     _GDN_EXTEND_BACKEND = str(name)
 
 
-def gated_delta_rule(q, k, v, g, beta, state, state_indices, seq_lens, has_state, q_start=None) -> torch.Tensor:
+_GDN_MAX_DK = 512       # key features the sequential kernel holds
+
+
+def _heads_like(t: torch.Tensor, heads: int) -> torch.Tensor:
+    return t if t.shape[1] == heads else t.repeat_interleave(heads // t.shape[1], dim=1)
+
+
+def gated_delta_rule(q, k, v, g, beta, state, state_indices, seq_lens, has_state, q_start=None, raw_gates=None,
+                     split_tf32: bool = False) -> torch.Tensor:
     """Gated delta rule over ragged sequences with per-request recurrent state (read when ``has_state``,
-    always written back).  q, k [T, H, Dk], v [T, H, Dv], g / beta [T, H] fp32."""
-    if (use_kernels(q) and hasattr(ext(), "gdn_recurrent") and q.shape[-1] == 128 and v.shape[-1] == 128
-            and _GDN_EXTEND_BACKEND != "pytorch"):
+    always written back).  q, k [T, Hk, Dk] (Hk divides H: value head h uses head ``h // (H / Hk)``), v [T, H, Dv],
+    g / beta [T, H] fp32; ``raw_gates = (b, a, a_log, dt_bias)`` instead of g and beta lets the kernel form them.
+    Tokens may be rows of wider matrices (heads of a token contiguous).  ``split_tf32``: the chunk-parallel kernel
+    carries its fp32 operands as two tf32 terms instead of one."""
+    H = v.shape[1]
+    if use_kernels(q) and q.shape[-1] <= _GDN_MAX_DK and _GDN_EXTEND_BACKEND != "pytorch":
         dev = q.device
         lens = seq_lens if isinstance(seq_lens, torch.Tensor) else torch.tensor(list(seq_lens), dtype=torch.int32, device=dev)
         has = has_state if isinstance(has_state, torch.Tensor) else torch.tensor([int(h) for h in has_state], dtype=torch.int32, device=dev)
         if q_start is None:
             q_start = torch.cumsum(lens, 0, dtype=torch.int32) - lens
-        out = torch.empty_like(v)
+        out = torch.empty((v.shape[0], H, v.shape[2]), dtype=v.dtype, device=dev)
+        meta = (state, state_indices.to(torch.int32), lens.to(torch.int32), has.to(torch.int32), q_start.to(torch.int32), out)
+        q, k, v = (t if t.stride(2) == 1 and t.stride(1) == t.shape[2] else t.contiguous() for t in (q, k, v))
         chunked = _GDN_EXTEND_BACKEND == "cuda_chunkwise" or (
             _GDN_EXTEND_BACKEND != "mllm_kernel" and q.shape[0] >= 32 * max(1, lens.numel()))
-        rule = ext().gdn_chunk if chunked and hasattr(ext(), "gdn_chunk") else ext().gdn_recurrent
-        rule(q.contiguous(), k.contiguous(), v.contiguous(), g.float().contiguous(), beta.float().contiguous(),
-             state, state_indices.to(torch.int32), lens.to(torch.int32), has.to(torch.int32), q_start.to(torch.int32), out)
+        if chunked and q.dtype != torch.float32:
+            if raw_gates is not None:
+                g, beta = gdn_gates(*raw_gates)
+                raw_gates = None
+            g, beta = g.float().contiguous(), beta.float().contiguous()
+            if ext().gdn_chunk(q, k, v, g, beta, *meta, split_tf32) == 0:
+                return out
+        if raw_gates is not None:
+            ext().gdn_recurrent_raw(q, k, v, *raw_gates, *meta)
+        else:
+            ext().gdn_recurrent(q, k, v, g.float().contiguous(), beta.float().contiguous(), *meta)
         return out
+    if raw_gates is not None:
+        g, beta = ref.gdn_gates(*raw_gates)
+    q, k = _heads_like(q, H), _heads_like(k, H)
     lens = seq_lens.tolist() if isinstance(seq_lens, torch.Tensor) else seq_lens
     has = has_state.tolist() if isinstance(has_state, torch.Tensor) else has_state
     if max(lens, default=0) > 16:  # prefill: the chunk-parallel form (matrix products) instead of a token loop

@@ -118,15 +118,15 @@ def interleave_gate_up(w: torch.Tensor, block: int) -> torch.Tensor:
     return torch.cat([g, u], dim=1).reshape(w.shape)
 
 
-def linear_swiglu(x: torch.Tensor, weight: torch.Tensor, block: int = 0) -> torch.Tensor:
-    """``silu(x Wg^T) * (x Wu^T)``; ``block`` = row interleave of ``weight`` (0: ``[gate ; up]``)."""
+def linear_swiglu(x: torch.Tensor, weight: torch.Tensor, block: int = 0, act: str = "silu") -> torch.Tensor:
+    """``act(x Wg^T) * (x Wu^T)``; ``block`` = row interleave of ``weight`` (0: ``[gate ; up]``)."""
     y = _f32(x) @ _f32(weight).t()
     if block:
         g, u = deinterleave_gate_up(y, block)
     else:
         d = y.shape[-1] // 2
         g, u = y[..., :d], y[..., d:]
-    return (F.silu(g) * u).to(x.dtype)
+    return ((F.gelu(g, approximate="tanh") if act == "gelu_tanh" else F.silu(g)) * u).to(x.dtype)
 
 
 def per_token_quant_int8(x: torch.Tensor) -> Tuple[torch.Tensor, torch.Tensor]:
@@ -273,10 +273,10 @@ def create_kv_indices(req_to_token: torch.Tensor, req_pool_indices: torch.Tensor
 # --------------------------------------------------------------------------
 # attention over the slot-indexed KV pool
 # --------------------------------------------------------------------------
-def _attend(q, k, v, scale, causal_offset: Optional[int], window: Optional[int] = None, logit_cap: float = 0.0):
+def _attend(q, k, v, scale, causal_offset: Optional[int], window: Optional[int] = None, logit_cap: float = 0.0, sink=None):
     """q [Tq,Hq,D] k,v [Tk,Hkv,D] fp32 -> [Tq,Hq,D]; key j visible to query i iff j <= i + causal_offset and,
     with a sliding ``window``, j > i + causal_offset - window (the last ``window`` keys, the query's own
-    included).  ``logit_cap`` > 0 soft-caps the scaled scores: ``cap * tanh(s / cap)``."""
+    included).  ``sink`` [Hq]: one more softmax term per head, without a value.  ``logit_cap`` > 0 soft-caps the scaled scores: ``cap * tanh(s / cap)``."""
     Hq, Hkv = q.shape[1], k.shape[1]
     g = Hq // Hkv
     kk = k.repeat_interleave(g, dim=1)
@@ -292,7 +292,7 @@ def _attend(q, k, v, scale, causal_offset: Optional[int], window: Optional[int] 
         if window:
             hidden = hidden | (j <= i + off - int(window))
         s = s.masked_fill(hidden, float("-inf"))
-    p = torch.softmax(s, dim=-1)
+    p = sink_softmax(s, sink)
     return torch.einsum("hqk,khd->qhd", p, vv)
 
 
@@ -322,7 +322,7 @@ def attention_prefill(
     q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, req_to_token: torch.Tensor,
     req_pool_indices: torch.Tensor, seq_lens: torch.Tensor, prefix_lens: torch.Tensor,
     q_start_loc: torch.Tensor, scale: float, out: Optional[torch.Tensor] = None, max_q_len: int = 0,
-    window: Optional[int] = None, logit_cap: float = 0.0,
+    window: Optional[int] = None, logit_cap: float = 0.0, sink: Optional[torch.Tensor] = None,
 ) -> torch.Tensor:
     """Causal attention of each request's new tokens over its cached prefix plus itself.
 
@@ -334,7 +334,7 @@ def attention_prefill(
         sl, pl, qs = int(seq_lens[b]), int(prefix_lens[b]), int(q_start_loc[b])
         n = sl - pl
         slots = req_to_token[int(req_pool_indices[b]), :sl].long()
-        o = _attend(_f32(q[qs : qs + n]), _f32(k_cache[slots]), _f32(v_cache[slots]), scale, pl, window, logit_cap)
+        o = _attend(_f32(q[qs : qs + n]), _f32(k_cache[slots]), _f32(v_cache[slots]), scale, pl, window, logit_cap, sink)
         out[qs : qs + n] = o.to(out.dtype)
     return out
 
@@ -360,14 +360,14 @@ def attention_prefill_sdpa(q, k_cache, v_cache, req_to_token, req_pool_indices, 
 def attention_decode(
     q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, req_to_token: torch.Tensor,
     req_pool_indices: torch.Tensor, seq_lens: torch.Tensor, scale: float, out: Optional[torch.Tensor] = None,
-    window: Optional[int] = None, logit_cap: float = 0.0,
+    window: Optional[int] = None, logit_cap: float = 0.0, sink: Optional[torch.Tensor] = None,
 ) -> torch.Tensor:
     """One query token per request over ``req_to_token[req, :seq_len]`` (the new token's K/V included)."""
     out = torch.empty_like(q) if out is None else out
     for b in range(req_pool_indices.numel()):
         sl = int(seq_lens[b])
         slots = req_to_token[int(req_pool_indices[b]), :sl].long()
-        o = _attend(_f32(q[b : b + 1]), _f32(k_cache[slots]), _f32(v_cache[slots]), scale, None, window, logit_cap)
+        o = _attend(_f32(q[b : b + 1]), _f32(k_cache[slots]), _f32(v_cache[slots]), scale, None, window, logit_cap, sink)
         out[b] = o[0].to(out.dtype)
     return out
 
@@ -506,13 +506,63 @@ def moe_experts(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_w: to
 
 
 # --------------------------------------------------------------------------
+# fp32 residual stream, Dynamic Tanh, latent attention
+# --------------------------------------------------------------------------
+def residual_dyt(x, y, mult, alpha, weight, bias, dtype):
+    if y is not None:
+        x.add_(_f32(y), alpha=float(mult))
+    return (torch.tanh(_f32(alpha) * x) * _f32(weight) + _f32(bias)).to(dtype)
+
+
+def latent_prologue(y, q_weight, kv_weight, eps, loc=None, cache=None):
+    def norm(t, w):
+        t = _f32(t)
+        return (t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps) * _f32(w)).to(y.dtype)
+
+    nq = q_weight.numel()
+    if kv_weight is not None:
+        cache[loc.long()] = norm(y[:, nq:nq + kv_weight.numel()], kv_weight)
+    return norm(y[:, :nq], q_weight)
+
+
+def latent_gather(cache, req_to_token, req, lens):
+    return torch.cat([cache[req_to_token[int(r), : int(n)].long()] for r, n in zip(req, lens)]) if len(req) else cache[:0]
+
+
+def latent_attention(q, cache, req_to_token, row_req, row_pos, scale, sink=None):
+    out = torch.empty_like(q)
+    for t in range(q.shape[0]):
+        c = _f32(cache[req_to_token[int(row_req[t]), : int(row_pos[t]) + 1].long()])      # [n, rank]
+        s = (_f32(q[t]) @ c.t()) * scale                                                  # [H, n]
+        p = sink_softmax(s, sink)
+        out[t] = (p @ c).to(q.dtype)
+    return out
+
+
+def sink_softmax(scores: torch.Tensor, sink: Optional[torch.Tensor]) -> torch.Tensor:
+    """Softmax over the last dimension of ``scores`` [H, ...]; a head's sink is one more term of the denominator."""
+    if sink is None:
+        return torch.softmax(scores, dim=-1)
+    extra = _f32(sink).view(-1, *([1] * (scores.dim() - 1))).expand(*scores.shape[:-1], 1)
+    return torch.softmax(torch.cat([scores, extra], dim=-1), dim=-1)[..., :-1]
+
+
+# --------------------------------------------------------------------------
 # gated delta net (linear attention of the Qwen3.5 hybrid models)
 # --------------------------------------------------------------------------
-def rmsnorm_gated(x: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float) -> torch.Tensor:
-    """``weight * round(rmsnorm(x)) * silu(gate)`` over the last dimension (norm before gate)."""
-    xf = _f32(x)
-    n = (xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps)).to(x.dtype)
-    return (_f32(weight) * _f32(n) * F.silu(_f32(gate))).to(x.dtype)
+def rmsnorm_gated(x: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, round_norm: bool = True) -> torch.Tensor:
+    """``weight * rmsnorm(x) * silu(gate)`` over runs of ``weight.numel()`` features (norm before gate; the normed
+    value is rounded to x's type first when ``round_norm``)."""
+    xf = _f32(x).reshape(*x.shape[:-1], -1, weight.numel())
+    n = xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps)
+    if round_norm:
+        n = _f32(n.to(x.dtype))
+    return ((_f32(weight) * n).reshape(x.shape) * F.silu(_f32(gate))).to(x.dtype)
+
+
+def gdn_gates(b, a, a_log, dt_bias):
+    g = -torch.exp(_f32(a_log)) * F.softplus(_f32(a) + _f32(dt_bias))
+    return g, torch.sigmoid(_f32(b))
 
 
 def causal_conv1d_silu(x: torch.Tensor, weight: torch.Tensor, conv_state: torch.Tensor, state_indices: torch.Tensor,
@@ -532,7 +582,7 @@ def causal_conv1d_silu(x: torch.Tensor, weight: torch.Tensor, conv_state: torch.
         seq = torch.cat([hist, _f32(x[off:off + n]).t()], dim=1)          # [C, K-1+n]
         y = F.conv1d(seq.unsqueeze(0), _f32(weight).unsqueeze(1), None, groups=weight.shape[0]).squeeze(0)  # [C, n]
         out[off:off + n] = F.silu(y).t().to(x.dtype)
-        conv_state[slot] = seq[:, -(K - 1):].to(conv_state.dtype)
+        conv_state[slot] = seq[:, seq.shape[1] - (K - 1):].to(conv_state.dtype)
         off += n
     return out
 

@@ -40,6 +40,7 @@ class ServerConfig:
     # -- scheduling / memory -------------------------------------------------
     mem_fraction_static: Optional[float] = None
     max_running_requests: Optional[int] = 1
+    spare_request_slots: int = 8      # request-table (and state) rows beyond max_running_requests, for prompts being prefilled
     max_queued_requests: Optional[int] = None
     max_total_tokens: Optional[int] = None
     chunked_prefill_size: Optional[int] = None
@@ -139,6 +140,7 @@ class ServerConfig:
             self.max_running_requests is None or self.max_running_requests > 0,
             "`max_running_requests` must be > 0 when set.",
         )
+        need(self.spare_request_slots >= 0, "`spare_request_slots` must be >= 0.")
         need(
             self.max_queued_requests is None or self.max_queued_requests >= 0,
             "`max_queued_requests` must be >= 0 when set.",

@@ -48,6 +48,8 @@ class ForwardBatch:
     extend_seq_lens_cpu: Optional[List[int]] = None
     extend_prefix_lens_cpu: Optional[List[int]] = None
     max_extend_len: int = 0
+    # rows of input_ids whose logits are wanted (None: the last row of each request)
+    logit_rows: Optional[torch.Tensor] = None
     # multimodal
     mrope_positions: Optional[torch.Tensor] = None      # [3, T]
     mrope_position_deltas: Optional[torch.Tensor] = None
@@ -65,3 +67,11 @@ class ForwardBatch:
     llm_decode_ms: Optional[float] = None
     benchmark_vision_timing: bool = False
     extra: dict = field(default_factory=dict)
+
+    def logit_row_index(self) -> Optional[torch.Tensor]:
+        """Rows whose logits the pass returns; None when it is every row."""
+        if self.logit_rows is not None:
+            return self.logit_rows
+        if self.forward_mode.is_extend() and self.extend_seq_lens is not None:
+            return torch.cumsum(self.extend_seq_lens, 0) - 1
+        return None

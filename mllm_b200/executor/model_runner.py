@@ -28,7 +28,7 @@ from .. import ops
 from ..configs import ServerConfig
 from ..engine.forward_batch import ForwardBatch, ForwardMode
 from ..mem_cache import KVPool, ReqToTokenPool, TokenToKVPoolAllocator
-from ..models import get_model_class
+from ..models import get_config_adapter, get_model_class
 from ..models.qwen3 import LogitsProcessorOutput
 from ..parallel import state as pstate
 
@@ -99,6 +99,12 @@ def load_hf_config(model_path) -> Any:
 
         return get_preset(s.split(":", 1)[1])
     cfg_file = Path(s) / "config.json"
+    if cfg_file.exists():
+        with open(cfg_file) as f:
+            raw = json.load(f)
+        adapt = get_config_adapter(raw)
+        if adapt is not None:
+            return adapt(raw)
     try:
         from transformers import AutoConfig
 
@@ -155,6 +161,8 @@ class ModelRunner:
         if self.hf_config is None:
             self.hf_config = load_hf_config(self.server_config.model_path)
         self.dtype = self._resolve_dtype()
+        if self.dtype == torch.float32:
+            torch.set_float32_matmul_precision("highest")     # no reduced-precision mode in a 32-bit run
         self._pre_load_avail_gib = get_available_gpu_memory(self.device.type, self.gpu_id)
         self.load_model()
         self._extract_model_metadata()
@@ -190,7 +198,8 @@ class ModelRunner:
     def _num_req_slots(self) -> int:
         """Rows of the request table: the running batch plus a few spare rows for requests being prefilled
         while it is full."""
-        return max(int(self.server_config.max_running_requests or 1), 1) + 8
+        spare = getattr(self.server_config, "spare_request_slots", 8)
+        return max(int(self.server_config.max_running_requests or 1), 1) + max(0, int(spare))
 
     def _tp_rendezvous(self) -> None:
         if pstate.get_tensor_model_parallel_world_size() > 1:
@@ -307,6 +316,7 @@ class ModelRunner:
         # layers under pipeline parallelism
         self.kv_layer_offset = 0
         self.num_kv_layers = int(getattr(self.model, "kv_layers", 0) or tc.num_hidden_layers)
+        self.own_kv_pool = hasattr(self.model, "make_kv_pool")     # the model's cache is not K and V rows per head
         if pstate.get_pipeline_parallel_world_size() > 1:
             if hasattr(self.model, "kv_layers") or not hasattr(getattr(self.model, "model", None), "pp_layers"):
                 raise NotImplementedError(f"{type(self.model).__name__} does not support pipeline parallelism")
@@ -406,6 +416,8 @@ class ModelRunner:
                 p.data.copy_((torch.rand(p.shape, device=self.device, generator=gen) * 0.5 + 0.75).mul_(std / 64).to(p.dtype))
             elif name.endswith("norm.weight") or ".norm" in name and name.endswith(".weight") and p.dim() == 1:
                 p.data.fill_(1.0)
+            elif name.endswith(".alpha"):
+                continue                                  # Dynamic Tanh slope: keep the initial value
             elif name.endswith(".bias"):
                 p.data.zero_()
             else:
@@ -454,6 +466,8 @@ class ModelRunner:
 
     # ------------------------------------------------------------------ memory
     def cell_bytes(self) -> int:
+        if self.own_kv_pool:
+            return max(1, int(self.model.kv_cell_bytes(self.kv_cache_dtype)))
         return KVPool.cell_bytes(self.num_kv_layers, self.num_kv_heads, self.head_dim, self.kv_cache_dtype)
 
     def _profile_max_num_tokens(self) -> MemoryProfileResult:
@@ -482,8 +496,11 @@ class ModelRunner:
         self.max_total_num_tokens = tokens
         self.max_running_requests = max(int(self.server_config.max_running_requests or 1), 1)
         self.req_to_token_pool = ReqToTokenPool(self._num_req_slots(), self.context_len + 4, self.device)
-        self.token_to_kv_pool = KVPool(tokens, self.num_kv_layers, self.num_kv_heads, self.head_dim,
-                                       self.kv_cache_dtype, self.device, page_size=page, layer_offset=self.kv_layer_offset)
+        if self.own_kv_pool:
+            self.token_to_kv_pool = self.model.make_kv_pool(tokens, self.kv_cache_dtype, self.device, page)
+        else:
+            self.token_to_kv_pool = KVPool(tokens, self.num_kv_layers, self.num_kv_heads, self.head_dim,
+                                           self.kv_cache_dtype, self.device, page_size=page, layer_offset=self.kv_layer_offset)
         self.token_to_kv_pool_allocator = TokenToKVPoolAllocator(tokens, page_size=page, device=self.device)
         logger.info("KV pool: %d tokens, %.2f GiB (%d B/token)", tokens, tokens * prof.cell_bytes / (1 << 30),
                     prof.cell_bytes)
@@ -493,7 +510,7 @@ class ModelRunner:
             return
         if pstate.get_pipeline_parallel_world_size() > 1:
             return      # stages exchange activations with point-to-point calls between the layers: eager only
-        if self.kv_cache_dtype != self.dtype and not ops.attention_kernels_cover(self.head_dim, self.kv_cache_dtype, self.dtype):
+        if not self.own_kv_pool and self.kv_cache_dtype != self.dtype and not ops.attention_kernels_cover(self.head_dim, self.kv_cache_dtype, self.dtype):
             return      # 8-bit cache off the kernels: attention runs on paths that are not captured
         from .cuda_graph_runner import CudaGraphRunner
 

@@ -1,4 +1,4 @@
-"""Gated DeltaNet token mixer of the Qwen3.5 hybrid models (roles of pymllm/layers/gated_delta_net.py,
+"""Gated DeltaNet token mixers.  :class:`GatedDeltaNet` is that of the Qwen3.5 hybrid models (roles of pymllm/layers/gated_delta_net.py,
 layers/attention/gdn_backend.py and rms_norm_gated.py; math of HF ``Qwen3_5GatedDeltaNet``):
 
     qkv = conv1d_silu(in_proj_qkv(x))      depth-wise causal conv over the last 4 inputs, SiLU
@@ -8,10 +8,14 @@ layers/attention/gdn_backend.py and rms_norm_gated.py; math of HF ``Qwen3_5Gated
 
 State (recurrent matrix and conv history) lives in a :class:`GDNPool` row per request, so prefill of a
 continuation (chunked prefill) and decode both resume from it.
+
+:class:`FusedGatedDeltaNet` is the same rule for models that give its sizes per layer: one projection for everything
+that is taken of the layer input, gates formed inside the rule's kernel, 32-bit products in the recurrence.
 """
 
 from __future__ import annotations
 
+from dataclasses import dataclass
 from typing import Optional
 
 import torch
@@ -19,6 +23,32 @@ from torch import nn
 
 from .. import ops
 from ..parallel import state as pstate
+
+
+@dataclass
+class GdnBatch:
+    """What the delta-net kernels need to know about a batch, shared by all layers of a forward pass."""
+
+    slots: torch.Tensor       # [B] state row of each request
+    lens: torch.Tensor        # [B] new tokens
+    has_state: torch.Tensor   # [B] 1 where earlier tokens left a state
+    q_start: Optional[torch.Tensor]   # [B] first row of each request
+    max_len: int              # longest run of new tokens (0: not known on the host)
+
+
+def gdn_batch(fb) -> GdnBatch:
+    got = fb.extra.get("gdn_batch")
+    if got is None:
+        slots = fb.req_pool_indices.to(torch.int32)
+        if fb.forward_mode.is_decode():
+            ones = torch.ones(fb.batch_size, dtype=torch.int32, device=slots.device)
+            got = GdnBatch(slots, ones, ones, torch.arange(fb.batch_size, dtype=torch.int32, device=slots.device), 1)
+        else:
+            start = fb.extend_start_loc
+            got = GdnBatch(slots, fb.extend_seq_lens.to(torch.int32), (fb.extend_prefix_lens > 0).to(torch.int32),
+                           None if start is None else start.to(torch.int32), int(fb.max_extend_len or 0))
+        fb.extra["gdn_batch"] = got
+    return got
 
 
 class GatedDeltaNet(nn.Module):
@@ -89,33 +119,21 @@ class GatedDeltaNet(nn.Module):
         pool = fb.extra["gdn_pool"]
         recurrent, conv = pool.layer(self.gdn_index)
         T = x.shape[0]
-        slots = fb.req_pool_indices
-        if fb.forward_mode.is_decode():
-            lens = fb.extra.get("gdn_ones")
-            if lens is None:
-                lens = torch.ones(fb.batch_size, dtype=torch.int32, device=x.device)
-                fb.extra["gdn_ones"] = lens
-            has, q_start = lens, torch.arange(fb.batch_size, dtype=torch.int32, device=x.device)
-        else:
-            lens = fb.extend_seq_lens.to(torch.int32)
-            has = (fb.extend_prefix_lens > 0).to(torch.int32)
-            q_start = fb.extend_start_loc.to(torch.int32) if fb.extend_start_loc is not None else None
+        m = gdn_batch(fb)
         qkv = ops.linear(x, self.in_proj_qkv.weight)
         z = ops.linear(x, self.in_proj_z.weight)
         ba = ops.linear(x, torch.cat([self.in_proj_b.weight, self.in_proj_a.weight], 0)) if not hasattr(self, "_ba") else \
             ops.linear(x, self._ba)
         b, a = ba[:, : self.num_v_heads], ba[:, self.num_v_heads:]
-        qkv = ops.causal_conv1d_silu(qkv, self.conv1d.weight, conv, slots, lens, has, q_start)
+        qkv = ops.causal_conv1d_silu(qkv, self.conv1d.weight, conv, m.slots, m.lens, m.has_state, m.q_start, m.max_len)
         q, k, v = torch.split(qkv, [self.key_dim, self.key_dim, self.value_dim], dim=-1)
-        q = q.reshape(T, self.num_k_heads, self.head_k_dim)
-        k = k.reshape(T, self.num_k_heads, self.head_k_dim)
-        v = v.reshape(T, self.num_v_heads, self.head_v_dim)
-        rep = self.num_v_heads // self.num_k_heads
-        if rep > 1:
-            q, k = q.repeat_interleave(rep, dim=1), k.repeat_interleave(rep, dim=1)
+        # views of the convolution's rows; value head h uses query / key head h // (value heads / key heads)
+        q = q.unflatten(1, (self.num_k_heads, self.head_k_dim))
+        k = k.unflatten(1, (self.num_k_heads, self.head_k_dim))
+        v = v.unflatten(1, (self.num_v_heads, self.head_v_dim))
         beta = torch.sigmoid(b.float())
         g = -torch.exp(self.A_log.float()) * torch.nn.functional.softplus(a.float() + self.dt_bias.float())
-        o = ops.gated_delta_rule(q, k, v, g, beta, recurrent, slots, lens, has, q_start)
+        o = ops.gated_delta_rule(q, k, v, g, beta, recurrent, m.slots, m.lens, m.has_state, m.q_start)
         o = ops.rmsnorm_gated(o.reshape(-1, self.head_v_dim), z.reshape(-1, self.head_v_dim), self.norm.weight, self.eps)
         y = ops.linear(o.reshape(T, self.value_dim), self.out_proj.weight)
         return pstate.tensor_model_parallel_all_reduce(y) if self.tp > 1 else y
@@ -123,3 +141,67 @@ class GatedDeltaNet(nn.Module):
     def fuse_small_projections(self) -> None:
         """One GEMM for the beta / decay projections (call after loading)."""
         self._ba = torch.cat([self.in_proj_b.weight.data, self.in_proj_a.weight.data], 0).contiguous()
+
+
+class FusedGatedDeltaNet(nn.Module):
+    """One delta-net mixer with its own sizes.  The projections of the layer input are the row blocks
+    ``[q | k | v | gate | b | a]`` of one matrix (zero rows up to a multiple of 8); q and k have ``kv_heads`` heads and
+    value head ``h`` uses head ``h // (heads / kv_heads)``.  Unit norms, gates and the recurrence are fp32."""
+
+    def __init__(self, hidden_size: int, heads: int, kv_heads: int, dim: int, vdim: int, conv: int, eps: float, gdn_index: int,
+                 params_dtype: torch.dtype) -> None:
+        super().__init__()
+        if heads % kv_heads:
+            raise ValueError(f"delta net: {heads} value heads over {kv_heads} key heads")
+        self.heads, self.kv_heads, self.dim, self.vdim, self.conv_kernel = heads, kv_heads, dim, vdim, conv
+        self.eps, self.gdn_index = eps, gdn_index
+        self.key_dim, self.value_dim = kv_heads * dim, heads * vdim
+        self.conv_dim = 2 * self.key_dim + self.value_dim
+        self.shards = {"q": self.key_dim, "k": self.key_dim, "v": self.value_dim, "g": self.value_dim, "b": heads, "a": heads}
+        self.offset, rows = {}, 0
+        for name, n in self.shards.items():
+            self.offset[name] = rows
+            rows += n
+
+        def p(*shape, dtype=params_dtype):
+            return nn.Parameter(torch.zeros(*shape, dtype=dtype), requires_grad=False)
+
+        self.in_proj = nn.Module()
+        self.in_proj.weight = p(-(-rows // 8) * 8, hidden_size)
+        self.conv1d = nn.Module()
+        self.conv1d.weight = p(self.conv_dim, conv)
+        self.A_log = p(heads, dtype=torch.float32)
+        self.dt_bias = p(heads, dtype=torch.float32)
+        self.norm = nn.Module()
+        self.norm.weight = nn.Parameter(torch.ones(vdim, dtype=params_dtype), requires_grad=False)
+        self.out_proj = nn.Module()
+        self.out_proj.weight = p(hidden_size, self.value_dim)
+
+    @property
+    def state_shape(self):
+        """(value heads, key features, value features, convolution channels, taps) of a request's state."""
+        return self.heads, self.dim, self.vdim, self.conv_dim, self.conv_kernel
+
+    def load_projection(self, name: str, full: torch.Tensor) -> None:
+        o = self.offset[name]
+        self.in_proj.weight.data[o:o + self.shards[name]].copy_(full)
+
+    def load_conv(self, name: str, full: torch.Tensor) -> None:
+        o = self.offset[name]
+        self.conv1d.weight.data[o:o + self.shards[name]].copy_(full.reshape(self.shards[name], self.conv_kernel))
+
+    def forward(self, x: torch.Tensor, fb) -> torch.Tensor:
+        recurrent, conv = fb.extra["gdn_pool"].layer(self.gdn_index)
+        m = gdn_batch(fb)
+        o, C = self.offset, self.conv_dim
+        y = ops.linear(x, self.in_proj.weight)
+        qkv = ops.causal_conv1d_silu(y[:, :C], self.conv1d.weight, conv, m.slots, m.lens, m.has_state, m.q_start, m.max_len)
+        q = qkv[:, : o["k"]].unflatten(1, (self.kv_heads, self.dim))
+        k = qkv[:, o["k"]: o["v"]].unflatten(1, (self.kv_heads, self.dim))
+        v = qkv[:, o["v"]:].unflatten(1, (self.heads, self.vdim))
+        gates = (y[:, o["b"]: o["b"] + self.heads], y[:, o["a"]: o["a"] + self.heads], self.A_log, self.dt_bias)
+        r = ops.gated_delta_rule(q, k, v, None, None, recurrent, m.slots, m.lens, m.has_state, m.q_start, raw_gates=gates,
+                                 split_tf32=True)
+        r = ops.rmsnorm_gated(r.reshape(-1, self.value_dim), y[:, o["g"]: o["g"] + self.value_dim], self.norm.weight, self.eps,
+                              round_norm=False)
+        return ops.linear(r, self.out_proj.weight)

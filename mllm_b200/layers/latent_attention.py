@@ -1,0 +1,223 @@
+"""Latent attention without positions: the cache holds one row ``c`` of ``kv_rank`` features per token, shared by all
+heads; head ``h``'s key and value of a token are ``W_uk[h] c`` and ``W_uv[h] c``.  Queries go through a latent of their
+own.  Each head has a sink, a logit that joins the softmax denominator only.  A layer may read the latents of an
+earlier layer instead of writing its own.
+
+Two evaluations of the same sum (``csrc/latent.cu``):
+
+* absorbed: ``q' = W_uk[h]^T q`` meets the cached rows directly and the weighted sum of rows passes through ``W_uv[h]``
+  once per query — decode, short extends, 32-bit runs and head sizes the attention kernels do not have;
+* expanded: requests with many new tokens form K and V of their context with two matrix products and run the
+  attention kernels of the other models on them.  Heads are zero-padded (in the weights) to 64 / 128 / 256 features.
+
+A batch may need both: :func:`latent_plan` sorts the requests once per forward pass."""
+
+from __future__ import annotations
+
+from dataclasses import dataclass
+from typing import List, Optional
+
+import torch
+from torch import nn
+
+from .. import ops
+
+EXPAND_MIN_TOKENS = 32          # new tokens from which forming K and V of the context pays
+EXPAND_MAX_CONTEXT = 1 << 16    # context tokens expanded at a time (bounds the K and V buffers)
+
+
+@dataclass
+class ExpandGroup:
+    """Requests whose contexts are expanded together."""
+
+    req: torch.Tensor          # [b] request-table rows
+    seq_lens: torch.Tensor     # [b]
+    prefix_lens: torch.Tensor  # [b]
+    q_start: torch.Tensor      # [b] first query row
+    ctx_start: torch.Tensor    # [b] first row of the request's expanded context
+    rows: torch.Tensor         # [b, longest context] the identity table: row of every context token
+    batch: torch.Tensor        # [b] 0 .. b - 1, the rows of that table
+    total: int
+    max_ctx: int
+    max_q: int
+
+
+@dataclass
+class LatentPlan:
+    groups: List[ExpandGroup]
+    rows: Optional[torch.Tensor]      # query rows of the absorbed part (None: all of them)
+    row_req: Optional[torch.Tensor]   # [rows] request-table row (None: the absorbed part is empty)
+    row_pos: Optional[torch.Tensor]   # [rows] position
+    max_ctx: int                      # longest context of the absorbed part
+
+
+def latent_plan(fb, expand: bool, min_tokens: Optional[int] = None) -> LatentPlan:
+    """Which requests of the batch run expanded and which absorbed; cached in ``fb.extra``."""
+    key = ("latent_plan", expand)
+    got = fb.extra.get(key)
+    if got is not None:
+        return got
+    if fb.forward_mode.is_decode():
+        plan = LatentPlan([], None, fb.req_pool_indices.to(torch.int32), fb.positions.to(torch.int64), int(fb.max_seq_len))
+        fb.extra[key] = plan
+        return plan
+    least = EXPAND_MIN_TOKENS if min_tokens is None else min_tokens
+    dev = fb.input_ids.device
+    ext, pre = list(fb.extend_seq_lens_cpu), list(fb.extend_prefix_lens_cpu)
+    starts, total = [], 0
+    for n in ext:
+        starts.append(total)
+        total += n
+    far = [i for i, n in enumerate(ext) if expand and n >= least]
+    near = [i for i in range(len(ext)) if i not in set(far)]
+
+    def dev_i32(v):
+        return torch.tensor(v, dtype=torch.int32).to(dev, non_blocking=True)
+
+    groups: List[ExpandGroup] = []
+    run: List[int] = []
+
+    def close():
+        if not run:
+            return
+        sel = torch.tensor(run, dtype=torch.int64).to(dev, non_blocking=True)
+        ctx = [ext[i] + pre[i] for i in run]
+        at, acc = [], 0
+        for n in ctx:
+            at.append(acc)
+            acc += n
+        cs = dev_i32(at)
+        table = cs.unsqueeze(1) + torch.arange(max(ctx), dtype=torch.int32, device=dev).unsqueeze(0)
+        groups.append(ExpandGroup(
+            req=fb.req_pool_indices.index_select(0, sel).to(torch.int32), seq_lens=dev_i32(ctx),
+            prefix_lens=dev_i32([pre[i] for i in run]), q_start=dev_i32([starts[i] for i in run]), ctx_start=cs,
+            rows=table.clamp_(max=acc - 1), batch=torch.arange(len(run), dtype=torch.int32, device=dev), total=acc,
+            max_ctx=max(ctx), max_q=max(ext[i] for i in run)))
+        run.clear()
+
+    size = 0
+    for i in far:
+        if run and size + ext[i] + pre[i] > EXPAND_MAX_CONTEXT:
+            close()
+            size = 0
+        run.append(i)
+        size += ext[i] + pre[i]
+    close()
+    rows = row_req = row_pos = None
+    max_ctx = max((ext[i] + pre[i] for i in near), default=0)
+    if near:
+        if not far:
+            row_req = torch.repeat_interleave(fb.req_pool_indices.to(torch.int32), fb.extend_seq_lens.long(), output_size=total)
+            row_pos = fb.positions.to(torch.int64)
+        else:
+            owner = [i for i in near for _ in range(ext[i])]
+            picked = [r for i in near for r in range(starts[i], starts[i] + ext[i])]
+            rows = torch.tensor(picked, dtype=torch.int64).to(dev, non_blocking=True)
+            row_req = fb.req_pool_indices.to(torch.int32).index_select(0, torch.tensor(owner, dtype=torch.int64).to(dev, non_blocking=True))
+            row_pos = fb.positions.to(torch.int64).index_select(0, rows)
+    plan = LatentPlan(groups, rows, row_req, row_pos, max_ctx)
+    fb.extra[key] = plan
+    return plan
+
+
+def _pad_heads(w: torch.Tensor, heads: int, width: int) -> torch.Tensor:
+    """Rows of every head padded with zero rows to ``width``: [heads * d, k] -> [heads * width, k]."""
+    d = w.shape[0] // heads
+    if d == width:
+        return w
+    out = torch.zeros(heads, width, w.shape[1], dtype=w.dtype, device=w.device)
+    out[:, :d] = w.view(heads, d, -1)
+    return out.view(heads * width, -1)
+
+
+class LatentAttention(nn.Module):
+    def __init__(self, hidden_size: int, heads: int, dim: int, vdim: int, q_rank: int, kv_rank: int, scale: float, eps: float,
+                 latent_index: int, writes_latent: bool, params_dtype: torch.dtype) -> None:
+        """``latent_index``: the buffer of the latent pool this layer reads; ``writes_latent``: whether the layer has a
+        down projection of its own and fills it."""
+        super().__init__()
+        self.heads, self.dim, self.vdim, self.q_rank, self.kv_rank = heads, dim, vdim, q_rank, kv_rank
+        self.scale, self.eps, self.latent_index, self.writes_latent = float(scale), eps, latent_index, writes_latent
+
+        def p(*shape, dtype=params_dtype):
+            return nn.Parameter(torch.zeros(*shape, dtype=dtype), requires_grad=False)
+
+        def lin(o, i):
+            m = nn.Module()
+            m.weight = p(o, i)
+            return m
+
+        rows = q_rank + (kv_rank if writes_latent else 0)
+        self.down_proj = lin(-(-rows // 8) * 8, hidden_size)       # [query latent | cache latent | zero rows]
+        self.q_latent_norm = nn.Module()
+        self.q_latent_norm.weight = nn.Parameter(torch.ones(q_rank, dtype=torch.float32), requires_grad=False)
+        if writes_latent:
+            self.kv_latent_norm = nn.Module()
+            self.kv_latent_norm.weight = nn.Parameter(torch.ones(kv_rank, dtype=torch.float32), requires_grad=False)
+        self.q_up = lin(heads * dim, q_rank)
+        self.k_up = lin(heads * dim, kv_rank)
+        self.v_up = lin(heads * vdim, kv_rank)
+        self.sink = p(heads, dtype=torch.float32)
+        self.o_proj = lin(hidden_size, heads * vdim)
+        width = max(dim, vdim)
+        self.pad = next((w for w in (64, 128, 256) if width <= w), None)   # head size of the expanded form
+
+    def load_down(self, name: str, full: torch.Tensor) -> None:
+        o = 0 if name == "q" else self.q_rank
+        self.down_proj.weight.data[o:o + full.shape[0]].copy_(full)
+
+    def post_load(self) -> None:
+        """Weights in the layouts of the two forms: per head and K-major for the absorbed products, heads padded to the
+        attention kernels' size for the expanded ones."""
+        H = self.heads
+
+        def keep(t):
+            return nn.Parameter(t.contiguous(), requires_grad=False)
+
+        self._uk_t = keep(self.k_up.weight.data.view(H, self.dim, self.kv_rank).transpose(1, 2))      # [H, rank, dim]
+        self._uv = self.v_up.weight.data.view(H, self.vdim, self.kv_rank)                             # [H, vdim, rank]
+        if self.pad is not None and self.expandable(self.q_up.weight):
+            self._uq_pad = keep(_pad_heads(self.q_up.weight.data, H, self.pad))
+            self._uk_pad = keep(_pad_heads(self.k_up.weight.data, H, self.pad))
+            self._uv_pad = keep(_pad_heads(self.v_up.weight.data, H, self.pad))
+
+    def expandable(self, like: torch.Tensor) -> bool:
+        """The expanded form needs the 16-bit attention kernels on a GPU; on the CPU it runs in any type."""
+        return self.pad is not None and (not like.is_cuda or ops.attention_kernels_cover(self.pad, like.dtype, like.dtype)
+                                         and like.dtype != torch.float32)
+
+    def forward(self, x: torch.Tensor, fb) -> torch.Tensor:
+        T, H = x.shape[0], self.heads
+        cache = fb.token_to_kv_pool.get_latent_buffer(self.latent_index)
+        rtt = fb.req_to_token_pool.req_to_token
+        plan = latent_plan(fb, self.expandable(x))
+        y = ops.linear(x, self.down_proj.weight)
+        cq = ops.latent_prologue(y, self.q_latent_norm.weight, self.kv_latent_norm.weight if self.writes_latent else None,
+                                 self.eps, fb.out_cache_loc, cache if self.writes_latent else None)
+        o = None
+        if plan.groups:
+            o = self._expanded(cq, cache, rtt, plan)
+        if plan.row_req is not None:
+            c = cq if plan.rows is None else cq.index_select(0, plan.rows)
+            q = ops.linear(c, self.q_up.weight).view(-1, H, self.dim)
+            q = ops.head_linear(q, self._uk_t)
+            u = ops.latent_attention(q, cache, rtt, plan.row_req, plan.row_pos, self.scale, self.sink, plan.max_ctx)
+            u = ops.head_linear(u, self._uv)
+            if plan.rows is None:
+                o = u
+            else:
+                o.index_copy_(0, plan.rows, u)
+        return ops.linear(o.reshape(T, H * self.vdim), self.o_proj.weight)
+
+    def _expanded(self, cq, cache, rtt, plan: LatentPlan) -> torch.Tensor:
+        """Attention of the plan's expanded requests: [T, H, vdim], rows of other requests left unset."""
+        H, W = self.heads, self.pad
+        q = ops.linear(cq, self._uq_pad).view(-1, H, W)
+        out = torch.empty_like(q)
+        for g in plan.groups:
+            c = ops.latent_gather(cache, rtt, g.req, g.seq_lens, g.ctx_start, g.total, g.max_ctx)
+            k = ops.linear(c, self._uk_pad).view(-1, H, W)
+            v = ops.linear(c, self._uv_pad).view(-1, H, W)
+            ops.attention_prefill(q, k, v, g.rows, g.batch, g.seq_lens, g.prefix_lens, g.q_start, self.scale, out=out,
+                                  max_q_len=g.max_q, sink=self.sink)
+        return out if W == self.vdim else out[..., : self.vdim].contiguous()

@@ -52,6 +52,22 @@ class GemmaRMSNorm(RMSNorm):
         self.weight.data.copy_((w.float() + 1.0).to(self.weight.dtype))
 
 
+class DynamicTanh(nn.Module):
+    """``tanh(alpha * x) * weight + bias`` (a norm that takes no statistic), for a residual stream kept in fp32: the
+    call also adds the previous sublayer's output, ``x += mult * y``, in the same pass."""
+
+    def __init__(self, hidden_size: int, out_dtype: torch.dtype) -> None:
+        super().__init__()
+        self.out_dtype = out_dtype
+        self.alpha = nn.Parameter(torch.full((1,), 0.5, dtype=torch.float32), requires_grad=False)
+        self.weight = nn.Parameter(torch.ones(hidden_size, dtype=torch.float32), requires_grad=False)
+        self.bias = nn.Parameter(torch.zeros(hidden_size, dtype=torch.float32), requires_grad=False)
+
+    def forward(self, x: torch.Tensor, y: Optional[torch.Tensor] = None, mult: float = 1.0) -> torch.Tensor:
+        """``x`` [T, W] fp32 is updated in place when ``y`` is given; the normed rows come back in ``out_dtype``."""
+        return ops.residual_dyt(x, y, mult, self.alpha, self.weight, self.bias, self.out_dtype)
+
+
 class LayerNorm(nn.Module):
     def __init__(self, hidden_size: int, eps: float = 1e-6, bias: bool = True,
                  params_dtype: Optional[torch.dtype] = None) -> None:

@@ -27,7 +27,7 @@ cache by slot does not see the difference.
 
 from __future__ import annotations
 
-from typing import List, Optional, Tuple
+from typing import List, Optional, Sequence, Tuple
 
 import numpy as np
 import torch
@@ -99,6 +99,37 @@ class KVPool:
 
     def clear(self) -> None:
         self.store.zero_()
+
+
+class LatentPool:
+    """Cache of latent-attention layers: one row of ``widths[i]`` features per slot for every layer that writes
+    latents (layers that read another layer's latents have no buffer).  Slots and pages are those of
+    :class:`KVPool`: page 0 is never handed out and slot 0 is the sink of padded batch entries."""
+
+    def __init__(self, size: int, widths: Sequence[int], dtype: torch.dtype, device: torch.device | str, page_size: int = 1) -> None:
+        if dtype not in (torch.bfloat16, torch.float16, torch.float32):
+            raise NotImplementedError(f"latents are cached in the activation dtype, not {dtype}")
+        self.page_size = int(page_size)
+        self.size = (int(size) // self.page_size) * self.page_size
+        self.num_slots = self.size + self.page_size
+        self.widths, self.layer_num = list(widths), len(widths)
+        self.dtype, self.device = dtype, torch.device(device)
+        # rows begin on 16-byte boundaries
+        unit = 16 // torch.empty((), dtype=dtype).element_size()
+        self._store = [torch.zeros((self.num_slots, -(-w // unit) * unit), dtype=dtype, device=self.device) for w in self.widths]
+
+    @staticmethod
+    def cell_bytes(widths: Sequence[int], dtype: torch.dtype) -> int:
+        """Bytes one token occupies over all layers."""
+        eb = torch.empty((), dtype=dtype).element_size()
+        return sum(-(-w * eb // 16) * 16 for w in widths)
+
+    def get_latent_buffer(self, index: int) -> torch.Tensor:
+        return self._store[index][:, : self.widths[index]]
+
+    def clear(self) -> None:
+        for s in self._store:
+            s.zero_()
 
 
 class TokenToKVPoolAllocator:
@@ -226,6 +257,37 @@ class GDNPool:
 
     def bytes(self) -> int:
         return self.recurrent.numel() * 4 + self.conv.numel() * self.conv.element_size()
+
+
+class LayeredGDNPool(GDNPool):
+    """:class:`GDNPool` for models whose delta-net layers differ in size: ``shapes[i]`` is layer i's
+    ``(value heads, Dk, Dv, convolution channels, taps)``, and each layer has tensors of its own."""
+
+    def __init__(self, shapes: Sequence[Tuple[int, int, int, int, int]], slots: int, device,
+                 conv_dtype: torch.dtype = torch.bfloat16, track_slots: int = 0) -> None:
+        self.num_layers, self.slots, self.track_slots = len(shapes), slots, int(track_slots)
+        rows = slots + self.track_slots
+        self.layers = [(torch.zeros((rows, h, dk, dv), dtype=torch.float32, device=device),
+                        torch.zeros((rows, c, k - 1), dtype=conv_dtype, device=device)) for h, dk, dv, c, k in shapes]
+        self._free_track = list(range(slots, rows))
+
+    def layer(self, idx: int) -> Tuple[torch.Tensor, torch.Tensor]:
+        return self.layers[idx]
+
+    def reset(self, slot) -> None:
+        for recurrent, conv in self.layers:
+            recurrent[slot] = 0
+            conv[slot] = 0
+
+    def copy(self, src: int, dst: int) -> None:
+        for recurrent, conv in self.layers:
+            recurrent[dst] = recurrent[src]
+            conv[dst] = conv[src]
+
+    copy_states = copy
+
+    def bytes(self) -> int:
+        return sum(r.numel() * 4 + c.numel() * c.element_size() for r, c in self.layers)
 
 
 class ReqToTokenPool:

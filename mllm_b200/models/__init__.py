@@ -25,7 +25,20 @@ _REGISTRY: Dict[str, Tuple[str, str]] = {
     "SmolLM3ForCausalLM": ("mllm_b200.models.llama", "SmolLM3ForCausalLM"),
     "MiniCPMForCausalLM": ("mllm_b200.models.minicpm", "MiniCPMForCausalLM"),
     "MiniCPM4ForCausalLM": ("mllm_b200.models.minicpm", "MiniCPMForCausalLM"),
+    "PebulixForCausalLM": ("mllm_b200.models.pebulix", "PebulixForCausalLM"),
 }
+
+# designs whose config.json names itself in "architecture" and has a layout of its own: a function that checks the
+# file's content and returns it with the field names the runner reads
+_CONFIG_ADAPTERS: Dict[str, Tuple[str, str]] = {
+    "Pebulix": ("mllm_b200.models.pebulix", "adapt_config"),
+}
+
+
+def get_config_adapter(raw: dict):
+    """The adapter for the content of a ``config.json``, or None when it is laid out as transformers writes it."""
+    entry = _CONFIG_ADAPTERS.get(raw.get("architecture", "")) if isinstance(raw, dict) else None
+    return None if entry is None else getattr(importlib.import_module(entry[0]), entry[1])
 
 
 def register_model(arch: str, module: str, cls: str) -> None:

@@ -307,9 +307,9 @@ class Qwen3ForCausalLM(nn.Module):
         return self.model.embed_tokens.weight if self.tie else self.lm_head.weight
 
     def compute_logits(self, hidden: torch.Tensor, forward_batch: ForwardBatch) -> torch.Tensor:
-        if forward_batch.forward_mode.is_extend() and forward_batch.extend_seq_lens is not None:
-            last = torch.cumsum(forward_batch.extend_seq_lens, 0) - 1
-            hidden = hidden.index_select(0, last)
+        rows = forward_batch.logit_row_index()
+        if rows is not None:
+            hidden = hidden.index_select(0, rows)
         logits = ops.linear(hidden, self.lm_head_weight)
         if self.tp_size > 1:
             if logits.is_cuda and torch.cuda.is_current_stream_capturing():

@@ -222,8 +222,9 @@ class Qwen3_5ForCausalLM(nn.Module):
         fb.extra["gdn_pool"] = self.gdn_pool(fb)
         t0 = time.perf_counter()
         hidden = self.model(input_ids, fb, input_embeds)
-        if fb.forward_mode.is_extend() and fb.extend_seq_lens is not None:
-            hidden = hidden.index_select(0, torch.cumsum(fb.extend_seq_lens, 0) - 1)
+        rows = fb.logit_row_index()
+        if rows is not None:
+            hidden = hidden.index_select(0, rows)
         logits = ops.linear(hidden, self.lm_head_weight)
         ms = (time.perf_counter() - t0) * 1e3
         if fb.forward_mode.is_decode():

@@ -192,13 +192,9 @@ class ModelRunnerProcess:
                 self.state_pool.copy(m.state_slot, req.req_pool_idx)
 
     # ------------------------------------------------------------------ forward passes
-    def extend(self, items: Sequence[Tuple[Req, int]], sampling: bool = True):
-        """Run new tokens of several requests in one pass.
-
-        ``items``: (request, number of new tokens) — the tokens are the next ones after
-        ``req.num_computed`` in ``prompt + generated``.  Returns (sampled ids or None, rows that
-        produced a token): a row produces a token when its range ends at the current end of the
-        request's sequence."""
+    def _run_extend(self, items: Sequence[Tuple[Req, int]], logit_rows: Optional[Sequence[int]] = None):
+        """One pass over the next ``n`` tokens of each ``(request, n)``: (model output, batch).  ``logit_rows``: rows of
+        the concatenated tokens whose logits are returned instead of each request's last."""
         r = self.runner
         rtt = r.req_to_token_pool.req_to_token
         ids: List[int] = []
@@ -207,9 +203,10 @@ class ModelRunnerProcess:
         loc = self._alloc_rows(items)
         off = 0
         for req, n in items:
-            seq = req.all_ids()
             start = req.num_computed
-            ids.extend(seq[start : start + n])
+            # the tokens after num_computed in prompt + generated (prompts are long: no copy of the whole sequence)
+            mine = req.input_ids[start : start + n]
+            ids.extend(mine if len(mine) == n else req.all_ids()[start : start + n])
             rtt[req.req_pool_idx, start : start + n] = loc[off : off + n].to(torch.int32)
             off += n
             ext_lens.append(n)
@@ -224,6 +221,8 @@ class ModelRunnerProcess:
         uses_mrope = bool(getattr(r.model, "uses_mrope", False))
         if uses_mrope:  # position offsets already known for continued requests
             extra["mrope_position_deltas"] = torch.tensor([q.mrope_delta for q, _ in items], dtype=torch.int64).to(dev)
+        if logit_rows is not None:
+            extra["logit_rows"] = torch.tensor(list(logit_rows), dtype=torch.int64).to(dev, non_blocking=True)
         fb = r.prepare_forward_batch_extend(t_ids, t_pool, t_ext + t_pre, t_ext, t_pre, loc,
                                             extend_seq_lens_cpu=ext_lens, extend_prefix_lens_cpu=pre_lens, **extra)
         out = r.forward(fb)
@@ -231,14 +230,23 @@ class ModelRunnerProcess:
             for (q, _), d in zip(items, fb.mrope_position_deltas.tolist()):
                 q.mrope_delta = int(d)
         self.stats["prefill_tokens"] += total
-        produced = []
-        for i, (req, n) in enumerate(items):
+        for req, n in items:
             req.num_computed += n
-            if req.num_computed == req.seq_len:
-                produced.append(i)
+        return out, fb
+
+    def extend(self, items: Sequence[Tuple[Req, int]], sampling: bool = True):
+        """Run new tokens of several requests in one pass.
+
+        ``items``: (request, number of new tokens) — the tokens are the next ones after
+        ``req.num_computed`` in ``prompt + generated``.  Returns (sampled ids or None, rows that
+        produced a token): a row produces a token when its range ends at the current end of the
+        request's sequence."""
+        r = self.runner
+        out, fb = self._run_extend(items)
+        produced = [i for i, (req, _) in enumerate(items) if req.num_computed == req.seq_len]
         next_ids = None
         if sampling and produced:
-            rows = torch.tensor(produced, device=dev)
+            rows = torch.tensor(produced, device=self.device)
             logits = out.next_token_logits.index_select(0, rows)
             out.next_token_logits = logits
             next_ids = r.sample(out, self._sampling_info([items[i][0] for i in produced]))
@@ -249,11 +257,14 @@ class ModelRunnerProcess:
                 self._insert(req, req.input_ids)
         return next_ids, produced, fb
 
-    def decode(self, reqs: Sequence[Req]):
-        """One new token for every running request (graph path of the runner)."""
+    def extend_logits(self, items: Sequence[Tuple[Req, int]], logit_rows: Sequence[int]) -> torch.Tensor:
+        """The pass of :meth:`extend` without sampling: logits at the given rows of the concatenated new tokens."""
+        out, _ = self._run_extend(items, logit_rows)
+        return out.next_token_logits
+
+    def _run_decode(self, reqs: Sequence[Req]):
         r = self.runner
         dev = self.device
-        bs = len(reqs)
         loc = self._alloc_rows([(q, 1) for q in reqs])
         pool = torch.tensor([q.req_pool_idx for q in reqs], dtype=torch.int32).to(dev, non_blocking=True)
         pos = torch.tensor([q.num_computed for q in reqs], dtype=torch.int64).to(dev, non_blocking=True)
@@ -269,6 +280,12 @@ class ModelRunnerProcess:
         out = r.forward(fb)
         for q in reqs:
             q.num_computed += 1
+        return out, fb
+
+    def decode(self, reqs: Sequence[Req]):
+        """One new token for every running request (graph path of the runner)."""
+        r = self.runner
+        out, fb = self._run_decode(reqs)
         info = self._sampling_info(reqs)
         pre = getattr(out, "next_token_ids", None)
         if pre is not None and info.all_greedy and not info.has_penalties:
@@ -278,6 +295,11 @@ class ModelRunnerProcess:
         if any(q.return_logprob for q in reqs):      # touching the logits may trigger a cross-rank gather
             self._record_logprobs(reqs, out.next_token_logits, nxt)
         return nxt, fb
+
+    def decode_logits(self, reqs: Sequence[Req]) -> torch.Tensor:
+        """The pass of :meth:`decode` without sampling: logits [requests, vocab] after each request's last token."""
+        out, _ = self._run_decode(reqs)
+        return out.next_token_logits
 
     @staticmethod
     def _record_logprobs(reqs: Sequence[Req], logits: torch.Tensor, next_ids: torch.Tensor) -> None:

@@ -75,6 +75,30 @@ PRESETS["qwen3.5-2b"] = _hybrid(2048, 24, 8, 2, 6144, 256, 16, 16)
 PRESETS["qwen3.5-tiny"] = dict(_hybrid(256, 4, 2, 1, 512, 128, 1, 2, vocab=1024),
                                rope_parameters=dict(rope_theta=1e4, partial_rotary_factor=0.25, rope_type="default",
                                                     mrope_section=[6, 5, 5]))
+
+
+def _pebulix(layers, width, ff, vocab, heads, dim, q_rank, kv_rank, delta_heads, delta_dim, conv=4) -> Dict[str, Any]:
+    """Three delta-net layers to one latent-attention layer; every second latent layer reads the latents of the one before."""
+    out, last = [], None
+    for i in range(layers):
+        mlp = dict(kind="dense", ff=ff)
+        if (i + 1) % 4:
+            out.append(dict(type="delta", mlp=mlp, mixer=dict(heads=delta_heads, kv_heads=delta_heads, dim=delta_dim,
+                                                              vdim=delta_dim, conv=conv)))
+            continue
+        m = dict(heads=heads, dim=dim, vdim=dim, q_rank=q_rank, kv_rank=kv_rank, scale=dim ** -0.5)
+        if last is not None:
+            m["kv_from"], last = last, None
+        else:
+            last = i
+        out.append(dict(type="latent_attention", mlp=mlp, mixer=m))
+    return dict(architecture="Pebulix", layers=out, norm=dict(eps=1e-6), residual_mult=1.0, vocab=vocab, width=width,
+                torch_dtype="bfloat16")
+
+
+# hidden size, depth, feed-forward, vocabulary and delta-net heads of qwen3.5-2b
+PRESETS["pebulix-2b"] = _pebulix(24, 2048, 6144, 151936, heads=16, dim=128, q_rank=1024, kv_rank=512, delta_heads=16, delta_dim=128)
+PRESETS["pebulix-tiny"] = _pebulix(4, 128, 256, 1024, heads=2, dim=64, q_rank=64, kv_rank=64, delta_heads=2, delta_dim=32)
 _VL_VISION = dict(
     depth=24, hidden_size=1024, num_heads=16, intermediate_size=4096, patch_size=16, temporal_patch_size=2,
     spatial_merge_size=2, in_channels=3, out_hidden_size=2048, num_position_embeddings=2304,
@@ -156,7 +180,10 @@ def get_preset(name: str, **overrides) -> SimpleNamespace:
         raise KeyError(f"unknown preset {name!r}; have {sorted(PRESETS)}")
     d = copy.deepcopy(PRESETS[key])
     d.update(overrides)
-    return _to_ns(d)
+    from . import get_config_adapter
+
+    adapt = get_config_adapter(d)
+    return adapt(d) if adapt is not None else _to_ns(d)
 
 
 def preset_to_config_json(name: str) -> Dict[str, Any]:

@@ -59,6 +59,10 @@ def parse() -> argparse.Namespace:
                     help="tp only: fused = peer-memory kernels of this package, nccl = library all-reduce after o_proj / down_proj")
     ap.add_argument("--device", choices=["cuda", "cpu"], default="cuda",
                     help="cpu runs the same control flow on the host reference ops (flow tests; not a measurement)")
+    ap.add_argument("--design-pair", default=None, metavar="NEW:CLOSEST",
+                    help="instead of the flagship workload: prefill and decode throughput of two presets side by side, and "
+                         "their kernels against the roofline (e.g. pebulix-2b:qwen3.5-2b); one GPU, one JSON line")
+    ap.add_argument("--design-part", choices=["all", "kernels", "models"], default="all")
     ap.add_argument("--watchdog-s", type=float, default=1500.0,
                     help="give up (stack dump, error line, exit 3) when the whole run takes longer than this")
     return ap.parse_args()
@@ -377,6 +381,14 @@ def run_reference(a: argparse.Namespace) -> dict:
 
 def main() -> None:
     a = parse()
+    if a.design_pair:
+        from mllm_b200.benchmarks.design_pair import run as run_pair
+
+        sampler = ClockSampler(0)
+        sampler.start()
+        res = run_pair(a.design_pair, max(a.steps, 3), a.design_part)
+        print(json.dumps({**res, "clocks": sampler.stop()}), flush=True)
+        return
     out = run_reference(a) if a.impl == "reference" else run_ours(a)
     if out:
         print(json.dumps(out), flush=True)

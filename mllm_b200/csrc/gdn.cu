@@ -18,12 +18,34 @@ namespace {
 
 constexpr int kMaxConvK = 16;
 
-__device__ __forceinline__ float silu(float v) { return v / (1.f + expf(-v)); }
+// SiLU of a value that is rounded to T next: the fast exponential and division for 16-bit results
+template <typename T>
+__device__ __forceinline__ float silu(float v) {
+  if constexpr (sizeof(T) == 2) return __fdividef(v, 1.f + __expf(-v));
+  return v / (1.f + expf(-v));
+}
 
-// grid (ceil(C / 256), chunks, B); a CTA handles 256 channels of a run of tokens of one request.  KT: taps known at
-// compile time (0: any number up to kMaxConvK).  own_state: no request has more than one run, so the CTA also writes
-// the new history (it has read the old one already).
-template <typename T, int KT>
+// V neighbouring elements (V * sizeof(T) a power of two, aligned) as floats, and back
+template <typename T, int V>
+__device__ __forceinline__ void load_v(const T* p, float (&f)[V]) {
+  struct alignas(sizeof(T) * V) Pack { T e[V]; };
+  const Pack r = *reinterpret_cast<const Pack*>(p);
+#pragma unroll
+  for (int i = 0; i < V; ++i) f[i] = to_f32(r.e[i]);
+}
+template <typename T, int V>
+__device__ __forceinline__ void store_v(T* p, const float (&f)[V]) {
+  struct alignas(sizeof(T) * V) Pack { T e[V]; };
+  Pack r;
+#pragma unroll
+  for (int i = 0; i < V; ++i) r.e[i] = from_f32<T>(f[i]);
+  *reinterpret_cast<Pack*>(p) = r;
+}
+
+// grid (ceil(C / 256 V), chunks, B); a thread handles V neighbouring channels of a run of tokens of one request.  KT:
+// taps known at compile time (0: any number up to kMaxConvK).  own_state: no request has more than one run, so the
+// CTA also writes the new history (it has read the old one already).
+template <typename T, int KT, int V>
 __global__ void gdn_conv1d_silu_kernel(const T* __restrict__ x, int64_t x_ld, const T* __restrict__ w, T* __restrict__ conv_state,
                                        const int* __restrict__ slots, const int* __restrict__ lens,
                                        const int* __restrict__ has_state, const int* __restrict__ q_start,
@@ -31,7 +53,7 @@ __global__ void gdn_conv1d_silu_kernel(const T* __restrict__ x, int64_t x_ld, co
   pdl_wait();
   constexpr int kCap = KT > 0 ? KT : kMaxConvK;
   const int K = KT > 0 ? KT : taps;
-  const int c = blockIdx.x * blockDim.x + threadIdx.x;
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
   const int b = blockIdx.z;
   const int n = lens[b];
   const int t0 = blockIdx.y * chunk_tokens;
@@ -40,34 +62,45 @@ __global__ void gdn_conv1d_silu_kernel(const T* __restrict__ x, int64_t x_ld, co
   const int64_t row0 = q_start[b];
   T* st = conv_state + (static_cast<int64_t>(slots[b]) * channels + c) * (K - 1);
   const bool hist = has_state[b] != 0;
-  float wv[kCap], win[kCap];
+  float wv[kCap][V], win[kCap][V];
 #pragma unroll
   for (int j = 0; j < kCap; ++j)
-    if (j < K) wv[j] = to_f32(w[static_cast<int64_t>(c) * K + j]);
+#pragma unroll
+    for (int i = 0; i < V; ++i)
+      if (j < K) wv[j][i] = to_f32(w[static_cast<int64_t>(c + i) * K + j]);
   // window = the K-1 inputs before token t0
 #pragma unroll
   for (int j = 0; j < kCap - 1; ++j) {
     if (j < K - 1) {
       const int t = t0 - (K - 1) + j;
-      win[j] = t >= 0 ? to_f32(x[(row0 + t) * x_ld + c]) : (hist ? to_f32(st[K - 1 + t]) : 0.f);
+#pragma unroll
+      for (int i = 0; i < V; ++i)
+        win[j][i] = t >= 0 ? to_f32(x[(row0 + t) * x_ld + c + i]) : (hist ? to_f32(st[i * (K - 1) + K - 1 + t]) : 0.f);
     }
   }
 #pragma unroll 4
   for (int t = t0; t < t1; ++t) {
-    const float cur = to_f32(x[(row0 + t) * x_ld + c]);
-    float acc = 0.f;
+    float cur[V], acc[V];
+    load_v<T, V>(x + (row0 + t) * x_ld + c, cur);
 #pragma unroll
-    for (int j = 0; j < kCap; ++j)
-      if (j < K) acc = fmaf(wv[j], j == K - 1 ? cur : win[j], acc);
-    out[(row0 + t) * channels + c] = from_f32<T>(silu(acc));
+    for (int i = 0; i < V; ++i) {
+      acc[i] = 0.f;
 #pragma unroll
-    for (int j = 0; j < kCap - 1; ++j)
-      if (j < K - 1) win[j] = j == K - 2 ? cur : win[j + 1];
+      for (int j = 0; j < kCap; ++j)
+        if (j < K) acc[i] = fmaf(wv[j][i], j == K - 1 ? cur[i] : win[j][i], acc[i]);
+      acc[i] = silu<T>(acc[i]);
+#pragma unroll
+      for (int j = 0; j < kCap - 1; ++j)
+        if (j < K - 1) win[j][i] = j == K - 2 ? cur[i] : win[j + 1][i];
+    }
+    store_v<T, V>(out + (row0 + t) * channels + c, acc);
   }
   if (own_state) {
 #pragma unroll
     for (int j = 0; j < kCap - 1; ++j)
-      if (j < K - 1) st[j] = from_f32<T>(win[j]);
+#pragma unroll
+      for (int i = 0; i < V; ++i)
+        if (j < K - 1) st[i * (K - 1) + j] = from_f32<T>(win[j][i]);
   }
 }
 
@@ -262,7 +295,7 @@ __global__ void __launch_bounds__(256) gdn_recurrent_kernel(const GdnRuleParams 
 
 // out = weight * rmsnorm(x) * silu(gate); one warp per row.  Row r = (token r / heads, head r % heads) of x and out
 // (contiguous); gate rows of a token start gate_ld apart.  round_norm: the normed value is rounded to T before the weight.
-template <typename T>
+template <typename T, int V>
 __global__ void rmsnorm_gated_kernel(const T* __restrict__ x, const T* __restrict__ gate, int64_t gate_ld, const T* __restrict__ w,
                                      T* __restrict__ out, int64_t rows, int heads, int width, float eps, int round_norm) {
   pdl_wait();
@@ -271,17 +304,25 @@ __global__ void rmsnorm_gated_kernel(const T* __restrict__ x, const T* __restric
   if (r >= rows) return;
   const T* xr = x + r * width;
   const T* gr = gate + (r / heads) * gate_ld + (r % heads) * width;
-  float ss = 0.f;
-  for (int c = lane; c < width; c += 32) {
-    const float f = to_f32(xr[c]);
-    ss += f * f;
+  float ss = 0.f, f[V], g[V], wv[V];
+  for (int c = lane * V; c < width; c += 32 * V) {
+    load_v<T, V>(xr + c, f);
+#pragma unroll
+    for (int i = 0; i < V; ++i) ss = fmaf(f[i], f[i], ss);
   }
   ss = warp_sum(ss);
   const float rstd = 1.f / sqrtf(ss / static_cast<float>(width) + eps);
-  for (int c = lane; c < width; c += 32) {
-    float nrm = to_f32(xr[c]) * rstd;
-    if (round_norm) nrm = to_f32(from_f32<T>(nrm));
-    out[r * width + c] = from_f32<T>(to_f32(w[c]) * nrm * silu(to_f32(gr[c])));
+  for (int c = lane * V; c < width; c += 32 * V) {
+    load_v<T, V>(xr + c, f);
+    load_v<T, V>(gr + c, g);
+    load_v<T, V>(w + c, wv);
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      float nrm = f[i] * rstd;
+      if (round_norm) nrm = to_f32(from_f32<T>(nrm));
+      f[i] = wv[i] * nrm * silu<T>(g[i]);
+    }
+    store_v<T, V>(out + r * width + c, f);
   }
 }
 
@@ -299,18 +340,19 @@ int launch_recurrent_t(const GdnRuleParams& p, cudaStream_t s) {
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
-template <typename T>
-void launch_conv_t(const dim3& grid, cudaStream_t s, const void* x, int64_t x_ld, const void* w, void* st, const int* slots, const int* lens,
-                   const int* has, const int* q_start, void* out, int channels, int K, int chunk, int own) {
+template <typename T, int V>
+void launch_conv_t(int chunks, int batch, cudaStream_t s, const void* x, int64_t x_ld, const void* w, void* st, const int* slots,
+                   const int* lens, const int* has, const int* q_start, void* out, int channels, int K, int chunk, int own) {
+  const dim3 grid((channels + 256 * V - 1) / (256 * V), chunks, batch);
   auto go = [&](auto kernel) {
     launch_pdl(kernel, grid, dim3(256), 0, s, static_cast<const T*>(x), x_ld, static_cast<const T*>(w), static_cast<T*>(st), slots,
                lens, has, q_start, static_cast<T*>(out), channels, K, chunk, own);
   };
   switch (K) {
-    case 2: go(gdn_conv1d_silu_kernel<T, 2>); break;
-    case 3: go(gdn_conv1d_silu_kernel<T, 3>); break;
-    case 4: go(gdn_conv1d_silu_kernel<T, 4>); break;
-    default: go(gdn_conv1d_silu_kernel<T, 0>); break;
+    case 2: go(gdn_conv1d_silu_kernel<T, 2, V>); break;
+    case 3: go(gdn_conv1d_silu_kernel<T, 3, V>); break;
+    case 4: go(gdn_conv1d_silu_kernel<T, 4, V>); break;
+    default: go(gdn_conv1d_silu_kernel<T, 0, V>); break;
   }
 }
 
@@ -323,10 +365,17 @@ int launch_gdn_conv1d_silu(const void* x, int64_t x_ld, const void* w, void* con
   if (K < 1 || K > kMaxConvK) return -1;
   const int chunk = 64;
   const int chunks = (max_tokens + chunk - 1) / chunk;
-  const dim3 grid((channels + 255) / 256, chunks, batch);
   const int own = chunks == 1 ? 1 : 0;
-  MB200_DISPATCH_FLOAT(dt, (launch_conv_t<T>(grid, s, x, x_ld, w, conv_state, slots, lens, has_state, q_start, out, channels, K,
-                                             chunk, own)));
+  // two channels per thread when the rows allow it and there is more than a decode step to do
+  const uintptr_t align = reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(out);
+  const bool pair = channels % 2 == 0 && x_ld % 2 == 0 && align % (dt == kF32 ? 8 : 4) == 0 && max_tokens > 1;
+  if (pair) {
+    MB200_DISPATCH_FLOAT(dt, (launch_conv_t<T, 2>(chunks, batch, s, x, x_ld, w, conv_state, slots, lens, has_state, q_start, out,
+                                                  channels, K, chunk, own)));
+  } else {
+    MB200_DISPATCH_FLOAT(dt, (launch_conv_t<T, 1>(chunks, batch, s, x, x_ld, w, conv_state, slots, lens, has_state, q_start, out,
+                                                  channels, K, chunk, own)));
+  }
   note_launch();
   if (!own && K > 1) {
     const dim3 grid2((channels + 255) / 256, batch);
@@ -358,9 +407,18 @@ void launch_rmsnorm_gated(const void* x, const void* gate, int64_t gate_ld, cons
                           int width, float eps, int round_norm, DType dt, cudaStream_t s) {
   if (rows <= 0) return;
   const int warps = 8;
-  MB200_DISPATCH_FLOAT(dt, (launch_pdl(rmsnorm_gated_kernel<T>, dim3(static_cast<unsigned>((rows + warps - 1) / warps)),
-                                       dim3(warps * 32), 0, s, static_cast<const T*>(x), static_cast<const T*>(gate), gate_ld,
-                                       static_cast<const T*>(w), static_cast<T*>(out), rows, heads, width, eps, round_norm)));
+  const dim3 grid(static_cast<unsigned>((rows + warps - 1) / warps)), block(warps * 32);
+  const uintptr_t align = reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(w) |
+                          reinterpret_cast<uintptr_t>(out);
+  if (width % 4 == 0 && gate_ld % 4 == 0 && align % (dt == kF32 ? 16 : 8) == 0) {
+    MB200_DISPATCH_FLOAT(dt, (launch_pdl(rmsnorm_gated_kernel<T, 4>, grid, block, 0, s, static_cast<const T*>(x),
+                                         static_cast<const T*>(gate), gate_ld, static_cast<const T*>(w), static_cast<T*>(out), rows,
+                                         heads, width, eps, round_norm)));
+  } else {
+    MB200_DISPATCH_FLOAT(dt, (launch_pdl(rmsnorm_gated_kernel<T, 1>, grid, block, 0, s, static_cast<const T*>(x),
+                                         static_cast<const T*>(gate), gate_ld, static_cast<const T*>(w), static_cast<T*>(out), rows,
+                                         heads, width, eps, round_norm)));
+  }
   note_launch();
 }
 

@@ -12,9 +12,10 @@
 // (request, head) and a block of BV value features: grid (128 / BV, heads, batch), 256 threads.  The products
 // K K^T, Q K^T, K S0, Q S0, P U and K^T U' run on the tensor cores through warp-level MMA on tf32 operands with
 // fp32 accumulation (tiles of 16 x 16 x 8 read from shared memory); the state stays in fp32 in shared memory for
-// the whole sequence and is rounded to tf32 only as an MMA operand.  SPLIT: every operand enters as two tf32 terms
-// (its rounding and the remainder), three products per tile, which carries 21 bits of each operand through the
-// recurrence.  Heads of fewer than 128 features are zero-padded on their way into shared memory.  The substitution is the one sequential step;
+// the whole sequence and is rounded to tf32 only as an MMA operand.  The unit norms of q and k are row factors, applied
+// in fp32 where the products are scaled anyway: the K and Q operands stay the 16-bit inputs, which tf32 holds exactly.
+// SPLIT: every other operand enters as two tf32 terms (its rounding and the remainder), which carries 21 bits of it
+// through the recurrence: one product per tile for K K^T and Q K^T, two against K or Q, three otherwise.  Heads of fewer than 128 features are zero-padded on their way into shared memory.  The substitution is the one sequential step;
 // it runs 16 rows at a time (one thread per value feature inside a block, a tensor-core product to carry a solved
 // block into the rows below): one thread walking all 64 rows kept the other warps at a barrier for a quarter of
 // the kernel's issue slots.
@@ -40,7 +41,7 @@ constexpr int kGWarps = kGThreads / 32;
 template <int BV>
 struct GdnChunkCfg {
   static constexpr int kLdV = BV + 4;   // row stride of everything that is BV wide
-  static constexpr int kFloats = 2 * kGC * kGLd + kGD * kLdV + 2 * kGC * kGLdC + 3 * kGC * kLdV + 6 * kGC;
+  static constexpr int kFloats = 2 * kGC * kGLd + kGD * kLdV + 2 * kGC * kGLdC + 3 * kGC * kLdV + 8 * kGC;
   static constexpr int kSmem = kFloats * 4 + kGC * BV * 2 + 128;    // + the staged 16-bit V block of the next chunk
 };
 
@@ -66,29 +67,30 @@ __device__ __forceinline__ void to_tf32(F& f) {
   for (int i = 0; i < f.num_elements; ++i) f.x[i] = wmma::__float_to_tf32(f.x[i]);
 }
 
-// acc += A B with fp32 operands: one tf32 product, or (SPLIT) the three leading products of two-term operands
-template <bool SPLIT, typename FA, typename FB>
+// f becomes its tf32 rounding, lo the tf32 rounding of the remainder
+template <typename F>
+__device__ __forceinline__ void split_tf32(F& f, F& lo) {
+#pragma unroll
+  for (int i = 0; i < f.num_elements; ++i) {
+    const float hi = wmma::__float_to_tf32(f.x[i]);
+    lo.x[i] = wmma::__float_to_tf32(f.x[i] - hi);
+    f.x[i] = hi;
+  }
+}
+// acc += A B with fp32 operands: one tf32 product, or (SPLIT) the leading products of two-term operands.  XA / XB: the
+// operand's values are exact in tf32 already.
+template <bool SPLIT, bool XA, bool XB, typename FA, typename FB>
 __device__ __forceinline__ void mma_f32(FragC& acc, FA& fa, FB& fb) {
   if constexpr (SPLIT) {
     FA la;
     FB lb;
-#pragma unroll
-    for (int i = 0; i < fa.num_elements; ++i) {
-      const float hi = wmma::__float_to_tf32(fa.x[i]);
-      la.x[i] = wmma::__float_to_tf32(fa.x[i] - hi);
-      fa.x[i] = hi;
-    }
-#pragma unroll
-    for (int i = 0; i < fb.num_elements; ++i) {
-      const float hi = wmma::__float_to_tf32(fb.x[i]);
-      lb.x[i] = wmma::__float_to_tf32(fb.x[i] - hi);
-      fb.x[i] = hi;
-    }
-    wmma::mma_sync(acc, la, fb, acc);
-    wmma::mma_sync(acc, fa, lb, acc);
+    if constexpr (!XA) split_tf32(fa, la);
+    if constexpr (!XB) split_tf32(fb, lb);
+    if constexpr (!XA) wmma::mma_sync(acc, la, fb, acc);
+    if constexpr (!XB) wmma::mma_sync(acc, fa, lb, acc);
   } else {
-    to_tf32(fa);
-    to_tf32(fb);
+    if constexpr (!XA) to_tf32(fa);
+    if constexpr (!XB) to_tf32(fb);
   }
   wmma::mma_sync(acc, fa, fb, acc);
 }
@@ -108,8 +110,8 @@ __global__ void __launch_bounds__(kGThreads, 1) gdn_chunk_kernel(const GdnRulePa
   constexpr int kVT = BV / 16;   // 16-wide tiles across the value block
   extern __shared__ uint8_t gdn_smem_raw[];
   float* sm = reinterpret_cast<float*>((reinterpret_cast<uintptr_t>(gdn_smem_raw) + 127) & ~uintptr_t(127));
-  float* sK = sm;                        // [64][132] l2-normalised keys
-  float* sQ = sK + kGC * kGLd;           // [64][132] l2-normalised, scaled queries
+  float* sK = sm;                        // [64][132] keys as they came
+  float* sQ = sK + kGC * kGLd;           // [64][132] queries as they came
   float* sS = sQ + kGC * kGLd;           // [128][BV+4] state block
   float* sA = sS + kGD * kLdV;           // [64][68] K K^T, then A
   float* sP = sA + kGC * kGLdC;          // [64][68] Q K^T, then M * (Q K^T)
@@ -122,7 +124,9 @@ __global__ void __launch_bounds__(kGThreads, 1) gdn_chunk_kernel(const GdnRulePa
   float* sT = sE + kGC;                  // [64] exp(G_C - G)
   float* sGn = sT + kGC;                 // [64] staged g of the next chunk
   float* sBn = sGn + kGC;                // [64] staged beta of the next chunk
-  T* sVn = reinterpret_cast<T*>(sBn + kGC);   // [64][BV] staged V block of the next chunk
+  float* sRk = sBn + kGC;                // [64] 1 / |k|
+  float* sRq = sRk + kGC;                // [64] Dk^-0.5 / |q|
+  T* sVn = reinterpret_cast<T*>(sRq + kGC);   // [64][BV] staged V block of the next chunk
   // The 16-bit K and Q rows of the next chunk are staged in the bytes of sQ, which nothing reads once Q K^T and
   // Q S0 of the current chunk are done: K rows at byte 0, Q rows at byte 16384, 256 bytes per row.
   T* sKn = reinterpret_cast<T*>(sQ);
@@ -173,7 +177,7 @@ __global__ void __launch_bounds__(kGThreads, 1) gdn_chunk_kernel(const GdnRulePa
     const int nv = min(kGC, n - c0);
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();      // the staged rows of this chunk are visible to every thread
-    // ---- K and Q rows normalised (a warp per row; all rows are read before any is written: the staged rows
+    // ---- K and Q rows widened, their norms taken (a warp per row; all rows are read before any is written: the staged rows
     // share their bytes with sQ), the V block widened, g and beta moved; rows past the end are zero ----
     {
       float kk[kGC / kGWarps][4], qq[kGC / kGWarps][4];
@@ -204,11 +208,12 @@ __global__ void __launch_bounds__(kGThreads, 1) gdn_chunk_kernel(const GdnRulePa
         const int r = warp + it * kGWarps;
         const float ks = warp_sum(kk[it][0] * kk[it][0] + kk[it][1] * kk[it][1] + kk[it][2] * kk[it][2] + kk[it][3] * kk[it][3]);
         const float qs = warp_sum(qq[it][0] * qq[it][0] + qq[it][1] * qq[it][1] + qq[it][2] * qq[it][2] + qq[it][3] * qq[it][3]);
-        const float kn = rsqrtf(ks + 1e-6f), qn = rsqrtf(qs + 1e-6f) * qscale;
-        *reinterpret_cast<float4*>(sK + r * kGLd + lane * 4) =
-            make_float4(kk[it][0] * kn, kk[it][1] * kn, kk[it][2] * kn, kk[it][3] * kn);
-        *reinterpret_cast<float4*>(sQ + r * kGLd + lane * 4) =
-            make_float4(qq[it][0] * qn, qq[it][1] * qn, qq[it][2] * qn, qq[it][3] * qn);
+        if (lane == 0) {
+          sRk[r] = 1.f / sqrtf(ks + 1e-6f);
+          sRq[r] = qscale / sqrtf(qs + 1e-6f);
+        }
+        *reinterpret_cast<float4*>(sK + r * kGLd + lane * 4) = make_float4(kk[it][0], kk[it][1], kk[it][2], kk[it][3]);
+        *reinterpret_cast<float4*>(sQ + r * kGLd + lane * 4) = make_float4(qq[it][0], qq[it][1], qq[it][2], qq[it][3]);
       }
     }
     __syncthreads();
@@ -249,7 +254,7 @@ __global__ void __launch_bounds__(kGThreads, 1) gdn_chunk_kernel(const GdnRulePa
           FragBT fb;
           wmma::load_matrix_sync(fa, left + k0, kGLd);
           wmma::load_matrix_sync(fb, right + k0, kGLd);     // B[k][j] = K[j][k]
-          mma_f32<SPLIT>(acc, fa, fb);
+          mma_f32<SPLIT, true, true>(acc, fa, fb);
         }
         wmma::store_matrix_sync((which ? sP : sA) + ti * 16 * kGLdC + tj * 16, acc, kGLdC, wmma::mem_row_major);
       } else {
@@ -261,7 +266,7 @@ __global__ void __launch_bounds__(kGThreads, 1) gdn_chunk_kernel(const GdnRulePa
           FragB fb;
           wmma::load_matrix_sync(fa, left + k0, kGLd);
           wmma::load_matrix_sync(fb, sS + k0 * kLdV + tc * 16, kLdV);
-          mma_f32<SPLIT>(acc, fa, fb);
+          mma_f32<SPLIT, true, false>(acc, fa, fb);
         }
         wmma::store_matrix_sync((which ? sY : sX) + ti * 16 * kLdV + tc * 16, acc, kLdV, wmma::mem_row_major);
       }
@@ -275,14 +280,15 @@ __global__ void __launch_bounds__(kGThreads, 1) gdn_chunk_kernel(const GdnRulePa
       const int i = idx >> 6, j = idx & 63;
       const float d = j <= i ? __expf(sG[i] - sG[j]) : 0.f;
       const float ka = sA[i * kGLdC + j], qa = sP[i * kGLdC + j];
-      sA[i * kGLdC + j] = j < i ? sB[i] * d * ka : 0.f;
-      sP[i * kGLdC + j] = j <= i ? d * qa : 0.f;
+      const float rk = sRk[j];
+      sA[i * kGLdC + j] = j < i ? sB[i] * d * (sRk[i] * rk * ka) : 0.f;
+      sP[i * kGLdC + j] = j <= i ? d * (sRq[i] * rk * qa) : 0.f;
     }
     for (int idx = tid; idx < kGC * BV; idx += kGThreads) {
       const int i = idx / BV, c = idx % BV;
       const float e = sE[i];
-      sU[i * kLdV + c] = sB[i] * (sU[i * kLdV + c] - e * sX[i * kLdV + c]);
-      sY[i * kLdV + c] *= e;
+      sU[i * kLdV + c] = sB[i] * (sU[i * kLdV + c] - e * sRk[i] * sX[i * kLdV + c]);
+      sY[i * kLdV + c] *= e * sRq[i];
     }
     __syncthreads();
 
@@ -310,7 +316,7 @@ __global__ void __launch_bounds__(kGThreads, 1) gdn_chunk_kernel(const GdnRulePa
         for (int i = 0; i < 16; ++i) {
           const int row = blk * 16 + i;
           sU[row * kLdV + tid] = u[i];
-          sX[row * kLdV + tid] = sT[row] * u[i];
+          sX[row * kLdV + tid] = sT[row] * sRk[row] * u[i];
         }
       }
       __syncthreads();
@@ -328,7 +334,7 @@ __global__ void __launch_bounds__(kGThreads, 1) gdn_chunk_kernel(const GdnRulePa
             wmma::load_matrix_sync(fb, sU + (blk * 16 + k0) * kLdV + tc * 16, kLdV);
 #pragma unroll
             for (int i = 0; i < fa.num_elements; ++i) fa.x[i] = -fa.x[i];
-            mma_f32<SPLIT>(acc, fa, fb);
+            mma_f32<SPLIT, false, false>(acc, fa, fb);
           }
           wmma::store_matrix_sync(tile, acc, kLdV, wmma::mem_row_major);
         }
@@ -349,7 +355,7 @@ __global__ void __launch_bounds__(kGThreads, 1) gdn_chunk_kernel(const GdnRulePa
           FragB fb;
           wmma::load_matrix_sync(fa, sP + ti * 16 * kGLdC + k0, kGLdC);
           wmma::load_matrix_sync(fb, sU + k0 * kLdV + tc * 16, kLdV);
-          mma_f32<SPLIT>(acc, fa, fb);
+          mma_f32<SPLIT, false, false>(acc, fa, fb);
         }
         wmma::store_matrix_sync(tile, acc, kLdV, wmma::mem_row_major);
       } else {
@@ -364,7 +370,7 @@ __global__ void __launch_bounds__(kGThreads, 1) gdn_chunk_kernel(const GdnRulePa
           FragB fb;
           wmma::load_matrix_sync(fa, sK + k0 * kGLd + tm * 16, kGLd);    // A[m][k] = K[k][m]
           wmma::load_matrix_sync(fb, sX + k0 * kLdV + tc * 16, kLdV);
-          mma_f32<SPLIT>(acc, fa, fb);
+          mma_f32<SPLIT, true, false>(acc, fa, fb);
         }
         wmma::store_matrix_sync(tile, acc, kLdV, wmma::mem_row_major);
       }

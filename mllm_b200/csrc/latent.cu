@@ -461,31 +461,40 @@ __global__ void __launch_bounds__(256) latent_attn_mma_kernel(const LatentParams
     }
 }
 
-// out = sum_s w_s * O_s, w_s = 2^(lse_s - max) / (sum + sink); grid (heads, rows)
+// out = sum_s w_s * O_s, w_s = 2^(lse_s - max) / (sum + sink); grid (heads, rows), splits <= 64.  The weights are formed
+// once by a warp (two splits per lane); then a thread sums four features over the splits with independent loads.
 template <typename T>
 __global__ void __launch_bounds__(128) latent_merge_kernel(const LatentParams p) {
   pdl_launch_dependents();
   pdl_wait();
-  const int h = blockIdx.x, row = blockIdx.y;
+  __shared__ float wt[64];
+  const int h = blockIdx.x, row = blockIdx.y, tid = threadIdx.x;
   const int64_t at = static_cast<int64_t>(row) * p.heads + h;
   const float* lse = p.part_lse + at * p.splits;
-  float m = -INFINITY;
-  for (int s = 0; s < p.splits; ++s) m = fmaxf(m, lse[s]);
-  float den = 0.f;
-  if (p.sink != nullptr) {
-    const float sl = p.sink[h] * kLatLog2e;
-    m = fmaxf(m, sl);
-    den = exp2f(sl - m);
+  if (tid < 32) {
+    const float l0 = tid < p.splits ? lse[tid] : -INFINITY, l1 = tid + 32 < p.splits ? lse[tid + 32] : -INFINITY;
+    const float sl = p.sink != nullptr ? p.sink[h] * kLatLog2e : -INFINITY;
+    const float m = fmaxf(warp_max(fmaxf(l0, l1)), sl);
+    const float w0 = exp2f(l0 - m), w1 = exp2f(l1 - m);
+    const float den = warp_sum(w0 + w1) + exp2f(sl - m);
+    wt[tid] = w0 / den;
+    wt[tid + 32] = w1 / den;
   }
-  for (int s = 0; s < p.splits; ++s) den += exp2f(lse[s] - m);
-  const float inv = 1.f / den;
-  for (int c = threadIdx.x; c < p.rank; c += blockDim.x) {
-    float acc = 0.f;
+  __syncthreads();
+  const float* po = p.part_o + at * p.splits * p.rank;
+  for (int c = tid * 4; c < p.rank; c += 512) {      // the rank is a multiple of 8
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
     for (int s = 0; s < p.splits; ++s) {
-      const float w = exp2f(lse[s] - m);
-      if (w > 0.f) acc = fmaf(w, p.part_o[(at * p.splits + s) * p.rank + c], acc);
+      const float w = wt[s];
+      const float4 v = *reinterpret_cast<const float4*>(po + static_cast<int64_t>(s) * p.rank + c);
+      acc.x = fmaf(w, v.x, acc.x);
+      acc.y = fmaf(w, v.y, acc.y);
+      acc.z = fmaf(w, v.z, acc.z);
+      acc.w = fmaf(w, v.w, acc.w);
     }
-    static_cast<T*>(p.out)[at * p.rank + c] = from_f32<T>(acc * inv);
+    T four[4] = {from_f32<T>(acc.x), from_f32<T>(acc.y), from_f32<T>(acc.z), from_f32<T>(acc.w)};
+    *reinterpret_cast<uint2*>(static_cast<T*>(p.out) + at * p.rank + c) = *reinterpret_cast<const uint2*>(four);
   }
 }
 

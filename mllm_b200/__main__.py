@@ -25,10 +25,13 @@ def show_config() -> dict:
         info["gpu"] = {"name": p.name, "capability": f"{p.major}.{p.minor}", "sms": p.multi_processor_count,
                        "memory_gib": round(p.total_memory / 2 ** 30, 1), "count": torch.cuda.device_count()}
     ext = {}
-    try:
-        ext["mllm_b200_C"] = ops.ext() is not None
-    except Exception as exc:
-        ext["mllm_b200_C"] = f"not loaded: {exc}"
+    from ._build import load_extension
+
+    for name in ("mllm_b200_C", "mllm_b200_X"):
+        try:
+            ext[name] = load_extension(name) is not None
+        except Exception as exc:
+            ext[name] = f"not loaded: {exc}"
     try:
         from .mem_cache.native import host_ext
 

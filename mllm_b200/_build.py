@@ -1,8 +1,10 @@
 """Build / load the native extensions in-tree.
 
-Two extensions live under ``mllm_b200/csrc``:
+Three extensions live under ``mllm_b200/csrc``:
 
-* ``mllm_b200_C``    — the sm_100a CUDA kernels plus their PyTorch binding;
+* ``mllm_b200_C``    — the sm_100a CUDA kernels of every decoder plus their PyTorch binding;
+* ``mllm_b200_X``    — kernels that only some models or layouts use (experts, 4-bit weights, vision towers, tensor- and
+  expert-parallel exchange), loaded, and where it is missing compiled, when one of them is first called;
 * ``mllm_b200_host`` — host-only C++ (radix tree, page allocator, ``.mllm`` file reader).
 
 They are compiled with ``torch.utils.cpp_extension.load`` into ``mllm_b200/_ext`` so the
@@ -35,9 +37,15 @@ CXX_FLAGS = ["-O3", "-std=c++17"]
 
 EXTENSIONS: Dict[str, Dict[str, List[str]]] = {
     "mllm_b200_C": {
-        "sources": ["bindings.cpp", "elementwise.cu", "gemm_tcgen05.cu", "attention.cu", "sampling.cu", "moe.cu",
-                    "comm.cu", "gemm_w4a16.cu", "vision.cu", "gdn.cu", "gdn_chunk.cu", "latent.cu", "no_alloc.cu", "ep_a2a.cu", "gemm_smallm.cu", "gemm_smallm_w4.cu"],
-        "headers": ["common.cuh", "kernels.h", "no_alloc.h"],
+        "sources": ["bindings.cpp", "runtime.cu", "elementwise.cu", "gemm_tcgen05.cu", "gemm_smallm.cu", "attention.cu",
+                    "sampling.cu", "gdn.cu", "gdn_chunk.cu", "latent.cu", "no_alloc.cu"],
+        "headers": ["bindings_common.h", "common.cuh", "kernels.h", "no_alloc.h"],
+        "cuda": True,
+    },
+    "mllm_b200_X": {
+        "sources": ["bindings_extra.cpp", "runtime.cu", "moe.cu", "comm.cu", "ep_a2a.cu", "gemm_w4a16.cu", "gemm_smallm_w4.cu",
+                    "vision.cu"],
+        "headers": ["bindings_common.h", "common.cuh", "kernels.h"],
         "cuda": True,
     },
     "mllm_b200_host": {

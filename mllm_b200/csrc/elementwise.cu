@@ -5,61 +5,12 @@
 // All of them move 16 bytes per thread per access and touch every byte once
 // (the norm kernels keep a row in registers between the reduction and the
 // scaling pass), so their ceiling is HBM bandwidth.
-#include <atomic>
 #include <cstdlib>
-#include <map>
-#include <mutex>
-#include <utility>
 
 #include "common.cuh"
 #include "kernels.h"
 
 namespace mb200 {
-
-static std::atomic<uint64_t> g_launches{0};
-uint64_t launch_count() { return g_launches.load(); }
-void note_launch(int n) { g_launches.fetch_add(n); }
-bool pdl_enabled() {
-  static const bool on = [] {
-    const char* v = std::getenv("MLLM_B200_PDL");
-    return !(v != nullptr && v[0] == '0');
-  }();
-  return on;
-}
-
-cudaError_t ensure_dynamic_smem(const void* kernel, int bytes) {
-  static std::mutex mu;
-  static std::map<std::pair<const void*, int>, int> set_to;  // (kernel, device) -> bytes granted
-  int dev = 0;
-  cudaError_t err = cudaGetDevice(&dev);
-  if (err != cudaSuccess) return err;
-  std::lock_guard<std::mutex> lock(mu);
-  auto it = set_to.find({kernel, dev});
-  if (it != set_to.end() && it->second >= bytes) return cudaSuccess;
-  err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
-  if (err == cudaSuccess) set_to[{kernel, dev}] = bytes;
-  return err;
-}
-
-void ensure_max_carveout(const void* kernel) {
-  static const bool on = [] {
-    // opt-in: measured neutral on the decode step (5.38 ms with, 5.34 ms without), so the default leaves every
-    // kernel's carve-out to the driver
-    const char* v = std::getenv("MLLM_B200_MAX_CARVEOUT");
-    return v != nullptr && v[0] == '1';
-  }();
-  if (!on) return;
-  static std::mutex mu;
-  static std::map<std::pair<const void*, int>, bool> done;
-  int dev = 0;
-  if (cudaGetDevice(&dev) != cudaSuccess) return;
-  std::lock_guard<std::mutex> lock(mu);
-  auto& d = done[{kernel, dev}];
-  if (d) return;
-  d = true;
-  cudaFuncSetAttribute(kernel, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
-  cudaGetLastError();   // a kernel that cannot take the hint keeps its default
-}
 
 namespace {
 

@@ -1215,49 +1215,15 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_consta
 // ---------------------------------------------------------------------------------------
 // host side
 // ---------------------------------------------------------------------------------------
-using EncodeFn = CUresult (*)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*,
-                              const cuuint64_t*, const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave,
-                              CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-
-EncodeFn get_encode_fn() {
-  static EncodeFn fn = nullptr;
-  static std::once_flag once;
-  std::call_once(once, [] {
-    void* sym = nullptr;
-    cudaDriverEntryPointQueryResult qres;
-    if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &sym, cudaEnableDefault, &qres) == cudaSuccess &&
-        qres == cudaDriverEntryPointSuccess) {
-      fn = reinterpret_cast<EncodeFn>(sym);
-    }
-  });
-  return fn;
-}
-
 int env_int(const char* name, int dflt) {
   const char* v = std::getenv(name);
   return (v != nullptr && *v != 0) ? std::atoi(v) : dflt;
 }
 
-CUtensorMapL2promotion l2_promotion() {
-  static const int v = env_int("MLLM_B200_GEMM_L2_PROMO", 256);
-  return v == 0 ? CU_TENSOR_MAP_L2_PROMOTION_NONE
-                : (v == 64 ? CU_TENSOR_MAP_L2_PROMOTION_L2_64B
-                           : (v == 128 ? CU_TENSOR_MAP_L2_PROMOTION_L2_128B : CU_TENSOR_MAP_L2_PROMOTION_L2_256B));
-}
-
-// 2-D row-major matrix [rows, k] (k contiguous, `ld` elements between rows); box = 128 bytes of k x box_rows.
 bool make_operand_map(CUtensorMap* map, const void* base, int64_t rows, int64_t k, int64_t ld, int elem_bytes,
                       CUtensorMapDataType type, int box_rows) {
-  EncodeFn fn = get_encode_fn();
-  if (fn == nullptr) return false;
-  cuuint64_t dims[2] = {static_cast<cuuint64_t>(k), static_cast<cuuint64_t>(rows)};
-  cuuint64_t strides[1] = {static_cast<cuuint64_t>(ld) * elem_bytes};
-  cuuint32_t box[2] = {static_cast<cuuint32_t>(kRowBytes / elem_bytes), static_cast<cuuint32_t>(box_rows)};
-  cuuint32_t estr[2] = {1, 1};
-  CUresult r = fn(map, type, 2, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
-                  CU_TENSOR_MAP_SWIZZLE_128B, l2_promotion(),
-                  CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-  return r == CUDA_SUCCESS;
+  const int code = type == CU_TENSOR_MAP_DATA_TYPE_UINT8 ? 2 : (type == CU_TENSOR_MAP_DATA_TYPE_FLOAT16 ? 1 : 0);
+  return make_tma_operand_map(map, base, rows, k, ld, elem_bytes, code, box_rows);
 }
 
 template <int BN, bool SWAP, bool SWIGLU, int RT = 1, int KD = 1>
@@ -1327,15 +1293,6 @@ int launch_pair_cfg(const CUtensorMap& tr, const CUtensorMap& tc, const KParams&
 }
 
 }  // namespace
-
-bool make_tma_operand_map(void* map, const void* base, int64_t rows, int64_t k, int64_t ld, int elem_bytes, int type,
-                          int box_rows) {
-  const CUtensorMapDataType t = type == 2 ? CU_TENSOR_MAP_DATA_TYPE_UINT8
-                                          : (type == 1 ? CU_TENSOR_MAP_DATA_TYPE_FLOAT16 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16);
-  return make_operand_map(static_cast<CUtensorMap*>(map), base, rows, k, ld, elem_bytes, t, box_rows);
-}
-
-size_t gemm_workspace_bytes(int, int, int, int) { return size_t(64) << 20; }
 
 int launch_gemm(const GemmArgs& a, cudaStream_t s) {
   if (a.m <= 0 || a.n <= 0) return 0;

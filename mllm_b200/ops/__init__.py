@@ -1,7 +1,7 @@
 """Operator front-end: one Python function per hot op.
 
 For tensors on a GPU every function launches the hand-written sm_100a kernel
-from the in-tree ``mllm_b200_C`` extension and raises if that extension cannot
+from the in-tree extension modules (``mllm_b200_C``, ``mllm_b200_X``) and raises if they cannot
 be loaded — there is no silent framework fallback on a GPU.  For CPU tensors
 (tests, fp32 oracle) the plain-PyTorch statement in :mod:`.reference` runs.
 ``MLLM_B200_FORCE_TORCH=1`` forces the PyTorch statement everywhere, which the
@@ -21,19 +21,49 @@ _FORCE_TORCH = os.environ.get("MLLM_B200_FORCE_TORCH", "0") == "1"
 _ext = None
 
 
-def ext():
-    """The CUDA extension module (loaded on first use; raises when unavailable)."""
-    global _ext
-    if _ext is None:
+class _Kernels:
+    """The kernel functions of the CUDA extension modules under one name; a module is loaded when one of its functions is
+    first asked for."""
+
+    def __init__(self) -> None:
+        self.__dict__["_mods"] = {}
+        self._load("mllm_b200_C")
+
+    def _load(self, name: str):
         from .._build import load_extension
 
-        mod = load_extension("mllm_b200_C")
+        mod = load_extension(name)
         if mod is None:
             raise RuntimeError(
-                "mllm_b200: the sm_100a kernel extension (mllm_b200_C) is not built; "
+                f"mllm_b200: the sm_100a kernel extension ({name}) is not built; "
                 "run `python -m mllm_b200._build` or `__graft_entry__.build()`."
             )
-        _ext = mod
+        self._mods[name] = mod
+        return mod
+
+    def __getattr__(self, name: str):
+        if name.startswith("_"):
+            raise AttributeError(name)
+        for module in ("mllm_b200_C", "mllm_b200_X"):
+            mod = self._mods.get(module) or self._load(module)
+            fn = getattr(mod, name, None)
+            if fn is not None:
+                self.__dict__[name] = fn
+                return fn
+        raise AttributeError(name)
+
+    def launch_count(self) -> int:
+        return sum(int(m.launch_count()) for m in self._mods.values())
+
+    def read_status(self, device: int) -> int:
+        return next((c for c in [int(m.read_status(device)) for m in self._mods.values()] if c), 0)
+
+
+def ext():
+    """The CUDA kernels (loaded on first use; raises when unavailable)."""
+    global _ext
+    if _ext is None:
+        _ext = _Kernels()
     return _ext
 
 

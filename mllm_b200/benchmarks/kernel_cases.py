@@ -175,9 +175,28 @@ def gdn(a) -> dict:
             "us_per_64_tokens": ms * 1e3 / (L / 64), "state_tflops": 6 * T * H * D * D / ms / 1e9}
 
 
+def latent(a) -> dict:
+    """Decode of latent attention: `--batch` requests of `--seq` tokens, `--hq` heads over latents of `--rank` features."""
+    dev = "cuda"
+    table = (torch.arange(a.batch * a.seq, device=dev, dtype=torch.int32) + 16).view(a.batch, a.seq)
+    req = torch.arange(a.batch, dtype=torch.int32, device=dev)
+    pos = torch.full((a.batch,), a.seq - 1, dtype=torch.int64, device=dev)
+    caches = [torch.randn(a.batch * a.seq + 16, a.rank, device=dev, dtype=torch.bfloat16) for _ in range(max(1, a.kv_sets))]
+    q = torch.randn(a.batch, a.hq, a.rank, device=dev, dtype=torch.bfloat16) * a.rank ** -0.5
+    sink = torch.zeros(a.hq, device=dev)
+
+    def run():
+        for c in caches:
+            ops.latent_attention(q, c, table, req, pos, 1.0, sink, a.seq)
+
+    ms = _time(run, a.iters) / len(caches)
+    return {"case": "latent", "batch": a.batch, "seq": a.seq, "heads": a.hq, "rank": a.rank, "ms": ms,
+            "gbs": a.batch * a.seq * a.rank * 2 / ms / 1e6, "tflops": 4 * a.batch * a.seq * a.hq * a.rank / ms / 1e9}
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
-    ap.add_argument("case", choices=["attn_decode", "attn_prefill", "gemm", "moe", "w4a16", "gdn"])
+    ap.add_argument("case", choices=["attn_decode", "attn_prefill", "gemm", "moe", "w4a16", "gdn", "latent"])
     ap.add_argument("--gdn-backend", default="auto", choices=["auto", "cuda_chunkwise", "mllm_kernel"],
                     help="gdn: chunk-parallel kernel, token-sequential kernel, or the default choice between them")
     ap.add_argument("--experts", type=int, default=16, help="moe: local experts")
@@ -185,6 +204,7 @@ def main() -> None:
     ap.add_argument("--seq", type=int, default=2050)
     ap.add_argument("--hq", type=int, default=32)
     ap.add_argument("--hkv", type=int, default=8)
+    ap.add_argument("--rank", type=int, default=512, help="latent: features of a cached row")
     ap.add_argument("--m", type=int, default=8)
     ap.add_argument("--n", type=int, default=4096)
     ap.add_argument("--k", type=int, default=4096)
@@ -195,7 +215,8 @@ def main() -> None:
     ap.add_argument("--iters", type=int, default=20)
     ap.add_argument("--kv-sets", type=int, default=4, help="attn_decode: KV caches used in turn (working set > L2)")
     a = ap.parse_args()
-    out = {"attn_decode": attn_decode, "attn_prefill": attn_prefill, "gemm": gemm, "moe": moe, "w4a16": w4a16, "gdn": gdn}[a.case](a)
+    out = {"attn_decode": attn_decode, "attn_prefill": attn_prefill, "gemm": gemm, "moe": moe, "w4a16": w4a16, "gdn": gdn,
+           "latent": latent}[a.case](a)
     ops.check_status()
     print(json.dumps(out))
 

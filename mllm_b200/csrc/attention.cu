@@ -84,18 +84,9 @@ __device__ __forceinline__ float tanh_approx(float x) {
   asm("tanh.approx.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
-// 1 / softmax denominator of a row with sum `l` over its keys, taken relative to 2^m.  A sink adds exp(sink) once: it
-// has no key and no value and is not scaled.
-__device__ __forceinline__ float inv_denominator(float l, float m, const float* sink, int head) {
-  if (!(l > 0.f)) return 0.f;
-  if (sink == nullptr) return 1.f / l;
-  const float d = sink[head] * kLog2e - m;
-  if (d > 0.f) {
-    const float e = exp2f(-d);
-    return e / fmaf(l, e, 1.f);
-  }
-  return 1.f / (l + exp2f(d));
-}
+// What a head's sink adds to a softmax denominator kept relative to 2^m: exp(sink) once; it has no key and no value and
+// is not scaled.  (Infinite when the sink is out of reach of every key: the row's output is then 0, as it should be.)
+__device__ __forceinline__ float sink_term(const float* sink, int head, float m) { return exp2f(sink[head] * kLog2e - m); }
 __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N>
 __device__ __forceinline__ void cp_async_wait() {
@@ -446,7 +437,8 @@ __global__ void __launch_bounds__(kAttnThreads, FwdCfg<NH>::kCtasPerSm) attn_fwd
   if (!ok_all && p.status != nullptr) atomicExch(p.status, kStatusPipelineTimeout);
 
   // ---- epilogue (partial results of a split leave the sink to the merge) ---------------------
-  const float inv_l = inv_denominator(l_sum, m_used, p.is_decode && p.num_splits > 1 ? nullptr : p.sink, row_head);
+  if (p.sink != nullptr && !(p.is_decode && p.num_splits > 1)) l_sum += sink_term(p.sink, row_head, m_used);
+  const float inv_l = l_sum > 0.f ? 1.f / l_sum : 0.f;
   if (p.is_decode && p.num_splits > 1) {
     float* po = p.part_o + ((static_cast<int64_t>(b) * p.hq + row_head) * p.num_splits + split) * kD;
 #pragma unroll 1
@@ -911,7 +903,11 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
       }
     }
     asm volatile("bar.sync 1, 128;" ::: "memory");
-    if (tid < g) red2[tid] = redt[tid] + redt[NQ + tid] + redt[2 * NQ + tid] + redt[3 * NQ + tid];
+    if (tid < g) {
+      float l = redt[tid] + redt[NQ + tid] + redt[2 * NQ + tid] + redt[3 * NQ + tid];
+      if (p.sink != nullptr && p.num_splits == 1) l += sink_term(p.sink, hk * g + tid, m_used_at(m_used, tid));
+      red2[tid] = l;
+    }
     asm volatile("bar.sync 1, 128;" ::: "memory");
     const bool good = ok_all && (*fail_flag == 0);
 
@@ -926,9 +922,8 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
         const int c = c0 + i;
         if (c < g && good) {
           const float l = red2[c];
+          const float v = l > 0.f ? __uint_as_float(o[i]) / l : 0.f;
           const int head = hk * g + c;
-          const float v = p.sink != nullptr && p.num_splits == 1 ? __uint_as_float(o[i]) * inv_denominator(l, m_used[c], p.sink, head)
-                          : l > 0.f ? __uint_as_float(o[i]) / l : 0.f;
           if (p.num_splits > 1) {
             p.part_o[((static_cast<int64_t>(b) * p.hq + head) * p.num_splits + split) * kD + tid] = v;
           } else {
@@ -1323,7 +1318,8 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
 
     // ---- epilogue: normalise, park the group's 128 rows x 256 B in its P buffer (free now), then store them
     // row by row: 16 lanes cover one output row, and the g rows of a token are adjacent in memory ----
-    const float inv_l = inv_denominator(l_sum, m_used, p.sink, hk * g + row % g);
+    if (p.sink != nullptr) l_sum += sink_term(p.sink, hk * g + row % g, m_used);
+    const float inv_l = l_sum > 0.f ? 1.f / l_sum : 0.f;
 #pragma unroll 1
     for (int c = 0; c < kD; c += 32) {
       uint32_t o[32];

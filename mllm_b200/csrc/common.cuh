@@ -423,6 +423,14 @@ __device__ __forceinline__ float warp_max(float v) {
   return v;
 }
 
+// Activation of the gate half of a gated product whose result is rounded to 16 bits: SiLU, or (GELU) the tanh form of
+// the GELU as v * sigmoid(2 sqrt(2 / pi) (v + 0.044715 v^3)), since 0.5 (1 + tanh(y)) = sigmoid(2 y).
+template <bool GELU>
+__device__ __forceinline__ float gate_act(float v) {
+  if constexpr (GELU) return v / (1.f + __expf(-v * fmaf(0.07135481627f, fminf(v * v, 1e30f), 1.5957691216f)));
+  return v / (1.f + __expf(-v));
+}
+
 // run a statement with T bound to the 16-bit element type named by a DType value
 #define MB200_DISPATCH_HALF(dt, ...)          \
   if ((dt) == ::mb200::kBF16) {               \

@@ -98,7 +98,7 @@ __device__ __forceinline__ uint16_t f_to_half(float v) {
   return *reinterpret_cast<const uint16_t*>(&h);
 }
 
-template <bool F16>
+template <bool F16, bool GELU>
 __global__ void __launch_bounds__(kSmThreads, 1) gemm_smallm_kernel(const SmallMParams p) {
   __shared__ float partial[2][kSmWarps][64];
   extern __shared__ __align__(16) uint8_t smem_dyn[];
@@ -284,7 +284,7 @@ __global__ void __launch_bounds__(kSmThreads, 1) gemm_smallm_kernel(const SmallM
                   for (int w8 = 0; w8 < kSmWarps; ++w8) up += partial[buf][w8][t + 4];
                   const int blk = cu >> 5, q = cu & 31;
                   const int64_t col = static_cast<int64_t>(blk) * 128 + q * 4 + slot;
-                  const float y = (p.swiglu == 2 ? gelu_tanh_f(v) : v / (1.f + __expf(-v))) * up;
+                  const float y = gate_act<GELU>(v) * up;
                   static_cast<uint16_t*>(p.out)[mrow * p.ldc + col] = f_to_half<F16>(y);
                 }
               } else {
@@ -360,14 +360,13 @@ int launch_gemm_smallm(const GemmArgs& a, cudaStream_t s) {
   p.units_per_cta = (p.units + slots - 1) / slots;
   const int grid = (p.units + p.units_per_cta - 1) / p.units_per_cta;
   const int smem = kSmRingBytes + 8 * (2 * a.k + kSmRowPad);
-  cudaError_t err;
-  if (a.dt == kF16) {
-    if (ensure_dynamic_smem(reinterpret_cast<const void*>(gemm_smallm_kernel<true>), kSmRingBytes + 8 * (2 * kSmMaxK + kSmRowPad)) != cudaSuccess) return -3;
-    err = launch_pdl(gemm_smallm_kernel<true>, dim3(grid), dim3(kSmThreads), smem, s, p);
-  } else {
-    if (ensure_dynamic_smem(reinterpret_cast<const void*>(gemm_smallm_kernel<false>), kSmRingBytes + 8 * (2 * kSmMaxK + kSmRowPad)) != cudaSuccess) return -3;
-    err = launch_pdl(gemm_smallm_kernel<false>, dim3(grid), dim3(kSmThreads), smem, s, p);
-  }
+  const bool gelu = a.swiglu == 2;
+  auto go = [&](auto kernel) -> cudaError_t {
+    const cudaError_t set = ensure_dynamic_smem(reinterpret_cast<const void*>(kernel), kSmRingBytes + 8 * (2 * kSmMaxK + kSmRowPad));
+    return set != cudaSuccess ? set : launch_pdl(kernel, dim3(grid), dim3(kSmThreads), smem, s, p);
+  };
+  const cudaError_t err = a.dt == kF16 ? (gelu ? go(gemm_smallm_kernel<true, true>) : go(gemm_smallm_kernel<true, false>))
+                                       : (gelu ? go(gemm_smallm_kernel<false, true>) : go(gemm_smallm_kernel<false, false>));
   note_launch();
   return err == cudaSuccess ? 0 : -4;
 }

@@ -57,7 +57,6 @@ struct KParams {
   int is_int8;
   int row_static;        // swap tiling: the row operand (weights) is not written by earlier kernels of the stream
   int cluster_k;         // swap tiling: > 1 = the k range of a tile is split over the CTAs of a cluster of this size
-  int gate_gelu;         // gated epilogue: GELU (tanh form) of the gate rows instead of SiLU
   int early_trigger;     // swap tiling: let the kernels behind this one start their set-up as soon as this one runs
   uint32_t idesc;
   // ---- tensor-parallel fusion (normal tiling only) ----
@@ -83,10 +82,11 @@ struct KParams {
 constexpr int kStageRowBytes = 144;                      // 128 bytes of output + 16 bytes of padding
 constexpr int kEpiStagingBytes = 4 * 32 * kStageRowBytes;  // four epilogue warps x 32 rows
 
+// SWIGLU: 0 plain product, 1 silu(gate) * up, 2 gelu_tanh(gate) * up.
 // RT = 128-row MMA tiles of the row operand per stage (small-batch tiling only; SwiGLU needs 2: a
 // gate block and its up block), KD = 128-byte K atoms per stage.  Larger stages mean fewer TMA boxes
 // and barrier round trips per byte streamed.
-template <int BN, bool SWAP, bool SWIGLU, int RT, int KD>
+template <int BN, bool SWAP, int SWIGLU, int RT, int KD>
 struct Cfg {
   static constexpr int R = SWAP ? RT : 1;
   static constexpr int kRowTileBytes = kBM * R * kRowBytes;   // 16 KB * R per K atom
@@ -136,9 +136,6 @@ __device__ __forceinline__ void st_cluster_v4f(uint32_t cluster_addr, float a, f
 }
 __device__ __forceinline__ void fence_acq_rel_cluster() { asm volatile("fence.acq_rel.cluster;" ::: "memory"); }
 
-__device__ __forceinline__ float silu_f(float v) { return v / (1.f + __expf(-v)); }
-// activation of the gate rows of a gated epilogue: SiLU, or the tanh form of the GELU
-__device__ __forceinline__ float gate_act(float v, int gelu) { return gelu ? gelu_tanh_f(v) : silu_f(v); }
 
 __device__ __forceinline__ uint32_t pack_out2(float lo, float hi, int out_f16) {
   if (out_f16) {
@@ -161,7 +158,7 @@ __device__ __forceinline__ float acc_to_float(uint32_t raw, int is_int8) {
   return is_int8 ? static_cast<float>(static_cast<int32_t>(raw)) : __uint_as_float(raw);
 }
 
-template <int BN, bool SWAP, bool SWIGLU, int RT, int KD>
+template <int BN, bool SWAP, int SWIGLU, int RT, int KD>
 __global__ void __launch_bounds__(kThreads, SWAP ? 2 : 1)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_constant__ CUtensorMap tm_col,
                     const KParams p) {
@@ -511,7 +508,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
                       x *= sa * p.b_scale[tc * BN + cc];
                       u *= sa * p.b_scale[tc * BN + BN / 2 + cc];
                     }
-                    x = gate_act(x, p.gate_gelu) * u;
+                    x = gate_act<SWIGLU == 2>(x) * u;
                   } else {
                     const int64_t col = col0 + cc;
                     if (p.is_int8 && col < n_out) x *= sa * p.b_scale[col];
@@ -568,7 +565,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
                   x *= sa * p.b_scale[tc * BN + c + v8 * 8 + j];
                   u *= sa * p.b_scale[tc * BN + BN / 2 + c + v8 * 8 + j];
                 }
-                x = gate_act(x, p.gate_gelu) * u;
+                x = gate_act<SWIGLU == 2>(x) * u;
               } else {
                 if (p.is_int8) x *= sa * p.b_scale[col + j];
                 if (p.bias != nullptr) x += load_out1(p.bias, col + j, p.out_f16);
@@ -711,7 +708,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
                       xv *= p.a_scale[j] * p.b_scale[wrow];
                       uv *= p.a_scale[j] * p.b_scale[wrow + kBM];
                     }
-                    xv = gate_act(xv, p.gate_gelu) * uv;
+                    xv = gate_act<SWIGLU == 2>(xv) * uv;
                     ocol = static_cast<int64_t>(tr) * kBM + row_in_tile;
                   } else {
                     if (p.is_int8) xv *= p.a_scale[j] * p.b_scale[wrow];
@@ -762,7 +759,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
                   x *= p.a_scale[mi] * p.b_scale[wrow];
                   u *= p.a_scale[mi] * p.b_scale[wrow + kBM];
                 }
-                x = gate_act(x, p.gate_gelu) * u;
+                x = gate_act<SWIGLU == 2>(x) * u;
                 ocol = static_cast<int64_t>(tr) * kBM + row_in_tile;
               } else {
                 if (p.is_int8) x *= p.a_scale[mi] * p.b_scale[wrow];
@@ -866,7 +863,7 @@ __device__ __forceinline__ void umma_commit_pair(uint32_t bar_cluster_addr) {
                : "memory");
 }
 
-template <bool SWIGLU>
+template <int SWIGLU>
 __global__ void __launch_bounds__(kThreads, 1)
 gemm_pair_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_constant__ CUtensorMap tm_col,
                  const KParams p) {
@@ -1160,7 +1157,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_consta
                 x *= sa * p.b_scale[tc * kPairBN + c + v8 * 8 + j];
                 u *= sa * p.b_scale[tc * kPairBN + kPairBN / 2 + c + v8 * 8 + j];
               }
-              x = gate_act(x, p.gate_gelu) * u;
+              x = gate_act<SWIGLU == 2>(x) * u;
             } else {
               if (p.is_int8) x *= sa * p.b_scale[col + j];
               if (p.bias != nullptr) x += load_out1(p.bias, col + j, p.out_f16);
@@ -1226,7 +1223,7 @@ bool make_operand_map(CUtensorMap* map, const void* base, int64_t rows, int64_t 
   return make_tma_operand_map(map, base, rows, k, ld, elem_bytes, code, box_rows);
 }
 
-template <int BN, bool SWAP, bool SWIGLU, int RT = 1, int KD = 1>
+template <int BN, bool SWAP, int SWIGLU, int RT = 1, int KD = 1>
 int launch_cfg(const CUtensorMap& tr, const CUtensorMap& tc, KParams p, int grid, cudaStream_t s) {
   using C = Cfg<BN, SWAP, SWIGLU, RT, KD>;
   // tuning knob: MLLM_B200_GEMM_STAGES caps the ring depth of the small-batch tiling
@@ -1268,7 +1265,7 @@ int launch_cfg(const CUtensorMap& tr, const CUtensorMap& tc, KParams p, int grid
   return err == cudaSuccess ? 0 : -4;
 }
 
-template <bool SWIGLU>
+template <int SWIGLU>
 int launch_pair_cfg(const CUtensorMap& tr, const CUtensorMap& tc, const KParams& p, int pairs, cudaStream_t s) {
   auto kern = gemm_pair_kernel<SWIGLU>;
   if (ensure_dynamic_smem(reinterpret_cast<const void*>(kern), kPairSmem) != cudaSuccess) return -3;
@@ -1323,7 +1320,6 @@ int launch_gemm(const GemmArgs& a, cudaStream_t s) {
   p.out_f16 = (a.dt == kF16) ? 1 : 0;
   p.is_int8 = a.is_int8;
   p.row_static = a.b_static;
-  p.gate_gelu = a.swiglu == 2 ? 1 : 0;
   {
     // The CTAs of a following small-batch GEMM fit beside ours when both keep their rings short: they are
     // then launched while this kernel still streams, fetch their first weight tiles, and take over the memory
@@ -1373,8 +1369,9 @@ int launch_gemm(const GemmArgs& a, cudaStream_t s) {
       if (!make_operand_map(&tm_row, a.a, a.m, a.k, a.lda, eb, type, kBM)) return -2;
       if (!make_operand_map(&tm_col, a.b, a.n, a.k, a.ldb, eb, type, kPairBN / 2)) return -2;
       const int pairs = static_cast<int>(std::min<int64_t>(tiles_pair, num_sms / 2));
-      return a.swiglu ? launch_pair_cfg<true>(tm_row, tm_col, p, pairs, s)
-                      : launch_pair_cfg<false>(tm_row, tm_col, p, pairs, s);
+      if (a.swiglu == 2) return launch_pair_cfg<2>(tm_row, tm_col, p, pairs, s);
+      return a.swiglu ? launch_pair_cfg<1>(tm_row, tm_col, p, pairs, s)
+                      : launch_pair_cfg<0>(tm_row, tm_col, p, pairs, s);
     }
     // ---- normal tiling: activations are the 128-row operand ----
     int bn = 256;
@@ -1389,9 +1386,10 @@ int launch_gemm(const GemmArgs& a, cudaStream_t s) {
     if (!make_operand_map(&tm_row, a.a, a.m, a.k, a.lda, eb, type, kBM)) return -2;
     if (!make_operand_map(&tm_col, a.b, a.n, a.k, a.ldb, eb, type, bn)) return -2;
     const int grid = std::min(p.tiles_r * p.tiles_c, num_sms);
-    if (a.swiglu) return launch_cfg<256, false, true>(tm_row, tm_col, p, grid, s);
-    if (bn == 256) return launch_cfg<256, false, false>(tm_row, tm_col, p, grid, s);
-    return launch_cfg<128, false, false>(tm_row, tm_col, p, grid, s);
+    if (a.swiglu == 2) return launch_cfg<256, false, 2>(tm_row, tm_col, p, grid, s);
+    if (a.swiglu) return launch_cfg<256, false, 1>(tm_row, tm_col, p, grid, s);
+    if (bn == 256) return launch_cfg<256, false, 0>(tm_row, tm_col, p, grid, s);
+    return launch_cfg<128, false, 0>(tm_row, tm_col, p, grid, s);
   }
 
   // ---- a handful of rows: stream the weights through registers (gemm_smallm.cu) ----
@@ -1465,18 +1463,22 @@ int launch_gemm(const GemmArgs& a, cudaStream_t s) {
   p.max_contrib = contributors(grid);
 #define MB200_SWAP_SMALL(BNV)                                                                       \
   case BNV:                                                                                         \
+    if (a.swiglu == 2)                                                                              \
+      return kd == 2 ? launch_cfg<BNV, true, 2, 2, 2>(tm_row, tm_col, p, grid, s)                   \
+                     : launch_cfg<BNV, true, 2, 2, 1>(tm_row, tm_col, p, grid, s);                  \
     if (a.swiglu)                                                                                   \
-      return kd == 2 ? launch_cfg<BNV, true, true, 2, 2>(tm_row, tm_col, p, grid, s)                \
-                     : launch_cfg<BNV, true, true, 2, 1>(tm_row, tm_col, p, grid, s);               \
+      return kd == 2 ? launch_cfg<BNV, true, 1, 2, 2>(tm_row, tm_col, p, grid, s)                   \
+                     : launch_cfg<BNV, true, 1, 2, 1>(tm_row, tm_col, p, grid, s);                  \
     if (rt == 2)                                                                                    \
-      return kd == 2 ? launch_cfg<BNV, true, false, 2, 2>(tm_row, tm_col, p, grid, s)               \
-                     : launch_cfg<BNV, true, false, 2, 1>(tm_row, tm_col, p, grid, s);              \
-    return kd == 2 ? launch_cfg<BNV, true, false, 1, 2>(tm_row, tm_col, p, grid, s)                 \
-                   : launch_cfg<BNV, true, false, 1, 1>(tm_row, tm_col, p, grid, s);
+      return kd == 2 ? launch_cfg<BNV, true, 0, 2, 2>(tm_row, tm_col, p, grid, s)               \
+                     : launch_cfg<BNV, true, 0, 2, 1>(tm_row, tm_col, p, grid, s);              \
+    return kd == 2 ? launch_cfg<BNV, true, 0, 1, 2>(tm_row, tm_col, p, grid, s)                 \
+                   : launch_cfg<BNV, true, 0, 1, 1>(tm_row, tm_col, p, grid, s);
 #define MB200_SWAP_LARGE(BNV)                                                                       \
   case BNV:                                                                                         \
-    return a.swiglu ? launch_cfg<BNV, true, true, 2, 1>(tm_row, tm_col, p, grid, s)                 \
-                    : launch_cfg<BNV, true, false, 1, 1>(tm_row, tm_col, p, grid, s);
+    if (a.swiglu == 2) return launch_cfg<BNV, true, 2, 2, 1>(tm_row, tm_col, p, grid, s);           \
+    return a.swiglu ? launch_cfg<BNV, true, 1, 2, 1>(tm_row, tm_col, p, grid, s)                    \
+                    : launch_cfg<BNV, true, 0, 1, 1>(tm_row, tm_col, p, grid, s);
   switch (bn) {
     MB200_SWAP_SMALL(16)
     MB200_SWAP_SMALL(32)

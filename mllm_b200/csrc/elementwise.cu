@@ -1,4 +1,4 @@
-// Memory-bound sm_100a kernels: RMSNorm / fused add+RMSNorm, LayerNorm, gated
+// Memory-bound sm_100a kernels: RMSNorm / fused add+RMSNorm, LayerNorm, Dynamic Tanh, gated
 // activations, embedding gather, the fused per-head QK-norm + rotary + KV-cache
 // write, the stand-alone KV write, per-token int8 quantisation and greedy argmax.
 //

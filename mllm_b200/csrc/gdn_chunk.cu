@@ -9,7 +9,7 @@
 //   S_end = exp(G_C) S0 + K^T (exp(G_C - G) * U)
 //
 // Every exponent is of a non-positive number.  The columns of S (the value features) never mix, so a CTA owns one
-// (request, head) and a block of BV value features: grid (128 / BV, heads, batch), 256 threads.  The products
+// (request, head) and a block of BV value features: grid (ceil(Dv / BV), heads, batch), 512 threads.  The products
 // K K^T, Q K^T, K S0, Q S0, P U and K^T U' run on the tensor cores through warp-level MMA on tf32 operands with
 // fp32 accumulation (tiles of 16 x 16 x 8 read from shared memory); the state stays in fp32 in shared memory for
 // the whole sequence and is rounded to tf32 only as an MMA operand.  The unit norms of q and k are row factors, applied

@@ -25,9 +25,9 @@ def show_config() -> dict:
         info["gpu"] = {"name": p.name, "capability": f"{p.major}.{p.minor}", "sms": p.multi_processor_count,
                        "memory_gib": round(p.total_memory / 2 ** 30, 1), "count": torch.cuda.device_count()}
     ext = {}
-    from ._build import load_extension
+    from ._build import cuda_modules, load_extension
 
-    for name in ("mllm_b200_C", "mllm_b200_X"):
+    for name in cuda_modules():
         try:
             ext[name] = load_extension(name) is not None
         except Exception as exc:

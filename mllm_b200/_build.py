@@ -1,11 +1,16 @@
 """Build / load the native extensions in-tree.
 
-Three extensions live under ``mllm_b200/csrc``:
+The extensions live under ``mllm_b200/csrc``:
 
 * ``mllm_b200_C``    — the sm_100a CUDA kernels of every decoder plus their PyTorch binding;
-* ``mllm_b200_X``    — kernels that only some models or layouts use (experts, 4-bit weights, vision towers, tensor- and
-  expert-parallel exchange), loaded, and where it is missing compiled, when one of them is first called;
+* ``mllm_b200_R``    — gated delta rule and latent attention;
+* ``mllm_b200_L``    — lightning attention (linear attention with a fixed decay per head);
+* ``mllm_b200_E``    — mixtures of experts;
+* ``mllm_b200_X``    — 4-bit weights, vision towers, tensor- and expert-parallel exchange;
 * ``mllm_b200_host`` — host-only C++ (radix tree, page allocator, ``.mllm`` file reader).
+
+A CUDA module other than the first is loaded, and where it is missing compiled, when one of its functions is first
+called: a model compiles what it needs.
 
 They are compiled with ``torch.utils.cpp_extension.load`` into ``mllm_b200/_ext`` so the
 shared objects sit beside the package (not in a user cache) and travel with the source
@@ -18,6 +23,7 @@ from __future__ import annotations
 import hashlib
 import importlib.util
 import os
+import re
 import sys
 import threading
 from pathlib import Path
@@ -35,17 +41,33 @@ CUDA_FLAGS = [
 ]
 CXX_FLAGS = ["-O3", "-std=c++17"]
 
+_COMMON = ["bindings_common.h", "common.cuh", "kernels.h", "mma.cuh"]
+
 EXTENSIONS: Dict[str, Dict[str, List[str]]] = {
     "mllm_b200_C": {
-        "sources": ["bindings.cpp", "runtime.cu", "elementwise.cu", "gemm_tcgen05.cu", "gemm_smallm.cu", "attention.cu",
-                    "sampling.cu", "gdn.cu", "gdn_chunk.cu", "latent.cu", "no_alloc.cu"],
-        "headers": ["bindings_common.h", "common.cuh", "kernels.h", "no_alloc.h"],
+        "sources": ["bindings.cpp", "runtime.cu", "elementwise.cu", "row_ops.cu", "gemm_tcgen05.cu", "gemm_smallm.cu", "attention.cu",
+                    "attention_rows.cu", "sampling.cu", "no_alloc.cu"],
+        "headers": _COMMON + ["no_alloc.h"],
+        "cuda": True,
+    },
+    "mllm_b200_R": {
+        "sources": ["bindings_recurrent.cpp", "runtime.cu", "gdn.cu", "gdn_chunk.cu", "latent.cu"],
+        "headers": _COMMON,
+        "cuda": True,
+    },
+    "mllm_b200_L": {
+        "sources": ["bindings_lightning.cpp", "runtime.cu", "lightning.cu"],
+        "headers": _COMMON,
+        "cuda": True,
+    },
+    "mllm_b200_E": {
+        "sources": ["bindings_moe.cpp", "runtime.cu", "moe.cu"],
+        "headers": _COMMON,
         "cuda": True,
     },
     "mllm_b200_X": {
-        "sources": ["bindings_extra.cpp", "runtime.cu", "moe.cu", "comm.cu", "ep_a2a.cu", "gemm_w4a16.cu", "gemm_smallm_w4.cu",
-                    "vision.cu"],
-        "headers": ["bindings_common.h", "common.cuh", "kernels.h"],
+        "sources": ["bindings_extra.cpp", "runtime.cu", "comm.cu", "ep_a2a.cu", "gemm_w4a16.cu", "gemm_smallm_w4.cu", "vision.cu"],
+        "headers": _COMMON,
         "cuda": True,
     },
     "mllm_b200_host": {
@@ -57,6 +79,16 @@ EXTENSIONS: Dict[str, Dict[str, List[str]]] = {
 
 _loaded: Dict[str, ModuleType] = {}
 _lock = threading.Lock()
+
+
+def cuda_modules() -> List[str]:
+    """The CUDA extension modules, the one of every decoder first."""
+    return [n for n, spec in EXTENSIONS.items() if spec["cuda"]]
+
+
+def module_functions(name: str) -> List[str]:
+    """Names of the functions a CUDA module binds, read from its binding source (the first of its sources)."""
+    return re.findall(r'm\.def\("(\w+)"', (_CSRC / EXTENSIONS[name]["sources"][0]).read_text())
 
 
 def _existing(names: List[str]) -> List[Path]:

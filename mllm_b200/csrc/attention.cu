@@ -41,7 +41,7 @@ struct AttnParams {
   const void* q;      // [T, Hq, D] with row stride q_stride (elements)
   const void* k_cache;
   const void* v_cache;
-  void* out;          // [T, Hq, D] contiguous
+  void* out;          // [T, Hq, D] with row stride out_stride (elements), heads of a token contiguous
   float* part_o;      // decode split: [B, Hq, splits, D]
   float* part_lse;    // decode split: [B, Hq, splits]
   const int* req_to_token;
@@ -51,7 +51,7 @@ struct AttnParams {
   int non_causal;          // prefill only: every query row sees the whole sequence
   const int* q_start;      // null in decode
   int* status;
-  int64_t q_stride;
+  int64_t q_stride, out_stride;
   int64_t rtt_stride;
   int64_t num_slots;
   int64_t kv_tok_stride, kv_head_stride;  // elements: row of head h of slot s at s * tok + h * head
@@ -460,7 +460,7 @@ __global__ void __launch_bounds__(kAttnThreads, FwdCfg<NH>::kCtasPerSm) attn_fwd
           l_sum > 0.f ? (m_used + log2f(l_sum)) : -INFINITY;
   } else {
     uint16_t* orow = static_cast<uint16_t*>(p.out) +
-                     (static_cast<int64_t>(q_row0 + q0 + (row_valid ? row_tok : 0)) * p.hq + row_head) * kD;
+                     static_cast<int64_t>(q_row0 + q0 + (row_valid ? row_tok : 0)) * p.out_stride + row_head * kD;
 #pragma unroll 1
     for (int c = 0; c < kD; c += 32) {
       uint32_t o[32];
@@ -643,7 +643,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
       if (tid < g) p.part_lse[(static_cast<int64_t>(b) * p.hq + hk * g + tid) * p.num_splits + split] = -INFINITY;
     } else {
       for (int i = tid; i < g * kD; i += kDecThreads)
-        static_cast<uint16_t*>(p.out)[(static_cast<int64_t>(b) * p.hq + hk * g) * kD + i] = 0;
+        static_cast<uint16_t*>(p.out)[b * p.out_stride + hk * g * kD + i] = 0;
     }
   } else if (warp == 4) {
     // =============================== producer warp ===============================
@@ -927,7 +927,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
           if (p.num_splits > 1) {
             p.part_o[((static_cast<int64_t>(b) * p.hq + head) * p.num_splits + split) * kD + tid] = v;
           } else {
-            const int64_t oi = (static_cast<int64_t>(b) * p.hq + head) * kD + tid;
+            const int64_t oi = b * p.out_stride + head * kD + tid;
             if (p.out_f16)
               static_cast<__half*>(p.out)[oi] = __float2half_rn(v);
             else
@@ -1359,7 +1359,7 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
         if (tok < tpt && tile_q0 + tok < q_len) {
           const uint4 v = *reinterpret_cast<const uint4*>(sP + grp_i * kPfTileBytes + r * 256 + ((chunk ^ (r & 7)) << 4));
           uint16_t* dst = static_cast<uint16_t*>(p.out) +
-                          (static_cast<int64_t>(q_row0 + tile_q0 + tok) * p.hq + hk * g + r % g) * kD + chunk * 8;
+                          static_cast<int64_t>(q_row0 + tile_q0 + tok) * p.out_stride + (hk * g + r % g) * kD + chunk * 8;
           *reinterpret_cast<uint4*>(dst) = v;
         }
       }
@@ -1383,7 +1383,8 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
 // combine decode partials: out[b, h, :] = sum_s w_s * O_s with w_s = 2^(lse_s - max) / sum; a head's sink is one more
 // term of the sum, without a value
 __global__ void attn_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_lse,
-                                  void* __restrict__ out, int hq, int splits, int out_f16, const float* __restrict__ sink) {
+                                  void* __restrict__ out, int64_t out_stride, int hq, int splits, int out_f16,
+                                  const float* __restrict__ sink) {
   pdl_launch_dependents();
   pdl_wait();
   const int b = blockIdx.y, h = blockIdx.x, d = threadIdx.x;
@@ -1404,7 +1405,7 @@ __global__ void attn_merge_kernel(const float* __restrict__ part_o, const float*
     acc += w * part_o[(base + s) * hd + d];
   }
   const float v = den > 0.f ? acc / den : 0.f;
-  const int64_t o = (static_cast<int64_t>(b) * hq + h) * hd + d;
+  const int64_t o = b * out_stride + h * hd + d;
   if (out_f16)
     static_cast<__half*>(out)[o] = __float2half_rn(v);
   else
@@ -1503,6 +1504,8 @@ int launch_attention(const AttnArgs& a, cudaStream_t s) {
   p.q_start = a.q_start;
   p.status = a.status;
   p.q_stride = a.q_stride;
+  p.out_stride = a.out_stride > 0 ? a.out_stride : static_cast<int64_t>(a.hq) * hd;
+  if (p.out_stride % 8 != 0 || (reinterpret_cast<uintptr_t>(a.out) & 15) != 0) return -1;
   p.rtt_stride = a.rtt_stride;
   p.num_slots = a.num_slots;
   p.kv_tok_stride = a.kv_tok_stride;
@@ -1546,7 +1549,7 @@ int launch_attention(const AttnArgs& a, cudaStream_t s) {
     const int rc = nq == 16 ? launch_decode_cfg<16>(p, a, grid, s) : launch_decode_cfg<32>(p, a, grid, s);
     if (rc != 0) return rc;
     if (p.num_splits > 1) {
-      launch_pdl(attn_merge_kernel, dim3(a.hq, a.batch), dim3(kD), 0, s, a.part_o, a.part_lse, a.out, a.hq, p.num_splits, p.out_f16, a.sink);
+      launch_pdl(attn_merge_kernel, dim3(a.hq, a.batch), dim3(kD), 0, s, a.part_o, a.part_lse, a.out, p.out_stride, a.hq, p.num_splits, p.out_f16, a.sink);
       note_launch();
     }
     return cudaGetLastError() == cudaSuccess ? 0 : -4;
@@ -1565,7 +1568,7 @@ int launch_attention(const AttnArgs& a, cudaStream_t s) {
   const int rc = hd == 64 ? launch_fwd_cfg<1>(p, grid, s) : hd == 128 ? launch_fwd_cfg<2>(p, grid, s) : launch_fwd_cfg<4>(p, grid, s);
   if (rc != 0) return rc;
   if (a.is_decode && p.num_splits > 1) {
-    launch_pdl(attn_merge_kernel, dim3(a.hq, a.batch), dim3(hd), 0, s, a.part_o, a.part_lse, a.out, a.hq, p.num_splits, p.out_f16, a.sink);
+    launch_pdl(attn_merge_kernel, dim3(a.hq, a.batch), dim3(hd), 0, s, a.part_o, a.part_lse, a.out, p.out_stride, a.hq, p.num_splits, p.out_f16, a.sink);
     note_launch();
   }
   return cudaGetLastError() == cudaSuccess ? 0 : -4;

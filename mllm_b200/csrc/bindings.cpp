@@ -224,154 +224,6 @@ void apply_penalties(Tensor& logits, const Tensor& counts, const c10::optional<T
                                 logits.size(1), stream_of(logits));
 }
 
-// ---- gated delta net ----
-void check_float(const Tensor& t, const char* name) {
-  check_cuda(t, name);
-  TORCH_CHECK(t.scalar_type() == at::kBFloat16 || t.scalar_type() == at::kHalf || t.scalar_type() == at::kFloat, "mllm_b200: ", name,
-              " must be bf16, fp16 or fp32");
-}
-void check_f32_vec(const Tensor& t, int64_t n, const char* name) {
-  TORCH_CHECK(t.is_cuda() && t.scalar_type() == at::kFloat && t.is_contiguous() && t.numel() == n, "mllm_b200: ", name,
-              " must be a contiguous fp32 device tensor of ", n, " elements");
-}
-
-// x, out [T, H * W] contiguous; gate [T, H * W] with any row stride; w [W]
-void rmsnorm_gated(const Tensor& x, const Tensor& gate, const Tensor& w, Tensor& out, double eps, bool round_norm) {
-  check_float(x, "x");
-  const int64_t width = w.numel();
-  TORCH_CHECK(x.dim() == 2 && x.is_contiguous() && gate.dim() == 2 && gate.sizes() == x.sizes() && gate.stride(1) == 1 &&
-                  out.is_contiguous() && out.sizes() == x.sizes() && x.size(1) % width == 0 && w.is_contiguous() &&
-                  w.scalar_type() == x.scalar_type() && gate.scalar_type() == x.scalar_type() && out.scalar_type() == x.scalar_type(),
-              "rmsnorm_gated: x, gate, out [T, H * W] and weight [W] of one type");
-  c10::cuda::CUDAGuard g(x.device());
-  const int64_t heads = x.size(1) / width;
-  mb200::launch_rmsnorm_gated(x.data_ptr(), gate.data_ptr(), gate.stride(0), w.data_ptr(), out.data_ptr(), x.size(0) * heads, heads,
-                              width, static_cast<float>(eps), round_norm ? 1 : 0, dtype_of(x), stream_of(x));
-}
-
-static void check_ragged(const Tensor& slots, const Tensor& lens, const Tensor& has, const Tensor& q_start) {
-  for (const Tensor* t : {&slots, &lens, &has, &q_start})
-    TORCH_CHECK(t->is_cuda() && t->scalar_type() == at::kInt && t->is_contiguous() && t->numel() == slots.numel(),
-                "ragged metadata: int32 device vectors of one length");
-}
-
-// x [T, C] with any row stride; max_len: longest run of new tokens of a request (0: unknown)
-void gdn_conv1d_silu(const Tensor& x, const Tensor& w, Tensor& conv_state, const Tensor& slots, const Tensor& lens,
-                     const Tensor& has, const Tensor& q_start, Tensor& out, int64_t max_len) {
-  check_float(x, "x");
-  check_ragged(slots, lens, has, q_start);
-  TORCH_CHECK(x.dim() == 2 && x.stride(1) == 1 && out.is_contiguous() && out.sizes() == x.sizes() && w.dim() == 2 &&
-                  w.is_contiguous() && w.size(0) == x.size(1) && conv_state.dim() == 3 && conv_state.is_contiguous() &&
-                  conv_state.size(1) == x.size(1) && conv_state.size(2) == w.size(1) - 1 && out.scalar_type() == x.scalar_type() &&
-                  w.scalar_type() == x.scalar_type() && conv_state.scalar_type() == x.scalar_type(),
-              "gdn_conv1d_silu: x [T, C], w [C, K], conv_state [slots, C, K-1]");
-  c10::cuda::CUDAGuard g(x.device());
-  const int rc = mb200::launch_gdn_conv1d_silu(x.data_ptr(), x.stride(0), w.data_ptr(), conv_state.data_ptr(), slots.data_ptr<int>(),
-                                               lens.data_ptr<int>(), has.data_ptr<int>(), q_start.data_ptr<int>(),
-                                               out.data_ptr(), slots.numel(), max_len > 0 ? std::min<int64_t>(max_len, x.size(0)) : x.size(0),
-                                               x.size(1), w.size(1), dtype_of(x), stream_of(x));
-  TORCH_CHECK(rc == 0, "gdn_conv1d_silu: unsupported kernel width");
-}
-
-// b, a [T, H] with one row stride -> g, beta fp32 [T, H]
-void gdn_gates(const Tensor& b, const Tensor& a, const Tensor& a_log, const Tensor& dt_bias, Tensor& g, Tensor& beta) {
-  check_float(b, "b");
-  TORCH_CHECK(b.dim() == 2 && a.sizes() == b.sizes() && b.stride(1) == 1 && a.strides() == b.strides() &&
-                  a.scalar_type() == b.scalar_type(),
-              "gdn_gates: b, a [T, H] of one layout");
-  check_f32_vec(a_log, b.size(1), "a_log");
-  check_f32_vec(dt_bias, b.size(1), "dt_bias");
-  check_f32_vec(g, b.numel(), "g");
-  check_f32_vec(beta, b.numel(), "beta");
-  c10::cuda::CUDAGuard gd(b.device());
-  mb200::launch_gdn_gates(b.data_ptr(), a.data_ptr(), b.stride(0), a_log.data_ptr<float>(), dt_bias.data_ptr<float>(),
-                          g.data_ptr<float>(), beta.data_ptr<float>(), b.size(0), b.size(1), dtype_of(b), stream_of(b));
-}
-
-static mb200::GdnRuleParams rule_params(const Tensor& q, const Tensor& k, const Tensor& v, Tensor& state, const Tensor& slots,
-                                        const Tensor& lens, const Tensor& has, const Tensor& q_start, Tensor& out) {
-  check_float(q, "q");
-  check_ragged(slots, lens, has, q_start);
-  for (const Tensor* t : {&q, &k, &v})
-    TORCH_CHECK(t->dim() == 3 && t->stride(2) == 1 && t->stride(1) == t->size(2) && t->size(0) == q.size(0) &&
-                    t->scalar_type() == q.scalar_type(),
-                "gated delta rule: q, k [T, Hk, Dk], v [T, H, Dv] of one type, heads of a token contiguous");
-  TORCH_CHECK(k.sizes() == q.sizes() && v.size(1) % q.size(1) == 0 && out.is_contiguous() && out.sizes() == v.sizes() &&
-                  out.scalar_type() == q.scalar_type() && state.scalar_type() == at::kFloat && state.is_contiguous() &&
-                  state.dim() == 4 && state.size(1) == v.size(1) && state.size(2) == q.size(2) && state.size(3) == v.size(2),
-              "gated delta rule: out [T, H, Dv], state fp32 [slots, H, Dk, Dv], H a multiple of Hk");
-  mb200::GdnRuleParams p{};
-  p.q = q.data_ptr();
-  p.k = k.data_ptr();
-  p.v = v.data_ptr();
-  p.out = out.data_ptr();
-  p.state = state.data_ptr<float>();
-  p.slots = slots.data_ptr<int>();
-  p.lens = lens.data_ptr<int>();
-  p.has_state = has.data_ptr<int>();
-  p.q_start = q_start.data_ptr<int>();
-  p.q_ld = q.stride(0);
-  p.k_ld = k.stride(0);
-  p.v_ld = v.stride(0);
-  p.batch = slots.numel();
-  p.heads = v.size(1);
-  p.k_heads = q.size(1);
-  p.dk = q.size(2);
-  p.dv = v.size(2);
-  p.dt = dtype_of(q);
-  return p;
-}
-
-static void set_gates(mb200::GdnRuleParams& p, const Tensor& g, const Tensor& beta, int64_t tokens) {
-  check_f32_vec(g, tokens * p.heads, "g");
-  check_f32_vec(beta, tokens * p.heads, "beta");
-  p.g = g.data_ptr<float>();
-  p.beta = beta.data_ptr<float>();
-}
-
-void gdn_recurrent(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& g, const Tensor& beta, Tensor& state,
-                   const Tensor& slots, const Tensor& lens, const Tensor& has, const Tensor& q_start, Tensor& out) {
-  mb200::GdnRuleParams p = rule_params(q, k, v, state, slots, lens, has, q_start, out);
-  set_gates(p, g, beta, q.size(0));
-  c10::cuda::CUDAGuard gd(q.device());
-  const int rc = mb200::launch_gdn_recurrent(p, stream_of(q));
-  TORCH_CHECK(rc == 0, "gdn_recurrent: unsupported head size (code ", rc, ")");
-}
-
-// the same with the gates computed inside from the raw projections b, a [T, H]
-void gdn_recurrent_raw(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& b, const Tensor& a, const Tensor& a_log,
-                       const Tensor& dt_bias, Tensor& state, const Tensor& slots, const Tensor& lens, const Tensor& has,
-                       const Tensor& q_start, Tensor& out) {
-  mb200::GdnRuleParams p = rule_params(q, k, v, state, slots, lens, has, q_start, out);
-  TORCH_CHECK(b.is_cuda() && b.dim() == 2 && b.size(0) == q.size(0) && b.size(1) == p.heads && a.sizes() == b.sizes() &&
-                  b.stride(1) == 1 && a.strides() == b.strides() && b.scalar_type() == q.scalar_type() &&
-                  a.scalar_type() == q.scalar_type(),
-              "gdn_recurrent_raw: b, a [T, H] of one layout");
-  check_f32_vec(a_log, p.heads, "a_log");
-  check_f32_vec(dt_bias, p.heads, "dt_bias");
-  p.b_raw = b.data_ptr();
-  p.a_raw = a.data_ptr();
-  p.gate_ld = b.stride(0);
-  p.a_log = a_log.data_ptr<float>();
-  p.dt_bias = dt_bias.data_ptr<float>();
-  c10::cuda::CUDAGuard gd(q.device());
-  const int rc = mb200::launch_gdn_recurrent(p, stream_of(q));
-  TORCH_CHECK(rc == 0, "gdn_recurrent_raw: unsupported head size (code ", rc, ")");
-}
-
-// Returns 1 (nothing launched) when the shape is not the chunk kernel's.
-int64_t gdn_chunk(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& g, const Tensor& beta, Tensor& state,
-                  const Tensor& slots, const Tensor& lens, const Tensor& has, const Tensor& q_start, Tensor& out, bool split_tf32) {
-  mb200::GdnRuleParams p = rule_params(q, k, v, state, slots, lens, has, q_start, out);
-  set_gates(p, g, beta, q.size(0));
-  p.split_tf32 = split_tf32 ? 1 : 0;
-  if (!mb200::gdn_chunk_covers(p)) return 1;
-  c10::cuda::CUDAGuard gd(q.device());
-  const int rc = mb200::launch_gdn_chunk(p, device_state(q.get_device()).num_sms, stream_of(q));
-  TORCH_CHECK(rc == 0, "gdn_chunk: launch failed (code ", rc, ")");
-  return 0;
-}
-
 // ---- fp32 residual stream, Dynamic Tanh ----
 void residual_dyt(Tensor& x, const c10::optional<Tensor>& y, double mult, const Tensor& alpha, const Tensor& w, const Tensor& b,
                   Tensor& h) {
@@ -390,121 +242,202 @@ void residual_dyt(Tensor& x, const c10::optional<Tensor>& y, double mult, const 
                              dtype_of(h), stream_of(x));
 }
 
-void embedding_f32(const Tensor& ids, const Tensor& table, Tensor& out) {
+void embedding_f32(const Tensor& ids, const Tensor& table, double scale, Tensor& out, c10::optional<Tensor> h) {
   check_float(table, "table");
   TORCH_CHECK(ids.is_cuda() && ids.scalar_type() == at::kLong && ids.is_contiguous() && table.dim() == 2 && table.is_contiguous() &&
                   out.is_contiguous() && out.scalar_type() == at::kFloat && out.numel() == ids.numel() * table.size(1),
               "embedding_f32: int64 ids, contiguous table, fp32 out");
+  if (h.has_value())
+    TORCH_CHECK(h->is_contiguous() && h->scalar_type() == table.scalar_type() && h->numel() == out.numel(), "embedding_f32: h");
   c10::cuda::CUDAGuard g(table.device());
   auto& st = device_state(table.get_device());
-  mb200::launch_embedding_f32(ids.data_ptr<int64_t>(), table.data_ptr(), out.data_ptr<float>(), ids.numel(), table.size(1),
-                              table.size(0), dtype_of(table), st.status.data_ptr<int>(), stream_of(table));
+  mb200::launch_embedding_f32(ids.data_ptr<int64_t>(), table.data_ptr(), static_cast<float>(scale), out.data_ptr<float>(),
+                              h.has_value() ? h->data_ptr() : nullptr, ids.numel(), table.size(1), table.size(0), dtype_of(table),
+                              st.status.data_ptr<int>(), stream_of(table));
 }
 
-// ---- latent attention ----
-// y [T, q_rank (+ kv_rank)]; cq [T, q_rank]; cache [slots, kv_rank] and loc only when the layer writes latents
-void latent_prologue(const Tensor& y, const Tensor& q_w, const c10::optional<Tensor>& kv_w, double eps, Tensor& cq,
-                     const c10::optional<Tensor>& loc, c10::optional<Tensor> cache) {
-  check_float(y, "y");
-  const int64_t q_rank = q_w.numel(), kv_rank = kv_w.has_value() ? kv_w->numel() : 0;
-  TORCH_CHECK(y.dim() == 2 && y.stride(1) == 1 && y.size(1) >= q_rank + kv_rank && cq.is_contiguous() && cq.dim() == 2 &&
-                  cq.size(0) == y.size(0) && cq.size(1) == q_rank && cq.scalar_type() == y.scalar_type(),
-              "latent_prologue: y [T, q_rank + kv_rank], cq [T, q_rank]");
-  check_f32_vec(q_w, q_rank, "q_w");
-  if (kv_rank > 0) {
-    check_f32_vec(*kv_w, kv_rank, "kv_w");
-    TORCH_CHECK(loc.has_value() && cache.has_value() && loc->is_cuda() && loc->scalar_type() == at::kLong && loc->is_contiguous() &&
-                    loc->numel() == y.size(0) && cache->dim() == 2 && cache->stride(1) == 1 && cache->size(1) == kv_rank &&
-                    cache->scalar_type() == y.scalar_type(),
-                "latent_prologue: loc int64 [T], cache [slots, kv_rank]");
+// x [T, W] fp32 (updated in place when `update`), y [T, W] or none, ls / w fp32 [W], h [T, W].  experts: (expert rows
+// [P, W], sorted_pos [T * top], topk_w [T, top], ids [T, top], token_in [T, W]) or empty
+void post_norm(Tensor& x, const c10::optional<Tensor>& y, const c10::optional<Tensor>& ls, double alpha, const Tensor& w, double eps,
+               Tensor& h, bool update, const std::vector<Tensor>& experts, int64_t identity_from) {
+  check_float(h, "h");
+  TORCH_CHECK(x.is_cuda() && x.scalar_type() == at::kFloat && x.dim() == 2 && x.is_contiguous() && h.is_contiguous() &&
+                  h.sizes() == x.sizes(),
+              "post_norm: x fp32 [T, W], h [T, W]");
+  const int64_t T = x.size(0), W = x.size(1);
+  check_f32_vec(w, W, "w");
+  if (ls.has_value()) check_f32_vec(*ls, W, "ls");
+  if (y.has_value())
+    TORCH_CHECK(y->is_cuda() && y->is_contiguous() && y->sizes() == x.sizes() && y->scalar_type() == h.scalar_type(), "post_norm: y [T, W]");
+  mb200::PostNormArgs a{};
+  if (!experts.empty()) {
+    TORCH_CHECK(experts.size() == 5, "post_norm: expert_rows, sorted_pos, topk_w, ids, token_in");
+    const Tensor &rows = experts[0], &pos = experts[1], &tw = experts[2], &ids = experts[3], &in = experts[4];
+    TORCH_CHECK(rows.is_cuda() && rows.is_contiguous() && rows.dim() == 2 && rows.size(1) == W && rows.scalar_type() == h.scalar_type() &&
+                    tw.is_cuda() && tw.scalar_type() == at::kFloat && tw.is_contiguous() && tw.dim() == 2 && tw.size(0) == T &&
+                    tw.size(1) <= 32 && pos.is_cuda() && pos.scalar_type() == at::kInt && pos.is_contiguous() &&
+                    pos.numel() >= tw.numel() && ids.is_cuda() && ids.scalar_type() == at::kInt && ids.is_contiguous() &&
+                    ids.sizes() == tw.sizes() && in.is_cuda() && in.is_contiguous() && in.sizes() == x.sizes() &&
+                    in.scalar_type() == h.scalar_type(),
+                "post_norm: expert tensors");
+    a.expert_rows = rows.data_ptr();
+    a.sorted_pos = pos.data_ptr<int>();
+    a.topk_w = tw.data_ptr<float>();
+    a.ids = ids.data_ptr<int>();
+    a.token_in = in.data_ptr();
+    a.top = tw.size(1);
+    a.identity_from = identity_from;
   }
-  c10::cuda::CUDAGuard g(y.device());
-  auto& st = device_state(y.get_device());
-  mb200::launch_latent_prologue(y.data_ptr(), y.stride(0), y.size(0), q_rank, kv_rank, q_w.data_ptr<float>(),
-                                kv_rank > 0 ? kv_w->data_ptr<float>() : nullptr, static_cast<float>(eps), cq.data_ptr(),
-                                kv_rank > 0 ? loc->data_ptr<int64_t>() : nullptr, kv_rank > 0 ? cache->data_ptr() : nullptr,
-                                kv_rank > 0 ? cache->stride(0) : 0, kv_rank > 0 ? cache->size(0) : 0, dtype_of(y),
-                                st.status.data_ptr<int>(), stream_of(y));
-}
-
-void latent_gather(const Tensor& cache, const Tensor& req_to_token, const Tensor& req, const Tensor& lens, const Tensor& start,
-                   int64_t max_len, Tensor& out) {
-  check_float(cache, "cache");
-  for (const Tensor* t : {&req_to_token, &req, &lens, &start})
-    TORCH_CHECK(t->scalar_type() == at::kInt && t->is_cuda(), "latent_gather: index tensors must be int32 CUDA tensors");
-  TORCH_CHECK(cache.dim() == 2 && cache.stride(1) == 1 && req_to_token.dim() == 2 && req_to_token.stride(1) == 1 &&
-                  max_len <= req_to_token.size(1) && req.numel() == lens.numel() && req.numel() == start.numel() &&
-                  out.is_contiguous() && out.dim() == 2 && out.size(1) == cache.size(1) && out.scalar_type() == cache.scalar_type(),
-              "latent_gather: cache [slots, rank], out [rows, rank]");
-  c10::cuda::CUDAGuard g(cache.device());
-  auto& st = device_state(cache.get_device());
-  mb200::launch_latent_gather(cache.data_ptr(), cache.stride(0), cache.size(1), cache.element_size(), req_to_token.data_ptr<int>(),
-                              req_to_token.stride(0), req.data_ptr<int>(), lens.data_ptr<int>(), start.data_ptr<int>(), req.numel(),
-                              max_len, out.data_ptr(), cache.size(0), st.status.data_ptr<int>(), stream_of(cache));
-}
-
-// out[t, h, :] = w[h] x[t, h, :].  Returns non-zero (nothing launched) when the shape is not the kernel's.
-int64_t head_linear(const Tensor& x, const Tensor& w, Tensor& out) {
-  check_float(x, "x");
-  TORCH_CHECK(x.dim() == 3 && x.stride(2) == 1 && w.dim() == 3 && w.is_contiguous() && w.size(0) == x.size(1) &&
-                  w.size(2) == x.size(2) && out.dim() == 3 && out.stride(2) == 1 && out.size(0) == x.size(0) &&
-                  out.size(1) == x.size(1) && out.size(2) == w.size(1) && w.scalar_type() == x.scalar_type() &&
-                  out.scalar_type() == x.scalar_type(),
-              "head_linear: x [T, H, K], w [H, N, K], out [T, H, N]");
-  if ((reinterpret_cast<uintptr_t>(x.data_ptr()) | reinterpret_cast<uintptr_t>(w.data_ptr())) & 15) return 1;
   c10::cuda::CUDAGuard g(x.device());
-  return mb200::launch_head_linear(x.data_ptr(), x.stride(0), x.stride(1), w.data_ptr(), out.data_ptr(), out.stride(0), out.stride(1),
-                                   x.size(0), x.size(1), w.size(1), w.size(2), device_state(x.get_device()).num_sms, dtype_of(x),
-                                   stream_of(x));
+  a.x = x.data_ptr<float>();
+  a.x_out = update ? x.data_ptr<float>() : nullptr;
+  a.y = y.has_value() ? y->data_ptr() : nullptr;
+  a.ls = ls.has_value() ? ls->data_ptr<float>() : nullptr;
+  a.w = w.data_ptr<float>();
+  a.h = h.data_ptr();
+  a.rows = T;
+  a.width = W;
+  a.alpha = static_cast<float>(alpha);
+  a.eps = static_cast<float>(eps);
+  a.dt = dtype_of(h);
+  const int rc = mb200::launch_post_norm(a, stream_of(x));
+  TORCH_CHECK(rc == 0, "post_norm: row too wide or too many choices (code ", rc, ")");
 }
 
-// q, out [rows, H, R]; cache [slots, R]; row_req int32, row_pos int64 [rows]; max_seq_len sizes the split of the context
-void latent_attention(const Tensor& q, const Tensor& cache, const Tensor& req_to_token, const Tensor& row_req, const Tensor& row_pos,
-                      double scale, const c10::optional<Tensor>& sink, Tensor& out, int64_t max_seq_len) {
+// x [T, W] contiguous, gate and out [T, W] with any row stride, w fp32 [W]
+void rmsnorm_sigmoid_gate(const Tensor& x, const Tensor& gate, const Tensor& w, Tensor& out, double eps) {
+  check_float(x, "x");
+  TORCH_CHECK(x.dim() == 2 && x.is_contiguous() && gate.sizes() == x.sizes() && gate.stride(1) == 1 && out.sizes() == x.sizes() &&
+                  out.stride(1) == 1 && gate.scalar_type() == x.scalar_type() && out.scalar_type() == x.scalar_type() &&
+                  gate.is_cuda() && out.is_cuda(),
+              "rmsnorm_sigmoid_gate: x, gate, out [T, W] of one type");
+  check_f32_vec(w, x.size(1), "w");
+  c10::cuda::CUDAGuard g(x.device());
+  const int rc = mb200::launch_rmsnorm_sigmoid_gate(x.data_ptr(), gate.data_ptr(), gate.stride(0), w.data_ptr<float>(), out.data_ptr(),
+                                                    out.stride(0), x.size(0), x.size(1), static_cast<float>(eps), dtype_of(x), stream_of(x));
+  TORCH_CHECK(rc == 0, "rmsnorm_sigmoid_gate: row too wide (code ", rc, ")");
+}
+
+// row [T, >= (heads + kv_heads) * dim + kv_heads * vdim]; q_out [T, heads, q_width]; caches [slots, kv_heads, >= width]
+void rownorm_rope_kv(const Tensor& row, const Tensor& q_w, const Tensor& k_w, const Tensor& inv_freq, const Tensor& positions,
+                     const Tensor& loc, Tensor& q_out, Tensor& k_cache, Tensor& v_cache, int64_t heads, int64_t kv_heads, int64_t dim,
+                     int64_t vdim, double eps) {
+  check_float(row, "row");
+  const int64_t T = row.size(0);
+  TORCH_CHECK(row.dim() == 2 && row.stride(1) == 1 && row.size(1) >= (heads + kv_heads) * dim + kv_heads * vdim &&
+                  q_out.is_contiguous() && q_out.dim() == 3 && q_out.size(0) == T && q_out.size(1) == heads && q_out.size(2) >= dim &&
+                  q_out.scalar_type() == row.scalar_type(),
+              "rownorm_rope_kv: row [T, q | k | v], q_out [T, heads, >= dim]");
+  check_f32_vec(q_w, heads * dim, "q_w");
+  check_f32_vec(k_w, kv_heads * dim, "k_w");
+  for (const Tensor* t : {&k_cache, &v_cache})
+    TORCH_CHECK(t->is_cuda() && t->dim() == 3 && t->stride(2) == 1 && t->size(1) == kv_heads && t->scalar_type() == row.scalar_type() &&
+                    t->size(0) == k_cache.size(0),
+                "rownorm_rope_kv: caches [slots, kv_heads, width] of the rows' type");
+  TORCH_CHECK(k_cache.size(2) >= dim && v_cache.size(2) >= vdim && positions.is_cuda() && positions.scalar_type() == at::kLong &&
+                  positions.is_contiguous() && positions.numel() == T && loc.is_cuda() && loc.scalar_type() == at::kLong &&
+                  loc.is_contiguous() && loc.numel() == T && inv_freq.is_cuda() && inv_freq.scalar_type() == at::kDouble &&
+                  inv_freq.is_contiguous(),
+              "rownorm_rope_kv: int64 positions and slots [T], fp64 frequencies");
+  c10::cuda::CUDAGuard g(row.device());
+  mb200::RowNormRopeArgs a{};
+  a.row = row.data_ptr();
+  a.q_w = q_w.data_ptr<float>();
+  a.k_w = k_w.data_ptr<float>();
+  a.inv_freq = inv_freq.data_ptr<double>();
+  a.positions = positions.data_ptr<int64_t>();
+  a.loc = loc.data_ptr<int64_t>();
+  a.q_out = q_out.data_ptr();
+  a.k_cache = k_cache.data_ptr();
+  a.v_cache = v_cache.data_ptr();
+  a.status = device_state(row.get_device()).status.data_ptr<int>();
+  a.row_ld = row.stride(0);
+  a.k_tok_stride = k_cache.stride(0);
+  a.k_head_stride = k_cache.stride(1);
+  a.v_tok_stride = v_cache.stride(0);
+  a.v_head_stride = v_cache.stride(1);
+  a.num_slots = k_cache.size(0);
+  a.tokens = T;
+  a.heads = heads;
+  a.kv_heads = kv_heads;
+  a.dim = dim;
+  a.vdim = vdim;
+  a.q_width = q_out.size(2);
+  a.rot_dims = 2 * inv_freq.numel();
+  a.eps = static_cast<float>(eps);
+  a.dt = dtype_of(row);
+  const int rc = mb200::launch_rownorm_rope_kv(a, stream_of(row));
+  TORCH_CHECK(rc == 0, "rownorm_rope_kv: unsupported sizes (code ", rc, ")");
+}
+
+// out fp32 [T, W] = cap * tanh(x / cap)
+void soft_cap(const Tensor& x, Tensor& out, double cap) {
+  check_float(x, "x");
+  TORCH_CHECK(x.dim() == 2 && x.stride(1) == 1 && out.is_contiguous() && out.sizes() == x.sizes() && out.scalar_type() == at::kFloat &&
+                  out.is_cuda() && cap > 0,
+              "soft_cap: x [T, W], fp32 out, cap > 0");
+  c10::cuda::CUDAGuard g(x.device());
+  mb200::launch_soft_cap(x.data_ptr(), x.stride(0), out.data_ptr<float>(), x.size(0), x.size(1), static_cast<float>(cap), dtype_of(x),
+                         stream_of(x));
+}
+
+void relu_squared(Tensor& x) {
+  check_float(x, "x");
+  TORCH_CHECK(x.is_contiguous(), "relu_squared: contiguous");
+  c10::cuda::CUDAGuard g(x.device());
+  mb200::launch_relu_squared(x.data_ptr(), x.numel(), dtype_of(x), stream_of(x));
+}
+
+// q [rows, H, D] and out [rows, H, Dv] with any row stride; caches [slots, G, D / Dv]
+void attention_rows(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& req_to_token, const Tensor& row_req,
+                    const Tensor& row_pos, double scale, Tensor& out, int64_t window, double logit_cap, const c10::optional<Tensor>& sink) {
   check_float(q, "q");
-  TORCH_CHECK(q.dim() == 3 && q.is_contiguous() && out.is_contiguous() && out.sizes() == q.sizes() &&
-                  out.scalar_type() == q.scalar_type() && cache.dim() == 2 && cache.stride(1) == 1 && cache.size(1) == q.size(2) &&
-                  cache.scalar_type() == q.scalar_type() && cache.is_cuda() && q.size(2) <= 1024 && q.size(0) <= 65535,
-              "latent_attention: q, out [rows <= 65535, H, R <= 1024], cache [slots, R] of one type");
-  TORCH_CHECK(req_to_token.is_cuda() && req_to_token.scalar_type() == at::kInt && req_to_token.dim() == 2 &&
-                  req_to_token.stride(1) == 1 && row_req.is_cuda() && row_req.scalar_type() == at::kInt && row_req.is_contiguous() &&
-                  row_req.numel() == q.size(0) && row_pos.is_cuda() && row_pos.scalar_type() == at::kLong &&
-                  row_pos.is_contiguous() && row_pos.numel() == q.size(0),
-              "latent_attention: row_req int32 [rows], row_pos int64 [rows]");
+  TORCH_CHECK(q.dim() == 3 && q.stride(2) == 1 && q.stride(1) == q.size(2) && out.dim() == 3 && out.stride(2) == 1 &&
+                  out.stride(1) == out.size(2) && out.size(0) == q.size(0) && out.size(1) == q.size(1) &&
+                  out.scalar_type() == q.scalar_type() && out.is_cuda(),
+              "attention_rows: q [rows, H, D], out [rows, H, Dv]");
+  for (const Tensor* t : {&k_cache, &v_cache})
+    TORCH_CHECK(t->is_cuda() && t->dim() == 3 && t->stride(2) == 1 && t->scalar_type() == q.scalar_type() &&
+                    t->size(0) == k_cache.size(0) && t->size(1) == k_cache.size(1),
+                "attention_rows: caches [slots, G, width] of q's type");
+  TORCH_CHECK(k_cache.size(2) == q.size(2) && v_cache.size(2) == out.size(2) && req_to_token.is_cuda() &&
+                  req_to_token.scalar_type() == at::kInt && req_to_token.dim() == 2 && req_to_token.stride(1) == 1 && row_req.is_cuda() &&
+                  row_req.scalar_type() == at::kInt && row_req.is_contiguous() && row_req.numel() == q.size(0) && row_pos.is_cuda() &&
+                  row_pos.scalar_type() == at::kLong && row_pos.is_contiguous() && row_pos.numel() == q.size(0),
+              "attention_rows: row_req int32 [rows], row_pos int64 [rows]");
   c10::cuda::CUDAGuard g(q.device());
-  auto& st = device_state(q.get_device());
-  mb200::LatentAttnArgs a{};
-  a.rows = q.size(0);
-  a.heads = q.size(1);
-  a.rank = q.size(2);
-  a.cache_ld = cache.stride(0);
-  a.dt = dtype_of(q);
-  if (sink.has_value()) {
-    check_f32_vec(*sink, a.heads, "sink");
-    a.sink = sink->data_ptr<float>();
-  }
-  a.splits = mb200::latent_mma_covers(a.rank, a.cache_ld, a.dt)
-                 ? mb200::latent_num_splits(a.rows, a.heads, max_seq_len > 0 ? max_seq_len : req_to_token.size(1), st.num_sms)
-                 : 1;
-  Tensor part_o, part_lse;
-  if (a.splits > 1) {
-    part_o = torch::empty({a.rows, a.heads, a.splits, a.rank}, q.options().dtype(torch::kFloat32));
-    part_lse = torch::empty({a.rows, a.heads, a.splits}, q.options().dtype(torch::kFloat32));
-    a.part_o = part_o.data_ptr<float>();
-    a.part_lse = part_lse.data_ptr<float>();
-  }
+  mb200::RowAttnArgs a{};
   a.q = q.data_ptr();
-  a.cache = cache.data_ptr();
+  a.k_cache = k_cache.data_ptr();
+  a.v_cache = v_cache.data_ptr();
   a.out = out.data_ptr();
   a.req_to_token = req_to_token.data_ptr<int>();
   a.row_req = row_req.data_ptr<int>();
   a.row_pos = row_pos.data_ptr<int64_t>();
-  a.status = st.status.data_ptr<int>();
+  a.heads = q.size(1);
+  if (sink.has_value()) {
+    check_f32_vec(*sink, a.heads, "sink");
+    a.sink = sink->data_ptr<float>();
+  }
+  a.status = device_state(q.get_device()).status.data_ptr<int>();
+  a.q_stride = q.stride(0);
+  a.out_stride = out.stride(0);
   a.rtt_stride = req_to_token.stride(0);
-  a.num_slots = cache.size(0);
+  a.num_slots = k_cache.size(0);
+  a.k_tok_stride = k_cache.stride(0);
+  a.k_head_stride = k_cache.stride(1);
+  a.v_tok_stride = v_cache.stride(0);
+  a.v_head_stride = v_cache.stride(1);
+  a.rows = q.size(0);
+  a.kv_heads = k_cache.size(1);
+  a.dim = q.size(2);
+  a.vdim = out.size(2);
+  a.window = static_cast<int>(window);
   a.scale = static_cast<float>(scale);
-  const int rc = mb200::launch_latent_attention(a, stream_of(q));
-  TORCH_CHECK(rc == 0, "latent_attention: unsupported configuration (code ", rc, ")");
+  a.logit_cap = static_cast<float>(logit_cap);
+  a.dt = dtype_of(q);
+  const int rc = mb200::launch_attention_rows(a, stream_of(q));
+  TORCH_CHECK(rc == 0, "attention_rows: unsupported sizes (code ", rc, ")");
 }
 
 // out = a @ b^T (+bias) (+residual) | swiglu.  a [M,K], b [N,K].
@@ -537,7 +470,7 @@ int64_t gemm_impl(const Tensor& a, const Tensor& b, Tensor& out, const c10::opti
                   out.stride(1) == 1,
               "gemm: 2-D row-major operands");
   TORCH_CHECK(a.size(1) == b.size(1) && a.scalar_type() == b.scalar_type(), "gemm: K / dtype mismatch");
-  TORCH_CHECK(out.size(0) == a.size(0) && out.size(1) == (swiglu ? b.size(0) / 2 : b.size(0)), "gemm: out shape");
+  TORCH_CHECK(out.size(0) == a.size(0) && out.size(1) == (swiglu == 1 || swiglu == 2 ? b.size(0) / 2 : b.size(0)), "gemm: out shape");
   if (is_int8) {
     TORCH_CHECK(a_scale.has_value() && b_scale.has_value(), "gemm: int8 needs scales");
     TORCH_CHECK(a_scale->scalar_type() == at::kFloat && b_scale->scalar_type() == at::kFloat &&
@@ -572,7 +505,7 @@ int64_t gemm_impl(const Tensor& a, const Tensor& b, Tensor& out, const c10::opti
   args.ldb = b.stride(0);
   args.ldc = out.stride(0);
   args.ld_res = residual.has_value() ? residual->stride(0) : 0;
-  args.swiglu = static_cast<int>(swiglu);   // 1: SiLU gate, 2: GELU (tanh form) gate
+  args.swiglu = static_cast<int>(swiglu);   // 1: SiLU gate, 2: GELU (tanh form) gate, 3: square of relu
   args.dt = dtype_of(out);
   args.is_int8 = is_int8 ? 1 : 0;
   args.workspace = st.workspace.data_ptr<float>();
@@ -691,7 +624,9 @@ void attention_prefill(const Tensor& q, const Tensor& k_cache, const Tensor& v_c
   TORCH_CHECK(q.dim() == 3, "q must be [T,Hq,D]");
   const int64_t hd = q.size(2);
   TORCH_CHECK((hd == 64 || hd == 128 || hd == 256) && q.stride(2) == 1 && q.stride(1) == hd, "q must be [T,Hq,D], D 64, 128 or 256");
-  TORCH_CHECK(out.is_contiguous() && out.sizes() == q.sizes() && out.scalar_type() == q.scalar_type(), "out");
+  TORCH_CHECK(out.dim() == 3 && out.stride(2) == 1 && out.stride(1) == hd && out.sizes() == q.sizes() &&
+                  out.scalar_type() == q.scalar_type(),
+              "out must be [T,Hq,D], heads of a token contiguous");
   const int kv_fmt = check_kv_cache(k_cache, v_cache, q.scalar_type(), k_cache.size(1), hd);
   for (const Tensor* t : {&req_to_token, &req_pool_indices, &seq_lens, &prefix_lens, &q_start})
     TORCH_CHECK(t->scalar_type() == at::kInt && t->is_cuda(), "index tensors must be int32 CUDA tensors");
@@ -712,6 +647,7 @@ void attention_prefill(const Tensor& q, const Tensor& k_cache, const Tensor& v_c
   a.q_start = q_start.data_ptr<int>();
   a.status = st.status.data_ptr<int>();
   a.q_stride = q.stride(0);
+  a.out_stride = out.stride(0);
   a.rtt_stride = req_to_token.stride(0);
   a.num_slots = k_cache.size(0);
   a.batch = req_pool_indices.numel();
@@ -739,7 +675,9 @@ void attention_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_ca
   TORCH_CHECK(q.dim() == 3, "q must be [B,Hq,D]");
   const int64_t hd = q.size(2);
   TORCH_CHECK((hd == 64 || hd == 128 || hd == 256) && q.stride(2) == 1 && q.stride(1) == hd, "q must be [B,Hq,D], D 64, 128 or 256");
-  TORCH_CHECK(out.is_contiguous() && out.sizes() == q.sizes() && out.scalar_type() == q.scalar_type(), "out");
+  TORCH_CHECK(out.dim() == 3 && out.stride(2) == 1 && out.stride(1) == hd && out.sizes() == q.sizes() &&
+                  out.scalar_type() == q.scalar_type(),
+              "out must be [T,Hq,D], heads of a token contiguous");
   const int kv_fmt = check_kv_cache(k_cache, v_cache, q.scalar_type(), k_cache.size(1), hd);
   for (const Tensor* t : {&req_to_token, &req_pool_indices, &seq_lens})
     TORCH_CHECK(t->scalar_type() == at::kInt && t->is_cuda(), "index tensors must be int32 CUDA tensors");
@@ -750,8 +688,9 @@ void attention_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_ca
   TORCH_CHECK(q.size(0) == a.batch, "decode: one query row per request");
   a.hq = q.size(1);
   a.hkv = k_cache.size(1);
-  a.num_splits = mb200::decode_num_splits(a.batch, a.hkv, max_seq_len > 0 ? max_seq_len : req_to_token.size(1),
-                                           st.num_sms);
+  int64_t longest = max_seq_len > 0 ? max_seq_len : req_to_token.size(1);
+  if (window > 0) longest = std::min(longest, window + 128);     // keys read, up to the tiles' alignment
+  a.num_splits = mb200::decode_num_splits(a.batch, a.hkv, longest, st.num_sms);
   Tensor part_o, part_lse;
   if (a.num_splits > 1) {
     part_o = torch::empty({a.batch, a.hq, a.num_splits, hd}, q.options().dtype(torch::kFloat32));
@@ -770,6 +709,7 @@ void attention_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_ca
   a.seq_lens = seq_lens.data_ptr<int>();
   a.status = st.status.data_ptr<int>();
   a.q_stride = q.stride(0);
+  a.out_stride = out.stride(0);
   a.rtt_stride = req_to_token.stride(0);
   a.num_slots = k_cache.size(0);
   a.head_dim = static_cast<int>(hd);
@@ -803,18 +743,14 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("gemm", &gemm);
   m.def("gemm_norm", &gemm_norm);
   m.def("gemm_tp", &gemm_tp);
-  m.def("rmsnorm_gated", &rmsnorm_gated);
-  m.def("gdn_conv1d_silu", &gdn_conv1d_silu);
-  m.def("gdn_gates", &gdn_gates);
-  m.def("gdn_recurrent", &gdn_recurrent);
-  m.def("gdn_recurrent_raw", &gdn_recurrent_raw);
   m.def("residual_dyt", &residual_dyt);
   m.def("embedding_f32", &embedding_f32);
-  m.def("latent_prologue", &latent_prologue);
-  m.def("latent_gather", &latent_gather);
-  m.def("head_linear", &head_linear);
-  m.def("latent_attention", &latent_attention);
-  m.def("gdn_chunk", &gdn_chunk);
+  m.def("post_norm", &post_norm);
+  m.def("rmsnorm_sigmoid_gate", &rmsnorm_sigmoid_gate);
+  m.def("rownorm_rope_kv", &rownorm_rope_kv);
+  m.def("soft_cap", &soft_cap);
+  m.def("relu_squared", &relu_squared);
+  m.def("attention_rows", &attention_rows);
   m.def("attention_prefill", &attention_prefill, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("req_to_token"),
         py::arg("req_pool_indices"), py::arg("seq_lens"), py::arg("prefix_lens"), py::arg("q_start"), py::arg("scale"),
         py::arg("out"), py::arg("max_q_len"), py::arg("causal"), py::arg("window"), py::arg("logit_cap"),

@@ -33,6 +33,22 @@ void check_half(const Tensor& t, const char* name) {
               " must be bf16 or fp16");
 }
 
+void check_float(const Tensor& t, const char* name) {
+  check_cuda(t, name);
+  TORCH_CHECK(t.scalar_type() == at::kBFloat16 || t.scalar_type() == at::kHalf || t.scalar_type() == at::kFloat, "mllm_b200: ", name,
+              " must be bf16, fp16 or fp32");
+}
+void check_f32_vec(const Tensor& t, int64_t n, const char* name) {
+  TORCH_CHECK(t.is_cuda() && t.scalar_type() == at::kFloat && t.is_contiguous() && t.numel() == n, "mllm_b200: ", name,
+              " must be a contiguous fp32 device tensor of ", n, " elements");
+}
+
+void check_ragged(const Tensor& slots, const Tensor& lens, const Tensor& has, const Tensor& q_start) {
+  for (const Tensor* t : {&slots, &lens, &has, &q_start})
+    TORCH_CHECK(t->is_cuda() && t->scalar_type() == at::kInt && t->is_contiguous() && t->numel() == slots.numel(),
+                "ragged metadata: int32 device vectors of one length");
+}
+
 struct DeviceState {
   Tensor status;     // int32[1]
   Tensor workspace;  // float, split-K partials

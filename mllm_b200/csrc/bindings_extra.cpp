@@ -1,4 +1,4 @@
-// PyTorch binding of the kernels that only some models or layouts use (module mllm_b200_X): experts, 4-bit weights,
+// PyTorch binding of the kernels that only some models or layouts use (module mllm_b200_X): 4-bit weights,
 // vision towers, tensor- and expert-parallel exchange.
 #include "bindings_common.h"
 
@@ -86,92 +86,6 @@ void gelu_erf(const Tensor& x, Tensor& out) {
               "gelu_erf: contiguous tensors of one shape");
   c10::cuda::CUDAGuard g(x.device());
   mb200::launch_gelu_erf(x.data_ptr(), out.data_ptr(), x.numel(), dtype_of(x), stream_of(x));
-}
-
-// ---- mixture of experts ----
-void moe_router_topk(const Tensor& logits, Tensor& w, Tensor& ids, bool renorm) {
-  check_cuda(logits, "logits");
-  TORCH_CHECK(logits.dim() == 2 && logits.stride(1) == 1 && logits.size(1) <= 256, "moe_router_topk: [T,E<=256] logits");
-  TORCH_CHECK(w.scalar_type() == at::kFloat && ids.scalar_type() == at::kInt && w.is_contiguous() && ids.is_contiguous() &&
-                  w.dim() == 2 && w.size(0) == logits.size(0) && w.size(1) <= 32 && ids.sizes() == w.sizes(),
-              "moe_router_topk: fp32 weights / int32 ids [T,k<=32]");
-  c10::cuda::CUDAGuard g(logits.device());
-  mb200::launch_moe_router_topk(logits.data_ptr(), logits.stride(0), w.data_ptr<float>(), ids.data_ptr<int>(),
-                                logits.size(0), logits.size(1), w.size(1), renorm ? 1 : 0, dtype_of(logits),
-                                stream_of(logits));
-}
-
-void moe_align(const Tensor& topk_ids, int64_t expert_offset, int64_t experts, int64_t bn, Tensor& sorted_pos,
-               Tensor& src_token, Tensor& expert_offsets, Tensor& work, Tensor& n_work) {
-  check_cuda(topk_ids, "topk_ids");
-  TORCH_CHECK(topk_ids.scalar_type() == at::kInt && topk_ids.is_contiguous() && topk_ids.dim() == 2, "moe_align: int32 [T,k] ids");
-  TORCH_CHECK(experts >= 1 && experts <= 256, "moe_align: 1..256 local experts");
-  const int64_t pairs = topk_ids.numel();
-  for (const Tensor* t : {&sorted_pos, &src_token, &expert_offsets, &work, &n_work})
-    TORCH_CHECK(t->is_cuda() && t->scalar_type() == at::kInt && t->is_contiguous(), "moe_align: int32 outputs");
-  TORCH_CHECK(sorted_pos.numel() >= pairs && src_token.numel() >= pairs && expert_offsets.numel() >= experts + 1 &&
-                  work.dim() == 2 && work.size(1) == 2 && n_work.numel() >= 1,
-              "moe_align: output sizes");
-  c10::cuda::CUDAGuard g(topk_ids.device());
-  mb200::launch_moe_align(topk_ids.data_ptr<int>(), pairs, topk_ids.size(1), expert_offset, experts, bn,
-                          sorted_pos.data_ptr<int>(), src_token.data_ptr<int>(), expert_offsets.data_ptr<int>(),
-                          work.data_ptr<int>(), n_work.data_ptr<int>(), work.size(0), stream_of(topk_ids));
-}
-
-void moe_gather(const Tensor& x, const Tensor& src_token, const Tensor& expert_offsets, Tensor& xs) {
-  check_cuda(x, "x");
-  TORCH_CHECK(x.dim() == 2 && x.stride(1) == 1 && x.size(1) % 8 == 0 && x.stride(0) % 8 == 0 && xs.is_contiguous() &&
-                  xs.size(1) == x.size(1) && x.element_size() == 2 && xs.scalar_type() == x.scalar_type(),
-              "moe_gather: 16-bit rows, hidden % 8 == 0");
-  c10::cuda::CUDAGuard g(x.device());
-  mb200::launch_moe_gather(x.data_ptr(), x.stride(0), src_token.data_ptr<int>(), expert_offsets.data_ptr<int>(),
-                           expert_offsets.numel() - 1, xs.data_ptr(), xs.size(0), x.size(1), stream_of(x));
-}
-
-void moe_combine(const Tensor& y, const Tensor& sorted_pos, const Tensor& topk_w, Tensor& out) {
-  check_cuda(y, "y");
-  TORCH_CHECK(y.is_contiguous() && out.is_contiguous() && y.size(1) == out.size(1) && y.size(1) % 8 == 0 &&
-                  topk_w.scalar_type() == at::kFloat && topk_w.is_contiguous() && topk_w.size(0) == out.size(0) &&
-                  sorted_pos.numel() >= topk_w.numel() && y.scalar_type() == out.scalar_type() && y.element_size() == 2,
-              "moe_combine: shapes");
-  c10::cuda::CUDAGuard g(y.device());
-  mb200::launch_moe_combine(y.data_ptr(), sorted_pos.data_ptr<int>(), topk_w.data_ptr<float>(), out.data_ptr(),
-                            out.size(0), out.size(1), topk_w.size(1), dtype_of(y), stream_of(y));
-}
-
-// out[rows of e] = x[rows of e] @ w[e]^T (SwiGLU-fused when swiglu) over the expert-sorted rows
-int64_t moe_grouped_gemm(const Tensor& x, const Tensor& w, Tensor& out, const Tensor& expert_offsets, const Tensor& work,
-                      const Tensor& n_work, int64_t bn, bool swiglu) {
-  check_cuda(x, "x");
-  check_cuda(w, "w");
-  TORCH_CHECK(x.dim() == 2 && w.dim() == 3 && out.dim() == 2 && x.stride(1) == 1 && w.is_contiguous() && out.stride(1) == 1 &&
-                  x.size(1) == w.size(2) && x.scalar_type() == w.scalar_type() && out.scalar_type() == x.scalar_type() &&
-                  x.element_size() == 2,
-              "moe_grouped_gemm: x [R,K], w [E,N,K], 16-bit");
-  TORCH_CHECK(out.size(0) == x.size(0) && out.size(1) == (swiglu ? w.size(1) / 2 : w.size(1)), "moe_grouped_gemm: out shape");
-  TORCH_CHECK(expert_offsets.numel() == w.size(0) + 1, "moe_grouped_gemm: offsets");
-  c10::cuda::CUDAGuard g(x.device());
-  DeviceState& st = device_state(x.get_device());
-  mb200::MoeGemmArgs a{};
-  a.x = x.data_ptr();
-  a.w = w.data_ptr();
-  a.out = out.data_ptr();
-  a.expert_offsets = expert_offsets.data_ptr<int>();
-  a.work = work.data_ptr<int>();
-  a.n_work = n_work.data_ptr<int>();
-  a.status = st.status.data_ptr<int>();
-  a.ldx = x.stride(0);
-  a.ldc = out.stride(0);
-  a.rows_cap = x.size(0);
-  a.experts = w.size(0);
-  a.n = w.size(1);
-  a.k = w.size(2);
-  a.bn = bn;
-  a.max_work = work.size(0);
-  a.swiglu = swiglu ? 1 : 0;
-  a.num_sms = st.num_sms;
-  a.dt = dtype_of(x);
-  return mb200::launch_moe_grouped_gemm(a, stream_of(x));
 }
 
 int64_t tp_rs_add_rmsnorm_ag(const Tensor& inbox, const Tensor& tile_flags, Tensor& residual_shard, const Tensor& weight,
@@ -303,11 +217,6 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("vision_rope_split_pad", &vision_rope_split_pad);
   m.def("vision_pos_embed_add", &vision_pos_embed_add);
   m.def("gelu_erf", &gelu_erf);
-  m.def("moe_router_topk", &moe_router_topk);
-  m.def("moe_align", &moe_align);
-  m.def("moe_gather", &moe_gather);
-  m.def("moe_combine", &moe_combine);
-  m.def("moe_grouped_gemm", &moe_grouped_gemm);
   m.def("tp_rs_add_rmsnorm_ag", &tp_rs_add_rmsnorm_ag);
   m.def("tp_wait_flags", &tp_wait_flags);
   m.def("ep_plan", &ep_plan);

@@ -1,0 +1,67 @@
+// PyTorch binding of lightning attention (module mllm_b200_L).
+#include "bindings_common.h"
+
+namespace {
+
+mb200::LightningArgs lightning_args(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& decay, Tensor& state,
+                                    const Tensor& slots, const Tensor& lens, const Tensor& has, const Tensor& q_start, Tensor& out) {
+  check_float(q, "q");
+  check_ragged(slots, lens, has, q_start);
+  for (const Tensor* t : {&q, &k, &v})
+    TORCH_CHECK(t->is_cuda() && t->dim() == 3 && t->stride(2) == 1 && t->stride(1) == t->size(2) && t->size(0) == q.size(0) &&
+                    t->size(1) == q.size(1) && t->scalar_type() == q.scalar_type(),
+                "lightning attention: q, k [T, H, Dk], v [T, H, Dv] of one type, heads of a token contiguous");
+  TORCH_CHECK(k.size(2) == q.size(2) && out.is_cuda() && out.is_contiguous() && out.sizes() == v.sizes() &&
+                  out.scalar_type() == q.scalar_type() && state.is_cuda() && state.scalar_type() == at::kFloat && state.is_contiguous() &&
+                  state.dim() == 4 && state.size(1) == q.size(1) && state.size(2) == q.size(2) && state.size(3) == v.size(2),
+              "lightning attention: out [T, H, Dv], state fp32 [slots, H, Dk, Dv]");
+  check_f32_vec(decay, q.size(1), "decay");
+  mb200::LightningArgs a{};
+  a.q = q.data_ptr();
+  a.k = k.data_ptr();
+  a.v = v.data_ptr();
+  a.out = out.data_ptr();
+  a.decay = decay.data_ptr<float>();
+  a.state = state.data_ptr<float>();
+  a.slots = slots.data_ptr<int>();
+  a.lens = lens.data_ptr<int>();
+  a.has_state = has.data_ptr<int>();
+  a.q_start = q_start.data_ptr<int>();
+  a.q_ld = q.stride(0);
+  a.k_ld = k.stride(0);
+  a.v_ld = v.stride(0);
+  a.batch = slots.numel();
+  a.heads = q.size(1);
+  a.dk = q.size(2);
+  a.dv = v.size(2);
+  a.dt = dtype_of(q);
+  return a;
+}
+
+void lightning_recurrent(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& decay, Tensor& state, const Tensor& slots,
+                         const Tensor& lens, const Tensor& has, const Tensor& q_start, Tensor& out) {
+  const mb200::LightningArgs a = lightning_args(q, k, v, decay, state, slots, lens, has, q_start, out);
+  c10::cuda::CUDAGuard g(q.device());
+  const int rc = mb200::launch_lightning_recurrent(a, stream_of(q));
+  TORCH_CHECK(rc == 0, "lightning_recurrent: unsupported head size (code ", rc, ")");
+}
+
+// Returns 1 (nothing launched) when the sizes are not the chunk kernel's.
+int64_t lightning_chunk(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& decay, Tensor& state, const Tensor& slots,
+                        const Tensor& lens, const Tensor& has, const Tensor& q_start, Tensor& out) {
+  const mb200::LightningArgs a = lightning_args(q, k, v, decay, state, slots, lens, has, q_start, out);
+  if (!mb200::lightning_chunk_covers(a)) return 1;
+  c10::cuda::CUDAGuard g(q.device());
+  const int rc = mb200::launch_lightning_chunk(a, stream_of(q));
+  TORCH_CHECK(rc == 0, "lightning_chunk: launch failed (code ", rc, ")");
+  return 0;
+}
+
+}  // namespace
+
+PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
+  m.def("lightning_recurrent", &lightning_recurrent);
+  m.def("lightning_chunk", &lightning_chunk);
+  m.def("read_status", &read_status);
+  m.def("launch_count", &launch_count);
+}

@@ -278,17 +278,21 @@ __global__ void residual_dyt_kernel(float* __restrict__ x, const T* __restrict__
   }
 }
 
-// embedding rows widened to fp32 (the start of an fp32 residual stream); one CTA per token
+// embedding rows times a constant, in fp32 (the start of an fp32 residual stream); h (may be null): the same in the
+// table's type; one CTA per token
 template <typename T>
-__global__ void embedding_f32_kernel(const int64_t* __restrict__ ids, const T* __restrict__ table, float* __restrict__ out,
-                                     int width, int vocab, int* status) {
+__global__ void embedding_f32_kernel(const int64_t* __restrict__ ids, const T* __restrict__ table, float scale, float* __restrict__ out,
+                                     T* __restrict__ h, int width, int vocab, int* status) {
   pdl_launch_dependents();
   pdl_wait();
   const int64_t id = ids[blockIdx.x];
   const bool ok = id >= 0 && id < vocab;
   if (!ok && threadIdx.x == 0 && status != nullptr) atomicExch(status, kStatusBadIndex);
-  for (int c = threadIdx.x; c < width; c += blockDim.x)
-    out[static_cast<int64_t>(blockIdx.x) * width + c] = ok ? to_f32(table[id * width + c]) : 0.f;
+  for (int c = threadIdx.x; c < width; c += blockDim.x) {
+    const float v = ok ? to_f32(table[id * width + c]) * scale : 0.f;
+    out[static_cast<int64_t>(blockIdx.x) * width + c] = v;
+    if (h != nullptr) h[static_cast<int64_t>(blockIdx.x) * width + c] = from_f32<T>(v);
+  }
 }
 
 template <typename T>
@@ -725,12 +729,12 @@ void launch_residual_dyt(float* x, const void* y, float mult, const float* alpha
   note_launch();
 }
 
-void launch_embedding_f32(const int64_t* ids, const void* table, float* out, int tokens, int width, int vocab, DType dt,
-                          int* status, cudaStream_t s) {
+void launch_embedding_f32(const int64_t* ids, const void* table, float scale, float* out, void* h, int tokens, int width, int vocab,
+                          DType dt, int* status, cudaStream_t s) {
   if (tokens == 0) return;
   const int threads = width >= 256 ? 256 : (width + 31) / 32 * 32;
   MB200_DISPATCH_FLOAT(dt, (launch_pdl(embedding_f32_kernel<T>, dim3(tokens), dim3(threads), 0, s, ids, static_cast<const T*>(table),
-                                       out, width, vocab, status)));
+                                       scale, out, static_cast<T*>(h), width, vocab, status)));
   note_launch();
 }
 

@@ -98,7 +98,7 @@ __device__ __forceinline__ uint16_t f_to_half(float v) {
   return *reinterpret_cast<const uint16_t*>(&h);
 }
 
-template <bool F16, bool GELU>
+template <bool F16, int ACT>   // ACT: activation of the gate (0 SiLU, 1 GELU) or, 2, square of relu without a gate
 __global__ void __launch_bounds__(kSmThreads, 1) gemm_smallm_kernel(const SmallMParams p) {
   __shared__ float partial[2][kSmWarps][64];
   extern __shared__ __align__(16) uint8_t smem_dyn[];
@@ -284,11 +284,15 @@ __global__ void __launch_bounds__(kSmThreads, 1) gemm_smallm_kernel(const SmallM
                   for (int w8 = 0; w8 < kSmWarps; ++w8) up += partial[buf][w8][t + 4];
                   const int blk = cu >> 5, q = cu & 31;
                   const int64_t col = static_cast<int64_t>(blk) * 128 + q * 4 + slot;
-                  const float y = gate_act<GELU>(v) * up;
+                  const float y = gate_act<ACT == 1>(v) * up;
                   static_cast<uint16_t*>(p.out)[mrow * p.ldc + col] = f_to_half<F16>(y);
                 }
               } else {
                 const int64_t col = static_cast<int64_t>(cu) * 8 + slot;
+                if constexpr (ACT == 2) {
+                  v = fmaxf(v, 0.f);
+                  v *= v;
+                }
                 if (p.bias != nullptr) v += half_to_f<F16>(static_cast<const uint16_t*>(p.bias)[col]);
                 if (p.residual != nullptr)
                   v += half_to_f<F16>(static_cast<const uint16_t*>(p.residual)[mrow * p.ld_res + col]);
@@ -317,7 +321,8 @@ int launch_gemm_smallm(const GemmArgs& a, cudaStream_t s) {
   // matrices of hundreds of MB (the vocabulary head) stream at the full copy rate through the TMA ring of the
   // tcgen05 path, whose set-up cost no longer shows; this kernel is for the projections of a layer
   if (static_cast<int64_t>(a.n) * a.k * 2 > (int64_t(384) << 20)) return 1;
-  if (a.swiglu && (a.n % 256 != 0 || a.bias != nullptr || a.residual != nullptr)) return 1;
+  const bool relu2 = a.swiglu == 3;
+  if (a.swiglu && !relu2 && (a.n % 256 != 0 || a.bias != nullptr || a.residual != nullptr)) return 1;
   if ((a.lda * 2) % 16 != 0 || (a.ldb * 2) % 16 != 0) return 1;
   if (a.norm_weight != nullptr &&
       ((a.norm_residual_ld * 2) % 16 != 0 || (a.norm_residual_out_ld * 2) % 16 != 0 ||
@@ -340,7 +345,7 @@ int launch_gemm_smallm(const GemmArgs& a, cudaStream_t s) {
   p.ld_res = a.ld_res;
   p.units = a.n / 8;
   p.steps_per_warp = a.k / (32 * kSmWarps);
-  p.swiglu = a.swiglu;
+  p.swiglu = relu2 ? 0 : a.swiglu;
   p.b_static = a.b_static;
   p.norm_w = a.norm_weight;
   p.norm_res = static_cast<const uint8_t*>(a.norm_residual);
@@ -365,8 +370,9 @@ int launch_gemm_smallm(const GemmArgs& a, cudaStream_t s) {
     const cudaError_t set = ensure_dynamic_smem(reinterpret_cast<const void*>(kernel), kSmRingBytes + 8 * (2 * kSmMaxK + kSmRowPad));
     return set != cudaSuccess ? set : launch_pdl(kernel, dim3(grid), dim3(kSmThreads), smem, s, p);
   };
-  const cudaError_t err = a.dt == kF16 ? (gelu ? go(gemm_smallm_kernel<true, true>) : go(gemm_smallm_kernel<true, false>))
-                                       : (gelu ? go(gemm_smallm_kernel<false, true>) : go(gemm_smallm_kernel<false, false>));
+  const cudaError_t err =
+      a.dt == kF16 ? (relu2 ? go(gemm_smallm_kernel<true, 2>) : gelu ? go(gemm_smallm_kernel<true, 1>) : go(gemm_smallm_kernel<true, 0>))
+                   : (relu2 ? go(gemm_smallm_kernel<false, 2>) : gelu ? go(gemm_smallm_kernel<false, 1>) : go(gemm_smallm_kernel<false, 0>));
   note_launch();
   return err == cudaSuccess ? 0 : -4;
 }

@@ -82,7 +82,18 @@ struct KParams {
 constexpr int kStageRowBytes = 144;                      // 128 bytes of output + 16 bytes of padding
 constexpr int kEpiStagingBytes = 4 * 32 * kStageRowBytes;  // four epilogue warps x 32 rows
 
-// SWIGLU: 0 plain product, 1 silu(gate) * up, 2 gelu_tanh(gate) * up.
+template <int SWIGLU>
+constexpr bool kGated = SWIGLU == 1 || SWIGLU == 2;
+template <int SWIGLU>
+__device__ __forceinline__ float plain_act(float x) {
+  if constexpr (SWIGLU == 3) {
+    x = fmaxf(x, 0.f);
+    return x * x;
+  }
+  return x;
+}
+
+// SWIGLU: 0 plain product, 1 silu(gate) * up, 2 gelu_tanh(gate) * up, 3 square of relu (no gate: as the plain product).
 // RT = 128-row MMA tiles of the row operand per stage (small-batch tiling only; SwiGLU needs 2: a
 // gate block and its up block), KD = 128-byte K atoms per stage.  Larger stages mean fewer TMA boxes
 // and barrier round trips per byte streamed.
@@ -96,14 +107,14 @@ struct Cfg {
   // one or two CTAs per SM: the ring takes the shared memory that is left
   static constexpr int kStagesRaw = 200704 / kStageBytes;
   static constexpr int kStages = kStagesRaw > 12 ? 12 : kStagesRaw;
-  static constexpr int kSub = SWIGLU ? 1 : R;                 // output rows finalised per epilogue thread
+  static constexpr int kSub = kGated<SWIGLU> ? 1 : R;                 // output rows finalised per epilogue thread
   static constexpr int kAccCols = R * BN;
   static constexpr int kAccBufs = (2 * kAccCols <= 512) ? 2 : 1;
   static constexpr int kTmemColsRaw = kAccBufs * kAccCols;
   static constexpr int kTmemCols =
       kTmemColsRaw <= 32 ? 32 : (kTmemColsRaw <= 64 ? 64 : (kTmemColsRaw <= 128 ? 128 : (kTmemColsRaw <= 256 ? 256 : 512)));
   static_assert(kStages >= 2, "stage too large for shared memory");
-  static_assert(!SWIGLU || !SWAP || RT == 2, "SwiGLU small-batch tiles hold a gate block and an up block");
+  static_assert(!kGated<SWIGLU> || !SWAP || RT == 2, "SwiGLU small-batch tiles hold a gate block and an up block");
   static_assert(SWAP || (RT == 1 && KD == 1), "normal tiling uses single-atom stages");
   static_assert(kTmemColsRaw <= 512, "accumulators exceed tensor memory");
   static_assert(BN % 16 == 0 && BN >= 16 && BN <= 256, "invalid MMA N");
@@ -465,9 +476,9 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
       const uint32_t t_base = tmem_base + (static_cast<uint32_t>(ew * 32) << 16) + acc * C::kAccCols;
 
       if constexpr (!SWAP) {
-        constexpr int kOutCols = SWIGLU ? BN / 2 : BN;
+        constexpr int kOutCols = kGated<SWIGLU> ? BN / 2 : BN;
         const int64_t col0 = static_cast<int64_t>(tc) * kOutCols;
-        const int n_out = SWIGLU ? p.n / 2 : p.n;
+        const int n_out = kGated<SWIGLU> ? p.n / 2 : p.n;
         if (p.rs_tp > 0) {
           // Staged epilogue (reduce-scatter stores only): a thread owns one accumulator row; 64 output columns at a time are
           // rounded, parked in shared memory and written back so that eight lanes cover 128
@@ -493,7 +504,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
             for (int h = 0; h < 2; ++h) {
               uint32_t r0[32], r1[32];
               tmem_ld_32x32(t_base + c + h * 32, r0);
-              if constexpr (SWIGLU) tmem_ld_32x32(t_base + BN / 2 + c + h * 32, r1);
+              if constexpr (kGated<SWIGLU>) tmem_ld_32x32(t_base + BN / 2 + c + h * 32, r1);
               tmem_ld_wait();
 #pragma unroll
               for (int j = 0; j < 32; j += 2) {
@@ -502,7 +513,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
                 for (int q = 0; q < 2; ++q) {
                   const int cc = c + h * 32 + j + q;  // column inside the tile's output
                   float x = acc_to_float(r0[j + q], p.is_int8);
-                  if constexpr (SWIGLU) {
+                  if constexpr (kGated<SWIGLU>) {
                     float u = acc_to_float(r1[j + q], p.is_int8);
                     if (p.is_int8) {
                       x *= sa * p.b_scale[tc * BN + cc];
@@ -548,7 +559,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
         for (int c = 0; c < kOutCols; c += 32) {
           uint32_t r0[32], r1[32];
           tmem_ld_32x32(t_base + c, r0);
-          if constexpr (SWIGLU) tmem_ld_32x32(t_base + BN / 2 + c, r1);
+          if constexpr (kGated<SWIGLU>) tmem_ld_32x32(t_base + BN / 2 + c, r1);
           tmem_ld_wait();
           if (!row_ok) continue;
 #pragma unroll
@@ -559,7 +570,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
               float x = acc_to_float(r0[v8 * 8 + j], p.is_int8);
-              if constexpr (SWIGLU) {
+              if constexpr (kGated<SWIGLU>) {
                 float u = acc_to_float(r1[v8 * 8 + j], p.is_int8);
                 if (p.is_int8) {
                   x *= sa * p.b_scale[tc * BN + c + v8 * 8 + j];
@@ -569,10 +580,11 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
               } else {
                 if (p.is_int8) x *= sa * p.b_scale[col + j];
                 if (p.bias != nullptr) x += load_out1(p.bias, col + j, p.out_f16);
+                x = plain_act<SWIGLU>(x);
               }
               f[j] = x;
             }
-            if (!SWIGLU && p.residual != nullptr) {
+            if (!kGated<SWIGLU> && p.residual != nullptr) {
               const uint4 rv = *reinterpret_cast<const uint4*>(static_cast<const uint16_t*>(p.residual) +
                                                                row * p.ld_res + col);
               const uint32_t* ru = reinterpret_cast<const uint32_t*>(&rv);
@@ -695,14 +707,14 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
               for (int c0 = 0; c0 < m_cols; c0 += 16) {
                 float x[16], u[16];
                 reduce16(sub * kBM + row_in_tile, c0, x);
-                if constexpr (SWIGLU) reduce16(kBM + row_in_tile, c0, u);
+                if constexpr (kGated<SWIGLU>) reduce16(kBM + row_in_tile, c0, u);
 #pragma unroll
                 for (int jj = 0; jj < 16; ++jj) {
                   const int j = c0 + jj;
                   if (j >= m_cols) break;
                   float xv = x[jj];
                   int64_t ocol;
-                  if constexpr (SWIGLU) {
+                  if constexpr (kGated<SWIGLU>) {
                     float uv = u[jj];
                     if (p.is_int8) {
                       xv *= p.a_scale[j] * p.b_scale[wrow];
@@ -738,7 +750,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
           for (int c = 0; c < BN; c += 16) {
             uint32_t v0[16], v1[16];
             tmem_ld_32x16(t_base + sub * BN + c, v0);
-            if constexpr (SWIGLU) tmem_ld_32x16(t_base + BN + c, v1);
+            if constexpr (kGated<SWIGLU>) tmem_ld_32x16(t_base + BN + c, v1);
             tmem_ld_wait();
             if (wrow >= p.n) continue;
 #pragma unroll
@@ -750,10 +762,10 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
               for (int s2 = 1; s2 < p.cluster_k; ++s2) {   // partners in rank order: the sum does not depend on timing
                 const float* part = red_buf + static_cast<size_t>(s2 - 1) * kTileRows * BN;
                 x += part[(sub * kBM + row_in_tile) * BN + mi];
-                if constexpr (SWIGLU) u_extra += part[(kBM + row_in_tile) * BN + mi];
+                if constexpr (kGated<SWIGLU>) u_extra += part[(kBM + row_in_tile) * BN + mi];
               }
               int64_t ocol;
-              if constexpr (SWIGLU) {
+              if constexpr (kGated<SWIGLU>) {
                 float u = acc_to_float(v1[j], p.is_int8) + u_extra;
                 if (p.is_int8) {
                   x *= p.a_scale[mi] * p.b_scale[wrow];
@@ -1064,8 +1076,8 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_consta
     const int row_in_tile = ew * 32 + lane;
     bool ok = true;
     int tr, tc;
-    constexpr int kOutCols = SWIGLU ? kPairBN / 2 : kPairBN;
-    const int n_out = SWIGLU ? p.n / 2 : p.n;
+    constexpr int kOutCols = kGated<SWIGLU> ? kPairBN / 2 : kPairBN;
+    const int n_out = kGated<SWIGLU> ? p.n / 2 : p.n;
     for (int idx = 0; ok && get_tile(idx, tr, tc); ++idx) {
       const int acc = idx & 1;
       const uint32_t acc_phase = (idx >> 1) & 1;
@@ -1079,7 +1091,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_consta
       const bool row_ok = row < p.m;
       const int64_t col0 = static_cast<int64_t>(tc) * kOutCols;
       const float sa = (p.is_int8 && row_ok) ? p.a_scale[row] : 1.f;
-      if constexpr (!SWIGLU) {
+      if constexpr (!kGated<SWIGLU>) {
         if (p.rs_tp > 0) {
           // reduce-scatter: 64 output columns at a time are rounded, parked in shared memory and written so that
           // eight lanes cover 128 contiguous bytes of one row of the owner's inbox (full-line peer stores)
@@ -1140,7 +1152,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_consta
       for (int c = 0; c < kOutCols; c += 32) {
         uint32_t r0[32], r1[32];
         tmem_ld_32x32(t_base + c, r0);
-        if constexpr (SWIGLU) tmem_ld_32x32(t_base + kPairBN / 2 + c, r1);
+        if constexpr (kGated<SWIGLU>) tmem_ld_32x32(t_base + kPairBN / 2 + c, r1);
         tmem_ld_wait();
         if (!row_ok) continue;
 #pragma unroll
@@ -1151,7 +1163,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_consta
 #pragma unroll
           for (int j = 0; j < 8; ++j) {
             float x = acc_to_float(r0[v8 * 8 + j], p.is_int8);
-            if constexpr (SWIGLU) {
+            if constexpr (kGated<SWIGLU>) {
               float u = acc_to_float(r1[v8 * 8 + j], p.is_int8);
               if (p.is_int8) {
                 x *= sa * p.b_scale[tc * kPairBN + c + v8 * 8 + j];
@@ -1161,10 +1173,11 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_consta
             } else {
               if (p.is_int8) x *= sa * p.b_scale[col + j];
               if (p.bias != nullptr) x += load_out1(p.bias, col + j, p.out_f16);
+              x = plain_act<SWIGLU>(x);
             }
             f[j] = x;
           }
-          if (!SWIGLU && p.residual != nullptr) {
+          if (!kGated<SWIGLU> && p.residual != nullptr) {
             const uint4 rv = *reinterpret_cast<const uint4*>(static_cast<const uint16_t*>(p.residual) +
                                                              row * p.ld_res + col);
             const uint32_t* ru = reinterpret_cast<const uint32_t*>(&rv);
@@ -1298,7 +1311,9 @@ int launch_gemm(const GemmArgs& a, cudaStream_t s) {
   const int k_per_block = kRowBytes / eb;
   if (a.k % (16 / eb) != 0 || a.lda % (16 / eb) != 0 || a.ldb % (16 / eb) != 0) return -1;
   if (a.n % 8 != 0 || a.ldc % 8 != 0) return -1;
-  if (a.swiglu && (a.n % 256 != 0 || a.bias != nullptr || a.residual != nullptr)) return -1;
+  const bool gated = a.swiglu == 1 || a.swiglu == 2, relu2 = a.swiglu == 3;
+  if (gated && (a.n % 256 != 0 || a.bias != nullptr || a.residual != nullptr)) return -1;
+  if (relu2 && (a.bias != nullptr || a.residual != nullptr || a.rs_tp > 0)) return -1;
   if ((reinterpret_cast<uintptr_t>(a.a) | reinterpret_cast<uintptr_t>(a.b) | reinterpret_cast<uintptr_t>(a.out)) & 15)
     return -1;
   if (a.residual != nullptr && ((reinterpret_cast<uintptr_t>(a.residual) & 15) || a.ld_res % 8 != 0)) return -1;
@@ -1359,7 +1374,7 @@ int launch_gemm(const GemmArgs& a, cudaStream_t s) {
     // ---- two-CTA tiling: 256 x 256 tiles per pair of SMs, when there are enough of them to fill the GPU ----
     static const int pair_knob = env_int("MLLM_B200_GEMM_PAIR", 1);
     const int64_t tiles_pair = static_cast<int64_t>((a.m + 2 * kBM - 1) / (2 * kBM)) * ((a.n + kPairBN - 1) / kPairBN);
-    const bool pair_rs_ok = a.rs_tp == 0 || (!a.swiglu && (a.m / kBM / a.rs_tp) % 2 == 0);
+    const bool pair_rs_ok = a.rs_tp == 0 || (!gated && (a.m / kBM / a.rs_tp) % 2 == 0);
     const int rs_first_owner = a.rs_tp > 0 ? (a.rs_rank + 1) % a.rs_tp : 0;
     if (pair_knob && a.n % 256 == 0 && tiles_pair >= num_sms / 2 && pair_rs_ok) {
       if (a.rs_tp > 0) p.rs_shift = rs_first_owner * (p.rs_tiles_per_rank / 2);
@@ -1369,13 +1384,14 @@ int launch_gemm(const GemmArgs& a, cudaStream_t s) {
       if (!make_operand_map(&tm_row, a.a, a.m, a.k, a.lda, eb, type, kBM)) return -2;
       if (!make_operand_map(&tm_col, a.b, a.n, a.k, a.ldb, eb, type, kPairBN / 2)) return -2;
       const int pairs = static_cast<int>(std::min<int64_t>(tiles_pair, num_sms / 2));
+      if (relu2) return launch_pair_cfg<3>(tm_row, tm_col, p, pairs, s);
       if (a.swiglu == 2) return launch_pair_cfg<2>(tm_row, tm_col, p, pairs, s);
-      return a.swiglu ? launch_pair_cfg<1>(tm_row, tm_col, p, pairs, s)
+      return gated ? launch_pair_cfg<1>(tm_row, tm_col, p, pairs, s)
                       : launch_pair_cfg<0>(tm_row, tm_col, p, pairs, s);
     }
     // ---- normal tiling: activations are the 128-row operand ----
     int bn = 256;
-    if (!a.swiglu) {
+    if (!gated) {
       const int64_t tiles256 = static_cast<int64_t>((a.m + kBM - 1) / kBM) * ((a.n + 255) / 256);
       if (tiles256 < num_sms || a.n % 256 != 0) bn = 128;
     }
@@ -1386,8 +1402,10 @@ int launch_gemm(const GemmArgs& a, cudaStream_t s) {
     if (!make_operand_map(&tm_row, a.a, a.m, a.k, a.lda, eb, type, kBM)) return -2;
     if (!make_operand_map(&tm_col, a.b, a.n, a.k, a.ldb, eb, type, bn)) return -2;
     const int grid = std::min(p.tiles_r * p.tiles_c, num_sms);
+    if (relu2)
+      return bn == 256 ? launch_cfg<256, false, 3>(tm_row, tm_col, p, grid, s) : launch_cfg<128, false, 3>(tm_row, tm_col, p, grid, s);
     if (a.swiglu == 2) return launch_cfg<256, false, 2>(tm_row, tm_col, p, grid, s);
-    if (a.swiglu) return launch_cfg<256, false, 1>(tm_row, tm_col, p, grid, s);
+    if (gated) return launch_cfg<256, false, 1>(tm_row, tm_col, p, grid, s);
     if (bn == 256) return launch_cfg<256, false, 0>(tm_row, tm_col, p, grid, s);
     return launch_cfg<128, false, 0>(tm_row, tm_col, p, grid, s);
   }
@@ -1397,6 +1415,7 @@ int launch_gemm(const GemmArgs& a, cudaStream_t s) {
     const int rc = launch_gemm_smallm(a, s);
     if (rc <= 0) return rc;
   }
+  if (relu2) return 1;                       // 9 to 256 rows: the caller applies the activation itself
   if (a.norm_weight != nullptr) return -1;   // the fused norm prologue exists in that kernel only
 
   // ---- swap tiling: weights are the 128-row operand, the batch is MMA N ----

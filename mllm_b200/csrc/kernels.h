@@ -27,8 +27,55 @@ void launch_act_and_mul(const void* x, void* out, int rows, int inter, int act, 
 // fp32 residual stream with a Dynamic Tanh norm: x += mult * y (y may be null), h = tanh(alpha x) * w + b
 void launch_residual_dyt(float* x, const void* y, float mult, const float* alpha, const float* w, const float* b, void* h,
                          int rows, int width, DType dt, cudaStream_t s);
-void launch_embedding_f32(const int64_t* ids, const void* table, float* out, int tokens, int width, int vocab, DType dt,
-                          int* status, cudaStream_t s);
+// embedding rows times `scale` in fp32; h (may be null): the same rounded to dt
+void launch_embedding_f32(const int64_t* ids, const void* table, float scale, float* out, void* h, int tokens, int width, int vocab,
+                          DType dt, int* status, cudaStream_t s);
+
+// ----- row-wise kernels of decoders with an fp32 residual stream (row_ops.cu) -----------------
+// x_out, h = rmsnorm(alpha * x + ls * (y + sum of the token's expert rows)) * w, x and x_out fp32 (x_out may be x, or null)
+struct PostNormArgs {
+  const float* x;           // [rows, width]
+  float* x_out;             // [rows, width] or null
+  const void* y;            // [rows, width] or null
+  const float* ls;          // [width] or null (1)
+  const float* w;           // [width]
+  void* h;                  // [rows, width]
+  // weighted sum of expert outputs (expert_rows null: none); choice j of token t is row sorted_pos[t * top + j] of
+  // expert_rows, or, where that is negative and its id is >= identity_from > 0, the row t of token_in
+  const void* expert_rows;
+  const int* sorted_pos;
+  const float* topk_w;
+  const int* ids;
+  const void* token_in;
+  int rows, width, top, identity_from;
+  float alpha, eps;
+  DType dt;                 // of y, h, expert_rows, token_in
+};
+int launch_post_norm(const PostNormArgs& args, cudaStream_t s);
+// out = rmsnorm over the whole row of x, times w and sigmoid(gate)
+int launch_rmsnorm_sigmoid_gate(const void* x, const void* gate, int64_t gate_ld, const float* w, void* out, int64_t out_ld, int rows,
+                                int width, float eps, DType dt, cudaStream_t s);
+// rows [q | k | v] of tokens: RMS norm over all query heads and over all key heads, rotation of neighbouring features,
+// q to q_out [tokens, heads, q_width] (zeros behind dim), k and v to the cache slots loc
+struct RowNormRopeArgs {
+  const void* row;          // row t at t * row_ld: heads * dim, kv_heads * dim and kv_heads * vdim features
+  const float* q_w;         // [heads * dim]
+  const float* k_w;         // [kv_heads * dim]
+  const double* inv_freq;   // [rot_dims / 2]
+  const int64_t* positions; // [tokens]
+  const int64_t* loc;       // [tokens]
+  void* q_out;
+  void* k_cache;            // head h of slot s at s * tok + h * head (elements)
+  void* v_cache;
+  int* status;
+  int64_t row_ld, k_tok_stride, k_head_stride, v_tok_stride, v_head_stride, num_slots;
+  int tokens, heads, kv_heads, dim, vdim, q_width, rot_dims;
+  float eps;
+  DType dt;
+};
+int launch_rownorm_rope_kv(const RowNormRopeArgs& args, cudaStream_t s);
+void launch_soft_cap(const void* x, int64_t x_ld, float* out, int rows, int width, float cap, DType dt, cudaStream_t s);
+void launch_relu_squared(void* x, int64_t n, DType dt, cudaStream_t s);
 void launch_gelu_tanh(const void* x, void* out, int64_t n, DType dt, cudaStream_t s);
 void launch_embedding(const int64_t* ids, const void* table, void* out, int tokens, int hidden, int vocab,
                       DType dt, int* status, cudaStream_t s);
@@ -89,7 +136,8 @@ struct GemmArgs {
   const float* b_scale;  // int8 only: per-column scale [n]
   int m, n, k;
   int64_t lda, ldb, ldc, ld_res;
-  int swiglu;            // 1: b rows alternate 128 gate / 128 up rows; out is [m, n/2] = silu(gate) * up; 2: gelu_tanh(gate) * up
+  int swiglu;            // 1: b rows alternate 128 gate / 128 up rows; out is [m, n/2] = silu(gate) * up; 2: gelu_tanh(gate) * up;
+                         // 3: out is [m, n] = max(a b^T, 0)^2 (launch_gemm returns 1 for 9 to 256 rows: not fused there)
   DType dt;              // element type of a, b (kBF16 / kF16) ; out has the same type
   int is_int8;           // 1: a, b are int8, out type given by dt
   float* workspace;      // split-K partial sums (small-m path), may be null when not needed
@@ -177,16 +225,20 @@ int launch_ep_dispatch(const EpA2AArgs& a, const void* x, int64_t x_stride, int 
 int launch_ep_return(const EpA2AArgs& a, const void* ys, const int* recv_rows, int* done_count, cudaStream_t s);
 
 // ----- mixture of experts ----------------------------------------------------------------
-// router: fp32 softmax over `experts` (<= 256) logits -> top_k (<= 32, sorted, lowest index wins ties)
-void launch_moe_router_topk(const void* logits, int64_t stride, float* w, int* ids, int tokens, int experts, int top_k,
-                            int renorm, DType dt, cudaStream_t s);
+// logits[t, e] = x[t] . w[e] in fp32 (products of 16-bit values are exact in it)
+int launch_moe_router_logits(const void* x, int64_t x_ld, const void* w, float* logits, int tokens, int experts, int hidden,
+                             int num_sms, DType dt, cudaStream_t s);
+// router: fp32 softmax over `experts` (<= 256) logits -> top_k (<= 32, sorted, lowest index wins ties).  The choice goes by
+// the scores plus `correction` (may be null), the weights are the scores; renorm divides them by their sum + renorm_eps
+void launch_moe_router_topk(const void* logits, int64_t stride, const float* correction, float* w, int* ids, int tokens, int experts,
+                            int top_k, int renorm, float renorm_eps, DType dt, cudaStream_t s);
 // counting sort of the (token, choice) pairs by local expert.  sorted_pos[pair] = row in the sorted
 // matrix or -1 (expert on another rank); src_token[row] = token; expert_offsets[experts + 1];
 // work[i] = (expert, chunk of bn rows), *n_work items.
 void launch_moe_align(const int* topk_ids, int pairs, int top_k, int expert_offset, int experts, int bn, int* sorted_pos,
                       int* src_token, int* expert_offsets, int* work, int* n_work, int max_work, cudaStream_t s);
 void launch_moe_gather(const void* x, int64_t x_stride, const int* src_token, const int* expert_offsets, int experts,
-                       void* xs, int pairs, int hidden, cudaStream_t s);
+                       void* xs, int pairs, int hidden, int elem_bytes, cudaStream_t s);
 void launch_moe_combine(const void* y, const int* sorted_pos, const float* topk_w, void* out, int tokens, int hidden,
                         int top_k, DType dt, cudaStream_t s);
 struct MoeGemmArgs {
@@ -202,6 +254,8 @@ struct MoeGemmArgs {
   DType dt;
 };
 int launch_moe_grouped_gemm(const MoeGemmArgs& args, cudaStream_t s);
+// the plain product (no SwiGLU) for fp32 and for sizes that the tensor-core kernel does not take
+int launch_moe_grouped_gemm_any(const MoeGemmArgs& args, cudaStream_t s);
 
 // ----- attention over the slot-indexed KV pool (tcgen05, head_dim 128) -----------------
 struct AttnArgs {
@@ -210,7 +264,7 @@ struct AttnArgs {
   const void* v_cache;
   int64_t kv_tok_stride;    // slot-major [slots, Hkv, 128]: Hkv * 128 and 128; head-major [Hkv, slots, 128]:
   int64_t kv_head_stride;   // 128 and slots * 128 (consecutive slots of a head are then contiguous)
-  void* out;                // [T, Hq, 128] contiguous
+  void* out;                // [T, Hq, D], rows of a token out_stride apart (0: contiguous)
   float* part_o;            // decode with num_splits > 1: [B, Hq, splits, 128]
   float* part_lse;          // decode with num_splits > 1: [B, Hq, splits]
   const int* req_to_token;  // [reqs, rtt_stride]
@@ -219,7 +273,7 @@ struct AttnArgs {
   const int* prefix_lens;       // [B], prefill only
   const int* q_start;           // [B], prefill only: first query row of each request
   int* status;
-  int64_t q_stride, rtt_stride, num_slots;
+  int64_t q_stride, out_stride, rtt_stride, num_slots;
   int batch, hq, hkv, head_dim;
   int max_q_len;            // prefill: longest run of new tokens in the batch
   int num_splits;           // decode
@@ -234,6 +288,48 @@ struct AttnArgs {
 };
 int launch_attention(const AttnArgs& args, cudaStream_t s);
 int decode_num_splits(int batch, int hkv, int max_seq_len, int num_sms);
+
+// ----- attention of single rows, any head sizes, fp32 arithmetic (attention_rows.cu) -----------
+struct RowAttnArgs {
+  const void* q;            // [rows, heads, dim], rows q_stride apart
+  const void* k_cache;      // head g of slot s at s * tok + g * head (elements), dim features
+  const void* v_cache;      // the same with vdim features
+  void* out;                // [rows, heads, vdim], rows out_stride apart
+  const int* req_to_token;
+  const int* row_req;       // [rows] request-table row
+  const int64_t* row_pos;   // [rows] position: keys 0 .. position (the last `window` of them when window > 0)
+  const float* sink;        // [heads] or null
+  int* status;
+  int64_t q_stride, out_stride, rtt_stride, num_slots, k_tok_stride, k_head_stride, v_tok_stride, v_head_stride;
+  int rows, heads, kv_heads, dim, vdim, window;
+  float scale, logit_cap;
+  DType dt;
+};
+int launch_attention_rows(const RowAttnArgs& args, cudaStream_t s);
+
+// ----- lightning attention (lightning.cu) --------------------------------------------------------
+// Per request and head, S <- decay S + k v^T and o = S^T q with q, k, v = silu of the given rows (rounded to dt), S fp32.
+// Ragged sequences as for the gated delta net below.
+struct LightningArgs {
+  const void* q;            // [T, heads, dk], token rows q_ld apart
+  const void* k;
+  const void* v;            // [T, heads, dv]
+  void* out;                // [T, heads, dv] contiguous
+  const float* decay;       // [heads]
+  float* state;             // [rows, heads, dk, dv]
+  const int* slots;
+  const int* lens;
+  const int* has_state;
+  const int* q_start;
+  int64_t q_ld, k_ld, v_ld;
+  int batch, heads, dk, dv;
+  DType dt;
+};
+// token by token; dk up to 512, any dv
+int launch_lightning_recurrent(const LightningArgs& args, cudaStream_t s);
+// 64 tokens at a time on the tensor cores; 16-bit types, dk up to 128
+int launch_lightning_chunk(const LightningArgs& args, cudaStream_t s);
+bool lightning_chunk_covers(const LightningArgs& args);
 
 // ----- latent attention (one cached row of `rank` features per token, shared by all heads) ------------
 // RMS norm of both parts of the down projections' rows [q_rank | kv_rank]: the first into cq [tokens, q_rank], the

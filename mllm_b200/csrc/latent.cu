@@ -19,6 +19,7 @@
 
 #include "common.cuh"
 #include "kernels.h"
+#include "mma.cuh"
 
 namespace mb200 {
 namespace {
@@ -93,20 +94,6 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const V* __restrict_
 // dimension) and tiles of 8 tokens; a lane feeds 16 contiguous bytes of W and of x to two MMAs, the same
 // permutation of k in both operands.  KS > 1: the warps of the CTA split k of the same 16 rows.
 // ---------------------------------------------------------------------------------------------
-template <typename T>
-__device__ __forceinline__ void mma_16816(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0,
-                                          uint32_t b1) {
-  if constexpr (sizeof(T) == 2 && std::is_same<T, __half>::value) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.f16.f16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-                 : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
-  } else {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-                 : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
-  }
-}
-
 constexpr int kHlTokTiles = 4;   // tiles of 8 tokens per CTA
 
 template <typename T, int KS>
@@ -208,23 +195,6 @@ __device__ __forceinline__ float lat_inv_denominator(float l, float m, const flo
   return 1.f / (l + exp2f(d));
 }
 
-__device__ __forceinline__ void lat_cp16(uint32_t dst, const void* src, bool valid) {
-  const int sz = valid ? 16 : 0;
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(sz) : "memory");
-}
-__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-               : "r"(addr)
-               : "memory");
-}
-__device__ __forceinline__ void ldsm4_t(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-               : "r"(addr)
-               : "memory");
-}
-
 constexpr int kLatTok = 32;        // context tokens per tile
 constexpr int kLatSLd = kLatTok + 8;
 
@@ -312,7 +282,7 @@ __global__ void __launch_bounds__(256) latent_attn_mma_kernel(const LatentParams
       const int s = __shfl_sync(0xffffffffu, my_slot, tk);
       const int c = c0 + ch * 8;
       const bool ok = s >= 0 && c < p.rank;
-      lat_cp16(dst + tk * C::kRowBytes + ch * 16, cache + (ok ? static_cast<int64_t>(s) * p.cache_ld + c : 0), ok);
+      cp16_zfill(dst + tk * C::kRowBytes + ch * 16, cache + (ok ? static_cast<int64_t>(s) * p.cache_ld + c : 0), ok);
     }
   };
 

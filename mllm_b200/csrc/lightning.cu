@@ -1,0 +1,406 @@
+// Lightning attention: linear attention with one fixed decay per head.  Per request and head,
+//
+//   S_t = decay S_(t-1) + k_t v_t^T,   o_t = S_t^T q_t,   q, k, v = silu of the projections' rows (rounded to their type)
+//
+// with S [dk, dv] in fp32, kept per request row between passes.  Two evaluations of the same sums:
+//
+// * token by token (decode, short extends, fp32, any size): the state in registers, one exchange per token;
+// * 64 tokens at a time (bf16 prefill): with S the state before the chunk and row i = 0 .. n - 1,
+//     O_i = decay^(i+1) Q_i S + sum_(j <= i) decay^(i-j) (Q_i . K_j) V_j
+//     S' = decay^n S + K^T diag(decay^(n-1-j)) V
+//   as warp-level tensor-core products.  Q, K and V are bf16 and enter as they are; fp32 operands are carried as sums of
+//   bf16 terms: two (16 bits) where the result is an output that is rounded to bf16 next, three (24 bits, all of fp32)
+//   where it stays in the state.  Nothing of the state passes through 16 bits.
+#include "common.cuh"
+#include "kernels.h"
+#include "mma.cuh"
+
+namespace mb200 {
+namespace {
+
+// SiLU of a value that is rounded to T next, and that rounding
+template <typename T>
+__device__ __forceinline__ float silu_as(float v) {
+  if constexpr (sizeof(T) == 2) return to_f32(from_f32<T>(__fdividef(v, 1.f + __expf(-v))));
+  return v / (1.f + expf(-v));
+}
+
+// ---------------------------------------------------------------------------------------------
+// token by token: grid (ceil(dv / 32), heads, batch), 256 threads; thread (rg, cl) = (tid / 8, tid % 8) holds rows rg,
+// rg + 32, ... of four columns of the state
+// ---------------------------------------------------------------------------------------------
+template <typename T, int RPT>
+__global__ void __launch_bounds__(256) lightning_recurrent_kernel(const LightningArgs p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float4 red[2][8][8];     // [parity][warp][column group]
+  const int h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int cl = tid & 7, rg = tid >> 3;
+  const int n = p.lens[b];
+  if (n <= 0) return;
+  const int c = blockIdx.x * 32 + cl * 4;
+  const int64_t row0 = p.q_start[b];
+  float* S = p.state + (static_cast<int64_t>(p.slots[b]) * p.heads + h) * p.dk * p.dv;   // [dk][dv]
+  const T* q = static_cast<const T*>(p.q) + row0 * p.q_ld + static_cast<int64_t>(h) * p.dk;
+  const T* k = static_cast<const T*>(p.k) + row0 * p.k_ld + static_cast<int64_t>(h) * p.dk;
+  const T* v = static_cast<const T*>(p.v) + row0 * p.v_ld + static_cast<int64_t>(h) * p.dv;
+  T* out = static_cast<T*>(p.out) + (row0 * p.heads + h) * p.dv;
+  const bool vec = (p.dv & 3) == 0;
+  const bool resume = p.has_state[b] != 0;
+  const float decay = p.decay[h];
+  float s[RPT][4];
+#pragma unroll
+  for (int r = 0; r < RPT; ++r) {
+    const int i = rg + 32 * r;
+    s[r][0] = s[r][1] = s[r][2] = s[r][3] = 0.f;
+    if (resume && i < p.dk) {
+      if (vec && c < p.dv) {
+        *reinterpret_cast<float4*>(s[r]) = *reinterpret_cast<const float4*>(S + static_cast<int64_t>(i) * p.dv + c);
+      } else {
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+          if (c + j < p.dv) s[r][j] = S[static_cast<int64_t>(i) * p.dv + c + j];
+      }
+    }
+  }
+  float kn[RPT], qn[RPT], vn[4];
+  auto load = [&](int t) {
+#pragma unroll
+    for (int r = 0; r < RPT; ++r) {
+      const int i = rg + 32 * r;
+      kn[r] = i < p.dk ? to_f32(k[t * p.k_ld + i]) : 0.f;
+      qn[r] = i < p.dk ? to_f32(q[t * p.q_ld + i]) : 0.f;
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j) vn[j] = c + j < p.dv ? to_f32(v[t * p.v_ld + c + j]) : 0.f;
+  };
+  load(0);
+  for (int t = 0; t < n; ++t) {
+    float o[4] = {0.f, 0.f, 0.f, 0.f}, v4[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) v4[j] = silu_as<T>(vn[j]);
+#pragma unroll
+    for (int r = 0; r < RPT; ++r) {
+      const float kr = silu_as<T>(kn[r]), qr = silu_as<T>(qn[r]);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        s[r][j] = fmaf(decay, s[r][j], kr * v4[j]);
+        o[j] = fmaf(s[r][j], qr, o[j]);
+      }
+    }
+    if (t + 1 < n) load(t + 1);
+#pragma unroll
+    for (int d = 8; d <= 16; d <<= 1)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) o[j] += __shfl_xor_sync(0xffffffffu, o[j], d);
+    const int par = t & 1;
+    if (lane < 8) red[par][warp][cl] = make_float4(o[0], o[1], o[2], o[3]);
+    __syncthreads();     // one barrier per token: the next token writes the other half of the buffer
+    if (rg == 0) {
+      float4 a = red[par][0][cl];
+#pragma unroll
+      for (int w = 1; w < 8; ++w) {
+        const float4 x = red[par][w][cl];
+        a.x += x.x;
+        a.y += x.y;
+        a.z += x.z;
+        a.w += x.w;
+      }
+      const float r4[4] = {a.x, a.y, a.z, a.w};
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (c + j < p.dv) out[static_cast<int64_t>(t) * p.heads * p.dv + c + j] = from_f32<T>(r4[j]);
+    }
+  }
+#pragma unroll
+  for (int r = 0; r < RPT; ++r) {
+    const int i = rg + 32 * r;
+    if (i < p.dk) {
+      if (vec && c < p.dv) {
+        *reinterpret_cast<float4*>(S + static_cast<int64_t>(i) * p.dv + c) = *reinterpret_cast<const float4*>(s[r]);
+      } else {
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+          if (c + j < p.dv) S[static_cast<int64_t>(i) * p.dv + c + j] = s[r][j];
+      }
+    }
+  }
+}
+
+// ---------------------------------------------------------------------------------------------
+// 64 tokens at a time: grid (ceil(dv / 64), heads, batch), 256 threads.  The columns of S never mix, so a CTA owns one
+// (request, head) and 64 of them, with the state in the accumulators of its 8 warps for the whole sequence.  DK: dk
+// rounded up to 32, 64 or 128 (missing features are zero).
+// ---------------------------------------------------------------------------------------------
+using bf16 = __nv_bfloat16;
+constexpr int kLcTok = 64, kLcV = 64, kLcLdV = kLcV + 8, kLcThreads = 256;
+
+template <int DK>
+struct LightningCfg {
+  static constexpr int kLd = DK + 8;
+  static constexpr int kElems = 2 * kLcTok * kLd + 4 * kLcTok * kLcLdV + 2 * DK * kLcLdV;
+  static constexpr int kSmem = kElems * 2 + (kLcTok + 1) * 4;
+};
+
+__device__ __forceinline__ float bf16_part(float x, float& rest) {
+  const float hi = __bfloat162float(__float2bfloat16_rn(x));
+  rest = x - hi;
+  return hi;
+}
+// a pair of fp32 values as two or three bf16 terms, each packed for an operand register
+__device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
+  float ra, rb;
+  const float ha = bf16_part(a, ra), hb = bf16_part(b, rb);
+  hi = pack_bf16x2(ha, hb);
+  lo = pack_bf16x2(ra, rb);
+}
+
+template <int DK>
+__global__ void __launch_bounds__(kLcThreads, 2) lightning_chunk_kernel(const LightningArgs p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  using C = LightningCfg<DK>;
+  constexpr int kLd = C::kLd, kMT = DK / 16, kCG = 8 / kMT, kNT = 8 / kCG;   // row tiles of S, column groups, n tiles per warp
+  extern __shared__ __align__(16) uint8_t lc_smem[];
+  bf16* sQ = reinterpret_cast<bf16*>(lc_smem);      // [64][DK + 8]
+  bf16* sK = sQ + kLcTok * kLd;                     // [64][DK + 8]
+  bf16* sV = sK + kLcTok * kLd;                     // [64][72] values
+  bf16* sW = sV + kLcTok * kLcLdV;                  // [3][64][72] terms of decay^(n-1-j) v_j
+  bf16* sS = sW + 3 * kLcTok * kLcLdV;              // [2][DK][72] terms of the state before the chunk
+  float* sPow = reinterpret_cast<float*>(sS + 2 * DK * kLcLdV);   // decay^0 .. decay^64
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int vb = blockIdx.x * kLcV, h = blockIdx.y, b = blockIdx.z;
+  const int n = p.lens[b];
+  if (n <= 0) return;
+  const int dk = p.dk, dv = p.dv, cols = min(kLcV, dv - vb);
+  const int64_t row0 = p.q_start[b];
+  const bf16* q = static_cast<const bf16*>(p.q) + row0 * p.q_ld + static_cast<int64_t>(h) * dk;
+  const bf16* k = static_cast<const bf16*>(p.k) + row0 * p.k_ld + static_cast<int64_t>(h) * dk;
+  const bf16* v = static_cast<const bf16*>(p.v) + row0 * p.v_ld + static_cast<int64_t>(h) * dv + vb;
+  bf16* out = static_cast<bf16*>(p.out) + (row0 * p.heads + h) * dv + vb;
+  float* S = p.state + (static_cast<int64_t>(p.slots[b]) * p.heads + h) * dk * dv + vb;
+  const bool resume = p.has_state[b] != 0;
+  if (tid <= kLcTok) sPow[tid] = powf(p.decay[h], static_cast<float>(tid));
+
+  // this warp's part of S: row tile mt, n tiles n0 .. n0 + kNT - 1
+  const int mt = warp % kMT, n0 = (warp / kMT) * kNT;
+  const int g = lane >> 2, c2 = (lane & 3) * 2;
+  float st[kNT][4];
+#pragma unroll
+  for (int nt = 0; nt < kNT; ++nt)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int i = mt * 16 + g + (e >> 1) * 8, c = (n0 + nt) * 8 + c2 + (e & 1);
+      st[nt][e] = resume && i < dk && c < cols ? S[static_cast<int64_t>(i) * dv + c] : 0.f;
+    }
+  __syncthreads();
+
+  for (int c0 = 0; c0 < n; c0 += kLcTok) {
+    const int nv = min(kLcTok, n - c0);
+    // ---- rows of the chunk: activated, missing rows and features zero; the values also scaled, in three terms ----
+    auto load8 = [&](const bf16* src, bool valid, float (&f)[8]) {
+      uint4 raw = make_uint4(0u, 0u, 0u, 0u);
+      if (valid) raw = *reinterpret_cast<const uint4*>(src);
+      const uint32_t* u = reinterpret_cast<const uint32_t*>(&raw);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float2 t = unpack_bf16x2(u[i]);
+        f[2 * i] = silu_as<bf16>(t.x);
+        f[2 * i + 1] = silu_as<bf16>(t.y);
+      }
+    };
+    auto pack8 = [](const float (&f)[8]) {
+      return make_uint4(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]), pack_bf16x2(f[4], f[5]), pack_bf16x2(f[6], f[7]));
+    };
+#pragma unroll
+    for (int it = 0; it < kLcTok * DK / 8 / kLcThreads; ++it) {
+      const int i = tid + it * kLcThreads, r = i / (DK / 8), d = (i % (DK / 8)) * 8;
+      const bool valid = r < nv && d < dk;
+      float f[8];
+      load8(q + static_cast<int64_t>(c0 + r) * p.q_ld + d, valid, f);
+      *reinterpret_cast<uint4*>(sQ + r * kLd + d) = pack8(f);
+      load8(k + static_cast<int64_t>(c0 + r) * p.k_ld + d, valid, f);
+      *reinterpret_cast<uint4*>(sK + r * kLd + d) = pack8(f);
+    }
+#pragma unroll
+    for (int it = 0; it < kLcTok * kLcV / 8 / kLcThreads; ++it) {
+      const int i = tid + it * kLcThreads, r = i / (kLcV / 8), d = (i % (kLcV / 8)) * 8;
+      float f[8], hi[8];
+      load8(v + static_cast<int64_t>(c0 + r) * p.v_ld + d, r < nv && d < cols, f);
+      *reinterpret_cast<uint4*>(sV + r * kLcLdV + d) = pack8(f);
+      const float w = r < nv ? sPow[nv - 1 - r] : 0.f;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) f[j] *= w;
+#pragma unroll
+      for (int t = 0; t < 3; ++t) {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) hi[j] = bf16_part(f[j], f[j]);
+        *reinterpret_cast<uint4*>(sW + (t * kLcTok + r) * kLcLdV + d) = pack8(hi);
+      }
+    }
+    // ---- the state before the chunk as an operand ----
+#pragma unroll
+    for (int nt = 0; nt < kNT; ++nt)
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        uint32_t hi, lo;
+        split2(st[nt][half * 2], st[nt][half * 2 + 1], hi, lo);
+        bf16* dst = sS + (mt * 16 + g + half * 8) * kLcLdV + (n0 + nt) * 8 + c2;
+        *reinterpret_cast<uint32_t*>(dst) = hi;
+        *reinterpret_cast<uint32_t*>(dst + DK * kLcLdV) = lo;
+      }
+    __syncthreads();
+
+    // ---- outputs: 16 rows and 32 columns per warp ----
+    {
+      const int rt = warp & 3, oc = (warp >> 2) * 32;
+      if (rt * 16 < nv) {
+        float o[4][4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+        uint32_t qa[kMT][4];
+#pragma unroll
+        for (int kk = 0; kk < kMT; ++kk) {
+          ldsm4(qa[kk], smem_u32(sQ + (rt * 16 + (lane & 15)) * kLd + kk * 16 + (lane >> 4) * 8));
+#pragma unroll
+          for (int t = 0; t < 2; ++t)
+#pragma unroll
+            for (int np = 0; np < 2; ++np) {
+              uint32_t bb[4];
+              ldsm4_t(bb, smem_u32(sS + (t * DK + kk * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * kLcLdV + oc + np * 16 + (lane >> 4) * 8));
+              mma_16816<bf16>(o[np * 2], qa[kk][0], qa[kk][1], qa[kk][2], qa[kk][3], bb[0], bb[1]);
+              mma_16816<bf16>(o[np * 2 + 1], qa[kk][0], qa[kk][1], qa[kk][2], qa[kk][3], bb[2], bb[3]);
+            }
+        }
+        const int ra = rt * 16 + g, rb = ra + 8;
+        const float da = sPow[ra + 1], db = sPow[rb + 1];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          o[i][0] *= da;
+          o[i][1] *= da;
+          o[i][2] *= db;
+          o[i][3] *= db;
+        }
+#pragma unroll 1
+        for (int jt = 0; jt <= rt; ++jt) {
+          float s[2][4];
+#pragma unroll
+          for (int i = 0; i < 2; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
+#pragma unroll
+          for (int kk = 0; kk < kMT; ++kk) {
+            uint32_t bb[4];
+            ldsm4(bb, smem_u32(sK + (jt * 16 + (lane >> 4) * 8 + (lane & 7)) * kLd + kk * 16 + ((lane >> 3) & 1) * 8));
+            mma_16816<bf16>(s[0], qa[kk][0], qa[kk][1], qa[kk][2], qa[kk][3], bb[0], bb[1]);
+            mma_16816<bf16>(s[1], qa[kk][0], qa[kk][1], qa[kk][2], qa[kk][3], bb[2], bb[3]);
+          }
+#pragma unroll
+          for (int i = 0; i < 2; ++i)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const int d = ((e >> 1) ? rb : ra) - (jt * 16 + i * 8 + c2 + (e & 1));
+              s[i][e] = d >= 0 ? s[i][e] * sPow[d] : 0.f;
+            }
+          uint32_t ph[4], pl[4];
+          split2(s[0][0], s[0][1], ph[0], pl[0]);
+          split2(s[0][2], s[0][3], ph[1], pl[1]);
+          split2(s[1][0], s[1][1], ph[2], pl[2]);
+          split2(s[1][2], s[1][3], ph[3], pl[3]);
+#pragma unroll
+          for (int np = 0; np < 2; ++np) {
+            uint32_t bb[4];
+            ldsm4_t(bb, smem_u32(sV + (jt * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * kLcLdV + oc + np * 16 + (lane >> 4) * 8));
+            mma_16816<bf16>(o[np * 2], ph[0], ph[1], ph[2], ph[3], bb[0], bb[1]);
+            mma_16816<bf16>(o[np * 2 + 1], ph[0], ph[1], ph[2], ph[3], bb[2], bb[3]);
+            mma_16816<bf16>(o[np * 2], pl[0], pl[1], pl[2], pl[3], bb[0], bb[1]);
+            mma_16816<bf16>(o[np * 2 + 1], pl[0], pl[1], pl[2], pl[3], bb[2], bb[3]);
+          }
+        }
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int c = oc + i * 8 + c2;
+          if (c < cols) {      // dv is even: pairs never straddle the end
+            if (ra < nv)
+              *reinterpret_cast<uint32_t*>(out + static_cast<int64_t>(c0 + ra) * p.heads * dv + c) = pack_bf16x2(o[i][0], o[i][1]);
+            if (rb < nv)
+              *reinterpret_cast<uint32_t*>(out + static_cast<int64_t>(c0 + rb) * p.heads * dv + c) = pack_bf16x2(o[i][2], o[i][3]);
+          }
+        }
+      }
+    }
+    // ---- S' = decay^n S + K^T W ----
+    const float carry = sPow[nv];
+#pragma unroll
+    for (int nt = 0; nt < kNT; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) st[nt][e] *= carry;
+#pragma unroll
+    for (int kt = 0; kt < kLcTok / 16; ++kt) {
+      if (kt * 16 < nv) {
+        uint32_t ka[4];
+        ldsm4_t(ka, smem_u32(sK + (kt * 16 + (lane >> 4) * 8 + (lane & 7)) * kLd + mt * 16 + ((lane >> 3) & 1) * 8));
+#pragma unroll
+        for (int t = 0; t < 3; ++t)
+#pragma unroll
+          for (int np = 0; np < kNT / 2; ++np) {
+            uint32_t bb[4];
+            ldsm4_t(bb, smem_u32(sW + (t * kLcTok + kt * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * kLcLdV + (n0 + np * 2) * 8 + (lane >> 4) * 8));
+            mma_16816<bf16>(st[np * 2], ka[0], ka[1], ka[2], ka[3], bb[0], bb[1]);
+            mma_16816<bf16>(st[np * 2 + 1], ka[0], ka[1], ka[2], ka[3], bb[2], bb[3]);
+          }
+      }
+    }
+    __syncthreads();      // every operand of this chunk has been read
+  }
+#pragma unroll
+  for (int nt = 0; nt < kNT; ++nt)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int i = mt * 16 + g + (e >> 1) * 8, c = (n0 + nt) * 8 + c2 + (e & 1);
+      if (i < dk && c < cols) S[static_cast<int64_t>(i) * dv + c] = st[nt][e];
+    }
+}
+
+template <typename T>
+int launch_recurrent_t(const LightningArgs& p, cudaStream_t s) {
+  const dim3 grid((p.dv + 31) / 32, p.heads, p.batch), block(256);
+  if (p.dk <= 32) launch_pdl(lightning_recurrent_kernel<T, 1>, grid, block, 0, s, p);
+  else if (p.dk <= 64) launch_pdl(lightning_recurrent_kernel<T, 2>, grid, block, 0, s, p);
+  else if (p.dk <= 128) launch_pdl(lightning_recurrent_kernel<T, 4>, grid, block, 0, s, p);
+  else if (p.dk <= 256) launch_pdl(lightning_recurrent_kernel<T, 8>, grid, block, 0, s, p);
+  else if (p.dk <= 512) launch_pdl(lightning_recurrent_kernel<T, 16>, grid, block, 0, s, p);
+  else return -1;
+  note_launch();
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+template <int DK>
+int launch_chunk_t(const LightningArgs& p, cudaStream_t s) {
+  if (ensure_dynamic_smem(reinterpret_cast<const void*>(lightning_chunk_kernel<DK>), LightningCfg<DK>::kSmem) != cudaSuccess) return -3;
+  const cudaError_t err = launch_pdl(lightning_chunk_kernel<DK>, dim3((p.dv + kLcV - 1) / kLcV, p.heads, p.batch), dim3(kLcThreads),
+                                     LightningCfg<DK>::kSmem, s, p);
+  note_launch();
+  return err == cudaSuccess ? 0 : -4;
+}
+
+}  // namespace
+
+int launch_lightning_recurrent(const LightningArgs& p, cudaStream_t s) {
+  if (p.batch <= 0) return 0;
+  int rc = 0;
+  MB200_DISPATCH_FLOAT(p.dt, rc = launch_recurrent_t<T>(p, s));
+  return rc;
+}
+
+bool lightning_chunk_covers(const LightningArgs& p) {
+  // rows move in 16-byte pieces
+  return p.dt == kBF16 && p.dk <= 128 && p.dk % 8 == 0 && p.dv % 8 == 0 && p.q_ld % 8 == 0 && p.k_ld % 8 == 0 && p.v_ld % 8 == 0 &&
+         ((reinterpret_cast<uintptr_t>(p.q) | reinterpret_cast<uintptr_t>(p.k) | reinterpret_cast<uintptr_t>(p.v)) & 15) == 0;
+}
+
+int launch_lightning_chunk(const LightningArgs& p, cudaStream_t s) {
+  if (p.batch <= 0) return 0;
+  if (!lightning_chunk_covers(p)) return -1;
+  return p.dk <= 32 ? launch_chunk_t<32>(p, s) : p.dk <= 64 ? launch_chunk_t<64>(p, s) : launch_chunk_t<128>(p, s);
+}
+
+}  // namespace mb200

@@ -17,6 +17,7 @@
 
 #include "common.cuh"
 #include "kernels.h"
+#include "mma.cuh"
 
 namespace mb200 {
 namespace {
@@ -31,8 +32,9 @@ constexpr int kMaxExperts = 256;
 // router: one warp per token
 // --------------------------------------------------------------------------------------------
 template <typename T>
-__global__ void moe_router_topk_kernel(const T* __restrict__ logits, int64_t stride, float* __restrict__ w_out,
-                                       int* __restrict__ id_out, int tokens, int experts, int top_k, int renorm) {
+__global__ void moe_router_topk_kernel(const T* __restrict__ logits, int64_t stride, const float* __restrict__ correction,
+                                       float* __restrict__ w_out, int* __restrict__ id_out, int tokens, int experts, int top_k,
+                                       int renorm, float renorm_eps) {
   pdl_wait();
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
@@ -50,49 +52,173 @@ __global__ void moe_router_topk_kernel(const T* __restrict__ logits, int64_t str
   float sum = 0.f;
 #pragma unroll
   for (int i = 0; i < kMaxExperts / 32; ++i) {
-    v[i] = (lane + 32 * i) < experts ? __expf(v[i] - mx) : -1.f;  // probabilities are >= 0; -1 = absent
-    if (v[i] > 0.f) sum += v[i];
+    v[i] = (lane + 32 * i) < experts ? expf(v[i] - mx) : 0.f;
+    sum += v[i];
   }
   sum = warp_sum(sum);
   const float inv = 1.f / sum;
+  // the key that is compared: the score, plus the expert's correction; -inf where there is no expert or it is taken
+  float key[kMaxExperts / 32];
+#pragma unroll
+  for (int i = 0; i < kMaxExperts / 32; ++i) {
+    const int e = lane + 32 * i;
+    v[i] *= inv;
+    key[i] = e < experts ? v[i] + (correction != nullptr ? correction[e] : 0.f) : -INFINITY;
+  }
   float chosen_w = 0.f;  // lane j keeps the j-th choice
   int chosen_e = 0;
   float ksum = 0.f;
   for (int j = 0; j < top_k; ++j) {
-    float best = -2.f;
+    float best = -INFINITY, score = 0.f;
     int bi = 0x7fffffff;
 #pragma unroll
     for (int i = 0; i < kMaxExperts / 32; ++i) {
-      if (v[i] > best) {  // ascending i: the lowest index wins ties inside a lane
-        best = v[i];
+      if (key[i] > best) {  // ascending i: the lowest index wins ties inside a lane
+        best = key[i];
+        score = v[i];
         bi = lane + 32 * i;
       }
     }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
       const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+      const float os = __shfl_xor_sync(0xffffffffu, score, o);
       const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
       if (ov > best || (ov == best && oi < bi)) {
         best = ov;
+        score = os;
         bi = oi;
       }
     }
     if ((bi & 31) == lane) {
 #pragma unroll
       for (int i = 0; i < kMaxExperts / 32; ++i)
-        if (i == (bi >> 5)) v[i] = -1.f;
+        if (i == (bi >> 5)) key[i] = -INFINITY;
     }
-    const float pw = best * inv;
-    ksum += pw;
+    ksum += score;
     if (lane == j) {
-      chosen_w = pw;
-      chosen_e = bi;
+      chosen_w = score;
+      chosen_e = bi == 0x7fffffff ? 0 : bi;
     }
   }
   if (lane < top_k) {
-    w_out[static_cast<int64_t>(t) * top_k + lane] = renorm ? chosen_w / ksum : chosen_w;
+    w_out[static_cast<int64_t>(t) * top_k + lane] = renorm ? chosen_w / (ksum + renorm_eps) : chosen_w;
     id_out[static_cast<int64_t>(t) * top_k + lane] = chosen_e;
   }
+}
+
+// --------------------------------------------------------------------------------------------
+// router logits in fp32
+// --------------------------------------------------------------------------------------------
+constexpr int kRlWarps = 4, kRlTokens = 4;
+
+// a warp takes one expert and four tokens (decode batches, fp32); V elements per access
+template <typename T, int V>
+__global__ void __launch_bounds__(kRlWarps * 32) moe_router_rows_kernel(const T* __restrict__ x, int64_t x_ld, const T* __restrict__ w,
+                                                                        float* __restrict__ logits, int tokens, int experts, int hidden) {
+  pdl_launch_dependents();
+  pdl_wait();
+  struct alignas(sizeof(T) * V) Pack { T e[V]; };
+  const int e = blockIdx.y * kRlWarps + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  const int t0 = blockIdx.x * kRlTokens;
+  if (e >= experts) return;
+  const T* we = w + static_cast<int64_t>(e) * hidden;
+  float acc[kRlTokens];
+#pragma unroll
+  for (int i = 0; i < kRlTokens; ++i) acc[i] = 0.f;
+#pragma unroll 4
+  for (int c = lane * V; c < hidden; c += 32 * V) {
+    const Pack wv = *reinterpret_cast<const Pack*>(we + c);
+#pragma unroll
+    for (int i = 0; i < kRlTokens; ++i) {
+      const Pack xv = *reinterpret_cast<const Pack*>(x + static_cast<int64_t>(min(t0 + i, tokens - 1)) * x_ld + c);
+#pragma unroll
+      for (int j = 0; j < V; ++j) acc[i] = fmaf(to_f32(xv.e[j]), to_f32(wv.e[j]), acc[i]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < kRlTokens; ++i) {
+    acc[i] = warp_sum(acc[i]);
+    if (lane == 0 && t0 + i < tokens) logits[static_cast<int64_t>(t0 + i) * experts + e] = acc[i];
+  }
+}
+
+// prefill: 64 tokens x all experts (NT tiles of 8) per CTA, 64 features at a time through a three-stage ring
+constexpr int kRmTok = 64, kRmK = 64, kRmLd = kRmK + 8, kRmStages = 3;
+
+template <typename T, int NT>
+__global__ void __launch_bounds__(128) moe_router_mma_kernel(const T* __restrict__ x, int64_t x_ld, const T* __restrict__ w,
+                                                             float* __restrict__ logits, int tokens, int experts, int hidden) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ __align__(16) uint8_t rm_smem[];
+  constexpr int kRows = kRmTok + NT * 8;                 // token rows, then expert rows
+  T* ring = reinterpret_cast<T*>(rm_smem);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int64_t t0 = static_cast<int64_t>(blockIdx.x) * kRmTok;
+  const int steps = (hidden + kRmK - 1) / kRmK;
+  auto load = [&](int step) {
+    T* dst = ring + (step % kRmStages) * kRows * kRmLd;
+    for (int i = tid; i < kRows * (kRmK / 8); i += 128) {
+      const int r = i / (kRmK / 8), c = (i % (kRmK / 8)) * 8, k = step * kRmK + c;
+      const bool tok = r < kRmTok;
+      const bool valid = k < hidden && (tok ? t0 + r < tokens : r - kRmTok < experts);
+      const T* src = tok ? x + (valid ? t0 + r : 0) * x_ld + (valid ? k : 0) : w + static_cast<int64_t>(valid ? r - kRmTok : 0) * hidden + (valid ? k : 0);
+      cp16_zfill(smem_u32(dst + r * kRmLd + c), src, valid);
+    }
+    cp_commit();
+  };
+  float acc[NT][4];
+#pragma unroll
+  for (int n = 0; n < NT; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
+#pragma unroll
+  for (int i = 0; i < kRmStages - 1; ++i) {
+    if (i < steps) load(i);
+    else cp_commit();
+  }
+  for (int step = 0; step < steps; ++step) {
+    cp_wait<kRmStages - 2>();
+    __syncthreads();
+    if (step + kRmStages - 1 < steps) load(step + kRmStages - 1);
+    else cp_commit();
+    const T* sx = ring + (step % kRmStages) * kRows * kRmLd;
+    const T* sw = sx + kRmTok * kRmLd;
+#pragma unroll
+    for (int kk = 0; kk < kRmK; kk += 16) {
+      uint32_t a[4];
+      ldsm4(a, smem_u32(sx + (warp * 16 + (lane & 15)) * kRmLd + kk + (lane >> 4) * 8));
+#pragma unroll
+      for (int n = 0; n < NT; n += 2) {
+        uint32_t b[4];      // two tiles of 8 experts: (lower, upper 8 features) of the first, then of the second
+        ldsm4(b, smem_u32(sw + (n * 8 + (lane >> 4) * 8 + (lane & 7)) * kRmLd + kk + ((lane >> 3) & 1) * 8));
+        mma_16816<T>(acc[n], a[0], a[1], a[2], a[3], b[0], b[1]);
+        mma_16816<T>(acc[n + 1], a[0], a[1], a[2], a[3], b[2], b[3]);
+      }
+    }
+  }
+#pragma unroll
+  for (int n = 0; n < NT; ++n) {
+    const int e = n * 8 + (lane & 3) * 2;
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int64_t t = t0 + warp * 16 + (lane >> 2) + half * 8;
+      if (t < tokens) {
+        if (e < experts) logits[t * experts + e] = acc[n][half * 2];
+        if (e + 1 < experts) logits[t * experts + e + 1] = acc[n][half * 2 + 1];
+      }
+    }
+  }
+}
+
+template <typename T, int NT>
+int launch_router_mma(const void* x, int64_t x_ld, const void* w, float* logits, int tokens, int experts, int hidden, cudaStream_t s) {
+  auto kern = moe_router_mma_kernel<T, NT>;
+  const int smem = kRmStages * (kRmTok + NT * 8) * kRmLd * static_cast<int>(sizeof(T));
+  if (ensure_dynamic_smem(reinterpret_cast<const void*>(kern), smem) != cudaSuccess) return -3;
+  const cudaError_t err = launch_pdl(kern, dim3((tokens + kRmTok - 1) / kRmTok), dim3(128), smem, s, static_cast<const T*>(x), x_ld,
+                                     static_cast<const T*>(w), logits, tokens, experts, hidden);
+  note_launch();
+  return err == cudaSuccess ? 0 : -4;
 }
 
 // --------------------------------------------------------------------------------------------
@@ -145,15 +271,16 @@ moe_align_kernel(const int* __restrict__ topk_ids, int pairs, int top_k, int exp
   }
 }
 
-// xs[pos, :] = x[src_token[pos], :] for the local pairs (16-byte vectors)
-__global__ void moe_gather_kernel(const uint4* __restrict__ x, int64_t x_stride_v, const int* __restrict__ src_token,
-                                  const int* __restrict__ expert_offsets, int experts, uint4* __restrict__ xs,
+// xs[pos, :] = x[src_token[pos], :] for the local pairs
+template <typename V>
+__global__ void moe_gather_kernel(const V* __restrict__ x, int64_t x_stride_v, const int* __restrict__ src_token,
+                                  const int* __restrict__ expert_offsets, int experts, V* __restrict__ xs,
                                   int row_vecs) {
   pdl_wait();
   const int pos = blockIdx.x;
   if (pos >= expert_offsets[experts]) return;
-  const uint4* src = x + static_cast<int64_t>(src_token[pos]) * x_stride_v;
-  uint4* dst = xs + static_cast<int64_t>(pos) * row_vecs;
+  const V* src = x + static_cast<int64_t>(src_token[pos]) * x_stride_v;
+  V* dst = xs + static_cast<int64_t>(pos) * row_vecs;
   for (int i = threadIdx.x; i < row_vecs; i += blockDim.x) dst[i] = __ldg(src + i);
 }
 
@@ -400,6 +527,50 @@ moe_grouped_gemm_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_c
   }
 }
 
+// The plain grouped product in fp32 arithmetic for any type and size: 64 weight rows x 16 tokens per tile, 256 threads
+// with four tokens each.  Work items are those of moe_align with chunks of 16 rows.
+constexpr int kGaRows = 64, kGaTok = 16, kGaK = 16;
+
+template <typename T>
+__global__ void __launch_bounds__(256) moe_grouped_any_kernel(const T* __restrict__ x, int64_t ldx, const T* __restrict__ w,
+                                                              T* __restrict__ out, int64_t ldc, const int* __restrict__ expert_offsets,
+                                                              const int2* __restrict__ work, const int* __restrict__ n_work, int n, int k) {
+  pdl_wait();
+  __shared__ float sw[kGaK][kGaRows + 1], sx[kGaK][kGaTok];
+  const int tiles = (n + kGaRows - 1) / kGaRows, total = *n_work * tiles;
+  const int col = threadIdx.x & 63, tg = threadIdx.x >> 6;
+  for (int item = blockIdx.x; item < total; item += gridDim.x) {
+    const int2 wk = work[item / tiles];
+    const int c0 = (item % tiles) * kGaRows, row0 = expert_offsets[wk.x] + wk.y * kGaTok;
+    const int valid = min(kGaTok, expert_offsets[wk.x + 1] - row0);
+    const T* we = w + static_cast<int64_t>(wk.x) * n * k;
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    for (int k0 = 0; k0 < k; k0 += kGaK) {
+      __syncthreads();
+      for (int i = threadIdx.x; i < kGaRows * kGaK; i += 256) {
+        const int r = i / kGaK, kk = i % kGaK;
+        sw[kk][r] = c0 + r < n && k0 + kk < k ? to_f32(we[static_cast<int64_t>(c0 + r) * k + k0 + kk]) : 0.f;
+      }
+      {
+        const int r = threadIdx.x / kGaK, kk = threadIdx.x % kGaK;
+        sx[kk][r] = r < valid && k0 + kk < k ? to_f32(x[static_cast<int64_t>(row0 + r) * ldx + k0 + kk]) : 0.f;
+      }
+      __syncthreads();
+#pragma unroll
+      for (int kk = 0; kk < kGaK; ++kk) {
+        const float a = sw[kk][col];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) acc[i] = fmaf(a, sx[kk][tg * 4 + i], acc[i]);
+      }
+    }
+    if (c0 + col < n) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        if (tg * 4 + i < valid) out[static_cast<int64_t>(row0 + tg * 4 + i) * ldc + c0 + col] = from_f32<T>(acc[i]);
+    }
+  }
+}
+
 template <int BN, bool SWIGLU>
 int launch_grouped_cfg(const CUtensorMap& tw, const CUtensorMap& tx, const GroupedParams& p, int grid, cudaStream_t s) {
   using C = GCfg<BN, SWIGLU>;
@@ -413,19 +584,37 @@ int launch_grouped_cfg(const CUtensorMap& tw, const CUtensorMap& tx, const Group
 
 }  // namespace
 
-void launch_moe_router_topk(const void* logits, int64_t stride, float* w, int* ids, int tokens, int experts, int top_k,
-                            int renorm, DType dt, cudaStream_t s) {
+void launch_moe_router_topk(const void* logits, int64_t stride, const float* correction, float* w, int* ids, int tokens, int experts,
+                            int top_k, int renorm, float renorm_eps, DType dt, cudaStream_t s) {
   if (tokens == 0) return;
   const int warps = 8;
   const dim3 grid((tokens + warps - 1) / warps), block(warps * 32);
-  if (dt == kF32) {
-    launch_pdl(moe_router_topk_kernel<float>, grid, block, 0, s, static_cast<const float*>(logits), stride, w, ids, tokens,
-               experts, top_k, renorm);
-  } else {
-    MB200_DISPATCH_HALF(dt, (launch_pdl(moe_router_topk_kernel<T>, grid, block, 0, s, static_cast<const T*>(logits), stride,
-                                        w, ids, tokens, experts, top_k, renorm)));
-  }
+  MB200_DISPATCH_FLOAT(dt, (launch_pdl(moe_router_topk_kernel<T>, grid, block, 0, s, static_cast<const T*>(logits), stride, correction,
+                                       w, ids, tokens, experts, top_k, renorm, renorm_eps)));
   note_launch();
+}
+
+int launch_moe_router_logits(const void* x, int64_t x_ld, const void* w, float* logits, int tokens, int experts, int hidden,
+                             int num_sms, DType dt, cudaStream_t s) {
+  if (tokens <= 0) return 0;
+  if (experts > kMaxExperts) return -1;
+  const uintptr_t ptrs = reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w);
+  const bool rows16 = ptrs % 16 == 0 && hidden % 8 == 0 && x_ld % 8 == 0;
+  if (tokens > 128 && dt != kF32 && rows16) {
+    int rc = 0;
+    MB200_DISPATCH_HALF(dt, rc = experts <= 64    ? (launch_router_mma<T, 8>(x, x_ld, w, logits, tokens, experts, hidden, s))
+                                 : experts <= 128 ? (launch_router_mma<T, 16>(x, x_ld, w, logits, tokens, experts, hidden, s))
+                                                  : (launch_router_mma<T, 32>(x, x_ld, w, logits, tokens, experts, hidden, s)));
+    return rc;
+  }
+  const dim3 grid((tokens + kRlTokens - 1) / kRlTokens, (experts + kRlWarps - 1) / kRlWarps), block(kRlWarps * 32);
+  const bool vec = rows16 && dt != kF32;
+  MB200_DISPATCH_FLOAT(dt, {
+    if (vec) launch_pdl(moe_router_rows_kernel<T, 8>, grid, block, 0, s, static_cast<const T*>(x), x_ld, static_cast<const T*>(w), logits, tokens, experts, hidden);
+    else launch_pdl(moe_router_rows_kernel<T, 1>, grid, block, 0, s, static_cast<const T*>(x), x_ld, static_cast<const T*>(w), logits, tokens, experts, hidden);
+  });
+  note_launch();
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
 void launch_moe_align(const int* topk_ids, int pairs, int top_k, int expert_offset, int experts, int bn, int* sorted_pos,
@@ -436,10 +625,18 @@ void launch_moe_align(const int* topk_ids, int pairs, int top_k, int expert_offs
 }
 
 void launch_moe_gather(const void* x, int64_t x_stride, const int* src_token, const int* expert_offsets, int experts,
-                       void* xs, int pairs, int hidden, cudaStream_t s) {
+                       void* xs, int pairs, int hidden, int elem_bytes, cudaStream_t s) {
   if (pairs == 0) return;
-  launch_pdl(moe_gather_kernel, dim3(pairs), dim3(128), 0, s, static_cast<const uint4*>(x), x_stride / 8, src_token,
-             expert_offsets, experts, static_cast<uint4*>(xs), hidden / 8);
+  auto go = [&](auto unit) {
+    using V = decltype(unit);
+    const int per = static_cast<int>(sizeof(V)) / elem_bytes;
+    launch_pdl(moe_gather_kernel<V>, dim3(pairs), dim3(128), 0, s, static_cast<const V*>(x), x_stride / per, src_token, expert_offsets,
+               experts, static_cast<V*>(xs), hidden / per);
+  };
+  const uintptr_t ptrs = reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(xs);
+  if (ptrs % 16 == 0 && (hidden * elem_bytes) % 16 == 0 && (x_stride * elem_bytes) % 16 == 0) go(uint4{});
+  else if (elem_bytes == 4) go(uint32_t{});
+  else go(uint16_t{});
   note_launch();
 }
 
@@ -488,6 +685,19 @@ int launch_moe_grouped_gemm(const MoeGemmArgs& a, cudaStream_t s) {
 #undef MB200_MOE_CASE
   }
   return -1;
+}
+
+int launch_moe_grouped_gemm_any(const MoeGemmArgs& a, cudaStream_t s) {
+  if (a.rows_cap <= 0) return 0;
+  if (a.swiglu || a.bn != kGaTok) return -1;
+  const int tiles = (a.n + kGaRows - 1) / kGaRows;
+  const int64_t items = static_cast<int64_t>(a.max_work) * tiles;
+  const int grid = static_cast<int>(std::min<int64_t>(std::max<int64_t>(1, items), 148 * 8));
+  MB200_DISPATCH_FLOAT(a.dt, (launch_pdl(moe_grouped_any_kernel<T>, dim3(grid), dim3(256), 0, s, static_cast<const T*>(a.x), a.ldx,
+                                         static_cast<const T*>(a.w), static_cast<T*>(a.out), a.ldc, a.expert_offsets,
+                                         reinterpret_cast<const int2*>(a.work), a.n_work, a.n, a.k)));
+  note_launch();
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
 }  // namespace mb200

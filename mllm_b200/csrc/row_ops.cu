@@ -1,0 +1,383 @@
+// Row-wise kernels of decoders that keep their residual stream in fp32: the norm after the residual sum (with the
+// weighted sum of expert outputs folded in), the prologue of attention layers whose query / key norm spans all heads,
+// the norm of a whole row with a gate, and small element-wise operations.
+//
+// All are bound by memory traffic: a CTA takes one row, 8 or 16 bytes per thread and access, and keeps it in registers
+// between the reduction and the scaling pass.  Rows that no vector access fits (odd widths) take the V = 1 form.
+#include <algorithm>
+
+#include "common.cuh"
+#include "kernels.h"
+
+namespace mb200 {
+namespace {
+
+template <typename T, int V>
+__device__ __forceinline__ void load_vec(const T* p, float (&f)[V]) {
+  struct alignas(sizeof(T) * V) Pack { T e[V]; };
+  const Pack r = *reinterpret_cast<const Pack*>(p);
+#pragma unroll
+  for (int i = 0; i < V; ++i) f[i] = to_f32(r.e[i]);
+}
+template <typename T, int V>
+__device__ __forceinline__ void store_vec(T* p, const float (&f)[V]) {
+  struct alignas(sizeof(T) * V) Pack { T e[V]; };
+  Pack r;
+#pragma unroll
+  for (int i = 0; i < V; ++i) r.e[i] = from_f32<T>(f[i]);
+  *reinterpret_cast<Pack*>(p) = r;
+}
+
+// sums of two values over the CTA (up to 32 warps)
+__device__ __forceinline__ float2 block_sum2(float a, float b) {
+  __shared__ float2 red[33];
+  a = warp_sum(a);
+  b = warp_sum(b);
+  const int w = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  if (lane_id() == 0) red[w] = make_float2(a, b);
+  __syncthreads();
+  if (w == 0) {
+    const float2 t = static_cast<int>(lane_id()) < nw ? red[lane_id()] : make_float2(0.f, 0.f);
+    a = warp_sum(t.x);
+    b = warp_sum(t.y);
+    if (lane_id() == 0) red[32] = make_float2(a, b);
+  }
+  __syncthreads();
+  return red[32];
+}
+
+constexpr int kRowVecs = 8;        // vectors of a row a thread may hold
+constexpr int kMaxChoices = 32;    // experts a token may use
+
+// threads for a row of `vecs` vectors: about two each, at most kRowVecs each (0: the row is too wide)
+inline int row_threads(int vecs) {
+  int t = std::min(1024, std::max(32, ((vecs + 1) / 2 + 31) / 32 * 32));
+  return static_cast<int64_t>(t) * kRowVecs >= vecs ? t : 0;
+}
+
+// ---------------------------------------------------------------------------------------------
+// x <- rmsnorm(alpha * x + ls * y) * w with x in fp32; h = x in the activations' type.  MOE: y is the sum of the row of
+// `y` (a shared expert; may be null), the token's expert rows times their weights and, for choices that name an identity
+// expert, the token's own input times its weight.
+// ---------------------------------------------------------------------------------------------
+template <typename T, int V, bool MOE>
+__global__ void __launch_bounds__(1024) post_norm_kernel(const PostNormArgs p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ int s_pos[kMaxChoices];
+  __shared__ float s_w[kMaxChoices];
+  const int64_t row = blockIdx.x;
+  const int vecs = p.width / V;
+  if constexpr (MOE) {
+    if (static_cast<int>(threadIdx.x) < p.top) {
+      const int64_t at = row * p.top + threadIdx.x;
+      const int pos = p.sorted_pos[at];
+      s_pos[threadIdx.x] = pos >= 0 ? pos : (p.identity_from > 0 && p.ids[at] >= p.identity_from ? -2 : -1);
+      s_w[threadIdx.x] = p.topk_w[at];
+    }
+    __syncthreads();
+  }
+  const float* x = p.x + row * p.width;
+  const T* y = p.y == nullptr ? nullptr : static_cast<const T*>(p.y) + row * p.width;
+  float z[kRowVecs][V];
+  float ss = 0.f;
+#pragma unroll
+  for (int it = 0; it < kRowVecs; ++it) {
+    const int v = threadIdx.x + it * blockDim.x;
+    if (v < vecs) {
+      const int c = v * V;
+      float acc[V], t[V];
+#pragma unroll
+      for (int i = 0; i < V; ++i) acc[i] = 0.f;
+      if (y != nullptr) load_vec<T, V>(y + c, acc);
+      if constexpr (MOE) {
+        for (int j = 0; j < p.top; ++j) {
+          const int pos = s_pos[j];
+          if (pos == -1) continue;
+          const T* src = pos >= 0 ? static_cast<const T*>(p.expert_rows) + static_cast<int64_t>(pos) * p.width
+                                  : static_cast<const T*>(p.token_in) + row * p.width;
+          load_vec<T, V>(src + c, t);
+          const float w = s_w[j];
+#pragma unroll
+          for (int i = 0; i < V; ++i) acc[i] = fmaf(w, t[i], acc[i]);
+        }
+      }
+      if (p.ls != nullptr) {
+        load_vec<float, V>(p.ls + c, t);
+#pragma unroll
+        for (int i = 0; i < V; ++i) acc[i] *= t[i];
+      }
+      load_vec<float, V>(x + c, t);
+#pragma unroll
+      for (int i = 0; i < V; ++i) {
+        z[it][i] = fmaf(p.alpha, t[i], acc[i]);
+        ss = fmaf(z[it][i], z[it][i], ss);
+      }
+    }
+  }
+  const float rstd = 1.f / sqrtf(block_sum2(ss, 0.f).x / static_cast<float>(p.width) + p.eps);
+#pragma unroll
+  for (int it = 0; it < kRowVecs; ++it) {
+    const int v = threadIdx.x + it * blockDim.x;
+    if (v < vecs) {
+      const int c = v * V;
+      float w[V];
+      load_vec<float, V>(p.w + c, w);
+#pragma unroll
+      for (int i = 0; i < V; ++i) z[it][i] *= rstd * w[i];
+      if (p.x_out != nullptr) store_vec<float, V>(p.x_out + row * p.width + c, z[it]);
+      store_vec<T, V>(static_cast<T*>(p.h) + row * p.width + c, z[it]);
+    }
+  }
+}
+
+// out = x * rsqrt(mean(x^2) + eps) * w * sigmoid(gate), the mean over the whole row
+template <typename T, int V>
+__global__ void __launch_bounds__(1024) rmsnorm_sigmoid_gate_kernel(const T* __restrict__ x, const T* __restrict__ gate, int64_t gate_ld,
+                                            const float* __restrict__ w, T* __restrict__ out, int64_t out_ld, int width, float eps) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int64_t row = blockIdx.x;
+  const int vecs = width / V;
+  const T* xr = x + row * width;
+  float z[kRowVecs][V], ss = 0.f;
+#pragma unroll
+  for (int it = 0; it < kRowVecs; ++it) {
+    const int v = threadIdx.x + it * blockDim.x;
+    if (v < vecs) {
+      load_vec<T, V>(xr + v * V, z[it]);
+#pragma unroll
+      for (int i = 0; i < V; ++i) ss = fmaf(z[it][i], z[it][i], ss);
+    }
+  }
+  const float rstd = 1.f / sqrtf(block_sum2(ss, 0.f).x / static_cast<float>(width) + eps);
+#pragma unroll
+  for (int it = 0; it < kRowVecs; ++it) {
+    const int v = threadIdx.x + it * blockDim.x;
+    if (v < vecs) {
+      float g[V], wv[V];
+      load_vec<T, V>(gate + row * gate_ld + v * V, g);
+      load_vec<float, V>(w + v * V, wv);
+#pragma unroll
+      for (int i = 0; i < V; ++i) z[it][i] *= rstd * wv[i] / (1.f + expf(-g[i]));
+      store_vec<T, V>(out + row * out_ld + v * V, z[it]);
+    }
+  }
+}
+
+// ---------------------------------------------------------------------------------------------
+// Attention prologue: row = [q: heads x dim | k: kv_heads x dim | v: kv_heads x vdim] of a token.  RMS norm over all of
+// q and over all of k, rotation of neighbouring features (2i, 2i + 1) below rot_dims, q written to [heads, q_width]
+// with zeros behind dim, K and V to the token's cache slot.  A CTA takes a token; its sines and cosines are computed
+// once.  Angles are formed and reduced in fp64: at large positions an fp32 product is off by more than the result's
+// own rounding, and the reduced argument keeps sincosf on its short path.  U: features per access (8, 2 or 1).
+// ---------------------------------------------------------------------------------------------
+template <typename T, int U>
+__global__ void __launch_bounds__(256) rownorm_rope_kv_kernel(const RowNormRopeArgs p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ float2 s_rot[];       // [rot_dims / 2] cosine, sine
+  const int64_t t = blockIdx.x;
+  const int tid = threadIdx.x, nt = blockDim.x;
+  const T* row = static_cast<const T*>(p.row) + t * p.row_ld;
+  const int nq = p.heads * p.dim, nk = p.kv_heads * p.dim, nv = p.kv_heads * p.vdim;
+  const int64_t slot = p.loc[t];
+  const bool slot_ok = slot >= 0 && slot < p.num_slots;
+  if (!slot_ok && tid == 0 && p.status != nullptr) atomicExch(p.status, kStatusBadIndex);
+  const double pos = static_cast<double>(p.positions[t]);
+  for (int i = tid; i < p.rot_dims / 2; i += nt) {
+    constexpr double kTurn = 6.283185307179586476925286766559;
+    double a = pos * p.inv_freq[i];
+    a -= kTurn * rint(a / kTurn);
+    float s, c;
+    sincosf(static_cast<float>(a), &s, &c);
+    s_rot[i] = make_float2(c, s);
+  }
+  float sq = 0.f, sk = 0.f;
+  for (int u = tid; u < (nq + nk) / U; u += nt) {
+    float f[U], part = 0.f;
+    load_vec<T, U>(row + u * U, f);
+#pragma unroll
+    for (int i = 0; i < U; ++i) part = fmaf(f[i], f[i], part);
+    if (u * U < nq) sq += part;
+    else sk += part;
+  }
+  const float2 sums = block_sum2(sq, sk);       // its barriers also publish s_rot
+  const float rq = 1.f / sqrtf(sums.x / static_cast<float>(nq) + p.eps), rk = 1.f / sqrtf(sums.y / static_cast<float>(nk) + p.eps);
+  for (int u = tid; u < (nq + nk) / U; u += nt) {
+    const int e = u * U;
+    const bool is_q = e < nq;
+    const int at = is_q ? e : e - nq, head = at / p.dim, d = at - head * p.dim;
+    const float r = is_q ? rq : rk;
+    const float* w = (is_q ? p.q_w : p.k_w) + at;
+    float f[U], wv[U];
+    load_vec<T, U>(row + e, f);
+    load_vec<float, U>(w, wv);
+#pragma unroll
+    for (int i = 0; i < U; ++i) f[i] *= r * wv[i];
+    if constexpr (U == 1) {
+      if (d < p.rot_dims) {
+        const int o = (d & 1) ? -1 : 1;
+        const float other = to_f32(row[e + o]) * r * w[o];
+        const float2 cs = s_rot[d >> 1];
+        f[0] = (d & 1) ? f[0] * cs.x + other * cs.y : f[0] * cs.x - other * cs.y;
+      }
+    } else {
+#pragma unroll
+      for (int i = 0; i < U; i += 2) {
+        if (d + i < p.rot_dims) {
+          const float2 cs = s_rot[(d + i) >> 1];
+          const float a = f[i], b = f[i + 1];
+          f[i] = a * cs.x - b * cs.y;
+          f[i + 1] = b * cs.x + a * cs.y;
+        }
+      }
+    }
+    if (is_q) {
+      store_vec<T, U>(static_cast<T*>(p.q_out) + (t * p.heads + head) * p.q_width + d, f);
+    } else if (slot_ok) {
+      store_vec<T, U>(static_cast<T*>(p.k_cache) + slot * p.k_tok_stride + head * p.k_head_stride + d, f);
+    }
+  }
+  if (slot_ok) {
+    for (int u = tid; u < nv / U; u += nt) {
+      const int e = u * U, head = e / p.vdim, d = e - head * p.vdim;
+      float f[U];
+      load_vec<T, U>(row + nq + nk + e, f);
+      store_vec<T, U>(static_cast<T*>(p.v_cache) + slot * p.v_tok_stride + head * p.v_head_stride + d, f);
+    }
+  }
+  const int gap = (p.q_width - p.dim) / U;
+  float zero[U];
+#pragma unroll
+  for (int i = 0; i < U; ++i) zero[i] = 0.f;
+  for (int u = tid; u < p.heads * gap; u += nt) {
+    const int head = u / gap;
+    store_vec<T, U>(static_cast<T*>(p.q_out) + (t * p.heads + head) * p.q_width + p.dim + (u - head * gap) * U, zero);
+  }
+}
+
+// out = cap * tanh(x / cap) in fp32
+template <typename T>
+__global__ void soft_cap_kernel(const T* __restrict__ x, int64_t x_ld, float* __restrict__ out, int64_t total, int width, float cap) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const float inv = 1.f / cap;
+  for (int64_t i = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x; i < total; i += static_cast<int64_t>(gridDim.x) * blockDim.x) {
+    const int64_t r = i / width;
+    out[i] = cap * tanhf(to_f32(x[r * x_ld + (i - r * width)]) * inv);
+  }
+}
+
+// x <- max(x, 0)^2
+template <typename T, int V>
+__global__ void relu_squared_kernel(T* __restrict__ x, int64_t vecs) {
+  pdl_launch_dependents();
+  pdl_wait();
+  for (int64_t i = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x; i < vecs; i += static_cast<int64_t>(gridDim.x) * blockDim.x) {
+    float f[V];
+    load_vec<T, V>(x + i * V, f);
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      const float m = fmaxf(f[j], 0.f);
+      f[j] = m * m;
+    }
+    store_vec<T, V>(x + i * V, f);
+  }
+}
+
+inline bool aligned(const void* p, uintptr_t n) { return (reinterpret_cast<uintptr_t>(p) & (n - 1)) == 0; }
+
+template <typename T, int V>
+int launch_post_norm_v(const PostNormArgs& p, cudaStream_t s) {
+  const int threads = row_threads(p.width / V);
+  if (threads == 0) return -1;
+  if (p.expert_rows != nullptr)
+    launch_pdl(post_norm_kernel<T, V, true>, dim3(p.rows), dim3(threads), 0, s, p);
+  else
+    launch_pdl(post_norm_kernel<T, V, false>, dim3(p.rows), dim3(threads), 0, s, p);
+  note_launch();
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+template <typename T, int V>
+int launch_gate_v(const void* x, const void* gate, int64_t gate_ld, const float* w, void* out, int64_t out_ld, int rows, int width,
+                  float eps, cudaStream_t s) {
+  const int threads = row_threads(width / V);
+  if (threads == 0) return -1;
+  launch_pdl(rmsnorm_sigmoid_gate_kernel<T, V>, dim3(rows), dim3(threads), 0, s, static_cast<const T*>(x), static_cast<const T*>(gate),
+             gate_ld, w, static_cast<T*>(out), out_ld, width, eps);
+  note_launch();
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+template <typename T>
+int launch_rownorm_rope_t(const RowNormRopeArgs& p, cudaStream_t s) {
+  const uintptr_t ptrs = reinterpret_cast<uintptr_t>(p.row) | reinterpret_cast<uintptr_t>(p.q_out) | reinterpret_cast<uintptr_t>(p.k_cache) |
+                         reinterpret_cast<uintptr_t>(p.v_cache) | reinterpret_cast<uintptr_t>(p.q_w) | reinterpret_cast<uintptr_t>(p.k_w);
+  const int64_t sizes = p.dim | p.vdim | p.q_width | p.row_ld | p.k_tok_stride | p.k_head_stride | p.v_tok_stride | p.v_head_stride;
+  const size_t smem = static_cast<size_t>(p.rot_dims / 2) * sizeof(float2) + 8;
+  auto go = [&](auto kernel) {
+    launch_pdl(kernel, dim3(p.tokens), dim3(256), smem, s, p);
+    note_launch();
+    return cudaGetLastError() == cudaSuccess ? 0 : -4;
+  };
+  if (sizes % 8 == 0 && ptrs % 32 == 0 && sizeof(T) == 2) return go(rownorm_rope_kv_kernel<T, 8>);
+  if (sizes % 2 == 0 && ptrs % 8 == 0) return go(rownorm_rope_kv_kernel<T, 2>);
+  return go(rownorm_rope_kv_kernel<T, 1>);
+}
+
+}  // namespace
+
+int launch_post_norm(const PostNormArgs& p, cudaStream_t s) {
+  if (p.rows <= 0) return 0;
+  if (p.expert_rows != nullptr && p.top > kMaxChoices) return -1;
+  const uintptr_t ptrs = reinterpret_cast<uintptr_t>(p.x) | reinterpret_cast<uintptr_t>(p.x_out) | reinterpret_cast<uintptr_t>(p.y) |
+                         reinterpret_cast<uintptr_t>(p.ls) | reinterpret_cast<uintptr_t>(p.w) | reinterpret_cast<uintptr_t>(p.h) |
+                         reinterpret_cast<uintptr_t>(p.expert_rows) | reinterpret_cast<uintptr_t>(p.token_in);
+  const bool vec = p.width % 4 == 0 && ptrs % 16 == 0;
+  int rc = 0;
+  MB200_DISPATCH_FLOAT(p.dt, rc = vec ? launch_post_norm_v<T, 4>(p, s) : launch_post_norm_v<T, 1>(p, s));
+  return rc;
+}
+
+int launch_rmsnorm_sigmoid_gate(const void* x, const void* gate, int64_t gate_ld, const float* w, void* out, int64_t out_ld, int rows,
+                                int width, float eps, DType dt, cudaStream_t s) {
+  if (rows <= 0) return 0;
+  const bool vec = width % 4 == 0 && gate_ld % 4 == 0 && out_ld % 4 == 0 && aligned(x, 16) && aligned(gate, dt == kF32 ? 16 : 8) &&
+                   aligned(w, 16) && aligned(out, dt == kF32 ? 16 : 8);
+  int rc = 0;
+  MB200_DISPATCH_FLOAT(dt, rc = vec ? (launch_gate_v<T, 4>(x, gate, gate_ld, w, out, out_ld, rows, width, eps, s))
+                                    : (launch_gate_v<T, 1>(x, gate, gate_ld, w, out, out_ld, rows, width, eps, s)));
+  return rc;
+}
+
+int launch_rownorm_rope_kv(const RowNormRopeArgs& p, cudaStream_t s) {
+  if (p.tokens <= 0) return 0;
+  if (p.rot_dims % 2 != 0 || p.rot_dims > p.dim || p.rot_dims > 4096 || p.q_width < p.dim) return -1;
+  int rc = 0;
+  MB200_DISPATCH_FLOAT(p.dt, rc = launch_rownorm_rope_t<T>(p, s));
+  return rc;
+}
+
+void launch_soft_cap(const void* x, int64_t x_ld, float* out, int rows, int width, float cap, DType dt, cudaStream_t s) {
+  const int64_t total = static_cast<int64_t>(rows) * width;
+  if (total <= 0) return;
+  const int grid = static_cast<int>(std::min<int64_t>((total + 255) / 256, 148 * 16));
+  MB200_DISPATCH_FLOAT(dt, (launch_pdl(soft_cap_kernel<T>, dim3(grid), dim3(256), 0, s, static_cast<const T*>(x), x_ld, out, total, width, cap)));
+  note_launch();
+}
+
+void launch_relu_squared(void* x, int64_t n, DType dt, cudaStream_t s) {
+  if (n <= 0) return;
+  const bool vec = n % 4 == 0 && aligned(x, 16);
+  const int64_t vecs = vec ? n / 4 : n;
+  const int grid = static_cast<int>(std::min<int64_t>((vecs + 255) / 256, 148 * 16));
+  MB200_DISPATCH_FLOAT(dt, {
+    if (vec) launch_pdl(relu_squared_kernel<T, 4>, dim3(grid), dim3(256), 0, s, static_cast<T*>(x), vecs);
+    else launch_pdl(relu_squared_kernel<T, 1>, dim3(grid), dim3(256), 0, s, static_cast<T*>(x), vecs);
+  });
+  note_launch();
+}
+
+}  // namespace mb200

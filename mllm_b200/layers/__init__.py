@@ -1,7 +1,9 @@
-from .attention import RadixAttention
+from .attention import RadixAttention, RowNormAttention
 from .embedding import VocabParallelEmbedding
 from .linear import ColumnParallelLinear, Linear, MergedLinear, RowParallelLinear
-from .mlp import MLP, ParallelMLP
+from .lightning import LightningAttention
+from .mlp import MLP, ParallelMLP, SquaredReluMLP
 from .latent_attention import LatentAttention, latent_plan
-from .norm import DynamicTanh, GemmaRMSNorm, LayerNorm, RMSNorm
+from .norm import DynamicTanh, GemmaRMSNorm, LayerNorm, PostRMSNorm, RMSNorm
+from .parallel_mixer import ParallelMixer
 from .quantize_base import LinearMethodBase, QuantizeMethodBase, UnquantizedLinearMethod, set_weight_attrs

@@ -9,6 +9,7 @@ from typing import Optional
 import torch
 from torch import nn
 
+from .. import ops
 from .linear import MergedLinear, RowParallelLinear
 
 
@@ -34,6 +35,20 @@ class MLP(nn.Module):
         if self.down_proj.tp_size > 1 and not self.down_proj.reduce_results:
             return self.down_proj.forward_partial(h)
         return self.down_proj(h)
+
+
+class SquaredReluMLP(nn.Module):
+    """``W_down max(W_up x, 0)^2``: no gate; the activation is part of the first GEMM where its kernel has it."""
+
+    def __init__(self, hidden_size: int, intermediate_size: int, params_dtype: Optional[torch.dtype] = None) -> None:
+        super().__init__()
+        dt = params_dtype or torch.get_default_dtype()
+        self.up_proj, self.down_proj = nn.Module(), nn.Module()
+        self.up_proj.weight = nn.Parameter(torch.zeros(intermediate_size, hidden_size, dtype=dt), requires_grad=False)
+        self.down_proj.weight = nn.Parameter(torch.zeros(hidden_size, intermediate_size, dtype=dt), requires_grad=False)
+
+    def forward(self, x: torch.Tensor) -> torch.Tensor:
+        return ops.linear(ops.linear_relu_squared(x, self.up_proj.weight), self.down_proj.weight)
 
 
 ParallelMLP = MLP

@@ -25,19 +25,29 @@ from ..parallel import state as pstate
 
 
 class MoEGate(nn.Module):
-    def __init__(self, hidden_size: int, num_experts: int, top_k: int, norm_topk_prob: bool, params_dtype=None) -> None:
+    """Router.  ``identity``: further outputs that stand for identity experts (the token's input comes back);
+    ``choice_bias``: a correction per output that takes part in the choice but not in the weights; ``renorm_eps`` is
+    added to the sum the weights are divided by.  ``fp32_logits``: the logits are not rounded to the activations' type."""
+
+    def __init__(self, hidden_size: int, num_experts: int, top_k: int, norm_topk_prob: bool, params_dtype=None, identity: int = 0,
+                 choice_bias: bool = False, renorm_eps: float = 0.0, fp32_logits: bool = False) -> None:
         super().__init__()
-        self.top_k, self.norm_topk_prob = top_k, norm_topk_prob
-        self.weight = nn.Parameter(torch.empty(num_experts, hidden_size, dtype=params_dtype or torch.get_default_dtype()),
+        self.top_k, self.norm_topk_prob, self.renorm_eps = top_k, norm_topk_prob, float(renorm_eps)
+        self.fp32_logits = fp32_logits or choice_bias or renorm_eps > 0
+        self.weight = nn.Parameter(torch.empty(num_experts + identity, hidden_size, dtype=params_dtype or torch.get_default_dtype()),
                                    requires_grad=False)
+        self.correction = nn.Parameter(torch.zeros(num_experts + identity, dtype=torch.float32), requires_grad=False) if choice_bias else None
 
     def forward(self, x: torch.Tensor):
+        if self.fp32_logits:
+            return ops.moe_route(x, self.weight, self.top_k, self.norm_topk_prob, self.correction, self.renorm_eps)
         return ops.moe_router_topk(x, self.weight, self.top_k, self.norm_topk_prob)
 
 
 class SparseMoeBlock(nn.Module):
     def __init__(self, hidden_size: int, moe_intermediate_size: int, num_experts: int, top_k: int,
-                 norm_topk_prob: bool = True, params_dtype=None, prefix: str = "") -> None:
+                 norm_topk_prob: bool = True, params_dtype=None, prefix: str = "", identity_experts: int = 0,
+                 choice_bias: bool = False, renorm_eps: float = 0.0, fp32_logits: bool = False) -> None:
         super().__init__()
         ep = pstate.get_ep_group()
         self.ep_size, self.ep_rank = ep.world_size, ep.rank_in_group
@@ -51,7 +61,10 @@ class SparseMoeBlock(nn.Module):
         self.inter_shard = 1 if self.ep_size > 1 else self.tp_size
         self.inter = moe_intermediate_size // self.inter_shard
         dt = params_dtype or torch.get_default_dtype()
-        self.gate = MoEGate(hidden_size, num_experts, top_k, norm_topk_prob, dt)
+        self.gate = MoEGate(hidden_size, num_experts, top_k, norm_topk_prob, dt, identity_experts, choice_bias, renorm_eps, fp32_logits)
+        self.identity_from = num_experts if identity_experts else 0     # router outputs from here on have no weights
+        if identity_experts and (self.ep_size > 1 or self.inter_shard > 1):
+            raise NotImplementedError("identity experts are not sharded over ranks")
         self.w13 = nn.Parameter(torch.empty(self.local_experts, 2 * self.inter, hidden_size, dtype=dt), requires_grad=False)
         self.w2 = nn.Parameter(torch.empty(self.local_experts, hidden_size, self.inter, dtype=dt), requires_grad=False)
         self.w13.weight_loader = self._load_w13
@@ -84,7 +97,8 @@ class SparseMoeBlock(nn.Module):
 
     def process_weights_after_loading(self) -> None:
         """Interleave gate/up rows in blocks of 128 so the first GEMM can fuse the SwiGLU."""
-        if self.swiglu_block == 0 and (2 * self.inter) % (2 * ops.SWIGLU_BLOCK) == 0 and self.w13.is_cuda:
+        if self.swiglu_block == 0 and (2 * self.inter) % (2 * ops.SWIGLU_BLOCK) == 0 and self.w13.is_cuda \
+                and self.w13.dtype != torch.float32 and self.w13.shape[2] % 8 == 0:
             w = self.w13.data
             for e in range(w.shape[0]):
                 w[e] = ops.ref.interleave_gate_up(w[e].clone(), ops.SWIGLU_BLOCK)
@@ -100,9 +114,16 @@ class SparseMoeBlock(nn.Module):
         shard = self._exchange(x)
         if shard is not None:
             return shard
+        if self.identity_from:
+            raise NotImplementedError("identity experts are summed by the norm behind the block: use expert_rows")
         topk_w, topk_ids = self.gate(x)
         return ops.moe_experts(x, self.w13, self.w2, topk_w, topk_ids, self.expert_offset, self.swiglu_block,
                                self.num_experts)
+
+    def expert_rows(self, x: torch.Tensor) -> "ops.ExpertRows":
+        """The routed experts' outputs before they are summed, for a norm that does it (one GPU per replica)."""
+        topk_w, topk_ids = self.gate(x)
+        return ops.moe_expert_rows(x, self.w13, self.w2, topk_w, topk_ids, self.swiglu_block, self.identity_from)
 
     def can_exchange(self, rows: int) -> bool:
         """Whether a batch of ``rows`` tokens can go through the expert-parallel exchange on this block."""

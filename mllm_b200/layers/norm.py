@@ -68,6 +68,24 @@ class DynamicTanh(nn.Module):
         return ops.residual_dyt(x, y, mult, self.alpha, self.weight, self.bias, self.out_dtype)
 
 
+class PostRMSNorm(nn.Module):
+    """Norm behind the residual sum, for a residual stream kept in fp32: ``x = rmsnorm(alpha * x + ls * y) * weight``, in
+    one pass.  ``y`` may be a sublayer's output, the expert rows of a mixture (weighted and summed on the way), or both."""
+
+    def __init__(self, hidden_size: int, eps: float, alpha: float, out_dtype: torch.dtype) -> None:
+        super().__init__()
+        self.eps, self.alpha, self.out_dtype = float(eps), float(alpha), out_dtype
+        self.weight = nn.Parameter(torch.ones(hidden_size, dtype=torch.float32), requires_grad=False)
+
+    def forward(self, x: torch.Tensor, y: Optional[torch.Tensor], ls: Optional[torch.Tensor] = None, experts=None) -> torch.Tensor:
+        """``x`` [T, W] fp32 is updated in place; the same rows come back in ``out_dtype``."""
+        return ops.post_norm(x, y, ls, self.alpha, self.weight, self.eps, self.out_dtype, experts=experts)
+
+    def read(self, x: torch.Tensor) -> torch.Tensor:
+        """The norm of ``x`` alone, which stays as it is."""
+        return ops.post_norm(x, None, None, 1.0, self.weight, self.eps, self.out_dtype, update=False)
+
+
 class LayerNorm(nn.Module):
     def __init__(self, hidden_size: int, eps: float = 1e-6, bias: bool = True,
                  params_dtype: Optional[torch.dtype] = None) -> None:

@@ -132,6 +132,38 @@ class LatentPool:
             s.zero_()
 
 
+class LayeredKVPool:
+    """K and V rows of models whose attention layers differ in size: ``shapes[i]`` is layer i's ``(kv heads, key width,
+    value width)``.  Storage of a layer is head-major as in :class:`KVPool`, and so are the slots and pages.  Rows may be
+    wider than the heads: the columns behind them are zero and stay zero."""
+
+    def __init__(self, size: int, shapes: Sequence[Tuple[int, int, int]], dtype: torch.dtype, device: torch.device | str,
+                 page_size: int = 1) -> None:
+        if dtype not in (torch.bfloat16, torch.float16, torch.float32):
+            raise NotImplementedError(f"K and V of layers of different sizes are cached in the activation dtype, not {dtype}")
+        self.page_size = int(page_size)
+        self.size = (int(size) // self.page_size) * self.page_size
+        self.num_slots = self.size + self.page_size
+        self.layer_num, self.shapes = len(shapes), [tuple(s) for s in shapes]
+        self.dtype, self.device = dtype, torch.device(device)
+        self.k_buffer, self.v_buffer = [], []
+        for heads, kw, vw in self.shapes:
+            for buf, width in ((self.k_buffer, kw), (self.v_buffer, vw)):
+                buf.append(torch.zeros((heads, self.num_slots, width), dtype=dtype, device=self.device).transpose(0, 1))
+
+    @staticmethod
+    def cell_bytes(shapes: Sequence[Tuple[int, int, int]], dtype: torch.dtype) -> int:
+        """Bytes one token occupies over all layers."""
+        return sum(h * (k + v) for h, k, v in shapes) * torch.empty((), dtype=dtype).element_size()
+
+    def get_kv_buffer(self, index: int) -> Tuple[torch.Tensor, torch.Tensor]:
+        return self.k_buffer[index], self.v_buffer[index]
+
+    def clear(self) -> None:
+        for t in self.k_buffer + self.v_buffer:
+            t.zero_()
+
+
 class TokenToKVPoolAllocator:
     """Host-side free list of KV slots / pages.
 
@@ -260,8 +292,9 @@ class GDNPool:
 
 
 class LayeredGDNPool(GDNPool):
-    """:class:`GDNPool` for models whose delta-net layers differ in size: ``shapes[i]`` is layer i's
-    ``(value heads, Dk, Dv, convolution channels, taps)``, and each layer has tensors of its own."""
+    """:class:`GDNPool` for models whose recurrent layers differ in size: ``shapes[i]`` is layer i's
+    ``(value heads, Dk, Dv, convolution channels, taps)`` — (0 channels, 1 tap) for a layer without a convolution — and
+    each layer has tensors of its own."""
 
     def __init__(self, shapes: Sequence[Tuple[int, int, int, int, int]], slots: int, device,
                  conv_dtype: torch.dtype = torch.bfloat16, track_slots: int = 0) -> None:

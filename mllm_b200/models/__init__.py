@@ -26,12 +26,14 @@ _REGISTRY: Dict[str, Tuple[str, str]] = {
     "MiniCPMForCausalLM": ("mllm_b200.models.minicpm", "MiniCPMForCausalLM"),
     "MiniCPM4ForCausalLM": ("mllm_b200.models.minicpm", "MiniCPMForCausalLM"),
     "PebulixForCausalLM": ("mllm_b200.models.pebulix", "PebulixForCausalLM"),
+    "KesovikForCausalLM": ("mllm_b200.models.kesovik", "KesovikForCausalLM"),
 }
 
 # designs whose config.json names itself in "architecture" and has a layout of its own: a function that checks the
 # file's content and returns it with the field names the runner reads
 _CONFIG_ADAPTERS: Dict[str, Tuple[str, str]] = {
     "Pebulix": ("mllm_b200.models.pebulix", "adapt_config"),
+    "Kesovik": ("mllm_b200.models.kesovik", "adapt_config"),
 }
 
 

@@ -1,7 +1,7 @@
 """Operator front-end: one Python function per hot op.
 
 For tensors on a GPU every function launches the hand-written sm_100a kernel
-from the in-tree extension modules (``mllm_b200_C``, ``mllm_b200_X``) and raises if they cannot
+from the in-tree extension modules (``mllm_b200_C`` and others) and raises if they cannot
 be loaded — there is no silent framework fallback on a GPU.  For CPU tensors
 (tests, fp32 oracle) the plain-PyTorch statement in :mod:`.reference` runs.
 ``MLLM_B200_FORCE_TORCH=1`` forces the PyTorch statement everywhere, which the
@@ -11,6 +11,7 @@ tests use to compare kernel output against it on the same device.
 from __future__ import annotations
 
 import os
+from dataclasses import dataclass
 from typing import Optional, Tuple
 
 import torch
@@ -26,7 +27,10 @@ class _Kernels:
     first asked for."""
 
     def __init__(self) -> None:
+        from .._build import cuda_modules, module_functions
+
         self.__dict__["_mods"] = {}
+        self.__dict__["_where"] = {fn: m for m in reversed(cuda_modules()) for fn in module_functions(m)}
         self._load("mllm_b200_C")
 
     def _load(self, name: str):
@@ -44,13 +48,11 @@ class _Kernels:
     def __getattr__(self, name: str):
         if name.startswith("_"):
             raise AttributeError(name)
-        for module in ("mllm_b200_C", "mllm_b200_X"):
-            mod = self._mods.get(module) or self._load(module)
-            fn = getattr(mod, name, None)
-            if fn is not None:
-                self.__dict__[name] = fn
-                return fn
-        raise AttributeError(name)
+        module = self._where.get(name)
+        if module is None:
+            raise AttributeError(name)
+        fn = self.__dict__[name] = getattr(self._mods.get(module) or self._load(module), name)
+        return fn
 
     def launch_count(self) -> int:
         return sum(int(m.launch_count()) for m in self._mods.values())
@@ -165,14 +167,80 @@ def embedding(ids: torch.Tensor, table: torch.Tensor) -> torch.Tensor:
     return out.view(*ids.shape, table.shape[1])
 
 
-def embedding_f32(ids: torch.Tensor, table: torch.Tensor) -> torch.Tensor:
-    """Embedding rows widened to fp32: the start of a residual stream that is kept in 32-bit."""
+def embedding_f32(ids: torch.Tensor, table: torch.Tensor, scale: float = 1.0, rounded: bool = False):
+    """Embedding rows times ``scale`` in fp32: the start of a residual stream that is kept in 32-bit.  ``rounded``: also
+    the same in the table's type, ``(stream, rounded stream)``."""
     if not use_kernels(table):
-        return ref.embedding(ids, table).float()
+        x = ref.embedding(ids, table).float() * scale
+        return (x, x.to(table.dtype)) if rounded else x
     flat = ids.reshape(-1).to(torch.int64).contiguous()
     out = torch.empty((flat.numel(), table.shape[1]), dtype=torch.float32, device=table.device)
-    ext().embedding_f32(flat, table, out)
-    return out.view(*ids.shape, table.shape[1])
+    h = torch.empty_like(out, dtype=table.dtype) if rounded else None
+    ext().embedding_f32(flat, table, float(scale), out, h)
+    out = out.view(*ids.shape, table.shape[1])
+    return (out, h.view(out.shape)) if rounded else out
+
+
+@dataclass
+class ExpertRows:
+    """Outputs of the chosen experts before they are weighted and summed."""
+
+    rows: torch.Tensor          # [pairs, W]
+    sorted_pos: torch.Tensor    # [T * k] row of every (token, choice); negative: no row
+    topk_w: torch.Tensor        # [T, k] fp32
+    ids: torch.Tensor           # [T, k] int32
+    token_in: torch.Tensor      # [T, W] the experts' input
+    identity_from: int = 0      # > 0: ids from here on return the token's input
+
+
+def post_norm(x: torch.Tensor, y: Optional[torch.Tensor], ls: Optional[torch.Tensor], alpha: float, weight: torch.Tensor, eps: float,
+              dtype: torch.dtype, update: bool = True, experts: Optional[ExpertRows] = None) -> torch.Tensor:
+    """``x = rmsnorm(alpha * x + ls * (y + weighted expert rows)) * weight`` for an fp32 stream ``x`` [T, W] (in place
+    when ``update``), returned in ``dtype`` too.  ``y`` [T, W] and ``ls`` [W] may be None."""
+    if not use_kernels(x):
+        return ref.post_norm(x, y, ls, alpha, weight, eps, dtype, update, experts)
+    h = torch.empty(x.shape, dtype=dtype, device=x.device)
+    e = experts
+    parts = [] if e is None else [e.rows, e.sorted_pos, e.topk_w, e.ids, e.token_in]
+    ext().post_norm(x, y, ls, float(alpha), weight, float(eps), h, update, parts, 0 if e is None else e.identity_from)
+    return h
+
+
+def rmsnorm_sigmoid_gate(x: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor) -> torch.Tensor:
+    """``out = rmsnorm(x) * weight * sigmoid(gate)``, the norm over whole rows; ``gate`` and ``out`` may be column slices."""
+    if not use_kernels(x):
+        return out.copy_(ref.rmsnorm_sigmoid_gate(x, gate, weight, eps))
+    ext().rmsnorm_sigmoid_gate(x, gate, weight, out, float(eps))
+    return out
+
+
+def rownorm_rope_kv(row, q_weight, k_weight, inv_freq, positions, loc, q_out, k_cache, v_cache, heads: int, kv_heads: int, dim: int,
+                    vdim: int, eps: float) -> None:
+    """Prologue of attention whose query / key norm spans all heads: ``row`` [T, q | k | v]; RMS norm over all of q and
+    over all of k, rotation of neighbouring features by ``positions * inv_freq`` (fp64, one per rotated pair), q into
+    ``q_out`` [T, heads, >= dim] (zeros behind), k and v into the cache slots ``loc``."""
+    args = (row, q_weight, k_weight, inv_freq, positions, loc, q_out, k_cache, v_cache, heads, kv_heads, dim, vdim, eps)
+    if not use_kernels(row):
+        return ref.rownorm_rope_kv(*args)
+    ext().rownorm_rope_kv(row, q_weight, k_weight, inv_freq, positions.to(torch.int64).contiguous(), loc.to(torch.int64).contiguous(),
+                          *args[6:])
+
+
+def soft_cap(x: torch.Tensor, cap: float) -> torch.Tensor:
+    """``cap * tanh(x / cap)`` in fp32."""
+    if not use_kernels(x):
+        return ref.soft_cap(x, cap)
+    out = torch.empty(x.shape, dtype=torch.float32, device=x.device)
+    ext().soft_cap(x, out, float(cap))
+    return out
+
+
+def relu_squared_(x: torch.Tensor) -> torch.Tensor:
+    """``max(x, 0)^2`` in place."""
+    if not use_kernels(x):
+        return ref.relu_squared(x)
+    ext().relu_squared(x)
+    return x
 
 
 def residual_dyt(x: torch.Tensor, y: Optional[torch.Tensor], mult: float, alpha: torch.Tensor, weight: torch.Tensor,
@@ -350,6 +418,22 @@ def linear_swiglu(x: torch.Tensor, weight: torch.Tensor, block: int = SWIGLU_BLO
     else:
         _gemm(x2, weight, o, None, None, 2 if act == "gelu_tanh" else 1, None, None)
     return o.view(*x.shape[:-1], weight.shape[0] // 2)
+
+
+def linear_relu_squared(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
+    """``max(x W^T, 0)^2``, the activation inside the GEMM where its kernel has it (up to 8 rows, more than 256)."""
+    x2 = _2d(x)
+    if use_kernels(x) and _gemm_shape_ok(x2, weight):
+        if x2.stride(-1) != 1 or (x2.stride(0) * x2.element_size()) % 16:
+            x2 = x2.contiguous()
+        if x2.shape[0] <= 8 or x2.shape[0] > 256:
+            o = torch.empty((x2.shape[0], weight.shape[0]), dtype=x.dtype, device=x.device)
+            rc = ext().gemm(x2, weight, o, None, None, 3, None, None, isinstance(weight, torch.nn.Parameter))
+            if rc == 0:
+                return o.view(*x.shape[:-1], weight.shape[0])
+            if rc != 1:
+                raise RuntimeError(f"mllm_b200 gemm: launch failure (code {rc})")
+    return relu_squared_(linear(x, weight))
 
 
 # Off by default: inside a CUDA graph the norm kernel already runs under the ring fill of the GEMM behind it
@@ -694,6 +778,16 @@ def attention_decode(q, k_cache, v_cache, req_to_token, req_pool_indices, seq_le
                                 window=window, logit_cap=logit_cap, sink=sink)
 
 
+def attention_rows(q, k_cache, v_cache, req_to_token, row_req, row_pos, scale: float, out, window: Optional[int] = None,
+                   logit_cap: float = 0.0, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Causal attention for fp32 and for head sizes the tensor-core kernels do not have (key and value widths may
+    differ): row t of ``q`` [rows, Hq, D] is a token of request ``row_req[t]`` at position ``row_pos[t]``."""
+    if not use_kernels(q):
+        return ref.attention_rows(q, k_cache, v_cache, req_to_token, row_req, row_pos, scale, out, int(window or 0), logit_cap, sink)
+    ext().attention_rows(q, k_cache, v_cache, req_to_token, row_req, row_pos, float(scale), out, int(window or 0), float(logit_cap), sink)
+    return out
+
+
 def attention_varlen_bidirectional(q, k, v, cu_seqlens, scale: float) -> torch.Tensor:
     """Bidirectional attention inside each segment; q, k, v [T, H, D].  On the GPU the tcgen05 prefill kernel runs
     without its causal mask, every segment being one "request" whose keys sit at rows ``cu[i]..cu[i+1]`` of k / v;
@@ -943,8 +1037,49 @@ def gated_delta_rule(q, k, v, g, beta, state, state_indices, seq_lens, has_state
 
 
 # --------------------------------------------------------------------------
+# lightning attention (linear attention with a fixed decay per head)
+# --------------------------------------------------------------------------
+def lightning_attention(q, k, v, decay, state, state_indices, seq_lens, has_state, q_start=None) -> torch.Tensor:
+    """``S <- decay S + k v^T``, ``o = S^T q`` with q, k [T, H, D] and v [T, H, Dv] taken through SiLU first; tokens may be
+    rows of wider matrices.  ``state`` fp32 [rows, H, D, Dv] is read where ``has_state`` and always written back;
+    metadata as for :func:`gated_delta_rule`, whose extend-backend choice also holds here."""
+    if not use_kernels(q):
+        lens = seq_lens.tolist() if isinstance(seq_lens, torch.Tensor) else seq_lens
+        has = has_state.tolist() if isinstance(has_state, torch.Tensor) else has_state
+        return ref.lightning_attention(q, k, v, decay, state, state_indices, lens, has).to(v.dtype)
+    lens = seq_lens.to(torch.int32)
+    if q_start is None:
+        q_start = torch.cumsum(lens, 0, dtype=torch.int32) - lens
+    out = torch.empty(v.shape, dtype=v.dtype, device=v.device)
+    q, k, v = (t if t.stride(2) == 1 and t.stride(1) == t.shape[2] else t.contiguous() for t in (q, k, v))
+    args = (q, k, v, decay, state, state_indices.to(torch.int32), lens, has_state.to(torch.int32), q_start.to(torch.int32), out)
+    chunked = _GDN_EXTEND_BACKEND == "cuda_chunkwise" or (
+        _GDN_EXTEND_BACKEND != "mllm_kernel" and q.shape[0] >= 32 * max(1, lens.numel()))
+    if not chunked or ext().lightning_chunk(*args) != 0:
+        ext().lightning_recurrent(*args)
+    return out
+
+
+# --------------------------------------------------------------------------
 # mixture of experts
 # --------------------------------------------------------------------------
+def moe_route(hidden: torch.Tensor, gate_weight: torch.Tensor, top_k: int, renormalize: bool = True,
+              correction: Optional[torch.Tensor] = None, renorm_eps: float = 0.0):
+    """Router with fp32 logits: softmax over all outputs, the ``top_k`` largest of ``scores + correction``, weights from
+    the scores alone (divided by their sum + ``renorm_eps`` when ``renormalize``)."""
+    if not use_kernels(hidden):
+        return ref.moe_router_topk(hidden, gate_weight, top_k, renormalize, correction, renorm_eps)
+    T, E = hidden.shape[0], gate_weight.shape[0]
+    if E > 256 or top_k > 32:
+        raise ValueError(f"moe_route: at most 256 outputs and 32 choices, not {E} and {top_k}")
+    logits = torch.empty((T, E), dtype=torch.float32, device=hidden.device)
+    w = torch.empty((T, top_k), dtype=torch.float32, device=hidden.device)
+    ids = torch.empty((T, top_k), dtype=torch.int32, device=hidden.device)
+    ext().moe_router_logits(hidden, gate_weight, logits)
+    ext().moe_router_topk(logits, w, ids, renormalize, correction, float(renorm_eps))
+    return w, ids
+
+
 def moe_router_topk(hidden: torch.Tensor, gate_weight: torch.Tensor, top_k: int, renormalize: bool = True):
     """Router: fp32 softmax over experts -> sorted top-k -> optional renormalisation."""
     if use_kernels(hidden) and hasattr(ext(), "moe_router_topk") and gate_weight.shape[0] <= 256 and top_k <= 8:
@@ -967,22 +1102,19 @@ def moe_chunk_rows(tokens: int, top_k: int, num_experts_global: int) -> int:
     return 128
 
 
-def _moe_gemm(x, w, out, offsets, work, n_work, bn, swiglu) -> None:
-    rc = ext().moe_grouped_gemm(x, w, out, offsets, work, n_work, bn, swiglu)
+def _moe_gemm(x, w, out, offsets, work, n_work, bn, swiglu, any_size: bool = False) -> None:
+    rc = ext().moe_grouped_gemm(x, w, out, offsets, work, n_work, bn, swiglu, any_size)
     if rc != 0:
         raise RuntimeError(f"mllm_b200 moe_grouped_gemm: unsupported shape or launch failure (code {rc}) for "
                            f"x={tuple(x.shape)} w={tuple(w.shape)}")
 
 
-def moe_experts(x, w13, w2, topk_w, topk_ids, expert_offset: int = 0, swiglu_block: int = 0,
-                num_experts_global: Optional[int] = None) -> torch.Tensor:
-    """Grouped expert MLPs.  On the GPU everything stays on the device (no host read of the routing,
-    so the step can be captured in a CUDA graph): pairs are counting-sorted by expert, activations
-    gathered into expert order, both expert GEMMs run as one grouped tcgen05 launch each (SwiGLU fused
-    into the first when ``w13`` is stored in 128-row gate/up blocks), and the k results per token are
-    summed with the router weights."""
-    if not use_kernels(x):
-        return ref.moe_experts(x, w13, w2, topk_w, topk_ids, expert_offset, swiglu_block)
+def _moe_sorted_rows(x, w13, w2, topk_ids, expert_offset: int, swiglu_block: int, num_experts_global: Optional[int]):
+    """Expert outputs in expert order [pairs, H] and the row of every pair.  Everything stays on the device (no host read
+    of the routing, so the step can be captured in a CUDA graph): pairs are counting-sorted by expert, activations
+    gathered into expert order, and both expert GEMMs run as one grouped launch each — on tcgen05, SwiGLU fused into
+    the first when ``w13`` is stored in 128-row gate/up blocks, or, for fp32 and sizes that are no multiple of 8, on a
+    plain kernel."""
     if swiglu_block not in (0, SWIGLU_BLOCK):
         raise ValueError(f"w13 interleave block must be 0 or {SWIGLU_BLOCK}")
     T, H = x.shape
@@ -991,7 +1123,8 @@ def moe_experts(x, w13, w2, topk_w, topk_ids, expert_offset: int = 0, swiglu_blo
     k = topk_ids.shape[1]
     P = T * k
     dev = x.device
-    bn = moe_chunk_rows(T, k, num_experts_global or E)
+    any_size = x.dtype == torch.float32 or H % 8 != 0 or inter % 8 != 0
+    bn = 16 if any_size else moe_chunk_rows(T, k, num_experts_global or E)
     max_work = E + (P + bn - 1) // bn
     i32 = dict(dtype=torch.int32, device=dev)
     sorted_pos = torch.empty(P, **i32)
@@ -1005,17 +1138,38 @@ def moe_experts(x, w13, w2, topk_w, topk_ids, expert_offset: int = 0, swiglu_blo
     xs = torch.empty((P, H), dtype=x.dtype, device=dev)
     e.moe_gather(x, src_token, offsets, xs)
     h = torch.empty((P, inter), dtype=x.dtype, device=dev)
-    if swiglu_block:
+    if swiglu_block and not any_size:
         _moe_gemm(xs, w13, h, offsets, work, n_work, bn, True)
     else:
+        if swiglu_block:
+            raise ValueError("interleaved gate/up rows need the fused product")
         gu = torch.empty((P, N13), dtype=x.dtype, device=dev)
-        _moe_gemm(xs, w13, gu, offsets, work, n_work, bn, False)
+        _moe_gemm(xs, w13, gu, offsets, work, n_work, bn, False, any_size)
         e.act_and_mul(gu, h, 0)
     ys = torch.empty((P, H), dtype=x.dtype, device=dev)
-    _moe_gemm(h, w2, ys, offsets, work, n_work, bn, False)
-    out = torch.empty((T, H), dtype=x.dtype, device=dev)
-    e.moe_combine(ys, sorted_pos, topk_w.contiguous(), out)
+    _moe_gemm(h, w2, ys, offsets, work, n_work, bn, False, any_size)
+    return ys, sorted_pos
+
+
+def moe_experts(x, w13, w2, topk_w, topk_ids, expert_offset: int = 0, swiglu_block: int = 0,
+                num_experts_global: Optional[int] = None) -> torch.Tensor:
+    """Sum over the k routed experts of ``w * down_e(silu(gate_e(x)) * up_e(x))``."""
+    if not use_kernels(x):
+        return ref.moe_experts(x, w13, w2, topk_w, topk_ids, expert_offset, swiglu_block)
+    ys, sorted_pos = _moe_sorted_rows(x, w13, w2, topk_ids, expert_offset, swiglu_block, num_experts_global)
+    out = torch.empty(x.shape, dtype=x.dtype, device=x.device)
+    ext().moe_combine(ys, sorted_pos, topk_w.contiguous(), out)
     return out
+
+
+def moe_expert_rows(x, w13, w2, topk_w, topk_ids, swiglu_block: int = 0, identity_from: int = 0) -> ExpertRows:
+    """The experts' outputs for a kernel that sums them itself (:func:`post_norm`).  ``identity_from`` > 0: ids from there
+    on are identity experts, which return the token's input and have no row."""
+    if not use_kernels(x):
+        rows, pos = ref.moe_expert_rows(x, w13, w2, topk_ids, swiglu_block)
+    else:
+        rows, pos = _moe_sorted_rows(x, w13, w2, topk_ids, 0, swiglu_block, None)
+    return ExpertRows(rows, pos, topk_w.contiguous(), topk_ids.contiguous(), x.contiguous(), int(identity_from))
 
 
 def ep_moe_exchange(x_own, w13, w2, topk_w, topk_ids, swiglu_block: int, comm) -> torch.Tensor:

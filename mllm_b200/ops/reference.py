@@ -473,15 +473,21 @@ def top_k_top_p_min_p_sample(
 # --------------------------------------------------------------------------
 # mixture of experts
 # --------------------------------------------------------------------------
-def moe_router_topk(hidden: torch.Tensor, gate_weight: torch.Tensor, top_k: int, renormalize: bool = True):
+def moe_router_topk(hidden: torch.Tensor, gate_weight: torch.Tensor, top_k: int, renormalize: bool = True,
+                    correction: Optional[torch.Tensor] = None, renorm_eps: float = 0.0):
     """fp32 ``softmax(hidden @ gate_weight.T)`` over all experts -> top-k (sorted by weight) ->
     optional renormalisation of the k weights (mllm/models/qwen3_moe/modeling_qwen3_moe_fa2.hpp:121-138).
+    With ``correction`` the choice goes by ``scores + correction``, the weights are the scores alone.
     Returns (weights fp32 [T, k], expert ids int32 [T, k])."""
     logits = _f32(hidden) @ _f32(gate_weight).t()
     scores = torch.softmax(logits, dim=-1)
-    w, idx = torch.topk(scores, top_k, dim=-1, sorted=True)
+    if correction is None:
+        w, idx = torch.topk(scores, top_k, dim=-1, sorted=True)
+    else:
+        idx = torch.topk(scores + _f32(correction), top_k, dim=-1, sorted=True).indices
+        w = scores.gather(-1, idx)
     if renormalize:
-        w = w / w.sum(-1, keepdim=True)
+        w = w / (w.sum(-1, keepdim=True) + renorm_eps)
     return w, idx.to(torch.int32)
 
 
@@ -505,9 +511,107 @@ def moe_experts(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_w: to
     return out.to(x.dtype)
 
 
+def moe_expert_rows(x, w13, w2, topk_ids, swiglu_block: int = 0):
+    """Outputs of the chosen experts, a row per (token, choice), and the row of every pair (-1: no such expert)."""
+    T, k = topk_ids.shape
+    rows = torch.zeros((T * k, x.shape[1]), dtype=x.dtype, device=x.device)
+    for e in range(w13.shape[0]):
+        tok, slot = (topk_ids == e).nonzero(as_tuple=True)
+        if tok.numel():
+            rows[tok * k + slot] = linear(linear_swiglu(x[tok], w13[e], swiglu_block), w2[e])
+    flat = topk_ids.reshape(-1)
+    pos = torch.arange(T * k, dtype=torch.int32, device=x.device)
+    return rows, torch.where((flat >= 0) & (flat < w13.shape[0]), pos, torch.full_like(pos, -1))
+
+
 # --------------------------------------------------------------------------
-# fp32 residual stream, Dynamic Tanh, latent attention
+# fp32 residual stream, norms after the sum, Dynamic Tanh, latent attention
 # --------------------------------------------------------------------------
+def post_norm(x, y, ls, alpha, weight, eps, dtype, update=True, experts=None):
+    z = torch.zeros_like(x) if y is None else _f32(y)
+    if experts is not None:
+        T, k = experts.topk_w.shape
+        pos = experts.sorted_pos[: T * k].view(T, k).long()
+        w = _f32(experts.topk_w)
+        part = torch.where((pos >= 0).unsqueeze(-1), _f32(experts.rows)[pos.clamp(min=0)], torch.zeros((), device=x.device))
+        z = z + (part * w.unsqueeze(-1)).sum(1)
+        if experts.identity_from > 0:
+            z = z + _f32(experts.token_in) * (w * (experts.ids >= experts.identity_from)).sum(1, keepdim=True)
+    z = float(alpha) * x + (z if ls is None else _f32(ls) * z)
+    z = z * torch.rsqrt(z.pow(2).mean(-1, keepdim=True) + eps) * _f32(weight)
+    if update:
+        x.copy_(z)
+    return z.to(dtype)
+
+
+def rmsnorm_sigmoid_gate(x, gate, weight, eps):
+    xf = _f32(x)
+    return (xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps) * _f32(weight) * torch.sigmoid(_f32(gate))).to(x.dtype)
+
+
+def rotate_pairs(x: torch.Tensor, positions: torch.Tensor, inv_freq: torch.Tensor) -> torch.Tensor:
+    """x [T, H, D] fp32: neighbouring features (2i, 2i + 1) turn by ``positions * inv_freq[i]``, later ones stay."""
+    n = inv_freq.numel()
+    a = (positions.double().unsqueeze(-1) * inv_freq.double()).unsqueeze(1)
+    c, s = torch.cos(a).float(), torch.sin(a).float()
+    u, v = x[..., 0:2 * n:2], x[..., 1:2 * n:2]
+    turned = torch.stack([u * c - v * s, v * c + u * s], -1).flatten(-2)
+    return torch.cat([turned, x[..., 2 * n:]], -1)
+
+
+def rownorm_rope_kv(row, q_w, k_w, inv_freq, positions, loc, q_out, k_cache, v_cache, heads, kv_heads, dim, vdim, eps):
+    T, nq, nk = row.shape[0], heads * dim, kv_heads * dim
+
+    def norm(t, w):
+        t = _f32(t)
+        return t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps) * _f32(w)
+
+    q = rotate_pairs(norm(row[:, :nq], q_w).view(T, heads, dim), positions, inv_freq)
+    k = rotate_pairs(norm(row[:, nq:nq + nk], k_w).view(T, kv_heads, dim), positions, inv_freq)
+    q_out.zero_()
+    q_out[..., :dim] = q.to(q_out.dtype)
+    k_cache[loc.long(), :, :dim] = k.to(k_cache.dtype)
+    v_cache[loc.long(), :, :vdim] = row[:, nq + nk:nq + nk + kv_heads * vdim].reshape(T, kv_heads, vdim)
+
+
+def soft_cap(x, cap):
+    return torch.tanh(_f32(x) / cap) * cap
+
+
+def relu_squared(x):
+    return x.copy_(torch.relu(x) ** 2)
+
+
+def attention_rows(q, k_cache, v_cache, req_to_token, row_req, row_pos, scale, out, window=0, logit_cap=0.0, sink=None):
+    rep = q.shape[1] // k_cache.shape[1]
+    for t in range(q.shape[0]):
+        pos = int(row_pos[t])
+        lo = max(0, pos - window + 1) if window else 0
+        slots = req_to_token[int(row_req[t]), lo: pos + 1].long()
+        k = _f32(k_cache[slots]).repeat_interleave(rep, 1)                 # [n, H, D]
+        v = _f32(v_cache[slots]).repeat_interleave(rep, 1)
+        s = torch.einsum("hd,nhd->hn", _f32(q[t]), k) * scale
+        if logit_cap:
+            s = logit_cap * torch.tanh(s / logit_cap)
+        out[t] = torch.einsum("hn,nhd->hd", sink_softmax(s, sink), v).to(q.dtype)
+    return out
+
+
+def lightning_attention(q, k, v, decay, state, state_indices, seq_lens, has_state):
+    """q, k [T, H, D], v [T, H, Dv] before their SiLU; the state rows are read where ``has_state`` and written back."""
+    q, k, v = (_f32(torch.nn.functional.silu(_f32(t)).to(t.dtype)) for t in (q, k, v))
+    out = torch.empty(v.shape, dtype=torch.float32, device=v.device)
+    g, at = _f32(decay).view(-1, 1, 1), 0
+    for slot, n, has in zip(state_indices.tolist(), seq_lens, has_state):
+        S = state[slot].clone() if has else torch.zeros_like(state[slot])
+        for t in range(at, at + n):
+            S = g * S + k[t].unsqueeze(-1) * v[t].unsqueeze(-2)
+            out[t] = (S * q[t].unsqueeze(-1)).sum(-2)
+        state[slot] = S
+        at += n
+    return out
+
+
 def residual_dyt(x, y, mult, alpha, weight, bias, dtype):
     if y is not None:
         x.add_(_f32(y), alpha=float(mult))

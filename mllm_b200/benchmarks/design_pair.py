@@ -1,11 +1,12 @@
 """Two decoder presets of equal size side by side, whole and kernel by kernel (random weights, one GPU).
 
     python bench.py --design-pair pebulix-2b:qwen3.5-2b
+    python bench.py --design-pair kesovik-6b:qwen3.5-moe-6b
 
 For each (batch, prompt length) both models prefill one batch and decode; times are CUDA-event medians, decode through
 the captured graphs.  Every step streams the weights and the caches of the model (several GB), so nothing is served
-from L2 between timed iterations.  The kernel table times the kernels that the latent / Dynamic Tanh / GeGLU /
-fp32-recurrence design adds next to the like kernel of the other model at the same size, each with its share of the
+from L2 between timed iterations.  The kernel table times the kernels that the new design adds next to the
+like kernel of the other model at the same size, each with its share of the
 measured roofline: algorithmic bytes over the copy bandwidth or FLOPs over the library GEMM rate, whichever bound is
 the longer one.  Kernel inputs are rotated over copies that together exceed L2."""
 
@@ -233,8 +234,7 @@ def gated_kernels(t: Table, rows: int, heads: int, dim: int) -> None:
           rows * heads * dim * 6.0)
 
 
-def kernel_rows() -> List[dict]:
-    t = Table()
+def pebulix_rows(t: Table) -> None:
     # decode: pebulix-2b (16 heads over latents of 512) and qwen3.5-2b (8 heads of 256 over 2 key / value heads)
     for batch, length in ((1, 2048), (8, 2048), (32, 1024), (4, 16384)):
         latent_kernels(t, batch, length, 16, 512, 128, f"{batch}x{length}")
@@ -252,6 +252,21 @@ def kernel_rows() -> List[dict]:
         product_kernels(t, rows, 2048, 6144)
         gated_kernels(t, rows, 16, 128)
         torch.cuda.empty_cache()
+
+
+def kesovik_rows(t: Table) -> None:
+    from .kesovik_kernels import add_rows
+
+    add_rows(t)
+
+
+# the kernels a design adds, by the first word of its presets
+KERNELS = {"pebulix": pebulix_rows, "kesovik": kesovik_rows}
+
+
+def kernel_rows(preset: str) -> List[dict]:
+    t = Table()
+    KERNELS[preset.split("-")[0]](t)
     ops.check_status()
     by_name = {r["kernel"]: r for r in t.rows}
     for r in t.rows:
@@ -268,7 +283,7 @@ def run(pair: str, reps: int, part: str = "all") -> dict:
     out: Dict[str, Any] = {"metric": "design_pair", "pair": names, "dtype": "bf16", "data": "synthetic (random weights and ids)",
                            "peaks": peaks()}
     if part in ("all", "kernels"):
-        out["kernels"] = kernel_rows()
+        out["kernels"] = kernel_rows(names[0])
     if part in ("all", "models"):
         out["models"] = [row for n in names for row in model_rows(n, SIZES, reps)]
     return out

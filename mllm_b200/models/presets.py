@@ -72,6 +72,10 @@ def _hybrid(hidden, layers, heads, kv_heads, inter, head_dim, lin_k_heads, lin_v
 
 
 PRESETS["qwen3.5-2b"] = _hybrid(2048, 24, 8, 2, 6144, 256, 16, 16)
+PRESETS["qwen3.5-moe-6b"] = dict(
+    PRESETS["qwen3.5-2b"], architectures=["Qwen3_5MoeForCausalLM"], model_type="qwen3_5_moe_text", num_experts=64, num_experts_per_tok=8,
+    moe_intermediate_size=512, shared_expert_intermediate_size=512, norm_topk_prob=True,
+)
 PRESETS["qwen3.5-tiny"] = dict(_hybrid(256, 4, 2, 1, 512, 128, 1, 2, vocab=1024),
                                rope_parameters=dict(rope_theta=1e4, partial_rotary_factor=0.25, rope_type="default",
                                                     mrope_section=[6, 5, 5]))
@@ -99,6 +103,34 @@ def _pebulix(layers, width, ff, vocab, heads, dim, q_rank, kv_rank, delta_heads,
 # hidden size, depth, feed-forward, vocabulary and delta-net heads of qwen3.5-2b
 PRESETS["pebulix-2b"] = _pebulix(24, 2048, 6144, 151936, heads=16, dim=128, q_rank=1024, kv_rank=512, delta_heads=16, delta_dim=128)
 PRESETS["pebulix-tiny"] = _pebulix(4, 128, 256, 1024, heads=2, dim=64, q_rank=64, kv_rank=64, delta_heads=2, delta_dim=32)
+
+
+def _kesovik(layers, width, ff, vocab, heads, kv_heads, dim, window, lin_heads, lin_dim, par_lin_heads, experts, identity, top, expert_ff,
+             shared_ff) -> Dict[str, Any]:
+    """Three lightning layers to one with sliding-window attention beside lightning attention; the first feed-forward is
+    dense, the others are mixtures."""
+    def lightning(n):
+        # half-lives from a few tokens to a few hundred, as a geometric series over the heads
+        return dict(heads=n, dim=lin_dim, vdim=lin_dim, decay=[1.0 - 2.0 ** (-2.0 - 7.0 * i / max(1, n - 1)) for i in range(n)])
+
+    out = []
+    for i in range(layers):
+        mlp = dict(kind="dense", ff=ff) if i == 0 else dict(kind="moe", expert=dict(ff=expert_ff), shared=dict(ff=shared_ff),
+                                                            router=dict(experts=experts, identity=identity, top=top))
+        if (i + 1) % 4:
+            out.append(dict(type="lightning", mlp=mlp, mixer=lightning(lin_heads)))
+        else:
+            left = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, mask=dict(size=window), rot=dict(base=1e6, dims=dim), scale=dim ** -0.5)
+            out.append(dict(type="parallel", mlp=mlp, mixer=dict(left=left, right=lightning(par_lin_heads), left_scale=1.0, right_scale=1.0)))
+    return dict(architecture="Kesovik", layers=out, norm=dict(eps=1e-6), postln_alpha=2.0, embedding=dict(scale=1.0), logit_softcap=30.0,
+                vocab=vocab, width=width, torch_dtype="bfloat16")
+
+
+# hidden size, depth, vocabulary, linear-attention heads and experts of qwen3.5-moe-6b
+PRESETS["kesovik-6b"] = _kesovik(24, 2048, 6144, 151936, heads=16, kv_heads=4, dim=128, window=2048, lin_heads=16, lin_dim=128,
+                                 par_lin_heads=8, experts=64, identity=8, top=8, expert_ff=512, shared_ff=512)
+PRESETS["kesovik-tiny"] = _kesovik(4, 128, 256, 1024, heads=4, kv_heads=2, dim=32, window=48, lin_heads=2, lin_dim=32, par_lin_heads=2,
+                                   experts=6, identity=2, top=2, expert_ff=64, shared_ff=64)
 _VL_VISION = dict(
     depth=24, hidden_size=1024, num_heads=16, intermediate_size=4096, patch_size=16, temporal_patch_size=2,
     spatial_merge_size=2, in_channels=3, out_hidden_size=2048, num_position_embeddings=2304,

@@ -7,7 +7,7 @@ import torch
 
 import pebulix_models as pm
 import pebulix_oracle as oracle
-from pebulix_schedules import cut, run_alone, run_together
+from session_schedules import cut, run_alone, run_together
 
 TOL = 2e-4
 

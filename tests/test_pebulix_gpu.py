@@ -5,7 +5,7 @@ import torch
 
 import pebulix_models as pm
 import pebulix_oracle as oracle
-from pebulix_schedules import cut, run_alone, run_together
+from session_schedules import cut, run_alone, run_together
 from test_pebulix_cpu import _generate, _greedy
 
 pytestmark = pytest.mark.gpu

@@ -280,7 +280,7 @@ __global__ void residual_dyt_kernel(float* __restrict__ x, const T* __restrict__
 
 // embedding rows times a constant, in fp32 (the start of an fp32 residual stream); h (may be null): the same in the
 // table's type; one CTA per token
-template <typename T>
+template <typename T, int V>
 __global__ void embedding_f32_kernel(const int64_t* __restrict__ ids, const T* __restrict__ table, float scale, float* __restrict__ out,
                                      T* __restrict__ h, int width, int vocab, int* status) {
   pdl_launch_dependents();
@@ -288,10 +288,21 @@ __global__ void embedding_f32_kernel(const int64_t* __restrict__ ids, const T* _
   const int64_t id = ids[blockIdx.x];
   const bool ok = id >= 0 && id < vocab;
   if (!ok && threadIdx.x == 0 && status != nullptr) atomicExch(status, kStatusBadIndex);
-  for (int c = threadIdx.x; c < width; c += blockDim.x) {
-    const float v = ok ? to_f32(table[id * width + c]) * scale : 0.f;
-    out[static_cast<int64_t>(blockIdx.x) * width + c] = v;
-    if (h != nullptr) h[static_cast<int64_t>(blockIdx.x) * width + c] = from_f32<T>(v);
+  struct alignas(sizeof(T) * V) Pack { T e[V]; };
+  struct alignas(V == 1 ? 4 : 16) PackF { float e[V]; };
+  const int64_t at = static_cast<int64_t>(blockIdx.x) * width;
+  for (int c = threadIdx.x * V; c < width; c += blockDim.x * V) {
+    Pack r{};
+    PackF f;
+    if (ok) r = *reinterpret_cast<const Pack*>(table + id * width + c);
+#pragma unroll
+    for (int i = 0; i < V; ++i) f.e[i] = ok ? to_f32(r.e[i]) * scale : 0.f;
+    *reinterpret_cast<PackF*>(out + at + c) = f;
+    if (h != nullptr) {
+#pragma unroll
+      for (int i = 0; i < V; ++i) r.e[i] = from_f32<T>(f.e[i]);
+      *reinterpret_cast<Pack*>(h + at + c) = r;
+    }
   }
 }
 
@@ -732,9 +743,15 @@ void launch_residual_dyt(float* x, const void* y, float mult, const float* alpha
 void launch_embedding_f32(const int64_t* ids, const void* table, float scale, float* out, void* h, int tokens, int width, int vocab,
                           DType dt, int* status, cudaStream_t s) {
   if (tokens == 0) return;
-  const int threads = width >= 256 ? 256 : (width + 31) / 32 * 32;
-  MB200_DISPATCH_FLOAT(dt, (launch_pdl(embedding_f32_kernel<T>, dim3(tokens), dim3(threads), 0, s, ids, static_cast<const T*>(table),
-                                       scale, out, static_cast<T*>(h), width, vocab, status)));
+  const uintptr_t ptrs = reinterpret_cast<uintptr_t>(table) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(h);
+  const bool vec = width % 4 == 0 && ptrs % 16 == 0;
+  const int units = vec ? width / 4 : width;
+  const int threads = units >= 512 ? 512 : (units + 31) / 32 * 32;
+  MB200_DISPATCH_FLOAT(dt, {
+    const T* tab = static_cast<const T*>(table);
+    if (vec) launch_pdl(embedding_f32_kernel<T, 4>, dim3(tokens), dim3(threads), 0, s, ids, tab, scale, out, static_cast<T*>(h), width, vocab, status);
+    else launch_pdl(embedding_f32_kernel<T, 1>, dim3(tokens), dim3(threads), 0, s, ids, tab, scale, out, static_cast<T*>(h), width, vocab, status);
+  });
   note_launch();
 }
 

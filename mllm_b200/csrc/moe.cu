@@ -221,6 +221,21 @@ int launch_router_mma(const void* x, int64_t x_ld, const void* w, float* logits,
   return err == cudaSuccess ? 0 : -4;
 }
 
+// the number of expert tiles is a compile-time loop bound: pairs of tiles up to 128 experts
+template <typename T>
+int launch_router_mma_t(const void* x, int64_t x_ld, const void* w, float* logits, int tokens, int experts, int hidden, cudaStream_t s) {
+  switch ((experts + 15) / 16) {
+    case 1: return launch_router_mma<T, 2>(x, x_ld, w, logits, tokens, experts, hidden, s);
+    case 2: return launch_router_mma<T, 4>(x, x_ld, w, logits, tokens, experts, hidden, s);
+    case 3: return launch_router_mma<T, 6>(x, x_ld, w, logits, tokens, experts, hidden, s);
+    case 4: return launch_router_mma<T, 8>(x, x_ld, w, logits, tokens, experts, hidden, s);
+    case 5: return launch_router_mma<T, 10>(x, x_ld, w, logits, tokens, experts, hidden, s);
+    case 6: return launch_router_mma<T, 12>(x, x_ld, w, logits, tokens, experts, hidden, s);
+    case 7: case 8: return launch_router_mma<T, 16>(x, x_ld, w, logits, tokens, experts, hidden, s);
+    default: return launch_router_mma<T, 32>(x, x_ld, w, logits, tokens, experts, hidden, s);
+  }
+}
+
 // --------------------------------------------------------------------------------------------
 // align: counting sort of the pairs by local expert + work list, one CTA
 // --------------------------------------------------------------------------------------------
@@ -602,9 +617,7 @@ int launch_moe_router_logits(const void* x, int64_t x_ld, const void* w, float* 
   const bool rows16 = ptrs % 16 == 0 && hidden % 8 == 0 && x_ld % 8 == 0;
   if (tokens > 128 && dt != kF32 && rows16) {
     int rc = 0;
-    MB200_DISPATCH_HALF(dt, rc = experts <= 64    ? (launch_router_mma<T, 8>(x, x_ld, w, logits, tokens, experts, hidden, s))
-                                 : experts <= 128 ? (launch_router_mma<T, 16>(x, x_ld, w, logits, tokens, experts, hidden, s))
-                                                  : (launch_router_mma<T, 32>(x, x_ld, w, logits, tokens, experts, hidden, s)));
+    MB200_DISPATCH_HALF(dt, rc = launch_router_mma_t<T>(x, x_ld, w, logits, tokens, experts, hidden, s));
     return rc;
   }
   const dim3 grid((tokens + kRlTokens - 1) / kRlTokens, (experts + kRlWarps - 1) / kRlWarps), block(kRlWarps * 32);

@@ -46,13 +46,16 @@ __device__ __forceinline__ float2 block_sum2(float a, float b) {
   return red[32];
 }
 
-constexpr int kRowVecs = 8;        // vectors of a row a thread may hold
+constexpr int kRowElems = 32;      // elements of a row a thread may hold
 constexpr int kMaxChoices = 32;    // experts a token may use
 
-// threads for a row of `vecs` vectors: about two each, at most kRowVecs each (0: the row is too wide)
-inline int row_threads(int vecs) {
-  int t = std::min(1024, std::max(32, ((vecs + 1) / 2 + 31) / 32 * 32));
-  return static_cast<int64_t>(t) * kRowVecs >= vecs ? t : 0;
+// threads for a row of `vecs` vectors of `v` elements: one each up to 256, then up to kRowElems elements each (0: the row
+// is too wide)
+inline int row_threads(int vecs, int v) {
+  const int most = kRowElems / v;
+  int t = std::min(256, (vecs + 31) / 32 * 32);
+  while (t < 1024 && static_cast<int64_t>(t) * most < vecs) t *= 2;
+  return static_cast<int64_t>(t) * most >= vecs ? t : 0;
 }
 
 // ---------------------------------------------------------------------------------------------
@@ -64,25 +67,36 @@ template <typename T, int V, bool MOE>
 __global__ void __launch_bounds__(1024) post_norm_kernel(const PostNormArgs p) {
   pdl_launch_dependents();
   pdl_wait();
-  __shared__ int s_pos[kMaxChoices];
+  __shared__ const T* s_src[kMaxChoices];
   __shared__ float s_w[kMaxChoices];
   const int64_t row = blockIdx.x;
   const int vecs = p.width / V;
+  int choices = 0;
   if constexpr (MOE) {
-    if (static_cast<int>(threadIdx.x) < p.top) {
-      const int64_t at = row * p.top + threadIdx.x;
-      const int pos = p.sorted_pos[at];
-      s_pos[threadIdx.x] = pos >= 0 ? pos : (p.identity_from > 0 && p.ids[at] >= p.identity_from ? -2 : -1);
-      s_w[threadIdx.x] = p.topk_w[at];
+    // a choice without a row gets weight zero and the token's own input to read: no branch in the loop below
+    choices = (p.top + 3) & ~3;
+    if (static_cast<int>(threadIdx.x) < choices) {
+      const T* self = static_cast<const T*>(p.token_in) + row * p.width;
+      const T* src = self;
+      float w = 0.f;
+      if (static_cast<int>(threadIdx.x) < p.top) {
+        const int64_t at = row * p.top + threadIdx.x;
+        const int pos = p.sorted_pos[at];
+        if (pos >= 0) src = static_cast<const T*>(p.expert_rows) + static_cast<int64_t>(pos) * p.width;
+        if (pos >= 0 || (p.identity_from > 0 && p.ids[at] >= p.identity_from)) w = p.topk_w[at];
+      }
+      s_src[threadIdx.x] = src;
+      s_w[threadIdx.x] = w;
     }
     __syncthreads();
   }
   const float* x = p.x + row * p.width;
   const T* y = p.y == nullptr ? nullptr : static_cast<const T*>(p.y) + row * p.width;
-  float z[kRowVecs][V];
+  constexpr int kIts = kRowElems / V;
+  float z[kIts][V];
   float ss = 0.f;
 #pragma unroll
-  for (int it = 0; it < kRowVecs; ++it) {
+  for (int it = 0; it < kIts; ++it) {
     const int v = threadIdx.x + it * blockDim.x;
     if (v < vecs) {
       const int c = v * V;
@@ -91,15 +105,16 @@ __global__ void __launch_bounds__(1024) post_norm_kernel(const PostNormArgs p) {
       for (int i = 0; i < V; ++i) acc[i] = 0.f;
       if (y != nullptr) load_vec<T, V>(y + c, acc);
       if constexpr (MOE) {
-        for (int j = 0; j < p.top; ++j) {
-          const int pos = s_pos[j];
-          if (pos == -1) continue;
-          const T* src = pos >= 0 ? static_cast<const T*>(p.expert_rows) + static_cast<int64_t>(pos) * p.width
-                                  : static_cast<const T*>(p.token_in) + row * p.width;
-          load_vec<T, V>(src + c, t);
-          const float w = s_w[j];
+        for (int j = 0; j < choices; j += 4) {
+          float r[4][V];
 #pragma unroll
-          for (int i = 0; i < V; ++i) acc[i] = fmaf(w, t[i], acc[i]);
+          for (int k = 0; k < 4; ++k) load_vec<T, V>(s_src[j + k] + c, r[k]);
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            const float w = s_w[j + k];
+#pragma unroll
+            for (int i = 0; i < V; ++i) acc[i] = fmaf(w, r[k][i], acc[i]);
+          }
         }
       }
       if (p.ls != nullptr) {
@@ -117,7 +132,7 @@ __global__ void __launch_bounds__(1024) post_norm_kernel(const PostNormArgs p) {
   }
   const float rstd = 1.f / sqrtf(block_sum2(ss, 0.f).x / static_cast<float>(p.width) + p.eps);
 #pragma unroll
-  for (int it = 0; it < kRowVecs; ++it) {
+  for (int it = 0; it < kIts; ++it) {
     const int v = threadIdx.x + it * blockDim.x;
     if (v < vecs) {
       const int c = v * V;
@@ -131,6 +146,13 @@ __global__ void __launch_bounds__(1024) post_norm_kernel(const PostNormArgs p) {
   }
 }
 
+// logistic function of a factor of a result that is rounded to T: the fast exponential and division for 16-bit results
+template <typename T>
+__device__ __forceinline__ float sigmoid_for(float v) {
+  if constexpr (sizeof(T) == 2) return __fdividef(1.f, 1.f + __expf(-v));
+  return 1.f / (1.f + expf(-v));
+}
+
 // out = x * rsqrt(mean(x^2) + eps) * w * sigmoid(gate), the mean over the whole row
 template <typename T, int V>
 __global__ void __launch_bounds__(1024) rmsnorm_sigmoid_gate_kernel(const T* __restrict__ x, const T* __restrict__ gate, int64_t gate_ld,
@@ -140,9 +162,10 @@ __global__ void __launch_bounds__(1024) rmsnorm_sigmoid_gate_kernel(const T* __r
   const int64_t row = blockIdx.x;
   const int vecs = width / V;
   const T* xr = x + row * width;
-  float z[kRowVecs][V], ss = 0.f;
+  constexpr int kIts = kRowElems / V;
+  float z[kIts][V], ss = 0.f;
 #pragma unroll
-  for (int it = 0; it < kRowVecs; ++it) {
+  for (int it = 0; it < kIts; ++it) {
     const int v = threadIdx.x + it * blockDim.x;
     if (v < vecs) {
       load_vec<T, V>(xr + v * V, z[it]);
@@ -152,14 +175,14 @@ __global__ void __launch_bounds__(1024) rmsnorm_sigmoid_gate_kernel(const T* __r
   }
   const float rstd = 1.f / sqrtf(block_sum2(ss, 0.f).x / static_cast<float>(width) + eps);
 #pragma unroll
-  for (int it = 0; it < kRowVecs; ++it) {
+  for (int it = 0; it < kIts; ++it) {
     const int v = threadIdx.x + it * blockDim.x;
     if (v < vecs) {
       float g[V], wv[V];
       load_vec<T, V>(gate + row * gate_ld + v * V, g);
       load_vec<float, V>(w + v * V, wv);
 #pragma unroll
-      for (int i = 0; i < V; ++i) z[it][i] *= rstd * wv[i] / (1.f + expf(-g[i]));
+      for (int i = 0; i < V; ++i) z[it][i] *= rstd * wv[i] * sigmoid_for<T>(g[i]);
       store_vec<T, V>(out + row * out_ld + v * V, z[it]);
     }
   }
@@ -173,7 +196,7 @@ __global__ void __launch_bounds__(1024) rmsnorm_sigmoid_gate_kernel(const T* __r
 // own rounding, and the reduced argument keeps sincosf on its short path.  U: features per access (8, 2 or 1).
 // ---------------------------------------------------------------------------------------------
 template <typename T, int U>
-__global__ void __launch_bounds__(256) rownorm_rope_kv_kernel(const RowNormRopeArgs p) {
+__global__ void __launch_bounds__(512) rownorm_rope_kv_kernel(const RowNormRopeArgs p) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ float2 s_rot[];       // [rot_dims / 2] cosine, sine
@@ -257,15 +280,20 @@ __global__ void __launch_bounds__(256) rownorm_rope_kv_kernel(const RowNormRopeA
   }
 }
 
-// out = cap * tanh(x / cap) in fp32
-template <typename T>
-__global__ void soft_cap_kernel(const T* __restrict__ x, int64_t x_ld, float* __restrict__ out, int64_t total, int width, float cap) {
+// out = cap * tanh(x / cap) in fp32; a CTA walks V neighbouring features at a time of one row
+template <typename T, int V>
+__global__ void soft_cap_kernel(const T* __restrict__ x, int64_t x_ld, float* __restrict__ out, int width, float cap) {
   pdl_launch_dependents();
   pdl_wait();
   const float inv = 1.f / cap;
-  for (int64_t i = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x; i < total; i += static_cast<int64_t>(gridDim.x) * blockDim.x) {
-    const int64_t r = i / width;
-    out[i] = cap * tanhf(to_f32(x[r * x_ld + (i - r * width)]) * inv);
+  const T* row = x + blockIdx.y * x_ld;
+  float* orow = out + static_cast<int64_t>(blockIdx.y) * width;
+  for (int c = (blockIdx.x * blockDim.x + threadIdx.x) * V; c < width; c += gridDim.x * blockDim.x * V) {
+    float f[V];
+    load_vec<T, V>(row + c, f);
+#pragma unroll
+    for (int i = 0; i < V; ++i) f[i] = cap * tanhf(f[i] * inv);
+    store_vec<float, V>(orow + c, f);
   }
 }
 
@@ -290,7 +318,7 @@ inline bool aligned(const void* p, uintptr_t n) { return (reinterpret_cast<uintp
 
 template <typename T, int V>
 int launch_post_norm_v(const PostNormArgs& p, cudaStream_t s) {
-  const int threads = row_threads(p.width / V);
+  const int threads = row_threads(p.width / V, V);
   if (threads == 0) return -1;
   if (p.expert_rows != nullptr)
     launch_pdl(post_norm_kernel<T, V, true>, dim3(p.rows), dim3(threads), 0, s, p);
@@ -303,7 +331,7 @@ int launch_post_norm_v(const PostNormArgs& p, cudaStream_t s) {
 template <typename T, int V>
 int launch_gate_v(const void* x, const void* gate, int64_t gate_ld, const float* w, void* out, int64_t out_ld, int rows, int width,
                   float eps, cudaStream_t s) {
-  const int threads = row_threads(width / V);
+  const int threads = row_threads(width / V, V);
   if (threads == 0) return -1;
   launch_pdl(rmsnorm_sigmoid_gate_kernel<T, V>, dim3(rows), dim3(threads), 0, s, static_cast<const T*>(x), static_cast<const T*>(gate),
              gate_ld, w, static_cast<T*>(out), out_ld, width, eps);
@@ -317,8 +345,11 @@ int launch_rownorm_rope_t(const RowNormRopeArgs& p, cudaStream_t s) {
                          reinterpret_cast<uintptr_t>(p.v_cache) | reinterpret_cast<uintptr_t>(p.q_w) | reinterpret_cast<uintptr_t>(p.k_w);
   const int64_t sizes = p.dim | p.vdim | p.q_width | p.row_ld | p.k_tok_stride | p.k_head_stride | p.v_tok_stride | p.v_head_stride;
   const size_t smem = static_cast<size_t>(p.rot_dims / 2) * sizeof(float2) + 8;
+  // decode batches: a thread per access; long runs: small CTAs, many of them
+  const int units = (p.heads + p.kv_heads) * p.dim / 8;
+  const int threads = p.tokens >= 1024 ? 128 : std::min(512, std::max(64, (units + 31) / 32 * 32));
   auto go = [&](auto kernel) {
-    launch_pdl(kernel, dim3(p.tokens), dim3(256), smem, s, p);
+    launch_pdl(kernel, dim3(p.tokens), dim3(threads), smem, s, p);
     note_launch();
     return cudaGetLastError() == cudaSuccess ? 0 : -4;
   };
@@ -335,9 +366,13 @@ int launch_post_norm(const PostNormArgs& p, cudaStream_t s) {
   const uintptr_t ptrs = reinterpret_cast<uintptr_t>(p.x) | reinterpret_cast<uintptr_t>(p.x_out) | reinterpret_cast<uintptr_t>(p.y) |
                          reinterpret_cast<uintptr_t>(p.ls) | reinterpret_cast<uintptr_t>(p.w) | reinterpret_cast<uintptr_t>(p.h) |
                          reinterpret_cast<uintptr_t>(p.expert_rows) | reinterpret_cast<uintptr_t>(p.token_in);
-  const bool vec = p.width % 4 == 0 && ptrs % 16 == 0;
+  const bool vec = p.width % 4 == 0 && ptrs % 16 == 0, wide = p.width % 8 == 0 && ptrs % 32 == 0 && p.dt != kF32;
   int rc = 0;
-  MB200_DISPATCH_FLOAT(p.dt, rc = vec ? launch_post_norm_v<T, 4>(p, s) : launch_post_norm_v<T, 1>(p, s));
+  if (wide) {
+    MB200_DISPATCH_HALF(p.dt, rc = (launch_post_norm_v<T, 8>(p, s)));
+  } else {
+    MB200_DISPATCH_FLOAT(p.dt, rc = vec ? launch_post_norm_v<T, 4>(p, s) : launch_post_norm_v<T, 1>(p, s));
+  }
   return rc;
 }
 
@@ -347,6 +382,11 @@ int launch_rmsnorm_sigmoid_gate(const void* x, const void* gate, int64_t gate_ld
   const bool vec = width % 4 == 0 && gate_ld % 4 == 0 && out_ld % 4 == 0 && aligned(x, 16) && aligned(gate, dt == kF32 ? 16 : 8) &&
                    aligned(w, 16) && aligned(out, dt == kF32 ? 16 : 8);
   int rc = 0;
+  if (width % 8 == 0 && gate_ld % 8 == 0 && out_ld % 8 == 0 && aligned(x, 16) && aligned(gate, 16) && aligned(w, 32) && aligned(out, 16) &&
+      dt != kF32) {
+    MB200_DISPATCH_HALF(dt, rc = (launch_gate_v<T, 8>(x, gate, gate_ld, w, out, out_ld, rows, width, eps, s)));
+    return rc;
+  }
   MB200_DISPATCH_FLOAT(dt, rc = vec ? (launch_gate_v<T, 4>(x, gate, gate_ld, w, out, out_ld, rows, width, eps, s))
                                     : (launch_gate_v<T, 1>(x, gate, gate_ld, w, out, out_ld, rows, width, eps, s)));
   return rc;
@@ -361,11 +401,20 @@ int launch_rownorm_rope_kv(const RowNormRopeArgs& p, cudaStream_t s) {
 }
 
 void launch_soft_cap(const void* x, int64_t x_ld, float* out, int rows, int width, float cap, DType dt, cudaStream_t s) {
-  const int64_t total = static_cast<int64_t>(rows) * width;
-  if (total <= 0) return;
-  const int grid = static_cast<int>(std::min<int64_t>((total + 255) / 256, 148 * 16));
-  MB200_DISPATCH_FLOAT(dt, (launch_pdl(soft_cap_kernel<T>, dim3(grid), dim3(256), 0, s, static_cast<const T*>(x), x_ld, out, total, width, cap)));
-  note_launch();
+  if (rows <= 0 || width <= 0) return;
+  const bool vec = width % 4 == 0 && x_ld % 4 == 0 && aligned(x, 16) && aligned(out, 16);
+  const int units = vec ? width / 4 : width;
+  for (int r = 0; r < rows; r += 32768) {          // rows are a grid dimension
+    const int m = std::min(32768, rows - r);
+    const dim3 grid(static_cast<unsigned>(std::min((units + 255) / 256, std::max(1, 148 * 8 / m + 1))), m);
+    MB200_DISPATCH_FLOAT(dt, {
+      const T* src = static_cast<const T*>(x) + r * x_ld;
+      float* dst = out + static_cast<int64_t>(r) * width;
+      if (vec) launch_pdl(soft_cap_kernel<T, 4>, grid, dim3(256), 0, s, src, x_ld, dst, width, cap);
+      else launch_pdl(soft_cap_kernel<T, 1>, grid, dim3(256), 0, s, src, x_ld, dst, width, cap);
+    });
+    note_launch();
+  }
 }
 
 void launch_relu_squared(void* x, int64_t n, DType dt, cudaStream_t s) {

@@ -28,7 +28,7 @@ def lightning_kernels(t: Table, batch: int, length: int, heads: int, dim: int) -
     decay = torch.linspace(0.8, 0.999, heads, device="cuda")
     t.add(f"lightning attention {tag}", f"delta rule {tag}",
           lambda i: ops.lightning_attention(*(xs[i][:, j * heads * dim:(j + 1) * heads * dim].unflatten(1, (heads, dim)) for j in range(3)),
-                                            decay, states[i], req, lens, has, start), n, nbytes, 4.0 * T * heads * dim * dim)
+                                            decay, states[i], req, lens, has, start, length), n, nbytes, 4.0 * T * heads * dim * dim)
     rule_kernels(t, batch, length, heads, dim)
 
 

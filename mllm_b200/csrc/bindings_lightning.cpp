@@ -46,12 +46,20 @@ void lightning_recurrent(const Tensor& q, const Tensor& k, const Tensor& v, cons
   TORCH_CHECK(rc == 0, "lightning_recurrent: unsupported head size (code ", rc, ")");
 }
 
-// Returns 1 (nothing launched) when the sizes are not the chunk kernel's.
+// max_len: the longest run of new tokens (0: not known).  Returns 1 (nothing launched) when the sizes are not the chunk
+// kernel's.
 int64_t lightning_chunk(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& decay, Tensor& state, const Tensor& slots,
-                        const Tensor& lens, const Tensor& has, const Tensor& q_start, Tensor& out) {
-  const mb200::LightningArgs a = lightning_args(q, k, v, decay, state, slots, lens, has, q_start, out);
+                        const Tensor& lens, const Tensor& has, const Tensor& q_start, Tensor& out, int64_t max_len) {
+  mb200::LightningArgs a = lightning_args(q, k, v, decay, state, slots, lens, has, q_start, out);
   if (!mb200::lightning_chunk_covers(a)) return 1;
   c10::cuda::CUDAGuard g(q.device());
+  a.segments = mb200::lightning_segments(a.batch, a.heads, a.dv, static_cast<int>(max_len), device_state(q.get_device()).num_sms);
+  Tensor ws;
+  if (a.segments > 1) {
+    a.seg_tokens = static_cast<int>((max_len + 64 * a.segments - 1) / (64 * a.segments) * 64);
+    ws = torch::empty({a.batch, a.segments, a.heads, a.dk, a.dv}, state.options());
+    a.ws = ws.data_ptr<float>();
+  }
   const int rc = mb200::launch_lightning_chunk(a, stream_of(q));
   TORCH_CHECK(rc == 0, "lightning_chunk: launch failed (code ", rc, ")");
   return 0;

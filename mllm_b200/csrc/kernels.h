@@ -323,8 +323,13 @@ struct LightningArgs {
   const int* q_start;
   int64_t q_ld, k_ld, v_ld;
   int batch, heads, dk, dv;
+  // chunk kernel: > 1 cuts every request's tokens into this many segments of seg_tokens (a multiple of 64; segments *
+  // seg_tokens >= the longest request) that run side by side; ws holds [batch][segments][heads][dk][dv] fp32
+  int segments, seg_tokens;
+  float* ws;
   DType dt;
 };
+int lightning_segments(int batch, int heads, int dv, int max_len, int num_sms);
 // token by token; dk up to 512, any dv
 int launch_lightning_recurrent(const LightningArgs& args, cudaStream_t s);
 // 64 tokens at a time on the tensor cores; 16-bit types, dk up to 128

@@ -11,6 +11,8 @@
 //   as warp-level tensor-core products.  Q, K and V are bf16 and enter as they are; fp32 operands are carried as sums of
 //   bf16 terms: two (16 bits) where the result is an output that is rounded to bf16 next, three (24 bits, all of fp32)
 //   where it stays in the state.  Nothing of the state passes through 16 bits.
+#include <algorithm>
+
 #include "common.cuh"
 #include "kernels.h"
 #include "mma.cuh"
@@ -128,9 +130,14 @@ __global__ void __launch_bounds__(256) lightning_recurrent_kernel(const Lightnin
 }
 
 // ---------------------------------------------------------------------------------------------
-// 64 tokens at a time: grid (ceil(dv / 64), heads, batch), 256 threads.  The columns of S never mix, so a CTA owns one
-// (request, head) and 64 of them, with the state in the accumulators of its 8 warps for the whole sequence.  DK: dk
-// rounded up to 32, 64 or 128 (missing features are zero).
+// 64 tokens at a time: grid (ceil(dv / 64) * segments, heads, batch), 256 threads.  The columns of S never mix, so a CTA
+// owns one (request, head) and 64 of them, with the state in the accumulators of its 8 warps.  DK: dk rounded up to 32,
+// 64 or 128 (missing features are zero).
+//
+// kWhole: one CTA walks all new tokens.  When that leaves SMs idle the tokens are cut into segments, and two launches
+// share the work through `ws` [batch][segments][heads][dk][dv]: kSums leaves the state before the request in slot 0 and
+// the sum K^T diag(decay^..) V of segment s in slot s + 1; kOutputs starts every segment from
+// (((slot 0) D + slot 1) D + ...), D = decay^(tokens of a segment), and the last segment writes the new state.
 // ---------------------------------------------------------------------------------------------
 using bf16 = __nv_bfloat16;
 constexpr int kLcTok = 64, kLcV = 64, kLcLdV = kLcV + 8, kLcThreads = 256;
@@ -155,9 +162,10 @@ __device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t&
   lo = pack_bf16x2(ra, rb);
 }
 
-template <int DK>
+enum LightningMode { kWhole, kSums, kOutputs };
+
+template <int DK, int MODE>
 __global__ void __launch_bounds__(kLcThreads, 2) lightning_chunk_kernel(const LightningArgs p) {
-  pdl_launch_dependents();
   pdl_wait();
   using C = LightningCfg<DK>;
   constexpr int kLd = C::kLd, kMT = DK / 16, kCG = 8 / kMT, kNT = 8 / kCG;   // row tiles of S, column groups, n tiles per warp
@@ -169,9 +177,11 @@ __global__ void __launch_bounds__(kLcThreads, 2) lightning_chunk_kernel(const Li
   bf16* sS = sW + 3 * kLcTok * kLcLdV;              // [2][DK][72] terms of the state before the chunk
   float* sPow = reinterpret_cast<float*>(sS + 2 * DK * kLcLdV);   // decay^0 .. decay^64
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int vb = blockIdx.x * kLcV, h = blockIdx.y, b = blockIdx.z;
+  const int seg = MODE == kWhole ? 0 : static_cast<int>(blockIdx.x) % p.segments;
+  const int vb = (MODE == kWhole ? static_cast<int>(blockIdx.x) : static_cast<int>(blockIdx.x) / p.segments) * kLcV, h = blockIdx.y, b = blockIdx.z;
   const int n = p.lens[b];
-  if (n <= 0) return;
+  const int t_begin = MODE == kWhole ? 0 : seg * p.seg_tokens, t_end = MODE == kWhole ? n : min(n, t_begin + p.seg_tokens);
+  if (n <= 0 || t_begin >= n) return;
   const int dk = p.dk, dv = p.dv, cols = min(kLcV, dv - vb);
   const int64_t row0 = p.q_start[b];
   const bf16* q = static_cast<const bf16*>(p.q) + row0 * p.q_ld + static_cast<int64_t>(h) * dk;
@@ -185,18 +195,34 @@ __global__ void __launch_bounds__(kLcThreads, 2) lightning_chunk_kernel(const Li
   // this warp's part of S: row tile mt, n tiles n0 .. n0 + kNT - 1
   const int mt = warp % kMT, n0 = (warp / kMT) * kNT;
   const int g = lane >> 2, c2 = (lane & 3) * 2;
+  const int64_t slot_elems = static_cast<int64_t>(p.heads) * dk * dv;
+  float* ws = MODE == kWhole ? nullptr : p.ws + (static_cast<int64_t>(b) * p.segments * p.heads + h) * dk * dv + vb;
   float st[kNT][4];
+  auto for_state = [&](auto&& f) {       // f(element of st, offset in a [dk][dv] matrix) for the elements that exist
 #pragma unroll
-  for (int nt = 0; nt < kNT; ++nt)
+    for (int nt = 0; nt < kNT; ++nt)
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int i = mt * 16 + g + (e >> 1) * 8, c = (n0 + nt) * 8 + c2 + (e & 1);
-      st[nt][e] = resume && i < dk && c < cols ? S[static_cast<int64_t>(i) * dv + c] : 0.f;
-    }
+      for (int e = 0; e < 4; ++e) {
+        const int i = mt * 16 + g + (e >> 1) * 8, c = (n0 + nt) * 8 + c2 + (e & 1);
+        if (i < dk && c < cols) f(st[nt][e], static_cast<int64_t>(i) * dv + c);
+      }
+  };
+#pragma unroll
+  for (int nt = 0; nt < kNT; ++nt) st[nt][0] = st[nt][1] = st[nt][2] = st[nt][3] = 0.f;
+  if constexpr (MODE == kWhole) {
+    if (resume) for_state([&](float& x, int64_t at) { x = S[at]; });
+  } else if constexpr (MODE == kSums) {
+    if (seg == 0) for_state([&](float&, int64_t at) { ws[at] = resume ? S[at] : 0.f; });
+    if (t_end == n) return;              // no later segment asks for this one's sum
+  } else {
+    const float full = powf(p.decay[h], static_cast<float>(p.seg_tokens));
+    for_state([&](float& x, int64_t at) { x = ws[at]; });
+    for (int k2 = 1; k2 <= seg; ++k2) for_state([&](float& x, int64_t at) { x = fmaf(x, full, ws[k2 * slot_elems + at]); });
+  }
   __syncthreads();
 
-  for (int c0 = 0; c0 < n; c0 += kLcTok) {
-    const int nv = min(kLcTok, n - c0);
+  for (int c0 = t_begin; c0 < t_end; c0 += kLcTok) {
+    const int nv = min(kLcTok, t_end - c0);
     // ---- rows of the chunk: activated, missing rows and features zero; the values also scaled, in three terms ----
     auto load8 = [&](const bf16* src, bool valid, float (&f)[8]) {
       uint4 raw = make_uint4(0u, 0u, 0u, 0u);
@@ -217,8 +243,10 @@ __global__ void __launch_bounds__(kLcThreads, 2) lightning_chunk_kernel(const Li
       const int i = tid + it * kLcThreads, r = i / (DK / 8), d = (i % (DK / 8)) * 8;
       const bool valid = r < nv && d < dk;
       float f[8];
-      load8(q + static_cast<int64_t>(c0 + r) * p.q_ld + d, valid, f);
-      *reinterpret_cast<uint4*>(sQ + r * kLd + d) = pack8(f);
+      if constexpr (MODE != kSums) {
+        load8(q + static_cast<int64_t>(c0 + r) * p.q_ld + d, valid, f);
+        *reinterpret_cast<uint4*>(sQ + r * kLd + d) = pack8(f);
+      }
       load8(k + static_cast<int64_t>(c0 + r) * p.k_ld + d, valid, f);
       *reinterpret_cast<uint4*>(sK + r * kLd + d) = pack8(f);
     }
@@ -240,7 +268,7 @@ __global__ void __launch_bounds__(kLcThreads, 2) lightning_chunk_kernel(const Li
     }
     // ---- the state before the chunk as an operand ----
 #pragma unroll
-    for (int nt = 0; nt < kNT; ++nt)
+    for (int nt = 0; nt < (MODE == kSums ? 0 : kNT); ++nt)
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
         uint32_t hi, lo;
@@ -252,7 +280,7 @@ __global__ void __launch_bounds__(kLcThreads, 2) lightning_chunk_kernel(const Li
     __syncthreads();
 
     // ---- outputs: 16 rows and 32 columns per warp ----
-    {
+    if constexpr (MODE != kSums) {
       const int rt = warp & 3, oc = (warp >> 2) * 32;
       if (rt * 16 < nv) {
         float o[4][4];
@@ -351,13 +379,12 @@ __global__ void __launch_bounds__(kLcThreads, 2) lightning_chunk_kernel(const Li
     }
     __syncthreads();      // every operand of this chunk has been read
   }
-#pragma unroll
-  for (int nt = 0; nt < kNT; ++nt)
-#pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int i = mt * 16 + g + (e >> 1) * 8, c = (n0 + nt) * 8 + c2 + (e & 1);
-      if (i < dk && c < cols) S[static_cast<int64_t>(i) * dv + c] = st[nt][e];
-    }
+  if constexpr (MODE == kSums) {
+    float* mine = ws + (seg + 1) * slot_elems;
+    for_state([&](float& x, int64_t at) { mine[at] = x; });
+  } else if (t_end == n) {
+    for_state([&](float& x, int64_t at) { S[at] = x; });
+  }
 }
 
 template <typename T>
@@ -373,13 +400,20 @@ int launch_recurrent_t(const LightningArgs& p, cudaStream_t s) {
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
-template <int DK>
-int launch_chunk_t(const LightningArgs& p, cudaStream_t s) {
-  if (ensure_dynamic_smem(reinterpret_cast<const void*>(lightning_chunk_kernel<DK>), LightningCfg<DK>::kSmem) != cudaSuccess) return -3;
-  const cudaError_t err = launch_pdl(lightning_chunk_kernel<DK>, dim3((p.dv + kLcV - 1) / kLcV, p.heads, p.batch), dim3(kLcThreads),
-                                     LightningCfg<DK>::kSmem, s, p);
+template <int DK, int MODE>
+int launch_chunk_mode(const LightningArgs& p, cudaStream_t s) {
+  auto kern = lightning_chunk_kernel<DK, MODE>;
+  if (ensure_dynamic_smem(reinterpret_cast<const void*>(kern), LightningCfg<DK>::kSmem) != cudaSuccess) return -3;
+  const int blocks = (p.dv + kLcV - 1) / kLcV * (MODE == kWhole ? 1 : p.segments);
+  const cudaError_t err = launch_pdl(kern, dim3(blocks, p.heads, p.batch), dim3(kLcThreads), LightningCfg<DK>::kSmem, s, p);
   note_launch();
   return err == cudaSuccess ? 0 : -4;
+}
+template <int DK>
+int launch_chunk_t(const LightningArgs& p, cudaStream_t s) {
+  if (p.segments <= 1) return launch_chunk_mode<DK, kWhole>(p, s);
+  const int rc = launch_chunk_mode<DK, kSums>(p, s);
+  return rc != 0 ? rc : launch_chunk_mode<DK, kOutputs>(p, s);
 }
 
 }  // namespace
@@ -397,9 +431,16 @@ bool lightning_chunk_covers(const LightningArgs& p) {
          ((reinterpret_cast<uintptr_t>(p.q) | reinterpret_cast<uintptr_t>(p.k) | reinterpret_cast<uintptr_t>(p.v)) & 15) == 0;
 }
 
+int lightning_segments(int batch, int heads, int dv, int max_len, int num_sms) {
+  // two CTAs are resident per SM; a segment has at least 256 tokens, and a start state is read from at most 16 slots
+  const int ctas = std::max(1, (dv + kLcV - 1) / kLcV * heads * batch);
+  return std::max(1, std::min({2 * num_sms / ctas, 16, max_len / 256}));
+}
+
 int launch_lightning_chunk(const LightningArgs& p, cudaStream_t s) {
   if (p.batch <= 0) return 0;
   if (!lightning_chunk_covers(p)) return -1;
+  if (p.segments > 1 && (p.ws == nullptr || p.seg_tokens <= 0 || p.seg_tokens % kLcTok != 0)) return -1;
   return p.dk <= 32 ? launch_chunk_t<32>(p, s) : p.dk <= 64 ? launch_chunk_t<64>(p, s) : launch_chunk_t<128>(p, s);
 }
 

@@ -31,7 +31,7 @@ constexpr int kMaxExperts = 256;
 // --------------------------------------------------------------------------------------------
 // router: one warp per token
 // --------------------------------------------------------------------------------------------
-template <typename T>
+template <typename T, int NV>   // NV: logits per lane
 __global__ void moe_router_topk_kernel(const T* __restrict__ logits, int64_t stride, const float* __restrict__ correction,
                                        float* __restrict__ w_out, int* __restrict__ id_out, int tokens, int experts, int top_k,
                                        int renorm, float renorm_eps) {
@@ -40,10 +40,10 @@ __global__ void moe_router_topk_kernel(const T* __restrict__ logits, int64_t str
   const int lane = threadIdx.x & 31;
   if (t >= tokens) return;
   const T* row = logits + static_cast<int64_t>(t) * stride;
-  float v[kMaxExperts / 32];
+  float v[NV];
   float mx = -INFINITY;
 #pragma unroll
-  for (int i = 0; i < kMaxExperts / 32; ++i) {
+  for (int i = 0; i < NV; ++i) {
     const int e = lane + 32 * i;
     v[i] = e < experts ? to_f32(row[e]) : -INFINITY;
     mx = fmaxf(mx, v[i]);
@@ -51,16 +51,16 @@ __global__ void moe_router_topk_kernel(const T* __restrict__ logits, int64_t str
   mx = warp_max(mx);
   float sum = 0.f;
 #pragma unroll
-  for (int i = 0; i < kMaxExperts / 32; ++i) {
+  for (int i = 0; i < NV; ++i) {
     v[i] = (lane + 32 * i) < experts ? expf(v[i] - mx) : 0.f;
     sum += v[i];
   }
   sum = warp_sum(sum);
   const float inv = 1.f / sum;
   // the key that is compared: the score, plus the expert's correction; -inf where there is no expert or it is taken
-  float key[kMaxExperts / 32];
+  float key[NV];
 #pragma unroll
-  for (int i = 0; i < kMaxExperts / 32; ++i) {
+  for (int i = 0; i < NV; ++i) {
     const int e = lane + 32 * i;
     v[i] *= inv;
     key[i] = e < experts ? v[i] + (correction != nullptr ? correction[e] : 0.f) : -INFINITY;
@@ -69,32 +69,34 @@ __global__ void moe_router_topk_kernel(const T* __restrict__ logits, int64_t str
   int chosen_e = 0;
   float ksum = 0.f;
   for (int j = 0; j < top_k; ++j) {
-    float best = -INFINITY, score = 0.f;
+    float best = -INFINITY;
     int bi = 0x7fffffff;
 #pragma unroll
-    for (int i = 0; i < kMaxExperts / 32; ++i) {
+    for (int i = 0; i < NV; ++i) {
       if (key[i] > best) {  // ascending i: the lowest index wins ties inside a lane
         best = key[i];
-        score = v[i];
         bi = lane + 32 * i;
       }
     }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
       const float ov = __shfl_xor_sync(0xffffffffu, best, o);
-      const float os = __shfl_xor_sync(0xffffffffu, score, o);
       const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
       if (ov > best || (ov == best && oi < bi)) {
         best = ov;
-        score = os;
         bi = oi;
       }
     }
+    float score = 0.f;
     if ((bi & 31) == lane) {
 #pragma unroll
-      for (int i = 0; i < kMaxExperts / 32; ++i)
-        if (i == (bi >> 5)) key[i] = -INFINITY;
+      for (int i = 0; i < NV; ++i)
+        if (i == (bi >> 5)) {
+          key[i] = -INFINITY;
+          score = v[i];
+        }
     }
+    score = __shfl_sync(0xffffffffu, score, bi & 31);
     ksum += score;
     if (lane == j) {
       chosen_w = score;
@@ -143,8 +145,10 @@ __global__ void __launch_bounds__(kRlWarps * 32) moe_router_rows_kernel(const T*
   }
 }
 
-// prefill: 64 tokens x all experts (NT tiles of 8) per CTA, 64 features at a time through a three-stage ring
-constexpr int kRmTok = 64, kRmK = 64, kRmLd = kRmK + 8, kRmStages = 3;
+// prefill: 32 tokens x all experts (NT tiles of 8) per CTA, 128 features at a time through a ring; warps 0 and 1 take
+// the two row tiles of the lower 64 features of a step, warps 2 and 3 those of the upper, and the halves meet at the end
+constexpr int kRmTok = 32, kRmK = 128, kRmLd = kRmK + 8;
+constexpr int rm_stages(int nt) { return nt <= 16 ? 3 : 2; }
 
 template <typename T, int NT>
 __global__ void __launch_bounds__(128) moe_router_mma_kernel(const T* __restrict__ x, int64_t x_ld, const T* __restrict__ w,
@@ -152,6 +156,7 @@ __global__ void __launch_bounds__(128) moe_router_mma_kernel(const T* __restrict
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) uint8_t rm_smem[];
+  constexpr int kRmStages = rm_stages(NT);
   constexpr int kRows = kRmTok + NT * 8;                 // token rows, then expert rows
   T* ring = reinterpret_cast<T*>(rm_smem);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -184,9 +189,10 @@ __global__ void __launch_bounds__(128) moe_router_mma_kernel(const T* __restrict
     const T* sx = ring + (step % kRmStages) * kRows * kRmLd;
     const T* sw = sx + kRmTok * kRmLd;
 #pragma unroll
-    for (int kk = 0; kk < kRmK; kk += 16) {
+    for (int k16 = 0; k16 < kRmK / 2; k16 += 16) {
+      const int kk = (warp >> 1) * (kRmK / 2) + k16;
       uint32_t a[4];
-      ldsm4(a, smem_u32(sx + (warp * 16 + (lane & 15)) * kRmLd + kk + (lane >> 4) * 8));
+      ldsm4(a, smem_u32(sx + ((warp & 1) * 16 + (lane & 15)) * kRmLd + kk + (lane >> 4) * 8));
 #pragma unroll
       for (int n = 0; n < NT; n += 2) {
         uint32_t b[4];      // two tiles of 8 experts: (lower, upper 8 features) of the first, then of the second
@@ -196,15 +202,26 @@ __global__ void __launch_bounds__(128) moe_router_mma_kernel(const T* __restrict
       }
     }
   }
+  cp_wait<0>();
+  __syncthreads();                       // the ring is free: it takes the partial sums of the upper features
+  float* part = reinterpret_cast<float*>(rm_smem) + (warp & 1) * 32 * NT * 4;
+  if (warp >= 2) {
+#pragma unroll
+    for (int n = 0; n < NT; ++n) *reinterpret_cast<float4*>(part + (n * 32 + lane) * 4) = make_float4(acc[n][0], acc[n][1], acc[n][2], acc[n][3]);
+  }
+  __syncthreads();
+  if (warp >= 2) return;
 #pragma unroll
   for (int n = 0; n < NT; ++n) {
+    const float4 o = *reinterpret_cast<const float4*>(part + (n * 32 + lane) * 4);
+    const float sum[4] = {acc[n][0] + o.x, acc[n][1] + o.y, acc[n][2] + o.z, acc[n][3] + o.w};
     const int e = n * 8 + (lane & 3) * 2;
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
       const int64_t t = t0 + warp * 16 + (lane >> 2) + half * 8;
       if (t < tokens) {
-        if (e < experts) logits[t * experts + e] = acc[n][half * 2];
-        if (e + 1 < experts) logits[t * experts + e + 1] = acc[n][half * 2 + 1];
+        if (e < experts) logits[t * experts + e] = sum[half * 2];
+        if (e + 1 < experts) logits[t * experts + e + 1] = sum[half * 2 + 1];
       }
     }
   }
@@ -213,7 +230,7 @@ __global__ void __launch_bounds__(128) moe_router_mma_kernel(const T* __restrict
 template <typename T, int NT>
 int launch_router_mma(const void* x, int64_t x_ld, const void* w, float* logits, int tokens, int experts, int hidden, cudaStream_t s) {
   auto kern = moe_router_mma_kernel<T, NT>;
-  const int smem = kRmStages * (kRmTok + NT * 8) * kRmLd * static_cast<int>(sizeof(T));
+  const int smem = rm_stages(NT) * (kRmTok + NT * 8) * kRmLd * static_cast<int>(sizeof(T));
   if (ensure_dynamic_smem(reinterpret_cast<const void*>(kern), smem) != cudaSuccess) return -3;
   const cudaError_t err = launch_pdl(kern, dim3((tokens + kRmTok - 1) / kRmTok), dim3(128), smem, s, static_cast<const T*>(x), x_ld,
                                      static_cast<const T*>(w), logits, tokens, experts, hidden);
@@ -604,8 +621,17 @@ void launch_moe_router_topk(const void* logits, int64_t stride, const float* cor
   if (tokens == 0) return;
   const int warps = 8;
   const dim3 grid((tokens + warps - 1) / warps), block(warps * 32);
-  MB200_DISPATCH_FLOAT(dt, (launch_pdl(moe_router_topk_kernel<T>, grid, block, 0, s, static_cast<const T*>(logits), stride, correction,
-                                       w, ids, tokens, experts, top_k, renorm, renorm_eps)));
+  auto go = [&](auto kernel, auto* typed) {
+    launch_pdl(kernel, grid, block, 0, s, typed, stride, correction, w, ids, tokens, experts, top_k, renorm, renorm_eps);
+  };
+  MB200_DISPATCH_FLOAT(dt, {
+    const T* l = static_cast<const T*>(logits);
+    if (experts <= 32) go(moe_router_topk_kernel<T, 1>, l);
+    else if (experts <= 64) go(moe_router_topk_kernel<T, 2>, l);
+    else if (experts <= 96) go(moe_router_topk_kernel<T, 3>, l);
+    else if (experts <= 128) go(moe_router_topk_kernel<T, 4>, l);
+    else go(moe_router_topk_kernel<T, 8>, l);
+  });
   note_launch();
 }
 

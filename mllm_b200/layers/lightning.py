@@ -54,5 +54,5 @@ class LightningAttention(nn.Module):
         q = row[:, :K].unflatten(1, (self.heads, self.dim))
         k = row[:, K:2 * K].unflatten(1, (self.heads, self.dim))
         v = row[:, 2 * K:2 * K + V].unflatten(1, (self.heads, self.vdim))
-        o = ops.lightning_attention(q, k, v, self.decay, state, m.slots, m.lens, m.has_state, m.q_start)
+        o = ops.lightning_attention(q, k, v, self.decay, state, m.slots, m.lens, m.has_state, m.q_start, m.max_len)
         ops.rmsnorm_sigmoid_gate(o.view(-1, V), row[:, 2 * K + V:2 * K + 2 * V], self.norm.weight, self.eps, out)

@@ -1039,10 +1039,11 @@ def gated_delta_rule(q, k, v, g, beta, state, state_indices, seq_lens, has_state
 # --------------------------------------------------------------------------
 # lightning attention (linear attention with a fixed decay per head)
 # --------------------------------------------------------------------------
-def lightning_attention(q, k, v, decay, state, state_indices, seq_lens, has_state, q_start=None) -> torch.Tensor:
+def lightning_attention(q, k, v, decay, state, state_indices, seq_lens, has_state, q_start=None, max_len: int = 0) -> torch.Tensor:
     """``S <- decay S + k v^T``, ``o = S^T q`` with q, k [T, H, D] and v [T, H, Dv] taken through SiLU first; tokens may be
     rows of wider matrices.  ``state`` fp32 [rows, H, D, Dv] is read where ``has_state`` and always written back;
-    metadata as for :func:`gated_delta_rule`, whose extend-backend choice also holds here."""
+    metadata as for :func:`gated_delta_rule`, whose extend-backend choice also holds here.  ``max_len``: the longest run
+    of new tokens, when the host knows it; long runs of few requests are then cut into segments that run side by side."""
     if not use_kernels(q):
         lens = seq_lens.tolist() if isinstance(seq_lens, torch.Tensor) else seq_lens
         has = has_state.tolist() if isinstance(has_state, torch.Tensor) else has_state
@@ -1055,7 +1056,7 @@ def lightning_attention(q, k, v, decay, state, state_indices, seq_lens, has_stat
     args = (q, k, v, decay, state, state_indices.to(torch.int32), lens, has_state.to(torch.int32), q_start.to(torch.int32), out)
     chunked = _GDN_EXTEND_BACKEND == "cuda_chunkwise" or (
         _GDN_EXTEND_BACKEND != "mllm_kernel" and q.shape[0] >= 32 * max(1, lens.numel()))
-    if not chunked or ext().lightning_chunk(*args) != 0:
+    if not chunked or ext().lightning_chunk(*args, int(max_len)) != 0:
         ext().lightning_recurrent(*args)
     return out
 

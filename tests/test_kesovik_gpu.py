@@ -313,6 +313,32 @@ def test_chunk_state_keeps_32_bits():
     assert ((y.double().cpu() - o).abs() / o).max() < 4.1e-3          # one rounding to bf16
 
 
+@pytest.mark.parametrize("heads,dim,vdim", [(2, 128, 128), (3, 40, 72), (1, 32, 64)])
+def test_long_prompts_cut_into_segments(heads, dim, vdim):
+    """Long runs of few requests run as segments side by side: the same outputs and states as one walk, for requests that
+    span all segments, end inside one or at its border, with and without an earlier state."""
+    from mllm_b200 import ops
+
+    lens, K, V = [1500, 512, 3, 300], heads * dim, heads * vdim
+    decay = torch.tensor([0.9995, 0.97, 0.6][:heads], device=DEV)
+    x = _r(sum(lens), 2 * K + V, seed=3).to(torch.bfloat16).to(DEV)
+    q, k, v = x[:, :K].unflatten(1, (heads, dim)), x[:, K:2 * K].unflatten(1, (heads, dim)), x[:, 2 * K:].unflatten(1, (heads, vdim))
+    first = _r(6, heads, dim, vdim, seed=4).to(DEV)
+    slots, ln, has = _i32([5, 1, 0, 2]), _i32(lens), _i32([1, 0, 1, 1])
+    got, want = [], []
+    for out, longest in ((want, 0), (got, max(lens))):
+        state = first.clone()
+        out.append(ops.lightning_attention(q, k, v, decay, state, slots, ln, has, None, longest).float())
+        out.append(state)
+    for a, b, tol in zip(got, want, (8e-3, 1e-5)):
+        assert (a - b).abs().max() <= tol * b.abs().max()
+    assert torch.equal(got[1][[3, 4]], first[[3, 4]])
+    o, S = oracle.decayed_sums(*(oracle.f64(oracle.silu(oracle.f64(t[2012:2015])).to(torch.bfloat16)) for t in (q, k, v)), decay.cpu(),
+                               oracle.f64(first[0]))
+    _close(got[0][2012:2015], o, 6e-3)
+    _close(got[1][0], S, 1e-3)
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("decay", [1.0, 0.999, 0.5, 0.0])
 def test_lightning_finds_a_far_token(dtype, decay):
@@ -334,7 +360,7 @@ def test_lightning_finds_a_far_token(dtype, decay):
         for p in portions:
             sl = slice(done, done + p)
             outs.append(ops.lightning_attention(q[sl], k[sl], v[sl], torch.tensor([decay], device=DEV), state, _i32([1]), _i32([p]),
-                                                _i32([int(done > 0)]), _i32([0])))
+                                                _i32([int(done > 0)]), _i32([0]), p))
             done += p
         got = torch.cat(outs)[:, 0].float().cpu()
         assert (got[:at].abs() < 1e-6).all()

@@ -194,9 +194,27 @@ def latent(a) -> dict:
             "gbs": a.batch * a.seq * a.rank * 2 / ms / 1e6, "tflops": 4 * a.batch * a.seq * a.hq * a.rank / ms / 1e9}
 
 
+def lightning(a) -> dict:
+    """Lightning attention over `--batch` requests of `--seq` new tokens, `--hq` heads of 128 x 128."""
+    dev, H, D, T = "cuda", a.hq, 128, a.batch * a.seq
+    xs = [torch.randn(T, 3 * H * D, device=dev, dtype=torch.bfloat16) for _ in range(max(1, a.kv_sets))]
+    state = torch.zeros(a.batch, H, D, D, device=dev)
+    req = torch.arange(a.batch, dtype=torch.int32, device=dev)
+    lens, decay = torch.full_like(req, a.seq), torch.linspace(0.8, 0.999, H, device=dev)
+
+    def run():
+        for x in xs:
+            q, k, v = (t.unflatten(1, (H, D)) for t in x.split(H * D, 1))
+            ops.lightning_attention(q, k, v, decay, state, req, lens, torch.ones_like(req), req * a.seq, a.seq)
+
+    ms = _time(run, a.iters) / len(xs)
+    return {"case": "lightning", "batch": a.batch, "seq": a.seq, "heads": H, "ms": ms,
+            "gbs": (T * 4 * H * D * 2 + 2 * a.batch * H * D * D * 4) / ms / 1e6}
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
-    ap.add_argument("case", choices=["attn_decode", "attn_prefill", "gemm", "moe", "w4a16", "gdn", "latent"])
+    ap.add_argument("case", choices=["attn_decode", "attn_prefill", "gemm", "moe", "w4a16", "gdn", "latent", "lightning"])
     ap.add_argument("--gdn-backend", default="auto", choices=["auto", "cuda_chunkwise", "mllm_kernel"],
                     help="gdn: chunk-parallel kernel, token-sequential kernel, or the default choice between them")
     ap.add_argument("--experts", type=int, default=16, help="moe: local experts")
@@ -216,7 +234,7 @@ def main() -> None:
     ap.add_argument("--kv-sets", type=int, default=4, help="attn_decode: KV caches used in turn (working set > L2)")
     a = ap.parse_args()
     out = {"attn_decode": attn_decode, "attn_prefill": attn_prefill, "gemm": gemm, "moe": moe, "w4a16": w4a16, "gdn": gdn,
-           "latent": latent}[a.case](a)
+           "latent": latent, "lightning": lightning}[a.case](a)
     ops.check_status()
     print(json.dumps(out))
 

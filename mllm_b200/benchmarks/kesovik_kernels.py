@@ -32,7 +32,7 @@ def lightning_kernels(t: Table, batch: int, length: int, heads: int, dim: int) -
     rule_kernels(t, batch, length, heads, dim)
 
 
-def window_decode(t: Table, batch: int, length: int, window: int, heads: int, kv: int, dim: int, tag: str) -> None:
+def window_decode(t: Table, batch: int, length: int, window: int, heads: int, kv: int, dim: int, tag: str, like: str) -> None:
     slots = batch * length + 16
     n = _copies(2 * slots * kv * dim * 2)
     pool = [tuple(_rand(kv, slots, dim).transpose(0, 1) for _ in range(2)) for _ in range(n)]
@@ -40,7 +40,7 @@ def window_decode(t: Table, batch: int, length: int, window: int, heads: int, kv
     req = torch.arange(batch, device="cuda", dtype=torch.int32)
     lens, q = torch.full_like(req, length), _rand(batch, heads, dim)
     seen = min(window, length)
-    t.add(f"window attention decode {tag}, window {window}", f"attention_decode {tag}",
+    t.add(f"window attention decode {tag}, window {window}", f"attention_decode {like}",
           lambda i: ops.attention_decode(q, *pool[i], table, req, lens, dim ** -0.5, max_seq_len=length, window=window), n,
           2.0 * batch * seen * kv * dim * 2, 4.0 * batch * heads * seen * dim)
 
@@ -133,10 +133,11 @@ def add_rows(t: Table) -> None:
     for batch, length in ((1, 1), (8, 1), (32, 1), (1, 2048), (8, 2048)):
         lightning_kernels(t, batch, length, 16, 128)
         torch.cuda.empty_cache()
+    # the like kernel reads as many keys: it has no window in the other model
     for batch, length in ((1, 2048), (8, 2048), (32, 1024), (4, 16384)):
-        tag = f"{batch}x{length}"
-        window_decode(t, batch, length, 2048, 16, 4, 128, tag)
-        kv_decode_kernel(t, batch, length, 8, 2, 256, tag)
+        seen = min(2048, length)
+        window_decode(t, batch, length, 2048, 16, 4, 128, f"{batch}x{length}", f"{batch}x{seen}")
+        kv_decode_kernel(t, batch, seen, 8, 2, 256, f"{batch}x{seen}")
         torch.cuda.empty_cache()
     prefill(t, 8, 2048, 16, 4, 128, 2048, "attention_prefill 256-wide 8x2048")
     prefill(t, 8, 2048, 16, 4, 128, 512, "attention_prefill 256-wide 8x2048")

@@ -149,17 +149,26 @@ struct LightningCfg {
   static constexpr int kSmem = kElems * 2 + (kLcTok + 1) * 4;
 };
 
-__device__ __forceinline__ float bf16_part(float x, float& rest) {
-  const float hi = __bfloat162float(__float2bfloat16_rn(x));
-  rest = x - hi;
-  return hi;
+// Two fp32 values as sums of bf16 terms, each pair of terms packed for an operand register.  A leading term is the value
+// with its lower 16 bits cut off (one byte permutation for both), the last one is rounded.
+__device__ __forceinline__ uint32_t cut_term(float& a, float& b) {
+  const uint32_t ua = __float_as_uint(a), ub = __float_as_uint(b);
+  a -= __uint_as_float(ua & 0xffff0000u);
+  b -= __uint_as_float(ub & 0xffff0000u);
+  return __byte_perm(ua, ub, 0x7632);
 }
-// a pair of fp32 values as two or three bf16 terms, each packed for an operand register
 __device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
-  float ra, rb;
-  const float ha = bf16_part(a, ra), hb = bf16_part(b, rb);
-  hi = pack_bf16x2(ha, hb);
-  lo = pack_bf16x2(ra, rb);
+  hi = cut_term(a, b);
+  lo = pack_bf16x2(a, b);
+}
+
+// SiLU of two values with one reciprocal: 1 / x = y / (x y).  exp is bounded so that the product stays finite; below
+// -41 the result is then v * 1e-18 instead of v * exp(v), zero beside any other term.
+__device__ __forceinline__ void silu_pair(float& a, float& b) {
+  const float da = 1.f + fminf(__expf(-a), 1e18f), db = 1.f + fminf(__expf(-b), 1e18f);
+  const float r = __fdividef(1.f, da * db);
+  a *= db * r;
+  b *= da * r;
 }
 
 enum LightningMode { kWhole, kSums, kOutputs };
@@ -230,9 +239,10 @@ __global__ void __launch_bounds__(kLcThreads, 2) lightning_chunk_kernel(const Li
       const uint32_t* u = reinterpret_cast<const uint32_t*>(&raw);
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        const float2 t = unpack_bf16x2(u[i]);
-        f[2 * i] = silu_as<bf16>(t.x);
-        f[2 * i + 1] = silu_as<bf16>(t.y);
+        float2 t = unpack_bf16x2(u[i]);
+        silu_pair(t.x, t.y);
+        f[2 * i] = t.x;
+        f[2 * i + 1] = t.y;
       }
     };
     auto pack8 = [](const float (&f)[8]) {
@@ -253,18 +263,23 @@ __global__ void __launch_bounds__(kLcThreads, 2) lightning_chunk_kernel(const Li
 #pragma unroll
     for (int it = 0; it < kLcTok * kLcV / 8 / kLcThreads; ++it) {
       const int i = tid + it * kLcThreads, r = i / (kLcV / 8), d = (i % (kLcV / 8)) * 8;
-      float f[8], hi[8];
+      float f[8];
       load8(v + static_cast<int64_t>(c0 + r) * p.v_ld + d, r < nv && d < cols, f);
-      *reinterpret_cast<uint4*>(sV + r * kLcLdV + d) = pack8(f);
+      const uint4 raw = pack8(f);
+      *reinterpret_cast<uint4*>(sV + r * kLcLdV + d) = raw;
       const float w = r < nv ? sPow[nv - 1 - r] : 0.f;
+      const uint32_t* u = reinterpret_cast<const uint32_t*>(&raw);
 #pragma unroll
-      for (int j = 0; j < 8; ++j) f[j] *= w;
-#pragma unroll
-      for (int t = 0; t < 3; ++t) {
-#pragma unroll
-        for (int j = 0; j < 8; ++j) hi[j] = bf16_part(f[j], f[j]);
-        *reinterpret_cast<uint4*>(sW + (t * kLcTok + r) * kLcLdV + d) = pack8(hi);
+      for (int j = 0; j < 4; ++j) {        // the rounded value, scaled
+        const float2 t = unpack_bf16x2(u[j]);
+        f[2 * j] = t.x * w;
+        f[2 * j + 1] = t.y * w;
       }
+#pragma unroll
+      for (int t = 0; t < 2; ++t)
+        *reinterpret_cast<uint4*>(sW + (t * kLcTok + r) * kLcLdV + d) =
+            make_uint4(cut_term(f[0], f[1]), cut_term(f[2], f[3]), cut_term(f[4], f[5]), cut_term(f[6], f[7]));
+      *reinterpret_cast<uint4*>(sW + (2 * kLcTok + r) * kLcLdV + d) = pack8(f);
     }
     // ---- the state before the chunk as an operand ----
 #pragma unroll
@@ -355,28 +370,32 @@ __global__ void __launch_bounds__(kLcThreads, 2) lightning_chunk_kernel(const Li
         }
       }
     }
-    // ---- S' = decay^n S + K^T W ----
+    // ---- S' = decay^n S + K^T W.  The chunk's sum is formed by itself and added in one fp32 operation: the tensor core
+    // cuts off what an accumulator cannot hold, which would add up in the large S ----
     const float carry = sPow[nv];
+    float add[kNT][4];
 #pragma unroll
-    for (int nt = 0; nt < kNT; ++nt)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) st[nt][e] *= carry;
+    for (int nt = 0; nt < kNT; ++nt) add[nt][0] = add[nt][1] = add[nt][2] = add[nt][3] = 0.f;
 #pragma unroll
     for (int kt = 0; kt < kLcTok / 16; ++kt) {
       if (kt * 16 < nv) {
         uint32_t ka[4];
         ldsm4_t(ka, smem_u32(sK + (kt * 16 + (lane >> 4) * 8 + (lane & 7)) * kLd + mt * 16 + ((lane >> 3) & 1) * 8));
 #pragma unroll
-        for (int t = 0; t < 3; ++t)
+        for (int t = 2; t >= 0; --t)
 #pragma unroll
           for (int np = 0; np < kNT / 2; ++np) {
             uint32_t bb[4];
             ldsm4_t(bb, smem_u32(sW + (t * kLcTok + kt * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * kLcLdV + (n0 + np * 2) * 8 + (lane >> 4) * 8));
-            mma_16816<bf16>(st[np * 2], ka[0], ka[1], ka[2], ka[3], bb[0], bb[1]);
-            mma_16816<bf16>(st[np * 2 + 1], ka[0], ka[1], ka[2], ka[3], bb[2], bb[3]);
+            mma_16816<bf16>(add[np * 2], ka[0], ka[1], ka[2], ka[3], bb[0], bb[1]);
+            mma_16816<bf16>(add[np * 2 + 1], ka[0], ka[1], ka[2], ka[3], bb[2], bb[3]);
           }
       }
     }
+#pragma unroll
+    for (int nt = 0; nt < kNT; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) st[nt][e] = fmaf(st[nt][e], carry, add[nt][e]);
     __syncthreads();      // every operand of this chunk has been read
   }
   if constexpr (MODE == kSums) {

@@ -2,7 +2,7 @@
 
 Each preset is a plain attribute bag with the HF ``config.json`` field names the
 models read.  Shapes: Qwen3 dense (0.6B / 1.7B / 4B / 8B / 14B / 32B), Qwen3-30B-A3B
-(MoE), Llama / Qwen2 decoders, the Qwen3.5 hybrids, and the vision+language pairs Qwen3-VL-2B, Qwen2-VL-2B
+(MoE), Llama / Qwen2 decoders, the Qwen3.5 hybrids, Pebulix, Kesovik, and the vision+language pairs Qwen3-VL-2B, Qwen2-VL-2B
 and Qwen2.5-VL-3B (each with a ``-tiny`` shape for tests).
 """
 

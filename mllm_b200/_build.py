@@ -3,7 +3,8 @@
 The extensions live under ``mllm_b200/csrc``:
 
 * ``mllm_b200_C``    — the sm_100a CUDA kernels of every decoder plus their PyTorch binding;
-* ``mllm_b200_R``    — gated delta rule and latent attention;
+* ``mllm_b200_R``    — gated delta rule;
+* ``mllm_b200_A``    — latent attention;
 * ``mllm_b200_L``    — lightning attention (linear attention with a fixed decay per head);
 * ``mllm_b200_E``    — mixtures of experts;
 * ``mllm_b200_X``    — 4-bit weights, vision towers, tensor- and expert-parallel exchange;
@@ -51,7 +52,12 @@ EXTENSIONS: Dict[str, Dict[str, List[str]]] = {
         "cuda": True,
     },
     "mllm_b200_R": {
-        "sources": ["bindings_recurrent.cpp", "runtime.cu", "gdn.cu", "gdn_chunk.cu", "latent.cu"],
+        "sources": ["bindings_recurrent.cpp", "runtime.cu", "gdn.cu", "gdn_chunk.cu"],
+        "headers": _COMMON,
+        "cuda": True,
+    },
+    "mllm_b200_A": {
+        "sources": ["bindings_latent.cpp", "runtime.cu", "latent.cu"],
         "headers": _COMMON,
         "cuda": True,
     },

@@ -259,7 +259,8 @@ void embedding_f32(const Tensor& ids, const Tensor& table, double scale, Tensor&
 // x [T, W] fp32 (updated in place when `update`), y [T, W] or none, ls / w fp32 [W], h [T, W].  experts: (expert rows
 // [P, W], sorted_pos [T * top], topk_w [T, top], ids [T, top], token_in [T, W]) or empty
 void post_norm(Tensor& x, const c10::optional<Tensor>& y, const c10::optional<Tensor>& ls, double alpha, const Tensor& w, double eps,
-               Tensor& h, bool update, const std::vector<Tensor>& experts, int64_t identity_from) {
+               Tensor& h, bool update, const std::vector<Tensor>& experts, int64_t identity_from, bool inner,
+               const c10::optional<Tensor>& y_logit) {
   check_float(h, "h");
   TORCH_CHECK(x.is_cuda() && x.scalar_type() == at::kFloat && x.dim() == 2 && x.is_contiguous() && h.is_contiguous() &&
                   h.sizes() == x.sizes(),
@@ -299,6 +300,13 @@ void post_norm(Tensor& x, const c10::optional<Tensor>& y, const c10::optional<Te
   a.width = W;
   a.alpha = static_cast<float>(alpha);
   a.eps = static_cast<float>(eps);
+  a.inner = inner ? 1 : 0;
+  if (y_logit.has_value()) {
+    TORCH_CHECK(y_logit->is_cuda() && y_logit->scalar_type() == at::kFloat && y_logit->dim() == 1 && y_logit->size(0) == T,
+                "post_norm: y_logit fp32 [T]");
+    a.y_logit = y_logit->data_ptr<float>();
+    a.y_logit_ld = y_logit->stride(0);
+  }
   a.dt = dtype_of(h);
   const int rc = mb200::launch_post_norm(a, stream_of(x));
   TORCH_CHECK(rc == 0, "post_norm: row too wide or too many choices (code ", rc, ")");
@@ -368,6 +376,55 @@ void rownorm_rope_kv(const Tensor& row, const Tensor& q_w, const Tensor& k_w, co
   a.dt = dtype_of(row);
   const int rc = mb200::launch_rownorm_rope_kv(a, stream_of(row));
   TORCH_CHECK(rc == 0, "rownorm_rope_kv: unsupported sizes (code ", rc, ")");
+}
+
+// row [T, >= (heads + kv_heads) * dim] with values at column v_at; q_out [T, heads, q_width]; caches [slots, kv_heads, >= width]
+void headnorm_rope_kv(const Tensor& row, const Tensor& inv_freq, const Tensor& positions, const Tensor& loc, Tensor& q_out, Tensor& k_cache,
+                      Tensor& v_cache, int64_t heads, int64_t kv_heads, int64_t dim, int64_t vdim, int64_t v_at, bool halves, double eps) {
+  check_float(row, "row");
+  const int64_t T = row.size(0);
+  TORCH_CHECK(row.dim() == 2 && row.stride(1) == 1 && row.size(1) >= (heads + kv_heads) * dim && v_at >= 0 &&
+                  row.size(1) >= v_at + kv_heads * vdim && q_out.is_contiguous() && q_out.dim() == 3 && q_out.size(0) == T &&
+                  q_out.size(1) == heads && q_out.size(2) >= dim && q_out.scalar_type() == row.scalar_type() && q_out.is_cuda(),
+              "headnorm_rope_kv: row [T, q | k | ..], q_out [T, heads, >= dim]");
+  for (const Tensor* t : {&k_cache, &v_cache})
+    TORCH_CHECK(t->is_cuda() && t->dim() == 3 && t->stride(2) == 1 && t->size(1) == kv_heads && t->scalar_type() == row.scalar_type() &&
+                    t->size(0) == k_cache.size(0),
+                "headnorm_rope_kv: caches [slots, kv_heads, width] of the rows' type");
+  TORCH_CHECK(k_cache.size(2) >= dim && v_cache.size(2) >= vdim && positions.is_cuda() && positions.scalar_type() == at::kLong &&
+                  positions.is_contiguous() && positions.numel() == T && loc.is_cuda() && loc.scalar_type() == at::kLong &&
+                  loc.is_contiguous() && loc.numel() == T && inv_freq.is_cuda() && inv_freq.scalar_type() == at::kDouble &&
+                  inv_freq.is_contiguous(),
+              "headnorm_rope_kv: int64 positions and slots [T], fp64 frequencies");
+  c10::cuda::CUDAGuard g(row.device());
+  mb200::HeadNormRopeArgs a{};
+  a.row = row.data_ptr();
+  a.inv_freq = inv_freq.data_ptr<double>();
+  a.positions = positions.data_ptr<int64_t>();
+  a.loc = loc.data_ptr<int64_t>();
+  a.q_out = q_out.data_ptr();
+  a.k_cache = k_cache.data_ptr();
+  a.v_cache = v_cache.data_ptr();
+  a.status = device_state(row.get_device()).status.data_ptr<int>();
+  a.row_ld = row.stride(0);
+  a.k_tok_stride = k_cache.stride(0);
+  a.k_head_stride = k_cache.stride(1);
+  a.v_tok_stride = v_cache.stride(0);
+  a.v_head_stride = v_cache.stride(1);
+  a.num_slots = k_cache.size(0);
+  a.tokens = T;
+  a.heads = heads;
+  a.kv_heads = kv_heads;
+  a.dim = dim;
+  a.vdim = vdim;
+  a.v_at = v_at;
+  a.q_width = q_out.size(2);
+  a.rot_dims = 2 * inv_freq.numel();
+  a.halves = halves ? 1 : 0;
+  a.eps = static_cast<float>(eps);
+  a.dt = dtype_of(row);
+  const int rc = mb200::launch_headnorm_rope_kv(a, stream_of(row));
+  TORCH_CHECK(rc == 0, "headnorm_rope_kv: unsupported sizes (code ", rc, ")");
 }
 
 // out fp32 [T, W] = cap * tanh(x / cap)
@@ -745,9 +802,11 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("gemm_tp", &gemm_tp);
   m.def("residual_dyt", &residual_dyt);
   m.def("embedding_f32", &embedding_f32);
-  m.def("post_norm", &post_norm);
+  m.def("post_norm", &post_norm, py::arg("x"), py::arg("y"), py::arg("ls"), py::arg("alpha"), py::arg("w"), py::arg("eps"), py::arg("h"),
+        py::arg("update"), py::arg("experts"), py::arg("identity_from"), py::arg("inner") = false, py::arg("y_logit") = py::none());
   m.def("rmsnorm_sigmoid_gate", &rmsnorm_sigmoid_gate);
   m.def("rownorm_rope_kv", &rownorm_rope_kv);
+  m.def("headnorm_rope_kv", &headnorm_rope_kv);
   m.def("soft_cap", &soft_cap);
   m.def("relu_squared", &relu_squared);
   m.def("attention_rows", &attention_rows);

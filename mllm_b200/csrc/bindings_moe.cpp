@@ -17,8 +17,9 @@ void moe_router_logits(const Tensor& x, const Tensor& w, Tensor& logits) {
   TORCH_CHECK(rc == 0, "moe_router_logits: launch failed (code ", rc, ")");
 }
 
+// logits [T, >= experts] (a column slice will do); sigmoid, groups / keep, scale: see RouteArgs
 void moe_router_topk(const Tensor& logits, Tensor& w, Tensor& ids, bool renorm, const c10::optional<Tensor>& correction,
-                     double renorm_eps) {
+                     double renorm_eps, bool sigmoid, int64_t groups, int64_t keep, double scale) {
   check_cuda(logits, "logits");
   TORCH_CHECK(logits.dim() == 2 && logits.stride(1) == 1 && logits.size(1) <= 256, "moe_router_topk: [T,E<=256] logits");
   TORCH_CHECK(w.scalar_type() == at::kFloat && ids.scalar_type() == at::kInt && w.is_contiguous() && ids.is_contiguous() &&
@@ -27,9 +28,24 @@ void moe_router_topk(const Tensor& logits, Tensor& w, Tensor& ids, bool renorm, 
   c10::cuda::CUDAGuard g(logits.device());
   if (correction.has_value()) check_f32_vec(*correction, logits.size(1), "correction");
   TORCH_CHECK(w.size(1) <= logits.size(1), "moe_router_topk: more choices than experts");
-  mb200::launch_moe_router_topk(logits.data_ptr(), logits.stride(0), correction.has_value() ? correction->data_ptr<float>() : nullptr,
-                                w.data_ptr<float>(), ids.data_ptr<int>(), logits.size(0), logits.size(1), w.size(1), renorm ? 1 : 0,
-                                static_cast<float>(renorm_eps), dtype_of(logits), stream_of(logits));
+  mb200::RouteArgs a{};
+  a.logits = logits.data_ptr();
+  a.correction = correction.has_value() ? correction->data_ptr<float>() : nullptr;
+  a.w = w.data_ptr<float>();
+  a.ids = ids.data_ptr<int>();
+  a.stride = logits.stride(0);
+  a.tokens = logits.size(0);
+  a.experts = logits.size(1);
+  a.top_k = w.size(1);
+  a.sigmoid = sigmoid ? 1 : 0;
+  a.renorm = renorm ? 1 : 0;
+  a.groups = groups;
+  a.keep = keep;
+  a.renorm_eps = static_cast<float>(renorm_eps);
+  a.scale = static_cast<float>(scale);
+  a.dt = dtype_of(logits);
+  const int rc = mb200::launch_moe_router_topk(a, stream_of(logits));
+  TORCH_CHECK(rc == 0, "moe_router_topk: unsupported choice (code ", rc, "): at most 32 groups of equal size that hold the choices");
 }
 
 void moe_align(const Tensor& topk_ids, int64_t expert_offset, int64_t experts, int64_t bn, Tensor& sorted_pos,
@@ -113,7 +129,8 @@ int64_t moe_grouped_gemm(const Tensor& x, const Tensor& w, Tensor& out, const Te
 PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("moe_router_logits", &moe_router_logits);
   m.def("moe_router_topk", &moe_router_topk, py::arg("logits"), py::arg("w"), py::arg("ids"), py::arg("renorm"),
-        py::arg("correction") = py::none(), py::arg("renorm_eps") = 0.0);
+        py::arg("correction") = py::none(), py::arg("renorm_eps") = 0.0, py::arg("sigmoid") = false, py::arg("groups") = 1,
+        py::arg("keep") = 1, py::arg("scale") = 1.0);
   m.def("moe_align", &moe_align);
   m.def("moe_gather", &moe_gather);
   m.def("moe_combine", &moe_combine);

@@ -1,4 +1,4 @@
-// PyTorch binding of the gated delta rule and of latent attention (module mllm_b200_R).
+// PyTorch binding of the gated delta rule (module mllm_b200_R).
 #include "bindings_common.h"
 
 namespace {
@@ -135,112 +135,6 @@ int64_t gdn_chunk(const Tensor& q, const Tensor& k, const Tensor& v, const Tenso
   return 0;
 }
 
-// ---- latent attention ----
-// y [T, q_rank (+ kv_rank)]; cq [T, q_rank]; cache [slots, kv_rank] and loc only when the layer writes latents
-void latent_prologue(const Tensor& y, const Tensor& q_w, const c10::optional<Tensor>& kv_w, double eps, Tensor& cq,
-                     const c10::optional<Tensor>& loc, c10::optional<Tensor> cache) {
-  check_float(y, "y");
-  const int64_t q_rank = q_w.numel(), kv_rank = kv_w.has_value() ? kv_w->numel() : 0;
-  TORCH_CHECK(y.dim() == 2 && y.stride(1) == 1 && y.size(1) >= q_rank + kv_rank && cq.is_contiguous() && cq.dim() == 2 &&
-                  cq.size(0) == y.size(0) && cq.size(1) == q_rank && cq.scalar_type() == y.scalar_type(),
-              "latent_prologue: y [T, q_rank + kv_rank], cq [T, q_rank]");
-  check_f32_vec(q_w, q_rank, "q_w");
-  if (kv_rank > 0) {
-    check_f32_vec(*kv_w, kv_rank, "kv_w");
-    TORCH_CHECK(loc.has_value() && cache.has_value() && loc->is_cuda() && loc->scalar_type() == at::kLong && loc->is_contiguous() &&
-                    loc->numel() == y.size(0) && cache->dim() == 2 && cache->stride(1) == 1 && cache->size(1) == kv_rank &&
-                    cache->scalar_type() == y.scalar_type(),
-                "latent_prologue: loc int64 [T], cache [slots, kv_rank]");
-  }
-  c10::cuda::CUDAGuard g(y.device());
-  auto& st = device_state(y.get_device());
-  mb200::launch_latent_prologue(y.data_ptr(), y.stride(0), y.size(0), q_rank, kv_rank, q_w.data_ptr<float>(),
-                                kv_rank > 0 ? kv_w->data_ptr<float>() : nullptr, static_cast<float>(eps), cq.data_ptr(),
-                                kv_rank > 0 ? loc->data_ptr<int64_t>() : nullptr, kv_rank > 0 ? cache->data_ptr() : nullptr,
-                                kv_rank > 0 ? cache->stride(0) : 0, kv_rank > 0 ? cache->size(0) : 0, dtype_of(y),
-                                st.status.data_ptr<int>(), stream_of(y));
-}
-
-void latent_gather(const Tensor& cache, const Tensor& req_to_token, const Tensor& req, const Tensor& lens, const Tensor& start,
-                   int64_t max_len, Tensor& out) {
-  check_float(cache, "cache");
-  for (const Tensor* t : {&req_to_token, &req, &lens, &start})
-    TORCH_CHECK(t->scalar_type() == at::kInt && t->is_cuda(), "latent_gather: index tensors must be int32 CUDA tensors");
-  TORCH_CHECK(cache.dim() == 2 && cache.stride(1) == 1 && req_to_token.dim() == 2 && req_to_token.stride(1) == 1 &&
-                  max_len <= req_to_token.size(1) && req.numel() == lens.numel() && req.numel() == start.numel() &&
-                  out.is_contiguous() && out.dim() == 2 && out.size(1) == cache.size(1) && out.scalar_type() == cache.scalar_type(),
-              "latent_gather: cache [slots, rank], out [rows, rank]");
-  c10::cuda::CUDAGuard g(cache.device());
-  auto& st = device_state(cache.get_device());
-  mb200::launch_latent_gather(cache.data_ptr(), cache.stride(0), cache.size(1), cache.element_size(), req_to_token.data_ptr<int>(),
-                              req_to_token.stride(0), req.data_ptr<int>(), lens.data_ptr<int>(), start.data_ptr<int>(), req.numel(),
-                              max_len, out.data_ptr(), cache.size(0), st.status.data_ptr<int>(), stream_of(cache));
-}
-
-// out[t, h, :] = w[h] x[t, h, :].  Returns non-zero (nothing launched) when the shape is not the kernel's.
-int64_t head_linear(const Tensor& x, const Tensor& w, Tensor& out) {
-  check_float(x, "x");
-  TORCH_CHECK(x.dim() == 3 && x.stride(2) == 1 && w.dim() == 3 && w.is_contiguous() && w.size(0) == x.size(1) &&
-                  w.size(2) == x.size(2) && out.dim() == 3 && out.stride(2) == 1 && out.size(0) == x.size(0) &&
-                  out.size(1) == x.size(1) && out.size(2) == w.size(1) && w.scalar_type() == x.scalar_type() &&
-                  out.scalar_type() == x.scalar_type(),
-              "head_linear: x [T, H, K], w [H, N, K], out [T, H, N]");
-  if ((reinterpret_cast<uintptr_t>(x.data_ptr()) | reinterpret_cast<uintptr_t>(w.data_ptr())) & 15) return 1;
-  c10::cuda::CUDAGuard g(x.device());
-  return mb200::launch_head_linear(x.data_ptr(), x.stride(0), x.stride(1), w.data_ptr(), out.data_ptr(), out.stride(0), out.stride(1),
-                                   x.size(0), x.size(1), w.size(1), w.size(2), device_state(x.get_device()).num_sms, dtype_of(x),
-                                   stream_of(x));
-}
-
-// q, out [rows, H, R]; cache [slots, R]; row_req int32, row_pos int64 [rows]; max_seq_len sizes the split of the context
-void latent_attention(const Tensor& q, const Tensor& cache, const Tensor& req_to_token, const Tensor& row_req, const Tensor& row_pos,
-                      double scale, const c10::optional<Tensor>& sink, Tensor& out, int64_t max_seq_len) {
-  check_float(q, "q");
-  TORCH_CHECK(q.dim() == 3 && q.is_contiguous() && out.is_contiguous() && out.sizes() == q.sizes() &&
-                  out.scalar_type() == q.scalar_type() && cache.dim() == 2 && cache.stride(1) == 1 && cache.size(1) == q.size(2) &&
-                  cache.scalar_type() == q.scalar_type() && cache.is_cuda() && q.size(2) <= 1024 && q.size(0) <= 65535,
-              "latent_attention: q, out [rows <= 65535, H, R <= 1024], cache [slots, R] of one type");
-  TORCH_CHECK(req_to_token.is_cuda() && req_to_token.scalar_type() == at::kInt && req_to_token.dim() == 2 &&
-                  req_to_token.stride(1) == 1 && row_req.is_cuda() && row_req.scalar_type() == at::kInt && row_req.is_contiguous() &&
-                  row_req.numel() == q.size(0) && row_pos.is_cuda() && row_pos.scalar_type() == at::kLong &&
-                  row_pos.is_contiguous() && row_pos.numel() == q.size(0),
-              "latent_attention: row_req int32 [rows], row_pos int64 [rows]");
-  c10::cuda::CUDAGuard g(q.device());
-  auto& st = device_state(q.get_device());
-  mb200::LatentAttnArgs a{};
-  a.rows = q.size(0);
-  a.heads = q.size(1);
-  a.rank = q.size(2);
-  a.cache_ld = cache.stride(0);
-  a.dt = dtype_of(q);
-  if (sink.has_value()) {
-    check_f32_vec(*sink, a.heads, "sink");
-    a.sink = sink->data_ptr<float>();
-  }
-  a.splits = mb200::latent_mma_covers(a.rank, a.cache_ld, a.dt)
-                 ? mb200::latent_num_splits(a.rows, a.heads, max_seq_len > 0 ? max_seq_len : req_to_token.size(1), st.num_sms)
-                 : 1;
-  Tensor part_o, part_lse;
-  if (a.splits > 1) {
-    part_o = torch::empty({a.rows, a.heads, a.splits, a.rank}, q.options().dtype(torch::kFloat32));
-    part_lse = torch::empty({a.rows, a.heads, a.splits}, q.options().dtype(torch::kFloat32));
-    a.part_o = part_o.data_ptr<float>();
-    a.part_lse = part_lse.data_ptr<float>();
-  }
-  a.q = q.data_ptr();
-  a.cache = cache.data_ptr();
-  a.out = out.data_ptr();
-  a.req_to_token = req_to_token.data_ptr<int>();
-  a.row_req = row_req.data_ptr<int>();
-  a.row_pos = row_pos.data_ptr<int64_t>();
-  a.status = st.status.data_ptr<int>();
-  a.rtt_stride = req_to_token.stride(0);
-  a.num_slots = cache.size(0);
-  a.scale = static_cast<float>(scale);
-  const int rc = mb200::launch_latent_attention(a, stream_of(q));
-  TORCH_CHECK(rc == 0, "latent_attention: unsupported configuration (code ", rc, ")");
-}
-
 }  // namespace
 
 PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
@@ -249,10 +143,6 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("gdn_gates", &gdn_gates);
   m.def("gdn_recurrent", &gdn_recurrent);
   m.def("gdn_recurrent_raw", &gdn_recurrent_raw);
-  m.def("latent_prologue", &latent_prologue);
-  m.def("latent_gather", &latent_gather);
-  m.def("head_linear", &head_linear);
-  m.def("latent_attention", &latent_attention);
   m.def("gdn_chunk", &gdn_chunk);
   m.def("read_status", &read_status);
   m.def("launch_count", &launch_count);

@@ -47,7 +47,10 @@ struct PostNormArgs {
   const float* topk_w;
   const int* ids;
   const void* token_in;
+  const float* y_logit;     // one per row, y_logit_ld apart, or null: y times its logistic function
+  int64_t y_logit_ld;
   int rows, width, top, identity_from;
+  int inner;                // 0: x <- norm(alpha * x + ls * y), 1: x <- alpha * x + ls * norm(y)
   float alpha, eps;
   DType dt;                 // of y, h, expert_rows, token_in
 };
@@ -74,6 +77,24 @@ struct RowNormRopeArgs {
   DType dt;
 };
 int launch_rownorm_rope_kv(const RowNormRopeArgs& args, cudaStream_t s);
+// rows [q | k | ..] of tokens: rotation of part of every query and key head, each head divided by its root mean square,
+// q to q_out [tokens, heads, q_width] (zeros behind dim), k and the unchanged values to the cache slots loc
+struct HeadNormRopeArgs {
+  const void* row;          // row t at t * row_ld: heads * dim and kv_heads * dim features, kv_heads * vdim values at v_at
+  const double* inv_freq;   // [rot_dims / 2]
+  const int64_t* positions; // [tokens]
+  const int64_t* loc;       // [tokens]
+  void* q_out;
+  void* k_cache;            // head h of slot s at s * tok + h * head (elements)
+  void* v_cache;
+  int* status;
+  int64_t row_ld, k_tok_stride, k_head_stride, v_tok_stride, v_head_stride, num_slots;
+  int tokens, heads, kv_heads, dim, vdim, v_at, q_width, rot_dims;
+  int halves;               // pairs are (i, i + rot_dims / 2); 0: neighbours (2i, 2i + 1)
+  float eps;
+  DType dt;
+};
+int launch_headnorm_rope_kv(const HeadNormRopeArgs& args, cudaStream_t s);
 void launch_soft_cap(const void* x, int64_t x_ld, float* out, int rows, int width, float cap, DType dt, cudaStream_t s);
 void launch_relu_squared(void* x, int64_t n, DType dt, cudaStream_t s);
 void launch_gelu_tanh(const void* x, void* out, int64_t n, DType dt, cudaStream_t s);
@@ -228,10 +249,22 @@ int launch_ep_return(const EpA2AArgs& a, const void* ys, const int* recv_rows, i
 // logits[t, e] = x[t] . w[e] in fp32 (products of 16-bit values are exact in it)
 int launch_moe_router_logits(const void* x, int64_t x_ld, const void* w, float* logits, int tokens, int experts, int hidden,
                              int num_sms, DType dt, cudaStream_t s);
-// router: fp32 softmax over `experts` (<= 256) logits -> top_k (<= 32, sorted, lowest index wins ties).  The choice goes by
-// the scores plus `correction` (may be null), the weights are the scores; renorm divides them by their sum + renorm_eps
-void launch_moe_router_topk(const void* logits, int64_t stride, const float* correction, float* w, int* ids, int tokens, int experts,
-                            int top_k, int renorm, float renorm_eps, DType dt, cudaStream_t s);
+// router: fp32 scores of `experts` (<= 256) logits -> top_k (<= 32, sorted, lowest index wins ties).  The choice goes by
+// the scores plus `correction`, the weights are the scores
+struct RouteArgs {
+  const void* logits;       // [tokens, >= experts], rows `stride` apart
+  const float* correction;  // [experts] or null
+  float* w;                 // [tokens, top_k]
+  int* ids;                 // [tokens, top_k]
+  int64_t stride;
+  int tokens, experts, top_k;
+  int sigmoid;              // scores: 0 softmax over the experts, 1 logistic function of each logit
+  int renorm;               // weights divided by their sum + renorm_eps
+  int groups, keep;         // keep < groups: only experts of the `keep` groups with the largest sums of two choice scores
+  float renorm_eps, scale;  // scale: factor of the weights
+  DType dt;                 // of the logits
+};
+int launch_moe_router_topk(const RouteArgs& args, cudaStream_t s);
 // counting sort of the (token, choice) pairs by local expert.  sorted_pos[pair] = row in the sorted
 // matrix or -1 (expert on another rank); src_token[row] = token; expert_offsets[experts + 1];
 // work[i] = (expert, chunk of bn rows), *n_work items.
@@ -336,22 +369,54 @@ int launch_lightning_recurrent(const LightningArgs& args, cudaStream_t s);
 int launch_lightning_chunk(const LightningArgs& args, cudaStream_t s);
 bool lightning_chunk_covers(const LightningArgs& args);
 
-// ----- latent attention (one cached row of `rank` features per token, shared by all heads) ------------
-// RMS norm of both parts of the down projections' rows [q_rank | kv_rank]: the first into cq [tokens, q_rank], the
-// second into the cache row loc[t].  kv_rank 0: the layer reads another layer's latents and writes none.
-void launch_latent_prologue(const void* y, int64_t ld, int tokens, int q_rank, int kv_rank, const float* q_w, const float* kv_w,
-                            float eps, void* cq, const int64_t* loc, void* cache, int64_t cache_ld, int64_t num_slots, DType dt,
-                            int* status, cudaStream_t s);
+// ----- latent attention (one cached row of `rank` features per token, shared by all heads; `rot` rotated key features may
+// follow them in the row) ------------
+// Rows [q_rank | kv_rank | rot | ..] of the down projections: RMS norm of the first two, the first into cq, the second into
+// the cache row loc[t], where the third follows it, its neighbouring features turned by positions[t] * inv_freq.  kv_rank 0:
+// the layer reads another layer's rows and writes none.
+struct LatentPrologueArgs {
+  const void* y;            // [tokens, ..], rows ld apart
+  const float* q_w;         // [q_rank]
+  const float* kv_w;        // [kv_rank]
+  const double* inv_freq;   // [rot / 2]
+  const int64_t* positions; // [tokens]
+  float2* turns;            // [tokens, rot / 2]: cosine and sine of every token, written
+  void* cq;                 // [tokens, q_rank]
+  const int64_t* loc;       // [tokens]
+  void* cache;
+  int* status;
+  int64_t ld, cache_ld, num_slots;
+  int tokens, q_rank, kv_rank, rot;
+  float eps;
+  DType dt;
+};
+void launch_latent_prologue(const LatentPrologueArgs& args, cudaStream_t s);
+// neighbouring features of x [tokens, heads, rot] (strided) turn by turns [tokens, rot / 2]; out may be x
+void launch_turn_heads(const void* x, int64_t x_tok, int64_t x_head, const float2* turns, void* out, int64_t out_tok, int64_t out_head,
+                       int tokens, int heads, int rot, DType dt, cudaStream_t s);
+// out [tokens, heads, width] = x (strided) * sigmoid(gate[t, h]), rows of gate gate_ld apart
+void launch_gate_heads(const void* x, int64_t x_tok, int64_t x_head, const void* gate, int64_t gate_ld, void* out, int tokens, int heads,
+                       int width, DType dt, cudaStream_t s);
 // out[start[b] + j] = latent of token j of request b, j < lens[b]
 void launch_latent_gather(const void* cache, int64_t cache_ld, int rank, int elem_bytes, const int* rtt, int64_t rtt_stride,
                           const int* req, const int* lens, const int* start, int batch, int max_len, void* out,
                           int64_t num_slots, int* status, cudaStream_t s);
-// out[t, h, :] = w[h] x[t, h, :] with w [heads, N, K], K % 8 == 0, 16-bit types (else -1)
-int launch_head_linear(const void* x, int64_t x_tok, int64_t x_head, const void* w, void* out, int64_t out_tok, int64_t out_head,
-                       int tokens, int heads, int N, int K, int num_sms, DType dt, cudaStream_t s);
+// out[t, h, :N] = w[h] x[t, h, :K], times sigmoid(gate[t, h]) where gate is given; the `rot` features behind K are turned by
+// turns [tokens, rot / 2] and put behind N.  K % 8 == 0, 16-bit types (else -1)
+struct HeadLinearArgs {
+  const void* x;
+  const void* w;            // [heads, N, K]
+  void* out;
+  const void* gate;         // [tokens, heads] with rows gate_ld apart, or null
+  const float2* turns;
+  int64_t x_tok, x_head, out_tok, out_head, gate_ld;
+  int tokens, heads, N, K, rot;
+  DType dt;
+};
+int launch_head_linear(const HeadLinearArgs& args, int num_sms, cudaStream_t s);
 struct LatentAttnArgs {
-  const void* q;            // [rows, heads, rank] queries taken to the latent space
-  const void* cache;        // latent of slot s at s * cache_ld (elements)
+  const void* q;            // [rows, heads, key] queries taken to the latent space, key >= rank
+  const void* cache;        // row of slot s at s * cache_ld (elements): key features, values are the first rank of them
   void* out;                // [rows, heads, rank]
   float* part_o;            // splits > 1: [rows, heads, splits, rank]
   float* part_lse;          // splits > 1: [rows, heads, splits]
@@ -361,13 +426,13 @@ struct LatentAttnArgs {
   const float* sink;        // [heads] or null
   int* status;
   int64_t rtt_stride, cache_ld, num_slots;
-  int rows, heads, rank, splits;
+  int rows, heads, key, rank, splits;
   float scale;
   DType dt;
 };
 int launch_latent_attention(const LatentAttnArgs& args, cudaStream_t s);
 int latent_num_splits(int rows, int heads, int max_seq_len, int num_sms);
-bool latent_mma_covers(int rank, int64_t cache_ld, DType dt);   // false: the fp32 kernel runs, splits must be 1
+bool latent_mma_covers(int key, int rank, int64_t cache_ld, DType dt);   // false: the fp32 kernel runs, splits must be 1
 
 // ----- gated delta net (hybrid models) -----------------------------------------------------------
 // Ragged sequences: request b owns rows q_start[b] .. q_start[b] + lens[b] of the token-major inputs and

@@ -1,14 +1,17 @@
 // Latent attention: every token leaves ONE row c of `rank` features in the cache, shared by all heads; a head's keys
-// and values are W_uk[h] c and W_uv[h] c.  Two ways to evaluate it, both causal, both with an optional sink per head:
+// and values are W_uk[h] c and W_uv[h] c.  A cached row may carry `rot` features more, a rotated key part that all heads
+// share: keys are then `key` = rank + rot features wide in the latent space, values stay `rank` wide.  Two ways to evaluate
+// it, both causal, both with an optional sink per head:
 //
 //   expanded (many new tokens): K and V of the whole context are formed by matrix products and the ordinary
 //       attention kernels run on them; this file only gathers the context's latents (latent_gather).
 //   absorbed (decode, short extends): the products move to the query side.  q' = W_uk[h]^T q has `rank` features,
-//       score = q' . c, and the weighted sum of the c rows is carried through W_uv[h] once per query.  The cache is
-//       read once for all heads and nothing per head is stored.
+//       score = q' . c (plus the rotated parts' product: q' continues with the head's rotated query part), and the
+//       weighted sum of the c rows is carried through W_uv[h] once per query.  The cache is read once for all heads and
+//       nothing per head is stored.
 //
 // latent_attn_mma_kernel is the absorbed form for 16-bit types.  A CTA owns one query token, 16 or 32 heads (the MMA
-// M dimension) and a range of the context, 32 tokens at a time.  The rank features are dealt to the warps, CW each:
+// M dimension) and a range of the context, 32 tokens at a time.  The key features are dealt to the warps, CW each:
 // a warp moves its own feature slice of every c row with cp.async, keeps its slice of q' in registers, multiplies
 // the slice's share of the scores and owns the same slice of the output.  So c is read from shared memory twice (as
 // keys, and transposed as values) by the same warp, tiles need no block barrier on their way in, and the warps meet
@@ -27,33 +30,44 @@ namespace {
 constexpr float kLatLog2e = 1.4426950408889634f;
 
 // ---------------------------------------------------------------------------------------------
-// Prologue: the down projections' output rows are [query latent | cache latent]; both are RMS-normed in 32-bit, the
-// first goes to `cq`, the second to the cache row of the token.  grid (tokens, 1 or 2).
+// Prologue: the down projections' output rows are [query latent | cache latent | rotated key part]; both latents are
+// RMS-normed in 32-bit, the first goes to `cq`, the second to the cache row of the token.  The key part is turned by the
+// token's position (neighbouring features) and follows the latent in the cache row; the cosines and sines of the token are
+// left in `turns` for the query heads.  Angles are formed and reduced in fp64.  grid (tokens, 1 or 2).
 // ---------------------------------------------------------------------------------------------
 template <typename T>
-__global__ void __launch_bounds__(128) latent_prologue_kernel(const T* __restrict__ y, int64_t ld, int q_rank, int kv_rank,
-                                                              const float* __restrict__ q_w, const float* __restrict__ kv_w,
-                                                              float eps, T* __restrict__ cq, const int64_t* __restrict__ loc,
-                                                              T* __restrict__ cache, int64_t cache_ld, int64_t num_slots,
-                                                              int* status) {
+__global__ void __launch_bounds__(128) latent_prologue_kernel(const LatentPrologueArgs p) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float red[4];
   const int t = blockIdx.x, part = blockIdx.y, tid = threadIdx.x;
-  const int n = part == 0 ? q_rank : kv_rank;
-  const T* row = y + static_cast<int64_t>(t) * ld + (part == 0 ? 0 : q_rank);
-  const float* w = part == 0 ? q_w : kv_w;
-  T* dst;
-  if (part == 0) {
-    dst = cq + static_cast<int64_t>(t) * q_rank;
-  } else {
-    const int64_t slot = loc[t];
-    if (slot < 0 || slot >= num_slots) {
-      if (tid == 0 && status != nullptr) atomicExch(status, kStatusBadIndex);
-      return;
-    }
-    dst = cache + slot * cache_ld;
+  const int n = part == 0 ? p.q_rank : p.kv_rank;
+  const T* row = static_cast<const T*>(p.y) + static_cast<int64_t>(t) * p.ld + (part == 0 ? 0 : p.q_rank);
+  const float* w = part == 0 ? p.q_w : p.kv_w;
+  T* dst = static_cast<T*>(p.cq) + static_cast<int64_t>(t) * p.q_rank;
+  if (part == 1) {
+    const int64_t slot = p.loc[t];
+    const bool ok = slot >= 0 && slot < p.num_slots;
+    if (!ok && tid == 0 && p.status != nullptr) atomicExch(p.status, kStatusBadIndex);
+    dst = ok ? static_cast<T*>(p.cache) + slot * p.cache_ld : nullptr;
   }
+  if (part == static_cast<int>(gridDim.y) - 1) {
+    const double pos = p.rot > 0 ? static_cast<double>(p.positions[t]) : 0.0;
+    for (int i = tid; i < p.rot / 2; i += 128) {
+      constexpr double kTurn = 6.283185307179586476925286766559;
+      double a = pos * p.inv_freq[i];
+      a -= kTurn * rint(a / kTurn);
+      float s, c;
+      sincosf(static_cast<float>(a), &s, &c);
+      p.turns[static_cast<int64_t>(t) * (p.rot / 2) + i] = make_float2(c, s);
+      if (part == 1 && dst != nullptr) {
+        const float u = to_f32(row[n + 2 * i]), v = to_f32(row[n + 2 * i + 1]);
+        dst[n + 2 * i] = from_f32<T>(u * c - v * s);
+        dst[n + 2 * i + 1] = from_f32<T>(v * c + u * s);
+      }
+    }
+  }
+  if (dst == nullptr) return;
   float ss = 0.f;
   for (int c = tid; c < n; c += 128) {
     const float f = to_f32(row[c]);
@@ -63,8 +77,48 @@ __global__ void __launch_bounds__(128) latent_prologue_kernel(const T* __restric
   if ((tid & 31) == 0) red[tid >> 5] = ss;
   __syncthreads();
   ss = red[0] + red[1] + red[2] + red[3];
-  const float r = 1.f / sqrtf(ss / static_cast<float>(n) + eps);
+  const float r = 1.f / sqrtf(ss / static_cast<float>(n) + p.eps);
   for (int c = tid; c < n; c += 128) dst[c] = from_f32<T>(to_f32(row[c]) * r * w[c]);
+}
+
+// Neighbouring features of x [tokens, heads, rot] turn by the token's `turns` [tokens, rot / 2]; out may be x.  A thread
+// takes a pair.
+template <typename T>
+__global__ void __launch_bounds__(256) turn_heads_kernel(const T* x, int64_t x_tok, int64_t x_head, const float2* __restrict__ turns,
+                                                         T* out, int64_t out_tok, int64_t out_head, int heads, int half, int64_t pairs) {
+  pdl_launch_dependents();
+  pdl_wait();
+  for (int64_t e = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x; e < pairs; e += static_cast<int64_t>(gridDim.x) * blockDim.x) {
+    const int i = static_cast<int>(e % half);
+    const int64_t th = e / half, t = th / heads;
+    const int h = static_cast<int>(th - t * heads);
+    const T* src = x + t * x_tok + h * x_head + 2 * i;
+    T* dst = out + t * out_tok + h * out_head + 2 * i;
+    const float2 cs = turns[t * half + i];
+    const float u = to_f32(src[0]), v = to_f32(src[1]);
+    dst[0] = from_f32<T>(u * cs.x - v * cs.y);
+    dst[1] = from_f32<T>(v * cs.x + u * cs.y);
+  }
+}
+
+__device__ __forceinline__ float lat_sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
+
+// out[t, h, :] = x[t, h, :width] * sigmoid(gate[t, h]); V features per access
+template <typename T, int V>
+__global__ void __launch_bounds__(256) gate_heads_kernel(const T* x, int64_t x_tok, int64_t x_head, const T* __restrict__ gate,
+                                                         int64_t gate_ld, T* out, int heads, int vecs, int64_t total) {
+  pdl_launch_dependents();
+  pdl_wait();
+  struct alignas(sizeof(T) * V) Pack { T e[V]; };
+  for (int64_t e = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x; e < total; e += static_cast<int64_t>(gridDim.x) * blockDim.x) {
+    const int64_t th = e / vecs, t = th / heads;
+    const int c = static_cast<int>(e - th * vecs) * V, h = static_cast<int>(th - t * heads);
+    const float g = lat_sigmoid(to_f32(gate[t * gate_ld + h]));
+    Pack r = *reinterpret_cast<const Pack*>(x + t * x_tok + h * x_head + c);
+#pragma unroll
+    for (int i = 0; i < V; ++i) r.e[i] = from_f32<T>(to_f32(r.e[i]) * g);
+    *reinterpret_cast<Pack*>(out + th * vecs * V + c) = r;
+  }
 }
 
 // Rows of a request's context, in position order: out[start[b] + j] = cache[rtt[req[b]][j]] for j < lens[b].
@@ -92,14 +146,17 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const V* __restrict_
 // ---------------------------------------------------------------------------------------------
 // Per-head projection out[t, h, :] = W[h] x[t, h, :], W [H, N, K].  A warp owns 16 rows of one head's W (the MMA M
 // dimension) and tiles of 8 tokens; a lane feeds 16 contiguous bytes of W and of x to two MMAs, the same
-// permutation of k in both operands.  KS > 1: the warps of the CTA split k of the same 16 rows.
+// permutation of k in both operands.  KS > 1: the warps of the CTA split k of the same 16 rows.  gate: row t, head h is
+// multiplied by sigmoid(gate[t, h]).  rot > 0: the heads of x and of out go on with `rot` features behind K and N, which the
+// last CTAs of the x dimension turn by the tokens' `turns`.
 // ---------------------------------------------------------------------------------------------
 constexpr int kHlTokTiles = 4;   // tiles of 8 tokens per CTA
 
 template <typename T, int KS>
 __global__ void __launch_bounds__(128) head_linear_kernel(const T* __restrict__ x, int64_t x_tok, int64_t x_head,
                                                           const T* __restrict__ w, T* __restrict__ out, int64_t out_tok,
-                                                          int64_t out_head, int tokens, int N, int K) {
+                                                          int64_t out_head, int tokens, int N, int K, const T* __restrict__ gate,
+                                                          int64_t gate_ld, const float2* __restrict__ turns, int rot) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float part[KS > 1 ? KS : 1][kHlTokTiles][16][8];
@@ -107,6 +164,20 @@ __global__ void __launch_bounds__(128) head_linear_kernel(const T* __restrict__ 
   const int h = blockIdx.y;
   const int n0 = KS > 1 ? blockIdx.x * 16 : (blockIdx.x * 4 + warp) * 16;
   const int t0 = blockIdx.z * kHlTokTiles * 8;
+  if (rot > 0 && blockIdx.x == gridDim.x - 1) {
+    const int half = rot / 2, mine = min(tokens - t0, kHlTokTiles * 8);
+    for (int e = threadIdx.x; e < mine * half; e += 128) {
+      const int t = t0 + e / half, i = e % half;
+      const T* src = x + t * x_tok + h * x_head + K + 2 * i;
+      T* dst = out + t * out_tok + h * out_head + N + 2 * i;
+      const float2 cs = turns[static_cast<int64_t>(t) * half + i];
+      const float u = to_f32(src[0]), v = to_f32(src[1]);
+      dst[0] = from_f32<T>(u * cs.x - v * cs.y);
+      dst[1] = from_f32<T>(v * cs.x + u * cs.y);
+    }
+    return;
+  }
+  auto gate_of = [&](int t) { return gate == nullptr ? 1.f : lat_sigmoid(to_f32(gate[t * gate_ld + h])); };
   const int g = lane >> 2, q = lane & 3;
   float acc[kHlTokTiles][4];
 #pragma unroll
@@ -150,16 +221,22 @@ __global__ void __launch_bounds__(128) head_linear_kernel(const T* __restrict__ 
         float v = 0.f;
 #pragma unroll
         for (int s = 0; s < KS; ++s) v += part[s][i][r][tok];
-        out[t * out_tok + h * out_head + n0 + r] = from_f32<T>(v);
+        out[t * out_tok + h * out_head + n0 + r] = from_f32<T>(v * gate_of(t));
       }
     }
   } else if (n0 < N) {
 #pragma unroll
     for (int i = 0; i < kHlTokTiles; ++i) {
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int t = t0 + i * 8 + 2 * q + (j & 1), r = n0 + g + (j >> 1) * 8;
-        if (t < tokens && r < N) out[t * out_tok + h * out_head + r] = from_f32<T>(acc[i][j]);
+      for (int j = 0; j < 2; ++j) {
+        const int t = t0 + i * 8 + 2 * q + j;
+        if (t >= tokens) continue;
+        const float f = gate_of(t);
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+          const int r = n0 + g + k * 8;
+          if (r < N) out[t * out_tok + h * out_head + r] = from_f32<T>(acc[i][j + 2 * k] * f);
+        }
       }
     }
   }
@@ -169,8 +246,8 @@ __global__ void __launch_bounds__(128) head_linear_kernel(const T* __restrict__ 
 // Absorbed attention
 // ---------------------------------------------------------------------------------------------
 struct LatentParams {
-  const void* q;            // [rows, heads, rank]
-  const void* cache;        // latent of slot s at s * cache_ld
+  const void* q;            // [rows, heads, key]
+  const void* cache;        // row of slot s at s * cache_ld: `key` features, the first `rank` of them the latent
   void* out;                // [rows, heads, rank]
   float* part_o;            // splits > 1: [rows, heads, splits, rank]
   float* part_lse;          // splits > 1: [rows, heads, splits], log2 domain
@@ -180,7 +257,7 @@ struct LatentParams {
   const float* sink;        // [heads] or null
   int* status;
   int64_t rtt_stride, cache_ld, num_slots;
-  int rows, heads, rank, splits;
+  int rows, heads, key, rank, splits;
   float scale;
 };
 
@@ -208,8 +285,9 @@ struct LatCfg {
   }
 };
 
-template <typename T, int CW, int MT>
-__global__ void __launch_bounds__(256) latent_attn_mma_kernel(const LatentParams p) {
+// NW: the most warps of a CTA, eight for the latents of a power of two, nine when a rotated key part follows them
+template <typename T, int CW, int MT, int NW>
+__global__ void __launch_bounds__(NW * 32) latent_attn_mma_kernel(const LatentParams p) {
   using C = LatCfg<CW, MT>;
   constexpr int kM = MT * 16;
   pdl_launch_dependents();
@@ -243,7 +321,7 @@ __global__ void __launch_bounds__(256) latent_attn_mma_kernel(const LatentParams
   // this warp's slice of q' as MMA A fragments
   uint32_t qa[MT][CW / 16][4];
   {
-    const T* qb = static_cast<const T*>(p.q) + static_cast<int64_t>(row) * p.heads * p.rank;
+    const T* qb = static_cast<const T*>(p.q) + static_cast<int64_t>(row) * p.heads * p.key;
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
@@ -251,7 +329,7 @@ __global__ void __launch_bounds__(256) latent_attn_mma_kernel(const LatentParams
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           const int h = h0 + mt * 16 + g + (j & 1) * 8, c = c0 + ks * 16 + 2 * q + (j >> 1) * 8;
-          qa[mt][ks][j] = (h < p.heads && c < p.rank) ? *reinterpret_cast<const uint32_t*>(qb + static_cast<int64_t>(h) * p.rank + c) : 0u;
+          qa[mt][ks][j] = (h < p.heads && c < p.key) ? *reinterpret_cast<const uint32_t*>(qb + static_cast<int64_t>(h) * p.key + c) : 0u;
         }
   }
   float o[MT][CW / 8][4];
@@ -281,7 +359,7 @@ __global__ void __launch_bounds__(256) latent_attn_mma_kernel(const LatentParams
       const int piece = i * 32 + lane, tk = piece / kCh, ch = piece % kCh;
       const int s = __shfl_sync(0xffffffffu, my_slot, tk);
       const int c = c0 + ch * 8;
-      const bool ok = s >= 0 && c < p.rank;
+      const bool ok = s >= 0 && c < p.key;
       cp16_zfill(dst + tk * C::kRowBytes + ch * 16, cache + (ok ? static_cast<int64_t>(s) * p.cache_ld + c : 0), ok);
     }
   };
@@ -383,6 +461,7 @@ __global__ void __launch_bounds__(256) latent_attn_mma_kernel(const LatentParams
           o[mt][i][3] *= f[1];
         }
       }
+      if (c0 >= p.rank) continue;   // a slice of the rotated part: keys only
 #pragma unroll
       for (int ks = 0; ks < 2; ++ks)
 #pragma unroll
@@ -468,21 +547,22 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const LatentParams p)
   }
 }
 
-// Any element type and any rank up to 1024, all in fp32: one CTA per (query token, head), tiles of 64 context tokens.
-constexpr int kLatAnyTok = 64, kLatAnyThreads = 128, kLatAnyCols = 8;
+// Any element type and any rank up to 1024 (keys up to kLatAnyKeys), all in fp32: one CTA per (query token, head), tiles of
+// 64 context tokens.
+constexpr int kLatAnyTok = 64, kLatAnyThreads = 128, kLatAnyCols = 8, kLatAnyKeys = 1536;
 
 template <typename T>
 __global__ void __launch_bounds__(kLatAnyThreads) latent_attn_any_kernel(const LatentParams p) {
   pdl_launch_dependents();
   pdl_wait();
-  __shared__ float sq[kLatAnyThreads * kLatAnyCols];
+  __shared__ float sq[kLatAnyKeys];
   __shared__ float sc[kLatAnyTok];
   __shared__ int sl[kLatAnyTok];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int h = blockIdx.x, row = blockIdx.y;
   const int64_t at = (static_cast<int64_t>(row) * p.heads + h) * p.rank;
-  const T* qr = static_cast<const T*>(p.q) + at;
-  for (int c = tid; c < p.rank; c += kLatAnyThreads) sq[c] = to_f32(qr[c]);
+  const T* qr = static_cast<const T*>(p.q) + (static_cast<int64_t>(row) * p.heads + h) * p.key;
+  for (int c = tid; c < p.key; c += kLatAnyThreads) sq[c] = to_f32(qr[c]);
   const int n = static_cast<int>(p.row_pos[row]) + 1;
   const int* slots = p.rtt + static_cast<int64_t>(p.row_req[row]) * p.rtt_stride;
   const T* cache = static_cast<const T*>(p.cache);
@@ -505,7 +585,7 @@ __global__ void __launch_bounds__(kLatAnyThreads) latent_attn_any_kernel(const L
     for (int j = warp; j < nt; j += kLatAnyThreads / 32) {
       const T* cr = cache + static_cast<int64_t>(sl[j]) * p.cache_ld;
       float d = 0.f;
-      for (int c = lane; c < p.rank; c += 32) d = fmaf(sq[c], to_f32(cr[c]), d);
+      for (int c = lane; c < p.key; c += 32) d = fmaf(sq[c], to_f32(cr[c]), d);
       d = warp_sum(d);
       if (lane == 0) sc[j] = d * p.scale;
     }
@@ -545,32 +625,70 @@ __global__ void __launch_bounds__(kLatAnyThreads) latent_attn_any_kernel(const L
   }
 }
 
-template <typename T, int CW, int MT>
+template <typename T, int CW, int MT, int NW>
 int launch_latent_cfg(const LatentParams& p, cudaStream_t s) {
-  const int warps = (p.rank + CW - 1) / CW;
+  const int warps = (p.key + CW - 1) / CW;
   const int smem = LatCfg<CW, MT>::smem(warps);
-  if (ensure_dynamic_smem(reinterpret_cast<const void*>(latent_attn_mma_kernel<T, CW, MT>), LatCfg<CW, MT>::smem(8)) != cudaSuccess)
-    return -3;
-  const cudaError_t err = launch_pdl(latent_attn_mma_kernel<T, CW, MT>, dim3(p.splits, (p.heads + MT * 16 - 1) / (MT * 16), p.rows),
-                                     dim3(warps * 32), smem, s, p);
+  auto kern = latent_attn_mma_kernel<T, CW, MT, NW>;
+  if (ensure_dynamic_smem(reinterpret_cast<const void*>(kern), LatCfg<CW, MT>::smem(NW)) != cudaSuccess) return -3;
+  const cudaError_t err = launch_pdl(kern, dim3(p.splits, (p.heads + MT * 16 - 1) / (MT * 16), p.rows), dim3(warps * 32), smem, s, p);
   note_launch();
   return err == cudaSuccess ? 0 : -4;
 }
 
-template <typename T, int CW>
+constexpr int kLatMmaKeys = 1024;
+
+template <typename T, int CW, int NW>
 int launch_latent_mt(const LatentParams& p, cudaStream_t s) {
-  return p.heads > 16 ? launch_latent_cfg<T, CW, 2>(p, s) : launch_latent_cfg<T, CW, 1>(p, s);
+  return p.heads > 16 ? launch_latent_cfg<T, CW, 2, NW>(p, s) : launch_latent_cfg<T, CW, 1, NW>(p, s);
+}
+
+template <typename T>
+int launch_latent_mma(const LatentParams& p, cudaStream_t s) {
+  if (p.key <= 8 * 16) return launch_latent_mt<T, 16, 8>(p, s);
+  if (p.key <= 9 * 16) return launch_latent_mt<T, 16, 9>(p, s);
+  if (p.key <= 8 * 32) return launch_latent_mt<T, 32, 8>(p, s);
+  if (p.key <= 9 * 32) return launch_latent_mt<T, 32, 9>(p, s);
+  if (p.key <= 8 * 64) return launch_latent_mt<T, 64, 8>(p, s);
+  if (p.key <= 9 * 64) return launch_latent_mt<T, 64, 9>(p, s);
+  return launch_latent_mt<T, 128, 8>(p, s);
 }
 
 }  // namespace
 
-void launch_latent_prologue(const void* y, int64_t ld, int tokens, int q_rank, int kv_rank, const float* q_w, const float* kv_w,
-                            float eps, void* cq, const int64_t* loc, void* cache, int64_t cache_ld, int64_t num_slots, DType dt,
-                            int* status, cudaStream_t s) {
-  if (tokens == 0) return;
-  MB200_DISPATCH_FLOAT(dt, (launch_pdl(latent_prologue_kernel<T>, dim3(tokens, kv_rank > 0 ? 2 : 1), dim3(128), 0, s,
-                                       static_cast<const T*>(y), ld, q_rank, kv_rank, q_w, kv_w, eps, static_cast<T*>(cq), loc,
-                                       static_cast<T*>(cache), cache_ld, num_slots, status)));
+void launch_latent_prologue(const LatentPrologueArgs& p, cudaStream_t s) {
+  if (p.tokens == 0) return;
+  MB200_DISPATCH_FLOAT(p.dt, (launch_pdl(latent_prologue_kernel<T>, dim3(p.tokens, p.kv_rank > 0 ? 2 : 1), dim3(128), 0, s, p)));
+  note_launch();
+}
+
+void launch_turn_heads(const void* x, int64_t x_tok, int64_t x_head, const float2* turns, void* out, int64_t out_tok, int64_t out_head,
+                       int tokens, int heads, int rot, DType dt, cudaStream_t s) {
+  const int64_t pairs = static_cast<int64_t>(tokens) * heads * (rot / 2);
+  if (pairs == 0) return;
+  const int grid = static_cast<int>(std::min<int64_t>((pairs + 255) / 256, 148 * 32));
+  MB200_DISPATCH_FLOAT(dt, (launch_pdl(turn_heads_kernel<T>, dim3(grid), dim3(256), 0, s, static_cast<const T*>(x), x_tok, x_head, turns,
+                                       static_cast<T*>(out), out_tok, out_head, heads, rot / 2, pairs)));
+  note_launch();
+}
+
+void launch_gate_heads(const void* x, int64_t x_tok, int64_t x_head, const void* gate, int64_t gate_ld, void* out, int tokens, int heads,
+                       int width, DType dt, cudaStream_t s) {
+  if (tokens == 0 || width == 0) return;
+  const uintptr_t ptrs = reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(out);
+  auto go = [&](auto kernel, int v, const auto* xs, const auto* gs, auto* os) {
+    const int64_t total = static_cast<int64_t>(tokens) * heads * (width / v);
+    const int grid = static_cast<int>(std::min<int64_t>((total + 255) / 256, 148 * 32));
+    launch_pdl(kernel, dim3(grid), dim3(256), 0, s, xs, x_tok, x_head, gs, gate_ld, os, heads, width / v, total);
+  };
+  const bool vec = ptrs % 16 == 0 && width % 8 == 0 && x_tok % 8 == 0 && x_head % 8 == 0 && dt != kF32;
+  MB200_DISPATCH_FLOAT(dt, {
+    const T* xs = static_cast<const T*>(x);
+    const T* gs = static_cast<const T*>(gate);
+    T* os = static_cast<T*>(out);
+    if (vec) go(gate_heads_kernel<T, 8>, 8, xs, gs, os);
+    else go(gate_heads_kernel<T, 1>, 1, xs, gs, os);
+  });
   note_launch();
 }
 
@@ -591,19 +709,19 @@ void launch_latent_gather(const void* cache, int64_t cache_ld, int rank, int ele
   note_launch();
 }
 
-int launch_head_linear(const void* x, int64_t x_tok, int64_t x_head, const void* w, void* out, int64_t out_tok, int64_t out_head,
-                       int tokens, int heads, int N, int K, int num_sms, DType dt, cudaStream_t s) {
-  if (tokens == 0) return 0;
-  if (dt == kF32 || K % 8 != 0 || x_tok % 8 != 0 || x_head % 8 != 0) return -1;
-  const int groups = (tokens + kHlTokTiles * 8 - 1) / (kHlTokTiles * 8);
-  const bool split_k = static_cast<int64_t>(heads) * ((N + 63) / 64) * groups < num_sms && K >= 128;
-  MB200_DISPATCH_HALF(dt, {
-    if (split_k)
-      launch_pdl(head_linear_kernel<T, 4>, dim3((N + 15) / 16, heads, groups), dim3(128), 0, s, static_cast<const T*>(x), x_tok,
-                 x_head, static_cast<const T*>(w), static_cast<T*>(out), out_tok, out_head, tokens, N, K);
-    else
-      launch_pdl(head_linear_kernel<T, 1>, dim3((N + 63) / 64, heads, groups), dim3(128), 0, s, static_cast<const T*>(x), x_tok,
-                 x_head, static_cast<const T*>(w), static_cast<T*>(out), out_tok, out_head, tokens, N, K);
+int launch_head_linear(const HeadLinearArgs& a, int num_sms, cudaStream_t s) {
+  if (a.tokens == 0) return 0;
+  if (a.dt == kF32 || a.K % 8 != 0 || a.x_tok % 8 != 0 || a.x_head % 8 != 0) return -1;
+  const int groups = (a.tokens + kHlTokTiles * 8 - 1) / (kHlTokTiles * 8), extra = a.rot > 0 ? 1 : 0;
+  const bool split_k = static_cast<int64_t>(a.heads) * ((a.N + 63) / 64) * groups < num_sms && a.K >= 128;
+  MB200_DISPATCH_HALF(a.dt, {
+    auto go = [&](auto kernel, int tiles) {
+      launch_pdl(kernel, dim3(tiles + extra, a.heads, groups), dim3(128), 0, s, static_cast<const T*>(a.x), a.x_tok, a.x_head,
+                 static_cast<const T*>(a.w), static_cast<T*>(a.out), a.out_tok, a.out_head, a.tokens, a.N, a.K,
+                 static_cast<const T*>(a.gate), a.gate_ld, a.turns, a.rot);
+    };
+    if (split_k) go(head_linear_kernel<T, 4>, (a.N + 15) / 16);
+    else go(head_linear_kernel<T, 1>, (a.N + 63) / 64);
   });
   note_launch();
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
@@ -616,13 +734,13 @@ int latent_num_splits(int rows, int heads, int max_seq_len, int num_sms) {
   return std::max(1, std::min(splits, 64));
 }
 
-bool latent_mma_covers(int rank, int64_t cache_ld, DType dt) {
-  return dt != kF32 && rank % 8 == 0 && rank <= 1024 && cache_ld % 8 == 0;
+bool latent_mma_covers(int key, int rank, int64_t cache_ld, DType dt) {
+  return dt != kF32 && rank % 8 == 0 && key % 8 == 0 && key <= kLatMmaKeys && cache_ld % 8 == 0;
 }
 
 int launch_latent_attention(const LatentAttnArgs& a, cudaStream_t s) {
   if (a.rows == 0) return 0;
-  if (a.rank > kLatAnyThreads * kLatAnyCols || a.splits < 1) return -1;
+  if (a.rank > kLatAnyThreads * kLatAnyCols || a.key < a.rank || a.key > kLatAnyKeys || a.splits < 1) return -1;
   LatentParams p{};
   p.q = a.q;
   p.cache = a.cache;
@@ -639,20 +757,18 @@ int launch_latent_attention(const LatentAttnArgs& a, cudaStream_t s) {
   p.num_slots = a.num_slots;
   p.rows = a.rows;
   p.heads = a.heads;
+  p.key = a.key;
   p.rank = a.rank;
   p.splits = a.splits;
   p.scale = a.scale;
-  if (!latent_mma_covers(a.rank, a.cache_ld, a.dt)) {
+  if (!latent_mma_covers(a.key, a.rank, a.cache_ld, a.dt)) {
     if (a.splits != 1) return -1;
     MB200_DISPATCH_FLOAT(a.dt, (launch_pdl(latent_attn_any_kernel<T>, dim3(a.heads, a.rows), dim3(kLatAnyThreads), 0, s, p)));
     note_launch();
     return cudaGetLastError() == cudaSuccess ? 0 : -4;
   }
   int rc = 0;
-  MB200_DISPATCH_HALF(a.dt, (rc = a.rank <= 128   ? launch_latent_mt<T, 16>(p, s)
-                                  : a.rank <= 256 ? launch_latent_mt<T, 32>(p, s)
-                                  : a.rank <= 512 ? launch_latent_mt<T, 64>(p, s)
-                                                  : launch_latent_mt<T, 128>(p, s)));
+  MB200_DISPATCH_HALF(a.dt, (rc = launch_latent_mma<T>(p, s)));
   if (rc != 0) return rc;
   if (a.splits > 1) {
     MB200_DISPATCH_HALF(a.dt, (launch_pdl(latent_merge_kernel<T>, dim3(a.heads, a.rows), dim3(128), 0, s, p)));

@@ -14,6 +14,7 @@
 // Warp roles (256 threads): warp 0 TMA producer, warp 1 MMA issuer, warp 2 TMEM allocator,
 // warps 4-7 epilogue.  Every barrier wait is bounded (kStatusPipelineTimeout on expiry).
 #include <algorithm>
+#include <type_traits>
 
 #include "common.cuh"
 #include "kernels.h"
@@ -31,39 +32,76 @@ constexpr int kMaxExperts = 256;
 // --------------------------------------------------------------------------------------------
 // router: one warp per token
 // --------------------------------------------------------------------------------------------
-template <typename T, int NV>   // NV: logits per lane
-__global__ void moe_router_topk_kernel(const T* __restrict__ logits, int64_t stride, const float* __restrict__ correction,
-                                       float* __restrict__ w_out, int* __restrict__ id_out, int tokens, int experts, int top_k,
-                                       int renorm, float renorm_eps) {
+// larger two of two sorted pairs
+__device__ __forceinline__ float2 top_two(float2 a, float2 b) {
+  return make_float2(fmaxf(a.x, b.x), fmaxf(fminf(a.x, b.x), fmaxf(a.y, b.y)));
+}
+
+// NV: logits per lane; SIGMOID: scores are logistic functions of the logits instead of their softmax; GROUPS: only experts of
+// the p.keep best of p.groups (at most 32) runs of neighbours can be chosen, a run's score being the sum of its two largest keys
+template <typename T, int NV, bool SIGMOID, bool GROUPS>
+__global__ void moe_router_topk_kernel(const RouteArgs p) {
   pdl_wait();
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-  const int lane = threadIdx.x & 31;
-  if (t >= tokens) return;
-  const T* row = logits + static_cast<int64_t>(t) * stride;
+  const int lane = threadIdx.x & 31, experts = p.experts, top_k = p.top_k;
+  if (t >= p.tokens) return;
+  const T* row = static_cast<const T*>(p.logits) + static_cast<int64_t>(t) * p.stride;
   float v[NV];
-  float mx = -INFINITY;
+  if constexpr (SIGMOID) {
 #pragma unroll
-  for (int i = 0; i < NV; ++i) {
-    const int e = lane + 32 * i;
-    v[i] = e < experts ? to_f32(row[e]) : -INFINITY;
-    mx = fmaxf(mx, v[i]);
-  }
-  mx = warp_max(mx);
-  float sum = 0.f;
+    for (int i = 0; i < NV; ++i) v[i] = (lane + 32 * i) < experts ? 1.f / (1.f + expf(-to_f32(row[lane + 32 * i]))) : 0.f;
+  } else {
+    float mx = -INFINITY;
 #pragma unroll
-  for (int i = 0; i < NV; ++i) {
-    v[i] = (lane + 32 * i) < experts ? expf(v[i] - mx) : 0.f;
-    sum += v[i];
+    for (int i = 0; i < NV; ++i) {
+      const int e = lane + 32 * i;
+      v[i] = e < experts ? to_f32(row[e]) : -INFINITY;
+      mx = fmaxf(mx, v[i]);
+    }
+    mx = warp_max(mx);
+    float sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      v[i] = (lane + 32 * i) < experts ? expf(v[i] - mx) : 0.f;
+      sum += v[i];
+    }
+    sum = warp_sum(sum);
+    const float inv = 1.f / sum;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) v[i] *= inv;
   }
-  sum = warp_sum(sum);
-  const float inv = 1.f / sum;
   // the key that is compared: the score, plus the expert's correction; -inf where there is no expert or it is taken
   float key[NV];
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
     const int e = lane + 32 * i;
-    v[i] *= inv;
-    key[i] = e < experts ? v[i] + (correction != nullptr ? correction[e] : 0.f) : -INFINITY;
+    key[i] = e < experts ? v[i] + (p.correction != nullptr ? p.correction[e] : 0.f) : -INFINITY;
+  }
+  if constexpr (GROUPS) {
+    const int size = experts / p.groups;
+    int mine[NV];                 // the group of each of the lane's experts
+#pragma unroll
+    for (int i = 0; i < NV; ++i) mine[i] = (lane + 32 * i) / size;
+    float group_score = -INFINITY;        // lane g: the score of group g
+    for (int g = 0; g < p.groups; ++g) {
+      float2 two = make_float2(-INFINITY, -INFINITY);
+#pragma unroll
+      for (int i = 0; i < NV; ++i)
+        if (mine[i] == g) two = top_two(two, make_float2(key[i], -INFINITY));
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1)
+        two = top_two(two, make_float2(__shfl_xor_sync(0xffffffffu, two.x, o), __shfl_xor_sync(0xffffffffu, two.y, o)));
+      if (lane == g) group_score = size > 1 ? two.x + two.y : two.x;
+    }
+    int before = 0;                       // groups that come first: a larger score, or the same and a lower index
+    for (int g = 0; g < p.groups; ++g) {
+      const float other = __shfl_sync(0xffffffffu, group_score, g);
+      before += (other > group_score || (other == group_score && g < lane)) ? 1 : 0;
+    }
+    const unsigned open = __ballot_sync(0xffffffffu, lane < p.groups && before < p.keep);
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+      if ((lane + 32 * i) < experts && ((open >> mine[i]) & 1u) == 0) key[i] = -INFINITY;
   }
   float chosen_w = 0.f;  // lane j keeps the j-th choice
   int chosen_e = 0;
@@ -104,8 +142,8 @@ __global__ void moe_router_topk_kernel(const T* __restrict__ logits, int64_t str
     }
   }
   if (lane < top_k) {
-    w_out[static_cast<int64_t>(t) * top_k + lane] = renorm ? chosen_w / (ksum + renorm_eps) : chosen_w;
-    id_out[static_cast<int64_t>(t) * top_k + lane] = chosen_e;
+    p.w[static_cast<int64_t>(t) * top_k + lane] = (p.renorm ? chosen_w / (ksum + p.renorm_eps) : chosen_w) * p.scale;
+    p.ids[static_cast<int64_t>(t) * top_k + lane] = chosen_e;
   }
 }
 
@@ -616,23 +654,34 @@ int launch_grouped_cfg(const CUtensorMap& tw, const CUtensorMap& tx, const Group
 
 }  // namespace
 
-void launch_moe_router_topk(const void* logits, int64_t stride, const float* correction, float* w, int* ids, int tokens, int experts,
-                            int top_k, int renorm, float renorm_eps, DType dt, cudaStream_t s) {
-  if (tokens == 0) return;
+int launch_moe_router_topk(const RouteArgs& p, cudaStream_t s) {
+  if (p.tokens == 0) return 0;
+  const bool groups = p.groups > 1 && p.keep < p.groups;
+  if (p.experts > kMaxExperts || p.top_k > 32 || p.top_k > p.experts) return -1;
+  if (groups && (p.groups > 32 || p.experts % p.groups != 0 || p.keep < 1 || p.top_k > p.keep * (p.experts / p.groups))) return -1;
   const int warps = 8;
-  const dim3 grid((tokens + warps - 1) / warps), block(warps * 32);
-  auto go = [&](auto kernel, auto* typed) {
-    launch_pdl(kernel, grid, block, 0, s, typed, stride, correction, w, ids, tokens, experts, top_k, renorm, renorm_eps);
+  const dim3 grid((p.tokens + warps - 1) / warps), block(warps * 32);
+  auto go = [&](auto kernel) { launch_pdl(kernel, grid, block, 0, s, p); };
+  auto pick = [&](auto typed, auto nv) {
+    using T = decltype(typed);
+    constexpr int NV = decltype(nv)::value;
+    if (p.sigmoid) {
+      if (groups) go(moe_router_topk_kernel<T, NV, true, true>);
+      else go(moe_router_topk_kernel<T, NV, true, false>);
+    } else {
+      if (groups) go(moe_router_topk_kernel<T, NV, false, true>);
+      else go(moe_router_topk_kernel<T, NV, false, false>);
+    }
   };
-  MB200_DISPATCH_FLOAT(dt, {
-    const T* l = static_cast<const T*>(logits);
-    if (experts <= 32) go(moe_router_topk_kernel<T, 1>, l);
-    else if (experts <= 64) go(moe_router_topk_kernel<T, 2>, l);
-    else if (experts <= 96) go(moe_router_topk_kernel<T, 3>, l);
-    else if (experts <= 128) go(moe_router_topk_kernel<T, 4>, l);
-    else go(moe_router_topk_kernel<T, 8>, l);
+  MB200_DISPATCH_FLOAT(p.dt, {
+    if (p.experts <= 32) pick(T{}, std::integral_constant<int, 1>{});
+    else if (p.experts <= 64) pick(T{}, std::integral_constant<int, 2>{});
+    else if (p.experts <= 96) pick(T{}, std::integral_constant<int, 3>{});
+    else if (p.experts <= 128) pick(T{}, std::integral_constant<int, 4>{});
+    else pick(T{}, std::integral_constant<int, 8>{});
   });
   note_launch();
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
 int launch_moe_router_logits(const void* x, int64_t x_ld, const void* w, float* logits, int tokens, int experts, int hidden,

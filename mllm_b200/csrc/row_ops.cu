@@ -1,10 +1,11 @@
-// Row-wise kernels of decoders that keep their residual stream in fp32: the norm after the residual sum (with the
-// weighted sum of expert outputs folded in), the prologue of attention layers whose query / key norm spans all heads,
+// Row-wise kernels of decoders that keep their residual stream in fp32: the norm around the residual sum (with the
+// weighted sum of expert outputs folded in), prologues of attention layers (query / key norm over all heads or per head),
 // the norm of a whole row with a gate, and small element-wise operations.
 //
 // All are bound by memory traffic: a CTA takes one row, 8 or 16 bytes per thread and access, and keeps it in registers
 // between the reduction and the scaling pass.  Rows that no vector access fits (odd widths) take the V = 1 form.
 #include <algorithm>
+#include <type_traits>
 
 #include "common.cuh"
 #include "kernels.h"
@@ -48,22 +49,30 @@ __device__ __forceinline__ float2 block_sum2(float a, float b) {
 
 constexpr int kRowElems = 32;      // elements of a row a thread may hold
 constexpr int kMaxChoices = 32;    // experts a token may use
+// the norm on a sublayer's output holds the stream's elements beside them
+constexpr int row_elems(bool inner) { return inner ? kRowElems / 2 : kRowElems; }
 
-// threads for a row of `vecs` vectors of `v` elements: one each up to 256, then up to kRowElems elements each (0: the row
-// is too wide)
-inline int row_threads(int vecs, int v) {
-  const int most = kRowElems / v;
+// threads for a row of `vecs` vectors of `v` elements: one each up to 256, then up to `elems` elements each (0: the row is
+// too wide)
+inline int row_threads(int vecs, int v, int elems = kRowElems) {
+  const int most = elems / v;
   int t = std::min(256, (vecs + 31) / 32 * 32);
   while (t < 1024 && static_cast<int64_t>(t) * most < vecs) t *= 2;
   return static_cast<int64_t>(t) * most >= vecs ? t : 0;
 }
 
+// logistic function in full fp32
+__device__ __forceinline__ float sigmoid_f32(float v) { return 1.f / (1.f + expf(-v)); }
+
 // ---------------------------------------------------------------------------------------------
-// x <- rmsnorm(alpha * x + ls * y) * w with x in fp32; h = x in the activations' type.  MOE: y is the sum of the row of
-// `y` (a shared expert; may be null), the token's expert rows times their weights and, for choices that name an identity
-// expert, the token's own input times its weight.
+// The step behind a sublayer, x in fp32; h = the new x in the activations' type.
+//   INNER false: x <- rmsnorm(alpha * x + ls * y) * w      (the norm behind the sum)
+//   INNER true:  x <- alpha * x + ls * rmsnorm(y) * w      (the norm on the sublayer's output)
+// y_logit: a number per token; y is multiplied by its logistic function.  MOE: y is the sum of the row of `y` (a shared
+// expert; may be null), the token's expert rows times their weights and, for choices that name an identity expert, the
+// token's own input times its weight.
 // ---------------------------------------------------------------------------------------------
-template <typename T, int V, bool MOE>
+template <typename T, int V, bool MOE, bool INNER>
 __global__ void __launch_bounds__(1024) post_norm_kernel(const PostNormArgs p) {
   pdl_launch_dependents();
   pdl_wait();
@@ -92,8 +101,9 @@ __global__ void __launch_bounds__(1024) post_norm_kernel(const PostNormArgs p) {
   }
   const float* x = p.x + row * p.width;
   const T* y = p.y == nullptr ? nullptr : static_cast<const T*>(p.y) + row * p.width;
-  constexpr int kIts = kRowElems / V;
-  float z[kIts][V];
+  const float y_scale = p.y_logit == nullptr ? 1.f : sigmoid_f32(p.y_logit[row * p.y_logit_ld]);
+  constexpr int kIts = row_elems(INNER) / V;
+  float z[kIts][V], xr[INNER ? kIts : 1][V];
   float ss = 0.f;
 #pragma unroll
   for (int it = 0; it < kIts; ++it) {
@@ -103,7 +113,12 @@ __global__ void __launch_bounds__(1024) post_norm_kernel(const PostNormArgs p) {
       float acc[V], t[V];
 #pragma unroll
       for (int i = 0; i < V; ++i) acc[i] = 0.f;
-      if (y != nullptr) load_vec<T, V>(y + c, acc);
+      if constexpr (INNER) load_vec<float, V>(x + c, xr[it]);
+      if (y != nullptr) {
+        load_vec<T, V>(y + c, acc);
+#pragma unroll
+        for (int i = 0; i < V; ++i) acc[i] *= y_scale;
+      }
       if constexpr (MOE) {
         for (int j = 0; j < choices; j += 4) {
           float r[4][V];
@@ -117,17 +132,21 @@ __global__ void __launch_bounds__(1024) post_norm_kernel(const PostNormArgs p) {
           }
         }
       }
-      if (p.ls != nullptr) {
-        load_vec<float, V>(p.ls + c, t);
+      if constexpr (INNER) {
 #pragma unroll
-        for (int i = 0; i < V; ++i) acc[i] *= t[i];
-      }
-      load_vec<float, V>(x + c, t);
+        for (int i = 0; i < V; ++i) z[it][i] = acc[i];
+      } else {
+        if (p.ls != nullptr) {
+          load_vec<float, V>(p.ls + c, t);
 #pragma unroll
-      for (int i = 0; i < V; ++i) {
-        z[it][i] = fmaf(p.alpha, t[i], acc[i]);
-        ss = fmaf(z[it][i], z[it][i], ss);
+          for (int i = 0; i < V; ++i) acc[i] *= t[i];
+        }
+        load_vec<float, V>(x + c, t);
+#pragma unroll
+        for (int i = 0; i < V; ++i) z[it][i] = fmaf(p.alpha, t[i], acc[i]);
       }
+#pragma unroll
+      for (int i = 0; i < V; ++i) ss = fmaf(z[it][i], z[it][i], ss);
     }
   }
   const float rstd = 1.f / sqrtf(block_sum2(ss, 0.f).x / static_cast<float>(p.width) + p.eps);
@@ -140,6 +159,15 @@ __global__ void __launch_bounds__(1024) post_norm_kernel(const PostNormArgs p) {
       load_vec<float, V>(p.w + c, w);
 #pragma unroll
       for (int i = 0; i < V; ++i) z[it][i] *= rstd * w[i];
+      if constexpr (INNER) {
+        if (p.ls != nullptr) {
+          load_vec<float, V>(p.ls + c, w);
+#pragma unroll
+          for (int i = 0; i < V; ++i) z[it][i] *= w[i];
+        }
+#pragma unroll
+        for (int i = 0; i < V; ++i) z[it][i] = fmaf(p.alpha, xr[it][i], z[it][i]);
+      }
       if (p.x_out != nullptr) store_vec<float, V>(p.x_out + row * p.width + c, z[it]);
       store_vec<T, V>(static_cast<T*>(p.h) + row * p.width + c, z[it]);
     }
@@ -150,7 +178,7 @@ __global__ void __launch_bounds__(1024) post_norm_kernel(const PostNormArgs p) {
 template <typename T>
 __device__ __forceinline__ float sigmoid_for(float v) {
   if constexpr (sizeof(T) == 2) return __fdividef(1.f, 1.f + __expf(-v));
-  return 1.f / (1.f + expf(-v));
+  return sigmoid_f32(v);
 }
 
 // out = x * rsqrt(mean(x^2) + eps) * w * sigmoid(gate), the mean over the whole row
@@ -280,6 +308,105 @@ __global__ void __launch_bounds__(512) rownorm_rope_kv_kernel(const RowNormRopeA
   }
 }
 
+// ---------------------------------------------------------------------------------------------
+// Attention prologue with a norm per head: row = [q: heads x dim | k: kv_heads x dim | ..] of a token, values of kv_heads x
+// vdim at column v_at (the keys themselves where v_at = heads * dim).  Query and key heads are turned on their first
+// rot_dims features (halves: feature i with i + rot_dims / 2, else neighbours) and divided by their root mean square, which
+// turning does not change; values are cached as they came.  Groups of G lanes take a head each, U features per access.
+// ---------------------------------------------------------------------------------------------
+template <typename T, int U, bool HALVES>
+__global__ void __launch_bounds__(512) headnorm_rope_kv_kernel(const HeadNormRopeArgs p, int G) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ float2 s_rot[];       // [rot_dims / 2] cosine, sine
+  const int64_t t = blockIdx.x;
+  const int tid = threadIdx.x, nt = blockDim.x, half = p.rot_dims / 2;
+  const T* row = static_cast<const T*>(p.row) + t * p.row_ld;
+  const int64_t slot = p.loc[t];
+  const bool slot_ok = slot >= 0 && slot < p.num_slots;
+  if (!slot_ok && tid == 0 && p.status != nullptr) atomicExch(p.status, kStatusBadIndex);
+  const double pos = static_cast<double>(p.positions[t]);
+  for (int i = tid; i < half; i += nt) {
+    constexpr double kTurn = 6.283185307179586476925286766559;
+    double a = pos * p.inv_freq[i];
+    a -= kTurn * rint(a / kTurn);
+    float s, c;
+    sincosf(static_cast<float>(a), &s, &c);
+    s_rot[i] = make_float2(c, s);
+  }
+  if (slot_ok) {
+    for (int u = tid; u < p.kv_heads * p.vdim / U; u += nt) {
+      const int e = u * U, head = e / p.vdim, d = e - head * p.vdim;
+      float f[U];
+      load_vec<T, U>(row + p.v_at + e, f);
+      store_vec<T, U>(static_cast<T*>(p.v_cache) + slot * p.v_tok_stride + head * p.v_head_stride + d, f);
+    }
+  }
+  __syncthreads();
+  const int units = p.dim / U, all = p.heads + p.kv_heads, lane = tid % G, groups = nt / G;
+  const int rounds = (all + groups - 1) / groups;
+  for (int r = 0; r < rounds; ++r) {
+    const int h = r * groups + tid / G;
+    const bool on = h < all, is_q = h < p.heads;
+    const T* src = row + (on ? h : 0) * p.dim;       // key heads follow the query heads
+    float ss = 0.f;
+    for (int u = lane; u < units; u += G) {
+      float f[U];
+      load_vec<T, U>(src + u * U, f);
+#pragma unroll
+      for (int i = 0; i < U; ++i) ss = fmaf(f[i], f[i], ss);
+    }
+    for (int o = G / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (!on) continue;                               // no shuffle follows in this round
+    const float rstd = 1.f / sqrtf(ss / static_cast<float>(p.dim) + p.eps);
+    T* dst = nullptr;
+    if (is_q) dst = static_cast<T*>(p.q_out) + (t * p.heads + h) * p.q_width;
+    else if (slot_ok) dst = static_cast<T*>(p.k_cache) + slot * p.k_tok_stride + (h - p.heads) * p.k_head_stride;
+    if (dst != nullptr) {
+      for (int u = lane; u < units; u += G) {
+        const int d = u * U;
+        float f[U];
+        load_vec<T, U>(src + d, f);
+        if (d < p.rot_dims) {
+          if constexpr (HALVES) {
+            const bool low = d < half;               // U divides half: a unit lies on one side
+            float o[U];
+            load_vec<T, U>(src + (low ? d + half : d - half), o);
+#pragma unroll
+            for (int i = 0; i < U; ++i) {
+              const float2 cs = s_rot[(low ? d : d - half) + i];
+              f[i] = low ? f[i] * cs.x - o[i] * cs.y : f[i] * cs.x + o[i] * cs.y;
+            }
+          } else if constexpr (U == 1) {
+            const float other = to_f32(src[d ^ 1]);
+            const float2 cs = s_rot[d >> 1];
+            f[0] = (d & 1) ? f[0] * cs.x + other * cs.y : f[0] * cs.x - other * cs.y;
+          } else {
+#pragma unroll
+            for (int i = 0; i < U; i += 2) {
+              if (d + i < p.rot_dims) {
+                const float2 cs = s_rot[(d + i) >> 1];
+                const float a = f[i], b = f[i + 1];
+                f[i] = a * cs.x - b * cs.y;
+                f[i + 1] = b * cs.x + a * cs.y;
+              }
+            }
+          }
+        }
+#pragma unroll
+        for (int i = 0; i < U; ++i) f[i] *= rstd;
+        store_vec<T, U>(dst + d, f);
+      }
+    }
+    if (is_q) {
+      float zero[U];
+#pragma unroll
+      for (int i = 0; i < U; ++i) zero[i] = 0.f;
+      for (int d = p.dim + lane * U; d < p.q_width; d += G * U) store_vec<T, U>(dst + d, zero);
+    }
+  }
+}
+
 // out = cap * tanh(x / cap) in fp32; a CTA walks V neighbouring features at a time of one row
 template <typename T, int V>
 __global__ void soft_cap_kernel(const T* __restrict__ x, int64_t x_ld, float* __restrict__ out, int width, float cap) {
@@ -316,14 +443,14 @@ __global__ void relu_squared_kernel(T* __restrict__ x, int64_t vecs) {
 
 inline bool aligned(const void* p, uintptr_t n) { return (reinterpret_cast<uintptr_t>(p) & (n - 1)) == 0; }
 
-template <typename T, int V>
+template <typename T, int V, bool INNER>
 int launch_post_norm_v(const PostNormArgs& p, cudaStream_t s) {
-  const int threads = row_threads(p.width / V, V);
+  const int threads = row_threads(p.width / V, V, row_elems(INNER));
   if (threads == 0) return -1;
   if (p.expert_rows != nullptr)
-    launch_pdl(post_norm_kernel<T, V, true>, dim3(p.rows), dim3(threads), 0, s, p);
+    launch_pdl(post_norm_kernel<T, V, true, INNER>, dim3(p.rows), dim3(threads), 0, s, p);
   else
-    launch_pdl(post_norm_kernel<T, V, false>, dim3(p.rows), dim3(threads), 0, s, p);
+    launch_pdl(post_norm_kernel<T, V, false, INNER>, dim3(p.rows), dim3(threads), 0, s, p);
   note_launch();
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
@@ -358,6 +485,28 @@ int launch_rownorm_rope_t(const RowNormRopeArgs& p, cudaStream_t s) {
   return go(rownorm_rope_kv_kernel<T, 1>);
 }
 
+template <typename T, bool HALVES>
+int launch_headnorm_rope_t(const HeadNormRopeArgs& p, cudaStream_t s) {
+  const uintptr_t ptrs = reinterpret_cast<uintptr_t>(p.row) | reinterpret_cast<uintptr_t>(p.q_out) | reinterpret_cast<uintptr_t>(p.k_cache) |
+                         reinterpret_cast<uintptr_t>(p.v_cache);
+  int64_t sizes = p.dim | p.vdim | p.v_at | p.q_width | p.row_ld | p.k_tok_stride | p.k_head_stride | p.v_tok_stride | p.v_head_stride;
+  if (HALVES) sizes |= p.rot_dims / 2;               // a unit must not cross the middle or the end of the turned features
+  const size_t smem = static_cast<size_t>(p.rot_dims / 2) * sizeof(float2) + 8;
+  auto go = [&](auto kernel, int unit) {
+    int G = 1;
+    while (G < 32 && G * unit < p.dim) G *= 2;
+    // decode batches: a group of lanes per head; long runs: small CTAs, many of them
+    const int want = (p.heads + p.kv_heads) * G;
+    const int threads = p.tokens >= 1024 ? 128 : std::min(512, std::max(64, (want + 31) / 32 * 32));
+    launch_pdl(kernel, dim3(p.tokens), dim3(threads), smem, s, p, G);
+    note_launch();
+    return cudaGetLastError() == cudaSuccess ? 0 : -4;
+  };
+  if (sizes % 8 == 0 && ptrs % 16 == 0 && sizeof(T) == 2) return go(headnorm_rope_kv_kernel<T, 8, HALVES>, 8);
+  if (sizes % 2 == 0 && ptrs % 8 == 0) return go(headnorm_rope_kv_kernel<T, 2, HALVES>, 2);
+  return go(headnorm_rope_kv_kernel<T, 1, HALVES>, 1);
+}
+
 }  // namespace
 
 int launch_post_norm(const PostNormArgs& p, cudaStream_t s) {
@@ -368,11 +517,16 @@ int launch_post_norm(const PostNormArgs& p, cudaStream_t s) {
                          reinterpret_cast<uintptr_t>(p.expert_rows) | reinterpret_cast<uintptr_t>(p.token_in);
   const bool vec = p.width % 4 == 0 && ptrs % 16 == 0, wide = p.width % 8 == 0 && ptrs % 32 == 0 && p.dt != kF32;
   int rc = 0;
-  if (wide) {
-    MB200_DISPATCH_HALF(p.dt, rc = (launch_post_norm_v<T, 8>(p, s)));
-  } else {
-    MB200_DISPATCH_FLOAT(p.dt, rc = vec ? launch_post_norm_v<T, 4>(p, s) : launch_post_norm_v<T, 1>(p, s));
-  }
+  auto go = [&](auto inner) {
+    constexpr bool kInner = decltype(inner)::value;
+    if (wide) {
+      MB200_DISPATCH_HALF(p.dt, rc = (launch_post_norm_v<T, 8, kInner>(p, s)));
+    } else {
+      MB200_DISPATCH_FLOAT(p.dt, rc = vec ? (launch_post_norm_v<T, 4, kInner>(p, s)) : (launch_post_norm_v<T, 1, kInner>(p, s)));
+    }
+  };
+  if (p.inner) go(std::true_type{});
+  else go(std::false_type{});
   return rc;
 }
 
@@ -397,6 +551,14 @@ int launch_rownorm_rope_kv(const RowNormRopeArgs& p, cudaStream_t s) {
   if (p.rot_dims % 2 != 0 || p.rot_dims > p.dim || p.rot_dims > 4096 || p.q_width < p.dim) return -1;
   int rc = 0;
   MB200_DISPATCH_FLOAT(p.dt, rc = launch_rownorm_rope_t<T>(p, s));
+  return rc;
+}
+
+int launch_headnorm_rope_kv(const HeadNormRopeArgs& p, cudaStream_t s) {
+  if (p.tokens <= 0) return 0;
+  if (p.rot_dims % 2 != 0 || p.rot_dims > p.dim || p.rot_dims > 4096 || p.q_width < p.dim) return -1;
+  int rc = 0;
+  MB200_DISPATCH_FLOAT(p.dt, rc = p.halves ? (launch_headnorm_rope_t<T, true>(p, s)) : (launch_headnorm_rope_t<T, false>(p, s)));
   return rc;
 }
 

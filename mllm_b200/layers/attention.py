@@ -8,6 +8,7 @@ the request->slot table directly, so there is no per-step planning or index flat
 
 from __future__ import annotations
 
+import math
 from typing import Optional
 
 import torch
@@ -80,32 +81,44 @@ def query_rows(fb):
     return got
 
 
-class RowNormAttention(nn.Module):
+def rotation_frequencies(dims: int, base: float, scaling: Optional[dict] = None) -> torch.Tensor:
+    """One fp64 frequency per rotated pair, ``base^(-2i / dims)``.  ``scaling`` (factor, low, high, original): frequencies
+    whose wave is longer than ``original / low`` are divided by ``factor``, waves shorter than ``original / high`` stay, with
+    a linear blend (in original / wave) between."""
+    i = torch.arange(dims // 2, dtype=torch.float64)
+    f = torch.pow(torch.tensor(base, dtype=torch.float64), -2.0 * i / max(1, dims))
+    if scaling:
+        factor, lo, hi, old = (float(scaling[k]) for k in ("factor", "low", "high", "original"))
+        turns = old * f / (2.0 * math.pi)                   # over the original length: original / wavelength
+        keep = torch.where(turns > hi, 1.0, torch.where(turns < lo, 0.0, (turns - lo) / (hi - lo)))
+        f = (1.0 - keep) * f / factor + keep * f
+    return f
+
+
+class SizedAttention(nn.Module):
     """Causal attention core for layers that give their own sizes: grouped query heads, keys of ``dim`` and values of
-    ``vdim`` features, a query / key norm that spans all heads of the row, rotation of neighbouring features on the
-    first ``rot_dims`` of each head, any score scale, an optional sliding window.  It reads the projected rows
-    ``[q | k | v]`` and writes the concatenated heads; projections belong to the mixer around it.
+    ``vdim`` features, rotation of part of each head, any score scale, an optional sliding window, an optional sink per
+    head.  It reads the projected rows that ``shards`` names and writes the concatenated heads; projections belong to the
+    mixer around it.  Subclasses have the prologue (:meth:`prepare`): norms, rotation, cache write.
 
     16-bit runs use the attention kernels of the other models, with heads zero-padded to 64 / 128 / 256 features in the
     cache and in the rows that leave (``width``); fp32 runs and wider heads take the row kernel, unpadded."""
 
     folds_scale = False       # the output is linear in V only: a scale on it belongs to what follows
+    biased: tuple = ()
 
     def __init__(self, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, eps: float, kv_index: int, rot_dims: int = 0,
-                 rot_base: float = 1e4, window: Optional[int] = None, dtype: torch.dtype = torch.bfloat16, biased: bool = True) -> None:
+                 rot_base: float = 1e4, rot_scaling: Optional[dict] = None, window: Optional[int] = None,
+                 dtype: torch.dtype = torch.bfloat16) -> None:
         super().__init__()
         if heads % kv_heads or rot_dims % 2 or rot_dims > dim:
             raise ValueError(f"attention: {heads} heads over {kv_heads}, {rot_dims} of {dim} features rotated")
         self.heads, self.kv_heads, self.dim, self.vdim = heads, kv_heads, dim, vdim
         self.scale, self.eps, self.kv_index, self.window = float(scale), float(eps), kv_index, window
-        self.rot_dims, self.rot_base = rot_dims, float(rot_base)
-        self.shards = {"q": heads * dim, "k": kv_heads * dim, "v": kv_heads * vdim}
-        self.biased = tuple(self.shards) if biased else ()
+        self.rot_dims, self.rot_base, self.rot_scaling = rot_dims, float(rot_base), rot_scaling
         self.width = None if dtype == torch.float32 or heads // kv_heads > 128 else next(
             (w for w in (64, 128, 256) if w >= max(dim, vdim) and ops.attention_kernels_cover(w, dtype, dtype)), None)
-        self.q_norm, self.k_norm = nn.Module(), nn.Module()
-        self.q_norm.weight = nn.Parameter(torch.ones(heads * dim, dtype=torch.float32), requires_grad=False)
-        self.k_norm.weight = nn.Parameter(torch.ones(kv_heads * dim, dtype=torch.float32), requires_grad=False)
+        self.register_parameter("sink", None)
         self._inv_freq: Optional[torch.Tensor] = None
 
     @property
@@ -126,27 +139,71 @@ class RowNormAttention(nn.Module):
         return out.view(w.shape[0], -1)
 
     def inv_freq(self, device) -> torch.Tensor:
-        """One fp64 frequency per rotated pair: ``rot_base^(-2i / rot_dims)``."""
         if self._inv_freq is None or self._inv_freq.device != device:
-            i = torch.arange(self.rot_dims // 2, dtype=torch.float64)
-            self._inv_freq = torch.pow(torch.tensor(self.rot_base, dtype=torch.float64), -2.0 * i / max(1, self.rot_dims)).to(device)
+            self._inv_freq = rotation_frequencies(self.rot_dims, self.rot_base, self.rot_scaling).to(device)
         return self._inv_freq
 
+    def prepare(self, row: torch.Tensor, fb, q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor) -> None:
+        """Queries of ``row`` into ``q`` [T, heads, key width], keys and values into the cache slots of the batch."""
+        raise NotImplementedError
+
     def forward(self, row: torch.Tensor, fb, out: torch.Tensor) -> None:
-        """``row`` [T, >= q | k | v], ``out`` [T, out_width] (a column slice of a wider matrix will do)."""
+        """``row`` [T, >= the shards], ``out`` [T, out_width] (a column slice of a wider matrix will do)."""
         T = row.shape[0]
         kw, vw = self.kv_shape[1:]
         k_cache, v_cache = fb.token_to_kv_pool.get_kv_buffer(self.kv_index)
         rtt = fb.req_to_token_pool.req_to_token
         q = torch.empty((T, self.heads, kw), dtype=row.dtype, device=row.device)
-        ops.rownorm_rope_kv(row, self.q_norm.weight, self.k_norm.weight, self.inv_freq(row.device), fb.positions, fb.out_cache_loc, q,
-                            k_cache, v_cache, self.heads, self.kv_heads, self.dim, self.vdim, self.eps)
+        self.prepare(row, fb, q, k_cache, v_cache)
         o = out.unflatten(1, (self.heads, vw))
         if self.width is None or not row.is_cuda:
-            ops.attention_rows(q, k_cache, v_cache, rtt, *query_rows(fb), self.scale, o, window=self.window)
+            ops.attention_rows(q, k_cache, v_cache, rtt, *query_rows(fb), self.scale, o, window=self.window, sink=self.sink)
         elif fb.forward_mode.is_decode():
             ops.attention_decode(q, k_cache, v_cache, rtt, fb.req_pool_indices, fb.seq_lens, self.scale, out=o, max_seq_len=fb.max_seq_len,
-                                 window=self.window)
+                                 window=self.window, sink=self.sink)
         else:
             ops.attention_prefill(q, k_cache, v_cache, rtt, fb.req_pool_indices, fb.seq_lens, fb.extend_prefix_lens, fb.extend_start_loc,
-                                  self.scale, out=o, max_q_len=fb.max_extend_len, window=self.window)
+                                  self.scale, out=o, max_q_len=fb.max_extend_len, window=self.window, sink=self.sink)
+
+
+class RowNormAttention(SizedAttention):
+    """With a query / key norm that spans all heads of the row, then rotation of neighbouring features; rows are
+    ``[q | k | v]``."""
+
+    def __init__(self, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, eps: float, kv_index: int, rot_dims: int = 0,
+                 rot_base: float = 1e4, window: Optional[int] = None, dtype: torch.dtype = torch.bfloat16, biased: bool = True) -> None:
+        super().__init__(heads, kv_heads, dim, vdim, scale, eps, kv_index, rot_dims, rot_base, None, window, dtype)
+        self.shards = {"q": heads * dim, "k": kv_heads * dim, "v": kv_heads * vdim}
+        self.biased = tuple(self.shards) if biased else ()
+        self.q_norm, self.k_norm = nn.Module(), nn.Module()
+        self.q_norm.weight = nn.Parameter(torch.ones(heads * dim, dtype=torch.float32), requires_grad=False)
+        self.k_norm.weight = nn.Parameter(torch.ones(kv_heads * dim, dtype=torch.float32), requires_grad=False)
+
+    def prepare(self, row, fb, q, k_cache, v_cache) -> None:
+        ops.rownorm_rope_kv(row, self.q_norm.weight, self.k_norm.weight, self.inv_freq(row.device), fb.positions, fb.out_cache_loc, q,
+                            k_cache, v_cache, self.heads, self.kv_heads, self.dim, self.vdim, self.eps)
+
+
+class HeadNormAttention(SizedAttention):
+    """Query and key heads turn (``halves``: feature i with the one half the rotated features on, else neighbours) and are
+    then divided by their root mean square.  Rows are ``[q | k | v]``, or ``[q | k]`` with ``tied``: the values are the keys
+    as projected.  ``sinks``: a logit per head that joins the softmax denominator only."""
+
+    def __init__(self, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, eps: float, kv_index: int, rot_dims: int = 0,
+                 rot_base: float = 1e4, rot_scaling: Optional[dict] = None, halves: bool = True, tied: bool = False, sinks: bool = False,
+                 window: Optional[int] = None, dtype: torch.dtype = torch.bfloat16) -> None:
+        super().__init__(heads, kv_heads, dim, vdim, scale, eps, kv_index, rot_dims, rot_base, rot_scaling, window, dtype)
+        if tied and vdim != dim:
+            raise ValueError(f"attention: values that are the keys have {dim} features, not {vdim}")
+        self.halves, self.tied = halves, tied
+        self.shards = {"q": heads * dim, "k": kv_heads * dim}
+        self.v_at = heads * dim
+        if not tied:
+            self.v_at += kv_heads * dim
+            self.shards["v"] = kv_heads * vdim
+        if sinks:
+            self.sink = nn.Parameter(torch.zeros(heads, dtype=torch.float32), requires_grad=False)
+
+    def prepare(self, row, fb, q, k_cache, v_cache) -> None:
+        ops.headnorm_rope_kv(row, self.inv_freq(row.device), fb.positions, fb.out_cache_loc, q, k_cache, v_cache, self.heads, self.kv_heads,
+                             self.dim, self.vdim, self.v_at, self.halves, self.eps)

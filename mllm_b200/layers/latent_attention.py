@@ -1,14 +1,18 @@
-"""Latent attention without positions: the cache holds one row ``c`` of ``kv_rank`` features per token, shared by all
-heads; head ``h``'s key and value of a token are ``W_uk[h] c`` and ``W_uv[h] c``.  Queries go through a latent of their
-own.  Each head has a sink, a logit that joins the softmax denominator only.  A layer may read the latents of an
-earlier layer instead of writing its own.
+"""Latent attention: the cache holds one row ``c`` of ``kv_rank`` features per token, shared by all heads; head ``h``'s
+key and value of a token are ``W_uk[h] c`` and ``W_uv[h] c``.  Queries go through a latent of their own.  Options: a
+rotated key part of ``rot_dim`` features, shared by all heads, which follows the latent in the cache row and meets a
+rotated part of each query head (without it there are no positions); a sink per head, a logit that joins the softmax
+denominator only; a gate per head on the output.  A layer may read the latents of an earlier layer instead of writing its
+own.
 
 Two evaluations of the same sum (``csrc/latent.cu``):
 
-* absorbed: ``q' = W_uk[h]^T q`` meets the cached rows directly and the weighted sum of rows passes through ``W_uv[h]``
-  once per query — decode, short extends, 32-bit runs and head sizes the attention kernels do not have;
+* absorbed: ``q' = W_uk[h]^T q``, followed by the rotated query part, meets the cached rows directly and the weighted sum
+  of latents passes through ``W_uv[h]`` once per query — decode, short extends, 32-bit runs and head sizes the attention
+  kernels do not have;
 * expanded: requests with many new tokens form K and V of their context with two matrix products and run the
-  attention kernels of the other models on them.  Heads are zero-padded (in the weights) to 64 / 128 / 256 features.
+  attention kernels of the other models on them.  Heads are zero-padded (in the weights) to 64 / 128 / 256 features; the
+  shared key part reaches the heads through rows of the identity in the weights that form K, which copy it exactly.
 
 A batch may need both: :func:`latent_plan` sorts the requests once per forward pass."""
 
@@ -21,6 +25,7 @@ import torch
 from torch import nn
 
 from .. import ops
+from .attention import rotation_frequencies
 
 EXPAND_MIN_TOKENS = 32          # new tokens from which forming K and V of the context pays
 EXPAND_MAX_CONTEXT = 1 << 16    # context tokens expanded at a time (bounds the K and V buffers)
@@ -132,12 +137,15 @@ def _pad_heads(w: torch.Tensor, heads: int, width: int) -> torch.Tensor:
 
 class LatentAttention(nn.Module):
     def __init__(self, hidden_size: int, heads: int, dim: int, vdim: int, q_rank: int, kv_rank: int, scale: float, eps: float,
-                 latent_index: int, writes_latent: bool, params_dtype: torch.dtype) -> None:
+                 latent_index: int, writes_latent: bool, params_dtype: torch.dtype, rot_dim: int = 0, rot_base: float = 1e4,
+                 rot_scaling: Optional[dict] = None, sinks: bool = True, gated: bool = False) -> None:
         """``latent_index``: the buffer of the latent pool this layer reads; ``writes_latent``: whether the layer has a
         down projection of its own and fills it."""
         super().__init__()
         self.heads, self.dim, self.vdim, self.q_rank, self.kv_rank = heads, dim, vdim, q_rank, kv_rank
         self.scale, self.eps, self.latent_index, self.writes_latent = float(scale), eps, latent_index, writes_latent
+        self.rot_dim, self.rot_base, self.rot_scaling, self.gated = rot_dim, float(rot_base), rot_scaling, gated
+        self._inv_freq: Optional[torch.Tensor] = None
 
         def p(*shape, dtype=params_dtype):
             return nn.Parameter(torch.zeros(*shape, dtype=dtype), requires_grad=False)
@@ -147,44 +155,68 @@ class LatentAttention(nn.Module):
             m.weight = p(o, i)
             return m
 
-        rows = q_rank + (kv_rank if writes_latent else 0)
-        self.down_proj = lin(-(-rows // 8) * 8, hidden_size)       # [query latent | cache latent | zero rows]
+        # rows of the down projection: query latent, cache latent with the shared key part, gates; zero rows to a multiple of 8
+        self.down_at, rows = {}, 0
+        for name, n in (("q", q_rank), ("kv", kv_rank + rot_dim if writes_latent else 0), ("g", heads if gated else 0)):
+            self.down_at[name] = slice(rows, rows + n)
+            rows += n
+        self.down_proj = lin(-(-rows // 8) * 8, hidden_size)
         self.q_latent_norm = nn.Module()
         self.q_latent_norm.weight = nn.Parameter(torch.ones(q_rank, dtype=torch.float32), requires_grad=False)
         if writes_latent:
             self.kv_latent_norm = nn.Module()
             self.kv_latent_norm.weight = nn.Parameter(torch.ones(kv_rank, dtype=torch.float32), requires_grad=False)
-        self.q_up = lin(heads * dim, q_rank)
+        self.q_up = lin(heads * (dim + rot_dim), q_rank)        # per head [dim | rot_dim]
         self.k_up = lin(heads * dim, kv_rank)
         self.v_up = lin(heads * vdim, kv_rank)
-        self.sink = p(heads, dtype=torch.float32)
+        self.sink = p(heads, dtype=torch.float32) if sinks else None
         self.o_proj = lin(hidden_size, heads * vdim)
-        width = max(dim, vdim)
+        width = max(dim + rot_dim, vdim)
         self.pad = next((w for w in (64, 128, 256) if width <= w), None)   # head size of the expanded form
 
+    @property
+    def cache_width(self) -> int:
+        """Features of a cache row."""
+        return self.kv_rank + self.rot_dim
+
     def load_down(self, name: str, full: torch.Tensor) -> None:
-        o = 0 if name == "q" else self.q_rank
-        self.down_proj.weight.data[o:o + full.shape[0]].copy_(full)
+        """``name``: q (query latent), kv (cache latent and shared key part) or g (gates)."""
+        rows = self.down_proj.weight.data[self.down_at[name]]
+        if rows.shape != full.shape:
+            raise ValueError(f"a tensor of shape {tuple(full.shape)} does not fit {tuple(rows.shape)}")
+        rows.copy_(full)
 
     def post_load(self) -> None:
         """Weights in the layouts of the two forms: per head and K-major for the absorbed products, heads padded to the
         attention kernels' size for the expanded ones."""
-        H = self.heads
+        H, R = self.heads, self.rot_dim
 
         def keep(t):
             return nn.Parameter(t.contiguous(), requires_grad=False)
 
-        self._uk_t = keep(self.k_up.weight.data.view(H, self.dim, self.kv_rank).transpose(1, 2))      # [H, rank, dim]
+        k_up = self.k_up.weight.data.view(H, self.dim, self.kv_rank)
+        self._uk_t = keep(k_up.transpose(1, 2))                                                       # [H, rank, dim]
         self._uv = self.v_up.weight.data.view(H, self.vdim, self.kv_rank)                             # [H, vdim, rank]
         if self.pad is not None and self.expandable(self.q_up.weight):
+            v_up = self._uv
+            if R:       # products with whole cache rows: the shared key part is copied into K and left out of V
+                wide = k_up.new_zeros(H, self.dim + R, self.cache_width)
+                wide[:, : self.dim, : self.kv_rank] = k_up
+                wide[:, self.dim:, self.kv_rank:] = torch.eye(R, dtype=wide.dtype, device=wide.device)
+                k_up, v_up = wide, torch.cat([v_up, v_up.new_zeros(H, self.vdim, R)], -1)
             self._uq_pad = keep(_pad_heads(self.q_up.weight.data, H, self.pad))
-            self._uk_pad = keep(_pad_heads(self.k_up.weight.data, H, self.pad))
-            self._uv_pad = keep(_pad_heads(self.v_up.weight.data, H, self.pad))
+            self._uk_pad = keep(_pad_heads(k_up.reshape(-1, self.cache_width), H, self.pad))
+            self._uv_pad = keep(_pad_heads(v_up.reshape(-1, self.cache_width), H, self.pad))
 
     def expandable(self, like: torch.Tensor) -> bool:
         """The expanded form needs the 16-bit attention kernels on a GPU; on the CPU it runs in any type."""
         return self.pad is not None and (not like.is_cuda or ops.attention_kernels_cover(self.pad, like.dtype, like.dtype)
                                          and like.dtype != torch.float32)
+
+    def inv_freq(self, device) -> Optional[torch.Tensor]:
+        if self.rot_dim and (self._inv_freq is None or self._inv_freq.device != device):
+            self._inv_freq = rotation_frequencies(self.rot_dim, self.rot_base, self.rot_scaling).to(device)
+        return self._inv_freq
 
     def forward(self, x: torch.Tensor, fb) -> torch.Tensor:
         T, H = x.shape[0], self.heads
@@ -192,27 +224,33 @@ class LatentAttention(nn.Module):
         rtt = fb.req_to_token_pool.req_to_token
         plan = latent_plan(fb, self.expandable(x))
         y = ops.linear(x, self.down_proj.weight)
-        cq = ops.latent_prologue(y, self.q_latent_norm.weight, self.kv_latent_norm.weight if self.writes_latent else None,
-                                 self.eps, fb.out_cache_loc, cache if self.writes_latent else None)
+        cq, turns = ops.latent_prologue(y, self.q_latent_norm.weight, self.kv_latent_norm.weight if self.writes_latent else None,
+                                        self.eps, fb.out_cache_loc, cache if self.writes_latent else None, fb.positions,
+                                        self.inv_freq(x.device))
+        gate = y[:, self.down_at["g"]] if self.gated else None
         o = None
         if plan.groups:
-            o = self._expanded(cq, cache, rtt, plan)
+            o = self._expanded(cq, cache, rtt, plan, turns, gate)
         if plan.row_req is not None:
-            c = cq if plan.rows is None else cq.index_select(0, plan.rows)
-            q = ops.linear(c, self.q_up.weight).view(-1, H, self.dim)
-            q = ops.head_linear(q, self._uk_t)
-            u = ops.latent_attention(q, cache, rtt, plan.row_req, plan.row_pos, self.scale, self.sink, plan.max_ctx)
-            u = ops.head_linear(u, self._uv)
+            def near(t):
+                return t if plan.rows is None or t is None else t.index_select(0, plan.rows)
+
+            q = ops.linear(near(cq), self.q_up.weight).view(-1, H, self.dim + self.rot_dim)
+            q = ops.head_linear(q, self._uk_t, turns=near(turns))
+            u = ops.latent_attention(q, cache, rtt, plan.row_req, plan.row_pos, self.scale, self.sink, plan.max_ctx, self.kv_rank)
+            u = ops.head_linear(u, self._uv, gate=near(gate))
             if plan.rows is None:
                 o = u
             else:
                 o.index_copy_(0, plan.rows, u)
         return ops.linear(o.reshape(T, H * self.vdim), self.o_proj.weight)
 
-    def _expanded(self, cq, cache, rtt, plan: LatentPlan) -> torch.Tensor:
+    def _expanded(self, cq, cache, rtt, plan: LatentPlan, turns, gate) -> torch.Tensor:
         """Attention of the plan's expanded requests: [T, H, vdim], rows of other requests left unset."""
         H, W = self.heads, self.pad
         q = ops.linear(cq, self._uq_pad).view(-1, H, W)
+        if turns is not None:
+            ops.turn_heads(q[..., self.dim: self.dim + self.rot_dim], turns)
         out = torch.empty_like(q)
         for g in plan.groups:
             c = ops.latent_gather(cache, rtt, g.req, g.seq_lens, g.ctx_start, g.total, g.max_ctx)
@@ -220,4 +258,5 @@ class LatentAttention(nn.Module):
             v = ops.linear(c, self._uv_pad).view(-1, H, W)
             ops.attention_prefill(q, k, v, g.rows, g.batch, g.seq_lens, g.prefix_lens, g.q_start, self.scale, out=out,
                                   max_q_len=g.max_q, sink=self.sink)
-        return out if W == self.vdim else out[..., : self.vdim].contiguous()
+        out = out[..., : self.vdim]
+        return out.contiguous() if gate is None else ops.gate_heads(out, gate)

@@ -15,7 +15,7 @@ reduction that closes every tensor-parallel block.
 
 from __future__ import annotations
 
-from typing import Optional
+from typing import Optional, Tuple
 
 import torch
 from torch import nn
@@ -27,27 +27,35 @@ from ..parallel import state as pstate
 class MoEGate(nn.Module):
     """Router.  ``identity``: further outputs that stand for identity experts (the token's input comes back);
     ``choice_bias``: a correction per output that takes part in the choice but not in the weights; ``renorm_eps`` is
-    added to the sum the weights are divided by.  ``fp32_logits``: the logits are not rounded to the activations' type."""
+    added to the sum the weights are divided by.  ``fp32_logits``: the logits are not rounded to the activations' type.
+    ``sigmoid``: scores are logistic functions of the logits instead of their softmax; ``groups`` = (count, keep): only
+    experts of the best ``keep`` groups of neighbours can be chosen; ``scale``: factor of the weights; ``shared_gate``: one
+    more row of the weight, whose logit gates a shared expert."""
 
     def __init__(self, hidden_size: int, num_experts: int, top_k: int, norm_topk_prob: bool, params_dtype=None, identity: int = 0,
-                 choice_bias: bool = False, renorm_eps: float = 0.0, fp32_logits: bool = False) -> None:
+                 choice_bias: bool = False, renorm_eps: float = 0.0, fp32_logits: bool = False, sigmoid: bool = False,
+                 groups: Tuple[int, int] = (1, 1), scale: float = 1.0, shared_gate: bool = False) -> None:
         super().__init__()
         self.top_k, self.norm_topk_prob, self.renorm_eps = top_k, norm_topk_prob, float(renorm_eps)
-        self.fp32_logits = fp32_logits or choice_bias or renorm_eps > 0
-        self.weight = nn.Parameter(torch.empty(num_experts + identity, hidden_size, dtype=params_dtype or torch.get_default_dtype()),
+        self.sigmoid, self.groups, self.scale, self.extra = sigmoid, groups, float(scale), int(shared_gate)
+        self.fp32_logits = fp32_logits or choice_bias or renorm_eps > 0 or sigmoid or groups[1] < groups[0] or scale != 1.0 or shared_gate
+        self.outputs = num_experts + identity
+        self.weight = nn.Parameter(torch.empty(self.outputs + self.extra, hidden_size, dtype=params_dtype or torch.get_default_dtype()),
                                    requires_grad=False)
-        self.correction = nn.Parameter(torch.zeros(num_experts + identity, dtype=torch.float32), requires_grad=False) if choice_bias else None
+        self.correction = nn.Parameter(torch.zeros(self.outputs, dtype=torch.float32), requires_grad=False) if choice_bias else None
 
     def forward(self, x: torch.Tensor):
+        """(weights, ids), and with ``shared_gate`` the shared expert's logits [T, 1]."""
         if self.fp32_logits:
-            return ops.moe_route(x, self.weight, self.top_k, self.norm_topk_prob, self.correction, self.renorm_eps)
+            return ops.moe_route(x, self.weight, self.top_k, self.norm_topk_prob, self.correction, self.renorm_eps, self.sigmoid,
+                                 *self.groups, self.scale, self.extra)
         return ops.moe_router_topk(x, self.weight, self.top_k, self.norm_topk_prob)
 
 
 class SparseMoeBlock(nn.Module):
     def __init__(self, hidden_size: int, moe_intermediate_size: int, num_experts: int, top_k: int,
                  norm_topk_prob: bool = True, params_dtype=None, prefix: str = "", identity_experts: int = 0,
-                 choice_bias: bool = False, renorm_eps: float = 0.0, fp32_logits: bool = False) -> None:
+                 choice_bias: bool = False, renorm_eps: float = 0.0, fp32_logits: bool = False, **router) -> None:
         super().__init__()
         ep = pstate.get_ep_group()
         self.ep_size, self.ep_rank = ep.world_size, ep.rank_in_group
@@ -61,7 +69,8 @@ class SparseMoeBlock(nn.Module):
         self.inter_shard = 1 if self.ep_size > 1 else self.tp_size
         self.inter = moe_intermediate_size // self.inter_shard
         dt = params_dtype or torch.get_default_dtype()
-        self.gate = MoEGate(hidden_size, num_experts, top_k, norm_topk_prob, dt, identity_experts, choice_bias, renorm_eps, fp32_logits)
+        self.gate = MoEGate(hidden_size, num_experts, top_k, norm_topk_prob, dt, identity_experts, choice_bias, renorm_eps, fp32_logits,
+                            **router)
         self.identity_from = num_experts if identity_experts else 0     # router outputs from here on have no weights
         if identity_experts and (self.ep_size > 1 or self.inter_shard > 1):
             raise NotImplementedError("identity experts are not sharded over ranks")
@@ -114,16 +123,17 @@ class SparseMoeBlock(nn.Module):
         shard = self._exchange(x)
         if shard is not None:
             return shard
-        if self.identity_from:
-            raise NotImplementedError("identity experts are summed by the norm behind the block: use expert_rows")
+        if self.identity_from or self.gate.extra:
+            raise NotImplementedError("identity experts and a gated shared expert are summed by the norm behind the block: use expert_rows")
         topk_w, topk_ids = self.gate(x)
         return ops.moe_experts(x, self.w13, self.w2, topk_w, topk_ids, self.expert_offset, self.swiglu_block,
                                self.num_experts)
 
     def expert_rows(self, x: torch.Tensor) -> "ops.ExpertRows":
         """The routed experts' outputs before they are summed, for a norm that does it (one GPU per replica)."""
-        topk_w, topk_ids = self.gate(x)
-        return ops.moe_expert_rows(x, self.w13, self.w2, topk_w, topk_ids, self.swiglu_block, self.identity_from)
+        topk_w, topk_ids, *logit = self.gate(x)
+        return ops.moe_expert_rows(x, self.w13, self.w2, topk_w, topk_ids, self.swiglu_block, self.identity_from,
+                                   logit[0][:, 0] if logit else None)
 
     def can_exchange(self, rows: int) -> bool:
         """Whether a batch of ``rows`` tokens can go through the expert-parallel exchange on this block."""

@@ -86,6 +86,18 @@ class PostRMSNorm(nn.Module):
         return ops.post_norm(x, None, None, 1.0, self.weight, self.eps, self.out_dtype, update=False)
 
 
+class OutputRMSNorm(PostRMSNorm):
+    """Norm on a sublayer's output only, for a residual stream kept in fp32: ``x += rmsnorm(y) * weight``, in one pass that
+    weighs and sums a mixture's expert rows as :class:`PostRMSNorm` does."""
+
+    def __init__(self, hidden_size: int, eps: float, out_dtype: torch.dtype) -> None:
+        super().__init__(hidden_size, eps, 1.0, out_dtype)
+
+    def forward(self, x: torch.Tensor, y: Optional[torch.Tensor], experts=None) -> torch.Tensor:
+        """``x`` [T, W] fp32 is updated in place; its rows come back in ``out_dtype``."""
+        return ops.post_norm(x, y, None, 1.0, self.weight, self.eps, self.out_dtype, experts=experts, inner=True)
+
+
 class LayerNorm(nn.Module):
     def __init__(self, hidden_size: int, eps: float = 1e-6, bias: bool = True,
                  params_dtype: Optional[torch.dtype] = None) -> None:

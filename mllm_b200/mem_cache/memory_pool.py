@@ -164,6 +164,33 @@ class LayeredKVPool:
             t.zero_()
 
 
+class MixedPool:
+    """Cache of models that have both kinds of layer: K and V rows (:class:`LayeredKVPool`) and latent rows
+    (:class:`LatentPool`) over the same slots and pages."""
+
+    def __init__(self, size: int, shapes: Sequence[Tuple[int, int, int]], widths: Sequence[int], dtype: torch.dtype,
+                 device: torch.device | str, page_size: int = 1) -> None:
+        self.kv = LayeredKVPool(size, shapes, dtype, device, page_size)
+        self.latent = LatentPool(size, widths, dtype, device, page_size)
+        self.page_size, self.size, self.num_slots = self.kv.page_size, self.kv.size, self.kv.num_slots
+        self.layer_num, self.dtype, self.device = self.kv.layer_num + self.latent.layer_num, dtype, self.kv.device
+
+    @staticmethod
+    def cell_bytes(shapes: Sequence[Tuple[int, int, int]], widths: Sequence[int], dtype: torch.dtype) -> int:
+        """Bytes one token occupies over all layers."""
+        return LayeredKVPool.cell_bytes(shapes, dtype) + LatentPool.cell_bytes(widths, dtype)
+
+    def get_kv_buffer(self, index: int) -> Tuple[torch.Tensor, torch.Tensor]:
+        return self.kv.get_kv_buffer(index)
+
+    def get_latent_buffer(self, index: int) -> torch.Tensor:
+        return self.latent.get_latent_buffer(index)
+
+    def clear(self) -> None:
+        self.kv.clear()
+        self.latent.clear()
+
+
 class TokenToKVPoolAllocator:
     """Host-side free list of KV slots / pages.
 

@@ -27,6 +27,7 @@ _REGISTRY: Dict[str, Tuple[str, str]] = {
     "MiniCPM4ForCausalLM": ("mllm_b200.models.minicpm", "MiniCPMForCausalLM"),
     "PebulixForCausalLM": ("mllm_b200.models.pebulix", "PebulixForCausalLM"),
     "KesovikForCausalLM": ("mllm_b200.models.kesovik", "KesovikForCausalLM"),
+    "LufizenForCausalLM": ("mllm_b200.models.lufizen", "LufizenForCausalLM"),
 }
 
 # designs whose config.json names itself in "architecture" and has a layout of its own: a function that checks the
@@ -34,6 +35,7 @@ _REGISTRY: Dict[str, Tuple[str, str]] = {
 _CONFIG_ADAPTERS: Dict[str, Tuple[str, str]] = {
     "Pebulix": ("mllm_b200.models.pebulix", "adapt_config"),
     "Kesovik": ("mllm_b200.models.kesovik", "adapt_config"),
+    "Lufizen": ("mllm_b200.models.lufizen", "adapt_config"),
 }
 
 

@@ -29,20 +29,15 @@ from ..layers import MLP, LightningAttention, ParallelMixer, PostRMSNorm, RowNor
 from ..layers.moe import SparseMoeBlock
 from ..mem_cache import LayeredGDNPool, LayeredKVPool
 from ..parallel import state as pstate
+from .places import load_places, mixture_places, put, require_positive
 from .qwen3 import LogitsProcessorOutput
 
 PARALLEL, LIGHTNING = "parallel", "lightning"
 RENORM_EPS = 1e-20        # joins the sum that the chosen experts' scores are divided by
 
 
-def _positive(where: str, sizes: Dict[str, Any], names: Iterable[str]) -> None:
-    for n in names:
-        if int(sizes.get(n) or 0) <= 0:
-            raise ValueError(f"{where}: {n} must be given and positive")
-
-
 def _check_attention(where: str, m: Dict[str, Any]) -> None:
-    _positive(where, m, ("heads", "kv_heads", "dim", "vdim"))
+    require_positive(where, m, ("heads", "kv_heads", "dim", "vdim"))
     if m["heads"] % m["kv_heads"]:
         raise ValueError(f"{where}: {m['heads']} query heads over {m['kv_heads']} key/value heads")
     if "scale" not in m:
@@ -51,11 +46,11 @@ def _check_attention(where: str, m: Dict[str, Any]) -> None:
     if dims % 2 or not 0 <= dims <= m["dim"]:
         raise ValueError(f"{where}: {dims} of {m['dim']} features rotated")
     if m.get("mask") is not None:
-        _positive(f"{where}: mask", m["mask"], ("size",))
+        require_positive(f"{where}: mask", m["mask"], ("size",))
 
 
 def _check_lightning(where: str, m: Dict[str, Any]) -> None:
-    _positive(where, m, ("heads", "dim", "vdim"))
+    require_positive(where, m, ("heads", "dim", "vdim"))
     d = m.get("decay")
     if not isinstance(d, (int, float)) and (d is None or len(d) != m["heads"]):
         raise ValueError(f"{where}: decay must hold one factor for each of {m['heads']} heads")
@@ -65,16 +60,16 @@ def _check_mlp(where: str, mlp: Optional[Dict[str, Any]]) -> None:
     if mlp is None:
         return
     if mlp.get("kind") == "dense":
-        _positive(where, mlp, ("ff",))
+        require_positive(where, mlp, ("ff",))
     elif mlp.get("kind") == "moe":
         r = mlp["router"]
-        _positive(where, r, ("experts", "top"))
-        _positive(f"{where}: expert", mlp["expert"], ("ff",))
+        require_positive(where, r, ("experts", "top"))
+        require_positive(f"{where}: expert", mlp["expert"], ("ff",))
         outputs = int(r["experts"]) + int(r.get("identity") or 0)
         if r["top"] > min(outputs, 32) or outputs > 256:
             raise ValueError(f"{where}: {r['top']} of {outputs} router outputs (at most 32 of 256)")
         if mlp.get("shared") is not None:
-            _positive(f"{where}: shared", mlp["shared"], ("ff",))
+            require_positive(f"{where}: shared", mlp["shared"], ("ff",))
     else:
         raise ValueError(f"{where}: unknown feed-forward {mlp.get('kind')!r}")
 
@@ -239,28 +234,10 @@ class KesovikForCausalLM(nn.Module):
     def load_weights(self, weights: Iterable[Tuple[str, torch.Tensor]]) -> set:
         """Checkpoint names: ``embed``, ``head``, ``final.norm``, ``l<i>.norm1|norm2|ls1|ls2``, ``l<i>.mix.[left.|right.]<tensor>``,
         ``l<i>.mlp.<tensor>``.  Every tensor must have a place and every place a tensor."""
-        places = self._places()
-        loaded = set()
-        for name, t in weights:
-            put = places.get(name)
-            if put is None:
-                raise ValueError(f"unexpected tensor {name!r} in the checkpoint")
-            put(t.materialize() if hasattr(t, "materialize") else t)
-            loaded.add(name)
-        missing = sorted(set(places) - loaded)
-        if missing:
-            raise ValueError(f"the checkpoint lacks {len(missing)} tensors: {', '.join(missing[:8])}")
-        return loaded
+        return load_places(self._places(), weights)
 
     def _places(self) -> Dict[str, Any]:
         out: Dict[str, Any] = {}
-
-        def put(p):
-            def copy(t):
-                if t.shape != p.shape:
-                    raise ValueError(f"a tensor of shape {tuple(t.shape)} does not fit {tuple(p.shape)}")
-                p.data.copy_(t)
-            return copy
 
         out["embed"], out["head"], out["final.norm"] = put(self.embed.weight), put(self.head.weight), put(self.final_norm.weight)
         for i, layer in enumerate(self.layers):
@@ -284,17 +261,7 @@ class KesovikForCausalLM(nn.Module):
             if isinstance(layer.mlp, SquaredReluMLP):
                 out[at + "up"], out[at + "down"] = put(layer.mlp.up_proj.weight), put(layer.mlp.down_proj.weight)
                 continue
-            block, shared = layer.mlp.block, layer.mlp.shared
-            out[at + "router"], out[at + "correction"] = put(block.gate.weight), put(block.gate.correction)
-            for e in range(block.num_experts):
-                for n in ("gate", "up"):
-                    out[f"{at}e{e}.{n}"] = lambda t, b=block, e=e, n=n: b.w13.weight_loader(b.w13, t, e, n)
-                out[f"{at}e{e}.down"] = lambda t, b=block, e=e: b.w2.weight_loader(b.w2, t, e)
-            if shared is not None:
-                gu, down = shared.gate_up_proj.weight, shared.down_proj.weight
-                for j, n in enumerate(("gate", "up")):
-                    out[f"{at}shared.{n}"] = lambda t, p=gu, j=j: p.weight_loader(p, t, j)
-                out[at + "shared.down"] = lambda t, p=down: p.weight_loader(p, t)
+            out.update(mixture_places(at, layer.mlp.block, layer.mlp.shared))
         return out
 
     def post_load(self) -> None:

@@ -27,15 +27,10 @@ from ..layers import MLP, DynamicTanh, LatentAttention, VocabParallelEmbedding
 from ..layers.gdn import FusedGatedDeltaNet
 from ..mem_cache import LatentPool, LayeredGDNPool
 from ..parallel import state as pstate
+from .places import load_places, require_positive
 from .qwen3 import LogitsProcessorOutput
 
 LATENT, DELTA = "latent_attention", "delta"
-
-
-def _positive(where: str, sizes: Dict[str, Any], names: Iterable[str]) -> None:
-    for n in names:
-        if int(sizes.get(n) or 0) <= 0:
-            raise ValueError(f"{where}: {n} must be given and positive")
 
 
 def adapt_config(raw: Dict[str, Any]) -> SimpleNamespace:
@@ -44,7 +39,7 @@ def adapt_config(raw: Dict[str, Any]) -> SimpleNamespace:
     for i, layer in enumerate(layers):
         kind, m, mlp, where = layer["type"], layer["mixer"], layer.get("mlp"), f"layer {i}"
         if kind == LATENT:
-            _positive(where, m, ("heads", "dim", "vdim", "q_rank", "kv_rank"))
+            require_positive(where, m, ("heads", "dim", "vdim", "q_rank", "kv_rank"))
             j = m.get("kv_from")
             if j is not None:
                 src = layers[j] if 0 <= j < i else None
@@ -53,7 +48,7 @@ def adapt_config(raw: Dict[str, Any]) -> SimpleNamespace:
                     raise ValueError(f"{where}: kv_from {j} must name an earlier latent-attention layer with latents of its "
                                      "own and the same kv_rank")
         elif kind == DELTA:
-            _positive(where, m, ("heads", "kv_heads", "dim", "vdim", "conv"))
+            require_positive(where, m, ("heads", "kv_heads", "dim", "vdim", "conv"))
             if m["heads"] % m["kv_heads"]:
                 raise ValueError(f"{where}: {m['heads']} value heads over {m['kv_heads']} key heads")
         else:
@@ -165,18 +160,7 @@ class PebulixForCausalLM(nn.Module):
     def load_weights(self, weights: Iterable[Tuple[str, torch.Tensor]]) -> set:
         """Checkpoint names: ``embed``, ``l<i>.norm1|norm2`` and ``final.norm`` (each with ``.alpha`` and ``.b``),
         ``l<i>.mix.<tensor>``, ``l<i>.mlp.gate|up|down``.  Every tensor must have a place and every place a tensor."""
-        places = self._places()
-        loaded = set()
-        for name, t in weights:
-            put = places.get(name)
-            if put is None:
-                raise ValueError(f"unexpected tensor {name!r} in the checkpoint")
-            put(t.materialize() if hasattr(t, "materialize") else t)
-            loaded.add(name)
-        missing = sorted(set(places) - loaded)
-        if missing:
-            raise ValueError(f"the checkpoint lacks {len(missing)} tensors: {', '.join(missing[:8])}")
-        return loaded
+        return load_places(self._places(), weights)
 
     def _places(self) -> Dict[str, Any]:
         out: Dict[str, Any] = {}

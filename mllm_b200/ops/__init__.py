@@ -191,18 +191,21 @@ class ExpertRows:
     ids: torch.Tensor           # [T, k] int32
     token_in: torch.Tensor      # [T, W] the experts' input
     identity_from: int = 0      # > 0: ids from here on return the token's input
+    shared_logit: Optional[torch.Tensor] = None     # [T] fp32: the shared expert counts sigmoid(shared_logit) times
 
 
 def post_norm(x: torch.Tensor, y: Optional[torch.Tensor], ls: Optional[torch.Tensor], alpha: float, weight: torch.Tensor, eps: float,
-              dtype: torch.dtype, update: bool = True, experts: Optional[ExpertRows] = None) -> torch.Tensor:
+              dtype: torch.dtype, update: bool = True, experts: Optional[ExpertRows] = None, inner: bool = False) -> torch.Tensor:
     """``x = rmsnorm(alpha * x + ls * (y + weighted expert rows)) * weight`` for an fp32 stream ``x`` [T, W] (in place
-    when ``update``), returned in ``dtype`` too.  ``y`` [T, W] and ``ls`` [W] may be None."""
+    when ``update``), returned in ``dtype`` too.  ``y`` [T, W] and ``ls`` [W] may be None.  ``inner``: the norm is on the
+    sublayer's output alone, ``x = alpha * x + ls * rmsnorm(y + weighted expert rows) * weight``."""
+    logit = None if experts is None else experts.shared_logit
     if not use_kernels(x):
-        return ref.post_norm(x, y, ls, alpha, weight, eps, dtype, update, experts)
+        return ref.post_norm(x, y, ls, alpha, weight, eps, dtype, update, experts, inner, logit)
     h = torch.empty(x.shape, dtype=dtype, device=x.device)
     e = experts
     parts = [] if e is None else [e.rows, e.sorted_pos, e.topk_w, e.ids, e.token_in]
-    ext().post_norm(x, y, ls, float(alpha), weight, float(eps), h, update, parts, 0 if e is None else e.identity_from)
+    ext().post_norm(x, y, ls, float(alpha), weight, float(eps), h, update, parts, 0 if e is None else e.identity_from, inner, logit)
     return h
 
 
@@ -224,6 +227,18 @@ def rownorm_rope_kv(row, q_weight, k_weight, inv_freq, positions, loc, q_out, k_
         return ref.rownorm_rope_kv(*args)
     ext().rownorm_rope_kv(row, q_weight, k_weight, inv_freq, positions.to(torch.int64).contiguous(), loc.to(torch.int64).contiguous(),
                           *args[6:])
+
+
+def headnorm_rope_kv(row, inv_freq, positions, loc, q_out, k_cache, v_cache, heads: int, kv_heads: int, dim: int, vdim: int, v_at: int,
+                     halves: bool, eps: float) -> None:
+    """Prologue of attention with a norm per head: ``row`` [T, q | k | ..]; query and key heads turn by ``positions *
+    inv_freq`` (fp64, one per rotated pair; ``halves``: feature i with the one half the rotated features on, else
+    neighbours) and are divided by their root mean square; q goes to ``q_out`` [T, heads, >= dim] (zeros behind), k and the
+    values (columns from ``v_at``, unchanged) to the cache slots ``loc``."""
+    args = (row, inv_freq, positions, loc, q_out, k_cache, v_cache, heads, kv_heads, dim, vdim, v_at, halves, eps)
+    if not use_kernels(row):
+        return ref.headnorm_rope_kv(*args)
+    ext().headnorm_rope_kv(row, inv_freq, positions.to(torch.int64).contiguous(), loc.to(torch.int64).contiguous(), *args[4:])
 
 
 def soft_cap(x: torch.Tensor, cap: float) -> torch.Tensor:
@@ -877,15 +892,39 @@ def gelu_erf(x: torch.Tensor) -> torch.Tensor:
 # latent attention (one cached row per token, shared by all heads)
 # --------------------------------------------------------------------------
 def latent_prologue(y: torch.Tensor, q_weight: torch.Tensor, kv_weight: Optional[torch.Tensor], eps: float,
-                    loc: Optional[torch.Tensor] = None, cache: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """RMS norm (fp32) of the down projections' rows ``y = [query latent | cache latent]``: returns the normed query
-    latent [T, q_rank] and writes the normed cache latent to ``cache[loc]`` (``kv_weight`` None: the layer reads
-    another layer's latents and writes none)."""
+                    loc: Optional[torch.Tensor] = None, cache: Optional[torch.Tensor] = None,
+                    positions: Optional[torch.Tensor] = None, inv_freq: Optional[torch.Tensor] = None):
+    """RMS norm (fp32) of the down projections' rows ``y = [query latent | cache latent | rotated key part | ..]``: returns
+    the normed query latent [T, q_rank] and writes the normed cache latent to ``cache[loc]`` (``kv_weight`` None: the layer
+    reads another layer's latents and writes none).  With ``inv_freq`` (fp64, one per pair of neighbouring features) the key
+    part, turned by ``positions * inv_freq``, follows the latent in the cache row, and the cosines and sines [T, rot / 2, 2]
+    come back for the query heads (None without)."""
     if not use_kernels(y):
-        return ref.latent_prologue(y, q_weight, kv_weight, eps, loc, cache)
+        return ref.latent_prologue(y, q_weight, kv_weight, eps, loc, cache, positions, inv_freq)
     cq = torch.empty((y.shape[0], q_weight.numel()), dtype=y.dtype, device=y.device)
-    ext().latent_prologue(y, q_weight, kv_weight, eps, cq, None if loc is None else loc.to(torch.int64).contiguous(), cache)
-    return cq
+    turns = None if inv_freq is None else torch.empty((y.shape[0], inv_freq.numel(), 2), dtype=torch.float32, device=y.device)
+    ext().latent_prologue(y, q_weight, kv_weight, eps, cq, None if loc is None else loc.to(torch.int64).contiguous(), cache,
+                          None if inv_freq is None else positions.to(torch.int64).contiguous(), inv_freq, turns)
+    return cq, turns
+
+
+def turn_heads(x: torch.Tensor, turns: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """x [T, H, rot] (a slice of wider heads will do): neighbouring features turn by ``turns`` [T, rot / 2, 2]; in place
+    unless ``out`` is given."""
+    out = x if out is None else out
+    if not use_kernels(x):
+        return out.copy_(ref.turn_heads(x, turns))
+    ext().turn_heads(x, turns, out)
+    return out
+
+
+def gate_heads(x: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
+    """``x[t, h] * sigmoid(gate[t, h])``, contiguous; x [T, H, W] and gate [T, H] may be slices."""
+    if not use_kernels(x):
+        return (x.float() * torch.sigmoid(gate.float()).unsqueeze(-1)).to(x.dtype)
+    out = torch.empty(x.shape, dtype=x.dtype, device=x.device)
+    ext().gate_heads(x, gate, out)
+    return out
 
 
 def latent_gather(cache, req_to_token, req, lens, start, total: int, max_len: int) -> torch.Tensor:
@@ -897,28 +936,36 @@ def latent_gather(cache, req_to_token, req, lens, start, total: int, max_len: in
     return out
 
 
-def head_linear(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
-    """``out[t, h] = weight[h] @ x[t, h]``: x [T, H, K], weight [H, N, K] -> [T, H, N]."""
+def head_linear(x: torch.Tensor, weight: torch.Tensor, gate: Optional[torch.Tensor] = None, turns: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``out[t, h] = weight[h] @ x[t, h]``: x [T, H, K], weight [H, N, K] -> [T, H, N].  ``gate`` [T, H]: times its logistic
+    function.  ``turns`` [T, rot / 2, 2]: x is [T, H, K + rot], and the features behind K, turned, follow the N results."""
+    T, H, N, K = x.shape[0], x.shape[1], weight.shape[1], weight.shape[2]
+    out = torch.empty((T, H, N + x.shape[2] - K), dtype=x.dtype, device=x.device)
     if use_kernels(x) and x.dtype != torch.float32:
-        out = torch.empty((x.shape[0], x.shape[1], weight.shape[1]), dtype=x.dtype, device=x.device)
-        if x.shape[0] == 0 or ext().head_linear(x, weight, out) == 0:
+        if T == 0 or ext().head_linear(x, weight, out, gate, turns) == 0:
             return out
     # 32-bit and unaligned sizes: a library batched product
-    return torch.bmm(x.transpose(0, 1), weight.transpose(1, 2)).transpose(0, 1).contiguous()
+    torch.bmm(x[..., :K].transpose(0, 1), weight.transpose(1, 2), out=(y := torch.empty((H, T, N), dtype=x.dtype, device=x.device)))
+    out[..., :N] = y.transpose(0, 1)
+    if turns is not None:
+        turn_heads(x[..., K:], turns, out[..., N:])
+    return out if gate is None else gate_heads(out, gate)
 
 
 _LATENT_ROWS = 32768     # query rows of one launch (they are a grid dimension)
 
 
 def latent_attention(q: torch.Tensor, cache: torch.Tensor, req_to_token, row_req, row_pos, scale: float,
-                     sink: Optional[torch.Tensor] = None, max_seq_len: int = 0) -> torch.Tensor:
-    """Attention of queries in the latent space over the cached latents, which are keys and values at once: row t is a
-    token of request ``row_req[t]`` at position ``row_pos[t]`` and sees the keys 0 .. its position.
-    q [rows, H, rank] -> [rows, H, rank]; ``sink`` [H] fp32 joins the denominator as ``exp(sink)``."""
+                     sink: Optional[torch.Tensor] = None, max_seq_len: int = 0, rank: Optional[int] = None) -> torch.Tensor:
+    """Attention of queries in the latent space over the cached rows, which are keys and values at once: row t is a
+    token of request ``row_req[t]`` at position ``row_pos[t]`` and sees the keys 0 .. its position.  Keys are whole rows,
+    values their first ``rank`` features (default: all).  q [rows, H, key width] -> [rows, H, rank]; ``sink`` [H] fp32 joins
+    the denominator as ``exp(sink)``."""
+    rank = q.shape[2] if rank is None else rank
     if not use_kernels(q):
-        return ref.latent_attention(q, cache, req_to_token, row_req, row_pos, scale, sink)
+        return ref.latent_attention(q, cache, req_to_token, row_req, row_pos, scale, sink, rank)
     q = q.contiguous()
-    out = torch.empty_like(q)
+    out = torch.empty((q.shape[0], q.shape[1], rank), dtype=q.dtype, device=q.device)
     for r in range(0, q.shape[0], _LATENT_ROWS):
         e = min(q.shape[0], r + _LATENT_ROWS)
         ext().latent_attention(q[r:e], cache, req_to_token, row_req[r:e], row_pos[r:e], float(scale), sink, out[r:e], int(max_seq_len))
@@ -1065,20 +1112,32 @@ def lightning_attention(q, k, v, decay, state, state_indices, seq_lens, has_stat
 # mixture of experts
 # --------------------------------------------------------------------------
 def moe_route(hidden: torch.Tensor, gate_weight: torch.Tensor, top_k: int, renormalize: bool = True,
-              correction: Optional[torch.Tensor] = None, renorm_eps: float = 0.0):
-    """Router with fp32 logits: softmax over all outputs, the ``top_k`` largest of ``scores + correction``, weights from
-    the scores alone (divided by their sum + ``renorm_eps`` when ``renormalize``)."""
-    if not use_kernels(hidden):
-        return ref.moe_router_topk(hidden, gate_weight, top_k, renormalize, correction, renorm_eps)
-    T, E = hidden.shape[0], gate_weight.shape[0]
+              correction: Optional[torch.Tensor] = None, renorm_eps: float = 0.0, sigmoid: bool = False, groups: int = 1,
+              keep: int = 1, scale: float = 1.0, extra: int = 0):
+    """Router with fp32 logits: scores (softmax over all outputs, or ``sigmoid`` of each), the ``top_k`` largest of
+    ``scores + correction``, weights from the scores alone (divided by their sum + ``renorm_eps`` when ``renormalize``, times
+    ``scale``).  ``keep`` < ``groups``: only outputs of the ``keep`` groups of neighbours with the largest sums of their two
+    largest choice scores.  ``extra``: the last rows of ``gate_weight`` are no outputs to choose from; their logits come
+    back as a third result [T, extra]."""
+    T, E = hidden.shape[0], gate_weight.shape[0] - extra
     if E > 256 or top_k > 32:
         raise ValueError(f"moe_route: at most 256 outputs and 32 choices, not {E} and {top_k}")
-    logits = torch.empty((T, E), dtype=torch.float32, device=hidden.device)
+    if not use_kernels(hidden):
+        w, ids = ref.moe_router_topk(hidden, gate_weight[:E], top_k, renormalize, correction, renorm_eps, sigmoid, groups, keep, scale)
+        return (w, ids, hidden.float() @ gate_weight[E:].float().t()) if extra else (w, ids)
     w = torch.empty((T, top_k), dtype=torch.float32, device=hidden.device)
     ids = torch.empty((T, top_k), dtype=torch.int32, device=hidden.device)
-    ext().moe_router_logits(hidden, gate_weight, logits)
-    ext().moe_router_topk(logits, w, ids, renormalize, correction, float(renorm_eps))
-    return w, ids
+    together = E + extra <= 256
+    logits = torch.empty((T, E + extra if together else E), dtype=torch.float32, device=hidden.device)
+    ext().moe_router_logits(hidden, gate_weight if together else gate_weight[:E], logits)
+    ext().moe_router_topk(logits[:, :E], w, ids, renormalize, correction, float(renorm_eps), sigmoid, groups, keep, float(scale))
+    if not extra:
+        return w, ids
+    if together:
+        return w, ids, logits[:, E:]
+    rest = torch.empty((T, extra), dtype=torch.float32, device=hidden.device)
+    ext().moe_router_logits(hidden, gate_weight[E:], rest)
+    return w, ids, rest
 
 
 def moe_router_topk(hidden: torch.Tensor, gate_weight: torch.Tensor, top_k: int, renormalize: bool = True):
@@ -1163,14 +1222,15 @@ def moe_experts(x, w13, w2, topk_w, topk_ids, expert_offset: int = 0, swiglu_blo
     return out
 
 
-def moe_expert_rows(x, w13, w2, topk_w, topk_ids, swiglu_block: int = 0, identity_from: int = 0) -> ExpertRows:
+def moe_expert_rows(x, w13, w2, topk_w, topk_ids, swiglu_block: int = 0, identity_from: int = 0,
+                    shared_logit: Optional[torch.Tensor] = None) -> ExpertRows:
     """The experts' outputs for a kernel that sums them itself (:func:`post_norm`).  ``identity_from`` > 0: ids from there
     on are identity experts, which return the token's input and have no row."""
     if not use_kernels(x):
         rows, pos = ref.moe_expert_rows(x, w13, w2, topk_ids, swiglu_block)
     else:
         rows, pos = _moe_sorted_rows(x, w13, w2, topk_ids, 0, swiglu_block, None)
-    return ExpertRows(rows, pos, topk_w.contiguous(), topk_ids.contiguous(), x.contiguous(), int(identity_from))
+    return ExpertRows(rows, pos, topk_w.contiguous(), topk_ids.contiguous(), x.contiguous(), int(identity_from), shared_logit)
 
 
 def ep_moe_exchange(x_own, w13, w2, topk_w, topk_ids, swiglu_block: int, comm) -> torch.Tensor:

@@ -474,21 +474,27 @@ def top_k_top_p_min_p_sample(
 # mixture of experts
 # --------------------------------------------------------------------------
 def moe_router_topk(hidden: torch.Tensor, gate_weight: torch.Tensor, top_k: int, renormalize: bool = True,
-                    correction: Optional[torch.Tensor] = None, renorm_eps: float = 0.0):
+                    correction: Optional[torch.Tensor] = None, renorm_eps: float = 0.0, sigmoid: bool = False, groups: int = 1,
+                    keep: int = 1, scale: float = 1.0):
     """fp32 ``softmax(hidden @ gate_weight.T)`` over all experts -> top-k (sorted by weight) ->
     optional renormalisation of the k weights (mllm/models/qwen3_moe/modeling_qwen3_moe_fa2.hpp:121-138).
-    With ``correction`` the choice goes by ``scores + correction``, the weights are the scores alone.
+    With ``correction`` the choice goes by ``scores + correction``, the weights are the scores alone.  ``sigmoid``: the
+    scores are logistic functions of the logits.  ``keep`` < ``groups``: only experts of the ``keep`` groups of neighbours
+    with the largest sums of their two largest choice scores.  ``scale``: factor of the weights.
     Returns (weights fp32 [T, k], expert ids int32 [T, k])."""
     logits = _f32(hidden) @ _f32(gate_weight).t()
-    scores = torch.softmax(logits, dim=-1)
-    if correction is None:
-        w, idx = torch.topk(scores, top_k, dim=-1, sorted=True)
-    else:
-        idx = torch.topk(scores + _f32(correction), top_k, dim=-1, sorted=True).indices
-        w = scores.gather(-1, idx)
+    scores = torch.sigmoid(logits) if sigmoid else torch.softmax(logits, dim=-1)
+    choice = scores if correction is None else scores + _f32(correction)
+    if keep < groups:
+        by_group = choice.unflatten(-1, (groups, -1))
+        best = by_group.topk(min(2, by_group.shape[-1]), dim=-1).values.sum(-1).topk(keep, dim=-1).indices
+        closed = torch.ones_like(by_group[..., 0], dtype=torch.bool).scatter_(-1, best, False)
+        choice = by_group.masked_fill(closed.unsqueeze(-1), float("-inf")).flatten(-2)
+    idx = torch.topk(choice, top_k, dim=-1, sorted=True).indices
+    w = scores.gather(-1, idx)
     if renormalize:
         w = w / (w.sum(-1, keepdim=True) + renorm_eps)
-    return w, idx.to(torch.int32)
+    return w * scale, idx.to(torch.int32)
 
 
 def moe_experts(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_w: torch.Tensor, topk_ids: torch.Tensor,
@@ -527,8 +533,10 @@ def moe_expert_rows(x, w13, w2, topk_ids, swiglu_block: int = 0):
 # --------------------------------------------------------------------------
 # fp32 residual stream, norms after the sum, Dynamic Tanh, latent attention
 # --------------------------------------------------------------------------
-def post_norm(x, y, ls, alpha, weight, eps, dtype, update=True, experts=None):
+def post_norm(x, y, ls, alpha, weight, eps, dtype, update=True, experts=None, inner=False, y_logit=None):
     z = torch.zeros_like(x) if y is None else _f32(y)
+    if y_logit is not None:
+        z = z * torch.sigmoid(y_logit).unsqueeze(-1)
     if experts is not None:
         T, k = experts.topk_w.shape
         pos = experts.sorted_pos[: T * k].view(T, k).long()
@@ -537,8 +545,15 @@ def post_norm(x, y, ls, alpha, weight, eps, dtype, update=True, experts=None):
         z = z + (part * w.unsqueeze(-1)).sum(1)
         if experts.identity_from > 0:
             z = z + _f32(experts.token_in) * (w * (experts.ids >= experts.identity_from)).sum(1, keepdim=True)
+
+    def norm(t):
+        return t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps) * _f32(weight)
+
+    if inner:
+        z = norm(z)
     z = float(alpha) * x + (z if ls is None else _f32(ls) * z)
-    z = z * torch.rsqrt(z.pow(2).mean(-1, keepdim=True) + eps) * _f32(weight)
+    if not inner:
+        z = norm(z)
     if update:
         x.copy_(z)
     return z.to(dtype)
@@ -572,6 +587,28 @@ def rownorm_rope_kv(row, q_w, k_w, inv_freq, positions, loc, q_out, k_cache, v_c
     q_out[..., :dim] = q.to(q_out.dtype)
     k_cache[loc.long(), :, :dim] = k.to(k_cache.dtype)
     v_cache[loc.long(), :, :vdim] = row[:, nq + nk:nq + nk + kv_heads * vdim].reshape(T, kv_heads, vdim)
+
+
+def rotate_halves(x: torch.Tensor, positions: torch.Tensor, inv_freq: torch.Tensor) -> torch.Tensor:
+    """x [T, H, D] fp32: features i and i + n, n frequencies, turn by ``positions * inv_freq[i]``, later ones stay."""
+    n = inv_freq.numel()
+    a = (positions.double().unsqueeze(-1) * inv_freq.double()).unsqueeze(1)
+    c, s = torch.cos(a).float(), torch.sin(a).float()
+    u, v = x[..., :n], x[..., n:2 * n]
+    return torch.cat([u * c - v * s, v * c + u * s, x[..., 2 * n:]], -1)
+
+
+def headnorm_rope_kv(row, inv_freq, positions, loc, q_out, k_cache, v_cache, heads, kv_heads, dim, vdim, v_at, halves, eps):
+    T, turn = row.shape[0], rotate_halves if halves else rotate_pairs
+
+    def head(t, n):
+        t = turn(_f32(t).reshape(T, n, dim), positions, inv_freq)
+        return t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps)
+
+    q_out.zero_()
+    q_out[..., :dim] = head(row[:, : heads * dim], heads).to(q_out.dtype)
+    k_cache[loc.long(), :, :dim] = head(row[:, heads * dim: (heads + kv_heads) * dim], kv_heads).to(k_cache.dtype)
+    v_cache[loc.long(), :, :vdim] = row[:, v_at: v_at + kv_heads * vdim].reshape(T, kv_heads, vdim)
 
 
 def soft_cap(x, cap):
@@ -618,28 +655,46 @@ def residual_dyt(x, y, mult, alpha, weight, bias, dtype):
     return (torch.tanh(_f32(alpha) * x) * _f32(weight) + _f32(bias)).to(dtype)
 
 
-def latent_prologue(y, q_weight, kv_weight, eps, loc=None, cache=None):
+def turns_of(positions, inv_freq):
+    """[T, pairs, 2] fp32: cosine and sine of ``positions * inv_freq``."""
+    a = positions.double().unsqueeze(-1) * inv_freq.double()
+    return torch.stack([torch.cos(a), torch.sin(a)], -1).float()
+
+
+def turn_heads(x, turns):
+    """x [T, H, rot]: neighbouring features turn by ``turns`` [T, rot / 2, 2]."""
+    c, s = turns[:, None, :, 0], turns[:, None, :, 1]
+    u, v = _f32(x[..., 0::2]), _f32(x[..., 1::2])
+    return torch.stack([u * c - v * s, v * c + u * s], -1).flatten(-2).to(x.dtype)
+
+
+def latent_prologue(y, q_weight, kv_weight, eps, loc=None, cache=None, positions=None, inv_freq=None):
     def norm(t, w):
         t = _f32(t)
         return (t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps) * _f32(w)).to(y.dtype)
 
     nq = q_weight.numel()
+    turns = None if inv_freq is None else turns_of(positions, inv_freq)
     if kv_weight is not None:
-        cache[loc.long()] = norm(y[:, nq:nq + kv_weight.numel()], kv_weight)
-    return norm(y[:, :nq], q_weight)
+        rank = kv_weight.numel()
+        cache[loc.long(), :rank] = norm(y[:, nq:nq + rank], kv_weight)
+        if turns is not None:
+            cache[loc.long(), rank:] = turn_heads(y[:, None, nq + rank: nq + rank + 2 * turns.shape[1]], turns)[:, 0]
+    return norm(y[:, :nq], q_weight), turns
 
 
 def latent_gather(cache, req_to_token, req, lens):
     return torch.cat([cache[req_to_token[int(r), : int(n)].long()] for r, n in zip(req, lens)]) if len(req) else cache[:0]
 
 
-def latent_attention(q, cache, req_to_token, row_req, row_pos, scale, sink=None):
-    out = torch.empty_like(q)
+def latent_attention(q, cache, req_to_token, row_req, row_pos, scale, sink=None, rank=None):
+    rank = q.shape[2] if rank is None else rank
+    out = q.new_empty((*q.shape[:2], rank))
     for t in range(q.shape[0]):
         c = _f32(cache[req_to_token[int(row_req[t]), : int(row_pos[t]) + 1].long()])      # [n, rank]
         s = (_f32(q[t]) @ c.t()) * scale                                                  # [H, n]
         p = sink_softmax(s, sink)
-        out[t] = (p @ c).to(q.dtype)
+        out[t] = (p @ c[:, :rank]).to(q.dtype)
     return out
 
 

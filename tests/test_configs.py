@@ -151,6 +151,6 @@ def test_helper_command_lists_architectures_and_extensions(capsys):
     main(["show-config"])
     info = json.loads(capsys.readouterr().out)
     assert "Qwen3ForCausalLM" in info["architectures"] and "compressed-tensors" in info["quantization"]
-    assert set(info["extensions"]) == {"mllm_b200_C", "mllm_b200_R", "mllm_b200_L", "mllm_b200_E", "mllm_b200_X", "mllm_b200_host"}
+    assert set(info["extensions"]) == {"mllm_b200_C", "mllm_b200_R", "mllm_b200_A", "mllm_b200_L", "mllm_b200_E", "mllm_b200_X", "mllm_b200_host"}
     main(["models"])
     assert "Qwen3VLForConditionalGeneration" in capsys.readouterr().out.split()

@@ -41,6 +41,9 @@ CUDA_FLAGS = [
     "-Xptxas", "-v",
 ]
 CXX_FLAGS = ["-O3", "-std=c++17"]
+# the libstdc++ that torch uses, also where the compiler would link its own copy statically: with two copies in a process
+# the first number that is formatted into an error message crashes instead of raising
+LD_FLAGS = ["-l:libstdc++.so.6"]
 
 _COMMON = ["bindings_common.h", "common.cuh", "kernels.h", "mma.cuh"]
 
@@ -107,7 +110,7 @@ def _source_hash(name: str) -> str:
     for p in sorted(_existing(spec["sources"]) + _existing(spec["headers"])):
         h.update(p.name.encode())
         h.update(p.read_bytes())
-    h.update(" ".join(CUDA_FLAGS if spec["cuda"] else CXX_FLAGS).encode())
+    h.update(" ".join((CUDA_FLAGS if spec["cuda"] else CXX_FLAGS) + LD_FLAGS).encode())
     return h.hexdigest()
 
 
@@ -148,6 +151,7 @@ def build_extension(name: str, verbose: bool = False) -> ModuleType:
         extra_cflags=CXX_FLAGS,
         extra_cuda_cflags=CUDA_FLAGS if spec["cuda"] else None,
         extra_include_paths=[str(_CSRC)],
+        extra_ldflags=list(LD_FLAGS),      # load() appends to it
         build_directory=str(out),
         with_cuda=spec["cuda"],
         verbose=verbose,

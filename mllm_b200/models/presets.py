@@ -2,8 +2,8 @@
 
 Each preset is a plain attribute bag with the HF ``config.json`` field names the
 models read.  Shapes: Qwen3 dense (0.6B / 1.7B / 4B / 8B / 14B / 32B), Qwen3-30B-A3B
-(MoE), Llama / Qwen2 decoders, the Qwen3.5 hybrids, Pebulix, Kesovik, and the vision+language pairs Qwen3-VL-2B, Qwen2-VL-2B
-and Qwen2.5-VL-3B (each with a ``-tiny`` shape for tests).
+(MoE), Llama / Qwen2 decoders, the Qwen3.5 hybrids, Pebulix, Kesovik, Lufizen, and the vision+language pairs Qwen3-VL-2B,
+Qwen2-VL-2B and Qwen2.5-VL-3B (each with a ``-tiny`` shape for tests).
 """
 
 from __future__ import annotations
@@ -131,6 +131,36 @@ PRESETS["kesovik-6b"] = _kesovik(24, 2048, 6144, 151936, heads=16, kv_heads=4, d
                                  par_lin_heads=8, experts=64, identity=8, top=8, expert_ff=512, shared_ff=512)
 PRESETS["kesovik-tiny"] = _kesovik(4, 128, 256, 1024, heads=4, kv_heads=2, dim=32, window=48, lin_heads=2, lin_dim=32, par_lin_heads=2,
                                    experts=6, identity=2, top=2, expert_ff=64, shared_ff=64)
+
+
+def _lufizen(layers, width, vocab, heads, kv_heads, dim, rot_dim, vdim, q_rank, kv_rank, experts, groups, keep, top, expert_ff,
+             shared_ff) -> Dict[str, Any]:
+    """Latent attention and key-valued attention in turn, a mixture behind each."""
+    out = []
+    for i in range(layers):
+        mlp = dict(kind="moe", expert=dict(ff=expert_ff), shared=dict(ff=shared_ff),
+                   router=dict(experts=experts, groups=dict(count=groups, keep=keep), scale=2.5, top=top))
+        if i % 2 == 0:
+            m = dict(heads=heads, dim=dim, rot_dim=rot_dim, vdim=vdim, q_rank=q_rank, kv_rank=kv_rank, rot=dict(base=1e4, dims=rot_dim),
+                     scale=(dim + rot_dim) ** -0.5)
+            out.append(dict(type="latent_attention", mlp=mlp, mixer=m))
+        else:
+            rot = dict(base=5e5, dims=dim // 2, scaling=dict(factor=8.0, low=1.0, high=4.0, original=8192))
+            m = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, rot=rot, scale=dim ** -0.5)
+            out.append(dict(type="attention", mlp=mlp, mixer=m))
+    return dict(architecture="Lufizen", layers=out, norm=dict(eps=1e-6), embedding=dict(scale=1.0), logit_scale=1.0, vocab=vocab, width=width,
+                torch_dtype="bfloat16")
+
+
+# hidden size, depth, vocabulary, query and key heads and experts of qwen2-moe-6b
+PRESETS["lufizen-6b"] = _lufizen(24, 2048, 151936, heads=16, kv_heads=4, dim=128, rot_dim=64, vdim=128, q_rank=1024, kv_rank=512, experts=64,
+                                 groups=8, keep=4, top=8, expert_ff=512, shared_ff=512)
+PRESETS["lufizen-tiny"] = _lufizen(4, 128, 1024, heads=4, kv_heads=2, dim=32, rot_dim=16, vdim=32, q_rank=64, kv_rank=64, experts=8, groups=4,
+                                   keep=2, top=2, expert_ff=64, shared_ff=64)
+PRESETS["qwen2-moe-6b"] = dict(
+    _dense(2048, 24, 16, 4, 6144, False), architectures=["Qwen2MoeForCausalLM"], model_type="qwen2_moe", num_experts=64, num_experts_per_tok=8,
+    moe_intermediate_size=512, shared_expert_intermediate_size=512, norm_topk_prob=False, decoder_sparse_step=1, mlp_only_layers=[],
+)
 _VL_VISION = dict(
     depth=24, hidden_size=1024, num_heads=16, intermediate_size=4096, patch_size=16, temporal_patch_size=2,
     spatial_merge_size=2, in_channels=3, out_hidden_size=2048, num_position_embeddings=2304,

@@ -86,7 +86,7 @@ def test_latent_prologue(dtype, q_rank, kv_rank):
     qw, kw = 1 + _r(q_rank, seed=2, std=0.2), 1 + _r(max(kv_rank, 1), seed=3, std=0.2)
     loc = torch.randperm(S, generator=torch.Generator().manual_seed(4))[:T]
     cache = torch.full((S, kv_rank + 3), 7.0, dtype=dtype, device=DEV)
-    got = ops.latent_prologue(y.to(DEV), qw.to(DEV), kw.to(DEV) if kv_rank else None, 3e-5, loc.to(DEV) if kv_rank else None,
+    got, _ = ops.latent_prologue(y.to(DEV), qw.to(DEV), kw.to(DEV) if kv_rank else None, 3e-5, loc.to(DEV) if kv_rank else None,
                               cache[:, :kv_rank] if kv_rank else None)
     _close(got, oracle.rms_norm(oracle.f64(y[:, :q_rank]), oracle.f64(qw), 3e-5), _tol(dtype, 5e-3, 1e-6))
     if kv_rank:

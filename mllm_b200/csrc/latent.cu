@@ -153,7 +153,7 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const V* __restrict_
 constexpr int kHlTokTiles = 4;   // tiles of 8 tokens per CTA
 
 template <typename T, int KS>
-__global__ void __launch_bounds__(128) head_linear_kernel(const T* __restrict__ x, int64_t x_tok, int64_t x_head,
+__global__ void __launch_bounds__(KS > 1 ? KS * 32 : 128) head_linear_kernel(const T* __restrict__ x, int64_t x_tok, int64_t x_head,
                                                           const T* __restrict__ w, T* __restrict__ out, int64_t out_tok,
                                                           int64_t out_head, int tokens, int N, int K, const T* __restrict__ gate,
                                                           int64_t gate_ld, const float2* __restrict__ turns, int rot) {
@@ -166,7 +166,7 @@ __global__ void __launch_bounds__(128) head_linear_kernel(const T* __restrict__ 
   const int t0 = blockIdx.z * kHlTokTiles * 8;
   if (rot > 0 && blockIdx.x == gridDim.x - 1) {
     const int half = rot / 2, mine = min(tokens - t0, kHlTokTiles * 8);
-    for (int e = threadIdx.x; e < mine * half; e += 128) {
+    for (int e = threadIdx.x; e < mine * half; e += blockDim.x) {
       const int t = t0 + e / half, i = e % half;
       const T* src = x + t * x_tok + h * x_head + K + 2 * i;
       T* dst = out + t * out_tok + h * out_head + N + 2 * i;
@@ -177,7 +177,10 @@ __global__ void __launch_bounds__(128) head_linear_kernel(const T* __restrict__ 
     }
     return;
   }
-  auto gate_of = [&](int t) { return gate == nullptr ? 1.f : lat_sigmoid(to_f32(gate[t * gate_ld + h])); };
+  __shared__ float s_gate[kHlTokTiles * 8];
+  if (gate != nullptr && threadIdx.x < kHlTokTiles * 8)
+    s_gate[threadIdx.x] = t0 + static_cast<int>(threadIdx.x) < tokens ? lat_sigmoid(to_f32(gate[(t0 + threadIdx.x) * gate_ld + h])) : 0.f;
+  auto gate_of = [&](int t) { return gate == nullptr ? 1.f : s_gate[t - t0]; };      // after a barrier
   const int g = lane >> 2, q = lane & 3;
   float acc[kHlTokTiles][4];
 #pragma unroll
@@ -205,6 +208,7 @@ __global__ void __launch_bounds__(128) head_linear_kernel(const T* __restrict__ 
     }
   }
   // acc[i]: rows g and g + 8 of W, tokens i * 8 + 2 q and + 1
+  if (KS == 1 && gate != nullptr) __syncthreads();
   if constexpr (KS > 1) {
 #pragma unroll
     for (int i = 0; i < kHlTokTiles; ++i) {
@@ -214,7 +218,7 @@ __global__ void __launch_bounds__(128) head_linear_kernel(const T* __restrict__ 
       part[warp][i][g + 8][2 * q + 1] = acc[i][3];
     }
     __syncthreads();
-    for (int e = threadIdx.x; e < kHlTokTiles * 128; e += 128) {
+    for (int e = threadIdx.x; e < kHlTokTiles * 128; e += blockDim.x) {
       const int i = e >> 7, tok = (e >> 4) & 7, r = e & 15;
       const int t = t0 + i * 8 + tok;
       if (t < tokens && n0 + r < N) {
@@ -715,13 +719,14 @@ int launch_head_linear(const HeadLinearArgs& a, int num_sms, cudaStream_t s) {
   const int groups = (a.tokens + kHlTokTiles * 8 - 1) / (kHlTokTiles * 8), extra = a.rot > 0 ? 1 : 0;
   const bool split_k = static_cast<int64_t>(a.heads) * ((a.N + 63) / 64) * groups < num_sms && a.K >= 128;
   MB200_DISPATCH_HALF(a.dt, {
-    auto go = [&](auto kernel, int tiles) {
-      launch_pdl(kernel, dim3(tiles + extra, a.heads, groups), dim3(128), 0, s, static_cast<const T*>(a.x), a.x_tok, a.x_head,
+    auto go = [&](auto kernel, int tiles, int threads) {
+      launch_pdl(kernel, dim3(tiles + extra, a.heads, groups), dim3(threads), 0, s, static_cast<const T*>(a.x), a.x_tok, a.x_head,
                  static_cast<const T*>(a.w), static_cast<T*>(a.out), a.out_tok, a.out_head, a.tokens, a.N, a.K,
                  static_cast<const T*>(a.gate), a.gate_ld, a.turns, a.rot);
     };
-    if (split_k) go(head_linear_kernel<T, 4>, (a.N + 15) / 16);
-    else go(head_linear_kernel<T, 1>, (a.N + 63) / 64);
+    if (split_k && a.K >= 256) go(head_linear_kernel<T, 8>, (a.N + 15) / 16, 256);
+    else if (split_k) go(head_linear_kernel<T, 4>, (a.N + 15) / 16, 128);
+    else go(head_linear_kernel<T, 1>, (a.N + 63) / 64, 128);
   });
   note_launch();
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
@@ -730,7 +735,8 @@ int launch_head_linear(const HeadLinearArgs& a, int num_sms, cudaStream_t s) {
 int latent_num_splits(int rows, int heads, int max_seq_len, int num_sms) {
   const int ctas = std::max(1, rows * ((heads + 31) / 32));
   const int tiles = std::max(1, (max_seq_len + kLatTok - 1) / kLatTok);
-  const int splits = std::min(2 * num_sms / ctas, std::max(1, tiles / 4));   // two CTAs fit an SM
+  // two CTAs fit an SM; short contexts gain from every tile that runs beside another
+  const int splits = std::min(2 * num_sms / ctas, tiles <= 16 ? tiles : tiles / 2);
   return std::max(1, std::min(splits, 64));
 }
 

@@ -77,8 +77,34 @@ __global__ void moe_router_topk_kernel(const RouteArgs p) {
     const int e = lane + 32 * i;
     key[i] = e < experts ? v[i] + (p.correction != nullptr ? p.correction[e] : 0.f) : -INFINITY;
   }
-  if constexpr (GROUPS) {
-    const int size = experts / p.groups;
+  const int size = GROUPS ? experts / p.groups : 0;
+  if (GROUPS && size <= 32 && (size & (size - 1)) == 0) {
+    // groups are aligned runs of lanes
+    float score[NV];
+    int before[NV];               // groups that come first: a larger score, or the same and a lower index
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      float2 two = make_float2(key[i], -INFINITY);
+      for (int o = 1; o < size; o <<= 1)
+        two = top_two(two, make_float2(__shfl_xor_sync(0xffffffffu, two.x, o), __shfl_xor_sync(0xffffffffu, two.y, o)));
+      score[i] = size > 1 ? two.x + two.y : two.x;
+      before[i] = 0;
+    }
+#pragma unroll
+    for (int ii = 0; ii < NV; ++ii)
+      for (int l = 0; l < 32; l += size) {
+        const float other = __shfl_sync(0xffffffffu, score[ii], l);
+        const int at = ii * 32 + l;
+        if (at < experts) {
+#pragma unroll
+          for (int i = 0; i < NV; ++i)
+            before[i] += (other > score[i] || (other == score[i] && at < ((lane + 32 * i) & ~(size - 1)))) ? 1 : 0;
+        }
+      }
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+      if (before[i] >= p.keep) key[i] = -INFINITY;
+  } else if constexpr (GROUPS) {
     int mine[NV];                 // the group of each of the lane's experts
 #pragma unroll
     for (int i = 0; i < NV; ++i) mine[i] = (lane + 32 * i) / size;
@@ -103,34 +129,34 @@ __global__ void moe_router_topk_kernel(const RouteArgs p) {
     for (int i = 0; i < NV; ++i)
       if ((lane + 32 * i) < experts && ((open >> mine[i]) & 1u) == 0) key[i] = -INFINITY;
   }
+  // keys as integers of the same order; 0: no expert, closed or taken
+  unsigned order[NV];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const unsigned u = __float_as_uint(key[i]);
+    order[i] = key[i] == -INFINITY ? 0u : (u & 0x80000000u) ? ~u : u | 0x80000000u;
+  }
   float chosen_w = 0.f;  // lane j keeps the j-th choice
   int chosen_e = 0;
   float ksum = 0.f;
   for (int j = 0; j < top_k; ++j) {
-    float best = -INFINITY;
+    unsigned best = 0u;
     int bi = 0x7fffffff;
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-      if (key[i] > best) {  // ascending i: the lowest index wins ties inside a lane
-        best = key[i];
+      if (order[i] > best) {  // ascending i: the lowest index wins ties inside a lane
+        best = order[i];
         bi = lane + 32 * i;
       }
     }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ov = __shfl_xor_sync(0xffffffffu, best, o);
-      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-      if (ov > best || (ov == best && oi < bi)) {
-        best = ov;
-        bi = oi;
-      }
-    }
+    const unsigned most = __reduce_max_sync(0xffffffffu, best);
+    bi = static_cast<int>(__reduce_min_sync(0xffffffffu, best == most ? static_cast<unsigned>(bi) : 0x7fffffffu));
     float score = 0.f;
     if ((bi & 31) == lane) {
 #pragma unroll
       for (int i = 0; i < NV; ++i)
         if (i == (bi >> 5)) {
-          key[i] = -INFINITY;
+          order[i] = 0u;
           score = v[i];
         }
     }
@@ -183,31 +209,42 @@ __global__ void __launch_bounds__(kRlWarps * 32) moe_router_rows_kernel(const T*
   }
 }
 
-// prefill: 32 tokens x all experts (NT tiles of 8) per CTA, 128 features at a time through a ring; warps 0 and 1 take
-// the two row tiles of the lower 64 features of a step, warps 2 and 3 those of the upper, and the halves meet at the end
-constexpr int kRmTok = 32, kRmK = 128, kRmLd = kRmK + 8;
+// prefill: TT x 16 tokens x all experts (NT tiles of 8) per CTA, 128 features at a time through a ring; the first TT warps
+// take the row tiles of the lower 64 features of a step, the others those of the upper, and the halves meet at the end
+constexpr int kRmK = 128, kRmLd = kRmK + 8;
 constexpr int rm_stages(int nt) { return nt <= 16 ? 3 : 2; }
 
-template <typename T, int NT>
-__global__ void __launch_bounds__(128) moe_router_mma_kernel(const T* __restrict__ x, int64_t x_ld, const T* __restrict__ w,
-                                                             float* __restrict__ logits, int tokens, int experts, int hidden) {
+template <typename T, int NT, int TT>
+__global__ void __launch_bounds__(TT * 64) moe_router_mma_kernel(const T* __restrict__ x, int64_t x_ld, const T* __restrict__ w,
+                                                                 float* __restrict__ logits, int tokens, int experts, int hidden) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) uint8_t rm_smem[];
-  constexpr int kRmStages = rm_stages(NT);
-  constexpr int kRows = kRmTok + NT * 8;                 // token rows, then expert rows
+  constexpr int kRmStages = rm_stages(NT), kTok = TT * 16, kRmThreads = TT * 64;
+  constexpr int kRows = kTok + NT * 8;                   // token rows, then expert rows
+  constexpr int kStep = kRmThreads / (kRmK / 8);         // rows a pass of the CTA covers, 16 bytes per thread
+  static_assert(kTok % kStep == 0, "whole passes over the tokens");
   T* ring = reinterpret_cast<T*>(rm_smem);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int64_t t0 = static_cast<int64_t>(blockIdx.x) * kRmTok;
+  const int64_t t0 = static_cast<int64_t>(blockIdx.x) * kTok;
   const int steps = (hidden + kRmK - 1) / kRmK;
+  const int lr = tid / (kRmK / 8), lc = (tid % (kRmK / 8)) * 8;
+  const T* xp = x + (t0 + lr) * x_ld + lc;
+  const T* wp = w + static_cast<int64_t>(lr) * hidden + lc;
   auto load = [&](int step) {
-    T* dst = ring + (step % kRmStages) * kRows * kRmLd;
-    for (int i = tid; i < kRows * (kRmK / 8); i += 128) {
-      const int r = i / (kRmK / 8), c = (i % (kRmK / 8)) * 8, k = step * kRmK + c;
-      const bool tok = r < kRmTok;
-      const bool valid = k < hidden && (tok ? t0 + r < tokens : r - kRmTok < experts);
-      const T* src = tok ? x + (valid ? t0 + r : 0) * x_ld + (valid ? k : 0) : w + static_cast<int64_t>(valid ? r - kRmTok : 0) * hidden + (valid ? k : 0);
-      cp16_zfill(smem_u32(dst + r * kRmLd + c), src, valid);
+    T* dst = ring + ((step % kRmStages) * kRows + lr) * kRmLd + lc;
+    const int k0 = step * kRmK;
+    const bool okk = k0 + lc < hidden;
+#pragma unroll
+    for (int i = 0; i < kTok / kStep; ++i) {
+      const bool ok = okk && t0 + lr + i * kStep < tokens;
+      cp16_zfill(smem_u32(dst + i * kStep * kRmLd), ok ? xp + static_cast<int64_t>(i) * kStep * x_ld + k0 : x, ok);
+    }
+#pragma unroll
+    for (int i = 0; i < (NT * 8 + kStep - 1) / kStep; ++i) {
+      const bool ok = okk && lr + i * kStep < experts;
+      if ((i + 1) * kStep > NT * 8 && lr + i * kStep >= NT * 8) continue;      // behind the last tile
+      cp16_zfill(smem_u32(dst + (kTok + i * kStep) * kRmLd), ok ? wp + static_cast<int64_t>(i) * kStep * hidden + k0 : w, ok);
     }
     cp_commit();
   };
@@ -219,36 +256,37 @@ __global__ void __launch_bounds__(128) moe_router_mma_kernel(const T* __restrict
     if (i < steps) load(i);
     else cp_commit();
   }
+  const int rt = warp % TT, upper = warp / TT;
   for (int step = 0; step < steps; ++step) {
     cp_wait<kRmStages - 2>();
     __syncthreads();
     if (step + kRmStages - 1 < steps) load(step + kRmStages - 1);
     else cp_commit();
     const T* sx = ring + (step % kRmStages) * kRows * kRmLd;
-    const T* sw = sx + kRmTok * kRmLd;
+    const T* sw = sx + kTok * kRmLd;
 #pragma unroll
     for (int k16 = 0; k16 < kRmK / 2; k16 += 16) {
-      const int kk = (warp >> 1) * (kRmK / 2) + k16;
+      const int kk = upper * (kRmK / 2) + k16;
       uint32_t a[4];
-      ldsm4(a, smem_u32(sx + ((warp & 1) * 16 + (lane & 15)) * kRmLd + kk + (lane >> 4) * 8));
+      ldsm4(a, smem_u32(sx + (rt * 16 + (lane & 15)) * kRmLd + kk + (lane >> 4) * 8));
 #pragma unroll
       for (int n = 0; n < NT; n += 2) {
-        uint32_t b[4];      // two tiles of 8 experts: (lower, upper 8 features) of the first, then of the second
-        ldsm4(b, smem_u32(sw + (n * 8 + (lane >> 4) * 8 + (lane & 7)) * kRmLd + kk + ((lane >> 3) & 1) * 8));
+        uint32_t b[4];      // two tiles of 8 experts: (lower, upper 8 features) of the first, then of the second (or the first again)
+        ldsm4(b, smem_u32(sw + (n * 8 + (n + 1 < NT ? (lane >> 4) * 8 : 0) + (lane & 7)) * kRmLd + kk + ((lane >> 3) & 1) * 8));
         mma_16816<T>(acc[n], a[0], a[1], a[2], a[3], b[0], b[1]);
-        mma_16816<T>(acc[n + 1], a[0], a[1], a[2], a[3], b[2], b[3]);
+        if (n + 1 < NT) mma_16816<T>(acc[n + 1], a[0], a[1], a[2], a[3], b[2], b[3]);
       }
     }
   }
   cp_wait<0>();
   __syncthreads();                       // the ring is free: it takes the partial sums of the upper features
-  float* part = reinterpret_cast<float*>(rm_smem) + (warp & 1) * 32 * NT * 4;
-  if (warp >= 2) {
+  float* part = reinterpret_cast<float*>(rm_smem) + rt * 32 * NT * 4;
+  if (upper) {
 #pragma unroll
     for (int n = 0; n < NT; ++n) *reinterpret_cast<float4*>(part + (n * 32 + lane) * 4) = make_float4(acc[n][0], acc[n][1], acc[n][2], acc[n][3]);
   }
   __syncthreads();
-  if (warp >= 2) return;
+  if (upper) return;
 #pragma unroll
   for (int n = 0; n < NT; ++n) {
     const float4 o = *reinterpret_cast<const float4*>(part + (n * 32 + lane) * 4);
@@ -256,7 +294,7 @@ __global__ void __launch_bounds__(128) moe_router_mma_kernel(const T* __restrict
     const int e = n * 8 + (lane & 3) * 2;
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
-      const int64_t t = t0 + warp * 16 + (lane >> 2) + half * 8;
+      const int64_t t = t0 + rt * 16 + (lane >> 2) + half * 8;
       if (t < tokens) {
         if (e < experts) logits[t * experts + e] = sum[half * 2];
         if (e + 1 < experts) logits[t * experts + e + 1] = sum[half * 2 + 1];
@@ -265,15 +303,23 @@ __global__ void __launch_bounds__(128) moe_router_mma_kernel(const T* __restrict
   }
 }
 
-template <typename T, int NT>
-int launch_router_mma(const void* x, int64_t x_ld, const void* w, float* logits, int tokens, int experts, int hidden, cudaStream_t s) {
-  auto kern = moe_router_mma_kernel<T, NT>;
-  const int smem = rm_stages(NT) * (kRmTok + NT * 8) * kRmLd * static_cast<int>(sizeof(T));
+template <typename T, int NT, int TT>
+int launch_router_mma_tile(const void* x, int64_t x_ld, const void* w, float* logits, int tokens, int experts, int hidden, cudaStream_t s) {
+  auto kern = moe_router_mma_kernel<T, NT, TT>;
+  constexpr int smem = rm_stages(NT) * (TT * 16 + NT * 8) * kRmLd * static_cast<int>(sizeof(T));
+  static_assert(smem >= TT * 32 * NT * 16, "the partial sums fit the ring");
   if (ensure_dynamic_smem(reinterpret_cast<const void*>(kern), smem) != cudaSuccess) return -3;
-  const cudaError_t err = launch_pdl(kern, dim3((tokens + kRmTok - 1) / kRmTok), dim3(128), smem, s, static_cast<const T*>(x), x_ld,
+  const cudaError_t err = launch_pdl(kern, dim3((tokens + TT * 16 - 1) / (TT * 16)), dim3(TT * 64), smem, s, static_cast<const T*>(x), x_ld,
                                      static_cast<const T*>(w), logits, tokens, experts, hidden);
   note_launch();
   return err == cudaSuccess ? 0 : -4;
+}
+
+// 64 tokens a CTA halve the reads of the weights; few tokens spread over more CTAs of 32
+template <typename T, int NT>
+int launch_router_mma(const void* x, int64_t x_ld, const void* w, float* logits, int tokens, int experts, int hidden, cudaStream_t s) {
+  return tokens > 64 * 128 ? launch_router_mma_tile<T, NT, 4>(x, x_ld, w, logits, tokens, experts, hidden, s)
+                           : launch_router_mma_tile<T, NT, 2>(x, x_ld, w, logits, tokens, experts, hidden, s);
 }
 
 // the number of expert tiles is a compile-time loop bound: pairs of tiles up to 128 experts
@@ -284,7 +330,9 @@ int launch_router_mma_t(const void* x, int64_t x_ld, const void* w, float* logit
     case 2: return launch_router_mma<T, 4>(x, x_ld, w, logits, tokens, experts, hidden, s);
     case 3: return launch_router_mma<T, 6>(x, x_ld, w, logits, tokens, experts, hidden, s);
     case 4: return launch_router_mma<T, 8>(x, x_ld, w, logits, tokens, experts, hidden, s);
-    case 5: return launch_router_mma<T, 10>(x, x_ld, w, logits, tokens, experts, hidden, s);
+    case 5:       // nine tiles (64 outputs and a few more): three stages of two CTAs still fit an SM
+      return experts <= 72 ? launch_router_mma<T, 9>(x, x_ld, w, logits, tokens, experts, hidden, s)
+                           : launch_router_mma<T, 10>(x, x_ld, w, logits, tokens, experts, hidden, s);
     case 6: return launch_router_mma<T, 12>(x, x_ld, w, logits, tokens, experts, hidden, s);
     case 7: case 8: return launch_router_mma<T, 16>(x, x_ld, w, logits, tokens, experts, hidden, s);
     default: return launch_router_mma<T, 32>(x, x_ld, w, logits, tokens, experts, hidden, s);

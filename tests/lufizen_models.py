@@ -61,8 +61,9 @@ CONFIGS: Dict[str, dict] = {
 
 
 def weights(cfg: dict, seed: int = 0, steady: bool = False) -> Dict[str, torch.Tensor]:
-    """Values that bf16 holds exactly, scaled so that every mechanism shows in the logits.  ``steady``: corrections further
-    apart than any two scores, so that no rounding can turn a choice between experts."""
+    """Values that bf16 holds exactly, scaled so that every mechanism shows in the logits.  ``steady``: corrections
+    (and sums of two of them) further apart than any scores, so that no rounding can turn a choice between experts or
+    groups."""
     g = torch.Generator().manual_seed(seed)
     out: Dict[str, torch.Tensor] = {}
 
@@ -107,7 +108,7 @@ def weights(cfg: dict, seed: int = 0, steady: bool = False) -> Dict[str, torch.T
         from_stream(p + "router", r["experts"], 2.5)
         n(p + "correction", r["experts"], std=0.3)
         if steady:
-            out[p + "correction"] = (1.25 * torch.randperm(r["experts"], generator=g) - 5.0).to(torch.bfloat16)
+            out[p + "correction"] = (2.5 * 2.0 ** torch.randperm(r["experts"], generator=g)).to(torch.bfloat16)
         names = [f"e{e}" for e in range(r["experts"])] + (["shared"] if mlp.get("shared") else [])
         for name in names:
             ff = mlp["shared"]["ff"] if name == "shared" else mlp["expert"]["ff"]

@@ -176,22 +176,23 @@ def gdn(a) -> dict:
 
 
 def latent(a) -> dict:
-    """Decode of latent attention: `--batch` requests of `--seq` tokens, `--hq` heads over latents of `--rank` features."""
-    dev = "cuda"
+    """Decode of latent attention: `--batch` requests of `--seq` tokens, `--hq` heads over latents of `--rank` features and
+    a rotated key part of `--rot`."""
+    dev, key = "cuda", a.rank + a.rot
     table = (torch.arange(a.batch * a.seq, device=dev, dtype=torch.int32) + 16).view(a.batch, a.seq)
     req = torch.arange(a.batch, dtype=torch.int32, device=dev)
     pos = torch.full((a.batch,), a.seq - 1, dtype=torch.int64, device=dev)
-    caches = [torch.randn(a.batch * a.seq + 16, a.rank, device=dev, dtype=torch.bfloat16) for _ in range(max(1, a.kv_sets))]
-    q = torch.randn(a.batch, a.hq, a.rank, device=dev, dtype=torch.bfloat16) * a.rank ** -0.5
+    caches = [torch.randn(a.batch * a.seq + 16, key, device=dev, dtype=torch.bfloat16) for _ in range(max(1, a.kv_sets))]
+    q = torch.randn(a.batch, a.hq, key, device=dev, dtype=torch.bfloat16) * key ** -0.5
     sink = torch.zeros(a.hq, device=dev)
 
     def run():
         for c in caches:
-            ops.latent_attention(q, c, table, req, pos, 1.0, sink, a.seq)
+            ops.latent_attention(q, c, table, req, pos, 1.0, sink, a.seq, a.rank)
 
     ms = _time(run, a.iters) / len(caches)
-    return {"case": "latent", "batch": a.batch, "seq": a.seq, "heads": a.hq, "rank": a.rank, "ms": ms,
-            "gbs": a.batch * a.seq * a.rank * 2 / ms / 1e6, "tflops": 4 * a.batch * a.seq * a.hq * a.rank / ms / 1e9}
+    return {"case": "latent", "batch": a.batch, "seq": a.seq, "heads": a.hq, "rank": a.rank, "rot": a.rot, "ms": ms,
+            "gbs": a.batch * a.seq * key * 2 / ms / 1e6, "tflops": 2 * a.batch * a.seq * a.hq * (key + a.rank) / ms / 1e9}
 
 
 def lightning(a) -> dict:
@@ -222,7 +223,8 @@ def main() -> None:
     ap.add_argument("--seq", type=int, default=2050)
     ap.add_argument("--hq", type=int, default=32)
     ap.add_argument("--hkv", type=int, default=8)
-    ap.add_argument("--rank", type=int, default=512, help="latent: features of a cached row")
+    ap.add_argument("--rank", type=int, default=512, help="latent: features of a latent")
+    ap.add_argument("--rot", type=int, default=0, help="latent: features of the rotated key part behind it")
     ap.add_argument("--m", type=int, default=8)
     ap.add_argument("--n", type=int, default=4096)
     ap.add_argument("--k", type=int, default=4096)

@@ -45,17 +45,17 @@ CXX_FLAGS = ["-O3", "-std=c++17"]
 # the first number that is formatted into an error message crashes instead of raising
 LD_FLAGS = ["-l:libstdc++.so.6"]
 
-_COMMON = ["bindings_common.h", "common.cuh", "kernels.h", "mma.cuh"]
+_COMMON = ["bindings_common.h", "common.cuh", "kernels.h", "mma.cuh", "row.cuh"]
 
 EXTENSIONS: Dict[str, Dict[str, List[str]]] = {
     "mllm_b200_C": {
-        "sources": ["bindings.cpp", "runtime.cu", "elementwise.cu", "row_ops.cu", "gemm_tcgen05.cu", "gemm_smallm.cu", "attention.cu",
+        "sources": ["bindings.cpp", "runtime.cu", "elementwise.cu", "row_ops.cu", "depth.cu", "gemm_tcgen05.cu", "gemm_smallm.cu", "attention.cu",
                     "attention_rows.cu", "sampling.cu", "no_alloc.cu"],
         "headers": _COMMON + ["no_alloc.h"],
         "cuda": True,
     },
     "mllm_b200_R": {
-        "sources": ["bindings_recurrent.cpp", "runtime.cu", "gdn.cu", "gdn_chunk.cu"],
+        "sources": ["bindings_recurrent.cpp", "runtime.cu", "gdn.cu", "gdn_chunk.cu", "gdn_channel.cu"],
         "headers": _COMMON,
         "cuda": True,
     },

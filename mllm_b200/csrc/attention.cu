@@ -65,6 +65,7 @@ struct AttnParams {
   int out_f16;
   float scale_log2;        // softmax scale * log2(e)
   int window;              // sliding window: a query at position i sees keys i - window + 1 .. i (0 = everything)
+  int chunk;               // positions in chunks: a query at position i sees keys i / chunk * chunk .. i (0 = everything)
   float logit_cap;         // soft cap: score = cap * tanh(score / cap) before the softmax (0 = off)
   float scale;             // softmax scale (used with the soft cap)
   float cap_pre, cap_post; // soft cap: score in the log2 domain = cap_post * tanh(raw * cap_pre)
@@ -72,6 +73,12 @@ struct AttnParams {
   int kv_fmt;              // single-role kernel only: 1 / 2 = the caches hold unscaled e4m3 / e5m2 bytes
   uint32_t idesc_s, idesc_o;
 };
+
+// first key that a causal query at position i sees
+__device__ __forceinline__ int first_key(const AttnParams& p, int i) {
+  if (p.window > 0) return max(0, i - p.window + 1);
+  return p.chunk > 0 ? max(0, i / p.chunk * p.chunk) : 0;
+}
 
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool valid) {
   const int sz = valid ? 16 : 0;
@@ -147,7 +154,7 @@ __global__ void __launch_bounds__(kAttnThreads, FwdCfg<NH>::kCtasPerSm) attn_fwd
     q_len = 1;
     prefix = seq_len - 1;
     q_row0 = b;
-    const int lo = p.window > 0 ? max(0, seq_len - p.window) / kKV * kKV : 0;   // first tile the window touches
+    const int lo = first_key(p, seq_len - 1) / kKV * kKV;   // tile of the first key seen
     const int tiles = (seq_len - lo + kKV - 1) / kKV;
     const int per = (tiles + p.num_splits - 1) / p.num_splits;
     kv_begin = lo + blockIdx.x * per * kKV;
@@ -157,8 +164,8 @@ __global__ void __launch_bounds__(kAttnThreads, FwdCfg<NH>::kCtasPerSm) attn_fwd
     q_len = seq_len - prefix;
     q0 = blockIdx.x * p.tokens_per_tile;
     q_row0 = p.q_start[b];
-    // with a window the tile's first query row bounds the keys from below
-    kv_begin = (p.window > 0 && !p.non_causal) ? max(0, prefix + q0 - p.window + 1) / kKV * kKV : 0;
+    // the tile's first query row bounds the keys from below
+    kv_begin = p.non_causal ? 0 : first_key(p, prefix + q0) / kKV * kKV;
     kv_end = p.non_causal ? seq_len
                           : min(seq_len, prefix + min(q_len, q0 + p.tokens_per_tile));  // causal upper bound of the tile
     if (q0 >= q_len) return;
@@ -341,7 +348,7 @@ __global__ void __launch_bounds__(kAttnThreads, FwdCfg<NH>::kCtasPerSm) attn_fwd
     tmem_ld_wait();
     const int col0 = kv_begin + j * kKV;
     const int visible = min(kv_limit, kv_end - 1) - col0;  // columns 0..visible are allowed
-    const int first_vis = (p.window > 0 && !(p.non_causal && !p.is_decode)) ? kv_limit - p.window + 1 - col0 : -(1 << 30);
+    const int first_vis = p.non_causal && !p.is_decode ? -(1 << 30) : first_key(p, kv_limit) - col0;
     float sc[64];
     float m_tile = -INFINITY;
     if (p.logit_cap > 0.f) {   // uniform branch, kept outside the loop: the tanh must not be paid by plain scores
@@ -625,7 +632,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
 
   const int req = p.req_pool_indices[b];
   const int seq_len = p.seq_lens[b];
-  const int kv_lo = p.window > 0 ? max(0, seq_len - p.window) : 0;   // first key the (single) query sees
+  const int kv_lo = first_key(p, seq_len - 1);   // first key the (single) query sees
   const int lo_tile = kv_lo / kDT * kDT;
   const int tiles = (seq_len - lo_tile + kDT - 1) / kDT;
   const int per = (tiles + p.num_splits - 1) / p.num_splits;
@@ -1017,7 +1024,7 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
   const int q0 = (static_cast<int>(gridDim.x) - 1 - static_cast<int>(blockIdx.x)) * 2 * tpt;   // long rows first
   if (q0 >= q_len) return;
   const int q_row0 = p.q_start[b];
-  const int kv_begin = (p.window > 0 && !p.non_causal) ? max(0, prefix + q0 - p.window + 1) / kPfTile * kPfTile : 0;
+  const int kv_begin = p.non_causal ? 0 : first_key(p, prefix + q0) / kPfTile * kPfTile;
   const int kv_end = p.non_causal ? seq_len : min(seq_len, prefix + min(q_len, q0 + 2 * tpt));
   const int n_tiles = (kv_end - kv_begin + kPfTile - 1) / kPfTile;   // >= 1: the tile's first row sees itself
 
@@ -1223,7 +1230,7 @@ attn_prefill_ws_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
 
       const int col0 = kv_begin + t * kPfTile;
       const int visible = min(kv_limit, kv_end - 1) - col0;      // columns 0..visible are allowed
-      const int first_vis = (p.window > 0 && !p.non_causal) ? kv_limit - p.window + 1 - col0 : -(1 << 30);
+      const int first_vis = p.non_causal ? -(1 << 30) : first_key(p, kv_limit) - col0;
       const bool fast = __all_sync(0xffffffffu, plain_scores && visible >= kPfTile - 1 && first_vis <= 0);
       float mul = p.scale_log2;
       if (!fast) {
@@ -1531,6 +1538,7 @@ int launch_attention(const AttnArgs& a, cudaStream_t s) {
   p.scale_log2 = a.scale * kLog2e;
   p.scale = a.scale;
   p.window = a.window > 0 ? a.window : 0;
+  p.chunk = a.chunk > 0 ? a.chunk : 0;
   p.logit_cap = a.logit_cap > 0.f ? a.logit_cap : 0.f;
   p.cap_pre = p.logit_cap > 0.f ? a.scale / p.logit_cap : 0.f;
   p.cap_post = p.logit_cap * kLog2e;

@@ -26,7 +26,7 @@ __global__ void __launch_bounds__(kWarps * 32) attention_rows_kernel(const RowAt
   for (int i = lane; i < Dv; i += 32) acc[i] = 0.f;
   __syncwarp();
   const int64_t pos = p.row_pos[row];
-  const int64_t lo = p.window > 0 ? max(int64_t(0), pos - p.window + 1) : 0;
+  const int64_t lo = p.window > 0 ? max(int64_t(0), pos - p.window + 1) : p.chunk > 0 ? pos / p.chunk * p.chunk : 0;
   const int* table = p.req_to_token + static_cast<int64_t>(p.row_req[row]) * p.rtt_stride;
   float m = -INFINITY, l = 0.f;
   for (int64_t j0 = lo; j0 <= pos; j0 += 32) {

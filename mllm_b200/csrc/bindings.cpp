@@ -37,15 +37,15 @@ void layernorm(const Tensor& x, const Tensor& w, const c10::optional<Tensor>& b,
                           x.size(0), hidden, static_cast<float>(eps), dtype_of(x), stream_of(x));
 }
 
-void act_and_mul(const Tensor& x, Tensor& out, int64_t act) {
+void act_and_mul(const Tensor& x, Tensor& out, int64_t act, double limit) {
   check_cuda(x, "x");
   TORCH_CHECK(x.dim() == 2 && x.is_contiguous() && out.is_contiguous() && out.scalar_type() == x.scalar_type(),
               "act_and_mul: contiguous 2-D");
   const int inter = x.size(1) / 2;
   TORCH_CHECK(out.size(1) == inter && out.size(0) == x.size(0), "act_and_mul: width");
   c10::cuda::CUDAGuard g(x.device());
-  mb200::launch_act_and_mul(x.data_ptr(), out.data_ptr(), x.size(0), inter, static_cast<int>(act), dtype_of(x),
-                            stream_of(x));
+  mb200::launch_act_and_mul(x.data_ptr(), out.data_ptr(), x.size(0), inter, static_cast<int>(act), static_cast<float>(limit),
+                            dtype_of(x), stream_of(x));
 }
 
 void gelu_tanh(const Tensor& x, Tensor& out) {
@@ -326,6 +326,146 @@ void rmsnorm_sigmoid_gate(const Tensor& x, const Tensor& gate, const Tensor& w, 
   TORCH_CHECK(rc == 0, "rmsnorm_sigmoid_gate: row too wide (code ", rc, ")");
 }
 
+// x [T, W] contiguous, gate and out [T, W] with any row stride, w fp32 [W]; the mean is taken over each of `groups` parts
+void gated_rmsnorm(const Tensor& x, const Tensor& gate, const Tensor& w, Tensor& out, int64_t groups, double eps) {
+  check_float(x, "x");
+  TORCH_CHECK(x.dim() == 2 && x.is_contiguous() && gate.sizes() == x.sizes() && gate.stride(1) == 1 && out.sizes() == x.sizes() &&
+                  out.stride(1) == 1 && gate.scalar_type() == x.scalar_type() && out.scalar_type() == x.scalar_type() &&
+                  gate.is_cuda() && out.is_cuda() && groups >= 1 && x.size(1) % groups == 0,
+              "gated_rmsnorm: x, gate, out [T, W] of one type, equal groups");
+  check_f32_vec(w, x.size(1), "w");
+  c10::cuda::CUDAGuard g(x.device());
+  const int rc = mb200::launch_gated_rmsnorm(x.data_ptr(), gate.data_ptr(), gate.stride(0), w.data_ptr<float>(), out.data_ptr(), out.stride(0),
+                                             x.size(0), x.size(1), groups, static_cast<float>(eps), dtype_of(x), stream_of(x));
+  TORCH_CHECK(rc == 0, "gated_rmsnorm: row too wide (code ", rc, ")");
+}
+
+// outputs [h1] or [h1, h2] with their norm weights (one fp32 number each); conv: nothing, or [weight [W, K], state [rows, W,
+// K - 1], slots int32 [T]]
+static mb200::DepthInputs depth_inputs(const std::vector<Tensor>& h, const std::vector<Tensor>& g, const std::vector<Tensor>& conv, int64_t T,
+                                       int64_t W) {
+  TORCH_CHECK((h.size() == 1 || h.size() == 2) && g.size() == h.size(), "depth: one or two outputs, a norm weight for each");
+  for (const Tensor& t : h)
+    TORCH_CHECK(t.is_cuda() && t.is_contiguous() && t.dim() == 2 && t.size(0) == T && t.size(1) == W && t.scalar_type() == h[0].scalar_type(),
+                "depth: outputs [T, W] of one type");
+  for (const Tensor& t : g) check_f32_vec(t, 1, "norm weight");
+  mb200::DepthInputs a{};
+  a.h1 = h[0].data_ptr();
+  a.g1 = g[0].data_ptr<float>();
+  if (h.size() == 2) {
+    a.h2 = h[1].data_ptr();
+    a.g2 = g[1].data_ptr<float>();
+  }
+  if (!conv.empty()) {
+    TORCH_CHECK(conv.size() == 3, "depth: weight, state and slots of the convolution");
+    const Tensor &w = conv[0], &st = conv[1], &slots = conv[2];
+    TORCH_CHECK(w.is_cuda() && w.is_contiguous() && w.dim() == 2 && w.size(0) == W && w.size(1) >= 1 && w.scalar_type() == h[0].scalar_type() &&
+                    st.is_cuda() && st.is_contiguous() && st.dim() == 3 && st.size(1) == W && st.size(2) == w.size(1) - 1 &&
+                    st.scalar_type() == w.scalar_type() && slots.is_cuda() && slots.is_contiguous() && slots.scalar_type() == at::kInt &&
+                    slots.numel() == T,
+                "depth: weight [W, K], state [rows, W, K - 1], int32 slots [T]");
+    a.conv.w = w.data_ptr();
+    a.conv.state = st.data_ptr();
+    a.conv.slots = slots.data_ptr<int>();
+    a.conv.taps = w.size(1);
+  }
+  return a;
+}
+
+// x fp32 [T, W]; results: nothing or fp32 [>= n + keep, T, W] with dwa [n + 1]; mix: [a] or [a, b, a_w, b_w]; f [T, W] or nothing;
+// experts: nothing or [rows, sorted_pos, (topk_w)]
+void depth_step(const Tensor& x, const c10::optional<Tensor>& x_out, const c10::optional<Tensor>& results, int64_t n, bool keep,
+                const c10::optional<Tensor>& dwa, const std::vector<Tensor>& mix, double mix_scale, const c10::optional<Tensor>& f,
+                const std::vector<Tensor>& experts, int64_t top, double eps, const std::vector<Tensor>& h, const std::vector<Tensor>& g,
+                const std::vector<Tensor>& conv) {
+  TORCH_CHECK(x.is_cuda() && x.scalar_type() == at::kFloat && x.dim() == 2 && x.is_contiguous(), "depth_step: x fp32 [T, W]");
+  const int64_t T = x.size(0), W = x.size(1);
+  mb200::DepthStepArgs a{};
+  a.in = depth_inputs(h, g, conv, T, W);
+  check_float(h[0], "h");
+  const auto row_like = [&](const Tensor& t, const char* name) {
+    TORCH_CHECK(t.is_cuda() && t.is_contiguous() && t.dim() == 2 && t.size(0) == T && t.size(1) == W && t.scalar_type() == h[0].scalar_type(),
+                "depth_step: ", name, " [T, W] of the outputs' type");
+    return t.data_ptr();
+  };
+  TORCH_CHECK(mix.size() == 1 || mix.size() == 4, "depth_step: one mixer output, or two with their norm weights");
+  a.a = row_like(mix[0], "mixer output");
+  if (mix.size() == 4) {
+    a.b = row_like(mix[1], "second mixer output");
+    check_f32_vec(mix[2], W, "norm weight of the first output");
+    check_f32_vec(mix[3], W, "norm weight of the second output");
+    a.a_w = mix[2].data_ptr<float>();
+    a.b_w = mix[3].data_ptr<float>();
+  }
+  if (f.has_value()) a.f = row_like(*f, "feed-forward output");
+  if (x_out.has_value()) {
+    TORCH_CHECK(x_out->is_cuda() && x_out->scalar_type() == at::kFloat && x_out->is_contiguous() && x_out->sizes() == x.sizes(),
+                "depth_step: x_out fp32 [T, W]");
+    a.x_out = x_out->data_ptr<float>();
+  }
+  if (dwa.has_value()) {
+    check_f32_vec(*dwa, n + 1, "dwa");
+    TORCH_CHECK(results.has_value() && results->is_cuda() && results->scalar_type() == at::kFloat && results->is_contiguous() &&
+                    results->dim() == 3 && results->size(0) >= n + (keep ? 1 : 0) && results->size(1) == T && results->size(2) == W && n >= 0,
+                "depth_step: results fp32 [>= n (+ 1), T, W]");
+    a.dwa = dwa->data_ptr<float>();
+    a.results = results->data_ptr<float>();
+    a.result_stride = T * W;
+    a.n = n;
+    a.keep = keep ? 1 : 0;
+  }
+  if (!experts.empty()) {
+    const Tensor &rows = experts[0], &pos = experts[1];
+    TORCH_CHECK(experts.size() >= 2 && top >= 1 && top <= 32 && rows.is_cuda() && rows.is_contiguous() && rows.dim() == 2 && rows.size(1) == W &&
+                    rows.scalar_type() == h[0].scalar_type() && rows.size(0) >= 1 && pos.is_cuda() && pos.scalar_type() == at::kInt &&
+                    pos.is_contiguous() && pos.numel() >= T * top,
+                "depth_step: expert rows [pairs, W], row of every choice int32 [T * top]");
+    a.expert_rows = rows.data_ptr();
+    a.sorted_pos = pos.data_ptr<int>();
+    a.top = top;
+    if (experts.size() > 2) {
+      check_f32_vec(experts[2], T * top, "topk_w");
+      a.topk_w = experts[2].data_ptr<float>();
+    }
+  }
+  c10::cuda::CUDAGuard guard(x.device());
+  a.x = x.data_ptr<float>();
+  a.mix_scale = static_cast<float>(mix_scale);
+  a.rows = T;
+  a.width = W;
+  a.eps = static_cast<float>(eps);
+  a.dt = dtype_of(h[0]);
+  const int rc = mb200::launch_depth_step(a, stream_of(x));
+  TORCH_CHECK(rc == 0, "depth_step: row too wide or too many choices or taps (code ", rc, ")");
+}
+
+// x fp32 [T, W] = normed embedding rows of ids, h = the inputs of the first layer
+void embed_norm(const Tensor& ids, const Tensor& table, const Tensor& weight, Tensor& x, double eps, const std::vector<Tensor>& h,
+                const std::vector<Tensor>& g, const std::vector<Tensor>& conv) {
+  check_float(table, "table");
+  const int64_t T = ids.numel(), W = table.size(1);
+  TORCH_CHECK(ids.is_cuda() && ids.scalar_type() == at::kLong && ids.is_contiguous() && table.is_contiguous() && table.dim() == 2 && x.is_cuda() &&
+                  x.scalar_type() == at::kFloat && x.is_contiguous() && x.dim() == 2 && x.size(0) == T && x.size(1) == W,
+              "embed_norm: int64 ids [T], table [vocab, W], x fp32 [T, W]");
+  check_f32_vec(weight, 1, "weight");
+  mb200::EmbedNormArgs a{};
+  a.in = depth_inputs(h, g, conv, T, W);
+  TORCH_CHECK(h[0].scalar_type() == table.scalar_type(), "embed_norm: outputs of the table's type");
+  c10::cuda::CUDAGuard guard(table.device());
+  a.ids = ids.data_ptr<int64_t>();
+  a.table = table.data_ptr();
+  a.g = weight.data_ptr<float>();
+  a.x = x.data_ptr<float>();
+  a.status = device_state(table.get_device()).status.data_ptr<int>();
+  a.rows = T;
+  a.width = W;
+  a.vocab = table.size(0);
+  a.eps = static_cast<float>(eps);
+  a.dt = dtype_of(table);
+  const int rc = mb200::launch_embed_norm(a, stream_of(table));
+  TORCH_CHECK(rc == 0, "embed_norm: row too wide or too many taps (code ", rc, ")");
+}
+
 // row [T, >= (heads + kv_heads) * dim + kv_heads * vdim]; q_out [T, heads, q_width]; caches [slots, kv_heads, >= width]
 void rownorm_rope_kv(const Tensor& row, const Tensor& q_w, const Tensor& k_w, const Tensor& inv_freq, const Tensor& positions,
                      const Tensor& loc, Tensor& q_out, Tensor& k_cache, Tensor& v_cache, int64_t heads, int64_t kv_heads, int64_t dim,
@@ -380,7 +520,8 @@ void rownorm_rope_kv(const Tensor& row, const Tensor& q_w, const Tensor& k_w, co
 
 // row [T, >= (heads + kv_heads) * dim] with values at column v_at; q_out [T, heads, q_width]; caches [slots, kv_heads, >= width]
 void headnorm_rope_kv(const Tensor& row, const Tensor& inv_freq, const Tensor& positions, const Tensor& loc, Tensor& q_out, Tensor& k_cache,
-                      Tensor& v_cache, int64_t heads, int64_t kv_heads, int64_t dim, int64_t vdim, int64_t v_at, bool halves, double eps) {
+                      Tensor& v_cache, int64_t heads, int64_t kv_heads, int64_t dim, int64_t vdim, int64_t v_at, bool halves, double eps,
+                      bool norm, double magnitude) {
   check_float(row, "row");
   const int64_t T = row.size(0);
   TORCH_CHECK(row.dim() == 2 && row.stride(1) == 1 && row.size(1) >= (heads + kv_heads) * dim && v_at >= 0 &&
@@ -421,6 +562,8 @@ void headnorm_rope_kv(const Tensor& row, const Tensor& inv_freq, const Tensor& p
   a.q_width = q_out.size(2);
   a.rot_dims = 2 * inv_freq.numel();
   a.halves = halves ? 1 : 0;
+  a.norm = norm ? 1 : 0;
+  a.magnitude = static_cast<float>(magnitude);
   a.eps = static_cast<float>(eps);
   a.dt = dtype_of(row);
   const int rc = mb200::launch_headnorm_rope_kv(a, stream_of(row));
@@ -447,7 +590,7 @@ void relu_squared(Tensor& x) {
 
 // q [rows, H, D] and out [rows, H, Dv] with any row stride; caches [slots, G, D / Dv]
 void attention_rows(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& req_to_token, const Tensor& row_req,
-                    const Tensor& row_pos, double scale, Tensor& out, int64_t window, double logit_cap, const c10::optional<Tensor>& sink) {
+                    const Tensor& row_pos, double scale, Tensor& out, int64_t window, double logit_cap, const c10::optional<Tensor>& sink, int64_t chunk) {
   check_float(q, "q");
   TORCH_CHECK(q.dim() == 3 && q.stride(2) == 1 && q.stride(1) == q.size(2) && out.dim() == 3 && out.stride(2) == 1 &&
                   out.stride(1) == out.size(2) && out.size(0) == q.size(0) && out.size(1) == q.size(1) &&
@@ -490,6 +633,7 @@ void attention_rows(const Tensor& q, const Tensor& k_cache, const Tensor& v_cach
   a.dim = q.size(2);
   a.vdim = out.size(2);
   a.window = static_cast<int>(window);
+  a.chunk = static_cast<int>(chunk);
   a.scale = static_cast<float>(scale);
   a.logit_cap = static_cast<float>(logit_cap);
   a.dt = dtype_of(q);
@@ -519,7 +663,7 @@ struct NormFusion {
 int64_t gemm_impl(const Tensor& a, const Tensor& b, Tensor& out, const c10::optional<Tensor>& bias,
                   const c10::optional<Tensor>& residual, int64_t swiglu, const c10::optional<Tensor>& a_scale,
                   const c10::optional<Tensor>& b_scale, const TpFusion* tp, bool b_static = false,
-                  const NormFusion* norm = nullptr) {
+                  const NormFusion* norm = nullptr, double act_limit = 0.0) {
   check_cuda(a, "a");
   check_cuda(b, "b");
   const bool is_int8 = a.scalar_type() == at::kChar;
@@ -527,7 +671,7 @@ int64_t gemm_impl(const Tensor& a, const Tensor& b, Tensor& out, const c10::opti
                   out.stride(1) == 1,
               "gemm: 2-D row-major operands");
   TORCH_CHECK(a.size(1) == b.size(1) && a.scalar_type() == b.scalar_type(), "gemm: K / dtype mismatch");
-  TORCH_CHECK(out.size(0) == a.size(0) && out.size(1) == (swiglu == 1 || swiglu == 2 ? b.size(0) / 2 : b.size(0)), "gemm: out shape");
+  TORCH_CHECK(out.size(0) == a.size(0) && out.size(1) == (swiglu == 1 || swiglu == 2 || swiglu == 4 ? b.size(0) / 2 : b.size(0)), "gemm: out shape");
   if (is_int8) {
     TORCH_CHECK(a_scale.has_value() && b_scale.has_value(), "gemm: int8 needs scales");
     TORCH_CHECK(a_scale->scalar_type() == at::kFloat && b_scale->scalar_type() == at::kFloat &&
@@ -562,7 +706,8 @@ int64_t gemm_impl(const Tensor& a, const Tensor& b, Tensor& out, const c10::opti
   args.ldb = b.stride(0);
   args.ldc = out.stride(0);
   args.ld_res = residual.has_value() ? residual->stride(0) : 0;
-  args.swiglu = static_cast<int>(swiglu);   // 1: SiLU gate, 2: GELU (tanh form) gate, 3: square of relu
+  args.swiglu = static_cast<int>(swiglu);   // 1: SiLU gate, 2: GELU (tanh form) gate, 3: square of relu, 4: bounded gated unit
+  args.act_limit = static_cast<float>(act_limit);
   args.dt = dtype_of(out);
   args.is_int8 = is_int8 ? 1 : 0;
   args.workspace = st.workspace.data_ptr<float>();
@@ -614,8 +759,8 @@ int64_t gemm_impl(const Tensor& a, const Tensor& b, Tensor& out, const c10::opti
 // start streaming them before the kernels in front of this launch have finished.
 int64_t gemm(const Tensor& a, const Tensor& b, Tensor& out, const c10::optional<Tensor>& bias,
              const c10::optional<Tensor>& residual, int64_t swiglu, const c10::optional<Tensor>& a_scale,
-             const c10::optional<Tensor>& b_scale, bool b_static) {
-  return gemm_impl(a, b, out, bias, residual, swiglu, a_scale, b_scale, nullptr, b_static);
+             const c10::optional<Tensor>& b_scale, bool b_static, double act_limit) {
+  return gemm_impl(a, b, out, bias, residual, swiglu, a_scale, b_scale, nullptr, b_static, nullptr, act_limit);
 }
 
 // out = (rmsnorm(a + residual) * norm_weight) b^T [+ bias | SwiGLU] for up to 8 rows, with a + residual (rounded to
@@ -676,7 +821,7 @@ static const float* sink_ptr(const c10::optional<Tensor>& sink, int64_t heads) {
 void attention_prefill(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& req_to_token,
                        const Tensor& req_pool_indices, const Tensor& seq_lens, const Tensor& prefix_lens,
                        const Tensor& q_start, double scale, Tensor& out, int64_t max_q_len, bool causal, int64_t window,
-                       double logit_cap, const c10::optional<Tensor>& sink) {
+                       double logit_cap, const c10::optional<Tensor>& sink, int64_t chunk) {
   check_half(q, "q");
   TORCH_CHECK(q.dim() == 3, "q must be [T,Hq,D]");
   const int64_t hd = q.size(2);
@@ -718,6 +863,7 @@ void attention_prefill(const Tensor& q, const Tensor& k_cache, const Tensor& v_c
   a.non_causal = causal ? 0 : 1;
   a.scale = static_cast<float>(scale);
   a.window = static_cast<int>(window);
+  a.chunk = static_cast<int>(chunk);
   a.logit_cap = static_cast<float>(logit_cap);
   a.sink = sink_ptr(sink, a.hq);
   a.dt = dtype_of(q);
@@ -727,7 +873,7 @@ void attention_prefill(const Tensor& q, const Tensor& k_cache, const Tensor& v_c
 
 void attention_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& req_to_token,
                       const Tensor& req_pool_indices, const Tensor& seq_lens, double scale, Tensor& out,
-                      int64_t max_seq_len, int64_t window, double logit_cap, const c10::optional<Tensor>& sink) {
+                      int64_t max_seq_len, int64_t window, double logit_cap, const c10::optional<Tensor>& sink, int64_t chunk) {
   check_half(q, "q");
   TORCH_CHECK(q.dim() == 3, "q must be [B,Hq,D]");
   const int64_t hd = q.size(2);
@@ -746,7 +892,8 @@ void attention_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_ca
   a.hq = q.size(1);
   a.hkv = k_cache.size(1);
   int64_t longest = max_seq_len > 0 ? max_seq_len : req_to_token.size(1);
-  if (window > 0) longest = std::min(longest, window + 128);     // keys read, up to the tiles' alignment
+  const int64_t seen = window > 0 ? window : chunk;
+  if (seen > 0) longest = std::min(longest, seen + 128);     // keys read, up to the tiles' alignment
   a.num_splits = mb200::decode_num_splits(a.batch, a.hkv, longest, st.num_sms);
   Tensor part_o, part_lse;
   if (a.num_splits > 1) {
@@ -774,6 +921,7 @@ void attention_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_ca
   a.is_decode = 1;
   a.scale = static_cast<float>(scale);
   a.window = static_cast<int>(window);
+  a.chunk = static_cast<int>(chunk);
   a.logit_cap = static_cast<float>(logit_cap);
   a.sink = sink_ptr(sink, a.hq);
   a.dt = dtype_of(q);
@@ -787,7 +935,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("rmsnorm", &rmsnorm);
   m.def("fused_add_rmsnorm", &fused_add_rmsnorm);
   m.def("layernorm", &layernorm);
-  m.def("act_and_mul", &act_and_mul);
+  m.def("act_and_mul", &act_and_mul, py::arg("x"), py::arg("out"), py::arg("act"), py::arg("limit") = 0.0);
   m.def("gelu_tanh", &gelu_tanh);
   m.def("embedding", &embedding);
   m.def("qk_norm_rope_kv_write", &qk_norm_rope_kv_write);
@@ -797,7 +945,8 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("sample", &sample);
   m.def("apply_penalties", &apply_penalties);
   m.def("decode_prepare", &decode_prepare);
-  m.def("gemm", &gemm);
+  m.def("gemm", &gemm, py::arg("a"), py::arg("b"), py::arg("out"), py::arg("bias"), py::arg("residual"), py::arg("swiglu"),
+        py::arg("a_scale"), py::arg("b_scale"), py::arg("b_static"), py::arg("act_limit") = 0.0);
   m.def("gemm_norm", &gemm_norm);
   m.def("gemm_tp", &gemm_tp);
   m.def("residual_dyt", &residual_dyt);
@@ -806,17 +955,24 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
         py::arg("update"), py::arg("experts"), py::arg("identity_from"), py::arg("inner") = false, py::arg("y_logit") = py::none());
   m.def("rmsnorm_sigmoid_gate", &rmsnorm_sigmoid_gate);
   m.def("rownorm_rope_kv", &rownorm_rope_kv);
-  m.def("headnorm_rope_kv", &headnorm_rope_kv);
+  m.def("headnorm_rope_kv", &headnorm_rope_kv, py::arg("row"), py::arg("inv_freq"), py::arg("positions"), py::arg("loc"), py::arg("q_out"),
+        py::arg("k_cache"), py::arg("v_cache"), py::arg("heads"), py::arg("kv_heads"), py::arg("dim"), py::arg("vdim"), py::arg("v_at"),
+        py::arg("halves"), py::arg("eps"), py::arg("norm") = true, py::arg("magnitude") = 1.0);
+  m.def("gated_rmsnorm", &gated_rmsnorm);
+  m.def("depth_step", &depth_step);
+  m.def("embed_norm", &embed_norm);
   m.def("soft_cap", &soft_cap);
   m.def("relu_squared", &relu_squared);
-  m.def("attention_rows", &attention_rows);
+  m.def("attention_rows", &attention_rows, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("req_to_token"),
+        py::arg("row_req"), py::arg("row_pos"), py::arg("scale"), py::arg("out"), py::arg("window"), py::arg("logit_cap"),
+        py::arg("sink") = py::none(), py::arg("chunk") = 0);
   m.def("attention_prefill", &attention_prefill, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("req_to_token"),
         py::arg("req_pool_indices"), py::arg("seq_lens"), py::arg("prefix_lens"), py::arg("q_start"), py::arg("scale"),
         py::arg("out"), py::arg("max_q_len"), py::arg("causal"), py::arg("window"), py::arg("logit_cap"),
-        py::arg("sink") = py::none());
+        py::arg("sink") = py::none(), py::arg("chunk") = 0);
   m.def("attention_decode", &attention_decode, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("req_to_token"),
         py::arg("req_pool_indices"), py::arg("seq_lens"), py::arg("scale"), py::arg("out"), py::arg("max_seq_len"),
-        py::arg("window"), py::arg("logit_cap"), py::arg("sink") = py::none());
+        py::arg("window"), py::arg("logit_cap"), py::arg("sink") = py::none(), py::arg("chunk") = 0);
   m.def("read_status", &read_status);
   m.def("launch_count", &launch_count);
 }

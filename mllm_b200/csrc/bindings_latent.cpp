@@ -11,18 +11,26 @@ void check_turns(const Tensor& turns, int64_t tokens) {
 }
 float2* turns_ptr(const Tensor& t) { return reinterpret_cast<float2*>(t.data_ptr<float>()); }
 
-// y [T, q_rank (+ kv_rank) (+ rot)]; cq [T, q_rank]; cache [slots, kv_rank + rot] and loc only when the layer writes latents;
+// y [T, q_rank (+ kv_rank) (+ rot)]; q_w and cq [T, q_rank] only where queries have a latent; cache [slots, kv_rank + rot] and loc only when the layer writes latents;
 // positions int64 [T], inv_freq fp64 [rot / 2] and turns only with a rotated key part
-void latent_prologue(const Tensor& y, const Tensor& q_w, const c10::optional<Tensor>& kv_w, double eps, Tensor& cq,
+void latent_prologue(const Tensor& y, const c10::optional<Tensor>& q_w, const c10::optional<Tensor>& kv_w, double eps,
+                     const c10::optional<Tensor>& cq,
                      const c10::optional<Tensor>& loc, const c10::optional<Tensor>& cache, const c10::optional<Tensor>& positions,
-                     const c10::optional<Tensor>& inv_freq, const c10::optional<Tensor>& turns) {
+                     const c10::optional<Tensor>& inv_freq, const c10::optional<Tensor>& turns, bool halves) {
   check_float(y, "y");
-  const int64_t q_rank = q_w.numel(), kv_rank = kv_w.has_value() ? kv_w->numel() : 0, rot = inv_freq.has_value() ? 2 * inv_freq->numel() : 0;
-  TORCH_CHECK(y.dim() == 2 && y.stride(1) == 1 && y.size(1) >= q_rank + kv_rank + (kv_rank > 0 ? rot : 0) && cq.is_contiguous() &&
-                  cq.dim() == 2 && cq.size(0) == y.size(0) && cq.size(1) == q_rank && cq.scalar_type() == y.scalar_type() && cq.is_cuda(),
-              "latent_prologue: y [T, q_rank + kv_rank + rot], cq [T, q_rank]");
-  check_f32_vec(q_w, q_rank, "q_w");
+  const int64_t q_rank = q_w.has_value() ? q_w->numel() : 0, kv_rank = kv_w.has_value() ? kv_w->numel() : 0, rot = inv_freq.has_value() ? 2 * inv_freq->numel() : 0;
+  TORCH_CHECK(y.dim() == 2 && y.stride(1) == 1 && y.size(1) >= q_rank + kv_rank + (kv_rank > 0 ? rot : 0) &&
+                  cq.has_value() == q_w.has_value(),
+              "latent_prologue: y [T, q_rank + kv_rank + rot]");
   mb200::LatentPrologueArgs a{};
+  if (q_rank > 0) {
+    check_f32_vec(*q_w, q_rank, "q_w");
+    TORCH_CHECK(cq->is_contiguous() && cq->dim() == 2 && cq->size(0) == y.size(0) && cq->size(1) == q_rank &&
+                    cq->scalar_type() == y.scalar_type() && cq->is_cuda(),
+                "latent_prologue: cq [T, q_rank]");
+    a.q_w = q_w->data_ptr<float>();
+    a.cq = cq->data_ptr();
+  }
   if (kv_rank > 0) {
     check_f32_vec(*kv_w, kv_rank, "kv_w");
     TORCH_CHECK(loc.has_value() && cache.has_value() && loc->is_cuda() && loc->scalar_type() == at::kLong && loc->is_contiguous() &&
@@ -48,8 +56,7 @@ void latent_prologue(const Tensor& y, const Tensor& q_w, const c10::optional<Ten
   }
   c10::cuda::CUDAGuard g(y.device());
   a.y = y.data_ptr();
-  a.q_w = q_w.data_ptr<float>();
-  a.cq = cq.data_ptr();
+  a.halves = halves ? 1 : 0;
   a.status = device_state(y.get_device()).status.data_ptr<int>();
   a.ld = y.stride(0);
   a.tokens = y.size(0);
@@ -62,7 +69,7 @@ void latent_prologue(const Tensor& y, const Tensor& q_w, const c10::optional<Ten
 }
 
 // x, out [T, H, rot] with any token and head strides (out may be x)
-void turn_heads(const Tensor& x, const Tensor& turns, Tensor& out) {
+void turn_heads(const Tensor& x, const Tensor& turns, Tensor& out, bool halves) {
   check_float(x, "x");
   check_turns(turns, x.size(0));
   TORCH_CHECK(x.dim() == 3 && x.stride(2) == 1 && out.sizes() == x.sizes() && out.stride(2) == 1 && out.is_cuda() &&
@@ -70,23 +77,24 @@ void turn_heads(const Tensor& x, const Tensor& turns, Tensor& out) {
               "turn_heads: x, out [T, H, rot]");
   c10::cuda::CUDAGuard g(x.device());
   mb200::launch_turn_heads(x.data_ptr(), x.stride(0), x.stride(1), turns_ptr(turns), out.data_ptr(), out.stride(0), out.stride(1), x.size(0),
-                           x.size(1), x.size(2), dtype_of(x), stream_of(x));
+                           x.size(1), x.size(2), halves ? 1 : 0, dtype_of(x), stream_of(x));
 }
 
-// x [T, H, W] with any token and head strides, gate [T, H] with any row stride, out [T, H, W] contiguous
+// x, out [T, H, W] with any token and head strides (out may be x), gate [T, H] or [T, H * W] with any row stride
 void gate_heads(const Tensor& x, const Tensor& gate, Tensor& out) {
   check_float(x, "x");
+  const bool per_feature = gate.dim() == 2 && gate.size(1) != x.size(1);
   TORCH_CHECK(x.dim() == 3 && x.stride(2) == 1 && gate.is_cuda() && gate.dim() == 2 && gate.stride(1) == 1 && gate.size(0) == x.size(0) &&
-                  gate.size(1) == x.size(1) && gate.scalar_type() == x.scalar_type() && out.is_cuda() && out.is_contiguous() &&
-                  out.sizes() == x.sizes() && out.scalar_type() == x.scalar_type(),
-              "gate_heads: x, out [T, H, W], gate [T, H]");
+                  (!per_feature || gate.size(1) == x.size(1) * x.size(2)) && gate.scalar_type() == x.scalar_type() && out.is_cuda() &&
+                  out.stride(2) == 1 && out.sizes() == x.sizes() && out.scalar_type() == x.scalar_type(),
+              "gate_heads: x, out [T, H, W], gate [T, H] or [T, H * W]");
   c10::cuda::CUDAGuard g(x.device());
-  mb200::launch_gate_heads(x.data_ptr(), x.stride(0), x.stride(1), gate.data_ptr(), gate.stride(0), out.data_ptr(), x.size(0), x.size(1),
-                           x.size(2), dtype_of(x), stream_of(x));
+  mb200::launch_gate_heads(x.data_ptr(), x.stride(0), x.stride(1), gate.data_ptr(), gate.stride(0), out.data_ptr(), out.stride(0), out.stride(1),
+                           x.size(0), x.size(1), x.size(2), per_feature ? 1 : 0, dtype_of(x), stream_of(x));
 }
 
 void latent_gather(const Tensor& cache, const Tensor& req_to_token, const Tensor& req, const Tensor& lens, const Tensor& start,
-                   int64_t max_len, Tensor& out) {
+                   int64_t max_len, Tensor& out, const c10::optional<Tensor>& first) {
   check_float(cache, "cache");
   for (const Tensor* t : {&req_to_token, &req, &lens, &start})
     TORCH_CHECK(t->scalar_type() == at::kInt && t->is_cuda(), "latent_gather: index tensors must be int32 CUDA tensors");
@@ -94,16 +102,21 @@ void latent_gather(const Tensor& cache, const Tensor& req_to_token, const Tensor
                   max_len <= req_to_token.size(1) && req.numel() == lens.numel() && req.numel() == start.numel() &&
                   out.is_contiguous() && out.dim() == 2 && out.size(1) == cache.size(1) && out.scalar_type() == cache.scalar_type(),
               "latent_gather: cache [slots, rank], out [rows, rank]");
+  if (first.has_value())
+    TORCH_CHECK(first->is_cuda() && first->scalar_type() == at::kInt && first->is_contiguous() && first->numel() == req.numel(),
+                "latent_gather: first int32 [requests]");
   c10::cuda::CUDAGuard g(cache.device());
   auto& st = device_state(cache.get_device());
   mb200::launch_latent_gather(cache.data_ptr(), cache.stride(0), cache.size(1), cache.element_size(), req_to_token.data_ptr<int>(),
-                              req_to_token.stride(0), req.data_ptr<int>(), lens.data_ptr<int>(), start.data_ptr<int>(), req.numel(),
+                              req_to_token.stride(0), req.data_ptr<int>(), lens.data_ptr<int>(), start.data_ptr<int>(),
+                              first.has_value() ? first->data_ptr<int>() : nullptr, req.numel(),
                               max_len, out.data_ptr(), cache.size(0), st.status.data_ptr<int>(), stream_of(cache));
 }
 
-// out[t, h, :] = w[h] x[t, h, :] (times sigmoid(gate[t, h])).  With turns, x and out are [T, H, K + rot] and [T, H, N + rot]:
+// out[t, h, :] = w[h] x[t, h, :] (times sigmoid(gate[t, h]), or sigmoid(gate[t, h, :])).  With turns, x and out are [T, H, K + rot] and [T, H, N + rot]:
 // the features behind K are turned and put behind N.  Returns non-zero (nothing launched) when the shape is not the kernel's.
-int64_t head_linear(const Tensor& x, const Tensor& w, Tensor& out, const c10::optional<Tensor>& gate, const c10::optional<Tensor>& turns) {
+int64_t head_linear(const Tensor& x, const Tensor& w, Tensor& out, const c10::optional<Tensor>& gate, const c10::optional<Tensor>& turns,
+                    bool halves) {
   check_float(x, "x");
   const int64_t rot = turns.has_value() ? 2 * turns->size(1) : 0;
   if (turns.has_value()) check_turns(*turns, x.size(0));
@@ -114,9 +127,10 @@ int64_t head_linear(const Tensor& x, const Tensor& w, Tensor& out, const c10::op
               "head_linear: x [T, H, K (+ rot)], w [H, N, K], out [T, H, N (+ rot)]");
   mb200::HeadLinearArgs a{};
   if (gate.has_value()) {
-    TORCH_CHECK(gate->is_cuda() && gate->dim() == 2 && gate->stride(1) == 1 && gate->size(0) == x.size(0) && gate->size(1) == x.size(1) &&
-                    gate->scalar_type() == x.scalar_type(),
-                "head_linear: gate [T, H]");
+    TORCH_CHECK(gate->is_cuda() && gate->dim() == 2 && gate->stride(1) == 1 && gate->size(0) == x.size(0) &&
+                    (gate->size(1) == x.size(1) || gate->size(1) == x.size(1) * w.size(1)) && gate->scalar_type() == x.scalar_type(),
+                "head_linear: gate [T, H] or [T, H * N]");
+    a.gate_feat = gate->size(1) != x.size(1) ? 1 : 0;
     a.gate = gate->data_ptr();
     a.gate_ld = gate->stride(0);
   }
@@ -135,13 +149,14 @@ int64_t head_linear(const Tensor& x, const Tensor& w, Tensor& out, const c10::op
   a.N = w.size(1);
   a.K = w.size(2);
   a.rot = rot;
+  a.halves = halves ? 1 : 0;
   a.dt = dtype_of(x);
   return mb200::launch_head_linear(a, device_state(x.get_device()).num_sms, stream_of(x));
 }
 
 // q [rows, H, K]; out [rows, H, R <= K]; cache [slots, K], values its first R features; row_req int32, row_pos int64 [rows]; max_seq_len sizes the split of the context
 void latent_attention(const Tensor& q, const Tensor& cache, const Tensor& req_to_token, const Tensor& row_req, const Tensor& row_pos,
-                      double scale, const c10::optional<Tensor>& sink, Tensor& out, int64_t max_seq_len) {
+                      double scale, const c10::optional<Tensor>& sink, Tensor& out, int64_t max_seq_len, int64_t window) {
   check_float(q, "q");
   TORCH_CHECK(q.dim() == 3 && q.is_contiguous() && out.is_contiguous() && out.dim() == 3 && out.size(0) == q.size(0) &&
                   out.size(1) == q.size(1) && out.size(2) <= q.size(2) && out.scalar_type() == q.scalar_type() && cache.dim() == 2 &&
@@ -166,8 +181,11 @@ void latent_attention(const Tensor& q, const Tensor& cache, const Tensor& req_to
     check_f32_vec(*sink, a.heads, "sink");
     a.sink = sink->data_ptr<float>();
   }
+  a.window = static_cast<int>(window);
+  int64_t longest = max_seq_len > 0 ? max_seq_len : req_to_token.size(1);
+  if (window > 0) longest = std::min(longest, window + 32);      // keys read, up to the tiles' alignment
   a.splits = mb200::latent_mma_covers(a.key, a.rank, a.cache_ld, a.dt)
-                 ? mb200::latent_num_splits(a.rows, a.heads, max_seq_len > 0 ? max_seq_len : req_to_token.size(1), st.num_sms)
+                 ? mb200::latent_num_splits(a.rows, a.heads, longest, st.num_sms)
                  : 1;
   Tensor part_o, part_lse;
   if (a.splits > 1) {
@@ -194,12 +212,16 @@ void latent_attention(const Tensor& q, const Tensor& cache, const Tensor& req_to
 
 PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("latent_prologue", &latent_prologue, py::arg("y"), py::arg("q_w"), py::arg("kv_w"), py::arg("eps"), py::arg("cq"), py::arg("loc"),
-        py::arg("cache"), py::arg("positions") = py::none(), py::arg("inv_freq") = py::none(), py::arg("turns") = py::none());
-  m.def("turn_heads", &turn_heads);
+        py::arg("cache"), py::arg("positions") = py::none(), py::arg("inv_freq") = py::none(), py::arg("turns") = py::none(),
+        py::arg("halves") = false);
+  m.def("turn_heads", &turn_heads, py::arg("x"), py::arg("turns"), py::arg("out"), py::arg("halves") = false);
   m.def("gate_heads", &gate_heads);
-  m.def("latent_gather", &latent_gather);
-  m.def("head_linear", &head_linear, py::arg("x"), py::arg("w"), py::arg("out"), py::arg("gate") = py::none(), py::arg("turns") = py::none());
-  m.def("latent_attention", &latent_attention);
+  m.def("latent_gather", &latent_gather, py::arg("cache"), py::arg("req_to_token"), py::arg("req"), py::arg("lens"), py::arg("start"),
+        py::arg("max_len"), py::arg("out"), py::arg("first") = py::none());
+  m.def("head_linear", &head_linear, py::arg("x"), py::arg("w"), py::arg("out"), py::arg("gate") = py::none(), py::arg("turns") = py::none(),
+        py::arg("halves") = false);
+  m.def("latent_attention", &latent_attention, py::arg("q"), py::arg("cache"), py::arg("req_to_token"), py::arg("row_req"), py::arg("row_pos"),
+        py::arg("scale"), py::arg("sink"), py::arg("out"), py::arg("max_seq_len"), py::arg("window") = 0);
   m.def("read_status", &read_status);
   m.def("launch_count", &launch_count);
 }

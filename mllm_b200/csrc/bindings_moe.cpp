@@ -49,7 +49,8 @@ void moe_router_topk(const Tensor& logits, Tensor& w, Tensor& ids, bool renorm, 
 }
 
 void moe_align(const Tensor& topk_ids, int64_t expert_offset, int64_t experts, int64_t bn, Tensor& sorted_pos,
-               Tensor& src_token, Tensor& expert_offsets, Tensor& work, Tensor& n_work) {
+               Tensor& src_token, Tensor& expert_offsets, Tensor& work, Tensor& n_work, const c10::optional<Tensor>& topk_w,
+               const c10::optional<Tensor>& src_w) {
   check_cuda(topk_ids, "topk_ids");
   TORCH_CHECK(topk_ids.scalar_type() == at::kInt && topk_ids.is_contiguous() && topk_ids.dim() == 2, "moe_align: int32 [T,k] ids");
   TORCH_CHECK(experts >= 1 && experts <= 256, "moe_align: 1..256 local experts");
@@ -59,10 +60,17 @@ void moe_align(const Tensor& topk_ids, int64_t expert_offset, int64_t experts, i
   TORCH_CHECK(sorted_pos.numel() >= pairs && src_token.numel() >= pairs && expert_offsets.numel() >= experts + 1 &&
                   work.dim() == 2 && work.size(1) == 2 && n_work.numel() >= 1,
               "moe_align: output sizes");
+  TORCH_CHECK(topk_w.has_value() == src_w.has_value(), "moe_align: weights in and out");
+  if (topk_w.has_value()) {
+    check_f32_vec(*topk_w, pairs, "topk_w");
+    check_f32_vec(*src_w, pairs, "src_w");
+  }
   c10::cuda::CUDAGuard g(topk_ids.device());
   mb200::launch_moe_align(topk_ids.data_ptr<int>(), pairs, topk_ids.size(1), expert_offset, experts, bn,
                           sorted_pos.data_ptr<int>(), src_token.data_ptr<int>(), expert_offsets.data_ptr<int>(),
-                          work.data_ptr<int>(), n_work.data_ptr<int>(), work.size(0), stream_of(topk_ids));
+                          work.data_ptr<int>(), n_work.data_ptr<int>(), work.size(0),
+                          topk_w.has_value() ? topk_w->data_ptr<float>() : nullptr, src_w.has_value() ? src_w->data_ptr<float>() : nullptr,
+                          stream_of(topk_ids));
 }
 
 void moe_gather(const Tensor& x, const Tensor& src_token, const Tensor& expert_offsets, Tensor& xs) {
@@ -73,6 +81,17 @@ void moe_gather(const Tensor& x, const Tensor& src_token, const Tensor& expert_o
   c10::cuda::CUDAGuard g(x.device());
   mb200::launch_moe_gather(x.data_ptr(), x.stride(0), src_token.data_ptr<int>(), expert_offsets.data_ptr<int>(),
                            expert_offsets.numel() - 1, xs.data_ptr(), xs.size(0), x.size(1), x.element_size(), stream_of(x));
+}
+
+// xs[row] = x[src_token[row]] * src_w[row]
+void moe_gather_scaled(const Tensor& x, const Tensor& src_token, const Tensor& src_w, const Tensor& expert_offsets, Tensor& xs) {
+  check_float(x, "x");
+  check_f32_vec(src_w, xs.size(0), "src_w");
+  TORCH_CHECK(x.dim() == 2 && x.stride(1) == 1 && xs.is_contiguous() && xs.size(1) == x.size(1) && xs.scalar_type() == x.scalar_type(),
+              "moe_gather_scaled: rows of one type and width");
+  c10::cuda::CUDAGuard g(x.device());
+  mb200::launch_moe_gather_scaled(x.data_ptr(), x.stride(0), src_token.data_ptr<int>(), src_w.data_ptr<float>(), expert_offsets.data_ptr<int>(),
+                                  expert_offsets.numel() - 1, xs.data_ptr(), xs.size(0), x.size(1), dtype_of(x), stream_of(x));
 }
 
 void moe_combine(const Tensor& y, const Tensor& sorted_pos, const Tensor& topk_w, Tensor& out) {
@@ -86,10 +105,10 @@ void moe_combine(const Tensor& y, const Tensor& sorted_pos, const Tensor& topk_w
                             out.size(0), out.size(1), topk_w.size(1), dtype_of(y), stream_of(y));
 }
 
-// out[rows of e] = x[rows of e] @ w[e]^T (SwiGLU-fused when swiglu) over the expert-sorted rows; any: the kernel for fp32 and
+// out[rows of e] = x[rows of e] @ w[e]^T (SwiGLU-fused when swiglu) over the expert-sorted rows (gelu: the exact GELU of it); any: the kernel for fp32 and
 // sizes of any kind (work items of 16 rows, no SwiGLU)
 int64_t moe_grouped_gemm(const Tensor& x, const Tensor& w, Tensor& out, const Tensor& expert_offsets, const Tensor& work,
-                      const Tensor& n_work, int64_t bn, bool swiglu, bool any) {
+                      const Tensor& n_work, int64_t bn, bool swiglu, bool any, bool gelu) {
   check_cuda(x, "x");
   check_cuda(w, "w");
   TORCH_CHECK(x.dim() == 2 && w.dim() == 3 && out.dim() == 2 && x.stride(1) == 1 && w.is_contiguous() && out.stride(1) == 1 &&
@@ -117,6 +136,7 @@ int64_t moe_grouped_gemm(const Tensor& x, const Tensor& w, Tensor& out, const Te
   a.bn = bn;
   a.max_work = work.size(0);
   a.swiglu = swiglu ? 1 : 0;
+  a.gelu = gelu ? 1 : 0;
   a.num_sms = st.num_sms;
   a.dt = dtype_of(x);
   if (any) return mb200::launch_moe_grouped_gemm_any(a, stream_of(x));
@@ -131,11 +151,14 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("moe_router_topk", &moe_router_topk, py::arg("logits"), py::arg("w"), py::arg("ids"), py::arg("renorm"),
         py::arg("correction") = py::none(), py::arg("renorm_eps") = 0.0, py::arg("sigmoid") = false, py::arg("groups") = 1,
         py::arg("keep") = 1, py::arg("scale") = 1.0);
-  m.def("moe_align", &moe_align);
+  m.def("moe_align", &moe_align, py::arg("topk_ids"), py::arg("expert_offset"), py::arg("experts"), py::arg("bn"), py::arg("sorted_pos"),
+        py::arg("src_token"), py::arg("expert_offsets"), py::arg("work"), py::arg("n_work"), py::arg("topk_w") = py::none(),
+        py::arg("src_w") = py::none());
+  m.def("moe_gather_scaled", &moe_gather_scaled);
   m.def("moe_gather", &moe_gather);
   m.def("moe_combine", &moe_combine);
   m.def("moe_grouped_gemm", &moe_grouped_gemm, py::arg("x"), py::arg("w"), py::arg("out"), py::arg("expert_offsets"), py::arg("work"),
-        py::arg("n_work"), py::arg("bn"), py::arg("swiglu"), py::arg("any") = false);
+        py::arg("n_work"), py::arg("bn"), py::arg("swiglu"), py::arg("any") = false, py::arg("gelu") = false);
   m.def("read_status", &read_status);
   m.def("launch_count", &launch_count);
 }

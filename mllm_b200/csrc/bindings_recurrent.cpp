@@ -5,7 +5,7 @@ namespace {
 
 // ---- gated delta net ----
 // x, out [T, H * W] contiguous; gate [T, H * W] with any row stride; w [W]
-void rmsnorm_gated(const Tensor& x, const Tensor& gate, const Tensor& w, Tensor& out, double eps, bool round_norm) {
+void rmsnorm_gated(const Tensor& x, const Tensor& gate, const Tensor& w, Tensor& out, double eps, bool round_norm, bool sigmoid) {
   check_float(x, "x");
   const int64_t width = w.numel();
   TORCH_CHECK(x.dim() == 2 && x.is_contiguous() && gate.dim() == 2 && gate.sizes() == x.sizes() && gate.stride(1) == 1 &&
@@ -15,12 +15,13 @@ void rmsnorm_gated(const Tensor& x, const Tensor& gate, const Tensor& w, Tensor&
   c10::cuda::CUDAGuard g(x.device());
   const int64_t heads = x.size(1) / width;
   mb200::launch_rmsnorm_gated(x.data_ptr(), gate.data_ptr(), gate.stride(0), w.data_ptr(), out.data_ptr(), x.size(0) * heads, heads,
-                              width, static_cast<float>(eps), round_norm ? 1 : 0, dtype_of(x), stream_of(x));
+                              width, static_cast<float>(eps), round_norm ? 1 : 0, sigmoid ? 1 : 0, dtype_of(x), stream_of(x));
 }
 
 // x [T, C] with any row stride; max_len: longest run of new tokens of a request (0: unknown)
 void gdn_conv1d_silu(const Tensor& x, const Tensor& w, Tensor& conv_state, const Tensor& slots, const Tensor& lens,
-                     const Tensor& has, const Tensor& q_start, Tensor& out, int64_t max_len) {
+                     const Tensor& has, const Tensor& q_start, Tensor& out, int64_t max_len, const c10::optional<Tensor>& bias,
+                     bool add_input) {
   check_float(x, "x");
   check_ragged(slots, lens, has, q_start);
   TORCH_CHECK(x.dim() == 2 && x.stride(1) == 1 && out.is_contiguous() && out.sizes() == x.sizes() && w.dim() == 2 &&
@@ -28,11 +29,15 @@ void gdn_conv1d_silu(const Tensor& x, const Tensor& w, Tensor& conv_state, const
                   conv_state.size(1) == x.size(1) && conv_state.size(2) == w.size(1) - 1 && out.scalar_type() == x.scalar_type() &&
                   w.scalar_type() == x.scalar_type() && conv_state.scalar_type() == x.scalar_type(),
               "gdn_conv1d_silu: x [T, C], w [C, K], conv_state [slots, C, K-1]");
+  if (bias.has_value())
+    TORCH_CHECK(bias->is_cuda() && bias->is_contiguous() && bias->numel() == x.size(1) && bias->scalar_type() == x.scalar_type(),
+                "gdn_conv1d_silu: bias [C]");
   c10::cuda::CUDAGuard g(x.device());
   const int rc = mb200::launch_gdn_conv1d_silu(x.data_ptr(), x.stride(0), w.data_ptr(), conv_state.data_ptr(), slots.data_ptr<int>(),
                                                lens.data_ptr<int>(), has.data_ptr<int>(), q_start.data_ptr<int>(),
                                                out.data_ptr(), slots.numel(), max_len > 0 ? std::min<int64_t>(max_len, x.size(0)) : x.size(0),
-                                               x.size(1), w.size(1), dtype_of(x), stream_of(x));
+                                               x.size(1), w.size(1), bias.has_value() ? bias->data_ptr() : nullptr, add_input ? 1 : 0,
+                                               dtype_of(x), stream_of(x));
   TORCH_CHECK(rc == 0, "gdn_conv1d_silu: unsupported kernel width");
 }
 
@@ -122,6 +127,50 @@ void gdn_recurrent_raw(const Tensor& q, const Tensor& k, const Tensor& v, const 
   TORCH_CHECK(rc == 0, "gdn_recurrent_raw: unsupported head size (code ", rc, ")");
 }
 
+// decays per key channel: b [T, H] and a [T, H * Dk], rows of wider matrices, a_log [H], dt_bias [H * Dk]
+static void set_channel_gates(mb200::GdnRuleParams& p, const Tensor& b, const Tensor& a, const Tensor& a_log, const Tensor& dt_bias,
+                              const Tensor& q) {
+  TORCH_CHECK(b.is_cuda() && b.dim() == 2 && b.size(0) == q.size(0) && b.size(1) == p.heads && b.stride(1) == 1 && a.is_cuda() && a.dim() == 2 &&
+                  a.size(0) == q.size(0) && a.size(1) == static_cast<int64_t>(p.heads) * p.dk && a.stride(1) == 1 && a.stride(0) > 0 &&
+                  b.scalar_type() == q.scalar_type() && a.scalar_type() == q.scalar_type(),
+              "gated delta rule: b [T, H], a [T, H * Dk] of q's type");
+  check_f32_vec(a_log, p.heads, "a_log");
+  check_f32_vec(dt_bias, static_cast<int64_t>(p.heads) * p.dk, "dt_bias");
+  p.b_raw = b.data_ptr();
+  p.a_raw = a.data_ptr();
+  p.gate_ld = b.stride(0);
+  p.a_ld = a.stride(0);
+  p.a_log = a_log.data_ptr<float>();
+  p.dt_bias = dt_bias.data_ptr<float>();
+}
+
+void gdn_channel_recurrent(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& b, const Tensor& a, const Tensor& a_log,
+                           const Tensor& dt_bias, Tensor& state, const Tensor& slots, const Tensor& lens, const Tensor& has,
+                           const Tensor& q_start, Tensor& out) {
+  mb200::GdnRuleParams p = rule_params(q, k, v, state, slots, lens, has, q_start, out);
+  set_channel_gates(p, b, a, a_log, dt_bias, q);
+  c10::cuda::CUDAGuard gd(q.device());
+  const int rc = mb200::launch_gdn_recurrent(p, stream_of(q));
+  TORCH_CHECK(rc == 0, "gdn_channel_recurrent: unsupported head size (code ", rc, ")");
+}
+
+// max_len: the longest run of new tokens (0: not known).  Returns 1 (nothing launched) when the sizes are not the chunk
+// kernel's.
+int64_t gdn_channel_chunk(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& b, const Tensor& a, const Tensor& a_log,
+                          const Tensor& dt_bias, Tensor& state, const Tensor& slots, const Tensor& lens, const Tensor& has,
+                          const Tensor& q_start, Tensor& out, int64_t max_len) {
+  mb200::GdnRuleParams p = rule_params(q, k, v, state, slots, lens, has, q_start, out);
+  set_channel_gates(p, b, a, a_log, dt_bias, q);
+  if (!mb200::gdn_channel_chunk_covers(p)) return 1;
+  c10::cuda::CUDAGuard gd(q.device());
+  const int longest = static_cast<int>(max_len > 0 ? std::min<int64_t>(max_len, q.size(0)) : q.size(0));
+  const mb200::GdnChannelPlan plan = mb200::gdn_channel_plan(p, longest);
+  Tensor ws = torch::empty({plan.ws_floats}, state.options());
+  const int rc = mb200::launch_gdn_channel_chunk(p, ws.data_ptr<float>(), plan.span, longest, device_state(q.get_device()).num_sms, stream_of(q));
+  TORCH_CHECK(rc == 0, "gdn_channel_chunk: launch failed (code ", rc, ")");
+  return 0;
+}
+
 // Returns 1 (nothing launched) when the shape is not the chunk kernel's.
 int64_t gdn_chunk(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& g, const Tensor& beta, Tensor& state,
                   const Tensor& slots, const Tensor& lens, const Tensor& has, const Tensor& q_start, Tensor& out, bool split_tf32) {
@@ -138,12 +187,16 @@ int64_t gdn_chunk(const Tensor& q, const Tensor& k, const Tensor& v, const Tenso
 }  // namespace
 
 PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
-  m.def("rmsnorm_gated", &rmsnorm_gated);
-  m.def("gdn_conv1d_silu", &gdn_conv1d_silu);
+  m.def("rmsnorm_gated", &rmsnorm_gated, py::arg("x"), py::arg("gate"), py::arg("w"), py::arg("out"), py::arg("eps"), py::arg("round_norm"),
+        py::arg("sigmoid") = false);
+  m.def("gdn_conv1d_silu", &gdn_conv1d_silu, py::arg("x"), py::arg("w"), py::arg("conv_state"), py::arg("slots"), py::arg("lens"),
+        py::arg("has"), py::arg("q_start"), py::arg("out"), py::arg("max_len"), py::arg("bias") = py::none(), py::arg("add_input") = false);
   m.def("gdn_gates", &gdn_gates);
   m.def("gdn_recurrent", &gdn_recurrent);
   m.def("gdn_recurrent_raw", &gdn_recurrent_raw);
   m.def("gdn_chunk", &gdn_chunk);
+  m.def("gdn_channel_recurrent", &gdn_channel_recurrent);
+  m.def("gdn_channel_chunk", &gdn_channel_chunk);
   m.def("read_status", &read_status);
   m.def("launch_count", &launch_count);
 }

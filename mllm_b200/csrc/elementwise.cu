@@ -194,7 +194,7 @@ __global__ void layernorm_kernel(const T* __restrict__ x, const T* __restrict__ 
 // ---------------------------------------------------------------------------
 __device__ __forceinline__ float silu_f(float v) { return v / (1.f + __expf(-v)); }
 template <typename T, int kAct>
-__global__ void act_and_mul_kernel(const T* __restrict__ x, T* __restrict__ out, int rows, int inter) {
+__global__ void act_and_mul_kernel(const T* __restrict__ x, T* __restrict__ out, int rows, int inter, float limit) {
   pdl_launch_dependents();
   pdl_wait();
   const int vec_per_row = inter >> 3;
@@ -208,14 +208,14 @@ __global__ void act_and_mul_kernel(const T* __restrict__ x, T* __restrict__ out,
     unpack8<T>(row[v], g);
     unpack8<T>(row[vec_per_row + v], u);
 #pragma unroll
-    for (int j = 0; j < 8; ++j) o[j] = (kAct == 0 ? silu_f(g[j]) : gelu_tanh_f(g[j])) * u[j];
+    for (int j = 0; j < 8; ++j) o[j] = kAct == 2 ? clamped_gate(g[j], u[j], limit) : (kAct == 0 ? silu_f(g[j]) : gelu_tanh_f(g[j])) * u[j];
     reinterpret_cast<uint4*>(out + r * inter)[v] = pack8<T>(o);
   }
 }
 
 // the same one element at a time: fp32 tensors and widths that are no multiple of 8
 template <typename T>
-__global__ void act_and_mul_any_kernel(const T* __restrict__ x, T* __restrict__ out, int64_t total, int inter, int act) {
+__global__ void act_and_mul_any_kernel(const T* __restrict__ x, T* __restrict__ out, int64_t total, int inter, int act, float limit) {
   pdl_launch_dependents();
   pdl_wait();
   for (int64_t i = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x; i < total;
@@ -223,7 +223,12 @@ __global__ void act_and_mul_any_kernel(const T* __restrict__ x, T* __restrict__ 
     const int64_t r = i / inter;
     const int64_t at = r * 2 * inter + (i - r * inter);
     const float g = to_f32(x[at]), u = to_f32(x[at + inter]);
-    out[i] = from_f32<T>((act == 0 ? g / (1.f + expf(-g)) : gelu_tanh_f(g)) * u);
+    if (act == 2) {
+      const float c = fminf(g, limit);
+      out[i] = from_f32<T>(c / (1.f + expf(-1.702f * c)) * (fminf(fmaxf(u, -limit), limit) + 1.f));
+    } else {
+      out[i] = from_f32<T>((act == 0 ? g / (1.f + expf(-g)) : gelu_tanh_f(g)) * u);
+    }
   }
 }
 
@@ -700,26 +705,27 @@ void launch_layernorm(const void* x, const void* w, const void* b, void* out, in
   note_launch();
 }
 
-void launch_act_and_mul(const void* x, void* out, int rows, int inter, int act, DType dt, cudaStream_t s) {
+void launch_act_and_mul(const void* x, void* out, int rows, int inter, int act, float limit, DType dt, cudaStream_t s) {
   if (rows == 0) return;
   const int threads = 256;
   if (dt == kF32 || inter % 8 != 0) {
     const int64_t n = static_cast<int64_t>(rows) * inter;
     const int grid = static_cast<int>(std::min<int64_t>((n + threads - 1) / threads, 148 * 16));
     MB200_DISPATCH_FLOAT(dt, (launch_pdl(act_and_mul_any_kernel<T>, dim3(grid), dim3(threads), 0, s, static_cast<const T*>(x),
-                                         static_cast<T*>(out), n, inter, act)));
+                                         static_cast<T*>(out), n, inter, act, limit)));
     note_launch();
     return;
   }
   const int64_t total = static_cast<int64_t>(rows) * (inter >> 3);
   const int blocks = static_cast<int>(std::min<int64_t>((total + threads - 1) / threads, 148 * 16));
-  if (act == 0) {
-    MB200_DISPATCH_HALF(dt, (launch_pdl(act_and_mul_kernel<T, 0>, dim3(blocks), dim3(threads), 0, s, static_cast<const T*>(x),
-                                                                                  static_cast<T*>(out), rows, inter)));
-  } else {
-    MB200_DISPATCH_HALF(dt, (launch_pdl(act_and_mul_kernel<T, 1>, dim3(blocks), dim3(threads), 0, s, static_cast<const T*>(x),
-                                                                                  static_cast<T*>(out), rows, inter)));
-  }
+  MB200_DISPATCH_HALF(dt, {
+    auto go = [&](auto kernel) {
+      launch_pdl(kernel, dim3(blocks), dim3(threads), 0, s, static_cast<const T*>(x), static_cast<T*>(out), rows, inter, limit);
+    };
+    if (act == 0) go(act_and_mul_kernel<T, 0>);
+    else if (act == 1) go(act_and_mul_kernel<T, 1>);
+    else go(act_and_mul_kernel<T, 2>);
+  });
   note_launch();
 }
 

@@ -1,13 +1,15 @@
-// Gated-delta-net kernels of the hybrid models (Qwen3.5, Pebulix): depth-wise causal convolution + SiLU over
+// Gated-delta-net kernels of the hybrid models (Qwen3.5, Pebulix, Nikedra): depth-wise causal convolution over
 // ragged sequences with per-request history, the gates, the recurrent gated delta rule with the state matrix held
 // in registers, and the gated RMSNorm that follows it.  Every kernel takes its per-request metadata
 // (state row, new-token count, "has history" flag, first token row) from device arrays, so a decode
 // step needs no host synchronisation and can be captured in a CUDA graph.
 //
 //   conv:  y[t, c] = silu(sum_j w[c, j] * in[t - (K-1) + j, c]),  inputs before the first new token come
-//          from conv_state[slot, c, :] (or are zero); afterwards conv_state keeps the last K-1 inputs.
+//          from conv_state[slot, c, :] (or are zero); afterwards conv_state keeps the last K-1 inputs.  Options: a bias per
+//          channel in front of the SiLU; the convolution added to its input instead of the SiLU.
 //   gates: beta = sigmoid(b), g = -exp(A_log) * softplus(a + dt_bias)
-//   rule:  S *= exp(g_t);  S += k_t (x) ((v_t - S^T k_t) * beta_t);  o_t = S^T q_t
+//          or, with a decay per key channel, g[d] = -exp(A_log) * softplus(a[d] + dt_bias[d])
+//   rule:  S *= exp(g_t) (row by row with a decay per channel);  S += k_t (x) ((v_t - S^T k_t) * beta_t);  o_t = S^T q_t
 //          with q, k l2-normalised and q scaled by Dk^-0.5; S is [Dk, Dv] fp32 per (request, head).
 //          Value head h uses query / key head h / (heads / key heads).
 #include "common.cuh"
@@ -49,7 +51,8 @@ template <typename T, int KT, int V>
 __global__ void gdn_conv1d_silu_kernel(const T* __restrict__ x, int64_t x_ld, const T* __restrict__ w, T* __restrict__ conv_state,
                                        const int* __restrict__ slots, const int* __restrict__ lens,
                                        const int* __restrict__ has_state, const int* __restrict__ q_start,
-                                       T* __restrict__ out, int channels, int taps, int chunk_tokens, int own_state) {
+                                       T* __restrict__ out, int channels, int taps, int chunk_tokens, int own_state,
+                                       const T* __restrict__ bias, int add_input) {
   pdl_wait();
   constexpr int kCap = KT > 0 ? KT : kMaxConvK;
   const int K = KT > 0 ? KT : taps;
@@ -62,7 +65,9 @@ __global__ void gdn_conv1d_silu_kernel(const T* __restrict__ x, int64_t x_ld, co
   const int64_t row0 = q_start[b];
   T* st = conv_state + (static_cast<int64_t>(slots[b]) * channels + c) * (K - 1);
   const bool hist = has_state[b] != 0;
-  float wv[kCap][V], win[kCap][V];
+  float wv[kCap][V], win[kCap][V], bv[V];
+#pragma unroll
+  for (int i = 0; i < V; ++i) bv[i] = bias != nullptr ? to_f32(bias[c + i]) : 0.f;
 #pragma unroll
   for (int j = 0; j < kCap; ++j)
 #pragma unroll
@@ -84,11 +89,11 @@ __global__ void gdn_conv1d_silu_kernel(const T* __restrict__ x, int64_t x_ld, co
     load_v<T, V>(x + (row0 + t) * x_ld + c, cur);
 #pragma unroll
     for (int i = 0; i < V; ++i) {
-      acc[i] = 0.f;
+      acc[i] = bv[i];
 #pragma unroll
       for (int j = 0; j < kCap; ++j)
         if (j < K) acc[i] = fmaf(wv[j][i], j == K - 1 ? cur[i] : win[j][i], acc[i]);
-      acc[i] = silu<T>(acc[i]);
+      acc[i] = add_input ? cur[i] + acc[i] : silu<T>(acc[i]);
 #pragma unroll
       for (int j = 0; j < kCap - 1; ++j)
         if (j < K - 1) win[j][i] = j == K - 2 ? cur[i] : win[j + 1][i];
@@ -148,7 +153,8 @@ __global__ void gdn_gates_kernel(const T* __restrict__ b, const T* __restrict__ 
 // columns of the state.  With the decayed state S', S'^T k and S'^T q are summed over the rows together, since
 // o = (S' + k u^T)^T q = S'^T q + u (k . q): one exchange between the warps per token.  The norms of q and k and their
 // product ride along in the same exchange.
-template <typename T, int RPT>
+// CHANNEL: a decay per key channel, formed here from a_raw.
+template <typename T, int RPT, bool CHANNEL>
 __global__ void __launch_bounds__(256) gdn_recurrent_kernel(const GdnRuleParams p) {
   pdl_wait();
   __shared__ float4 red[2][8][16];    // [parity][warp][S'^T k of 8 column groups | S'^T q]
@@ -183,7 +189,13 @@ __global__ void __launch_bounds__(256) gdn_recurrent_kernel(const GdnRuleParams 
     }
   }
   const float qscale = 1.f / sqrtf(static_cast<float>(p.dk));
-  float kn[RPT], qn[RPT], vn[4], gn, bn;
+  float kn[RPT], qn[RPT], vn[4], gn = 0.f, bn;
+  float an[CHANNEL ? RPT : 1], bias[CHANNEL ? RPT : 1], rate = 0.f;
+  if constexpr (CHANNEL) {
+    rate = -expf(p.a_log[h]);
+#pragma unroll
+    for (int r = 0; r < RPT; ++r) bias[r] = rg + 32 * r < p.dk ? p.dt_bias[static_cast<int64_t>(h) * p.dk + rg + 32 * r] : 0.f;
+  }
   auto load = [&](int t) {
 #pragma unroll
     for (int r = 0; r < RPT; ++r) {
@@ -193,7 +205,15 @@ __global__ void __launch_bounds__(256) gdn_recurrent_kernel(const GdnRuleParams 
     }
 #pragma unroll
     for (int j = 0; j < 4; ++j) vn[j] = c + j < p.dv ? to_f32(v[t * p.v_ld + c + j]) : 0.f;
-    if (p.g != nullptr) {
+    if constexpr (CHANNEL) {
+      const T* a = static_cast<const T*>(p.a_raw) + (row0 + t) * p.a_ld + static_cast<int64_t>(h) * p.dk;
+#pragma unroll
+      for (int r = 0; r < RPT; ++r) {
+        const float z = rg + 32 * r < p.dk ? to_f32(a[rg + 32 * r]) + bias[r] : 0.f;
+        an[r] = expf(rate * (fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)))));
+      }
+      bn = 1.f / (1.f + expf(-to_f32(static_cast<const T*>(p.b_raw)[(row0 + t) * p.gate_ld + h])));
+    } else if (p.g != nullptr) {
       gn = p.g[(row0 + t) * p.heads + h];
       bn = p.beta[(row0 + t) * p.heads + h];
     } else {
@@ -204,7 +224,7 @@ __global__ void __launch_bounds__(256) gdn_recurrent_kernel(const GdnRuleParams 
   load(0);
   for (int t = 0; t < n; ++t) {
     float kv[RPT], qv[RPT];
-    const float decay = expf(gn), beta = bn;
+    const float decay = CHANNEL ? 1.f : expf(gn), beta = bn;
     const float v4[4] = {vn[0], vn[1], vn[2], vn[3]};
     float sk[4] = {0.f, 0.f, 0.f, 0.f}, sq[4] = {0.f, 0.f, 0.f, 0.f}, kk = 0.f, qq = 0.f, kq = 0.f;
 #pragma unroll
@@ -216,7 +236,7 @@ __global__ void __launch_bounds__(256) gdn_recurrent_kernel(const GdnRuleParams 
       kq = fmaf(kv[r], qv[r], kq);
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-        s[r][j] *= decay;
+        s[r][j] *= CHANNEL ? an[r] : decay;
         sk[j] = fmaf(s[r][j], kv[r], sk[j]);
         sq[j] = fmaf(s[r][j], qv[r], sq[j]);
       }
@@ -293,9 +313,9 @@ __global__ void __launch_bounds__(256) gdn_recurrent_kernel(const GdnRuleParams 
   }
 }
 
-// out = weight * rmsnorm(x) * silu(gate); one warp per row.  Row r = (token r / heads, head r % heads) of x and out
+// out = weight * rmsnorm(x) * silu(gate), or sigmoid(gate) (SIG); one warp per row.  Row r = (token r / heads, head r % heads) of x and out
 // (contiguous); gate rows of a token start gate_ld apart.  round_norm: the normed value is rounded to T before the weight.
-template <typename T, int V>
+template <typename T, int V, bool SIG>
 __global__ void rmsnorm_gated_kernel(const T* __restrict__ x, const T* __restrict__ gate, int64_t gate_ld, const T* __restrict__ w,
                                      T* __restrict__ out, int64_t rows, int heads, int width, float eps, int round_norm) {
   pdl_wait();
@@ -320,21 +340,22 @@ __global__ void rmsnorm_gated_kernel(const T* __restrict__ x, const T* __restric
     for (int i = 0; i < V; ++i) {
       float nrm = f[i] * rstd;
       if (round_norm) nrm = to_f32(from_f32<T>(nrm));
-      f[i] = wv[i] * nrm * silu<T>(g[i]);
+      if constexpr (SIG) f[i] = wv[i] * nrm * (sizeof(T) == 2 ? __fdividef(1.f, 1.f + __expf(-g[i])) : 1.f / (1.f + expf(-g[i])));
+      else f[i] = wv[i] * nrm * silu<T>(g[i]);
     }
     store_v<T, V>(out + r * width + c, f);
   }
 }
 
 // rows per thread of the recurrent kernel: 32 row groups cover Dk
-template <typename T>
+template <typename T, bool CHANNEL>
 int launch_recurrent_t(const GdnRuleParams& p, cudaStream_t s) {
   const dim3 grid((p.dv + 31) / 32, p.heads, p.batch), block(256);
-  if (p.dk <= 32) launch_pdl(gdn_recurrent_kernel<T, 1>, grid, block, 0, s, p);
-  else if (p.dk <= 64) launch_pdl(gdn_recurrent_kernel<T, 2>, grid, block, 0, s, p);
-  else if (p.dk <= 128) launch_pdl(gdn_recurrent_kernel<T, 4>, grid, block, 0, s, p);
-  else if (p.dk <= 256) launch_pdl(gdn_recurrent_kernel<T, 8>, grid, block, 0, s, p);
-  else if (p.dk <= 512) launch_pdl(gdn_recurrent_kernel<T, 16>, grid, block, 0, s, p);
+  if (p.dk <= 32) launch_pdl(gdn_recurrent_kernel<T, 1, CHANNEL>, grid, block, 0, s, p);
+  else if (p.dk <= 64) launch_pdl(gdn_recurrent_kernel<T, 2, CHANNEL>, grid, block, 0, s, p);
+  else if (p.dk <= 128) launch_pdl(gdn_recurrent_kernel<T, 4, CHANNEL>, grid, block, 0, s, p);
+  else if (p.dk <= 256) launch_pdl(gdn_recurrent_kernel<T, 8, CHANNEL>, grid, block, 0, s, p);
+  else if (p.dk <= 512) launch_pdl(gdn_recurrent_kernel<T, 16, CHANNEL>, grid, block, 0, s, p);
   else return -1;
   note_launch();
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
@@ -342,11 +363,12 @@ int launch_recurrent_t(const GdnRuleParams& p, cudaStream_t s) {
 
 template <typename T, int V>
 void launch_conv_t(int chunks, int batch, cudaStream_t s, const void* x, int64_t x_ld, const void* w, void* st, const int* slots,
-                   const int* lens, const int* has, const int* q_start, void* out, int channels, int K, int chunk, int own) {
+                   const int* lens, const int* has, const int* q_start, void* out, int channels, int K, int chunk, int own, const void* bias,
+                   int add_input) {
   const dim3 grid((channels + 256 * V - 1) / (256 * V), chunks, batch);
   auto go = [&](auto kernel) {
     launch_pdl(kernel, grid, dim3(256), 0, s, static_cast<const T*>(x), x_ld, static_cast<const T*>(w), static_cast<T*>(st), slots,
-               lens, has, q_start, static_cast<T*>(out), channels, K, chunk, own);
+               lens, has, q_start, static_cast<T*>(out), channels, K, chunk, own, static_cast<const T*>(bias), add_input);
   };
   switch (K) {
     case 2: go(gdn_conv1d_silu_kernel<T, 2, V>); break;
@@ -360,7 +382,7 @@ void launch_conv_t(int chunks, int batch, cudaStream_t s, const void* x, int64_t
 
 int launch_gdn_conv1d_silu(const void* x, int64_t x_ld, const void* w, void* conv_state, const int* slots, const int* lens,
                            const int* has_state, const int* q_start, void* out, int batch, int max_tokens, int channels, int K,
-                           DType dt, cudaStream_t s) {
+                           const void* bias, int add_input, DType dt, cudaStream_t s) {
   if (batch <= 0 || max_tokens <= 0) return 0;
   if (K < 1 || K > kMaxConvK) return -1;
   const int chunk = 64;
@@ -371,10 +393,10 @@ int launch_gdn_conv1d_silu(const void* x, int64_t x_ld, const void* w, void* con
   const bool pair = channels % 2 == 0 && x_ld % 2 == 0 && align % (dt == kF32 ? 8 : 4) == 0 && max_tokens > 1;
   if (pair) {
     MB200_DISPATCH_FLOAT(dt, (launch_conv_t<T, 2>(chunks, batch, s, x, x_ld, w, conv_state, slots, lens, has_state, q_start, out,
-                                                  channels, K, chunk, own)));
+                                                  channels, K, chunk, own, bias, add_input)));
   } else {
     MB200_DISPATCH_FLOAT(dt, (launch_conv_t<T, 1>(chunks, batch, s, x, x_ld, w, conv_state, slots, lens, has_state, q_start, out,
-                                                  channels, K, chunk, own)));
+                                                  channels, K, chunk, own, bias, add_input)));
   }
   note_launch();
   if (!own && K > 1) {
@@ -399,26 +421,32 @@ int launch_gdn_recurrent(const GdnRuleParams& p, cudaStream_t s) {
   if (p.batch <= 0) return 0;
   if (p.heads % p.k_heads != 0) return -1;
   int rc = 0;
-  MB200_DISPATCH_FLOAT(p.dt, rc = launch_recurrent_t<T>(p, s));
+  MB200_DISPATCH_FLOAT(p.dt, rc = p.a_ld > 0 ? (launch_recurrent_t<T, true>(p, s)) : (launch_recurrent_t<T, false>(p, s)));
   return rc;
 }
 
 void launch_rmsnorm_gated(const void* x, const void* gate, int64_t gate_ld, const void* w, void* out, int64_t rows, int heads,
-                          int width, float eps, int round_norm, DType dt, cudaStream_t s) {
+                          int width, float eps, int round_norm, int sigmoid, DType dt, cudaStream_t s) {
   if (rows <= 0) return;
   const int warps = 8;
   const dim3 grid(static_cast<unsigned>((rows + warps - 1) / warps)), block(warps * 32);
   const uintptr_t align = reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(w) |
                           reinterpret_cast<uintptr_t>(out);
-  if (width % 4 == 0 && gate_ld % 4 == 0 && align % (dt == kF32 ? 16 : 8) == 0) {
-    MB200_DISPATCH_FLOAT(dt, (launch_pdl(rmsnorm_gated_kernel<T, 4>, grid, block, 0, s, static_cast<const T*>(x),
-                                         static_cast<const T*>(gate), gate_ld, static_cast<const T*>(w), static_cast<T*>(out), rows,
-                                         heads, width, eps, round_norm)));
-  } else {
-    MB200_DISPATCH_FLOAT(dt, (launch_pdl(rmsnorm_gated_kernel<T, 1>, grid, block, 0, s, static_cast<const T*>(x),
-                                         static_cast<const T*>(gate), gate_ld, static_cast<const T*>(w), static_cast<T*>(out), rows,
-                                         heads, width, eps, round_norm)));
-  }
+  auto go = [&](auto typed, auto kernel) {
+    using T = decltype(typed);
+    launch_pdl(kernel, grid, block, 0, s, static_cast<const T*>(x), static_cast<const T*>(gate), gate_ld, static_cast<const T*>(w),
+               static_cast<T*>(out), rows, heads, width, eps, round_norm);
+  };
+  const bool vec = width % 4 == 0 && gate_ld % 4 == 0 && align % (dt == kF32 ? 16 : 8) == 0;
+  MB200_DISPATCH_FLOAT(dt, {
+    if (sigmoid) {
+      if (vec) go(T{}, rmsnorm_gated_kernel<T, 4, true>);
+      else go(T{}, rmsnorm_gated_kernel<T, 1, true>);
+    } else {
+      if (vec) go(T{}, rmsnorm_gated_kernel<T, 4, false>);
+      else go(T{}, rmsnorm_gated_kernel<T, 1, false>);
+    }
+  });
   note_launch();
 }
 

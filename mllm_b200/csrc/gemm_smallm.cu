@@ -29,6 +29,8 @@
 #include <algorithm>
 #include <cstdint>
 
+#include <type_traits>
+
 #include "common.cuh"
 #include "kernels.h"
 
@@ -54,6 +56,7 @@ struct SmallMParams {
   int units_per_cta;
   int steps_per_warp;    // k / 32 / kSmWarps
   int swiglu;
+  float act_limit;
   int b_static;
   int early_trigger;     // let the kernels behind this one start their set-up as soon as this one runs
   // fused prologue (norm_w != null): the rows fed to the product are rmsnorm(a + norm_res) * norm_w, with the sum
@@ -98,7 +101,7 @@ __device__ __forceinline__ uint16_t f_to_half(float v) {
   return *reinterpret_cast<const uint16_t*>(&h);
 }
 
-template <bool F16, int ACT>   // ACT: activation of the gate (0 SiLU, 1 GELU) or, 2, square of relu without a gate
+template <bool F16, int ACT>   // ACT: activation of the gate (0 SiLU, 1 GELU), 2 square of relu without a gate, 3 bounded gated unit with biases
 __global__ void __launch_bounds__(kSmThreads, 1) gemm_smallm_kernel(const SmallMParams p) {
   __shared__ float partial[2][kSmWarps][64];
   extern __shared__ __align__(16) uint8_t smem_dyn[];
@@ -284,7 +287,17 @@ __global__ void __launch_bounds__(kSmThreads, 1) gemm_smallm_kernel(const SmallM
                   for (int w8 = 0; w8 < kSmWarps; ++w8) up += partial[buf][w8][t + 4];
                   const int blk = cu >> 5, q = cu & 31;
                   const int64_t col = static_cast<int64_t>(blk) * 128 + q * 4 + slot;
-                  const float y = gate_act<ACT == 1>(v) * up;
+                  float y;
+                  if constexpr (ACT == 3) {
+                    const int64_t row = static_cast<int64_t>(blk) * 256 + q * 4 + slot;
+                    if (p.bias != nullptr) {
+                      v += half_to_f<F16>(static_cast<const uint16_t*>(p.bias)[row]);
+                      up += half_to_f<F16>(static_cast<const uint16_t*>(p.bias)[row + 128]);
+                    }
+                    y = clamped_gate(v, up, p.act_limit);
+                  } else {
+                    y = gate_act<ACT == 1>(v) * up;
+                  }
                   static_cast<uint16_t*>(p.out)[mrow * p.ldc + col] = f_to_half<F16>(y);
                 }
               } else {
@@ -321,8 +334,8 @@ int launch_gemm_smallm(const GemmArgs& a, cudaStream_t s) {
   // matrices of hundreds of MB (the vocabulary head) stream at the full copy rate through the TMA ring of the
   // tcgen05 path, whose set-up cost no longer shows; this kernel is for the projections of a layer
   if (static_cast<int64_t>(a.n) * a.k * 2 > (int64_t(384) << 20)) return 1;
-  const bool relu2 = a.swiglu == 3;
-  if (a.swiglu && !relu2 && (a.n % 256 != 0 || a.bias != nullptr || a.residual != nullptr)) return 1;
+  const bool relu2 = a.swiglu == 3, clamped = a.swiglu == 4;
+  if (a.swiglu && !relu2 && (a.n % 256 != 0 || (a.bias != nullptr && !clamped) || a.residual != nullptr)) return 1;
   if ((a.lda * 2) % 16 != 0 || (a.ldb * 2) % 16 != 0) return 1;
   if (a.norm_weight != nullptr &&
       ((a.norm_residual_ld * 2) % 16 != 0 || (a.norm_residual_out_ld * 2) % 16 != 0 ||
@@ -346,6 +359,7 @@ int launch_gemm_smallm(const GemmArgs& a, cudaStream_t s) {
   p.units = a.n / 8;
   p.steps_per_warp = a.k / (32 * kSmWarps);
   p.swiglu = relu2 ? 0 : a.swiglu;
+  p.act_limit = a.act_limit;
   p.b_static = a.b_static;
   p.norm_w = a.norm_weight;
   p.norm_res = static_cast<const uint8_t*>(a.norm_residual);
@@ -370,9 +384,13 @@ int launch_gemm_smallm(const GemmArgs& a, cudaStream_t s) {
     const cudaError_t set = ensure_dynamic_smem(reinterpret_cast<const void*>(kernel), kSmRingBytes + 8 * (2 * kSmMaxK + kSmRowPad));
     return set != cudaSuccess ? set : launch_pdl(kernel, dim3(grid), dim3(kSmThreads), smem, s, p);
   };
-  const cudaError_t err =
-      a.dt == kF16 ? (relu2 ? go(gemm_smallm_kernel<true, 2>) : gelu ? go(gemm_smallm_kernel<true, 1>) : go(gemm_smallm_kernel<true, 0>))
-                   : (relu2 ? go(gemm_smallm_kernel<false, 2>) : gelu ? go(gemm_smallm_kernel<false, 1>) : go(gemm_smallm_kernel<false, 0>));
+  auto pick = [&](auto f16) -> cudaError_t {
+    constexpr bool kF = decltype(f16)::value;
+    if (relu2) return go(gemm_smallm_kernel<kF, 2>);
+    if (clamped) return go(gemm_smallm_kernel<kF, 3>);
+    return gelu ? go(gemm_smallm_kernel<kF, 1>) : go(gemm_smallm_kernel<kF, 0>);
+  };
+  const cudaError_t err = a.dt == kF16 ? pick(std::true_type{}) : pick(std::false_type{});
   note_launch();
   return err == cudaSuccess ? 0 : -4;
 }

@@ -47,6 +47,7 @@ struct KParams {
   float* workspace;
   int* counters;
   int* status;
+  float act_limit;       // SWIGLU 4
   int m, n, k_blocks;
   int64_t ldc, ld_res;
   int tiles_r, tiles_c;  // tiles over the row-operand rows / column-operand rows
@@ -83,7 +84,7 @@ constexpr int kStageRowBytes = 144;                      // 128 bytes of output 
 constexpr int kEpiStagingBytes = 4 * 32 * kStageRowBytes;  // four epilogue warps x 32 rows
 
 template <int SWIGLU>
-constexpr bool kGated = SWIGLU == 1 || SWIGLU == 2;
+constexpr bool kGated = SWIGLU == 1 || SWIGLU == 2 || SWIGLU == 4;
 template <int SWIGLU>
 __device__ __forceinline__ float plain_act(float x) {
   if constexpr (SWIGLU == 3) {
@@ -93,7 +94,8 @@ __device__ __forceinline__ float plain_act(float x) {
   return x;
 }
 
-// SWIGLU: 0 plain product, 1 silu(gate) * up, 2 gelu_tanh(gate) * up, 3 square of relu (no gate: as the plain product).
+// SWIGLU: 0 plain product, 1 silu(gate) * up, 2 gelu_tanh(gate) * up, 3 square of relu (no gate: as the plain product),
+// 4 bounded gated unit of both halves with their biases.
 // RT = 128-row MMA tiles of the row operand per stage (small-batch tiling only; SwiGLU needs 2: a
 // gate block and its up block), KD = 128-byte K atoms per stage.  Larger stages mean fewer TMA boxes
 // and barrier round trips per byte streamed.
@@ -167,6 +169,19 @@ __device__ __forceinline__ void store_out1(void* base, int64_t idx, float v, int
 }
 __device__ __forceinline__ float acc_to_float(uint32_t raw, int is_int8) {
   return is_int8 ? static_cast<float>(static_cast<int32_t>(raw)) : __uint_as_float(raw);
+}
+
+// the gated unit of a gate product and its up product; `row`: weight row of the gate (the up row is kBM behind it)
+template <int SWIGLU>
+__device__ __forceinline__ float gated_unit(const KParams& p, float x, float u, int64_t row) {
+  if constexpr (SWIGLU == 4) {
+    if (p.bias != nullptr) {
+      x += load_out1(p.bias, row, p.out_f16);
+      u += load_out1(p.bias, row + kBM, p.out_f16);
+    }
+    return clamped_gate(x, u, p.act_limit);
+  }
+  return gate_act<SWIGLU == 2>(x) * u;
 }
 
 template <int BN, bool SWAP, int SWIGLU, int RT, int KD>
@@ -519,7 +534,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
                       x *= sa * p.b_scale[tc * BN + cc];
                       u *= sa * p.b_scale[tc * BN + BN / 2 + cc];
                     }
-                    x = gate_act<SWIGLU == 2>(x) * u;
+                    x = gated_unit<SWIGLU>(p, x, u, static_cast<int64_t>(tc) * BN + cc);
                   } else {
                     const int64_t col = col0 + cc;
                     if (p.is_int8 && col < n_out) x *= sa * p.b_scale[col];
@@ -576,7 +591,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
                   x *= sa * p.b_scale[tc * BN + c + v8 * 8 + j];
                   u *= sa * p.b_scale[tc * BN + BN / 2 + c + v8 * 8 + j];
                 }
-                x = gate_act<SWIGLU == 2>(x) * u;
+                x = gated_unit<SWIGLU>(p, x, u, static_cast<int64_t>(tc) * BN + c + v8 * 8 + j);
               } else {
                 if (p.is_int8) x *= sa * p.b_scale[col + j];
                 if (p.bias != nullptr) x += load_out1(p.bias, col + j, p.out_f16);
@@ -720,7 +735,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
                       xv *= p.a_scale[j] * p.b_scale[wrow];
                       uv *= p.a_scale[j] * p.b_scale[wrow + kBM];
                     }
-                    xv = gate_act<SWIGLU == 2>(xv) * uv;
+                    xv = gated_unit<SWIGLU>(p, xv, uv, wrow);
                     ocol = static_cast<int64_t>(tr) * kBM + row_in_tile;
                   } else {
                     if (p.is_int8) xv *= p.a_scale[j] * p.b_scale[wrow];
@@ -771,7 +786,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
                   x *= p.a_scale[mi] * p.b_scale[wrow];
                   u *= p.a_scale[mi] * p.b_scale[wrow + kBM];
                 }
-                x = gate_act<SWIGLU == 2>(x) * u;
+                x = gated_unit<SWIGLU>(p, x, u, wrow);
                 ocol = static_cast<int64_t>(tr) * kBM + row_in_tile;
               } else {
                 if (p.is_int8) x *= p.a_scale[mi] * p.b_scale[wrow];
@@ -1169,7 +1184,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_consta
                 x *= sa * p.b_scale[tc * kPairBN + c + v8 * 8 + j];
                 u *= sa * p.b_scale[tc * kPairBN + kPairBN / 2 + c + v8 * 8 + j];
               }
-              x = gate_act<SWIGLU == 2>(x) * u;
+              x = gated_unit<SWIGLU>(p, x, u, static_cast<int64_t>(tc) * kPairBN + c + v8 * 8 + j);
             } else {
               if (p.is_int8) x *= sa * p.b_scale[col + j];
               if (p.bias != nullptr) x += load_out1(p.bias, col + j, p.out_f16);
@@ -1311,8 +1326,9 @@ int launch_gemm(const GemmArgs& a, cudaStream_t s) {
   const int k_per_block = kRowBytes / eb;
   if (a.k % (16 / eb) != 0 || a.lda % (16 / eb) != 0 || a.ldb % (16 / eb) != 0) return -1;
   if (a.n % 8 != 0 || a.ldc % 8 != 0) return -1;
-  const bool gated = a.swiglu == 1 || a.swiglu == 2, relu2 = a.swiglu == 3;
-  if (gated && (a.n % 256 != 0 || a.bias != nullptr || a.residual != nullptr)) return -1;
+  const bool clamped = a.swiglu == 4, gated = a.swiglu == 1 || a.swiglu == 2 || clamped, relu2 = a.swiglu == 3;
+  if (gated && (a.n % 256 != 0 || (a.bias != nullptr && !clamped) || a.residual != nullptr)) return -1;
+  if (clamped && (a.is_int8 || a.gate_flags != nullptr || a.rs_tp > 0)) return -1;
   if (relu2 && (a.bias != nullptr || a.residual != nullptr || a.rs_tp > 0)) return -1;
   if ((reinterpret_cast<uintptr_t>(a.a) | reinterpret_cast<uintptr_t>(a.b) | reinterpret_cast<uintptr_t>(a.out)) & 15)
     return -1;
@@ -1327,6 +1343,7 @@ int launch_gemm(const GemmArgs& a, cudaStream_t s) {
   p.workspace = a.workspace;
   p.counters = a.counters;
   p.status = a.status;
+  p.act_limit = a.act_limit;
   p.m = a.m;
   p.n = a.n;
   p.k_blocks = (a.k + k_per_block - 1) / k_per_block;
@@ -1386,6 +1403,7 @@ int launch_gemm(const GemmArgs& a, cudaStream_t s) {
       const int pairs = static_cast<int>(std::min<int64_t>(tiles_pair, num_sms / 2));
       if (relu2) return launch_pair_cfg<3>(tm_row, tm_col, p, pairs, s);
       if (a.swiglu == 2) return launch_pair_cfg<2>(tm_row, tm_col, p, pairs, s);
+      if (clamped) return launch_pair_cfg<4>(tm_row, tm_col, p, pairs, s);
       return gated ? launch_pair_cfg<1>(tm_row, tm_col, p, pairs, s)
                       : launch_pair_cfg<0>(tm_row, tm_col, p, pairs, s);
     }
@@ -1405,6 +1423,7 @@ int launch_gemm(const GemmArgs& a, cudaStream_t s) {
     if (relu2)
       return bn == 256 ? launch_cfg<256, false, 3>(tm_row, tm_col, p, grid, s) : launch_cfg<128, false, 3>(tm_row, tm_col, p, grid, s);
     if (a.swiglu == 2) return launch_cfg<256, false, 2>(tm_row, tm_col, p, grid, s);
+    if (clamped) return launch_cfg<256, false, 4>(tm_row, tm_col, p, grid, s);
     if (gated) return launch_cfg<256, false, 1>(tm_row, tm_col, p, grid, s);
     if (bn == 256) return launch_cfg<256, false, 0>(tm_row, tm_col, p, grid, s);
     return launch_cfg<128, false, 0>(tm_row, tm_col, p, grid, s);
@@ -1485,6 +1504,9 @@ int launch_gemm(const GemmArgs& a, cudaStream_t s) {
     if (a.swiglu == 2)                                                                              \
       return kd == 2 ? launch_cfg<BNV, true, 2, 2, 2>(tm_row, tm_col, p, grid, s)                   \
                      : launch_cfg<BNV, true, 2, 2, 1>(tm_row, tm_col, p, grid, s);                  \
+    if (clamped)                                                                                    \
+      return kd == 2 ? launch_cfg<BNV, true, 4, 2, 2>(tm_row, tm_col, p, grid, s)                   \
+                     : launch_cfg<BNV, true, 4, 2, 1>(tm_row, tm_col, p, grid, s);                  \
     if (a.swiglu)                                                                                   \
       return kd == 2 ? launch_cfg<BNV, true, 1, 2, 2>(tm_row, tm_col, p, grid, s)                   \
                      : launch_cfg<BNV, true, 1, 2, 1>(tm_row, tm_col, p, grid, s);                  \
@@ -1496,6 +1518,7 @@ int launch_gemm(const GemmArgs& a, cudaStream_t s) {
 #define MB200_SWAP_LARGE(BNV)                                                                       \
   case BNV:                                                                                         \
     if (a.swiglu == 2) return launch_cfg<BNV, true, 2, 2, 1>(tm_row, tm_col, p, grid, s);           \
+    if (clamped) return launch_cfg<BNV, true, 4, 2, 1>(tm_row, tm_col, p, grid, s);                 \
     return a.swiglu ? launch_cfg<BNV, true, 1, 2, 1>(tm_row, tm_col, p, grid, s)                    \
                     : launch_cfg<BNV, true, 0, 1, 1>(tm_row, tm_col, p, grid, s);
   switch (bn) {

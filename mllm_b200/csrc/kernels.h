@@ -22,8 +22,8 @@ void launch_fused_add_rmsnorm(void* x, void* residual, const void* w, int rows, 
                               cudaStream_t s);
 void launch_layernorm(const void* x, const void* w, const void* b, void* out, int rows, int hidden, float eps,
                       DType dt, cudaStream_t s);
-// act: 0 = silu(gate)*up, 1 = gelu_tanh(gate)*up ; x is [rows, 2*inter] = [gate | up]
-void launch_act_and_mul(const void* x, void* out, int rows, int inter, int act, DType dt, cudaStream_t s);
+// act: 0 = silu(gate)*up, 1 = gelu_tanh(gate)*up, 2 = clamped gate (see clamped_gate in common.cuh); x is [rows, 2*inter] = [gate | up]
+void launch_act_and_mul(const void* x, void* out, int rows, int inter, int act, float limit, DType dt, cudaStream_t s);
 // fp32 residual stream with a Dynamic Tanh norm: x += mult * y (y may be null), h = tanh(alpha x) * w + b
 void launch_residual_dyt(float* x, const void* y, float mult, const float* alpha, const float* w, const float* b, void* h,
                          int rows, int width, DType dt, cudaStream_t s);
@@ -77,7 +77,7 @@ struct RowNormRopeArgs {
   DType dt;
 };
 int launch_rownorm_rope_kv(const RowNormRopeArgs& args, cudaStream_t s);
-// rows [q | k | ..] of tokens: rotation of part of every query and key head, each head divided by its root mean square,
+// rows [q | k | ..] of tokens: rotation of part of every query and key head, each head divided by its root mean square (norm),
 // q to q_out [tokens, heads, q_width] (zeros behind dim), k and the unchanged values to the cache slots loc
 struct HeadNormRopeArgs {
   const void* row;          // row t at t * row_ld: heads * dim and kv_heads * dim features, kv_heads * vdim values at v_at
@@ -91,10 +91,68 @@ struct HeadNormRopeArgs {
   int64_t row_ld, k_tok_stride, k_head_stride, v_tok_stride, v_head_stride, num_slots;
   int tokens, heads, kv_heads, dim, vdim, v_at, q_width, rot_dims;
   int halves;               // pairs are (i, i + rot_dims / 2); 0: neighbours (2i, 2i + 1)
-  float eps;
+  int norm;                 // 0: heads keep their length
+  float eps, magnitude;     // magnitude: factor of the sines and cosines
   DType dt;
 };
 int launch_headnorm_rope_kv(const HeadNormRopeArgs& args, cudaStream_t s);
+// out = rmsnorm of x * silu(gate), the mean over each of `groups` equal parts of the row, times w
+int launch_gated_rmsnorm(const void* x, const void* gate, int64_t gate_ld, const float* w, void* out, int64_t out_ld, int rows, int width,
+                         int groups, float eps, DType dt, cudaStream_t s);
+
+// ----- the step between layers whose sublayers run side by side, with an average over depth (depth.cu) -----
+// causal convolution of single tokens with their input added: row t is the next token of the request with state row slots[t]
+struct ConvStepArgs {
+  const void* w;            // [width, taps], column taps - 1 meets the token itself; null: no convolution
+  void* state;              // [rows, width, taps - 1] the last inputs, oldest first; moved on
+  const int* slots;
+  int taps;
+};
+// normed rows of a stream: h = x / sqrt(mean(x^2) + eps) * g with a single number g; h1 may pass a convolution
+struct DepthInputs {
+  const float* g1;
+  const float* g2;
+  void* h1;                 // [rows, width]
+  void* h2;                 // [rows, width] or null
+  ConvStepArgs conv;
+};
+struct DepthStepArgs {
+  const float* x;           // [rows, width] what the layer's sublayers read
+  float* x_out;             // [rows, width] what goes on, or null; may be x
+  float* results;           // results 0 .. n - 1, result_stride elements apart; result n is written where keep is set
+  int64_t result_stride;
+  int n, keep;
+  const float* dwa;         // [n + 1] weights of the average, or null: the layer's result goes on
+  const void* a;            // [rows, width] mixer output
+  const void* b;            // [rows, width] a second one, or null; then mix = mix_scale * (norm(a) * a_w + norm(b) * b_w)
+  const float* a_w;         // [width]
+  const float* b_w;         // [width]
+  float mix_scale;
+  const void* f;            // [rows, width] feed-forward output or null
+  const void* expert_rows;  // choice j of token t is row sorted_pos[t * top + j] (negative: none), or null
+  const int* sorted_pos;
+  const float* topk_w;      // [rows, top] or null (1)
+  int top;
+  DepthInputs in;
+  int rows, width;
+  float eps;
+  DType dt;                 // of a, b, f, expert_rows, h1, h2, the convolution
+};
+int launch_depth_step(const DepthStepArgs& args, cudaStream_t s);
+// x = embedding row / sqrt(mean of its squares + eps) * g, and the inputs of the first layer
+struct EmbedNormArgs {
+  const int64_t* ids;
+  const void* table;        // [vocab, width]
+  const float* g;
+  float* x;                 // [rows, width]
+  int* status;
+  DepthInputs in;
+  int rows, width, vocab;
+  float eps;
+  DType dt;
+};
+int launch_embed_norm(const EmbedNormArgs& args, cudaStream_t s);
+
 void launch_soft_cap(const void* x, int64_t x_ld, float* out, int rows, int width, float cap, DType dt, cudaStream_t s);
 void launch_relu_squared(void* x, int64_t n, DType dt, cudaStream_t s);
 void launch_gelu_tanh(const void* x, void* out, int64_t n, DType dt, cudaStream_t s);
@@ -153,11 +211,13 @@ struct GemmArgs {
   void* out;             // [m, n_out] row-major
   const void* bias;      // [n] or null
   const void* residual;  // [m, n] or null (added before rounding)
+  float act_limit;       // swiglu 4
   const float* a_scale;  // int8 only: per-row scale [m]
   const float* b_scale;  // int8 only: per-column scale [n]
   int m, n, k;
   int64_t lda, ldb, ldc, ld_res;
   int swiglu;            // 1: b rows alternate 128 gate / 128 up rows; out is [m, n/2] = silu(gate) * up; 2: gelu_tanh(gate) * up;
+                         // 4: clamped_gate(gate + bias, up + bias, act_limit), the only gated form with a bias (rows as b's);
                          // 3: out is [m, n] = max(a b^T, 0)^2 (launch_gemm returns 1 for 9 to 256 rows: not fused there)
   DType dt;              // element type of a, b (kBF16 / kF16) ; out has the same type
   int is_int8;           // 1: a, b are int8, out type given by dt
@@ -267,9 +327,13 @@ struct RouteArgs {
 int launch_moe_router_topk(const RouteArgs& args, cudaStream_t s);
 // counting sort of the (token, choice) pairs by local expert.  sorted_pos[pair] = row in the sorted
 // matrix or -1 (expert on another rank); src_token[row] = token; expert_offsets[experts + 1];
-// work[i] = (expert, chunk of bn rows), *n_work items.
+// work[i] = (expert, chunk of bn rows), *n_work items.  src_w (or null): src_w[row] = topk_w of the row's pair.
 void launch_moe_align(const int* topk_ids, int pairs, int top_k, int expert_offset, int experts, int bn, int* sorted_pos,
-                      int* src_token, int* expert_offsets, int* work, int* n_work, int max_work, cudaStream_t s);
+                      int* src_token, int* expert_offsets, int* work, int* n_work, int max_work, const float* topk_w, float* src_w,
+                      cudaStream_t s);
+// rows of the pairs' tokens in expert order, each times src_w of its row
+void launch_moe_gather_scaled(const void* x, int64_t x_stride, const int* src_token, const float* src_w, const int* expert_offsets, int experts,
+                              void* xs, int pairs, int hidden, DType dt, cudaStream_t s);
 void launch_moe_gather(const void* x, int64_t x_stride, const int* src_token, const int* expert_offsets, int experts,
                        void* xs, int pairs, int hidden, int elem_bytes, cudaStream_t s);
 void launch_moe_combine(const void* y, const int* sorted_pos, const float* topk_w, void* out, int tokens, int hidden,
@@ -284,6 +348,7 @@ struct MoeGemmArgs {
   int* status;
   int64_t ldx, ldc;
   int rows_cap, experts, n, k, bn, max_work, swiglu, num_sms;
+  int gelu;         // the exact GELU of the plain product
   DType dt;
 };
 int launch_moe_grouped_gemm(const MoeGemmArgs& args, cudaStream_t s);
@@ -314,6 +379,7 @@ struct AttnArgs {
   int non_causal;           // prefill only: bidirectional attention inside each sequence
   float scale;
   int window;               // > 0: a query at position i sees keys i - window + 1 .. i only (causal attention)
+  int chunk;                // > 0 (without a window): a query at position i sees keys i / chunk * chunk .. i only
   float logit_cap;          // > 0: scores pass through cap * tanh(score / cap) before the softmax
   DType dt;
   const float* sink;        // [Hq] or null: per head, exp(sink) joins the softmax denominator (no key, no value, unscaled)
@@ -330,11 +396,12 @@ struct RowAttnArgs {
   void* out;                // [rows, heads, vdim], rows out_stride apart
   const int* req_to_token;
   const int* row_req;       // [rows] request-table row
-  const int64_t* row_pos;   // [rows] position: keys 0 .. position (the last `window` of them when window > 0)
+  const int64_t* row_pos;   // [rows] position: keys 0 .. position (the last `window` of them when window > 0, those of its
+                            // chunk of positions when chunk > 0)
   const float* sink;        // [heads] or null
   int* status;
   int64_t q_stride, out_stride, rtt_stride, num_slots, k_tok_stride, k_head_stride, v_tok_stride, v_head_stride;
-  int rows, heads, kv_heads, dim, vdim, window;
+  int rows, heads, kv_heads, dim, vdim, window, chunk;
   float scale, logit_cap;
   DType dt;
 };
@@ -354,12 +421,21 @@ struct LightningArgs {
   const int* lens;
   const int* has_state;
   const int* q_start;
+  // state-space duality (dt_raw null: lightning attention): rows activated already, q and k [T, k_heads, dk],
+  // dt = softplus(dt_raw + dt_bias), decay exp(-exp(a_log) dt), S <- decay S + dt k v^T, o = S^T q + skip v
+  const void* dt_raw;       // [T, heads], rows dt_ld apart
+  const float* dt_bias;     // [heads]
+  const float* a_log;       // [heads]
+  const float* skip;        // [heads]
+  int64_t dt_ld;
+  int k_heads;
   int64_t q_ld, k_ld, v_ld;
   int batch, heads, dk, dv;
   // chunk kernel: > 1 cuts every request's tokens into this many segments of seg_tokens (a multiple of 64; segments *
   // seg_tokens >= the longest request) that run side by side; ws holds [batch][segments][heads][dk][dv] fp32
   int segments, seg_tokens;
   float* ws;
+  float* ws_log;            // state-space duality with segments: [batch][segments][heads]
   DType dt;
 };
 int lightning_segments(int batch, int heads, int dv, int max_len, int num_sms);
@@ -372,8 +448,8 @@ bool lightning_chunk_covers(const LightningArgs& args);
 // ----- latent attention (one cached row of `rank` features per token, shared by all heads; `rot` rotated key features may
 // follow them in the row) ------------
 // Rows [q_rank | kv_rank | rot | ..] of the down projections: RMS norm of the first two, the first into cq, the second into
-// the cache row loc[t], where the third follows it, its neighbouring features turned by positions[t] * inv_freq.  kv_rank 0:
-// the layer reads another layer's rows and writes none.
+// the cache row loc[t], where the third follows it, its neighbouring features (halves: feature i with i + rot / 2) turned by
+// positions[t] * inv_freq.  kv_rank 0: the layer reads another layer's rows and writes none; q_rank 0: queries have no latent.
 struct LatentPrologueArgs {
   const void* y;            // [tokens, ..], rows ld apart
   const float* q_w;         // [q_rank]
@@ -386,20 +462,21 @@ struct LatentPrologueArgs {
   void* cache;
   int* status;
   int64_t ld, cache_ld, num_slots;
-  int tokens, q_rank, kv_rank, rot;
+  int tokens, q_rank, kv_rank, rot, halves;
   float eps;
   DType dt;
 };
 void launch_latent_prologue(const LatentPrologueArgs& args, cudaStream_t s);
-// neighbouring features of x [tokens, heads, rot] (strided) turn by turns [tokens, rot / 2]; out may be x
+// neighbouring features (halves: i and i + rot / 2) of x [tokens, heads, rot] (strided) turn by turns [tokens, rot / 2]; out may be x
 void launch_turn_heads(const void* x, int64_t x_tok, int64_t x_head, const float2* turns, void* out, int64_t out_tok, int64_t out_head,
-                       int tokens, int heads, int rot, DType dt, cudaStream_t s);
-// out [tokens, heads, width] = x (strided) * sigmoid(gate[t, h]), rows of gate gate_ld apart
-void launch_gate_heads(const void* x, int64_t x_tok, int64_t x_head, const void* gate, int64_t gate_ld, void* out, int tokens, int heads,
-                       int width, DType dt, cudaStream_t s);
-// out[start[b] + j] = latent of token j of request b, j < lens[b]
+                       int tokens, int heads, int rot, int halves, DType dt, cudaStream_t s);
+// out [tokens, heads, width] (strided, may be x) = x (strided) * sigmoid(gate[t, h]), rows of gate gate_ld apart; per_feature:
+// gate is [tokens, heads * width], a number for every feature
+void launch_gate_heads(const void* x, int64_t x_tok, int64_t x_head, const void* gate, int64_t gate_ld, void* out, int64_t out_tok,
+                       int64_t out_head, int tokens, int heads, int width, int per_feature, DType dt, cudaStream_t s);
+// out[start[b] + j] = latent of token first[b] + j of request b, j < lens[b] (first null: 0)
 void launch_latent_gather(const void* cache, int64_t cache_ld, int rank, int elem_bytes, const int* rtt, int64_t rtt_stride,
-                          const int* req, const int* lens, const int* start, int batch, int max_len, void* out,
+                          const int* req, const int* lens, const int* start, const int* first, int batch, int max_len, void* out,
                           int64_t num_slots, int* status, cudaStream_t s);
 // out[t, h, :N] = w[h] x[t, h, :K], times sigmoid(gate[t, h]) where gate is given; the `rot` features behind K are turned by
 // turns [tokens, rot / 2] and put behind N.  K % 8 == 0, 16-bit types (else -1)
@@ -407,10 +484,10 @@ struct HeadLinearArgs {
   const void* x;
   const void* w;            // [heads, N, K]
   void* out;
-  const void* gate;         // [tokens, heads] with rows gate_ld apart, or null
+  const void* gate;         // [tokens, heads] (gate_feat: [tokens, heads * N]) with rows gate_ld apart, or null
   const float2* turns;
   int64_t x_tok, x_head, out_tok, out_head, gate_ld;
-  int tokens, heads, N, K, rot;
+  int tokens, heads, N, K, rot, halves, gate_feat;
   DType dt;
 };
 int launch_head_linear(const HeadLinearArgs& args, int num_sms, cudaStream_t s);
@@ -422,11 +499,11 @@ struct LatentAttnArgs {
   float* part_lse;          // splits > 1: [rows, heads, splits]
   const int* req_to_token;
   const int* row_req;       // [rows] request-table row of each query
-  const int64_t* row_pos;   // [rows] its position: it sees keys 0 .. position
+  const int64_t* row_pos;   // [rows] its position: it sees keys 0 .. position, with window > 0 the last `window` of them
   const float* sink;        // [heads] or null
   int* status;
   int64_t rtt_stride, cache_ld, num_slots;
-  int rows, heads, key, rank, splits;
+  int rows, heads, key, rank, splits, window;
   float scale;
   DType dt;
 };
@@ -434,12 +511,12 @@ int launch_latent_attention(const LatentAttnArgs& args, cudaStream_t s);
 int latent_num_splits(int rows, int heads, int max_seq_len, int num_sms);
 bool latent_mma_covers(int key, int rank, int64_t cache_ld, DType dt);   // false: the fp32 kernel runs, splits must be 1
 
-// ----- gated delta net (hybrid models) -----------------------------------------------------------
+// ----- gated delta net (hybrid models): causal convolution (bias [C] or null; add_input: x + conv(x) instead of the SiLU), rule -----------------------------------------------------------
 // Ragged sequences: request b owns rows q_start[b] .. q_start[b] + lens[b] of the token-major inputs and
 // row slots[b] of the state tensors; has_state[b] != 0 resumes from the stored state.
 int launch_gdn_conv1d_silu(const void* x, int64_t x_ld, const void* w, void* conv_state, const int* slots, const int* lens,
                            const int* has_state, const int* q_start, void* out, int batch, int max_tokens, int channels, int K,
-                           DType dt, cudaStream_t s);
+                           const void* bias, int add_input, DType dt, cudaStream_t s);
 // beta = sigmoid(b), g = -exp(a_log) * softplus(a + dt_bias); b and a [tokens, heads] with rows ld apart
 void launch_gdn_gates(const void* b, const void* a, int64_t ld, const float* a_log, const float* dt_bias, float* g, float* beta,
                       int64_t tokens, int heads, DType dt, cudaStream_t s);
@@ -451,15 +528,15 @@ struct GdnRuleParams {
   const float* g;           // log decay [T, heads], or null: gates from the four fields below (recurrent kernel only)
   const float* beta;
   const void* b_raw;        // [T, heads] with rows gate_ld apart
-  const void* a_raw;
+  const void* a_raw;        // [T, heads]; with a decay per key channel (a_ld > 0) [T, heads * dk] with rows a_ld apart
   const float* a_log;       // [heads]
-  const float* dt_bias;     // [heads]
+  const float* dt_bias;     // [heads], per channel [heads * dk]
   float* state;             // [rows, heads, dk, dv]
   const int* slots;
   const int* lens;
   const int* has_state;
   const int* q_start;
-  int64_t q_ld, k_ld, v_ld, gate_ld;
+  int64_t q_ld, k_ld, v_ld, gate_ld, a_ld;
   int batch, heads, k_heads, dk, dv;
   int split_tf32;           // chunk kernel: two-term tf32 operands (fp32-like products)
   DType dt;
@@ -469,9 +546,18 @@ int launch_gdn_recurrent(const GdnRuleParams& p, cudaStream_t s);
 // the same rule evaluated 64 tokens at a time with tensor-core products (prefill); dk up to 128, multiples of 8
 int launch_gdn_chunk(const GdnRuleParams& p, int num_sms, cudaStream_t s);
 bool gdn_chunk_covers(const GdnRuleParams& p);
+// decays per key channel, 16 tokens at a time (prefill); dk up to 128, multiples of 8, gates formed inside.  The workspace
+// holds `span` chunks of every request; longer runs loop over spans
+struct GdnChannelPlan {
+  int span;
+  int64_t ws_floats;
+};
+GdnChannelPlan gdn_channel_plan(const GdnRuleParams& p, int max_len);
+int launch_gdn_channel_chunk(const GdnRuleParams& p, float* ws, int span, int max_len, int num_sms, cudaStream_t s);
+bool gdn_channel_chunk_covers(const GdnRuleParams& p);
 // x, out [rows = tokens * heads, width] contiguous, gate [tokens, heads * width] with rows gate_ld apart
 void launch_rmsnorm_gated(const void* x, const void* gate, int64_t gate_ld, const void* w, void* out, int64_t rows, int heads,
-                          int width, float eps, int round_norm, DType dt, cudaStream_t s);
+                          int width, float eps, int round_norm, int sigmoid, DType dt, cudaStream_t s);
 
 // ----- vision tower helpers ------------------------------------------------------------------
 // qkv [T, 3, H, D] (D <= 128, D % 8 == 0) -> q, k, v [T, H, 128] zero-padded; q and k get the 2-D rotary

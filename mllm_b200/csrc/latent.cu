@@ -1,7 +1,7 @@
 // Latent attention: every token leaves ONE row c of `rank` features in the cache, shared by all heads; a head's keys
 // and values are W_uk[h] c and W_uv[h] c.  A cached row may carry `rot` features more, a rotated key part that all heads
 // share: keys are then `key` = rank + rot features wide in the latent space, values stay `rank` wide.  Two ways to evaluate
-// it, both causal, both with an optional sink per head:
+// it, both causal, both with an optional sink per head and an optional sliding window:
 //
 //   expanded (many new tokens): K and V of the whole context are formed by matrix products and the ordinary
 //       attention kernels run on them; this file only gathers the context's latents (latent_gather).
@@ -32,15 +32,16 @@ constexpr float kLatLog2e = 1.4426950408889634f;
 // ---------------------------------------------------------------------------------------------
 // Prologue: the down projections' output rows are [query latent | cache latent | rotated key part]; both latents are
 // RMS-normed in 32-bit, the first goes to `cq`, the second to the cache row of the token.  The key part is turned by the
-// token's position (neighbouring features) and follows the latent in the cache row; the cosines and sines of the token are
-// left in `turns` for the query heads.  Angles are formed and reduced in fp64.  grid (tokens, 1 or 2).
+// token's position (neighbouring features, or with `halves` feature i with i + rot / 2) and follows the latent in the cache row; the cosines and sines of the token are
+// left in `turns` for the query heads.  Angles are formed and reduced in fp64.  Either latent may be missing (a query
+// without one, a layer that reads another layer's rows).  grid (tokens, number of latents).
 // ---------------------------------------------------------------------------------------------
 template <typename T>
 __global__ void __launch_bounds__(128) latent_prologue_kernel(const LatentPrologueArgs p) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float red[4];
-  const int t = blockIdx.x, part = blockIdx.y, tid = threadIdx.x;
+  const int t = blockIdx.x, part = p.q_rank > 0 ? blockIdx.y : 1, tid = threadIdx.x;
   const int n = part == 0 ? p.q_rank : p.kv_rank;
   const T* row = static_cast<const T*>(p.y) + static_cast<int64_t>(t) * p.ld + (part == 0 ? 0 : p.q_rank);
   const float* w = part == 0 ? p.q_w : p.kv_w;
@@ -51,7 +52,7 @@ __global__ void __launch_bounds__(128) latent_prologue_kernel(const LatentProlog
     if (!ok && tid == 0 && p.status != nullptr) atomicExch(p.status, kStatusBadIndex);
     dst = ok ? static_cast<T*>(p.cache) + slot * p.cache_ld : nullptr;
   }
-  if (part == static_cast<int>(gridDim.y) - 1) {
+  if (blockIdx.y == gridDim.y - 1) {
     const double pos = p.rot > 0 ? static_cast<double>(p.positions[t]) : 0.0;
     for (int i = tid; i < p.rot / 2; i += 128) {
       constexpr double kTurn = 6.283185307179586476925286766559;
@@ -61,9 +62,10 @@ __global__ void __launch_bounds__(128) latent_prologue_kernel(const LatentProlog
       sincosf(static_cast<float>(a), &s, &c);
       p.turns[static_cast<int64_t>(t) * (p.rot / 2) + i] = make_float2(c, s);
       if (part == 1 && dst != nullptr) {
-        const float u = to_f32(row[n + 2 * i]), v = to_f32(row[n + 2 * i + 1]);
-        dst[n + 2 * i] = from_f32<T>(u * c - v * s);
-        dst[n + 2 * i + 1] = from_f32<T>(v * c + u * s);
+        const int a0 = n + (p.halves ? i : 2 * i), a1 = p.halves ? a0 + p.rot / 2 : a0 + 1;
+        const float u = to_f32(row[a0]), v = to_f32(row[a1]);
+        dst[a0] = from_f32<T>(u * c - v * s);
+        dst[a1] = from_f32<T>(v * c + u * s);
       }
     }
   }
@@ -81,58 +83,68 @@ __global__ void __launch_bounds__(128) latent_prologue_kernel(const LatentProlog
   for (int c = tid; c < n; c += 128) dst[c] = from_f32<T>(to_f32(row[c]) * r * w[c]);
 }
 
-// Neighbouring features of x [tokens, heads, rot] turn by the token's `turns` [tokens, rot / 2]; out may be x.  A thread
-// takes a pair.
+// Neighbouring features (halves: feature i and i + rot / 2) of x [tokens, heads, rot] turn by the token's `turns`
+// [tokens, rot / 2]; out may be x.  A thread takes a pair.
 template <typename T>
 __global__ void __launch_bounds__(256) turn_heads_kernel(const T* x, int64_t x_tok, int64_t x_head, const float2* __restrict__ turns,
-                                                         T* out, int64_t out_tok, int64_t out_head, int heads, int half, int64_t pairs) {
+                                                         T* out, int64_t out_tok, int64_t out_head, int heads, int half, int64_t pairs, int halves) {
   pdl_launch_dependents();
   pdl_wait();
   for (int64_t e = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x; e < pairs; e += static_cast<int64_t>(gridDim.x) * blockDim.x) {
     const int i = static_cast<int>(e % half);
     const int64_t th = e / half, t = th / heads;
     const int h = static_cast<int>(th - t * heads);
-    const T* src = x + t * x_tok + h * x_head + 2 * i;
-    T* dst = out + t * out_tok + h * out_head + 2 * i;
+    const int a = halves ? i : 2 * i, o = halves ? half : 1;
+    const T* src = x + t * x_tok + h * x_head + a;
+    T* dst = out + t * out_tok + h * out_head + a;
     const float2 cs = turns[t * half + i];
-    const float u = to_f32(src[0]), v = to_f32(src[1]);
+    const float u = to_f32(src[0]), v = to_f32(src[o]);
     dst[0] = from_f32<T>(u * cs.x - v * cs.y);
-    dst[1] = from_f32<T>(v * cs.x + u * cs.y);
+    dst[o] = from_f32<T>(v * cs.x + u * cs.y);
   }
 }
 
 __device__ __forceinline__ float lat_sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
 
-// out[t, h, :] = x[t, h, :width] * sigmoid(gate[t, h]); V features per access
-template <typename T, int V>
+// out[t, h, :] = x[t, h, :width] * sigmoid(gate[t, h]), or, with FEAT, of gate[t, h, :width]; V features per access; out may
+// be x
+template <typename T, int V, bool FEAT>
 __global__ void __launch_bounds__(256) gate_heads_kernel(const T* x, int64_t x_tok, int64_t x_head, const T* __restrict__ gate,
-                                                         int64_t gate_ld, T* out, int heads, int vecs, int64_t total) {
+                                                         int64_t gate_ld, T* out, int64_t out_tok, int64_t out_head, int heads, int vecs,
+                                                         int64_t total) {
   pdl_launch_dependents();
   pdl_wait();
   struct alignas(sizeof(T) * V) Pack { T e[V]; };
   for (int64_t e = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x; e < total; e += static_cast<int64_t>(gridDim.x) * blockDim.x) {
     const int64_t th = e / vecs, t = th / heads;
     const int c = static_cast<int>(e - th * vecs) * V, h = static_cast<int>(th - t * heads);
-    const float g = lat_sigmoid(to_f32(gate[t * gate_ld + h]));
     Pack r = *reinterpret_cast<const Pack*>(x + t * x_tok + h * x_head + c);
+    if constexpr (FEAT) {
+      const Pack z = *reinterpret_cast<const Pack*>(gate + t * gate_ld + static_cast<int64_t>(h) * vecs * V + c);
 #pragma unroll
-    for (int i = 0; i < V; ++i) r.e[i] = from_f32<T>(to_f32(r.e[i]) * g);
-    *reinterpret_cast<Pack*>(out + th * vecs * V + c) = r;
+      for (int i = 0; i < V; ++i) r.e[i] = from_f32<T>(to_f32(r.e[i]) * lat_sigmoid(to_f32(z.e[i])));
+    } else {
+      const float g = lat_sigmoid(to_f32(gate[t * gate_ld + h]));
+#pragma unroll
+      for (int i = 0; i < V; ++i) r.e[i] = from_f32<T>(to_f32(r.e[i]) * g);
+    }
+    *reinterpret_cast<Pack*>(out + t * out_tok + h * out_head + c) = r;
   }
 }
 
-// Rows of a request's context, in position order: out[start[b] + j] = cache[rtt[req[b]][j]] for j < lens[b].
+// Rows of a request's context, in position order: out[start[b] + j] = cache[rtt[req[b]][first[b] + j]] for j < lens[b] (first
+// may be null: 0).
 template <typename V>
 __global__ void __launch_bounds__(256) latent_gather_kernel(const V* __restrict__ cache, int64_t cache_ld_v, int row_v,
                                                             const int* __restrict__ rtt, int64_t rtt_stride,
                                                             const int* __restrict__ req, const int* __restrict__ lens,
-                                                            const int* __restrict__ start, V* __restrict__ out,
+                                                            const int* __restrict__ start, const int* __restrict__ first, V* __restrict__ out,
                                                             int64_t num_slots, int* status) {
   pdl_launch_dependents();
   pdl_wait();
   const int b = blockIdx.y, n = lens[b];
   const int lane = threadIdx.x & 31;
-  const int* slots = rtt + static_cast<int64_t>(req[b]) * rtt_stride;
+  const int* slots = rtt + static_cast<int64_t>(req[b]) * rtt_stride + (first != nullptr ? first[b] : 0);
   for (int j = blockIdx.x * 8 + (threadIdx.x >> 5); j < n; j += gridDim.x * 8) {
     const int s = slots[j];
     const bool ok = s >= 0 && s < num_slots;
@@ -147,7 +159,7 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const V* __restrict_
 // Per-head projection out[t, h, :] = W[h] x[t, h, :], W [H, N, K].  A warp owns 16 rows of one head's W (the MMA M
 // dimension) and tiles of 8 tokens; a lane feeds 16 contiguous bytes of W and of x to two MMAs, the same
 // permutation of k in both operands.  KS > 1: the warps of the CTA split k of the same 16 rows.  gate: row t, head h is
-// multiplied by sigmoid(gate[t, h]).  rot > 0: the heads of x and of out go on with `rot` features behind K and N, which the
+// multiplied by sigmoid(gate[t, h]) (gate_feat: output n of head h by sigmoid(gate[t, h, n])).  rot > 0: the heads of x and of out go on with `rot` features behind K and N, which the
 // last CTAs of the x dimension turn by the tokens' `turns`.
 // ---------------------------------------------------------------------------------------------
 constexpr int kHlTokTiles = 4;   // tiles of 8 tokens per CTA
@@ -156,7 +168,8 @@ template <typename T, int KS>
 __global__ void __launch_bounds__(KS > 1 ? KS * 32 : 128) head_linear_kernel(const T* __restrict__ x, int64_t x_tok, int64_t x_head,
                                                           const T* __restrict__ w, T* __restrict__ out, int64_t out_tok,
                                                           int64_t out_head, int tokens, int N, int K, const T* __restrict__ gate,
-                                                          int64_t gate_ld, const float2* __restrict__ turns, int rot) {
+                                                          int64_t gate_ld, const float2* __restrict__ turns, int rot, int halves,
+                                                          int gate_feat) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float part[KS > 1 ? KS : 1][kHlTokTiles][16][8];
@@ -168,19 +181,23 @@ __global__ void __launch_bounds__(KS > 1 ? KS * 32 : 128) head_linear_kernel(con
     const int half = rot / 2, mine = min(tokens - t0, kHlTokTiles * 8);
     for (int e = threadIdx.x; e < mine * half; e += blockDim.x) {
       const int t = t0 + e / half, i = e % half;
-      const T* src = x + t * x_tok + h * x_head + K + 2 * i;
-      T* dst = out + t * out_tok + h * out_head + N + 2 * i;
+      const int a = halves ? i : 2 * i, o = halves ? half : 1;
+      const T* src = x + t * x_tok + h * x_head + K + a;
+      T* dst = out + t * out_tok + h * out_head + N + a;
       const float2 cs = turns[static_cast<int64_t>(t) * half + i];
-      const float u = to_f32(src[0]), v = to_f32(src[1]);
+      const float u = to_f32(src[0]), v = to_f32(src[o]);
       dst[0] = from_f32<T>(u * cs.x - v * cs.y);
-      dst[1] = from_f32<T>(v * cs.x + u * cs.y);
+      dst[o] = from_f32<T>(v * cs.x + u * cs.y);
     }
     return;
   }
   __shared__ float s_gate[kHlTokTiles * 8];
-  if (gate != nullptr && threadIdx.x < kHlTokTiles * 8)
+  if (gate != nullptr && !gate_feat && threadIdx.x < kHlTokTiles * 8)
     s_gate[threadIdx.x] = t0 + static_cast<int>(threadIdx.x) < tokens ? lat_sigmoid(to_f32(gate[(t0 + threadIdx.x) * gate_ld + h])) : 0.f;
-  auto gate_of = [&](int t) { return gate == nullptr ? 1.f : s_gate[t - t0]; };      // after a barrier
+  auto gate_of = [&](int t, int n) {      // after a barrier
+    if (gate == nullptr) return 1.f;
+    return gate_feat ? lat_sigmoid(to_f32(gate[t * gate_ld + static_cast<int64_t>(h) * N + n])) : s_gate[t - t0];
+  };
   const int g = lane >> 2, q = lane & 3;
   float acc[kHlTokTiles][4];
 #pragma unroll
@@ -225,7 +242,7 @@ __global__ void __launch_bounds__(KS > 1 ? KS * 32 : 128) head_linear_kernel(con
         float v = 0.f;
 #pragma unroll
         for (int s = 0; s < KS; ++s) v += part[s][i][r][tok];
-        out[t * out_tok + h * out_head + n0 + r] = from_f32<T>(v * gate_of(t));
+        out[t * out_tok + h * out_head + n0 + r] = from_f32<T>(v * gate_of(t, n0 + r));
       }
     }
   } else if (n0 < N) {
@@ -235,11 +252,10 @@ __global__ void __launch_bounds__(KS > 1 ? KS * 32 : 128) head_linear_kernel(con
       for (int j = 0; j < 2; ++j) {
         const int t = t0 + i * 8 + 2 * q + j;
         if (t >= tokens) continue;
-        const float f = gate_of(t);
 #pragma unroll
         for (int k = 0; k < 2; ++k) {
           const int r = n0 + g + k * 8;
-          if (r < N) out[t * out_tok + h * out_head + r] = from_f32<T>(acc[i][j + 2 * k] * f);
+          if (r < N) out[t * out_tok + h * out_head + r] = from_f32<T>(acc[i][j + 2 * k] * gate_of(t, r));
         }
       }
     }
@@ -257,11 +273,11 @@ struct LatentParams {
   float* part_lse;          // splits > 1: [rows, heads, splits], log2 domain
   const int* rtt;
   const int* row_req;       // [rows] row of the request table
-  const int64_t* row_pos;   // [rows] position of the query: it sees keys 0 .. pos
+  const int64_t* row_pos;   // [rows] position of the query: it sees keys 0 .. pos, with a window the last `window` of them
   const float* sink;        // [heads] or null
   int* status;
   int64_t rtt_stride, cache_ld, num_slots;
-  int rows, heads, key, rank, splits;
+  int rows, heads, key, rank, splits, window;
   float scale;
 };
 
@@ -305,10 +321,10 @@ __global__ void __launch_bounds__(NW * 32) latent_attn_mma_kernel(const LatentPa
   const uint32_t slice0 = smem_u32(lat_smem) + warp * C::kSliceBytes;                     // stage s: + s * warps * kSliceBytes
   const uint32_t stage_step = warps * C::kSliceBytes;
 
-  const int n = static_cast<int>(p.row_pos[row]) + 1;
-  const int tiles = (n + kLatTok - 1) / kLatTok;
-  const int per = (tiles + p.splits - 1) / p.splits;
-  const int tile0 = split * per, tile1 = min(tiles, tile0 + per);
+  const int n = static_cast<int>(p.row_pos[row]) + 1, first = p.window > 0 ? max(0, n - p.window) : 0;   // keys first .. n - 1
+  const int tiles = (n + kLatTok - 1) / kLatTok, lo = first / kLatTok;
+  const int per = (tiles - lo + p.splits - 1) / p.splits;
+  const int tile0 = lo + split * per, tile1 = min(tiles, tile0 + per);
   if (tile0 >= tile1) {   // empty split: a neutral partial
     for (int i = tid; i < kM * p.rank; i += blockDim.x) {
       const int h = h0 + i / p.rank;
@@ -421,7 +437,8 @@ __global__ void __launch_bounds__(NW * 32) latent_attn_mma_kernel(const LatentPa
       const int at = (e / kLatTok) * kLatSLd + e % kLatTok;
       float v = 0.f;
       for (int w = 0; w < warps; ++w) v += sp[w * kM * kLatSLd + at];
-      ss[at] = (t * kLatTok + e % kLatTok < n) ? v * scale_log2 : -INFINITY;
+      const int tk = t * kLatTok + e % kLatTok;
+      ss[at] = (tk < n && tk >= first) ? v * scale_log2 : -INFINITY;
     }
     __syncthreads();
 
@@ -574,7 +591,7 @@ __global__ void __launch_bounds__(kLatAnyThreads) latent_attn_any_kernel(const L
 #pragma unroll
   for (int i = 0; i < kLatAnyCols; ++i) acc[i] = 0.f;
   float m = -INFINITY, l = 0.f;
-  for (int t0 = 0; t0 < n; t0 += kLatAnyTok) {
+  for (int t0 = p.window > 0 ? max(0, n - p.window) : 0; t0 < n; t0 += kLatAnyTok) {
     const int nt = min(kLatAnyTok, n - t0);
     __syncthreads();      // sc and sl of the previous tile are no longer read; sq is written
     if (tid < nt) {
@@ -662,42 +679,53 @@ int launch_latent_mma(const LatentParams& p, cudaStream_t s) {
 
 void launch_latent_prologue(const LatentPrologueArgs& p, cudaStream_t s) {
   if (p.tokens == 0) return;
-  MB200_DISPATCH_FLOAT(p.dt, (launch_pdl(latent_prologue_kernel<T>, dim3(p.tokens, p.kv_rank > 0 ? 2 : 1), dim3(128), 0, s, p)));
+  const int parts = (p.q_rank > 0 ? 1 : 0) + (p.kv_rank > 0 ? 1 : 0);
+  if (parts == 0) return;
+  MB200_DISPATCH_FLOAT(p.dt, (launch_pdl(latent_prologue_kernel<T>, dim3(p.tokens, parts), dim3(128), 0, s, p)));
   note_launch();
 }
 
 void launch_turn_heads(const void* x, int64_t x_tok, int64_t x_head, const float2* turns, void* out, int64_t out_tok, int64_t out_head,
-                       int tokens, int heads, int rot, DType dt, cudaStream_t s) {
+                       int tokens, int heads, int rot, int halves, DType dt, cudaStream_t s) {
   const int64_t pairs = static_cast<int64_t>(tokens) * heads * (rot / 2);
   if (pairs == 0) return;
   const int grid = static_cast<int>(std::min<int64_t>((pairs + 255) / 256, 148 * 32));
   MB200_DISPATCH_FLOAT(dt, (launch_pdl(turn_heads_kernel<T>, dim3(grid), dim3(256), 0, s, static_cast<const T*>(x), x_tok, x_head, turns,
-                                       static_cast<T*>(out), out_tok, out_head, heads, rot / 2, pairs)));
+                                       static_cast<T*>(out), out_tok, out_head, heads, rot / 2, pairs, halves)));
   note_launch();
 }
 
-void launch_gate_heads(const void* x, int64_t x_tok, int64_t x_head, const void* gate, int64_t gate_ld, void* out, int tokens, int heads,
-                       int width, DType dt, cudaStream_t s) {
+void launch_gate_heads(const void* x, int64_t x_tok, int64_t x_head, const void* gate, int64_t gate_ld, void* out, int64_t out_tok,
+                       int64_t out_head, int tokens, int heads, int width, int per_feature, DType dt, cudaStream_t s) {
   if (tokens == 0 || width == 0) return;
-  const uintptr_t ptrs = reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(out);
-  auto go = [&](auto kernel, int v, const auto* xs, const auto* gs, auto* os) {
-    const int64_t total = static_cast<int64_t>(tokens) * heads * (width / v);
-    const int grid = static_cast<int>(std::min<int64_t>((total + 255) / 256, 148 * 32));
-    launch_pdl(kernel, dim3(grid), dim3(256), 0, s, xs, x_tok, x_head, gs, gate_ld, os, heads, width / v, total);
-  };
-  const bool vec = ptrs % 16 == 0 && width % 8 == 0 && x_tok % 8 == 0 && x_head % 8 == 0 && dt != kF32;
+  uintptr_t ptrs = reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(out);
+  int64_t sizes = width | x_tok | x_head | out_tok | out_head;
+  if (per_feature) {
+    ptrs |= reinterpret_cast<uintptr_t>(gate);
+    sizes |= gate_ld;
+  }
+  const bool vec = ptrs % 16 == 0 && sizes % 8 == 0 && dt != kF32;
+  const int v = vec ? 8 : 1;
+  const int64_t total = static_cast<int64_t>(tokens) * heads * (width / v);
+  const int grid = static_cast<int>(std::min<int64_t>((total + 255) / 256, 148 * 32));
   MB200_DISPATCH_FLOAT(dt, {
-    const T* xs = static_cast<const T*>(x);
-    const T* gs = static_cast<const T*>(gate);
-    T* os = static_cast<T*>(out);
-    if (vec) go(gate_heads_kernel<T, 8>, 8, xs, gs, os);
-    else go(gate_heads_kernel<T, 1>, 1, xs, gs, os);
+    auto go = [&](auto kernel) {
+      launch_pdl(kernel, dim3(grid), dim3(256), 0, s, static_cast<const T*>(x), x_tok, x_head, static_cast<const T*>(gate), gate_ld,
+                 static_cast<T*>(out), out_tok, out_head, heads, width / v, total);
+    };
+    if (per_feature) {
+      if (vec) go(gate_heads_kernel<T, 8, true>);
+      else go(gate_heads_kernel<T, 1, true>);
+    } else {
+      if (vec) go(gate_heads_kernel<T, 8, false>);
+      else go(gate_heads_kernel<T, 1, false>);
+    }
   });
   note_launch();
 }
 
 void launch_latent_gather(const void* cache, int64_t cache_ld, int rank, int elem_bytes, const int* rtt, int64_t rtt_stride,
-                          const int* req, const int* lens, const int* start, int batch, int max_len, void* out,
+                          const int* req, const int* lens, const int* start, const int* first, int batch, int max_len, void* out,
                           int64_t num_slots, int* status, cudaStream_t s) {
   if (batch == 0 || max_len == 0) return;
   const dim3 grid(std::min((max_len + 7) / 8, 2048), batch), block(256);
@@ -705,10 +733,10 @@ void launch_latent_gather(const void* cache, int64_t cache_ld, int rank, int ele
   const int64_t ld_bytes = cache_ld * elem_bytes;
   if (row_bytes % 16 == 0 && ld_bytes % 16 == 0) {
     launch_pdl(latent_gather_kernel<uint4>, grid, block, 0, s, static_cast<const uint4*>(cache), ld_bytes / 16, row_bytes / 16, rtt,
-               rtt_stride, req, lens, start, static_cast<uint4*>(out), num_slots, status);
+               rtt_stride, req, lens, start, first, static_cast<uint4*>(out), num_slots, status);
   } else {
     launch_pdl(latent_gather_kernel<uint16_t>, grid, block, 0, s, static_cast<const uint16_t*>(cache), ld_bytes / 2, row_bytes / 2,
-               rtt, rtt_stride, req, lens, start, static_cast<uint16_t*>(out), num_slots, status);
+               rtt, rtt_stride, req, lens, start, first, static_cast<uint16_t*>(out), num_slots, status);
   }
   note_launch();
 }
@@ -722,7 +750,7 @@ int launch_head_linear(const HeadLinearArgs& a, int num_sms, cudaStream_t s) {
     auto go = [&](auto kernel, int tiles, int threads) {
       launch_pdl(kernel, dim3(tiles + extra, a.heads, groups), dim3(threads), 0, s, static_cast<const T*>(a.x), a.x_tok, a.x_head,
                  static_cast<const T*>(a.w), static_cast<T*>(a.out), a.out_tok, a.out_head, a.tokens, a.N, a.K,
-                 static_cast<const T*>(a.gate), a.gate_ld, a.turns, a.rot);
+                 static_cast<const T*>(a.gate), a.gate_ld, a.turns, a.rot, a.halves, a.gate_feat);
     };
     if (split_k && a.K >= 256) go(head_linear_kernel<T, 8>, (a.N + 15) / 16, 256);
     else if (split_k) go(head_linear_kernel<T, 4>, (a.N + 15) / 16, 128);
@@ -766,6 +794,7 @@ int launch_latent_attention(const LatentAttnArgs& a, cudaStream_t s) {
   p.key = a.key;
   p.rank = a.rank;
   p.splits = a.splits;
+  p.window = a.window;
   p.scale = a.scale;
   if (!latent_mma_covers(a.key, a.rank, a.cache_ld, a.dt)) {
     if (a.splits != 1) return -1;

@@ -1,6 +1,11 @@
-// Lightning attention: linear attention with one fixed decay per head.  Per request and head,
+// Linear attention whose state decays by one number per head.  Lightning attention has a fixed decay; per request and head,
 //
 //   S_t = decay S_(t-1) + k_t v_t^T,   o_t = S_t^T q_t,   q, k, v = silu of the projections' rows (rounded to their type)
+//
+// State-space duality (GATED) takes decay and step size from the token, shares keys and queries among groups of heads, and
+// adds a multiple of the value; its rows come activated:
+//
+//   dt_t = softplus(raw_t + dt_bias),  S_t = exp(-exp(a_log) dt_t) S_(t-1) + dt_t k_t v_t^T,  o_t = S_t^T q_t + skip v_t
 //
 // with S [dk, dv] in fp32, kept per request row between passes.  Two evaluations of the same sums:
 //
@@ -8,10 +13,12 @@
 // * 64 tokens at a time (bf16 prefill): with S the state before the chunk and row i = 0 .. n - 1,
 //     O_i = decay^(i+1) Q_i S + sum_(j <= i) decay^(i-j) (Q_i . K_j) V_j
 //     S' = decay^n S + K^T diag(decay^(n-1-j)) V
-//   as warp-level tensor-core products.  Q, K and V are bf16 and enter as they are; fp32 operands are carried as sums of
+//   as warp-level tensor-core products (GATED: powers of the decay become exponentials of differences of the running sum of
+//   its logarithm, times dt_j).  Q, K and V are bf16 and enter as they are; fp32 operands are carried as sums of
 //   bf16 terms: two (16 bits) where the result is an output that is rounded to bf16 next, three (24 bits, all of fp32)
 //   where it stays in the state.  Nothing of the state passes through 16 bits.
 #include <algorithm>
+#include <type_traits>
 
 #include "common.cuh"
 #include "kernels.h"
@@ -31,7 +38,13 @@ __device__ __forceinline__ float silu_as(float v) {
 // token by token: grid (ceil(dv / 32), heads, batch), 256 threads; thread (rg, cl) = (tid / 8, tid % 8) holds rows rg,
 // rg + 32, ... of four columns of the state
 // ---------------------------------------------------------------------------------------------
-template <typename T, int RPT>
+// dt = softplus(raw + bias)
+__device__ __forceinline__ float step_size(float raw, float bias) {
+  const float z = raw + bias;
+  return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
+}
+
+template <typename T, int RPT, bool GATED>
 __global__ void __launch_bounds__(256) lightning_recurrent_kernel(const LightningArgs p) {
   pdl_launch_dependents();
   pdl_wait();
@@ -42,14 +55,16 @@ __global__ void __launch_bounds__(256) lightning_recurrent_kernel(const Lightnin
   if (n <= 0) return;
   const int c = blockIdx.x * 32 + cl * 4;
   const int64_t row0 = p.q_start[b];
+  const int hk = GATED ? h / (p.heads / p.k_heads) : h;
   float* S = p.state + (static_cast<int64_t>(p.slots[b]) * p.heads + h) * p.dk * p.dv;   // [dk][dv]
-  const T* q = static_cast<const T*>(p.q) + row0 * p.q_ld + static_cast<int64_t>(h) * p.dk;
-  const T* k = static_cast<const T*>(p.k) + row0 * p.k_ld + static_cast<int64_t>(h) * p.dk;
+  const T* q = static_cast<const T*>(p.q) + row0 * p.q_ld + static_cast<int64_t>(hk) * p.dk;
+  const T* k = static_cast<const T*>(p.k) + row0 * p.k_ld + static_cast<int64_t>(hk) * p.dk;
   const T* v = static_cast<const T*>(p.v) + row0 * p.v_ld + static_cast<int64_t>(h) * p.dv;
   T* out = static_cast<T*>(p.out) + (row0 * p.heads + h) * p.dv;
   const bool vec = (p.dv & 3) == 0;
   const bool resume = p.has_state[b] != 0;
-  const float decay = p.decay[h];
+  float decay = GATED ? 1.f : p.decay[h];
+  const float rate = GATED ? -expf(p.a_log[h]) : 0.f, skip = GATED ? p.skip[h] : 0.f, bias = GATED ? p.dt_bias[h] : 0.f;
   float s[RPT][4];
 #pragma unroll
   for (int r = 0; r < RPT; ++r) {
@@ -65,7 +80,7 @@ __global__ void __launch_bounds__(256) lightning_recurrent_kernel(const Lightnin
       }
     }
   }
-  float kn[RPT], qn[RPT], vn[4];
+  float kn[RPT], qn[RPT], vn[4], dtn = 0.f;
   auto load = [&](int t) {
 #pragma unroll
     for (int r = 0; r < RPT; ++r) {
@@ -75,15 +90,20 @@ __global__ void __launch_bounds__(256) lightning_recurrent_kernel(const Lightnin
     }
 #pragma unroll
     for (int j = 0; j < 4; ++j) vn[j] = c + j < p.dv ? to_f32(v[t * p.v_ld + c + j]) : 0.f;
+    if constexpr (GATED) dtn = step_size(to_f32(static_cast<const T*>(p.dt_raw)[(row0 + t) * p.dt_ld + h]), bias);
   };
   load(0);
   for (int t = 0; t < n; ++t) {
-    float o[4] = {0.f, 0.f, 0.f, 0.f}, v4[4];
+    float o[4] = {0.f, 0.f, 0.f, 0.f}, v4[4], d4[4];
 #pragma unroll
-    for (int j = 0; j < 4; ++j) v4[j] = silu_as<T>(vn[j]);
+    for (int j = 0; j < 4; ++j) {
+      v4[j] = GATED ? dtn * vn[j] : silu_as<T>(vn[j]);
+      d4[j] = GATED ? skip * vn[j] : 0.f;
+    }
+    if constexpr (GATED) decay = expf(rate * dtn);
 #pragma unroll
     for (int r = 0; r < RPT; ++r) {
-      const float kr = silu_as<T>(kn[r]), qr = silu_as<T>(qn[r]);
+      const float kr = GATED ? kn[r] : silu_as<T>(kn[r]), qr = GATED ? qn[r] : silu_as<T>(qn[r]);
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         s[r][j] = fmaf(decay, s[r][j], kr * v4[j]);
@@ -108,7 +128,7 @@ __global__ void __launch_bounds__(256) lightning_recurrent_kernel(const Lightnin
         a.z += x.z;
         a.w += x.w;
       }
-      const float r4[4] = {a.x, a.y, a.z, a.w};
+      const float r4[4] = {a.x + d4[0], a.y + d4[1], a.z + d4[2], a.w + d4[3]};
 #pragma unroll
       for (int j = 0; j < 4; ++j)
         if (c + j < p.dv) out[static_cast<int64_t>(t) * p.heads * p.dv + c + j] = from_f32<T>(r4[j]);
@@ -137,16 +157,18 @@ __global__ void __launch_bounds__(256) lightning_recurrent_kernel(const Lightnin
 // kWhole: one CTA walks all new tokens.  When that leaves SMs idle the tokens are cut into segments, and two launches
 // share the work through `ws` [batch][segments][heads][dk][dv]: kSums leaves the state before the request in slot 0 and
 // the sum K^T diag(decay^..) V of segment s in slot s + 1; kOutputs starts every segment from
-// (((slot 0) D + slot 1) D + ...), D = decay^(tokens of a segment), and the last segment writes the new state.
+// (((slot 0) D + slot 1) D + ...), D = decay^(tokens of a segment) (GATED: kSums leaves log2 D of each segment in `ws_log`), and
+// the last segment writes the new state.
 // ---------------------------------------------------------------------------------------------
 using bf16 = __nv_bfloat16;
+constexpr float kLog2e = 1.4426950408889634f;
 constexpr int kLcTok = 64, kLcV = 64, kLcLdV = kLcV + 8, kLcThreads = 256;
 
 template <int DK>
 struct LightningCfg {
   static constexpr int kLd = DK + 8;
   static constexpr int kElems = 2 * kLcTok * kLd + 4 * kLcTok * kLcLdV + 2 * DK * kLcLdV;
-  static constexpr int kSmem = kElems * 2 + (kLcTok + 1) * 4;
+  static constexpr int kSmem = kElems * 2 + 4 * kLcTok * 4 + 16;
 };
 
 // Two fp32 values as sums of bf16 terms, each pair of terms packed for an operand register.  A leading term is the value
@@ -173,7 +195,7 @@ __device__ __forceinline__ void silu_pair(float& a, float& b) {
 
 enum LightningMode { kWhole, kSums, kOutputs };
 
-template <int DK, int MODE>
+template <int DK, int MODE, bool GATED>
 __global__ void __launch_bounds__(kLcThreads, 2) lightning_chunk_kernel(const LightningArgs p) {
   pdl_wait();
   using C = LightningCfg<DK>;
@@ -185,21 +207,25 @@ __global__ void __launch_bounds__(kLcThreads, 2) lightning_chunk_kernel(const Li
   bf16* sW = sV + kLcTok * kLcLdV;                  // [3][64][72] terms of decay^(n-1-j) v_j
   bf16* sS = sW + 3 * kLcTok * kLcLdV;              // [2][DK][72] terms of the state before the chunk
   float* sPow = reinterpret_cast<float*>(sS + 2 * DK * kLcLdV);   // decay^0 .. decay^64
+  // GATED: running sum G of log2 decay, 2^G, dt, and the weight 2^(G_end - G) dt of a token in the state after the chunk
+  float *sG = sPow, *sE = sG + kLcTok, *sDt = sE + kLcTok, *sWt = sDt + kLcTok;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int seg = MODE == kWhole ? 0 : static_cast<int>(blockIdx.x) % p.segments;
   const int vb = (MODE == kWhole ? static_cast<int>(blockIdx.x) : static_cast<int>(blockIdx.x) / p.segments) * kLcV, h = blockIdx.y, b = blockIdx.z;
   const int n = p.lens[b];
   const int t_begin = MODE == kWhole ? 0 : seg * p.seg_tokens, t_end = MODE == kWhole ? n : min(n, t_begin + p.seg_tokens);
   if (n <= 0 || t_begin >= n) return;
-  const int dk = p.dk, dv = p.dv, cols = min(kLcV, dv - vb);
+  const int dk = p.dk, dv = p.dv, cols = min(kLcV, dv - vb), hk = GATED ? h / (p.heads / p.k_heads) : h;
   const int64_t row0 = p.q_start[b];
-  const bf16* q = static_cast<const bf16*>(p.q) + row0 * p.q_ld + static_cast<int64_t>(h) * dk;
-  const bf16* k = static_cast<const bf16*>(p.k) + row0 * p.k_ld + static_cast<int64_t>(h) * dk;
+  const bf16* q = static_cast<const bf16*>(p.q) + row0 * p.q_ld + static_cast<int64_t>(hk) * dk;
+  const bf16* k = static_cast<const bf16*>(p.k) + row0 * p.k_ld + static_cast<int64_t>(hk) * dk;
   const bf16* v = static_cast<const bf16*>(p.v) + row0 * p.v_ld + static_cast<int64_t>(h) * dv + vb;
   bf16* out = static_cast<bf16*>(p.out) + (row0 * p.heads + h) * dv + vb;
   float* S = p.state + (static_cast<int64_t>(p.slots[b]) * p.heads + h) * dk * dv + vb;
   const bool resume = p.has_state[b] != 0;
-  if (tid <= kLcTok) sPow[tid] = powf(p.decay[h], static_cast<float>(tid));
+  if (!GATED && tid <= kLcTok) sPow[tid] = powf(p.decay[h], static_cast<float>(tid));
+  const float rate2 = GATED ? -expf(p.a_log[h]) * kLog2e : 0.f, bias = GATED ? p.dt_bias[h] : 0.f, skip = GATED ? p.skip[h] : 0.f;
+  float log_total = 0.f;                 // GATED: log2 of the segment's decay so far
 
   // this warp's part of S: row tile mt, n tiles n0 .. n0 + kNT - 1
   const int mt = warp % kMT, n0 = (warp / kMT) * kNT;
@@ -224,14 +250,44 @@ __global__ void __launch_bounds__(kLcThreads, 2) lightning_chunk_kernel(const Li
     if (seg == 0) for_state([&](float&, int64_t at) { ws[at] = resume ? S[at] : 0.f; });
     if (t_end == n) return;              // no later segment asks for this one's sum
   } else {
-    const float full = powf(p.decay[h], static_cast<float>(p.seg_tokens));
+    float full = GATED ? 1.f : powf(p.decay[h], static_cast<float>(p.seg_tokens));
     for_state([&](float& x, int64_t at) { x = ws[at]; });
-    for (int k2 = 1; k2 <= seg; ++k2) for_state([&](float& x, int64_t at) { x = fmaf(x, full, ws[k2 * slot_elems + at]); });
+    for (int k2 = 1; k2 <= seg; ++k2) {
+      if constexpr (GATED) full = exp2f(p.ws_log[(static_cast<int64_t>(b) * p.segments + k2 - 1) * p.heads + h]);
+      for_state([&](float& x, int64_t at) { x = fmaf(x, full, ws[k2 * slot_elems + at]); });
+    }
   }
   __syncthreads();
 
   for (int c0 = t_begin; c0 < t_end; c0 += kLcTok) {
     const int nv = min(kLcTok, t_end - c0);
+    if constexpr (GATED) {
+      if (warp == 0) {       // two tokens per lane; tokens past the end have dt = 0
+        float dt[2], a[2];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const int r = 2 * lane + i;
+          dt[i] = r < nv ? step_size(to_f32(static_cast<const bf16*>(p.dt_raw)[(row0 + c0 + r) * p.dt_ld + h]), bias) : 0.f;
+          a[i] = rate2 * dt[i];
+        }
+        float up = a[0] + a[1], down = up;             // running sums from both ends
+#pragma unroll
+        for (int d = 1; d < 32; d <<= 1) {
+          const float u = __shfl_up_sync(0xffffffffu, up, d), w = __shfl_down_sync(0xffffffffu, down, d);
+          if (lane >= d) up += u;
+          if (lane + d < 32) down += w;
+        }
+        const float before = up - (a[0] + a[1]);
+        float after = __shfl_down_sync(0xffffffffu, down, 1);
+        if (lane == 31) after = 0.f;
+        const float g0 = before + a[0];
+        *reinterpret_cast<float2*>(sG + 2 * lane) = make_float2(g0, up);
+        *reinterpret_cast<float2*>(sE + 2 * lane) = make_float2(exp2f(g0), exp2f(up));
+        *reinterpret_cast<float2*>(sDt + 2 * lane) = make_float2(dt[0], dt[1]);
+        *reinterpret_cast<float2*>(sWt + 2 * lane) = make_float2(exp2f(after + a[1]) * dt[0], exp2f(after) * dt[1]);
+      }
+      __syncthreads();
+    }
     // ---- rows of the chunk: activated, missing rows and features zero; the values also scaled, in three terms ----
     auto load8 = [&](const bf16* src, bool valid, float (&f)[8]) {
       uint4 raw = make_uint4(0u, 0u, 0u, 0u);
@@ -240,7 +296,7 @@ __global__ void __launch_bounds__(kLcThreads, 2) lightning_chunk_kernel(const Li
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         float2 t = unpack_bf16x2(u[i]);
-        silu_pair(t.x, t.y);
+        if constexpr (!GATED) silu_pair(t.x, t.y);
         f[2 * i] = t.x;
         f[2 * i + 1] = t.y;
       }
@@ -267,7 +323,7 @@ __global__ void __launch_bounds__(kLcThreads, 2) lightning_chunk_kernel(const Li
       load8(v + static_cast<int64_t>(c0 + r) * p.v_ld + d, r < nv && d < cols, f);
       const uint4 raw = pack8(f);
       *reinterpret_cast<uint4*>(sV + r * kLcLdV + d) = raw;
-      const float w = r < nv ? sPow[nv - 1 - r] : 0.f;
+      const float w = GATED ? sWt[r] : r < nv ? sPow[nv - 1 - r] : 0.f;
       const uint32_t* u = reinterpret_cast<const uint32_t*>(&raw);
 #pragma unroll
       for (int j = 0; j < 4; ++j) {        // the rounded value, scaled
@@ -316,7 +372,8 @@ __global__ void __launch_bounds__(kLcThreads, 2) lightning_chunk_kernel(const Li
             }
         }
         const int ra = rt * 16 + g, rb = ra + 8;
-        const float da = sPow[ra + 1], db = sPow[rb + 1];
+        const float da = GATED ? sE[ra] : sPow[ra + 1], db = GATED ? sE[rb] : sPow[rb + 1];
+        const float ga = GATED ? sG[ra] : 0.f, gb = GATED ? sG[rb] : 0.f;
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
           o[i][0] *= da;
@@ -340,8 +397,9 @@ __global__ void __launch_bounds__(kLcThreads, 2) lightning_chunk_kernel(const Li
           for (int i = 0; i < 2; ++i)
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-              const int d = ((e >> 1) ? rb : ra) - (jt * 16 + i * 8 + c2 + (e & 1));
-              s[i][e] = d >= 0 ? s[i][e] * sPow[d] : 0.f;
+              const int j = jt * 16 + i * 8 + c2 + (e & 1), d = ((e >> 1) ? rb : ra) - j;
+              if constexpr (GATED) s[i][e] = d >= 0 ? s[i][e] * (exp2f(((e >> 1) ? gb : ga) - sG[j]) * sDt[j]) : 0.f;
+              else s[i][e] = d >= 0 ? s[i][e] * sPow[d] : 0.f;
             }
           uint32_t ph[4], pl[4];
           split2(s[0][0], s[0][1], ph[0], pl[0]);
@@ -362,6 +420,14 @@ __global__ void __launch_bounds__(kLcThreads, 2) lightning_chunk_kernel(const Li
         for (int i = 0; i < 4; ++i) {
           const int c = oc + i * 8 + c2;
           if (c < cols) {      // dv is even: pairs never straddle the end
+            if constexpr (GATED) {
+              const float2 va = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(sV + ra * kLcLdV + c));
+              const float2 vc = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(sV + rb * kLcLdV + c));
+              o[i][0] = fmaf(skip, va.x, o[i][0]);
+              o[i][1] = fmaf(skip, va.y, o[i][1]);
+              o[i][2] = fmaf(skip, vc.x, o[i][2]);
+              o[i][3] = fmaf(skip, vc.y, o[i][3]);
+            }
             if (ra < nv)
               *reinterpret_cast<uint32_t*>(out + static_cast<int64_t>(c0 + ra) * p.heads * dv + c) = pack_bf16x2(o[i][0], o[i][1]);
             if (rb < nv)
@@ -372,7 +438,8 @@ __global__ void __launch_bounds__(kLcThreads, 2) lightning_chunk_kernel(const Li
     }
     // ---- S' = decay^n S + K^T W.  The chunk's sum is formed by itself and added in one fp32 operation: the tensor core
     // cuts off what an accumulator cannot hold, which would add up in the large S ----
-    const float carry = sPow[nv];
+    const float carry = GATED ? sE[kLcTok - 1] : sPow[nv];
+    if constexpr (GATED && MODE == kSums) log_total += sG[kLcTok - 1];
     float add[kNT][4];
 #pragma unroll
     for (int nt = 0; nt < kNT; ++nt) add[nt][0] = add[nt][1] = add[nt][2] = add[nt][3] = 0.f;
@@ -400,39 +467,40 @@ __global__ void __launch_bounds__(kLcThreads, 2) lightning_chunk_kernel(const Li
   }
   if constexpr (MODE == kSums) {
     float* mine = ws + (seg + 1) * slot_elems;
+    if (GATED && tid == 0 && vb == 0) p.ws_log[(static_cast<int64_t>(b) * p.segments + seg) * p.heads + h] = log_total;
     for_state([&](float& x, int64_t at) { mine[at] = x; });
   } else if (t_end == n) {
     for_state([&](float& x, int64_t at) { S[at] = x; });
   }
 }
 
-template <typename T>
+template <typename T, bool GATED>
 int launch_recurrent_t(const LightningArgs& p, cudaStream_t s) {
   const dim3 grid((p.dv + 31) / 32, p.heads, p.batch), block(256);
-  if (p.dk <= 32) launch_pdl(lightning_recurrent_kernel<T, 1>, grid, block, 0, s, p);
-  else if (p.dk <= 64) launch_pdl(lightning_recurrent_kernel<T, 2>, grid, block, 0, s, p);
-  else if (p.dk <= 128) launch_pdl(lightning_recurrent_kernel<T, 4>, grid, block, 0, s, p);
-  else if (p.dk <= 256) launch_pdl(lightning_recurrent_kernel<T, 8>, grid, block, 0, s, p);
-  else if (p.dk <= 512) launch_pdl(lightning_recurrent_kernel<T, 16>, grid, block, 0, s, p);
+  if (p.dk <= 32) launch_pdl(lightning_recurrent_kernel<T, 1, GATED>, grid, block, 0, s, p);
+  else if (p.dk <= 64) launch_pdl(lightning_recurrent_kernel<T, 2, GATED>, grid, block, 0, s, p);
+  else if (p.dk <= 128) launch_pdl(lightning_recurrent_kernel<T, 4, GATED>, grid, block, 0, s, p);
+  else if (p.dk <= 256) launch_pdl(lightning_recurrent_kernel<T, 8, GATED>, grid, block, 0, s, p);
+  else if (p.dk <= 512) launch_pdl(lightning_recurrent_kernel<T, 16, GATED>, grid, block, 0, s, p);
   else return -1;
   note_launch();
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
-template <int DK, int MODE>
+template <int DK, int MODE, bool GATED>
 int launch_chunk_mode(const LightningArgs& p, cudaStream_t s) {
-  auto kern = lightning_chunk_kernel<DK, MODE>;
+  auto kern = lightning_chunk_kernel<DK, MODE, GATED>;
   if (ensure_dynamic_smem(reinterpret_cast<const void*>(kern), LightningCfg<DK>::kSmem) != cudaSuccess) return -3;
   const int blocks = (p.dv + kLcV - 1) / kLcV * (MODE == kWhole ? 1 : p.segments);
   const cudaError_t err = launch_pdl(kern, dim3(blocks, p.heads, p.batch), dim3(kLcThreads), LightningCfg<DK>::kSmem, s, p);
   note_launch();
   return err == cudaSuccess ? 0 : -4;
 }
-template <int DK>
+template <int DK, bool GATED>
 int launch_chunk_t(const LightningArgs& p, cudaStream_t s) {
-  if (p.segments <= 1) return launch_chunk_mode<DK, kWhole>(p, s);
-  const int rc = launch_chunk_mode<DK, kSums>(p, s);
-  return rc != 0 ? rc : launch_chunk_mode<DK, kOutputs>(p, s);
+  if (p.segments <= 1) return launch_chunk_mode<DK, kWhole, GATED>(p, s);
+  const int rc = launch_chunk_mode<DK, kSums, GATED>(p, s);
+  return rc != 0 ? rc : launch_chunk_mode<DK, kOutputs, GATED>(p, s);
 }
 
 }  // namespace
@@ -440,7 +508,7 @@ int launch_chunk_t(const LightningArgs& p, cudaStream_t s) {
 int launch_lightning_recurrent(const LightningArgs& p, cudaStream_t s) {
   if (p.batch <= 0) return 0;
   int rc = 0;
-  MB200_DISPATCH_FLOAT(p.dt, rc = launch_recurrent_t<T>(p, s));
+  MB200_DISPATCH_FLOAT(p.dt, rc = p.dt_raw != nullptr ? (launch_recurrent_t<T, true>(p, s)) : (launch_recurrent_t<T, false>(p, s)));
   return rc;
 }
 
@@ -460,7 +528,13 @@ int launch_lightning_chunk(const LightningArgs& p, cudaStream_t s) {
   if (p.batch <= 0) return 0;
   if (!lightning_chunk_covers(p)) return -1;
   if (p.segments > 1 && (p.ws == nullptr || p.seg_tokens <= 0 || p.seg_tokens % kLcTok != 0)) return -1;
-  return p.dk <= 32 ? launch_chunk_t<32>(p, s) : p.dk <= 64 ? launch_chunk_t<64>(p, s) : launch_chunk_t<128>(p, s);
+  auto go = [&](auto gated) {
+    constexpr bool kGated = decltype(gated)::value;
+    return p.dk <= 32 ? launch_chunk_t<32, kGated>(p, s) : p.dk <= 64 ? launch_chunk_t<64, kGated>(p, s) : launch_chunk_t<128, kGated>(p, s);
+  };
+  if (p.dt_raw == nullptr) return go(std::false_type{});
+  if (p.heads % p.k_heads != 0 || (p.segments > 1 && p.ws_log == nullptr)) return -1;
+  return go(std::true_type{});
 }
 
 }  // namespace mb200

@@ -9,7 +9,7 @@
 // handful of tokens still issues full-width MMAs and the kernel streams every active expert's
 // weights exactly once.  Work items (expert, token chunk) are written by the align kernel; CTAs
 // are persistent and walk item x weight-row-tile pairs.  With SWIGLU the weights hold alternating
-// 128-row gate / up blocks and the epilogue writes silu(gate) * up.
+// 128-row gate / up blocks and the epilogue writes silu(gate) * up; with GELU there is no gate and it writes the exact GELU.
 //
 // Warp roles (256 threads): warp 0 TMA producer, warp 1 MMA issuer, warp 2 TMEM allocator,
 // warps 4-7 epilogue.  Every barrier wait is bounded (kStatusPipelineTimeout on expiry).
@@ -345,7 +345,7 @@ int launch_router_mma_t(const void* x, int64_t x_ld, const void* w, float* logit
 __global__ void __launch_bounds__(1024)
 moe_align_kernel(const int* __restrict__ topk_ids, int pairs, int top_k, int expert_offset, int experts, int bn,
                  int* __restrict__ sorted_pos, int* __restrict__ src_token, int* __restrict__ expert_offsets,
-                 int2* __restrict__ work, int* __restrict__ n_work, int max_work) {
+                 int2* __restrict__ work, int* __restrict__ n_work, int max_work, const float* __restrict__ topk_w, float* __restrict__ src_w) {
   pdl_wait();
   __shared__ int cnt[kMaxExperts], off[kMaxExperts + 1], wbase[kMaxExperts + 1], fill[kMaxExperts];
   for (int e = threadIdx.x; e < kMaxExperts; e += blockDim.x) {
@@ -383,6 +383,7 @@ moe_align_kernel(const int* __restrict__ topk_ids, int pairs, int top_k, int exp
       const int pos = off[e] + atomicAdd(&fill[e], 1);
       sorted_pos[i] = pos;
       src_token[pos] = i / top_k;
+      if (src_w != nullptr) src_w[pos] = topk_w[i];
     } else {
       sorted_pos[i] = -1;
     }
@@ -400,6 +401,26 @@ __global__ void moe_gather_kernel(const V* __restrict__ x, int64_t x_stride_v, c
   const V* src = x + static_cast<int64_t>(src_token[pos]) * x_stride_v;
   V* dst = xs + static_cast<int64_t>(pos) * row_vecs;
   for (int i = threadIdx.x; i < row_vecs; i += blockDim.x) dst[i] = __ldg(src + i);
+}
+
+// the same with every row times the weight of its pair
+template <typename T, int V>
+__global__ void moe_gather_scaled_kernel(const T* __restrict__ x, int64_t x_stride, const int* __restrict__ src_token,
+                                         const float* __restrict__ src_w, const int* __restrict__ expert_offsets, int experts,
+                                         T* __restrict__ xs, int vecs) {
+  pdl_wait();
+  const int pos = blockIdx.x;
+  if (pos >= expert_offsets[experts]) return;
+  struct alignas(sizeof(T) * V) Pack { T e[V]; };
+  const T* src = x + static_cast<int64_t>(src_token[pos]) * x_stride;
+  T* dst = xs + static_cast<int64_t>(pos) * vecs * V;
+  const float w = src_w[pos];
+  for (int i = threadIdx.x; i < vecs; i += blockDim.x) {
+    Pack r = *reinterpret_cast<const Pack*>(src + i * V);
+#pragma unroll
+    for (int j = 0; j < V; ++j) r.e[j] = from_f32<T>(to_f32(r.e[j]) * w);
+    *reinterpret_cast<Pack*>(dst + i * V) = r;
+  }
 }
 
 // out[t, :] = sum_j w[t, j] * y[sorted_pos[t*k + j], :]   (choices on other ranks contribute nothing)
@@ -459,8 +480,9 @@ struct GCfg {
 };
 
 __device__ __forceinline__ float silu_f(float v) { return v / (1.f + __expf(-v)); }
+__device__ __forceinline__ float gelu_erf_f(float v) { return 0.5f * v * (1.f + erff(v * 0.70710678118654752f)); }
 
-template <int BN, bool SWIGLU>
+template <int BN, bool SWIGLU, bool GELU>
 __global__ void __launch_bounds__(kThreads, 1)
 moe_grouped_gemm_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__ CUtensorMap tm_x,
                         const GroupedParams p) {
@@ -616,6 +638,7 @@ moe_grouped_gemm_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_c
           if (c + j >= valid) break;
           float x = __uint_as_float(v0[j]);
           if constexpr (SWIGLU) x = silu_f(x) * __uint_as_float(v1[j]);
+          if constexpr (GELU) x = gelu_erf_f(x);
           const int64_t o = static_cast<int64_t>(row0 + c + j) * p.ldc + ocol;
           if (p.out_f16)
             static_cast<__half*>(p.out)[o] = __float2half_rn(x);
@@ -649,7 +672,7 @@ moe_grouped_gemm_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_c
 // with four tokens each.  Work items are those of moe_align with chunks of 16 rows.
 constexpr int kGaRows = 64, kGaTok = 16, kGaK = 16;
 
-template <typename T>
+template <typename T, bool GELU>
 __global__ void __launch_bounds__(256) moe_grouped_any_kernel(const T* __restrict__ x, int64_t ldx, const T* __restrict__ w,
                                                               T* __restrict__ out, int64_t ldc, const int* __restrict__ expert_offsets,
                                                               const int2* __restrict__ work, const int* __restrict__ n_work, int n, int k) {
@@ -684,15 +707,15 @@ __global__ void __launch_bounds__(256) moe_grouped_any_kernel(const T* __restric
     if (c0 + col < n) {
 #pragma unroll
       for (int i = 0; i < 4; ++i)
-        if (tg * 4 + i < valid) out[static_cast<int64_t>(row0 + tg * 4 + i) * ldc + c0 + col] = from_f32<T>(acc[i]);
+        if (tg * 4 + i < valid) out[static_cast<int64_t>(row0 + tg * 4 + i) * ldc + c0 + col] = from_f32<T>(GELU ? gelu_erf_f(acc[i]) : acc[i]);
     }
   }
 }
 
-template <int BN, bool SWIGLU>
+template <int BN, bool SWIGLU, bool GELU>
 int launch_grouped_cfg(const CUtensorMap& tw, const CUtensorMap& tx, const GroupedParams& p, int grid, cudaStream_t s) {
   using C = GCfg<BN, SWIGLU>;
-  auto kern = moe_grouped_gemm_kernel<BN, SWIGLU>;
+  auto kern = moe_grouped_gemm_kernel<BN, SWIGLU, GELU>;
   const size_t smem = static_cast<size_t>(C::kStages) * C::kStageBytes + 1024 + 512;
   if (ensure_dynamic_smem(reinterpret_cast<const void*>(kern), static_cast<int>(smem)) != cudaSuccess) return -3;
   const cudaError_t err = launch_pdl(kern, dim3(grid), dim3(kThreads), smem, s, tw, tx, p);
@@ -754,9 +777,10 @@ int launch_moe_router_logits(const void* x, int64_t x_ld, const void* w, float* 
 }
 
 void launch_moe_align(const int* topk_ids, int pairs, int top_k, int expert_offset, int experts, int bn, int* sorted_pos,
-                      int* src_token, int* expert_offsets, int* work, int* n_work, int max_work, cudaStream_t s) {
+                      int* src_token, int* expert_offsets, int* work, int* n_work, int max_work, const float* topk_w, float* src_w,
+                       cudaStream_t s) {
   launch_pdl(moe_align_kernel, dim3(1), dim3(1024), 0, s, topk_ids, pairs, top_k, expert_offset, experts, bn, sorted_pos,
-             src_token, expert_offsets, reinterpret_cast<int2*>(work), n_work, max_work);
+             src_token, expert_offsets, reinterpret_cast<int2*>(work), n_work, max_work, topk_w, src_w);
   note_launch();
 }
 
@@ -776,6 +800,24 @@ void launch_moe_gather(const void* x, int64_t x_stride, const int* src_token, co
   note_launch();
 }
 
+void launch_moe_gather_scaled(const void* x, int64_t x_stride, const int* src_token, const float* src_w, const int* expert_offsets, int experts,
+                              void* xs, int pairs, int hidden, DType dt, cudaStream_t s) {
+  if (pairs == 0) return;
+  const uintptr_t ptrs = reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(xs);
+  const int v = dt == kF32 ? 4 : 8;
+  const bool vec = ptrs % 16 == 0 && hidden % v == 0 && x_stride % v == 0;
+  MB200_DISPATCH_FLOAT(dt, {
+    constexpr int kV = 16 / static_cast<int>(sizeof(T));
+    auto go = [&](auto kernel, int vecs) {
+      launch_pdl(kernel, dim3(pairs), dim3(128), 0, s, static_cast<const T*>(x), x_stride, src_token, src_w, expert_offsets, experts,
+                 static_cast<T*>(xs), vecs);
+    };
+    if (vec) go(moe_gather_scaled_kernel<T, kV>, hidden / kV);
+    else go(moe_gather_scaled_kernel<T, 1>, hidden);
+  });
+  note_launch();
+}
+
 void launch_moe_combine(const void* y, const int* sorted_pos, const float* topk_w, void* out, int tokens, int hidden,
                         int top_k, DType dt, cudaStream_t s) {
   if (tokens == 0) return;
@@ -787,7 +829,7 @@ void launch_moe_combine(const void* y, const int* sorted_pos, const float* topk_
 int launch_moe_grouped_gemm(const MoeGemmArgs& a, cudaStream_t s) {
   if (a.rows_cap <= 0) return 0;
   if (a.k % 8 != 0 || a.ldc % 8 != 0 || a.n % 8 != 0) return -1;
-  if (a.swiglu && a.n % 256 != 0) return -1;
+  if (a.swiglu && (a.n % 256 != 0 || a.gelu)) return -1;
   if ((reinterpret_cast<uintptr_t>(a.x) | reinterpret_cast<uintptr_t>(a.w) | reinterpret_cast<uintptr_t>(a.out)) & 15) return -1;
   const int r = a.swiglu ? 2 : 1;
   GroupedParams p{};
@@ -813,7 +855,8 @@ int launch_moe_grouped_gemm(const MoeGemmArgs& a, cudaStream_t s) {
   switch (a.bn) {
 #define MB200_MOE_CASE(BNV) \
   case BNV:                 \
-    return a.swiglu ? launch_grouped_cfg<BNV, true>(tw, tx, p, grid, s) : launch_grouped_cfg<BNV, false>(tw, tx, p, grid, s);
+    if (a.gelu) return launch_grouped_cfg<BNV, false, true>(tw, tx, p, grid, s); \
+    return a.swiglu ? launch_grouped_cfg<BNV, true, false>(tw, tx, p, grid, s) : launch_grouped_cfg<BNV, false, false>(tw, tx, p, grid, s);
     MB200_MOE_CASE(16)
     MB200_MOE_CASE(32)
     MB200_MOE_CASE(64)
@@ -829,9 +872,14 @@ int launch_moe_grouped_gemm_any(const MoeGemmArgs& a, cudaStream_t s) {
   const int tiles = (a.n + kGaRows - 1) / kGaRows;
   const int64_t items = static_cast<int64_t>(a.max_work) * tiles;
   const int grid = static_cast<int>(std::min<int64_t>(std::max<int64_t>(1, items), 148 * 8));
-  MB200_DISPATCH_FLOAT(a.dt, (launch_pdl(moe_grouped_any_kernel<T>, dim3(grid), dim3(256), 0, s, static_cast<const T*>(a.x), a.ldx,
-                                         static_cast<const T*>(a.w), static_cast<T*>(a.out), a.ldc, a.expert_offsets,
-                                         reinterpret_cast<const int2*>(a.work), a.n_work, a.n, a.k)));
+  MB200_DISPATCH_FLOAT(a.dt, {
+    auto go = [&](auto kernel) {
+      launch_pdl(kernel, dim3(grid), dim3(256), 0, s, static_cast<const T*>(a.x), a.ldx, static_cast<const T*>(a.w), static_cast<T*>(a.out),
+                 a.ldc, a.expert_offsets, reinterpret_cast<const int2*>(a.work), a.n_work, a.n, a.k);
+    };
+    if (a.gelu) go(moe_grouped_any_kernel<T, true>);
+    else go(moe_grouped_any_kernel<T, false>);
+  });
   note_launch();
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }

@@ -9,60 +9,14 @@
 
 #include "common.cuh"
 #include "kernels.h"
+#include "row.cuh"
 
 namespace mb200 {
 namespace {
 
-template <typename T, int V>
-__device__ __forceinline__ void load_vec(const T* p, float (&f)[V]) {
-  struct alignas(sizeof(T) * V) Pack { T e[V]; };
-  const Pack r = *reinterpret_cast<const Pack*>(p);
-#pragma unroll
-  for (int i = 0; i < V; ++i) f[i] = to_f32(r.e[i]);
-}
-template <typename T, int V>
-__device__ __forceinline__ void store_vec(T* p, const float (&f)[V]) {
-  struct alignas(sizeof(T) * V) Pack { T e[V]; };
-  Pack r;
-#pragma unroll
-  for (int i = 0; i < V; ++i) r.e[i] = from_f32<T>(f[i]);
-  *reinterpret_cast<Pack*>(p) = r;
-}
-
-// sums of two values over the CTA (up to 32 warps)
-__device__ __forceinline__ float2 block_sum2(float a, float b) {
-  __shared__ float2 red[33];
-  a = warp_sum(a);
-  b = warp_sum(b);
-  const int w = threadIdx.x >> 5, nw = blockDim.x >> 5;
-  if (lane_id() == 0) red[w] = make_float2(a, b);
-  __syncthreads();
-  if (w == 0) {
-    const float2 t = static_cast<int>(lane_id()) < nw ? red[lane_id()] : make_float2(0.f, 0.f);
-    a = warp_sum(t.x);
-    b = warp_sum(t.y);
-    if (lane_id() == 0) red[32] = make_float2(a, b);
-  }
-  __syncthreads();
-  return red[32];
-}
-
-constexpr int kRowElems = 32;      // elements of a row a thread may hold
 constexpr int kMaxChoices = 32;    // experts a token may use
 // the norm on a sublayer's output holds the stream's elements beside them
 constexpr int row_elems(bool inner) { return inner ? kRowElems / 2 : kRowElems; }
-
-// threads for a row of `vecs` vectors of `v` elements: one each up to 256, then up to `elems` elements each (0: the row is
-// too wide)
-inline int row_threads(int vecs, int v, int elems = kRowElems) {
-  const int most = elems / v;
-  int t = std::min(256, (vecs + 31) / 32 * 32);
-  while (t < 1024 && static_cast<int64_t>(t) * most < vecs) t *= 2;
-  return static_cast<int64_t>(t) * most >= vecs ? t : 0;
-}
-
-// logistic function in full fp32
-__device__ __forceinline__ float sigmoid_f32(float v) { return 1.f / (1.f + expf(-v)); }
 
 // ---------------------------------------------------------------------------------------------
 // The step behind a sublayer, x in fp32; h = the new x in the activations' type.
@@ -174,11 +128,45 @@ __global__ void __launch_bounds__(1024) post_norm_kernel(const PostNormArgs p) {
   }
 }
 
-// logistic function of a factor of a result that is rounded to T: the fast exponential and division for 16-bit results
-template <typename T>
-__device__ __forceinline__ float sigmoid_for(float v) {
-  if constexpr (sizeof(T) == 2) return __fdividef(1.f, 1.f + __expf(-v));
-  return sigmoid_f32(v);
+// out = z * rsqrt(mean(z^2) + eps) * w with z = x * silu(gate): the gate comes before the norm, whose mean is taken over
+// each of `groups` equal parts of the row.  A CTA takes one part.
+template <typename T, int V>
+__global__ void __launch_bounds__(1024) gated_rmsnorm_kernel(const T* __restrict__ x, const T* __restrict__ gate, int64_t gate_ld,
+                                                             const float* __restrict__ w, T* __restrict__ out, int64_t out_ld, int width,
+                                                             int groups, float eps) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int64_t row = blockIdx.x / groups;
+  const int at = static_cast<int>(blockIdx.x - row * groups) * width, vecs = width / V;
+  const T* xr = x + row * groups * width + at;
+  constexpr int kIts = kRowElems / V;
+  float z[kIts][V], ss = 0.f;
+#pragma unroll
+  for (int it = 0; it < kIts; ++it) {
+    const int v = threadIdx.x + it * blockDim.x;
+    if (v < vecs) {
+      float g[V];
+      load_vec<T, V>(xr + v * V, z[it]);
+      load_vec<T, V>(gate + row * gate_ld + at + v * V, g);
+#pragma unroll
+      for (int i = 0; i < V; ++i) {
+        z[it][i] *= g[i] * sigmoid_for<T>(g[i]);
+        ss = fmaf(z[it][i], z[it][i], ss);
+      }
+    }
+  }
+  const float rstd = 1.f / sqrtf(block_sum2(ss, 0.f).x / static_cast<float>(width) + eps);
+#pragma unroll
+  for (int it = 0; it < kIts; ++it) {
+    const int v = threadIdx.x + it * blockDim.x;
+    if (v < vecs) {
+      float wv[V];
+      load_vec<float, V>(w + at + v * V, wv);
+#pragma unroll
+      for (int i = 0; i < V; ++i) z[it][i] *= rstd * wv[i];
+      store_vec<T, V>(out + row * out_ld + at + v * V, z[it]);
+    }
+  }
 }
 
 // out = x * rsqrt(mean(x^2) + eps) * w * sigmoid(gate), the mean over the whole row
@@ -309,10 +297,10 @@ __global__ void __launch_bounds__(512) rownorm_rope_kv_kernel(const RowNormRopeA
 }
 
 // ---------------------------------------------------------------------------------------------
-// Attention prologue with a norm per head: row = [q: heads x dim | k: kv_heads x dim | ..] of a token, values of kv_heads x
+// Attention prologue with a norm per head, or none: row = [q: heads x dim | k: kv_heads x dim | ..] of a token, values of kv_heads x
 // vdim at column v_at (the keys themselves where v_at = heads * dim).  Query and key heads are turned on their first
-// rot_dims features (halves: feature i with i + rot_dims / 2, else neighbours) and divided by their root mean square, which
-// turning does not change; values are cached as they came.  Groups of G lanes take a head each, U features per access.
+// rot_dims features (halves: feature i with i + rot_dims / 2, else neighbours), these times `magnitude`, and where `norm` is
+// set divided by their root mean square, which turning does not change; values are cached as they came.  Groups of G lanes take a head each, U features per access.
 // ---------------------------------------------------------------------------------------------
 template <typename T, int U, bool HALVES>
 __global__ void __launch_bounds__(512) headnorm_rope_kv_kernel(const HeadNormRopeArgs p, int G) {
@@ -332,7 +320,7 @@ __global__ void __launch_bounds__(512) headnorm_rope_kv_kernel(const HeadNormRop
     a -= kTurn * rint(a / kTurn);
     float s, c;
     sincosf(static_cast<float>(a), &s, &c);
-    s_rot[i] = make_float2(c, s);
+    s_rot[i] = make_float2(c * p.magnitude, s * p.magnitude);
   }
   if (slot_ok) {
     for (int u = tid; u < p.kv_heads * p.vdim / U; u += nt) {
@@ -349,16 +337,19 @@ __global__ void __launch_bounds__(512) headnorm_rope_kv_kernel(const HeadNormRop
     const int h = r * groups + tid / G;
     const bool on = h < all, is_q = h < p.heads;
     const T* src = row + (on ? h : 0) * p.dim;       // key heads follow the query heads
-    float ss = 0.f;
-    for (int u = lane; u < units; u += G) {
-      float f[U];
-      load_vec<T, U>(src + u * U, f);
+    float rstd = 1.f;
+    if (p.norm) {
+      float ss = 0.f;
+      for (int u = lane; u < units; u += G) {
+        float f[U];
+        load_vec<T, U>(src + u * U, f);
 #pragma unroll
-      for (int i = 0; i < U; ++i) ss = fmaf(f[i], f[i], ss);
+        for (int i = 0; i < U; ++i) ss = fmaf(f[i], f[i], ss);
+      }
+      for (int o = G / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      rstd = 1.f / sqrtf(ss / static_cast<float>(p.dim) + p.eps);
     }
-    for (int o = G / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
     if (!on) continue;                               // no shuffle follows in this round
-    const float rstd = 1.f / sqrtf(ss / static_cast<float>(p.dim) + p.eps);
     T* dst = nullptr;
     if (is_q) dst = static_cast<T*>(p.q_out) + (t * p.heads + h) * p.q_width;
     else if (slot_ok) dst = static_cast<T*>(p.k_cache) + slot * p.k_tok_stride + (h - p.heads) * p.k_head_stride;
@@ -441,8 +432,6 @@ __global__ void relu_squared_kernel(T* __restrict__ x, int64_t vecs) {
   }
 }
 
-inline bool aligned(const void* p, uintptr_t n) { return (reinterpret_cast<uintptr_t>(p) & (n - 1)) == 0; }
-
 template <typename T, int V, bool INNER>
 int launch_post_norm_v(const PostNormArgs& p, cudaStream_t s) {
   const int threads = row_threads(p.width / V, V, row_elems(INNER));
@@ -462,6 +451,17 @@ int launch_gate_v(const void* x, const void* gate, int64_t gate_ld, const float*
   if (threads == 0) return -1;
   launch_pdl(rmsnorm_sigmoid_gate_kernel<T, V>, dim3(rows), dim3(threads), 0, s, static_cast<const T*>(x), static_cast<const T*>(gate),
              gate_ld, w, static_cast<T*>(out), out_ld, width, eps);
+  note_launch();
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+template <typename T, int V>
+int launch_gated_rmsnorm_v(const void* x, const void* gate, int64_t gate_ld, const float* w, void* out, int64_t out_ld, int rows, int width,
+                           int groups, float eps, cudaStream_t s) {
+  const int threads = row_threads(width / V, V);
+  if (threads == 0) return -1;
+  launch_pdl(gated_rmsnorm_kernel<T, V>, dim3(static_cast<unsigned>(rows) * groups), dim3(threads), 0, s, static_cast<const T*>(x),
+             static_cast<const T*>(gate), gate_ld, w, static_cast<T*>(out), out_ld, width, groups, eps);
   note_launch();
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
@@ -543,6 +543,25 @@ int launch_rmsnorm_sigmoid_gate(const void* x, const void* gate, int64_t gate_ld
   }
   MB200_DISPATCH_FLOAT(dt, rc = vec ? (launch_gate_v<T, 4>(x, gate, gate_ld, w, out, out_ld, rows, width, eps, s))
                                     : (launch_gate_v<T, 1>(x, gate, gate_ld, w, out, out_ld, rows, width, eps, s)));
+  return rc;
+}
+
+int launch_gated_rmsnorm(const void* x, const void* gate, int64_t gate_ld, const float* w, void* out, int64_t out_ld, int rows, int width,
+                         int groups, float eps, DType dt, cudaStream_t s) {
+  if (rows <= 0) return 0;
+  if (groups < 1 || width % groups != 0) return -1;
+  const int part = width / groups;
+  const uintptr_t ptrs = reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(w) |
+                         reinterpret_cast<uintptr_t>(out);
+  const int64_t sizes = part | gate_ld | out_ld;
+  int rc = 0;
+  if (sizes % 8 == 0 && ptrs % 16 == 0 && aligned(w, 32) && dt != kF32) {
+    MB200_DISPATCH_HALF(dt, rc = (launch_gated_rmsnorm_v<T, 8>(x, gate, gate_ld, w, out, out_ld, rows, part, groups, eps, s)));
+    return rc;
+  }
+  const bool vec = sizes % 4 == 0 && aligned(w, 16) && ptrs % (dt == kF32 ? 16 : 8) == 0;
+  MB200_DISPATCH_FLOAT(dt, rc = vec ? (launch_gated_rmsnorm_v<T, 4>(x, gate, gate_ld, w, out, out_ld, rows, part, groups, eps, s))
+                                    : (launch_gated_rmsnorm_v<T, 1>(x, gate, gate_ld, w, out, out_ld, rows, part, groups, eps, s)));
   return rc;
 }
 

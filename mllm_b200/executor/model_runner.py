@@ -483,6 +483,8 @@ class ModelRunner:
         tokens = prof.max_total_num_tokens
         if self.device.type == "cpu":
             tokens = min(tokens, 1 << 16)
+        if self.own_kv_pool and not self.model.kv_cell_bytes(self.kv_cache_dtype):
+            tokens = min(tokens, self._num_req_slots() * self.context_len)     # no layer keeps anything per token
         if self.server_config.max_total_tokens is not None:
             tokens = min(tokens, int(self.server_config.max_total_tokens))
         if tokens <= 0:

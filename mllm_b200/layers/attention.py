@@ -84,9 +84,18 @@ def query_rows(fb):
 def rotation_frequencies(dims: int, base: float, scaling: Optional[dict] = None) -> torch.Tensor:
     """One fp64 frequency per rotated pair, ``base^(-2i / dims)``.  ``scaling`` (factor, low, high, original): frequencies
     whose wave is longer than ``original / low`` are divided by ``factor``, waves shorter than ``original / high`` stay, with
-    a linear blend (in original / wave) between."""
+    a linear blend (in original / wave) between.  ``scaling`` with (factor, original, fast, slow) is YaRN's: pair i is divided by
+    ``factor`` to a degree that rises linearly from 0 at the pair that makes ``fast`` turns over ``original`` positions to 1 at
+    the pair that makes ``slow``."""
     i = torch.arange(dims // 2, dtype=torch.float64)
     f = torch.pow(torch.tensor(base, dtype=torch.float64), -2.0 * i / max(1, dims))
+    if scaling and "fast" in scaling:
+        def pair_of(turns: float) -> float:
+            return dims * math.log(float(scaling["original"]) / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+
+        lo, hi = max(math.floor(pair_of(float(scaling["fast"]))), 0), min(math.ceil(pair_of(float(scaling["slow"]))), dims - 1)
+        ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+        return f / float(scaling["factor"]) * ramp + f * (1.0 - ramp)
     if scaling:
         factor, lo, hi, old = (float(scaling[k]) for k in ("factor", "low", "high", "original"))
         turns = old * f / (2.0 * math.pi)                   # over the original length: original / wavelength
@@ -95,10 +104,15 @@ def rotation_frequencies(dims: int, base: float, scaling: Optional[dict] = None)
     return f
 
 
+def rotation_magnitude(scaling: Optional[dict]) -> float:
+    """Factor of the sines and cosines that comes with YaRN's frequencies."""
+    return 0.1 * math.log(float(scaling["factor"])) + 1.0 if scaling and "fast" in scaling else 1.0
+
+
 class SizedAttention(nn.Module):
     """Causal attention core for layers that give their own sizes: grouped query heads, keys of ``dim`` and values of
-    ``vdim`` features, rotation of part of each head, any score scale, an optional sliding window, an optional sink per
-    head.  It reads the projected rows that ``shards`` names and writes the concatenated heads; projections belong to the
+    ``vdim`` features, rotation of part of each head, any score scale, an optional sliding window or chunks of positions, an
+    optional sink per head, an optional gate per head (``gate_at``: the column of its logits).  It reads the projected rows that ``shards`` names and writes the concatenated heads; projections belong to the
     mixer around it.  Subclasses have the prologue (:meth:`prepare`): norms, rotation, cache write.
 
     16-bit runs use the attention kernels of the other models, with heads zero-padded to 64 / 128 / 256 features in the
@@ -109,12 +123,13 @@ class SizedAttention(nn.Module):
 
     def __init__(self, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, eps: float, kv_index: int, rot_dims: int = 0,
                  rot_base: float = 1e4, rot_scaling: Optional[dict] = None, window: Optional[int] = None,
-                 dtype: torch.dtype = torch.bfloat16) -> None:
+                 dtype: torch.dtype = torch.bfloat16, chunk: Optional[int] = None) -> None:
         super().__init__()
         if heads % kv_heads or rot_dims % 2 or rot_dims > dim:
             raise ValueError(f"attention: {heads} heads over {kv_heads}, {rot_dims} of {dim} features rotated")
         self.heads, self.kv_heads, self.dim, self.vdim = heads, kv_heads, dim, vdim
-        self.scale, self.eps, self.kv_index, self.window = float(scale), float(eps), kv_index, window
+        self.scale, self.eps, self.kv_index, self.window, self.chunk = float(scale), float(eps), kv_index, window, chunk
+        self.gate_at: Optional[int] = None
         self.rot_dims, self.rot_base, self.rot_scaling = rot_dims, float(rot_base), rot_scaling
         self.width = None if dtype == torch.float32 or heads // kv_heads > 128 else next(
             (w for w in (64, 128, 256) if w >= max(dim, vdim) and ops.attention_kernels_cover(w, dtype, dtype)), None)
@@ -157,13 +172,16 @@ class SizedAttention(nn.Module):
         self.prepare(row, fb, q, k_cache, v_cache)
         o = out.unflatten(1, (self.heads, vw))
         if self.width is None or not row.is_cuda:
-            ops.attention_rows(q, k_cache, v_cache, rtt, *query_rows(fb), self.scale, o, window=self.window, sink=self.sink)
+            ops.attention_rows(q, k_cache, v_cache, rtt, *query_rows(fb), self.scale, o, window=self.window, sink=self.sink, chunk=self.chunk)
         elif fb.forward_mode.is_decode():
             ops.attention_decode(q, k_cache, v_cache, rtt, fb.req_pool_indices, fb.seq_lens, self.scale, out=o, max_seq_len=fb.max_seq_len,
-                                 window=self.window, sink=self.sink)
+                                 window=self.window, sink=self.sink, chunk=self.chunk)
         else:
             ops.attention_prefill(q, k_cache, v_cache, rtt, fb.req_pool_indices, fb.seq_lens, fb.extend_prefix_lens, fb.extend_start_loc,
-                                  self.scale, out=o, max_q_len=fb.max_extend_len, window=self.window, sink=self.sink)
+                                  self.scale, out=o, max_q_len=fb.max_extend_len, window=self.window, sink=self.sink,
+                                  chunk=self.chunk)
+        if self.gate_at is not None:
+            ops.gate_heads(o, row[:, self.gate_at: self.gate_at + self.heads], out=o)
 
 
 class RowNormAttention(SizedAttention):
@@ -207,3 +225,24 @@ class HeadNormAttention(SizedAttention):
     def prepare(self, row, fb, q, k_cache, v_cache) -> None:
         ops.headnorm_rope_kv(row, self.inv_freq(row.device), fb.positions, fb.out_cache_loc, q, k_cache, v_cache, self.heads, self.kv_heads,
                              self.dim, self.vdim, self.v_at, self.halves, self.eps)
+
+
+class RotaryAttention(SizedAttention):
+    """Query and key heads turn (feature i with the one half the rotated features on) and keep their length, up to the
+    magnitude that comes with scaled frequencies.  Rows are ``[q | k | v]``, with ``gated`` ``[q | k | v | g]``: each head's output
+    is multiplied by the logistic function of its own logit."""
+
+    def __init__(self, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, kv_index: int, rot_dims: int = 0, rot_base: float = 1e4,
+                 rot_scaling: Optional[dict] = None, window: Optional[int] = None, chunk: Optional[int] = None, gated: bool = False,
+                 dtype: torch.dtype = torch.bfloat16) -> None:
+        super().__init__(heads, kv_heads, dim, vdim, scale, 0.0, kv_index, rot_dims, rot_base, rot_scaling, window, dtype, chunk)
+        self.shards = {"q": heads * dim, "k": kv_heads * dim, "v": kv_heads * vdim}
+        self.v_at = (heads + kv_heads) * dim
+        self.magnitude = rotation_magnitude(rot_scaling)
+        if gated:
+            self.shards["g"] = heads
+            self.gate_at = self.v_at + kv_heads * vdim
+
+    def prepare(self, row, fb, q, k_cache, v_cache) -> None:
+        ops.headnorm_rope_kv(row, self.inv_freq(row.device), fb.positions, fb.out_cache_loc, q, k_cache, v_cache, self.heads, self.kv_heads,
+                             self.dim, self.vdim, self.v_at, True, 0.0, norm=False, magnitude=self.magnitude)

@@ -9,14 +9,14 @@ layers/attention/gdn_backend.py and rms_norm_gated.py; math of HF ``Qwen3_5Gated
 State (recurrent matrix and conv history) lives in a :class:`GDNPool` row per request, so prefill of a
 continuation (chunked prefill) and decode both resume from it.
 
-:class:`FusedGatedDeltaNet` is the same rule for models that give its sizes per layer: one projection for everything
+:class:`ChannelDeltaNet` is the rule with a decay per key channel.  :class:`FusedGatedDeltaNet` is the same rule for models that give its sizes per layer: one projection for everything
 that is taken of the layer input, gates formed inside the rule's kernel, 32-bit products in the recurrence.
 """
 
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import Optional
+from typing import Dict, Optional
 
 import torch
 from torch import nn
@@ -205,3 +205,129 @@ class FusedGatedDeltaNet(nn.Module):
         r = ops.rmsnorm_gated(r.reshape(-1, self.value_dim), y[:, o["g"]: o["g"] + self.value_dim], self.norm.weight, self.eps,
                               round_norm=False)
         return ops.linear(r, self.out_proj.weight)
+
+
+class ChannelDeltaNet(nn.Module):
+    """One delta-net mixer whose state decays by a factor per key channel:
+
+        q, k, v = silu(conv1d(W x));  beta = sigmoid(W_b x);  g = -exp(A_log) * softplus(W_a2 W_a1 x + dt_bias)
+        S <- diag(exp(g)) S;  S <- S + k (beta (v - S^T k))^T;  o = S^T q          (q, k unit vectors, q / sqrt(dim))
+        y = W_o (rmsnorm(o) * w * sigmoid(W_g2 W_g1 x))
+
+    The projections of the input are the row blocks ``[q | k | v | b | a1 | g1]`` of one matrix; the second factors of the decays
+    and of the gates are one product with a matrix of two blocks.  Blocks begin at multiples of 8.  q and k have ``kv_heads``
+    heads and value head ``h`` uses head ``h // (heads / kv_heads)``.  Unit norms, gates and the recurrence are fp32."""
+
+    def __init__(self, hidden_size: int, heads: int, kv_heads: int, dim: int, vdim: int, conv: int, a_rank: int, g_rank: int, eps: float,
+                 gdn_index: int, params_dtype: torch.dtype) -> None:
+        super().__init__()
+        if heads % kv_heads:
+            raise ValueError(f"delta net: {heads} value heads over {kv_heads} key heads")
+        self.heads, self.kv_heads, self.dim, self.vdim, self.conv_kernel = heads, kv_heads, dim, vdim, conv
+        self.eps, self.gdn_index, self.dtype = eps, gdn_index, params_dtype
+        self.key_dim, self.value_dim, self.decay_dim = kv_heads * dim, heads * vdim, heads * dim
+        self.conv_dim = 2 * self.key_dim + self.value_dim
+        self.hidden_size = hidden_size
+
+        def p(*shape, dtype=params_dtype):
+            old = getattr(getattr(self, "in_proj", None), "weight", None)       # later calls stay on the module's device
+            return nn.Parameter(torch.zeros(*shape, dtype=dtype, device=None if old is None else old.device), requires_grad=False)
+
+        self._p = p
+        self._low_rank: Dict[str, torch.Tensor] = {}
+        self.in_proj, self.low_rank, self.conv1d, self.norm, self.out_proj = (nn.Module() for _ in range(5))
+        self.set_ranks(a_rank, g_rank)
+        self.conv1d.weight = p(self.conv_dim, conv)
+        self.A_log = p(heads, dtype=torch.float32)
+        self.dt_bias = p(self.decay_dim, dtype=torch.float32)
+        self.norm.weight = nn.Parameter(torch.ones(vdim, dtype=params_dtype), requires_grad=False)
+        self.out_proj.weight = p(hidden_size, self.value_dim)
+
+    def set_ranks(self, a_rank: int, g_rank: int) -> None:
+        """Inner sizes of the decays' and of the gates' projections.  Rows of the other projections that were loaded stay."""
+        old = getattr(self.in_proj, "weight", None)
+        self.shards = {"q": self.key_dim, "k": self.key_dim, "v": self.value_dim, "b": self.heads, "a1": a_rank, "g1": g_rank}
+        self.offset, rows = {}, 0
+        for name, n in self.shards.items():
+            if name not in ("k", "v"):        # q, k and v are neighbours: one convolution
+                rows = -(-rows // 8) * 8
+            self.offset[name] = rows
+            rows += n
+        self.in_proj.weight = self._p(-(-rows // 8) * 8, self.hidden_size)
+        if old is not None:
+            self.in_proj.weight.data[: self.offset["a1"]].copy_(old.data[: self.offset["a1"]])
+        self.inner = slice(self.offset["a1"], -(-rows // 8) * 8)
+        self.gate_at = -(-self.decay_dim // 8) * 8
+        self.low_rank.weight = self._p(self.gate_at + -(-self.value_dim // 8) * 8, self.inner.stop - self.inner.start)
+
+    @property
+    def state_shape(self):
+        """(value heads, key features, value features, convolution channels, taps) of a request's state."""
+        return self.heads, self.dim, self.vdim, self.conv_dim, self.conv_kernel
+
+    def load_projection(self, name: str, full: torch.Tensor) -> None:
+        self._fit(self.in_proj.weight.data[self.offset[name]: self.offset[name] + self.shards[name]], full)
+
+    def load_low_rank(self, name: str, full: torch.Tensor) -> None:
+        """``name``: a1, a2 (decays), g1 or g2 (gates).  Their shapes alone give the inner sizes, so the four are placed together."""
+        parts = self._low_rank
+        parts[name] = full
+        if len(parts) < 4:
+            return
+        self.set_ranks(parts["a1"].shape[0], parts["g1"].shape[0])
+        for first, second, row, rows in (("a1", "a2", 0, self.decay_dim), ("g1", "g2", self.gate_at, self.value_dim)):
+            self.load_projection(first, parts[first])
+            col = self.offset[first] - self.inner.start
+            self._fit(self.low_rank.weight.data[row: row + rows, col: col + self.shards[first]], parts[second])
+        parts.clear()
+
+    @staticmethod
+    def _fit(dst: torch.Tensor, full: torch.Tensor) -> None:
+        if dst.shape != full.shape:
+            raise ValueError(f"a tensor of shape {tuple(full.shape)} does not fit {tuple(dst.shape)}")
+        dst.copy_(full)
+
+    def load_conv(self, name: str, full: torch.Tensor) -> None:
+        self._fit(self.conv1d.weight.data[self.offset[name]: self.offset[name] + self.shards[name]], full)
+
+    def forward(self, x: torch.Tensor, fb) -> torch.Tensor:
+        recurrent, conv = fb.extra["gdn_pool"].layer(self.gdn_index)
+        m = gdn_batch(fb)
+        o, C = self.offset, self.conv_dim
+        y = ops.linear(x, self.in_proj.weight)
+        second = ops.linear(y[:, self.inner], self.low_rank.weight)
+        qkv = ops.causal_conv1d_silu(y[:, :C], self.conv1d.weight, conv, m.slots, m.lens, m.has_state, m.q_start, m.max_len)
+        q = qkv[:, : o["k"]].unflatten(1, (self.kv_heads, self.dim))
+        k = qkv[:, o["k"]: o["v"]].unflatten(1, (self.kv_heads, self.dim))
+        v = qkv[:, o["v"]:].unflatten(1, (self.heads, self.vdim))
+        r = ops.channel_delta_rule(q, k, v, y[:, o["b"]: o["b"] + self.heads], second[:, : self.decay_dim], self.A_log, self.dt_bias,
+                                   recurrent, m.slots, m.lens, m.has_state, m.q_start, m.max_len)
+        r = ops.rmsnorm_gated(r.reshape(-1, self.value_dim), second[:, self.gate_at: self.gate_at + self.value_dim], self.norm.weight,
+                              self.eps, round_norm=False, sigmoid=True)
+        return ops.linear(r, self.out_proj.weight)
+
+
+class CausalConvolution(nn.Module):
+    """``x + conv(x)``, a causal convolution over time on each channel without an activation.  The last taps - 1 inputs of a
+    request live in its row of the state pool.  A decode step may leave the work to the kernel that writes ``x``
+    (:meth:`step`)."""
+
+    def __init__(self, channels: int, taps: int, gdn_index: int, params_dtype: torch.dtype) -> None:
+        super().__init__()
+        self.channels, self.taps, self.gdn_index = channels, taps, gdn_index
+        self.weight = nn.Parameter(torch.zeros(channels, taps, dtype=params_dtype), requires_grad=False)
+
+    @property
+    def state_shape(self):
+        return 0, 0, 0, self.channels, self.taps
+
+    def step(self, fb) -> Optional["ops.ConvStep"]:
+        """What the kernel in front needs to apply the convolution itself; None where rows have neighbours in the batch."""
+        if not fb.forward_mode.is_decode():
+            return None
+        return ops.ConvStep(self.weight, fb.extra["gdn_pool"].layer(self.gdn_index)[1], gdn_batch(fb).slots)
+
+    def forward(self, x: torch.Tensor, fb) -> torch.Tensor:
+        m = gdn_batch(fb)
+        return ops.causal_conv1d_silu(x, self.weight, fb.extra["gdn_pool"].layer(self.gdn_index)[1], m.slots, m.lens, m.has_state, m.q_start,
+                                      m.max_len, add_input=True)

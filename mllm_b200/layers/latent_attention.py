@@ -1,8 +1,8 @@
 """Latent attention: the cache holds one row ``c`` of ``kv_rank`` features per token, shared by all heads; head ``h``'s
-key and value of a token are ``W_uk[h] c`` and ``W_uv[h] c``.  Queries go through a latent of their own.  Options: a
-rotated key part of ``rot_dim`` features, shared by all heads, which follows the latent in the cache row and meets a
-rotated part of each query head (without it there are no positions); a sink per head, a logit that joins the softmax
-denominator only; a gate per head on the output.  A layer may read the latents of an earlier layer instead of writing its
+key and value of a token are ``W_uk[h] c`` and ``W_uv[h] c``.  Queries go through a latent of their own or are projected
+directly.  Options: a rotated key part of ``rot_dim`` features, shared by all heads, which follows the latent in the cache row and meets a
+rotated part of each query head (without it there are no positions); a sliding window; a sink per head, a logit that joins
+the softmax denominator only; a gate on the output, one per head or one per feature.  A layer may read the latents of an earlier layer instead of writing its
 own.
 
 Two evaluations of the same sum (``csrc/latent.cu``):
@@ -19,7 +19,7 @@ A batch may need both: :func:`latent_plan` sorts the requests once per forward p
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import List, Optional
+from typing import List, Optional, Union
 
 import torch
 from torch import nn
@@ -40,6 +40,7 @@ class ExpandGroup:
     prefix_lens: torch.Tensor  # [b]
     q_start: torch.Tensor      # [b] first query row
     ctx_start: torch.Tensor    # [b] first row of the request's expanded context
+    first: Optional[torch.Tensor]   # [b] token that context begins with (None: 0); the lengths above count from it
     rows: torch.Tensor         # [b, longest context] the identity table: row of every context token
     batch: torch.Tensor        # [b] 0 .. b - 1, the rows of that table
     total: int
@@ -56,9 +57,10 @@ class LatentPlan:
     max_ctx: int                      # longest context of the absorbed part
 
 
-def latent_plan(fb, expand: bool, min_tokens: Optional[int] = None) -> LatentPlan:
-    """Which requests of the batch run expanded and which absorbed; cached in ``fb.extra``."""
-    key = ("latent_plan", expand)
+def latent_plan(fb, expand: bool, min_tokens: Optional[int] = None, window: Optional[int] = None) -> LatentPlan:
+    """Which requests of the batch run expanded and which absorbed; cached in ``fb.extra``.  With a ``window`` a request is
+    expanded from the first token that its new tokens see."""
+    key = ("latent_plan", expand, window)
     got = fb.extra.get(key)
     if got is not None:
         return got
@@ -69,6 +71,7 @@ def latent_plan(fb, expand: bool, min_tokens: Optional[int] = None) -> LatentPla
     least = EXPAND_MIN_TOKENS if min_tokens is None else min_tokens
     dev = fb.input_ids.device
     ext, pre = list(fb.extend_seq_lens_cpu), list(fb.extend_prefix_lens_cpu)
+    skip = [max(0, p - window + 1) if window else 0 for p in pre]      # tokens in front of the expanded context
     starts, total = [], 0
     for n in ext:
         starts.append(total)
@@ -86,7 +89,7 @@ def latent_plan(fb, expand: bool, min_tokens: Optional[int] = None) -> LatentPla
         if not run:
             return
         sel = torch.tensor(run, dtype=torch.int64).to(dev, non_blocking=True)
-        ctx = [ext[i] + pre[i] for i in run]
+        ctx = [ext[i] + pre[i] - skip[i] for i in run]
         at, acc = [], 0
         for n in ctx:
             at.append(acc)
@@ -95,18 +98,20 @@ def latent_plan(fb, expand: bool, min_tokens: Optional[int] = None) -> LatentPla
         table = cs.unsqueeze(1) + torch.arange(max(ctx), dtype=torch.int32, device=dev).unsqueeze(0)
         groups.append(ExpandGroup(
             req=fb.req_pool_indices.index_select(0, sel).to(torch.int32), seq_lens=dev_i32(ctx),
-            prefix_lens=dev_i32([pre[i] for i in run]), q_start=dev_i32([starts[i] for i in run]), ctx_start=cs,
+            prefix_lens=dev_i32([pre[i] - skip[i] for i in run]), q_start=dev_i32([starts[i] for i in run]), ctx_start=cs,
+            first=dev_i32([skip[i] for i in run]) if window else None,
             rows=table.clamp_(max=acc - 1), batch=torch.arange(len(run), dtype=torch.int32, device=dev), total=acc,
             max_ctx=max(ctx), max_q=max(ext[i] for i in run)))
         run.clear()
 
     size = 0
     for i in far:
-        if run and size + ext[i] + pre[i] > EXPAND_MAX_CONTEXT:
+        ctx = ext[i] + pre[i] - skip[i]
+        if run and size + ctx > EXPAND_MAX_CONTEXT:
             close()
             size = 0
         run.append(i)
-        size += ext[i] + pre[i]
+        size += ctx
     close()
     rows = row_req = row_pos = None
     max_ctx = max((ext[i] + pre[i] for i in near), default=0)
@@ -136,15 +141,20 @@ def _pad_heads(w: torch.Tensor, heads: int, width: int) -> torch.Tensor:
 
 
 class LatentAttention(nn.Module):
-    def __init__(self, hidden_size: int, heads: int, dim: int, vdim: int, q_rank: int, kv_rank: int, scale: float, eps: float,
+    def __init__(self, hidden_size: int, heads: int, dim: int, vdim: int, q_rank: Optional[int], kv_rank: int, scale: float, eps: float,
                  latent_index: int, writes_latent: bool, params_dtype: torch.dtype, rot_dim: int = 0, rot_base: float = 1e4,
-                 rot_scaling: Optional[dict] = None, sinks: bool = True, gated: bool = False) -> None:
+                 rot_scaling: Optional[dict] = None, sinks: bool = True, gated: Union[bool, str] = False, halves: bool = False,
+                 window: Optional[int] = None) -> None:
         """``latent_index``: the buffer of the latent pool this layer reads; ``writes_latent``: whether the layer has a
-        down projection of its own and fills it."""
+        down projection of its own and fills it; ``q_rank`` None: queries are projected from the layer's input; ``gated``: True
+        for a gate per head, "features" for one per feature; ``halves``: feature i of the rotated part turns with feature i +
+        rot_dim / 2 instead of its neighbour; ``window``: a token sees the last ``window`` ones, itself among them."""
         super().__init__()
+        gates = heads * vdim if gated == "features" else heads if gated else 0
         self.heads, self.dim, self.vdim, self.q_rank, self.kv_rank = heads, dim, vdim, q_rank, kv_rank
         self.scale, self.eps, self.latent_index, self.writes_latent = float(scale), eps, latent_index, writes_latent
         self.rot_dim, self.rot_base, self.rot_scaling, self.gated = rot_dim, float(rot_base), rot_scaling, gated
+        self.halves, self.window = halves, window
         self._inv_freq: Optional[torch.Tensor] = None
 
         def p(*shape, dtype=params_dtype):
@@ -155,18 +165,24 @@ class LatentAttention(nn.Module):
             m.weight = p(o, i)
             return m
 
-        # rows of the down projection: query latent, cache latent with the shared key part, gates; zero rows to a multiple of 8
+        # rows of the down projection: query latent, cache latent with the shared key part, gates; zero rows to a multiple of 8.
+        # Queries without a latent come last: decode steps form them with the rest, prompts that run expanded on their own
         self.down_at, rows = {}, 0
-        for name, n in (("q", q_rank), ("kv", kv_rank + rot_dim if writes_latent else 0), ("g", heads if gated else 0)):
+        for name, n in (("q", q_rank or 0), ("kv", kv_rank + rot_dim if writes_latent else 0), ("g", gates)):
             self.down_at[name] = slice(rows, rows + n)
             rows += n
-        self.down_proj = lin(-(-rows // 8) * 8, hidden_size)
+        rows = -(-rows // 8) * 8
+        self.down_rows = rows
+        if q_rank is None:
+            self.down_at["q"] = slice(rows, rows + heads * (dim + rot_dim))
+            rows = -(-self.down_at["q"].stop // 8) * 8
+        self.down_proj = lin(rows, hidden_size)
         self.q_latent_norm = nn.Module()
-        self.q_latent_norm.weight = nn.Parameter(torch.ones(q_rank, dtype=torch.float32), requires_grad=False)
+        self.q_latent_norm.weight = None if q_rank is None else nn.Parameter(torch.ones(q_rank, dtype=torch.float32), requires_grad=False)
         if writes_latent:
             self.kv_latent_norm = nn.Module()
             self.kv_latent_norm.weight = nn.Parameter(torch.ones(kv_rank, dtype=torch.float32), requires_grad=False)
-        self.q_up = lin(heads * (dim + rot_dim), q_rank)        # per head [dim | rot_dim]
+        self.q_up = None if q_rank is None else lin(heads * (dim + rot_dim), q_rank)        # per head [dim | rot_dim]
         self.k_up = lin(heads * dim, kv_rank)
         self.v_up = lin(heads * vdim, kv_rank)
         self.sink = p(heads, dtype=torch.float32) if sinks else None
@@ -180,7 +196,7 @@ class LatentAttention(nn.Module):
         return self.kv_rank + self.rot_dim
 
     def load_down(self, name: str, full: torch.Tensor) -> None:
-        """``name``: q (query latent), kv (cache latent and shared key part) or g (gates)."""
+        """``name``: q (query latent, or the queries), kv (cache latent and shared key part) or g (gates)."""
         rows = self.down_proj.weight.data[self.down_at[name]]
         if rows.shape != full.shape:
             raise ValueError(f"a tensor of shape {tuple(full.shape)} does not fit {tuple(rows.shape)}")
@@ -197,14 +213,18 @@ class LatentAttention(nn.Module):
         k_up = self.k_up.weight.data.view(H, self.dim, self.kv_rank)
         self._uk_t = keep(k_up.transpose(1, 2))                                                       # [H, rank, dim]
         self._uv = self.v_up.weight.data.view(H, self.vdim, self.kv_rank)                             # [H, vdim, rank]
-        if self.pad is not None and self.expandable(self.q_up.weight):
+        q_up = self.down_proj.weight[self.down_at["q"]] if self.q_up is None else self.q_up.weight
+        # the projections of a prompt whose queries are formed apart
+        self._down_rest = self.down_proj.weight if self.q_up is not None else nn.Parameter(self.down_proj.weight.data[: self.down_rows],
+                                                                                            requires_grad=False)
+        if self.pad is not None and self.expandable(q_up):
             v_up = self._uv
             if R:       # products with whole cache rows: the shared key part is copied into K and left out of V
                 wide = k_up.new_zeros(H, self.dim + R, self.cache_width)
                 wide[:, : self.dim, : self.kv_rank] = k_up
                 wide[:, self.dim:, self.kv_rank:] = torch.eye(R, dtype=wide.dtype, device=wide.device)
                 k_up, v_up = wide, torch.cat([v_up, v_up.new_zeros(H, self.vdim, R)], -1)
-            self._uq_pad = keep(_pad_heads(self.q_up.weight.data, H, self.pad))
+            self._uq_pad = keep(_pad_heads(q_up.data, H, self.pad))
             self._uk_pad = keep(_pad_heads(k_up.reshape(-1, self.cache_width), H, self.pad))
             self._uv_pad = keep(_pad_heads(v_up.reshape(-1, self.cache_width), H, self.pad))
 
@@ -222,22 +242,31 @@ class LatentAttention(nn.Module):
         T, H = x.shape[0], self.heads
         cache = fb.token_to_kv_pool.get_latent_buffer(self.latent_index)
         rtt = fb.req_to_token_pool.req_to_token
-        plan = latent_plan(fb, self.expandable(x))
-        y = ops.linear(x, self.down_proj.weight)
+        plan = latent_plan(fb, self.expandable(x), window=self.window)
+
+        def near(t):
+            return t if plan.rows is None or t is None else t.index_select(0, plan.rows)
+
+        # without a query latent the expanded form takes its queries from the input, in heads of its own width
+        apart = self.q_up is None and bool(plan.groups)
+        y = ops.linear(x, self._down_rest if apart else self.down_proj.weight)
         cq, turns = ops.latent_prologue(y, self.q_latent_norm.weight, self.kv_latent_norm.weight if self.writes_latent else None,
                                         self.eps, fb.out_cache_loc, cache if self.writes_latent else None, fb.positions,
-                                        self.inv_freq(x.device))
+                                        self.inv_freq(x.device), self.halves)
         gate = y[:, self.down_at["g"]] if self.gated else None
         o = None
         if plan.groups:
-            o = self._expanded(cq, cache, rtt, plan, turns, gate)
+            o = self._expanded(x if cq is None else cq, cache, rtt, plan, turns, gate)
         if plan.row_req is not None:
-            def near(t):
-                return t if plan.rows is None or t is None else t.index_select(0, plan.rows)
-
-            q = ops.linear(near(cq), self.q_up.weight).view(-1, H, self.dim + self.rot_dim)
-            q = ops.head_linear(q, self._uk_t, turns=near(turns))
-            u = ops.latent_attention(q, cache, rtt, plan.row_req, plan.row_pos, self.scale, self.sink, plan.max_ctx, self.kv_rank)
+            if self.q_up is not None:
+                q = ops.linear(near(cq), self.q_up.weight)
+            elif apart:
+                q = ops.linear(near(x), self.down_proj.weight[self.down_at["q"]])
+            else:
+                q = y[:, self.down_at["q"]]
+            q = q.unflatten(1, (H, self.dim + self.rot_dim))
+            q = ops.head_linear(q, self._uk_t, turns=near(turns), halves=self.halves)
+            u = ops.latent_attention(q, cache, rtt, plan.row_req, plan.row_pos, self.scale, self.sink, plan.max_ctx, self.kv_rank, self.window)
             u = ops.head_linear(u, self._uv, gate=near(gate))
             if plan.rows is None:
                 o = u
@@ -250,13 +279,13 @@ class LatentAttention(nn.Module):
         H, W = self.heads, self.pad
         q = ops.linear(cq, self._uq_pad).view(-1, H, W)
         if turns is not None:
-            ops.turn_heads(q[..., self.dim: self.dim + self.rot_dim], turns)
+            ops.turn_heads(q[..., self.dim: self.dim + self.rot_dim], turns, halves=self.halves)
         out = torch.empty_like(q)
         for g in plan.groups:
-            c = ops.latent_gather(cache, rtt, g.req, g.seq_lens, g.ctx_start, g.total, g.max_ctx)
+            c = ops.latent_gather(cache, rtt, g.req, g.seq_lens, g.ctx_start, g.total, g.max_ctx, g.first)
             k = ops.linear(c, self._uk_pad).view(-1, H, W)
             v = ops.linear(c, self._uv_pad).view(-1, H, W)
             ops.attention_prefill(q, k, v, g.rows, g.batch, g.seq_lens, g.prefix_lens, g.q_start, self.scale, out=out,
-                                  max_q_len=g.max_q, sink=self.sink)
+                                  max_q_len=g.max_q, sink=self.sink, window=self.window)
         out = out[..., : self.vdim]
         return out.contiguous() if gate is None else ops.gate_heads(out, gate)

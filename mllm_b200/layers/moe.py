@@ -55,8 +55,12 @@ class MoEGate(nn.Module):
 class SparseMoeBlock(nn.Module):
     def __init__(self, hidden_size: int, moe_intermediate_size: int, num_experts: int, top_k: int,
                  norm_topk_prob: bool = True, params_dtype=None, prefix: str = "", identity_experts: int = 0,
-                 choice_bias: bool = False, renorm_eps: float = 0.0, fp32_logits: bool = False, **router) -> None:
+                 choice_bias: bool = False, renorm_eps: float = 0.0, fp32_logits: bool = False, gated: bool = True,
+                 weigh_input: bool = False, **router) -> None:
+        """``gated`` False: an expert is ``W_down gelu(W_up x)`` (the exact GELU) and ``w13`` holds the up projections alone;
+        ``weigh_input``: an expert's weight multiplies what it reads instead of its result.  Both need :meth:`expert_rows`."""
         super().__init__()
+        self.gated, self.weigh_input = gated, weigh_input
         ep = pstate.get_ep_group()
         self.ep_size, self.ep_rank = ep.world_size, ep.rank_in_group
         self.tp_size = pstate.get_tensor_model_parallel_world_size()
@@ -72,9 +76,9 @@ class SparseMoeBlock(nn.Module):
         self.gate = MoEGate(hidden_size, num_experts, top_k, norm_topk_prob, dt, identity_experts, choice_bias, renorm_eps, fp32_logits,
                             **router)
         self.identity_from = num_experts if identity_experts else 0     # router outputs from here on have no weights
-        if identity_experts and (self.ep_size > 1 or self.inter_shard > 1):
-            raise NotImplementedError("identity experts are not sharded over ranks")
-        self.w13 = nn.Parameter(torch.empty(self.local_experts, 2 * self.inter, hidden_size, dtype=dt), requires_grad=False)
+        if (identity_experts or not gated or weigh_input) and (self.ep_size > 1 or self.inter_shard > 1):
+            raise NotImplementedError("identity experts, experts without a gate and weighted inputs are not sharded over ranks")
+        self.w13 = nn.Parameter(torch.empty(self.local_experts, (2 if gated else 1) * self.inter, hidden_size, dtype=dt), requires_grad=False)
         self.w2 = nn.Parameter(torch.empty(self.local_experts, hidden_size, self.inter, dtype=dt), requires_grad=False)
         self.w13.weight_loader = self._load_w13
         self.w2.weight_loader = self._load_w2
@@ -96,7 +100,7 @@ class SparseMoeBlock(nn.Module):
             return
         e = expert - self.expert_offset
         part = self._shard(loaded, 0)
-        off = 0 if which == "gate" else self.inter
+        off = 0 if which == "gate" or not self.gated else self.inter
         param.data[e, off : off + self.inter].copy_(part)
 
     def _load_w2(self, param, loaded: torch.Tensor, expert: int, which: str = "down") -> None:
@@ -106,7 +110,7 @@ class SparseMoeBlock(nn.Module):
 
     def process_weights_after_loading(self) -> None:
         """Interleave gate/up rows in blocks of 128 so the first GEMM can fuse the SwiGLU."""
-        if self.swiglu_block == 0 and (2 * self.inter) % (2 * ops.SWIGLU_BLOCK) == 0 and self.w13.is_cuda \
+        if self.gated and self.swiglu_block == 0 and (2 * self.inter) % (2 * ops.SWIGLU_BLOCK) == 0 and self.w13.is_cuda \
                 and self.w13.dtype != torch.float32 and self.w13.shape[2] % 8 == 0:
             w = self.w13.data
             for e in range(w.shape[0]):
@@ -123,8 +127,9 @@ class SparseMoeBlock(nn.Module):
         shard = self._exchange(x)
         if shard is not None:
             return shard
-        if self.identity_from or self.gate.extra:
-            raise NotImplementedError("identity experts and a gated shared expert are summed by the norm behind the block: use expert_rows")
+        if self.identity_from or self.gate.extra or not self.gated or self.weigh_input:
+            raise NotImplementedError("identity experts, a gated shared expert, experts without a gate and weighted inputs are summed "
+                                      "by the step behind the block: use expert_rows")
         topk_w, topk_ids = self.gate(x)
         return ops.moe_experts(x, self.w13, self.w2, topk_w, topk_ids, self.expert_offset, self.swiglu_block,
                                self.num_experts)
@@ -133,7 +138,7 @@ class SparseMoeBlock(nn.Module):
         """The routed experts' outputs before they are summed, for a norm that does it (one GPU per replica)."""
         topk_w, topk_ids, *logit = self.gate(x)
         return ops.moe_expert_rows(x, self.w13, self.w2, topk_w, topk_ids, self.swiglu_block, self.identity_from,
-                                   logit[0][:, 0] if logit else None)
+                                   logit[0][:, 0] if logit else None, self.gated, self.weigh_input)
 
     def can_exchange(self, rows: int) -> bool:
         """Whether a batch of ``rows`` tokens can go through the expert-parallel exchange on this block."""

@@ -1,8 +1,9 @@
 """Token mixers side by side on the same input, ``sum_i scale_i * W_o,i branch_i(W_in,i x)``, as one projection in, the
 branches, and one projection out: the branches write neighbouring columns of one matrix, so their weighted sum is the
-inner dimension of the output product.  A single branch is the ordinary mixer.
+inner dimension of the output product.  A single branch is the ordinary mixer.  Where each branch's result has a norm of its
+own (:class:`NormedParallelMixer`), the output projections stay apart and the step behind the layer norms and averages them.
 
-A branch (:class:`.RowNormAttention`, :class:`.LightningAttention`) lists the projections it reads (``shards``: name ->
+A branch (:class:`.RowNormAttention`, :class:`.LightningAttention`, :class:`.StateSpace`) lists the projections it reads (``shards``: name ->
 rows, in order; ``biased``: which have a bias), the columns it writes (``out_width``) and how an output projection's
 columns are laid out for it (``expand_columns``); ``forward(row, fb, out)`` does the work."""
 
@@ -38,6 +39,7 @@ class ParallelMixer(nn.Module):
             if any(b.biased for b in branches) else None
         self.out_proj.weight = nn.Parameter(torch.zeros(hidden_size, cols, dtype=params_dtype), requires_grad=False)
         self.gaps = cols != sum(b.out_width for b in branches)
+        self.out_width = cols
         self.result_scale = 1.0        # set by fold_scales: what the sum of the branches is still to be multiplied with
 
     # ------------------------------------------------------------------ loading
@@ -73,10 +75,40 @@ class ParallelMixer(nn.Module):
         self.result_scale = base
 
     # ------------------------------------------------------------------ forward
-    def forward(self, x: torch.Tensor, fb) -> torch.Tensor:
+    def run_branches(self, x: torch.Tensor, fb) -> torch.Tensor:
+        """The branches' outputs side by side."""
         rows = ops.linear(x, self.in_proj.weight, self.in_proj.bias)
-        shape = (x.shape[0], self.out_proj.weight.shape[1])
+        shape = (x.shape[0], self.out_width)
         mixed = (torch.zeros if self.gaps else torch.empty)(shape, dtype=x.dtype, device=x.device)
         for b, r, c in zip(self.branches, self.row_at, self.out_at):
             b(rows[:, r:], fb, mixed[:, c: c + b.out_width])
-        return ops.linear(mixed, self.out_proj.weight)
+        return mixed
+
+    def forward(self, x: torch.Tensor, fb) -> torch.Tensor:
+        return ops.linear(self.run_branches(x, fb), self.out_proj.weight)
+
+
+class NormedParallelMixer(ParallelMixer):
+    """Two branches whose results ``W_o,i branch_i`` are RMS-normed one by one: the forward pass returns them with their norm
+    weights, for a step that norms and adds them (:func:`..ops.depth_step`)."""
+
+    def __init__(self, hidden_size: int, branches: Sequence[nn.Module], params_dtype: torch.dtype) -> None:
+        super().__init__(hidden_size, branches, [1.0] * len(branches), params_dtype)
+        del self.out_proj
+        self.out_projs, self.out_norms = nn.ModuleList(), nn.ParameterList()
+        for b in branches:
+            m = nn.Module()
+            m.weight = nn.Parameter(torch.zeros(hidden_size, b.out_width, dtype=params_dtype), requires_grad=False)
+            self.out_projs.append(m)
+            self.out_norms.append(nn.Parameter(torch.ones(hidden_size, dtype=torch.float32), requires_grad=False))
+
+    def load_out(self, branch: int, w: torch.Tensor) -> None:
+        dst, src = self.out_projs[branch].weight.data, self.branches[branch].expand_columns(w)
+        if dst.shape != src.shape:
+            raise ValueError(f"a tensor of shape {tuple(w.shape)} does not fit the branch's {tuple(dst.shape)}")
+        dst.copy_(src)
+
+    def forward(self, x: torch.Tensor, fb):
+        mixed = self.run_branches(x, fb)
+        return (*(ops.linear(mixed[:, c: c + b.out_width], m.weight) for b, c, m in zip(self.branches, self.out_at, self.out_projs)),
+                *self.out_norms)

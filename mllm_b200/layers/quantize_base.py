@@ -45,9 +45,10 @@ class LinearMethodBase(QuantizeMethodBase):
         raise NotImplementedError
 
     def apply_swiglu(self, layer: nn.Module, x: torch.Tensor) -> torch.Tensor:
-        """Fused gate/up projection + gated activation (``layer.gate_activation``, SiLU unless set); default =
-        apply then activation."""
-        return ops.act_and_mul(self.apply(layer, x), getattr(layer, "gate_activation", "silu"))
+        """Fused gate/up projection + gated activation (``layer.gate_activation``, SiLU unless set, with the bound
+        ``layer.gate_limit`` where it has one); default = apply then activation."""
+        return ops.act_and_mul(self.apply(layer, x, getattr(layer, "bias", None)), getattr(layer, "gate_activation", "silu"),
+                               getattr(layer, "gate_limit", 0.0))
 
 
 class UnquantizedLinearMethod(LinearMethodBase):
@@ -68,13 +69,15 @@ class UnquantizedLinearMethod(LinearMethodBase):
             w = layer.weight.data
             if w.shape[0] % (2 * ops.SWIGLU_BLOCK) == 0:
                 layer.weight.data = ops.ref.interleave_gate_up(w, ops.SWIGLU_BLOCK).contiguous()
+                if getattr(layer, "bias", None) is not None:
+                    layer.bias.data = ops.ref.interleave_gate_up(layer.bias.data.unsqueeze(-1), ops.SWIGLU_BLOCK).reshape(-1).contiguous()
                 layer._gate_up_interleaved = True
 
     def apply(self, layer, x, bias=None, residual=None):
         return ops.linear(x, layer.weight, bias, residual)
 
     def apply_swiglu(self, layer, x):
-        act = getattr(layer, "gate_activation", "silu")
+        act, limit, bias = getattr(layer, "gate_activation", "silu"), getattr(layer, "gate_limit", 0.0), getattr(layer, "bias", None)
         if getattr(layer, "_gate_up_interleaved", False):
-            return ops.linear_swiglu(x, layer.weight, ops.SWIGLU_BLOCK, act)
-        return ops.act_and_mul(ops.linear(x, layer.weight), act)
+            return ops.linear_swiglu(x, layer.weight, ops.SWIGLU_BLOCK, act, bias, limit)
+        return ops.act_and_mul(ops.linear(x, layer.weight, bias), act, limit)

@@ -28,6 +28,7 @@ _REGISTRY: Dict[str, Tuple[str, str]] = {
     "PebulixForCausalLM": ("mllm_b200.models.pebulix", "PebulixForCausalLM"),
     "KesovikForCausalLM": ("mllm_b200.models.kesovik", "KesovikForCausalLM"),
     "LufizenForCausalLM": ("mllm_b200.models.lufizen", "LufizenForCausalLM"),
+    "NikedraForCausalLM": ("mllm_b200.models.nikedra", "NikedraForCausalLM"),
 }
 
 # designs whose config.json names itself in "architecture" and has a layout of its own: a function that checks the
@@ -36,6 +37,7 @@ _CONFIG_ADAPTERS: Dict[str, Tuple[str, str]] = {
     "Pebulix": ("mllm_b200.models.pebulix", "adapt_config"),
     "Kesovik": ("mllm_b200.models.kesovik", "adapt_config"),
     "Lufizen": ("mllm_b200.models.lufizen", "adapt_config"),
+    "Nikedra": ("mllm_b200.models.nikedra", "adapt_config"),
 }
 
 

@@ -28,11 +28,13 @@ def put(p: torch.Tensor) -> Callable[[torch.Tensor], None]:
 
 
 def mixture_places(at: str, block, shared: Optional[torch.nn.Module]) -> Places:
-    """Places of a :class:`..layers.moe.SparseMoeBlock` with a corrected router and of a shared gated MLP beside it."""
+    """Places of a :class:`..layers.moe.SparseMoeBlock` and of a shared gated MLP beside it."""
     gate = block.gate
-    out: Places = {at + "router": put(gate.weight[: gate.outputs]), at + "correction": put(gate.correction)}
+    out: Places = {at + "router": put(gate.weight[: gate.outputs])}
+    if gate.correction is not None:
+        out[at + "correction"] = put(gate.correction)
     for e in range(block.num_experts):
-        for n in ("gate", "up"):
+        for n in ("gate", "up") if block.gated else ("up",):
             out[f"{at}e{e}.{n}"] = lambda t, e=e, n=n: block.w13.weight_loader(block.w13, t, e, n)
         out[f"{at}e{e}.down"] = lambda t, e=e: block.w2.weight_loader(block.w2, t, e)
     if shared is not None:
@@ -45,7 +47,8 @@ def mixture_places(at: str, block, shared: Optional[torch.nn.Module]) -> Places:
     return out
 
 
-def load_places(places: Places, weights: Iterable[Tuple[str, torch.Tensor]]) -> set:
+def load_places(places: Places, weights: Iterable[Tuple[str, torch.Tensor]], optional: Iterable[str] = ()) -> set:
+    """``optional``: tensors that a checkpoint may lack."""
     loaded = set()
     for name, t in weights:
         place = places.get(name)
@@ -53,7 +56,7 @@ def load_places(places: Places, weights: Iterable[Tuple[str, torch.Tensor]]) -> 
             raise ValueError(f"unexpected tensor {name!r} in the checkpoint")
         place(t.materialize() if hasattr(t, "materialize") else t)
         loaded.add(name)
-    missing = sorted(set(places) - loaded)
+    missing = sorted(set(places) - loaded - set(optional))
     if missing:
         raise ValueError(f"the checkpoint lacks {len(missing)} tensors: {', '.join(missing[:8])}")
     return loaded

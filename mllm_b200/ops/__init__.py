@@ -144,8 +144,15 @@ def gelu_tanh_and_mul(x: torch.Tensor) -> torch.Tensor:
     return out.view(*x.shape[:-1], -1)
 
 
-def act_and_mul(x: torch.Tensor, act: str) -> torch.Tensor:
-    """``act(gate) * up`` over the two halves of the last dimension; ``act``: ``silu`` or ``gelu_tanh``."""
+def act_and_mul(x: torch.Tensor, act: str, limit: float = 0.0) -> torch.Tensor:
+    """``x = [gate | up]`` -> the gated unit ``act`` (``silu``, ``gelu_tanh``, ``clamped``: see :func:`linear_swiglu`)."""
+    if act == "clamped":
+        if not use_kernels(x):
+            return ref.clamped_gate(*x.chunk(2, dim=-1), limit)
+        x2 = _2d(x).contiguous()
+        out = torch.empty((x2.shape[0], x2.shape[1] // 2), dtype=x.dtype, device=x.device)
+        ext().act_and_mul(x2, out, 2, float(limit))
+        return out.view(*x.shape[:-1], out.shape[1])
     return gelu_tanh_and_mul(x) if act == "gelu_tanh" else silu_and_mul(x)
 
 
@@ -187,7 +194,7 @@ class ExpertRows:
 
     rows: torch.Tensor          # [pairs, W]
     sorted_pos: torch.Tensor    # [T * k] row of every (token, choice); negative: no row
-    topk_w: torch.Tensor        # [T, k] fp32
+    topk_w: Optional[torch.Tensor]   # [T, k] fp32; None: the experts' inputs were weighted
     ids: torch.Tensor           # [T, k] int32
     token_in: torch.Tensor      # [T, W] the experts' input
     identity_from: int = 0      # > 0: ids from here on return the token's input
@@ -230,15 +237,71 @@ def rownorm_rope_kv(row, q_weight, k_weight, inv_freq, positions, loc, q_out, k_
 
 
 def headnorm_rope_kv(row, inv_freq, positions, loc, q_out, k_cache, v_cache, heads: int, kv_heads: int, dim: int, vdim: int, v_at: int,
-                     halves: bool, eps: float) -> None:
+                     halves: bool, eps: float, norm: bool = True, magnitude: float = 1.0) -> None:
     """Prologue of attention with a norm per head: ``row`` [T, q | k | ..]; query and key heads turn by ``positions *
     inv_freq`` (fp64, one per rotated pair; ``halves``: feature i with the one half the rotated features on, else
     neighbours) and are divided by their root mean square; q goes to ``q_out`` [T, heads, >= dim] (zeros behind), k and the
-    values (columns from ``v_at``, unchanged) to the cache slots ``loc``."""
-    args = (row, inv_freq, positions, loc, q_out, k_cache, v_cache, heads, kv_heads, dim, vdim, v_at, halves, eps)
+    values (columns from ``v_at``, unchanged) to the cache slots ``loc``.  ``norm`` False: heads keep their length.
+    ``magnitude``: factor of the sines and cosines."""
+    args = (row, inv_freq, positions, loc, q_out, k_cache, v_cache, heads, kv_heads, dim, vdim, v_at, halves, eps, norm, float(magnitude))
     if not use_kernels(row):
         return ref.headnorm_rope_kv(*args)
     ext().headnorm_rope_kv(row, inv_freq, positions.to(torch.int64).contiguous(), loc.to(torch.int64).contiguous(), *args[4:])
+
+
+def gated_rmsnorm(x: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, groups: int, eps: float, out: torch.Tensor) -> torch.Tensor:
+    """``out = rmsnorm(x * silu(gate)) * weight``, the mean over each of ``groups`` equal parts of a row; ``gate`` and ``out``
+    may be column slices."""
+    if not use_kernels(x):
+        return out.copy_(ref.gated_rmsnorm(x, gate, weight, groups, eps))
+    ext().gated_rmsnorm(x, gate, weight, out, int(groups), float(eps))
+    return out
+
+
+@dataclass
+class ConvStep:
+    """The causal convolution on the first of a layer's inputs, for batches in which every row is the next token of a request."""
+
+    weight: torch.Tensor        # [W, K]
+    state: torch.Tensor         # [rows, W, K - 1]
+    slots: torch.Tensor         # [T] int32
+
+
+def depth_step(x: torch.Tensor, mix, f: Optional[torch.Tensor], experts: Optional[ExpertRows], results: Optional[torch.Tensor], n: int,
+               dwa: Optional[torch.Tensor], norms, eps: float, dtype: torch.dtype, x_out: Optional[torch.Tensor], keep: bool = True,
+               mix_scale: float = 0.5, conv: Optional[ConvStep] = None):
+    """The step behind a layer whose mixer and feed-forward read the same fp32 stream ``x`` [T, W].  ``mix``: ``(a,)``, the
+    mixer's output, or ``(a, b, a_w, b_w)`` for ``mix_scale * (rmsnorm(a) * a_w + rmsnorm(b) * b_w)``; ``f`` and ``experts``: the
+    feed-forward's output, or expert rows to sum (either may be None).
+
+    ``z = x + mix + ff``; with ``dwa`` (fp32 [n + 1]) ``x' = dwa[n] z + sum_(j < n) dwa[j] results[j]`` and ``z`` is kept as
+    ``results[n]`` when ``keep``; without, ``x' = z``.  ``x'`` goes to ``x_out`` (may be ``x``; None: not written) and
+    ``x' / sqrt(mean(x'^2) + eps) * g`` comes back in ``dtype`` for every one-number weight ``g`` of ``norms`` (one or two).
+    ``conv``: the first of them passes a causal convolution that is added to it."""
+    T, W = x.shape
+    if not use_kernels(x):
+        return ref.depth_step(x, mix, f, experts, results, n, dwa, norms, eps, dtype, x_out, keep, mix_scale, conv)
+    h = [torch.empty((T, W), dtype=dtype, device=x.device) for _ in norms]
+    rows, top = [], 0
+    if experts is not None:
+        rows, top = [experts.rows, experts.sorted_pos], experts.ids.shape[1]
+        if experts.topk_w is not None:
+            rows.append(experts.topk_w.view(-1))
+    ext().depth_step(x, x_out, results, int(n), bool(keep), dwa, list(mix), float(mix_scale), f, rows, top, float(eps), h, list(norms),
+                     [] if conv is None else [conv.weight, conv.state, conv.slots])
+    return h
+
+
+def embed_norm(ids: torch.Tensor, table: torch.Tensor, weight: torch.Tensor, x: torch.Tensor, eps: float, norms,
+               conv: Optional[ConvStep] = None):
+    """Embedding rows divided by their root mean square, times the one number ``weight``, into the fp32 stream ``x`` [T, W];
+    returns the normed inputs of the first layer as :func:`depth_step` does."""
+    if not use_kernels(table):
+        return ref.embed_norm(ids, table, weight, x, eps, norms, conv)
+    h = [torch.empty(x.shape, dtype=table.dtype, device=x.device) for _ in norms]
+    ext().embed_norm(ids.reshape(-1).to(torch.int64).contiguous(), table, weight, x, float(eps), h, list(norms),
+                     [] if conv is None else [conv.weight, conv.state, conv.slots])
+    return h
 
 
 def soft_cap(x: torch.Tensor, cap: float) -> torch.Tensor:
@@ -272,9 +335,9 @@ def residual_dyt(x: torch.Tensor, y: Optional[torch.Tensor], mult: float, alpha:
 # --------------------------------------------------------------------------
 # GEMMs
 # --------------------------------------------------------------------------
-def _gemm(a, b, out, bias, residual, swiglu, a_scale, b_scale) -> None:
+def _gemm(a, b, out, bias, residual, swiglu, a_scale, b_scale, act_limit: float = 0.0) -> None:
     # a Parameter is a model weight: nothing in the stream writes it, so the kernel may fetch it early
-    rc = ext().gemm(a, b, out, bias, residual, int(swiglu), a_scale, b_scale, isinstance(b, torch.nn.Parameter))
+    rc = ext().gemm(a, b, out, bias, residual, int(swiglu), a_scale, b_scale, isinstance(b, torch.nn.Parameter), float(act_limit))
     if rc != 0:
         raise RuntimeError(f"mllm_b200 gemm: unsupported shape or launch failure (code {rc}) for "
                            f"M={a.shape[0]} N={b.shape[0]} K={a.shape[1]}")
@@ -418,12 +481,16 @@ def linear(
     return o.view(*x.shape[:-1], weight.shape[0]) if out is None else out
 
 
-def linear_swiglu(x: torch.Tensor, weight: torch.Tensor, block: int = SWIGLU_BLOCK, act: str = "silu") -> torch.Tensor:
+def linear_swiglu(x: torch.Tensor, weight: torch.Tensor, block: int = SWIGLU_BLOCK, act: str = "silu", bias: Optional[torch.Tensor] = None,
+                  limit: float = 0.0) -> torch.Tensor:
     """``act(x Wg^T) * (x Wu^T)`` in one GEMM; ``weight`` rows alternate ``block`` gate / ``block`` up rows.
-    ``act``: ``silu`` or ``gelu_tanh``."""
+    ``act``: ``silu``, ``gelu_tanh``, or ``clamped``, which takes a bias (in the order of the rows) and a bound: with
+    ``g = min(x Wg^T + b, limit)`` and ``u = clamp(x Wu^T + b, -limit, limit)``, ``g * sigmoid(1.702 g) * (u + 1)``."""
     x2 = _2d(x)
     if not use_kernels(x) or block != SWIGLU_BLOCK or weight.shape[0] % 256 or not _gemm_shape_ok(x2, weight):
-        return ref.linear_swiglu(x, weight, block, act)
+        return ref.linear_swiglu(x, weight, block, act, bias, limit)
+    if bias is not None and act != "clamped":
+        raise ValueError(f"linear_swiglu: no bias with {act!r}")
     if x2.stride(-1) != 1 or (x2.stride(0) * x2.element_size()) % 16:
         x2 = x2.contiguous()
     o = torch.empty((x2.shape[0], weight.shape[0] // 2), dtype=x.dtype, device=x.device)
@@ -431,7 +498,7 @@ def linear_swiglu(x: torch.Tensor, weight: torch.Tensor, block: int = SWIGLU_BLO
     if gate is not None:
         _gemm_tp(x2, weight, o, True, gate=gate)
     else:
-        _gemm(x2, weight, o, None, None, 2 if act == "gelu_tanh" else 1, None, None)
+        _gemm(x2, weight, o, bias, None, {"silu": 1, "gelu_tanh": 2, "clamped": 4}[act], None, None, limit)
     return o.view(*x.shape[:-1], weight.shape[0] // 2)
 
 
@@ -754,19 +821,20 @@ def _attention_kernel_ok(q: torch.Tensor, k_cache: torch.Tensor, window, logit_c
 
 def attention_prefill(q, k_cache, v_cache, req_to_token, req_pool_indices, seq_lens, prefix_lens,
                       q_start_loc, scale: float, out=None, max_q_len: int = 0, window: Optional[int] = None,
-                      logit_cap: float = 0.0, seq_lens_cpu=None, prefix_lens_cpu=None, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+                      logit_cap: float = 0.0, seq_lens_cpu=None, prefix_lens_cpu=None, sink: Optional[torch.Tensor] = None,
+                      chunk: Optional[int] = None) -> torch.Tensor:
     """Causal attention of new tokens over cached prefix + themselves.  ``window``: sliding-window attention
-    (each query sees its last ``window`` keys); ``logit_cap``: soft-capping of the scores; both are mask /
-    score options of the tcgen05 kernels.  ``sink`` [Hq] fp32: ``exp(sink)`` joins each head's softmax denominator.
+    (each query sees its last ``window`` keys); ``chunk``: positions are cut into chunks and each query sees the keys of its own;
+    ``logit_cap``: soft-capping of the scores; all are mask / score options of the tcgen05 kernels.  ``sink`` [Hq] fp32: ``exp(sink)`` joins each head's softmax denominator.
     Head sizes other than 64 / 128 / 256 and caches that hold neither the
     activation dtype nor an 8-bit float take library / PyTorch fallbacks."""
     if _attention_kernel_ok(q, k_cache, window, logit_cap) and hasattr(ext(), "attention_prefill"):
         if out is None:
             out = torch.empty((q.shape[0], q.shape[1], q.shape[2]), dtype=q.dtype, device=q.device)
         ext().attention_prefill(q, k_cache, v_cache, req_to_token, req_pool_indices, seq_lens, prefix_lens,
-                                q_start_loc, scale, out, max_q_len, True, int(window or 0), float(logit_cap or 0.0), sink)
+                                q_start_loc, scale, out, max_q_len, True, int(window or 0), float(logit_cap or 0.0), sink, int(chunk or 0))
         return out
-    if q.is_cuda and not logit_cap and sink is None:
+    if q.is_cuda and not logit_cap and sink is None and not chunk:
         o = ref.attention_prefill_sdpa(q, k_cache, v_cache, req_to_token, req_pool_indices, seq_lens, prefix_lens,
                                        q_start_loc, scale, seq_lens_cpu, prefix_lens_cpu, window)
         if out is None:
@@ -774,32 +842,32 @@ def attention_prefill(q, k_cache, v_cache, req_to_token, req_pool_indices, seq_l
         out.copy_(o)
         return out
     return ref.attention_prefill(q, k_cache, v_cache, req_to_token, req_pool_indices, seq_lens, prefix_lens,
-                                 q_start_loc, scale, out, window=window, logit_cap=logit_cap, sink=sink)
+                                 q_start_loc, scale, out, window=window, logit_cap=logit_cap, sink=sink, chunk=chunk)
 
 
 def attention_decode(q, k_cache, v_cache, req_to_token, req_pool_indices, seq_lens, scale: float,
                      out=None, max_seq_len: int = 0, window: Optional[int] = None, logit_cap: float = 0.0,
-                     sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     sink: Optional[torch.Tensor] = None, chunk: Optional[int] = None) -> torch.Tensor:
     if _attention_kernel_ok(q, k_cache, window, logit_cap) and hasattr(ext(), "attention_decode"):
         if out is None:
             out = torch.empty((q.shape[0], q.shape[1], q.shape[2]), dtype=q.dtype, device=q.device)
         ext().attention_decode(q, k_cache, v_cache, req_to_token, req_pool_indices, seq_lens, scale, out, max_seq_len,
-                               int(window or 0), float(logit_cap or 0.0), sink)
+                               int(window or 0), float(logit_cap or 0.0), sink, int(chunk or 0))
         return out
-    if q.is_cuda and max_seq_len and sink is None:
+    if q.is_cuda and max_seq_len and sink is None and not chunk:
         return ref.attention_decode_batched(q, k_cache, v_cache, req_to_token, req_pool_indices, seq_lens, scale,
                                             max_seq_len, out, window, logit_cap)
     return ref.attention_decode(q, k_cache, v_cache, req_to_token, req_pool_indices, seq_lens, scale, out,
-                                window=window, logit_cap=logit_cap, sink=sink)
+                                window=window, logit_cap=logit_cap, sink=sink, chunk=chunk)
 
 
 def attention_rows(q, k_cache, v_cache, req_to_token, row_req, row_pos, scale: float, out, window: Optional[int] = None,
-                   logit_cap: float = 0.0, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+                   logit_cap: float = 0.0, sink: Optional[torch.Tensor] = None, chunk: Optional[int] = None) -> torch.Tensor:
     """Causal attention for fp32 and for head sizes the tensor-core kernels do not have (key and value widths may
     differ): row t of ``q`` [rows, Hq, D] is a token of request ``row_req[t]`` at position ``row_pos[t]``."""
     if not use_kernels(q):
-        return ref.attention_rows(q, k_cache, v_cache, req_to_token, row_req, row_pos, scale, out, int(window or 0), logit_cap, sink)
-    ext().attention_rows(q, k_cache, v_cache, req_to_token, row_req, row_pos, float(scale), out, int(window or 0), float(logit_cap), sink)
+        return ref.attention_rows(q, k_cache, v_cache, req_to_token, row_req, row_pos, scale, out, int(window or 0), logit_cap, sink, int(chunk or 0))
+    ext().attention_rows(q, k_cache, v_cache, req_to_token, row_req, row_pos, float(scale), out, int(window or 0), float(logit_cap), sink, int(chunk or 0))
     return out
 
 
@@ -891,64 +959,70 @@ def gelu_erf(x: torch.Tensor) -> torch.Tensor:
 # --------------------------------------------------------------------------
 # latent attention (one cached row per token, shared by all heads)
 # --------------------------------------------------------------------------
-def latent_prologue(y: torch.Tensor, q_weight: torch.Tensor, kv_weight: Optional[torch.Tensor], eps: float,
+def latent_prologue(y: torch.Tensor, q_weight: Optional[torch.Tensor], kv_weight: Optional[torch.Tensor], eps: float,
                     loc: Optional[torch.Tensor] = None, cache: Optional[torch.Tensor] = None,
-                    positions: Optional[torch.Tensor] = None, inv_freq: Optional[torch.Tensor] = None):
+                    positions: Optional[torch.Tensor] = None, inv_freq: Optional[torch.Tensor] = None, halves: bool = False):
     """RMS norm (fp32) of the down projections' rows ``y = [query latent | cache latent | rotated key part | ..]``: returns
     the normed query latent [T, q_rank] and writes the normed cache latent to ``cache[loc]`` (``kv_weight`` None: the layer
     reads another layer's latents and writes none).  With ``inv_freq`` (fp64, one per pair of neighbouring features) the key
     part, turned by ``positions * inv_freq``, follows the latent in the cache row, and the cosines and sines [T, rot / 2, 2]
-    come back for the query heads (None without)."""
+    come back for the query heads (None without).  ``q_weight`` None: queries have no latent (``y`` begins with the cache
+    latent).  ``halves``: feature i turns with feature i + rot / 2."""
     if not use_kernels(y):
-        return ref.latent_prologue(y, q_weight, kv_weight, eps, loc, cache, positions, inv_freq)
-    cq = torch.empty((y.shape[0], q_weight.numel()), dtype=y.dtype, device=y.device)
+        return ref.latent_prologue(y, q_weight, kv_weight, eps, loc, cache, positions, inv_freq, halves)
+    cq = None if q_weight is None else torch.empty((y.shape[0], q_weight.numel()), dtype=y.dtype, device=y.device)
     turns = None if inv_freq is None else torch.empty((y.shape[0], inv_freq.numel(), 2), dtype=torch.float32, device=y.device)
     ext().latent_prologue(y, q_weight, kv_weight, eps, cq, None if loc is None else loc.to(torch.int64).contiguous(), cache,
-                          None if inv_freq is None else positions.to(torch.int64).contiguous(), inv_freq, turns)
+                          None if inv_freq is None else positions.to(torch.int64).contiguous(), inv_freq, turns, halves)
     return cq, turns
 
 
-def turn_heads(x: torch.Tensor, turns: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """x [T, H, rot] (a slice of wider heads will do): neighbouring features turn by ``turns`` [T, rot / 2, 2]; in place
-    unless ``out`` is given."""
+def turn_heads(x: torch.Tensor, turns: torch.Tensor, out: Optional[torch.Tensor] = None, halves: bool = False) -> torch.Tensor:
+    """x [T, H, rot] (a slice of wider heads will do): neighbouring features (``halves``: feature i and i + rot / 2) turn by
+    ``turns`` [T, rot / 2, 2]; in place unless ``out`` is given."""
     out = x if out is None else out
     if not use_kernels(x):
-        return out.copy_(ref.turn_heads(x, turns))
-    ext().turn_heads(x, turns, out)
+        return out.copy_(ref.turn_heads(x, turns, halves))
+    ext().turn_heads(x, turns, out, halves)
     return out
 
 
-def gate_heads(x: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
-    """``x[t, h] * sigmoid(gate[t, h])``, contiguous; x [T, H, W] and gate [T, H] may be slices."""
+def gate_heads(x: torch.Tensor, gate: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``x[t, h] * sigmoid(gate[t, h])``; x [T, H, W] and gate may be slices.  ``gate`` [T, H] has a number per head, [T, H * W]
+    one per feature.  The result is contiguous unless ``out`` (which may be ``x``) is given."""
+    out = torch.empty(x.shape, dtype=x.dtype, device=x.device) if out is None else out
     if not use_kernels(x):
-        return (x.float() * torch.sigmoid(gate.float()).unsqueeze(-1)).to(x.dtype)
-    out = torch.empty(x.shape, dtype=x.dtype, device=x.device)
+        g = torch.sigmoid(gate.float())
+        return out.copy_((x.float() * (g.unsqueeze(-1) if g.shape[1] == x.shape[1] else g.reshape(x.shape))).to(x.dtype))
     ext().gate_heads(x, gate, out)
     return out
 
 
-def latent_gather(cache, req_to_token, req, lens, start, total: int, max_len: int) -> torch.Tensor:
-    """[total, rank]: the latents of every request's context back to back (request b's rows begin at ``start[b]``)."""
+def latent_gather(cache, req_to_token, req, lens, start, total: int, max_len: int, first: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """[total, rank]: the latents of every request's context back to back (request b's rows begin at ``start[b]``), from its
+    token ``first[b]`` on."""
     if not use_kernels(cache):
-        return ref.latent_gather(cache, req_to_token, req, lens)
+        return ref.latent_gather(cache, req_to_token, req, lens, first)
     out = torch.empty((total, cache.shape[1]), dtype=cache.dtype, device=cache.device)
-    ext().latent_gather(cache, req_to_token, req, lens, start, max_len, out)
+    ext().latent_gather(cache, req_to_token, req, lens, start, max_len, out, first)
     return out
 
 
-def head_linear(x: torch.Tensor, weight: torch.Tensor, gate: Optional[torch.Tensor] = None, turns: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """``out[t, h] = weight[h] @ x[t, h]``: x [T, H, K], weight [H, N, K] -> [T, H, N].  ``gate`` [T, H]: times its logistic
-    function.  ``turns`` [T, rot / 2, 2]: x is [T, H, K + rot], and the features behind K, turned, follow the N results."""
+def head_linear(x: torch.Tensor, weight: torch.Tensor, gate: Optional[torch.Tensor] = None, turns: Optional[torch.Tensor] = None,
+                halves: bool = False) -> torch.Tensor:
+    """``out[t, h] = weight[h] @ x[t, h]``: x [T, H, K], weight [H, N, K] -> [T, H, N].  ``gate`` [T, H] or [T, H * N]: times its
+    logistic function.  ``turns`` [T, rot / 2, 2]: x is [T, H, K + rot], and the features behind K, turned (``halves``: as in
+    :func:`turn_heads`), follow the N results."""
     T, H, N, K = x.shape[0], x.shape[1], weight.shape[1], weight.shape[2]
     out = torch.empty((T, H, N + x.shape[2] - K), dtype=x.dtype, device=x.device)
     if use_kernels(x) and x.dtype != torch.float32:
-        if T == 0 or ext().head_linear(x, weight, out, gate, turns) == 0:
+        if T == 0 or ext().head_linear(x, weight, out, gate, turns, halves) == 0:
             return out
     # 32-bit and unaligned sizes: a library batched product
     torch.bmm(x[..., :K].transpose(0, 1), weight.transpose(1, 2), out=(y := torch.empty((H, T, N), dtype=x.dtype, device=x.device)))
     out[..., :N] = y.transpose(0, 1)
     if turns is not None:
-        turn_heads(x[..., K:], turns, out[..., N:])
+        turn_heads(x[..., K:], turns, out[..., N:], halves)
     return out if gate is None else gate_heads(out, gate)
 
 
@@ -956,27 +1030,30 @@ _LATENT_ROWS = 32768     # query rows of one launch (they are a grid dimension)
 
 
 def latent_attention(q: torch.Tensor, cache: torch.Tensor, req_to_token, row_req, row_pos, scale: float,
-                     sink: Optional[torch.Tensor] = None, max_seq_len: int = 0, rank: Optional[int] = None) -> torch.Tensor:
+                     sink: Optional[torch.Tensor] = None, max_seq_len: int = 0, rank: Optional[int] = None,
+                     window: Optional[int] = None) -> torch.Tensor:
     """Attention of queries in the latent space over the cached rows, which are keys and values at once: row t is a
-    token of request ``row_req[t]`` at position ``row_pos[t]`` and sees the keys 0 .. its position.  Keys are whole rows,
+    token of request ``row_req[t]`` at position ``row_pos[t]`` and sees the keys 0 .. its position, the last ``window`` of them
+    where that is given.  Keys are whole rows,
     values their first ``rank`` features (default: all).  q [rows, H, key width] -> [rows, H, rank]; ``sink`` [H] fp32 joins
     the denominator as ``exp(sink)``."""
     rank = q.shape[2] if rank is None else rank
     if not use_kernels(q):
-        return ref.latent_attention(q, cache, req_to_token, row_req, row_pos, scale, sink, rank)
+        return ref.latent_attention(q, cache, req_to_token, row_req, row_pos, scale, sink, rank, int(window or 0))
     q = q.contiguous()
     out = torch.empty((q.shape[0], q.shape[1], rank), dtype=q.dtype, device=q.device)
     for r in range(0, q.shape[0], _LATENT_ROWS):
         e = min(q.shape[0], r + _LATENT_ROWS)
-        ext().latent_attention(q[r:e], cache, req_to_token, row_req[r:e], row_pos[r:e], float(scale), sink, out[r:e], int(max_seq_len))
+        ext().latent_attention(q[r:e], cache, req_to_token, row_req[r:e], row_pos[r:e], float(scale), sink, out[r:e], int(max_seq_len), int(window or 0))
     return out
 
 
 # --------------------------------------------------------------------------
 # gated delta net (linear attention of the hybrid models)
 # --------------------------------------------------------------------------
-def rmsnorm_gated(x: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, round_norm: bool = True) -> torch.Tensor:
-    """``weight * rmsnorm(x) * silu(gate)``, the norm taken over runs of ``weight.numel()`` features of the last
+def rmsnorm_gated(x: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, round_norm: bool = True,
+                  sigmoid: bool = False) -> torch.Tensor:
+    """``weight * rmsnorm(x) * silu(gate)`` (``sigmoid``: times ``sigmoid(gate)``), the norm taken over runs of ``weight.numel()`` features of the last
     dimension.  ``gate`` may be a column slice of a wider matrix.  ``round_norm``: the normed value is rounded to the
     tensors' type before it is multiplied."""
     if use_kernels(x):
@@ -987,16 +1064,18 @@ def rmsnorm_gated(x: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps
             raise ValueError("rmsnorm_gated: the last dimension must hold whole heads")
         x2 = x2.contiguous()
         out = torch.empty_like(x2)
-        ext().rmsnorm_gated(x2, g2, weight, out, eps, round_norm)
+        ext().rmsnorm_gated(x2, g2, weight, out, eps, round_norm, sigmoid)
         return out.view(x.shape)
-    return ref.rmsnorm_gated(x, gate, weight, eps, round_norm)
+    return ref.rmsnorm_gated(x, gate, weight, eps, round_norm, sigmoid)
 
 
-def causal_conv1d_silu(x, weight, conv_state, state_indices, seq_lens, has_state, q_start=None, max_len: int = 0) -> torch.Tensor:
+def causal_conv1d_silu(x, weight, conv_state, state_indices, seq_lens, has_state, q_start=None, max_len: int = 0,
+                       bias: Optional[torch.Tensor] = None, add_input: bool = False) -> torch.Tensor:
     """Depth-wise causal conv (kernel K) + SiLU over the new tokens of every request, reading / updating
     the per-request history rows of ``conv_state``.  ``seq_lens`` / ``has_state`` may be host lists (CPU
     path) or device int32 tensors (GPU path, no host sync; ``q_start`` = first row of each request).  ``x`` may be a
-    column slice of a wider matrix; ``max_len``: the longest run of new tokens, when the host knows it."""
+    column slice of a wider matrix; ``max_len``: the longest run of new tokens, when the host knows it.  ``bias`` [C] joins
+    the convolution; ``add_input``: the result is ``x + conv(x)``, without the SiLU."""
     if use_kernels(x):
         dev = x.device
         lens = seq_lens if isinstance(seq_lens, torch.Tensor) else torch.tensor(list(seq_lens), dtype=torch.int32, device=dev)
@@ -1006,11 +1085,11 @@ def causal_conv1d_silu(x, weight, conv_state, state_indices, seq_lens, has_state
         out = torch.empty(x.shape, dtype=x.dtype, device=dev)
         ext().gdn_conv1d_silu(x if x.stride(-1) == 1 else x.contiguous(), weight.contiguous(), conv_state,
                               state_indices.to(torch.int32), lens.to(torch.int32), has.to(torch.int32), q_start.to(torch.int32),
-                              out, int(max_len))
+                              out, int(max_len), bias, add_input)
         return out
     lens = seq_lens.tolist() if isinstance(seq_lens, torch.Tensor) else seq_lens
     has = has_state.tolist() if isinstance(has_state, torch.Tensor) else has_state
-    return ref.causal_conv1d_silu(x, weight, conv_state, state_indices, lens, has)
+    return ref.causal_conv1d_silu(x, weight, conv_state, state_indices, lens, has, bias, add_input)
 
 
 def gdn_gates(b: torch.Tensor, a: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor) -> Tuple[torch.Tensor, torch.Tensor]:
@@ -1083,8 +1162,32 @@ def gated_delta_rule(q, k, v, g, beta, state, state_indices, seq_lens, has_state
     return ref.gated_delta_rule(q, k, v, g, beta, state, state_indices, lens, has)
 
 
+def channel_delta_rule(q, k, v, b, a, a_log, dt_bias, state, state_indices, seq_lens, has_state, q_start=None, max_len: int = 0) -> torch.Tensor:
+    """Gated delta rule with a decay per key channel: ``S <- diag(exp(g)) S``, ``S <- S + k (beta (v - S^T k))^T``, ``o = S^T q``,
+    with unit q and k (q also times ``Dk^-0.5``), ``g[h, d] = -exp(a_log[h]) * softplus(a[h, d] + dt_bias[h, d])`` and
+    ``beta = sigmoid(b)``.  q, k [T, Hk, Dk] (value head h uses head ``h // (H / Hk)``), v [T, H, Dv], b [T, H] and a [T, H * Dk] raw
+    projections (all may be rows of wider matrices), a_log [H] and dt_bias [H * Dk] fp32; state and metadata as for
+    :func:`gated_delta_rule`, whose extend-backend choice also holds here."""
+    H = v.shape[1]
+    if use_kernels(q) and q.shape[-1] <= _GDN_MAX_DK and _GDN_EXTEND_BACKEND != "pytorch":
+        lens = seq_lens.to(torch.int32)
+        if q_start is None:
+            q_start = torch.cumsum(lens, 0, dtype=torch.int32) - lens
+        out = torch.empty((v.shape[0], H, v.shape[2]), dtype=v.dtype, device=v.device)
+        q, k, v = (t if t.stride(2) == 1 and t.stride(1) == t.shape[2] else t.contiguous() for t in (q, k, v))
+        args = (q, k, v, b, a, a_log, dt_bias, state, state_indices.to(torch.int32), lens, has_state.to(torch.int32), q_start.to(torch.int32), out)
+        chunked = _GDN_EXTEND_BACKEND == "cuda_chunkwise" or (
+            _GDN_EXTEND_BACKEND != "mllm_kernel" and q.shape[0] >= 32 * max(1, lens.numel()))
+        if not chunked or ext().gdn_channel_chunk(*args, int(max_len)) != 0:
+            ext().gdn_channel_recurrent(*args)
+        return out
+    lens = seq_lens.tolist() if isinstance(seq_lens, torch.Tensor) else seq_lens
+    has = has_state.tolist() if isinstance(has_state, torch.Tensor) else has_state
+    return ref.channel_delta_rule(_heads_like(q, H), _heads_like(k, H), v, b, a, a_log, dt_bias, state, state_indices, lens, has)
+
+
 # --------------------------------------------------------------------------
-# lightning attention (linear attention with a fixed decay per head)
+# lightning attention (linear attention with a fixed decay per head), state-space duality
 # --------------------------------------------------------------------------
 def lightning_attention(q, k, v, decay, state, state_indices, seq_lens, has_state, q_start=None, max_len: int = 0) -> torch.Tensor:
     """``S <- decay S + k v^T``, ``o = S^T q`` with q, k [T, H, D] and v [T, H, Dv] taken through SiLU first; tokens may be
@@ -1105,6 +1208,28 @@ def lightning_attention(q, k, v, decay, state, state_indices, seq_lens, has_stat
         _GDN_EXTEND_BACKEND != "mllm_kernel" and q.shape[0] >= 32 * max(1, lens.numel()))
     if not chunked or ext().lightning_chunk(*args, int(max_len)) != 0:
         ext().lightning_recurrent(*args)
+    return out
+
+
+def state_space(x, B, C, dt, dt_bias, a_log, skip, state, state_indices, seq_lens, has_state, q_start=None, max_len: int = 0) -> torch.Tensor:
+    """State-space duality: ``S <- exp(-exp(a_log) dt) S + dt B x^T``, ``y = S^T C + skip x`` with
+    ``dt = softplus(dt + dt_bias)``.  x [T, H, P], B and C [T, G, N] (head h uses group ``h // (H / G)``), activated already, dt [T, H]
+    raw; tokens may be rows of wider matrices; ``dt_bias``, ``a_log``, ``skip`` fp32 [H].  ``state`` fp32 [rows, H, N, P]; metadata,
+    extend-backend choice and ``max_len`` as for :func:`lightning_attention`."""
+    if not use_kernels(x):
+        lens = seq_lens.tolist() if isinstance(seq_lens, torch.Tensor) else seq_lens
+        has = has_state.tolist() if isinstance(has_state, torch.Tensor) else has_state
+        return ref.state_space(x, B, C, dt, dt_bias, a_log, skip, state, state_indices, lens, has).to(x.dtype)
+    lens = seq_lens.to(torch.int32)
+    if q_start is None:
+        q_start = torch.cumsum(lens, 0, dtype=torch.int32) - lens
+    out = torch.empty(x.shape, dtype=x.dtype, device=x.device)
+    x, B, C = (t if t.stride(2) == 1 and t.stride(1) == t.shape[2] else t.contiguous() for t in (x, B, C))
+    args = (x, B, C, dt, dt_bias, a_log, skip, state, state_indices.to(torch.int32), lens, has_state.to(torch.int32), q_start.to(torch.int32), out)
+    chunked = _GDN_EXTEND_BACKEND == "cuda_chunkwise" or (
+        _GDN_EXTEND_BACKEND != "mllm_kernel" and x.shape[0] >= 32 * max(1, lens.numel()))
+    if not chunked or ext().state_space_chunk(*args, int(max_len)) != 0:
+        ext().state_space_recurrent(*args)
     return out
 
 
@@ -1162,24 +1287,26 @@ def moe_chunk_rows(tokens: int, top_k: int, num_experts_global: int) -> int:
     return 128
 
 
-def _moe_gemm(x, w, out, offsets, work, n_work, bn, swiglu, any_size: bool = False) -> None:
-    rc = ext().moe_grouped_gemm(x, w, out, offsets, work, n_work, bn, swiglu, any_size)
+def _moe_gemm(x, w, out, offsets, work, n_work, bn, swiglu, any_size: bool = False, gelu: bool = False) -> None:
+    rc = ext().moe_grouped_gemm(x, w, out, offsets, work, n_work, bn, swiglu, any_size, gelu)
     if rc != 0:
         raise RuntimeError(f"mllm_b200 moe_grouped_gemm: unsupported shape or launch failure (code {rc}) for "
                            f"x={tuple(x.shape)} w={tuple(w.shape)}")
 
 
-def _moe_sorted_rows(x, w13, w2, topk_ids, expert_offset: int, swiglu_block: int, num_experts_global: Optional[int]):
+def _moe_sorted_rows(x, w13, w2, topk_ids, expert_offset: int, swiglu_block: int, num_experts_global: Optional[int],
+                     input_w: Optional[torch.Tensor] = None, gated: bool = True):
     """Expert outputs in expert order [pairs, H] and the row of every pair.  Everything stays on the device (no host read
     of the routing, so the step can be captured in a CUDA graph): pairs are counting-sorted by expert, activations
     gathered into expert order, and both expert GEMMs run as one grouped launch each — on tcgen05, SwiGLU fused into
     the first when ``w13`` is stored in 128-row gate/up blocks, or, for fp32 and sizes that are no multiple of 8, on a
-    plain kernel."""
+    plain kernel.  ``gated`` False: experts are ``w2 gelu(w13 x)`` without a gate, the exact GELU inside the first product.
+    ``input_w`` [T, k]: what an expert reads is multiplied by the pair's weight."""
     if swiglu_block not in (0, SWIGLU_BLOCK):
         raise ValueError(f"w13 interleave block must be 0 or {SWIGLU_BLOCK}")
     T, H = x.shape
     E, N13, _ = w13.shape
-    inter = N13 // 2
+    inter = N13 // 2 if gated else N13
     k = topk_ids.shape[1]
     P = T * k
     dev = x.device
@@ -1194,11 +1321,18 @@ def _moe_sorted_rows(x, w13, w2, topk_ids, expert_offset: int, swiglu_block: int
     n_work = torch.empty(1, **i32)
     e = ext()
     ids = topk_ids if topk_ids.dtype == torch.int32 else topk_ids.to(torch.int32)
-    e.moe_align(ids.contiguous(), int(expert_offset), E, bn, sorted_pos, src_token, offsets, work, n_work)
     xs = torch.empty((P, H), dtype=x.dtype, device=dev)
-    e.moe_gather(x, src_token, offsets, xs)
+    if input_w is None:
+        e.moe_align(ids.contiguous(), int(expert_offset), E, bn, sorted_pos, src_token, offsets, work, n_work)
+        e.moe_gather(x, src_token, offsets, xs)
+    else:
+        src_w = torch.empty(P, dtype=torch.float32, device=dev)
+        e.moe_align(ids.contiguous(), int(expert_offset), E, bn, sorted_pos, src_token, offsets, work, n_work, input_w.reshape(-1), src_w)
+        e.moe_gather_scaled(x, src_token, src_w, offsets, xs)
     h = torch.empty((P, inter), dtype=x.dtype, device=dev)
-    if swiglu_block and not any_size:
+    if not gated:
+        _moe_gemm(xs, w13, h, offsets, work, n_work, bn, False, any_size, True)
+    elif swiglu_block and not any_size:
         _moe_gemm(xs, w13, h, offsets, work, n_work, bn, True)
     else:
         if swiglu_block:
@@ -1223,14 +1357,16 @@ def moe_experts(x, w13, w2, topk_w, topk_ids, expert_offset: int = 0, swiglu_blo
 
 
 def moe_expert_rows(x, w13, w2, topk_w, topk_ids, swiglu_block: int = 0, identity_from: int = 0,
-                    shared_logit: Optional[torch.Tensor] = None) -> ExpertRows:
+                    shared_logit: Optional[torch.Tensor] = None, gated: bool = True, weigh_input: bool = False) -> ExpertRows:
     """The experts' outputs for a kernel that sums them itself (:func:`post_norm`).  ``identity_from`` > 0: ids from there
-    on are identity experts, which return the token's input and have no row."""
+    on are identity experts, which return the token's input and have no row.  ``gated`` False: experts without a gate
+    (:func:`_moe_sorted_rows`); ``weigh_input``: the weights scale what the experts read, and their rows are just summed."""
+    w_in = topk_w.contiguous() if weigh_input else None
     if not use_kernels(x):
-        rows, pos = ref.moe_expert_rows(x, w13, w2, topk_ids, swiglu_block)
+        rows, pos = ref.moe_expert_rows(x, w13, w2, topk_ids, swiglu_block, gated, w_in)
     else:
-        rows, pos = _moe_sorted_rows(x, w13, w2, topk_ids, 0, swiglu_block, None)
-    return ExpertRows(rows, pos, topk_w.contiguous(), topk_ids.contiguous(), x.contiguous(), int(identity_from), shared_logit)
+        rows, pos = _moe_sorted_rows(x, w13, w2, topk_ids, 0, swiglu_block, None, w_in, gated)
+    return ExpertRows(rows, pos, None if weigh_input else topk_w.contiguous(), topk_ids.contiguous(), x.contiguous(), int(identity_from), shared_logit)
 
 
 def ep_moe_exchange(x_own, w13, w2, topk_w, topk_ids, swiglu_block: int, comm) -> torch.Tensor:

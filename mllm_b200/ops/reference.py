@@ -118,14 +118,25 @@ def interleave_gate_up(w: torch.Tensor, block: int) -> torch.Tensor:
     return torch.cat([g, u], dim=1).reshape(w.shape)
 
 
-def linear_swiglu(x: torch.Tensor, weight: torch.Tensor, block: int = 0, act: str = "silu") -> torch.Tensor:
-    """``act(x Wg^T) * (x Wu^T)``; ``block`` = row interleave of ``weight`` (0: ``[gate ; up]``)."""
+def clamped_gate(gate: torch.Tensor, up: torch.Tensor, limit: float) -> torch.Tensor:
+    """Gated unit with bounds: ``g = min(gate, limit)``, ``u = clamp(up, -limit, limit)``, ``g * sigmoid(1.702 g) * (u + 1)``."""
+    g, u = _f32(gate).clamp(max=limit), _f32(up).clamp(-limit, limit)
+    return (g * torch.sigmoid(1.702 * g) * (u + 1.0)).to(gate.dtype)
+
+
+def linear_swiglu(x: torch.Tensor, weight: torch.Tensor, block: int = 0, act: str = "silu", bias: Optional[torch.Tensor] = None,
+                  limit: float = 0.0) -> torch.Tensor:
+    """``act(x Wg^T) * (x Wu^T)``; ``block`` = row interleave of ``weight`` (0: ``[gate ; up]``) and of ``bias``."""
     y = _f32(x) @ _f32(weight).t()
+    if bias is not None:
+        y = y + _f32(bias)
     if block:
         g, u = deinterleave_gate_up(y, block)
     else:
         d = y.shape[-1] // 2
         g, u = y[..., :d], y[..., d:]
+    if act == "clamped":
+        return clamped_gate(g, u, limit).to(x.dtype)
     return ((F.gelu(g, approximate="tanh") if act == "gelu_tanh" else F.silu(g)) * u).to(x.dtype)
 
 
@@ -273,10 +284,11 @@ def create_kv_indices(req_to_token: torch.Tensor, req_pool_indices: torch.Tensor
 # --------------------------------------------------------------------------
 # attention over the slot-indexed KV pool
 # --------------------------------------------------------------------------
-def _attend(q, k, v, scale, causal_offset: Optional[int], window: Optional[int] = None, logit_cap: float = 0.0, sink=None):
+def _attend(q, k, v, scale, causal_offset: Optional[int], window: Optional[int] = None, logit_cap: float = 0.0, sink=None,
+            chunk: Optional[int] = None):
     """q [Tq,Hq,D] k,v [Tk,Hkv,D] fp32 -> [Tq,Hq,D]; key j visible to query i iff j <= i + causal_offset and,
     with a sliding ``window``, j > i + causal_offset - window (the last ``window`` keys, the query's own
-    included).  ``sink`` [Hq]: one more softmax term per head, without a value.  ``logit_cap`` > 0 soft-caps the scaled scores: ``cap * tanh(s / cap)``."""
+    included); with ``chunk``, keys before the start of the query's chunk of positions are hidden too.  ``sink`` [Hq]: one more softmax term per head, without a value.  ``logit_cap`` > 0 soft-caps the scaled scores: ``cap * tanh(s / cap)``."""
     Hq, Hkv = q.shape[1], k.shape[1]
     g = Hq // Hkv
     kk = k.repeat_interleave(g, dim=1)
@@ -284,13 +296,15 @@ def _attend(q, k, v, scale, causal_offset: Optional[int], window: Optional[int] 
     s = torch.einsum("qhd,khd->hqk", q, kk) * scale
     if logit_cap and logit_cap > 0:
         s = logit_cap * torch.tanh(s / logit_cap)
-    if causal_offset is not None or window:
+    if causal_offset is not None or window or chunk:
         off = causal_offset if causal_offset is not None else k.shape[0] - q.shape[0]
         i = torch.arange(q.shape[0], device=q.device).unsqueeze(-1)
         j = torch.arange(k.shape[0], device=q.device).unsqueeze(0)
         hidden = j > i + off if causal_offset is not None else torch.zeros_like(j > i)
         if window:
             hidden = hidden | (j <= i + off - int(window))
+        elif chunk:
+            hidden = hidden | (j < (i + off) // int(chunk) * int(chunk))
         s = s.masked_fill(hidden, float("-inf"))
     p = sink_softmax(s, sink)
     return torch.einsum("hqk,khd->qhd", p, vv)
@@ -322,7 +336,7 @@ def attention_prefill(
     q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, req_to_token: torch.Tensor,
     req_pool_indices: torch.Tensor, seq_lens: torch.Tensor, prefix_lens: torch.Tensor,
     q_start_loc: torch.Tensor, scale: float, out: Optional[torch.Tensor] = None, max_q_len: int = 0,
-    window: Optional[int] = None, logit_cap: float = 0.0, sink: Optional[torch.Tensor] = None,
+    window: Optional[int] = None, logit_cap: float = 0.0, sink: Optional[torch.Tensor] = None, chunk: Optional[int] = None,
 ) -> torch.Tensor:
     """Causal attention of each request's new tokens over its cached prefix plus itself.
 
@@ -334,7 +348,7 @@ def attention_prefill(
         sl, pl, qs = int(seq_lens[b]), int(prefix_lens[b]), int(q_start_loc[b])
         n = sl - pl
         slots = req_to_token[int(req_pool_indices[b]), :sl].long()
-        o = _attend(_f32(q[qs : qs + n]), _f32(k_cache[slots]), _f32(v_cache[slots]), scale, pl, window, logit_cap, sink)
+        o = _attend(_f32(q[qs : qs + n]), _f32(k_cache[slots]), _f32(v_cache[slots]), scale, pl, window, logit_cap, sink, chunk)
         out[qs : qs + n] = o.to(out.dtype)
     return out
 
@@ -360,14 +374,14 @@ def attention_prefill_sdpa(q, k_cache, v_cache, req_to_token, req_pool_indices, 
 def attention_decode(
     q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, req_to_token: torch.Tensor,
     req_pool_indices: torch.Tensor, seq_lens: torch.Tensor, scale: float, out: Optional[torch.Tensor] = None,
-    window: Optional[int] = None, logit_cap: float = 0.0, sink: Optional[torch.Tensor] = None,
+    window: Optional[int] = None, logit_cap: float = 0.0, sink: Optional[torch.Tensor] = None, chunk: Optional[int] = None,
 ) -> torch.Tensor:
     """One query token per request over ``req_to_token[req, :seq_len]`` (the new token's K/V included)."""
     out = torch.empty_like(q) if out is None else out
     for b in range(req_pool_indices.numel()):
         sl = int(seq_lens[b])
         slots = req_to_token[int(req_pool_indices[b]), :sl].long()
-        o = _attend(_f32(q[b : b + 1]), _f32(k_cache[slots]), _f32(v_cache[slots]), scale, None, window, logit_cap, sink)
+        o = _attend(_f32(q[b : b + 1]), _f32(k_cache[slots]), _f32(v_cache[slots]), scale, None, window, logit_cap, sink, chunk)
         out[b] = o[0].to(out.dtype)
     return out
 
@@ -517,14 +531,16 @@ def moe_experts(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_w: to
     return out.to(x.dtype)
 
 
-def moe_expert_rows(x, w13, w2, topk_ids, swiglu_block: int = 0):
+def moe_expert_rows(x, w13, w2, topk_ids, swiglu_block: int = 0, gated: bool = True, input_w: Optional[torch.Tensor] = None):
     """Outputs of the chosen experts, a row per (token, choice), and the row of every pair (-1: no such expert)."""
     T, k = topk_ids.shape
     rows = torch.zeros((T * k, x.shape[1]), dtype=x.dtype, device=x.device)
     for e in range(w13.shape[0]):
         tok, slot = (topk_ids == e).nonzero(as_tuple=True)
         if tok.numel():
-            rows[tok * k + slot] = linear(linear_swiglu(x[tok], w13[e], swiglu_block), w2[e])
+            xe = x[tok] if input_w is None else (_f32(x[tok]) * input_w[tok, slot].unsqueeze(-1)).to(x.dtype)
+            h = linear_swiglu(xe, w13[e], swiglu_block) if gated else F.gelu(_f32(linear(xe, w13[e], out_dtype=torch.float32))).to(x.dtype)
+            rows[tok * k + slot] = linear(h, w2[e])
     flat = topk_ids.reshape(-1)
     pos = torch.arange(T * k, dtype=torch.int32, device=x.device)
     return rows, torch.where((flat >= 0) & (flat < w13.shape[0]), pos, torch.full_like(pos, -1))
@@ -598,17 +614,68 @@ def rotate_halves(x: torch.Tensor, positions: torch.Tensor, inv_freq: torch.Tens
     return torch.cat([u * c - v * s, v * c + u * s, x[..., 2 * n:]], -1)
 
 
-def headnorm_rope_kv(row, inv_freq, positions, loc, q_out, k_cache, v_cache, heads, kv_heads, dim, vdim, v_at, halves, eps):
-    T, turn = row.shape[0], rotate_halves if halves else rotate_pairs
+def headnorm_rope_kv(row, inv_freq, positions, loc, q_out, k_cache, v_cache, heads, kv_heads, dim, vdim, v_at, halves, eps, norm=True,
+                     magnitude=1.0):
+    T, turn, R = row.shape[0], rotate_halves if halves else rotate_pairs, 2 * inv_freq.numel()
 
     def head(t, n):
         t = turn(_f32(t).reshape(T, n, dim), positions, inv_freq)
-        return t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps)
+        t = torch.cat([t[..., :R] * magnitude, t[..., R:]], -1)
+        return t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps) if norm else t
 
     q_out.zero_()
     q_out[..., :dim] = head(row[:, : heads * dim], heads).to(q_out.dtype)
     k_cache[loc.long(), :, :dim] = head(row[:, heads * dim: (heads + kv_heads) * dim], kv_heads).to(k_cache.dtype)
     v_cache[loc.long(), :, :vdim] = row[:, v_at: v_at + kv_heads * vdim].reshape(T, kv_heads, vdim)
+
+
+def gated_rmsnorm(x, gate, weight, groups, eps):
+    z = (_f32(x) * F.silu(_f32(gate))).unflatten(-1, (groups, -1))
+    z = (z * torch.rsqrt(z.pow(2).mean(-1, keepdim=True) + eps)).flatten(-2)
+    return (z * _f32(weight)).to(x.dtype)
+
+
+def _depth_inputs(x, norms, eps, dtype, conv):
+    r = torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)
+    h = [(x * r * _f32(g)).to(dtype) for g in norms]
+    if conv is not None:        # every row is the next token of the request with state row slots[t]
+        at = conv.slots.long()
+        seq = torch.cat([conv.state[at], h[0].unsqueeze(-1)], -1)
+        h[0] = (_f32(h[0]) + (_f32(seq) * _f32(conv.weight)).sum(-1)).to(dtype)
+        conv.state[at] = seq[..., 1:]
+    return h
+
+
+def depth_step(x, mix, f, experts, results, n, dwa, norms, eps, dtype, x_out, keep=True, mix_scale=0.5, conv=None):
+    def norm(t, w):
+        t = _f32(t)
+        return t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps) * _f32(w)
+
+    z = _f32(mix[0]) if len(mix) == 1 else mix_scale * (norm(mix[0], mix[2]) + norm(mix[1], mix[3]))
+    if f is not None:
+        z = z + _f32(f)
+    if experts is not None:
+        T, k = experts.ids.shape
+        pos = experts.sorted_pos[: T * k].view(T, k).long()
+        part = torch.where((pos >= 0).unsqueeze(-1), _f32(experts.rows)[pos.clamp(min=0)], torch.zeros((), device=x.device))
+        z = z + (part if experts.topk_w is None else part * _f32(experts.topk_w).unsqueeze(-1)).sum(1)
+    z = x + z
+    out = z
+    if dwa is not None:
+        if keep:
+            results[n] = z
+        out = dwa[n] * z
+        for j in range(n):
+            out = out + dwa[j] * results[j]
+    if x_out is not None:
+        x_out.copy_(out)
+    return _depth_inputs(out, norms, eps, dtype, conv)
+
+
+def embed_norm(ids, table, weight, x, eps, norms, conv=None):
+    e = _f32(embedding(ids, table)).view(x.shape)
+    x.copy_(e * torch.rsqrt(e.pow(2).mean(-1, keepdim=True) + eps) * _f32(weight))
+    return _depth_inputs(x, norms, eps, table.dtype, conv)
 
 
 def soft_cap(x, cap):
@@ -619,11 +686,11 @@ def relu_squared(x):
     return x.copy_(torch.relu(x) ** 2)
 
 
-def attention_rows(q, k_cache, v_cache, req_to_token, row_req, row_pos, scale, out, window=0, logit_cap=0.0, sink=None):
+def attention_rows(q, k_cache, v_cache, req_to_token, row_req, row_pos, scale, out, window=0, logit_cap=0.0, sink=None, chunk=0):
     rep = q.shape[1] // k_cache.shape[1]
     for t in range(q.shape[0]):
         pos = int(row_pos[t])
-        lo = max(0, pos - window + 1) if window else 0
+        lo = max(0, pos - window + 1) if window else pos // chunk * chunk if chunk else 0
         slots = req_to_token[int(row_req[t]), lo: pos + 1].long()
         k = _f32(k_cache[slots]).repeat_interleave(rep, 1)                 # [n, H, D]
         v = _f32(v_cache[slots]).repeat_interleave(rep, 1)
@@ -649,6 +716,46 @@ def lightning_attention(q, k, v, decay, state, state_indices, seq_lens, has_stat
     return out
 
 
+def state_space(x, B, C, dt, dt_bias, a_log, skip, state, state_indices, seq_lens, has_state):
+    """x [T, H, P], B and C [T, G, N] activated, dt [T, H] raw; the state rows [H, N, P] are read where ``has_state`` and written
+    back."""
+    H = x.shape[1]
+    xf, B, C = _f32(x), _f32(B).repeat_interleave(H // B.shape[1], 1), _f32(C).repeat_interleave(H // C.shape[1], 1)
+    step = F.softplus(_f32(dt) + _f32(dt_bias))                                  # [T, H]
+    decay = torch.exp(-torch.exp(_f32(a_log)) * step)
+    out, at = torch.empty(x.shape, dtype=torch.float32, device=x.device), 0
+    for slot, n, has in zip(state_indices.tolist(), seq_lens, has_state):
+        S = state[slot].clone() if has else torch.zeros_like(state[slot])
+        for t in range(at, at + n):
+            S = decay[t].view(-1, 1, 1) * S + B[t].unsqueeze(-1) * (step[t].unsqueeze(-1) * xf[t]).unsqueeze(-2)
+            out[t] = (S * C[t].unsqueeze(-1)).sum(-2) + _f32(skip).unsqueeze(-1) * xf[t]
+        state[slot] = S
+        at += n
+    return out
+
+
+def channel_delta_rule(q, k, v, b, a, a_log, dt_bias, state, state_indices, seq_lens, has_state):
+    """q, k [T, H, Dk], v [T, H, Dv], b [T, H], a [T, H * Dk] raw; the state rows [H, Dk, Dv] are read where ``has_state`` and
+    written back."""
+    T, H, Dk = q.shape
+    qf, kf, vf = _f32(q), _f32(k), _f32(v)
+    qf = qf * torch.rsqrt((qf * qf).sum(-1, keepdim=True) + 1e-6) * Dk ** -0.5
+    kf = kf * torch.rsqrt((kf * kf).sum(-1, keepdim=True) + 1e-6)
+    decay = torch.exp(-torch.exp(_f32(a_log)).view(1, H, 1) * F.softplus(_f32(a) + _f32(dt_bias)).view(T, H, Dk))
+    beta = torch.sigmoid(_f32(b))
+    out, at = torch.empty(v.shape, dtype=torch.float32, device=v.device), 0
+    for slot, n, has in zip(state_indices.tolist(), seq_lens, has_state):
+        S = state[slot].clone() if has else torch.zeros_like(state[slot])
+        for t in range(at, at + int(n)):
+            S = decay[t].unsqueeze(-1) * S
+            u = beta[t].unsqueeze(-1) * (vf[t] - (S * kf[t].unsqueeze(-1)).sum(-2))
+            S = S + kf[t].unsqueeze(-1) * u.unsqueeze(-2)
+            out[t] = (S * qf[t].unsqueeze(-1)).sum(-2)
+        state[slot] = S
+        at += int(n)
+    return out.to(v.dtype)
+
+
 def residual_dyt(x, y, mult, alpha, weight, bias, dtype):
     if y is not None:
         x.add_(_f32(y), alpha=float(mult))
@@ -661,37 +768,42 @@ def turns_of(positions, inv_freq):
     return torch.stack([torch.cos(a), torch.sin(a)], -1).float()
 
 
-def turn_heads(x, turns):
-    """x [T, H, rot]: neighbouring features turn by ``turns`` [T, rot / 2, 2]."""
+def turn_heads(x, turns, halves=False):
+    """x [T, H, rot]: neighbouring features (``halves``: feature i and i + rot / 2) turn by ``turns`` [T, rot / 2, 2]."""
     c, s = turns[:, None, :, 0], turns[:, None, :, 1]
+    if halves:
+        u, v = _f32(x).chunk(2, dim=-1)
+        return torch.cat([u * c - v * s, v * c + u * s], -1).to(x.dtype)
     u, v = _f32(x[..., 0::2]), _f32(x[..., 1::2])
     return torch.stack([u * c - v * s, v * c + u * s], -1).flatten(-2).to(x.dtype)
 
 
-def latent_prologue(y, q_weight, kv_weight, eps, loc=None, cache=None, positions=None, inv_freq=None):
+def latent_prologue(y, q_weight, kv_weight, eps, loc=None, cache=None, positions=None, inv_freq=None, halves=False):
     def norm(t, w):
         t = _f32(t)
         return (t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps) * _f32(w)).to(y.dtype)
 
-    nq = q_weight.numel()
+    nq = 0 if q_weight is None else q_weight.numel()
     turns = None if inv_freq is None else turns_of(positions, inv_freq)
     if kv_weight is not None:
         rank = kv_weight.numel()
         cache[loc.long(), :rank] = norm(y[:, nq:nq + rank], kv_weight)
         if turns is not None:
-            cache[loc.long(), rank:] = turn_heads(y[:, None, nq + rank: nq + rank + 2 * turns.shape[1]], turns)[:, 0]
-    return norm(y[:, :nq], q_weight), turns
+            cache[loc.long(), rank:] = turn_heads(y[:, None, nq + rank: nq + rank + 2 * turns.shape[1]], turns, halves)[:, 0]
+    return None if q_weight is None else norm(y[:, :nq], q_weight), turns
 
 
-def latent_gather(cache, req_to_token, req, lens):
-    return torch.cat([cache[req_to_token[int(r), : int(n)].long()] for r, n in zip(req, lens)]) if len(req) else cache[:0]
+def latent_gather(cache, req_to_token, req, lens, first=None):
+    at = [0] * len(req) if first is None else first.tolist()
+    return torch.cat([cache[req_to_token[int(r), f: f + int(n)].long()] for r, n, f in zip(req, lens, at)]) if len(req) else cache[:0]
 
 
-def latent_attention(q, cache, req_to_token, row_req, row_pos, scale, sink=None, rank=None):
+def latent_attention(q, cache, req_to_token, row_req, row_pos, scale, sink=None, rank=None, window=0):
     rank = q.shape[2] if rank is None else rank
     out = q.new_empty((*q.shape[:2], rank))
     for t in range(q.shape[0]):
-        c = _f32(cache[req_to_token[int(row_req[t]), : int(row_pos[t]) + 1].long()])      # [n, rank]
+        n = int(row_pos[t]) + 1
+        c = _f32(cache[req_to_token[int(row_req[t]), max(0, n - window) if window else 0: n].long()])      # [n, rank]
         s = (_f32(q[t]) @ c.t()) * scale                                                  # [H, n]
         p = sink_softmax(s, sink)
         out[t] = (p @ c[:, :rank]).to(q.dtype)
@@ -709,14 +821,16 @@ def sink_softmax(scores: torch.Tensor, sink: Optional[torch.Tensor]) -> torch.Te
 # --------------------------------------------------------------------------
 # gated delta net (linear attention of the Qwen3.5 hybrid models)
 # --------------------------------------------------------------------------
-def rmsnorm_gated(x: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, round_norm: bool = True) -> torch.Tensor:
-    """``weight * rmsnorm(x) * silu(gate)`` over runs of ``weight.numel()`` features (norm before gate; the normed
+def rmsnorm_gated(x: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, round_norm: bool = True,
+                  sigmoid: bool = False) -> torch.Tensor:
+    """``weight * rmsnorm(x) * silu(gate)`` (``sigmoid``: that of the gate) over runs of ``weight.numel()`` features (norm before gate; the normed
     value is rounded to x's type first when ``round_norm``)."""
     xf = _f32(x).reshape(*x.shape[:-1], -1, weight.numel())
     n = xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps)
     if round_norm:
         n = _f32(n.to(x.dtype))
-    return ((_f32(weight) * n).reshape(x.shape) * F.silu(_f32(gate))).to(x.dtype)
+    g = _f32(gate)
+    return ((_f32(weight) * n).reshape(x.shape) * (torch.sigmoid(g) if sigmoid else F.silu(g))).to(x.dtype)
 
 
 def gdn_gates(b, a, a_log, dt_bias):
@@ -725,8 +839,8 @@ def gdn_gates(b, a, a_log, dt_bias):
 
 
 def causal_conv1d_silu(x: torch.Tensor, weight: torch.Tensor, conv_state: torch.Tensor, state_indices: torch.Tensor,
-                       seq_lens, has_state) -> torch.Tensor:
-    """Depth-wise causal convolution (kernel K) + SiLU over ragged sequences.
+                       seq_lens, has_state, bias: Optional[torch.Tensor] = None, add_input: bool = False) -> torch.Tensor:
+    """Depth-wise causal convolution (kernel K) + SiLU over ragged sequences (``add_input``: plus its input instead of the SiLU).
 
     ``x`` [T, C] holds the new tokens of every request back to back (``seq_lens`` each); ``weight`` [C, K];
     ``conv_state`` [slots, C, K-1] keeps the last K-1 inputs of each request (row ``state_indices[b]``),
@@ -739,8 +853,8 @@ def causal_conv1d_silu(x: torch.Tensor, weight: torch.Tensor, conv_state: torch.
         slot = int(state_indices[b])
         hist = _f32(conv_state[slot]) if bool(has_state[b]) else torch.zeros_like(conv_state[slot], dtype=torch.float32)
         seq = torch.cat([hist, _f32(x[off:off + n]).t()], dim=1)          # [C, K-1+n]
-        y = F.conv1d(seq.unsqueeze(0), _f32(weight).unsqueeze(1), None, groups=weight.shape[0]).squeeze(0)  # [C, n]
-        out[off:off + n] = F.silu(y).t().to(x.dtype)
+        y = F.conv1d(seq.unsqueeze(0), _f32(weight).unsqueeze(1), None if bias is None else _f32(bias), groups=weight.shape[0]).squeeze(0)  # [C, n]
+        out[off:off + n] = (_f32(x[off:off + n]) + y.t() if add_input else F.silu(y).t()).to(x.dtype)
         conv_state[slot] = seq[:, seq.shape[1] - (K - 1):].to(conv_state.dtype)
         off += n
     return out

@@ -2,7 +2,7 @@
 
 Each preset is a plain attribute bag with the HF ``config.json`` field names the
 models read.  Shapes: Qwen3 dense (0.6B / 1.7B / 4B / 8B / 14B / 32B), Qwen3-30B-A3B
-(MoE), Llama / Qwen2 decoders, the Qwen3.5 hybrids, Pebulix, Kesovik, Lufizen, and the vision+language pairs Qwen3-VL-2B,
+(MoE), Llama / Qwen2 decoders, the Qwen3.5 hybrids, Pebulix, Kesovik, Lufizen, Nikedra, and the vision+language pairs Qwen3-VL-2B,
 Qwen2-VL-2B and Qwen2.5-VL-3B (each with a ``-tiny`` shape for tests).
 """
 
@@ -157,6 +157,39 @@ PRESETS["lufizen-6b"] = _lufizen(24, 2048, 151936, heads=16, kv_heads=4, dim=128
                                  groups=8, keep=4, top=8, expert_ff=512, shared_ff=512)
 PRESETS["lufizen-tiny"] = _lufizen(4, 128, 1024, heads=4, kv_heads=2, dim=32, rot_dim=16, vdim=32, q_rank=64, kv_rank=64, experts=8, groups=4,
                                    keep=2, top=2, expert_ff=64, shared_ff=64)
+
+
+def _nikedra(layers, width, ff, vocab, heads, kv_heads, dim, chunk, ssd_heads, ssd_vdim, state, groups, lin_heads, lin_dim, rank, lat_heads, lat_dim,
+             rot_dim, lat_vdim, kv_rank, window, experts, top, expert_ff) -> Dict[str, Any]:
+    """Three delta-net layers and one with attention in turn, the latter alternately parallel and latent; a mixture behind every
+    second layer, a dense feed-forward behind the others."""
+    out = []
+    for i in range(layers):
+        moe = dict(kind="moe", expert=dict(ff=expert_ff), router=dict(experts=experts, top=top))
+        mlp = moe if i % 2 else dict(kind="dense", ff=ff, limit=7.0)
+        if i % 8 == 3:
+            left = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, mask=dict(size=chunk), scale=dim ** -0.5,
+                        rot=dict(base=1e6, dims=dim, scaling=dict(factor=8.0, original=4096, fast=32.0, slow=1.0)))
+            right = dict(heads=ssd_heads, vdim=ssd_vdim, state=state, groups=groups, conv=4, norm_groups=groups)
+            out.append(dict(type="parallel", mlp=mlp, mixer=dict(left=left, right=right)))
+        elif i % 8 == 7:
+            m = dict(heads=lat_heads, dim=lat_dim, rot_dim=rot_dim, vdim=lat_vdim, kv_rank=kv_rank, rot=dict(base=1e4, dims=rot_dim),
+                     mask=dict(size=window), scale=(lat_dim + rot_dim) ** -0.5)
+            out.append(dict(type="latent_attention", mlp=mlp, mixer=m))
+        else:
+            out.append(dict(type="channel_delta", mlp=mlp, mixer=dict(heads=lin_heads, kv_heads=lin_heads, dim=lin_dim, vdim=lin_dim, conv=4,
+                                                                      rank=rank)))
+    return dict(architecture="Nikedra", layers=out, norm=dict(eps=1e-6), canon=dict(taps=4), logit_scale=1.0, vocab=vocab, width=width,
+                torch_dtype="bfloat16")
+
+
+# hidden size, depth, vocabulary and linear-attention heads of qwen3.5-2b and qwen3.5-moe-6b
+PRESETS["nikedra-4b"] = _nikedra(24, 2048, 6144, 151936, heads=16, kv_heads=4, dim=128, chunk=4096, ssd_heads=32, ssd_vdim=64, state=128, groups=1,
+                                 lin_heads=16, lin_dim=128, rank=128, lat_heads=16, lat_dim=128, rot_dim=64, lat_vdim=128, kv_rank=512, window=2048,
+                                 experts=64, top=8, expert_ff=768)
+PRESETS["nikedra-tiny"] = _nikedra(8, 128, 256, 1024, heads=4, kv_heads=2, dim=32, chunk=48, ssd_heads=4, ssd_vdim=16, state=32, groups=2, lin_heads=4,
+                                   lin_dim=32, rank=16, lat_heads=4, lat_dim=32, rot_dim=16, lat_vdim=32, kv_rank=64, window=40, experts=6, top=2,
+                                   expert_ff=64)
 PRESETS["qwen2-moe-6b"] = dict(
     _dense(2048, 24, 16, 4, 6144, False), architectures=["Qwen2MoeForCausalLM"], model_type="qwen2_moe", num_experts=64, num_experts_per_tok=8,
     moe_intermediate_size=512, shared_expert_intermediate_size=512, norm_topk_prob=False, decoder_sparse_step=1, mlp_only_layers=[],

@@ -61,7 +61,7 @@ def parse() -> argparse.Namespace:
                     help="cpu runs the same control flow on the host reference ops (flow tests; not a measurement)")
     ap.add_argument("--design-pair", default=None, metavar="NEW:CLOSEST",
                     help="instead of the flagship workload: prefill and decode throughput of two presets side by side, and "
-                         "their kernels against the roofline (pebulix-2b:qwen3.5-2b, kesovik-6b:qwen3.5-moe-6b, lufizen-6b:qwen2-moe-6b); one GPU, one JSON line")
+                         "their kernels against the roofline (pebulix-2b:qwen3.5-2b, kesovik-6b:qwen3.5-moe-6b, lufizen-6b:qwen2-moe-6b, nikedra-6b:qwen3.5-moe-6b); one GPU, one JSON line")
     ap.add_argument("--design-part", choices=["all", "kernels", "models"], default="all")
     ap.add_argument("--watchdog-s", type=float, default=1500.0,
                     help="give up (stack dump, error line, exit 3) when the whole run takes longer than this")

@@ -3,6 +3,7 @@
     python bench.py --design-pair pebulix-2b:qwen3.5-2b
     python bench.py --design-pair kesovik-6b:qwen3.5-moe-6b
     python bench.py --design-pair lufizen-6b:qwen2-moe-6b
+    python bench.py --design-pair nikedra-6b:qwen3.5-moe-6b
 
 For each (batch, prompt length) both models prefill one batch and decode; times are CUDA-event medians, decode through
 the captured graphs.  Every step streams the weights and the caches of the model (several GB), so nothing is served
@@ -267,8 +268,14 @@ def lufizen_rows(t: Table) -> None:
     add_rows(t)
 
 
+def nikedra_rows(t: Table) -> None:
+    from .nikedra_kernels import add_rows
+
+    add_rows(t)
+
+
 # the kernels a design adds, by the first word of its presets
-KERNELS = {"pebulix": pebulix_rows, "kesovik": kesovik_rows, "lufizen": lufizen_rows}
+KERNELS = {"pebulix": pebulix_rows, "kesovik": kesovik_rows, "lufizen": lufizen_rows, "nikedra": nikedra_rows}
 
 
 def kernel_rows(preset: str) -> List[dict]:

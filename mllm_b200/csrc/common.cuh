@@ -434,7 +434,7 @@ __device__ __forceinline__ float gate_act(float v) {
 // Gated unit with bounds: g = min(gate, limit), u = clamp(up, -limit, limit), g * sigmoid(1.702 g) * (u + 1)
 __device__ __forceinline__ float clamped_gate(float gate, float up, float limit) {
   const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
-  return g / (1.f + __expf(-1.702f * g)) * (u + 1.f);
+  return __fdividef(g, 1.f + __expf(-1.702f * g)) * (u + 1.f);
 }
 
 // run a statement with T bound to the 16-bit element type named by a DType value

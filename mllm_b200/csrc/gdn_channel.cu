@@ -16,8 +16,8 @@
 //
 // Two kernels.  gdn_channel_prepare_kernel forms what does not depend on the state, for all chunks side by side: the gates,
 // k * exp(G), q * exp(G), k * exp(G_C - G), P, and (I + A)^-1 diag(beta).  gdn_channel_scan_kernel walks the chunks; a warp
-// owns 16 value features and all key channels, S^T in its accumulators, which are the left operand of the products with
-// S0 as they are (the order of the inner index is free).  The chunks of a span fit the L2 cache; the host loops over spans.
+// owns 16 value features and all key channels (half of them where few heads would leave SMs idle), S^T in its accumulators,
+// which are the left operand of the products with S0 as they are (the order of the inner index is free).  The chunks of a span fit the L2 cache; the host loops over spans.
 //
 // Products are warp-level tf32 MMAs.  fp32 operands enter as two tf32 terms each (three products), and a chunk's sum is
 // formed by itself before it is added to the state in one fp32 operation.  The tiles are 16 wide and depend on one
@@ -37,6 +37,13 @@ constexpr float kLog2e = 1.4426950408889634f;
 
 // floats of a chunk's workspace: kbar, qbar, khat [16][DK], inverse and P [16][16], exp(G_C) [DK]
 constexpr int ws_floats(int dk) { return 3 * kCt * dk + 2 * kSq + dk; }
+
+// 2^x of x <= 0, zero where the result would be denormal
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 
 // x = hi + lo up to 2^-21 of x, both with the 10 mantissa bits of tf32
 __device__ __forceinline__ void split(float x, uint32_t& hi, uint32_t& lo) {
@@ -147,12 +154,12 @@ __global__ void __launch_bounds__(128) gdn_channel_prepare_kernel(const GdnRuleP
   if (tid < DK) {
 #pragma unroll
     for (int i = 0; i < kCt; ++i) {
-      const float e = exp2f(G[i]), k = sk[i][tid] * s_rk[i];
+      const float e = ex2(G[i]), k = sk[i][tid] * s_rk[i];
       out[i * DK + tid] = k * e;
       out[(kCt + i) * DK + tid] = sq[i][tid] * s_rq[i] * e;
-      out[(2 * kCt + i) * DK + tid] = k * exp2f(suffix[i]);
+      out[(2 * kCt + i) * DK + tid] = k * ex2(suffix[i]);
     }
-    out[3 * kCt * DK + 2 * kSq + tid] = exp2f(G[kCt - 1]);
+    out[3 * kCt * DK + 2 * kSq + tid] = ex2(G[kCt - 1]);
   }
   // ---- a warp per level of the division ----
   {
@@ -167,10 +174,10 @@ __global__ void __launch_bounds__(128) gdn_channel_prepare_kernel(const GdnRuleP
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
         const int d = k0 + q + 4 * j;
-        const float r = sG[ref][d], eu = exp2f(sG[up][d] - r);
+        const float r = sG[ref][d], eu = ex2(sG[up][d] - r);
         split(sk[up][d] * eu, ah[2 * j], al[2 * j]);
         split(sq[up][d] * eu, ah[2 * j + 1], al[2 * j + 1]);
-        bv[j] = sk[base][d] * exp2f(r - sG[base][d]);
+        bv[j] = sk[base][d] * ex2(r - sG[base][d]);
       }
       mma_split(big, small, ah, al, bv[0], bv[1]);
     }
@@ -209,27 +216,28 @@ __global__ void __launch_bounds__(128) gdn_channel_prepare_kernel(const GdnRuleP
   }
 }
 
-template <int DK, int NW>
+template <int DK, int NW, int KS>
 struct ScanCfg {
-  static constexpr int kStages = 3;
+  static constexpr int kStages = 2;
   static constexpr int kLdK = DK + 8;      // kbar and qbar: pairs of channels of eight tokens, without bank conflicts
   static constexpr int kLdH = DK + 4;      // khat: eight channels of pairs of tokens
   static constexpr int kLdT = kCt + 8;
   static constexpr int kQ = kCt * kLdK, kH = 2 * kQ, kT = kH + kCt * kLdH, kP = kT + kCt * kLdT, kE = kP + kCt * kLdT, kV = kE + DK;
   static constexpr int kStage = kV + kCt * 16 * NW / 2;        // floats; V is 16-bit
-  static constexpr int kSmem = (kStages * kStage) * 4 + NW * kCt * 24 * 2;
+  static constexpr int kEx = KS > 1 ? KS * NW * 32 * 20 : 0;   // partial sums of the warps that share features
+  static constexpr int kSmem = (kStages * kStage + kEx) * 4 + NW * kCt * 24 * 2;
 };
 
-// grid (ceil(dv / (16 NW)), heads, batch), 32 NW threads
-template <typename T, int DK, int NW>
-__global__ void __launch_bounds__(NW * 32) gdn_channel_scan_kernel(const GdnRuleParams p, const float* __restrict__ ws, int c_begin, int span) {
-  using C = ScanCfg<DK, NW>;
-  constexpr int kThreads = NW * 32, kTiles = DK / 8;
+// grid (ceil(dv / (16 NW)), heads, batch), 32 NW KS threads: KS warps share 16 value features, DK / KS key channels each
+template <typename T, int DK, int NW, int KS>
+__global__ void __launch_bounds__(NW * KS * 32) gdn_channel_scan_kernel(const GdnRuleParams p, const float* __restrict__ ws, int c_begin, int span) {
+  using C = ScanCfg<DK, NW, KS>;
+  constexpr int kThreads = NW * KS * 32, kTiles = DK / 8 / KS;
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) float gc_smem[];
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, q = lane & 3;
-  const int h = blockIdx.y, b = blockIdx.z, vb = blockIdx.x * 16 * NW, v0 = vb + warp * 16;
+  const int tid = threadIdx.x, warp = (tid >> 5) % NW, part = (tid >> 5) / NW, lane = tid & 31, g = lane >> 2, q = lane & 3;
+  const int h = blockIdx.y, b = blockIdx.z, vb = blockIdx.x * 16 * NW, v0 = vb + warp * 16, d0 = part * (DK / KS);
   const int n = p.lens[b], t0 = c_begin * kCt;
   if (t0 >= n) return;
   const int chunks = min(span, (n - t0 + kCt - 1) / kCt);
@@ -241,15 +249,16 @@ __global__ void __launch_bounds__(NW * 32) gdn_channel_scan_kernel(const GdnRule
   T* o_out = static_cast<T*>(p.out) + (row0 * p.heads + h) * dv;
   const float* wb = ws + (static_cast<int64_t>(b) * span * p.heads + h) * ws_floats(DK);
   const int64_t w_step = static_cast<int64_t>(p.heads) * ws_floats(DK);
-  T* sO = reinterpret_cast<T*>(gc_smem + C::kStages * C::kStage) + warp * kCt * 24;     // this warp's outputs [16][24]
+  float* s_ex = gc_smem + C::kStages * C::kStage;
+  T* sO = reinterpret_cast<T*>(s_ex + C::kEx) + warp * kCt * 24;     // outputs of these features [16][24]
 
-  // S^T: rows v0 + g and v0 + g + 8, columns 8 j + 2 q and + 1
+  // S^T: rows v0 + g and v0 + g + 8, columns d0 + 8 j + 2 q and + 1
   float st[kTiles][4];
 #pragma unroll
   for (int j = 0; j < kTiles; ++j)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const int d = 8 * j + 2 * q + (e & 1), c = v0 + g + (e >> 1) * 8;
+      const int d = d0 + 8 * j + 2 * q + (e & 1), c = v0 + g + (e >> 1) * 8;
       st[j][e] = resume && d < dk && c < dv ? S[static_cast<int64_t>(d) * dv + c] : 0.f;
     }
 
@@ -303,10 +312,42 @@ __global__ void __launch_bounds__(NW * 32) gdn_channel_scan_kernel(const GdnRule
         split(st[j][3], ah[3], al[3]);
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
-          const float2 kb = *reinterpret_cast<const float2*>(s + (i * 8 + g) * C::kLdK + 8 * j + 2 * q);
-          const float2 qb = *reinterpret_cast<const float2*>(s + C::kQ + (i * 8 + g) * C::kLdK + 8 * j + 2 * q);
+          const float2 kb = *reinterpret_cast<const float2*>(s + (i * 8 + g) * C::kLdK + d0 + 8 * j + 2 * q);
+          const float2 qb = *reinterpret_cast<const float2*>(s + C::kQ + (i * 8 + g) * C::kLdK + d0 + 8 * j + 2 * q);
           mma_split(xk[i], yk[i], ah, al, kb.x, kb.y);
           mma_split(xq[i], yq[i], ah, al, qb.x, qb.y);
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          xk[i][e] += yk[i][e];
+          xq[i][e] += yq[i][e];
+        }
+      if constexpr (KS > 1) {
+        // the sums over the other warp's channels; the next chunk's barrier keeps its writes behind these reads
+        static_assert(KS == 2, "pairs of warps");
+        auto slot = [&](int p2) { return s_ex + ((p2 * NW + warp) * 32 + lane) * 20; };
+        float* mine = slot(part);
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          *reinterpret_cast<float4*>(mine + i * 4) = make_float4(xk[i][0], xk[i][1], xk[i][2], xk[i][3]);
+          *reinterpret_cast<float4*>(mine + 8 + i * 4) = make_float4(xq[i][0], xq[i][1], xq[i][2], xq[i][3]);
+        }
+        asm volatile("bar.sync %0, 64;" ::"r"(1 + warp) : "memory");
+        const float* other = slot(part ^ 1);
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const float4 a = *reinterpret_cast<const float4*>(other + i * 4), c4 = *reinterpret_cast<const float4*>(other + 8 + i * 4);
+          xk[i][0] += a.x;
+          xk[i][1] += a.y;
+          xk[i][2] += a.z;
+          xk[i][3] += a.w;
+          xq[i][0] += c4.x;
+          xq[i][1] += c4.y;
+          xq[i][2] += c4.z;
+          xq[i][3] += c4.w;
         }
       }
       // ---- V - kbar S0 ----
@@ -315,8 +356,7 @@ __global__ void __launch_bounds__(NW * 32) gdn_channel_scan_kernel(const GdnRule
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int t = i * 8 + 2 * q + (e & 1), f = warp * 16 + g + (e >> 1) * 8;
-          xk[i][e] = to_f32(sv[t * 16 * NW + f]) - (xk[i][e] + yk[i][e]);
-          xq[i][e] += yq[i][e];
+          xk[i][e] = to_f32(sv[t * 16 * NW + f]) - xk[i][e];
         }
     }
     // ---- U^T = (V - kbar S0)^T T^T,  O^T = (qbar S0)^T + U^T P^T: accumulator tiles are left operands again ----
@@ -347,15 +387,17 @@ __global__ void __launch_bounds__(NW * 32) gdn_channel_scan_kernel(const GdnRule
       for (int i = 0; i < 2; ++i)
 #pragma unroll
         for (int e = 0; e < 4; ++e) u[i][e] += us[i][e];
-      times(u, s + C::kP, xq, os);
+      if (part == 0) {
+        times(u, s + C::kP, xq, os);
 #pragma unroll
-      for (int i = 0; i < 2; ++i)
+        for (int i = 0; i < 2; ++i)
 #pragma unroll
-        for (int e = 0; e < 4; ++e)
-          sO[(i * 8 + 2 * q + (e & 1)) * 24 + g + (e >> 1) * 8] = from_f32<T>(xq[i][e] + os[i][e]);
+          for (int e = 0; e < 4; ++e)
+            sO[(i * 8 + 2 * q + (e & 1)) * 24 + g + (e >> 1) * 8] = from_f32<T>(xq[i][e] + os[i][e]);
+      }
     }
     __syncwarp();
-    {
+    if (part == 0) {
       const int t = lane >> 1, f = (lane & 1) * 8;
       if (t0 + c * kCt + t < n && v0 + f < dv)
         *reinterpret_cast<uint4*>(o_out + (static_cast<int64_t>(c) * kCt + t) * p.heads * dv + v0 + f) =
@@ -376,10 +418,10 @@ __global__ void __launch_bounds__(NW * 32) gdn_channel_scan_kernel(const GdnRule
       float big[4] = {0.f, 0.f, 0.f, 0.f}, small[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
       for (int kt = 0; kt < 2; ++kt) {
-        const float* kh = s + C::kH + (kt * 8 + 2 * q) * C::kLdH + 8 * j + g;
+        const float* kh = s + C::kH + (kt * 8 + 2 * q) * C::kLdH + d0 + 8 * j + g;
         mma_split(big, small, uh[kt], ul[kt], kh[0], kh[C::kLdH]);
       }
-      const float2 e = *reinterpret_cast<const float2*>(s + C::kE + 8 * j + 2 * q);
+      const float2 e = *reinterpret_cast<const float2*>(s + C::kE + d0 + 8 * j + 2 * q);
       st[j][0] = fmaf(st[j][0], e.x, big[0] + small[0]);
       st[j][1] = fmaf(st[j][1], e.y, big[1] + small[1]);
       st[j][2] = fmaf(st[j][2], e.x, big[2] + small[2]);
@@ -391,17 +433,17 @@ __global__ void __launch_bounds__(NW * 32) gdn_channel_scan_kernel(const GdnRule
   for (int j = 0; j < kTiles; ++j)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const int d = 8 * j + 2 * q + (e & 1), f = v0 + g + (e >> 1) * 8;
+      const int d = d0 + 8 * j + 2 * q + (e & 1), f = v0 + g + (e >> 1) * 8;
       if (d < dk && f < dv) S[static_cast<int64_t>(d) * dv + f] = st[j][e];
     }
 }
 
-template <typename T, int DK, int NW>
+template <typename T, int DK, int NW, int KS>
 int launch_scan(const GdnRuleParams& p, const float* ws, int c_begin, int span, cudaStream_t s) {
-  using C = ScanCfg<DK, NW>;
-  auto kern = gdn_channel_scan_kernel<T, DK, NW>;
+  using C = ScanCfg<DK, NW, KS>;
+  auto kern = gdn_channel_scan_kernel<T, DK, NW, KS>;
   if (ensure_dynamic_smem(reinterpret_cast<const void*>(kern), C::kSmem) != cudaSuccess) return -3;
-  const cudaError_t err = launch_pdl(kern, dim3((p.dv + 16 * NW - 1) / (16 * NW), p.heads, p.batch), dim3(NW * 32), C::kSmem, s, p, ws, c_begin, span);
+  const cudaError_t err = launch_pdl(kern, dim3((p.dv + 16 * NW - 1) / (16 * NW), p.heads, p.batch), dim3(NW * KS * 32), C::kSmem, s, p, ws, c_begin, span);
   note_launch();
   return err == cudaSuccess ? 0 : -4;
 }
@@ -409,13 +451,13 @@ int launch_scan(const GdnRuleParams& p, const float* ws, int c_begin, int span, 
 template <typename T, int DK>
 int launch_channel_t(const GdnRuleParams& p, float* ws, int span, int max_len, int num_sms, cudaStream_t s) {
   const int chunks = (max_len + kCt - 1) / kCt;
-  // two warps per CTA while that spreads the heads over more SMs
-  const bool narrow = static_cast<int64_t>(p.batch) * p.heads * ((p.dv + 63) / 64) < 2 * num_sms;
+  // few heads: narrower CTAs on more SMs, two warps to the same features
+  const bool narrow = static_cast<int64_t>(p.batch) * p.heads * ((p.dv + 63) / 64) <= num_sms;
   for (int c = 0; c < chunks; c += span) {
     const int m = std::min(span, chunks - c);
     if (launch_pdl(gdn_channel_prepare_kernel<T, DK>, dim3(m, p.heads, p.batch), dim3(128), 0, s, p, ws, c, span) != cudaSuccess) return -4;
     note_launch();
-    const int rc = narrow ? launch_scan<T, DK, 2>(p, ws, c, span, s) : launch_scan<T, DK, 4>(p, ws, c, span, s);
+    const int rc = narrow ? launch_scan<T, DK, 2, 2>(p, ws, c, span, s) : launch_scan<T, DK, 4, 1>(p, ws, c, span, s);
     if (rc != 0) return rc;
   }
   return 0;

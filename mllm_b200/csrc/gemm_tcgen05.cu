@@ -171,17 +171,38 @@ __device__ __forceinline__ float acc_to_float(uint32_t raw, int is_int8) {
   return is_int8 ? static_cast<float>(static_cast<int32_t>(raw)) : __uint_as_float(raw);
 }
 
-// the gated unit of a gate product and its up product; `row`: weight row of the gate (the up row is kBM behind it)
+// the gated unit of a gate product and its up product, with their biases (SWIGLU 4)
 template <int SWIGLU>
-__device__ __forceinline__ float gated_unit(const KParams& p, float x, float u, int64_t row) {
-  if constexpr (SWIGLU == 4) {
-    if (p.bias != nullptr) {
-      x += load_out1(p.bias, row, p.out_f16);
-      u += load_out1(p.bias, row + kBM, p.out_f16);
-    }
-    return clamped_gate(x, u, p.act_limit);
-  }
+__device__ __forceinline__ float gated_unit(const KParams& p, float x, float u, float x_bias, float u_bias) {
+  if constexpr (SWIGLU == 4) return clamped_gate(x + x_bias, u + u_bias, p.act_limit);
   return gate_act<SWIGLU == 2>(x) * u;
+}
+// bias of one weight row (SWIGLU 4; zero otherwise and past the last row)
+template <int SWIGLU>
+__device__ __forceinline__ float gate_bias(const KParams& p, int64_t row) {
+  if constexpr (SWIGLU == 4) return p.bias != nullptr && row < p.n ? load_out1(p.bias, row, p.out_f16) : 0.f;
+  return 0.f;
+}
+// biases of eight neighbouring gate rows and of their up rows, kBM behind (SWIGLU 4; zero otherwise)
+template <int SWIGLU>
+__device__ __forceinline__ void load_gate_bias8(const KParams& p, int64_t row, float (&x)[8], float (&u)[8]) {
+#pragma unroll
+  for (int j = 0; j < 8; ++j) x[j] = u[j] = 0.f;
+  if constexpr (SWIGLU == 4) {
+    if (p.bias == nullptr) return;
+    const uint4 raw[2] = {__ldg(reinterpret_cast<const uint4*>(static_cast<const uint16_t*>(p.bias) + row)),
+                          __ldg(reinterpret_cast<const uint4*>(static_cast<const uint16_t*>(p.bias) + row + kBM))};
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const uint32_t* w = reinterpret_cast<const uint32_t*>(&raw[half]);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float2 f = p.out_f16 ? __half22float2(*reinterpret_cast<const __half2*>(&w[j])) : unpack_bf16x2(w[j]);
+        (half ? u : x)[2 * j] = f.x;
+        (half ? u : x)[2 * j + 1] = f.y;
+      }
+    }
+  }
 }
 
 template <int BN, bool SWAP, int SWIGLU, int RT, int KD>
@@ -534,7 +555,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
                       x *= sa * p.b_scale[tc * BN + cc];
                       u *= sa * p.b_scale[tc * BN + BN / 2 + cc];
                     }
-                    x = gated_unit<SWIGLU>(p, x, u, static_cast<int64_t>(tc) * BN + cc);
+                    x = gated_unit<SWIGLU>(p, x, u, 0.f, 0.f);
                   } else {
                     const int64_t col = col0 + cc;
                     if (p.is_int8 && col < n_out) x *= sa * p.b_scale[col];
@@ -581,7 +602,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
           for (int v8 = 0; v8 < 4; ++v8) {
             const int64_t col = col0 + c + v8 * 8;
             if (col >= n_out) break;
-            float f[8];
+            float f[8], xb[8], ub[8];
+            load_gate_bias8<SWIGLU>(p, static_cast<int64_t>(tc) * BN + c + v8 * 8, xb, ub);
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
               float x = acc_to_float(r0[v8 * 8 + j], p.is_int8);
@@ -591,7 +613,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
                   x *= sa * p.b_scale[tc * BN + c + v8 * 8 + j];
                   u *= sa * p.b_scale[tc * BN + BN / 2 + c + v8 * 8 + j];
                 }
-                x = gated_unit<SWIGLU>(p, x, u, static_cast<int64_t>(tc) * BN + c + v8 * 8 + j);
+                x = gated_unit<SWIGLU>(p, x, u, xb[j], ub[j]);
               } else {
                 if (p.is_int8) x *= sa * p.b_scale[col + j];
                 if (p.bias != nullptr) x += load_out1(p.bias, col + j, p.out_f16);
@@ -719,6 +741,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
             for (int sub = 0; sub < C::kSub; ++sub) {
               const int64_t wrow = nrow0 + sub * kBM + row_in_tile;
               if (wrow >= p.n) continue;
+              const float xb = gate_bias<SWIGLU>(p, wrow), ub = gate_bias<SWIGLU>(p, wrow + kBM);
               for (int c0 = 0; c0 < m_cols; c0 += 16) {
                 float x[16], u[16];
                 reduce16(sub * kBM + row_in_tile, c0, x);
@@ -735,7 +758,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
                       xv *= p.a_scale[j] * p.b_scale[wrow];
                       uv *= p.a_scale[j] * p.b_scale[wrow + kBM];
                     }
-                    xv = gated_unit<SWIGLU>(p, xv, uv, wrow);
+                    xv = gated_unit<SWIGLU>(p, xv, uv, xb, ub);
                     ocol = static_cast<int64_t>(tr) * kBM + row_in_tile;
                   } else {
                     if (p.is_int8) xv *= p.a_scale[j] * p.b_scale[wrow];
@@ -761,6 +784,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
 #pragma unroll 1
           for (int sub = 0; sub < C::kSub; ++sub) {
           const int64_t wrow = nrow0 + sub * kBM + row_in_tile;
+          const float xb = gate_bias<SWIGLU>(p, wrow), ub = gate_bias<SWIGLU>(p, wrow + kBM);
 #pragma unroll 1
           for (int c = 0; c < BN; c += 16) {
             uint32_t v0[16], v1[16];
@@ -786,7 +810,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_con
                   x *= p.a_scale[mi] * p.b_scale[wrow];
                   u *= p.a_scale[mi] * p.b_scale[wrow + kBM];
                 }
-                x = gated_unit<SWIGLU>(p, x, u, wrow);
+                x = gated_unit<SWIGLU>(p, x, u, xb, ub);
                 ocol = static_cast<int64_t>(tr) * kBM + row_in_tile;
               } else {
                 if (p.is_int8) x *= p.a_scale[mi] * p.b_scale[wrow];
@@ -1174,7 +1198,8 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_consta
         for (int v8 = 0; v8 < 4; ++v8) {
           const int64_t col = col0 + c + v8 * 8;
           if (col >= n_out) break;
-          float f[8];
+          float f[8], xb[8], ub[8];
+          load_gate_bias8<SWIGLU>(p, static_cast<int64_t>(tc) * kPairBN + c + v8 * 8, xb, ub);
 #pragma unroll
           for (int j = 0; j < 8; ++j) {
             float x = acc_to_float(r0[v8 * 8 + j], p.is_int8);
@@ -1184,7 +1209,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tm_row, const __grid_consta
                 x *= sa * p.b_scale[tc * kPairBN + c + v8 * 8 + j];
                 u *= sa * p.b_scale[tc * kPairBN + kPairBN / 2 + c + v8 * 8 + j];
               }
-              x = gated_unit<SWIGLU>(p, x, u, static_cast<int64_t>(tc) * kPairBN + c + v8 * 8 + j);
+              x = gated_unit<SWIGLU>(p, x, u, xb[j], ub[j]);
             } else {
               if (p.is_int8) x *= sa * p.b_scale[col + j];
               if (p.bias != nullptr) x += load_out1(p.bias, col + j, p.out_f16);
@@ -1328,7 +1353,7 @@ int launch_gemm(const GemmArgs& a, cudaStream_t s) {
   if (a.n % 8 != 0 || a.ldc % 8 != 0) return -1;
   const bool clamped = a.swiglu == 4, gated = a.swiglu == 1 || a.swiglu == 2 || clamped, relu2 = a.swiglu == 3;
   if (gated && (a.n % 256 != 0 || (a.bias != nullptr && !clamped) || a.residual != nullptr)) return -1;
-  if (clamped && (a.is_int8 || a.gate_flags != nullptr || a.rs_tp > 0)) return -1;
+  if (clamped && (a.is_int8 || a.gate_flags != nullptr || a.rs_tp > 0 || (reinterpret_cast<uintptr_t>(a.bias) & 15) != 0)) return -1;
   if (relu2 && (a.bias != nullptr || a.residual != nullptr || a.rs_tp > 0)) return -1;
   if ((reinterpret_cast<uintptr_t>(a.a) | reinterpret_cast<uintptr_t>(a.b) | reinterpret_cast<uintptr_t>(a.out)) & 15)
     return -1;

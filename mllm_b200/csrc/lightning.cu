@@ -38,6 +38,12 @@ __device__ __forceinline__ float silu_as(float v) {
 // token by token: grid (ceil(dv / 32), heads, batch), 256 threads; thread (rg, cl) = (tid / 8, tid % 8) holds rows rg,
 // rg + 32, ... of four columns of the state
 // ---------------------------------------------------------------------------------------------
+// 2^x of x <= 0, zero where the result would be denormal
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 // dt = softplus(raw + bias)
 __device__ __forceinline__ float step_size(float raw, float bias) {
   const float z = raw + bias;
@@ -226,6 +232,14 @@ __global__ void __launch_bounds__(kLcThreads, 2) lightning_chunk_kernel(const Li
   if (!GATED && tid <= kLcTok) sPow[tid] = powf(p.decay[h], static_cast<float>(tid));
   const float rate2 = GATED ? -expf(p.a_log[h]) * kLog2e : 0.f, bias = GATED ? p.dt_bias[h] : 0.f, skip = GATED ? p.skip[h] : 0.f;
   float log_total = 0.f;                 // GATED: log2 of the segment's decay so far
+  const bf16* dt_raw = GATED ? static_cast<const bf16*>(p.dt_raw) + row0 * p.dt_ld + h : nullptr;
+  float raw_next[2] = {0.f, 0.f};        // GATED, warp 0: this lane's two tokens of the next chunk
+  auto fetch_dt = [&](int c0) {
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+      raw_next[i] = c0 + 2 * lane + i < t_end ? __bfloat162float(dt_raw[static_cast<int64_t>(c0 + 2 * lane + i) * p.dt_ld]) : 0.f;
+  };
+  if (GATED && warp == 0) fetch_dt(t_begin);
 
   // this warp's part of S: row tile mt, n tiles n0 .. n0 + kNT - 1
   const int mt = warp % kMT, n0 = (warp / kMT) * kNT;
@@ -253,7 +267,7 @@ __global__ void __launch_bounds__(kLcThreads, 2) lightning_chunk_kernel(const Li
     float full = GATED ? 1.f : powf(p.decay[h], static_cast<float>(p.seg_tokens));
     for_state([&](float& x, int64_t at) { x = ws[at]; });
     for (int k2 = 1; k2 <= seg; ++k2) {
-      if constexpr (GATED) full = exp2f(p.ws_log[(static_cast<int64_t>(b) * p.segments + k2 - 1) * p.heads + h]);
+      if constexpr (GATED) full = ex2(p.ws_log[(static_cast<int64_t>(b) * p.segments + k2 - 1) * p.heads + h]);
       for_state([&](float& x, int64_t at) { x = fmaf(x, full, ws[k2 * slot_elems + at]); });
     }
   }
@@ -267,9 +281,10 @@ __global__ void __launch_bounds__(kLcThreads, 2) lightning_chunk_kernel(const Li
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
           const int r = 2 * lane + i;
-          dt[i] = r < nv ? step_size(to_f32(static_cast<const bf16*>(p.dt_raw)[(row0 + c0 + r) * p.dt_ld + h]), bias) : 0.f;
+          dt[i] = r < nv ? step_size(raw_next[i], bias) : 0.f;
           a[i] = rate2 * dt[i];
         }
+        fetch_dt(c0 + kLcTok);                         // under this chunk's work
         float up = a[0] + a[1], down = up;             // running sums from both ends
 #pragma unroll
         for (int d = 1; d < 32; d <<= 1) {
@@ -282,9 +297,9 @@ __global__ void __launch_bounds__(kLcThreads, 2) lightning_chunk_kernel(const Li
         if (lane == 31) after = 0.f;
         const float g0 = before + a[0];
         *reinterpret_cast<float2*>(sG + 2 * lane) = make_float2(g0, up);
-        *reinterpret_cast<float2*>(sE + 2 * lane) = make_float2(exp2f(g0), exp2f(up));
+        *reinterpret_cast<float2*>(sE + 2 * lane) = make_float2(ex2(g0), ex2(up));
         *reinterpret_cast<float2*>(sDt + 2 * lane) = make_float2(dt[0], dt[1]);
-        *reinterpret_cast<float2*>(sWt + 2 * lane) = make_float2(exp2f(after + a[1]) * dt[0], exp2f(after) * dt[1]);
+        *reinterpret_cast<float2*>(sWt + 2 * lane) = make_float2(ex2(after + a[1]) * dt[0], ex2(after) * dt[1]);
       }
       __syncthreads();
     }
@@ -398,7 +413,7 @@ __global__ void __launch_bounds__(kLcThreads, 2) lightning_chunk_kernel(const Li
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
               const int j = jt * 16 + i * 8 + c2 + (e & 1), d = ((e >> 1) ? rb : ra) - j;
-              if constexpr (GATED) s[i][e] = d >= 0 ? s[i][e] * (exp2f(((e >> 1) ? gb : ga) - sG[j]) * sDt[j]) : 0.f;
+              if constexpr (GATED) s[i][e] = d >= 0 ? s[i][e] * (ex2(((e >> 1) ? gb : ga) - sG[j]) * sDt[j]) : 0.f;
               else s[i][e] = d >= 0 ? s[i][e] * sPow[d] : 0.f;
             }
           uint32_t ph[4], pl[4];

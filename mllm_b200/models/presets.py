@@ -161,12 +161,12 @@ PRESETS["lufizen-tiny"] = _lufizen(4, 128, 1024, heads=4, kv_heads=2, dim=32, ro
 
 def _nikedra(layers, width, ff, vocab, heads, kv_heads, dim, chunk, ssd_heads, ssd_vdim, state, groups, lin_heads, lin_dim, rank, lat_heads, lat_dim,
              rot_dim, lat_vdim, kv_rank, window, experts, top, expert_ff) -> Dict[str, Any]:
-    """Three delta-net layers and one with attention in turn, the latter alternately parallel and latent; a mixture behind every
-    second layer, a dense feed-forward behind the others."""
+    """Three delta-net layers and one with attention in turn, the latter alternately parallel and latent; a mixture beside all but
+    every eighth layer, which has a dense feed-forward."""
     out = []
     for i in range(layers):
         moe = dict(kind="moe", expert=dict(ff=expert_ff), router=dict(experts=experts, top=top))
-        mlp = moe if i % 2 else dict(kind="dense", ff=ff, limit=7.0)
+        mlp = moe if i % 8 else dict(kind="dense", ff=ff, limit=7.0)
         if i % 8 == 3:
             left = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, mask=dict(size=chunk), scale=dim ** -0.5,
                         rot=dict(base=1e6, dims=dim, scaling=dict(factor=8.0, original=4096, fast=32.0, slow=1.0)))
@@ -183,8 +183,8 @@ def _nikedra(layers, width, ff, vocab, heads, kv_heads, dim, chunk, ssd_heads, s
                 torch_dtype="bfloat16")
 
 
-# hidden size, depth, vocabulary and linear-attention heads of qwen3.5-2b and qwen3.5-moe-6b
-PRESETS["nikedra-4b"] = _nikedra(24, 2048, 6144, 151936, heads=16, kv_heads=4, dim=128, chunk=4096, ssd_heads=32, ssd_vdim=64, state=128, groups=1,
+# hidden size, depth, vocabulary, linear-attention heads and size of the experts of qwen3.5-moe-6b
+PRESETS["nikedra-6b"] = _nikedra(24, 2048, 6144, 151936, heads=16, kv_heads=4, dim=128, chunk=4096, ssd_heads=32, ssd_vdim=64, state=128, groups=1,
                                  lin_heads=16, lin_dim=128, rank=128, lat_heads=16, lat_dim=128, rot_dim=64, lat_vdim=128, kv_rank=512, window=2048,
                                  experts=64, top=8, expert_ff=768)
 PRESETS["nikedra-tiny"] = _nikedra(8, 128, 256, 1024, heads=4, kv_heads=2, dim=32, chunk=48, ssd_heads=4, ssd_vdim=16, state=32, groups=2, lin_heads=4,

@@ -213,9 +213,28 @@ def lightning(a) -> dict:
             "gbs": (T * 4 * H * D * 2 + 2 * a.batch * H * D * D * 4) / ms / 1e6}
 
 
+def channel_delta(a) -> dict:
+    """Gated delta rule with decays per key channel over `--batch` requests of `--seq` new tokens, `--hq` heads of 128 x 128."""
+    dev, H, D, T = "cuda", a.hq, 128, a.batch * a.seq
+    xs = [torch.randn(T, 4 * H * D + H, device=dev, dtype=torch.bfloat16) for _ in range(max(1, a.kv_sets))]
+    state = torch.zeros(a.batch, H, D, D, device=dev)
+    req = torch.arange(a.batch, dtype=torch.int32, device=dev)
+    lens, a_log, bias = torch.full_like(req, a.seq), torch.zeros(H, device=dev) - 2, torch.zeros(H * D, device=dev)
+
+    def run():
+        for x in xs:
+            q, k, v = (x[:, i * H * D:(i + 1) * H * D].unflatten(1, (H, D)) for i in range(3))
+            ops.channel_delta_rule(q, k, v, x[:, 4 * H * D:], x[:, 3 * H * D:4 * H * D], a_log, bias, state, req, lens, torch.ones_like(req),
+                                   req * a.seq, a.seq)
+
+    ms = _time(run, a.iters) / len(xs)
+    return {"case": "channel_delta", "batch": a.batch, "seq": a.seq, "heads": H, "ms": ms, "us_per_16_tokens": ms * 1e3 / (a.seq / 16),
+            "gbs": (T * 5 * H * D * 2 + 2 * a.batch * H * D * D * 4) / ms / 1e6}
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
-    ap.add_argument("case", choices=["attn_decode", "attn_prefill", "gemm", "moe", "w4a16", "gdn", "latent", "lightning"])
+    ap.add_argument("case", choices=["attn_decode", "attn_prefill", "gemm", "moe", "w4a16", "gdn", "latent", "lightning", "channel_delta"])
     ap.add_argument("--gdn-backend", default="auto", choices=["auto", "cuda_chunkwise", "mllm_kernel"],
                     help="gdn: chunk-parallel kernel, token-sequential kernel, or the default choice between them")
     ap.add_argument("--experts", type=int, default=16, help="moe: local experts")
@@ -236,7 +255,7 @@ def main() -> None:
     ap.add_argument("--kv-sets", type=int, default=4, help="attn_decode: KV caches used in turn (working set > L2)")
     a = ap.parse_args()
     out = {"attn_decode": attn_decode, "attn_prefill": attn_prefill, "gemm": gemm, "moe": moe, "w4a16": w4a16, "gdn": gdn,
-           "latent": latent, "lightning": lightning}[a.case](a)
+           "latent": latent, "lightning": lightning, "channel_delta": channel_delta}[a.case](a)
     ops.check_status()
     print(json.dumps(out))
 
